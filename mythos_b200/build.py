@@ -1,9 +1,11 @@
 """In-tree build of the native code.
 
-Three artefacts are produced next to the Python sources (never in a user cache directory, so
+Four artefacts are produced next to the Python sources (never in a user cache directory, so
 they travel with a checkout):
 
 * ``mythos_b200/_C*.so``      kernels (``csrc/kernels/*.cu``, sm_100a only) + torch binding
+* ``mythos_b200/_H*.so``      the kernels that serve layer-list models (``HYBRID_SOURCES``) + their binding;
+                              :func:`build_hybrid` compiles these sources only
 * ``mythos_b200/libmythos_kernels.so``  the same kernels with a plain C ABI, no torch
 * ``mythos_b200/liboil_host.so``        host runtime: ``.oil`` container, SHA-256, BPE, RNG,
                                          page allocator, C API (``csrc/host/*.cpp``)
@@ -23,6 +25,10 @@ from pathlib import Path
 PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 OBJ = PKG / "csrc" / "build"
+
+# Sources of the layer-list model module: those it has to itself, and those it shares with ``_C``.
+HYBRID_ONLY = ["hybrid_ops", "recurrent"]
+HYBRID_SOURCES = HYBRID_ONLY + ["host_util", "gemm", "gemm_2cta", "sampler"]
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -64,13 +70,16 @@ def _torch_paths():
     return inc, lib
 
 
-def build_kernels(verbose: bool = False) -> list[Path]:
+def build_kernels(verbose: bool = False, only=None) -> list[Path]:
+    """Objects of the kernel sources (all of them, or the stems in ``only``)."""
     OBJ.mkdir(parents=True, exist_ok=True)
     kdir = CSRC / "kernels"
     headers = list(kdir.glob("*.h")) + list(kdir.glob("*.cuh"))
     jobs = []
     objs = []
     for src in sorted(kdir.glob("*.cu")):
+        if only is not None and src.stem not in only:
+            continue
         obj = OBJ / (src.stem + ".o")
         objs.append(obj)
         if _newer(obj, [src] + headers):
@@ -87,15 +96,13 @@ def build_kernels(verbose: bool = False) -> list[Path]:
     return objs
 
 
-def build_binding(objs, verbose: bool = False) -> Path:
-    inc, torch_lib = _torch_paths()
-    ext = sysconfig.get_config_var("EXT_SUFFIX") or ".so"
-    target = PKG / ("_C" + ext)
-    bsrc = CSRC / "bindings.cpp"
-    bobj = OBJ / "bindings.o"
-    headers = list((CSRC / "kernels").glob("*.h"))
+def _compile_binding(stem: str, module: str, verbose: bool = False) -> Path:
+    inc, _ = _torch_paths()
+    bsrc, bobj = CSRC / (stem + ".cpp"), OBJ / (stem + ".o")
+    OBJ.mkdir(parents=True, exist_ok=True)
+    headers = list((CSRC / "kernels").glob("*.h")) + list(CSRC.glob("binding_*.h"))
     if _newer(bobj, [bsrc] + headers):
-        cmd = ["g++", "-O2", "-std=c++17", "-fPIC", "-DTORCH_EXTENSION_NAME=_C", "-DTORCH_API_INCLUDE_EXTENSION_H",
+        cmd = ["g++", "-O2", "-std=c++17", "-fPIC", f"-DTORCH_EXTENSION_NAME={module}", "-DTORCH_API_INCLUDE_EXTENSION_H",
                "-D_GLIBCXX_USE_CXX11_ABI=1", "-I", str(CSRC), "-I", "/usr/local/cuda/include",
                "-I", sysconfig.get_paths()["include"]]
         for p in inc:
@@ -103,13 +110,42 @@ def build_binding(objs, verbose: bool = False) -> Path:
         cmd += ["-c", str(bsrc), "-o", str(bobj)]
         _run(cmd)
         if verbose:
-            print("g++ bindings.cpp")
+            print("g++", bsrc.name)
+    return bobj
+
+
+def _link_binding(module: str, bobj: Path, objs) -> Path:
+    _, torch_lib = _torch_paths()
+    target = PKG / (module + (sysconfig.get_config_var("EXT_SUFFIX") or ".so"))
     if _newer(target, list(objs) + [bobj]):
         cmd = ["g++", "-shared", "-o", str(target), str(bobj), *map(str, objs), "-L", torch_lib,
                "-L", "/usr/local/cuda/lib64", "-lc10", "-lc10_cuda", "-ltorch_cpu", "-ltorch_cuda", "-ltorch",
                "-ltorch_python", "-lcudart", "-Wl,-rpath," + torch_lib, "-Wl,-rpath,/usr/local/cuda/lib64"]
         _run(cmd)
     return target
+
+
+def build_binding(objs, verbose: bool = False) -> Path:
+    return _link_binding("_C", _compile_binding("bindings", "_C", verbose),
+                         [o for o in objs if o.stem not in HYBRID_ONLY])
+
+
+def build_hybrid(verbose: bool = False) -> Path:
+    """Module ``mythos_b200._H`` from its own sources (the binding compiles beside the kernels)."""
+    with ThreadPoolExecutor(max_workers=1) as ex:
+        binding = ex.submit(_compile_binding, "bindings_hybrid", "_H", verbose)
+        objs = build_kernels(verbose, only=HYBRID_SOURCES)
+        return _link_binding("_H", binding.result(), objs)
+
+
+def ensure_hybrid(verbose: bool = False) -> Path:
+    """:func:`build_hybrid`, with one process at a time in a checkout (the others wait for it)."""
+    import fcntl
+
+    OBJ.mkdir(parents=True, exist_ok=True)
+    with open(OBJ / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build_hybrid(verbose)
 
 
 def build_kernel_clib(objs) -> Path:
@@ -181,7 +217,8 @@ def build_capi(verbose: bool = False) -> Path:
 
 def build_all(verbose: bool = False) -> dict:
     objs = build_kernels(verbose)
-    out = {"binding": build_binding(objs, verbose), "kernels_c": build_kernel_clib(objs), "host": build_host(verbose),
+    out = {"binding": build_binding(objs, verbose), "hybrid": build_hybrid(verbose),
+           "kernels_c": build_kernel_clib([o for o in objs if o.stem not in HYBRID_ONLY]), "host": build_host(verbose),
            "capi": build_capi(verbose)}
     return out
 

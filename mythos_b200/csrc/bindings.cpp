@@ -5,35 +5,10 @@
 #include <c10/cuda/CUDAGuard.h>
 #include <torch/extension.h>
 
+#include "binding_sampler.h"
 #include "kernels/api.h"
 
 namespace {
-
-using torch::Tensor;
-using OptTensor = c10::optional<Tensor>;
-
-cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
-
-void chk(const Tensor& t, c10::ScalarType dt, const char* name) {
-  TORCH_CHECK(t.is_cuda(), name, " must be a CUDA tensor");
-  TORCH_CHECK(t.scalar_type() == dt, name, " has dtype ", t.scalar_type(), ", expected ", dt);
-}
-void chk_c(const Tensor& t, c10::ScalarType dt, const char* name) {
-  chk(t, dt, name);
-  TORCH_CHECK(t.is_contiguous(), name, " must be contiguous");
-}
-const void* cptr(const OptTensor& t) { return t.has_value() ? t->data_ptr() : nullptr; }
-void* mptr(OptTensor& t) { return t.has_value() ? t->data_ptr() : nullptr; }
-int* status_ptr(const OptTensor& s) {
-  if (!s.has_value()) return nullptr;
-  chk_c(*s, torch::kInt32, "status");
-  return s->data_ptr<int>();
-}
-
-constexpr auto BF16 = torch::kBFloat16;
-constexpr auto F32 = torch::kFloat32;
-constexpr auto I32 = torch::kInt32;
-constexpr auto U8 = torch::kUInt8;
 
 // out[M,N] (+)= alpha * op(a) * op(b)^T. a: [M,K] or, with a_mn, [K,M]; b: [N,K] or, with b_mn, [K,N].
 void gemm(const Tensor& a, const Tensor& b, Tensor& out, bool a_mn, bool b_mn, int64_t epi, double alpha,
@@ -908,28 +883,6 @@ void paged_attn_decode_int8(const Tensor& q, const Tensor& k_cache, const Tensor
                              out.data_ptr(), scratch.data_ptr<float>(), counters.data_ptr<int>(), (int)B, (int)H,
                              (int)Hkv, (int)D, (int)k_cache.size(1), (int)block_table.size(1), (int)k_cache.size(0),
                              (int)splits, (float)scale, status_ptr(status), cur_stream(), q.stride(0));
-}
-
-void sample_tokens(const Tensor& logits, const OptTensor& history, const OptTensor& allow_mask, double temperature,
-                   int64_t top_k, double top_p, double repetition_penalty, int64_t seed, Tensor& out_tokens,
-                   OptTensor out_logprob) {
-  chk(logits, BF16, "logits");
-  chk_c(out_tokens, I32, "out_tokens");
-  TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1, "sample_tokens: logits must be [rows, vocab]");
-  const int* hist = nullptr;
-  int hist_len = 0;
-  if (history.has_value()) {
-    chk_c(*history, I32, "history");
-    hist = history->data_ptr<int>();
-    hist_len = (int)history->size(1);
-  }
-  mb::SamplerArgs a{(float)temperature, (float)top_p, (float)repetition_penalty, (int)top_k,
-                    (unsigned long long)seed};
-  c10::cuda::CUDAGuard guard(logits.device());
-  mb::sample_tokens(logits.data_ptr(), logits.stride(0), (int)logits.size(0), (int)logits.size(1), hist, hist_len,
-                    allow_mask.has_value() ? allow_mask->data_ptr<unsigned char>() : nullptr, a,
-                    out_tokens.data_ptr<int>(), out_logprob.has_value() ? out_logprob->data_ptr<float>() : nullptr,
-                    nullptr, cur_stream());
 }
 
 void peer_add_f32(const Tensor& part, const std::vector<int64_t>& ptrs) {

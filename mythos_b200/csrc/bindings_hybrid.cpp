@@ -1,0 +1,283 @@
+// Python binding of the kernels that serve layer-list models (kernels/hybrid_api.h), a module of its
+// own (mythos_b200._H) so that serving such a model needs a fraction of the library's sources compiled.
+#include "binding_sampler.h"
+#include "kernels/api.h"
+#include "kernels/host_util.h"
+#include "kernels/hybrid_api.h"
+
+namespace {
+
+bool is_f32(const Tensor& t, const char* name) {
+  TORCH_CHECK(t.is_cuda(), name, " must be a CUDA tensor");
+  TORCH_CHECK(t.scalar_type() == BF16 || t.scalar_type() == F32, name, " must be bf16 or fp32");
+  return t.scalar_type() == F32;
+}
+// 2-D activations with unit inner stride, of the given type.
+void chk_rows(const Tensor& t, bool f32, int64_t rows, int64_t cols, const char* name) {
+  chk(t, f32 ? F32 : BF16, name);
+  TORCH_CHECK(t.dim() == 2 && t.stride(1) == 1 && t.size(0) >= rows && t.size(1) >= cols, name,
+              ": expected at least [", rows, ", ", cols, "]");
+}
+const float* fptr(const OptTensor& t, int64_t n, const char* name) {
+  if (!t.has_value()) return nullptr;
+  chk_c(*t, F32, name);
+  TORCH_CHECK(t->numel() >= n, name, ": expected ", n, " values");
+  return t->data_ptr<float>();
+}
+const float* fptr(const Tensor& t, int64_t n, const char* name) { return fptr(OptTensor(t), n, name); }
+
+// batch = (cu_q, kv_lens, slots, row_seq, pos)
+mb::RaggedBatch ragged(const std::vector<Tensor>& batch) {
+  TORCH_CHECK(batch.size() == 5, "ragged batch: cu_q, kv_lens, slots, row_seq, pos");
+  for (const auto& t : batch) chk_c(t, I32, "ragged batch");
+  const int64_t n = batch[1].numel(), rows = batch[4].numel();
+  TORCH_CHECK(batch[0].numel() == n + 1 && batch[2].numel() == n && batch[3].numel() == rows, "ragged batch: sizes");
+  return mb::RaggedBatch{batch[0].data_ptr<int>(), batch[1].data_ptr<int>(), batch[2].data_ptr<int>(),
+                         batch[3].data_ptr<int>(), batch[4].data_ptr<int>(), (int)n, (int)rows};
+}
+
+void embed_pos_norm(const Tensor& ids, const Tensor& pos, const Tensor& embed, const OptTensor& pos_table, double scale,
+                    const Tensor& gamma, Tensor& x, Tensor& h, double eps) {
+  const bool f32 = is_f32(h, "h");
+  const int64_t rows = ids.numel(), dim = embed.size(1);
+  chk_c(ids, I32, "ids");
+  chk_c(pos, I32, "pos");
+  chk_c(embed, f32 ? F32 : BF16, "embed");
+  chk_c(x, F32, "x");
+  chk_rows(h, f32, rows, dim, "h");
+  TORCH_CHECK(pos.numel() == rows && x.numel() == rows * dim, "embed_pos_norm: sizes");
+  if (pos_table.has_value()) {
+    chk_c(*pos_table, f32 ? F32 : BF16, "pos_table");
+    TORCH_CHECK(pos_table->size(1) == dim, "pos_table width");
+  }
+  c10::cuda::CUDAGuard guard(h.device());
+  mb::embed_pos_norm(f32, ids.data_ptr<int>(), pos.data_ptr<int>(), embed.data_ptr(), cptr(pos_table),
+                     (int)embed.size(0), pos_table.has_value() ? (int)pos_table->size(0) : 1, (float)scale,
+                     fptr(gamma, dim, "gamma"), x.data_ptr<float>(), h.data_ptr(), h.stride(0), (int)rows, (int)dim,
+                     (float)eps, cur_stream());
+}
+
+void sandwich_norm(const Tensor& y1, const OptTensor& y2, const OptTensor& w1, const OptTensor& w2, const Tensor& w_post,
+                   Tensor& x, const Tensor& w_next, Tensor& h, double eps) {
+  const bool f32 = is_f32(h, "h");
+  chk_c(x, F32, "x");
+  const int64_t rows = x.size(0), dim = x.size(1);
+  chk_rows(y1, f32, rows, dim, "y1");
+  chk_rows(h, f32, rows, dim, "h");
+  if (y2.has_value()) {
+    chk_rows(*y2, f32, rows, dim, "y2");
+    TORCH_CHECK(y2->stride(0) == y1.stride(0), "sandwich_norm: y1 and y2 need the same row stride");
+  }
+  c10::cuda::CUDAGuard guard(h.device());
+  mb::sandwich_norm(f32, y1.data_ptr(), cptr(y2), y1.stride(0), fptr(w1, dim, "w1"), fptr(w2, dim, "w2"),
+                    fptr(w_post, dim, "w_post"), x.data_ptr<float>(), fptr(w_next, dim, "w_next"), h.data_ptr(),
+                    h.stride(0), (int)rows, (int)dim, (float)eps, cur_stream());
+}
+
+struct Pages {
+  const int* table;
+  int stride, page_size, kv_heads, dk, dv;
+};
+Pages pages(const Tensor& table, const Tensor& k_cache, const Tensor& v_cache, bool f32, int n_seq) {
+  chk_c(table, I32, "block_table");
+  chk_c(k_cache, f32 ? F32 : BF16, "k_cache");
+  chk_c(v_cache, f32 ? F32 : BF16, "v_cache");
+  TORCH_CHECK(table.dim() == 2 && table.size(0) >= n_seq, "block_table: one row per sequence of the batch");
+  TORCH_CHECK(k_cache.dim() == 4 && v_cache.dim() == 4 && k_cache.size(0) == v_cache.size(0) &&
+                  k_cache.size(1) == v_cache.size(1) && k_cache.size(2) == v_cache.size(2),
+              "caches: [pages, page_size, kv_heads, width]");
+  return Pages{table.data_ptr<int>(), (int)table.size(1), (int)k_cache.size(1), (int)k_cache.size(2),
+               (int)k_cache.size(3), (int)v_cache.size(3)};
+}
+
+void qk_norm_append(const Tensor& proj, int64_t q_off, int64_t k_off, int64_t v_off, const Tensor& q_gamma,
+                    const Tensor& k_gamma, const std::vector<Tensor>& batch, const Tensor& table, Tensor& q_out,
+                    Tensor& k_cache, Tensor& v_cache, double eps) {
+  const bool f32 = is_f32(q_out, "q_out");
+  const auto rb = ragged(batch);
+  const Pages pg = pages(table, k_cache, v_cache, f32, rb.n_seq);
+  chk_c(q_out, f32 ? F32 : BF16, "q_out");
+  TORCH_CHECK(q_out.dim() == 3 && q_out.size(0) == rb.rows && q_out.size(2) == pg.dk, "q_out: [rows, heads, dk]");
+  const int heads = (int)q_out.size(1);
+  chk_rows(proj, f32, rb.rows, std::max({q_off + heads * pg.dk, k_off + pg.kv_heads * pg.dk, v_off + pg.kv_heads * pg.dv}),
+           "proj");
+  c10::cuda::CUDAGuard guard(q_out.device());
+  mb::qk_norm_append(f32, proj.data_ptr(), proj.stride(0), (int)q_off, (int)k_off, (int)v_off,
+                     fptr(q_gamma, pg.dk, "q_gamma"), fptr(k_gamma, pg.dk, "k_gamma"), rb, pg.table, pg.stride,
+                     pg.page_size, q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), heads, pg.kv_heads, pg.dk,
+                     pg.dv, (float)eps, cur_stream());
+}
+
+void paged_attn_any(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const std::vector<Tensor>& batch,
+                    const Tensor& table, const OptTensor& gate, Tensor& o, double scale) {
+  const bool f32 = is_f32(q, "q");
+  const auto rb = ragged(batch);
+  const Pages pg = pages(table, k_cache, v_cache, f32, rb.n_seq);
+  chk_c(q, f32 ? F32 : BF16, "q");
+  TORCH_CHECK(q.dim() == 3 && q.size(0) == rb.rows && q.size(2) == pg.dk, "q: [rows, heads, dk]");
+  const int heads = (int)q.size(1);
+  chk_rows(o, f32, rb.rows, (int64_t)heads * pg.dv, "o");
+  if (gate.has_value()) chk_rows(*gate, f32, rb.rows, heads, "gate");
+  c10::cuda::CUDAGuard guard(q.device());
+  mb::paged_attn_any(f32, q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), rb, pg.table, pg.stride, pg.page_size,
+                     cptr(gate), gate.has_value() ? gate->stride(0) : 0, o.data_ptr(), o.stride(0), heads, pg.kv_heads,
+                     pg.dk, pg.dv, (float)scale, cur_stream());
+}
+
+// out = alpha * a b^T; bf16 operands run the tcgen05 GEMM (bf16 or fp32 output), fp32 operands the fp32 kernel.
+void gemm_nt(const Tensor& a, const Tensor& b, Tensor& out, double alpha, const OptTensor& status) {
+  const bool f32 = is_f32(a, "a");
+  chk(b, f32 ? F32 : BF16, "b");
+  TORCH_CHECK(a.dim() == 2 && b.dim() == 2 && out.dim() == 2 && a.stride(1) == 1 && b.stride(1) == 1 && out.stride(1) == 1,
+              "gemm_nt: 2-D operands with unit inner stride");
+  TORCH_CHECK(a.size(1) == b.size(1) && out.size(0) == a.size(0) && out.size(1) == b.size(0), "gemm_nt: shapes");
+  c10::cuda::CUDAGuard guard(a.device());
+  if (f32) {
+    chk(out, F32, "out");
+    mb::gemm_f32(a.data_ptr<float>(), a.stride(0), b.data_ptr<float>(), b.stride(0), out.data_ptr<float>(), out.stride(0),
+                 (int)a.size(0), (int)b.size(0), (int)a.size(1), (float)alpha, cur_stream());
+  } else {
+    const bool of32 = is_f32(out, "out");
+    mb::gemm_bf16(a.data_ptr(), a.stride(0), false, b.data_ptr(), b.stride(0), false, out.data_ptr(), out.stride(0),
+                  (int)a.size(0), (int)b.size(0), (int)a.size(1), of32 ? mb::EPI_F32 : mb::EPI_BF16, (float)alpha,
+                  status_ptr(status), cur_stream());
+  }
+}
+
+void silu_gate(const Tensor& gu, int64_t f, int64_t f_off, Tensor& h) {
+  const bool f32 = is_f32(h, "h");
+  chk_rows(h, f32, h.size(0), f, "h");
+  chk_rows(gu, f32, h.size(0), f_off + f, "gu");
+  TORCH_CHECK(h.stride(0) == h.size(1), "silu_gate: h must be contiguous");
+  c10::cuda::CUDAGuard guard(h.device());
+  mb::silu_gate(f32, gu.data_ptr(), gu.stride(0), (int)f, (int)f_off, h.data_ptr(), h.stride(0), (int)h.size(0),
+                cur_stream());
+}
+
+// The recurrence of one layer with its parameters and state, built once per layer.
+struct Recurrent {
+  mb::RecurrentSpec s{};
+  int q_off = 0, k_off = 0, v_off = 0, b_off = 0;
+  OptTensor z_bias, a_log, conv_w, conv_state, gamma, a2, g2;
+  Tensor state;
+
+  int channels() const { return 2 * s.kv_heads * s.dim + s.heads * s.vdim; }
+  void validate() const {
+    chk_c(state, F32, "state");
+    TORCH_CHECK(state.dim() == 4 && state.size(1) == s.heads && state.size(2) == s.vdim && state.size(3) == s.dim,
+                "state: [slots, heads, vdim, dim]");
+    TORCH_CHECK(z_bias.has_value(), "recurrent: z_bias");
+    fptr(z_bias, (int64_t)s.heads * s.dim, "z_bias");
+    TORCH_CHECK(s.decay_kind == 0 || a_log.has_value(), "recurrent: a_log");
+    fptr(a_log, s.heads, "a_log");
+    if (s.taps > 0) {
+      TORCH_CHECK(conv_w.has_value(), "recurrent: conv_w");
+      fptr(conv_w, (int64_t)channels() * s.taps, "conv_w");
+      if (s.taps > 1) {
+        TORCH_CHECK(conv_state.has_value(), "recurrent: conv_state");
+        fptr(conv_state, state.size(0) * (s.taps - 1) * channels(), "conv_state");
+      }
+    }
+  }
+  mb::RecurrentInputs inputs(const Tensor& proj, const OptTensor& z, int64_t rows) {
+    const bool f32 = is_f32(proj, "proj");
+    const int64_t cq = (int64_t)s.kv_heads * s.dim, cv = (int64_t)s.heads * s.vdim;
+    chk_rows(proj, f32, rows, std::max({q_off + cq, k_off + cq, v_off + cv, (int64_t)(s.delta ? b_off + s.heads : 0)}),
+             "proj");
+    mb::RecurrentInputs in{};
+    in.proj = proj.data_ptr();
+    in.ld = proj.stride(0);
+    in.q_off = q_off;
+    in.k_off = k_off;
+    in.v_off = v_off;
+    in.b_off = b_off;
+    if (z.has_value()) {
+      chk_rows(*z, true, rows, (int64_t)s.heads * s.dim, "z");
+      in.z = z->data_ptr<float>();
+      in.ldz = z->stride(0);
+    }
+    in.z_bias = z_bias->data_ptr<float>();
+    in.a_log = fptr(a_log, s.heads, "a_log");
+    in.conv_w = fptr(conv_w, 0, "conv_w");
+    in.conv_state = const_cast<float*>(fptr(conv_state, 0, "conv_state"));
+    in.state = state.data_ptr<float>();
+    return in;
+  }
+  // o [rows, heads, vdim] fp32; the recurrence state and the convolution state advance.
+  void scan_seq(const Tensor& proj, const Tensor& z, const std::vector<Tensor>& batch, Tensor& scratch, Tensor& o) {
+    const auto rb = ragged(batch);
+    const int64_t need = (int64_t)rb.rows * (2 * s.kv_heads * s.dim + s.heads * (s.vdim + s.dim + 1));
+    chk_c(scratch, F32, "scratch");
+    chk_c(o, F32, "o");
+    TORCH_CHECK(scratch.numel() >= need && o.numel() >= (int64_t)rb.rows * s.heads * s.vdim, "scan_seq: buffers");
+    const auto in = inputs(proj, z, rb.rows);
+    c10::cuda::CUDAGuard guard(proj.device());
+    const bool f32 = is_f32(proj, "proj");
+    mb::recurrent_scan_seq(f32, s, in, rb, scratch.data_ptr<float>(), o.data_ptr<float>(), cur_stream());
+    mb::conv_state_update(f32, s, in, rb, cur_stream());
+  }
+  void norm_gate(const Tensor& o, const Tensor& gate, Tensor& out) {
+    const bool f32 = is_f32(out, "out");
+    const int64_t rows = out.size(0), cv = (int64_t)s.heads * s.vdim;
+    chk_c(o, F32, "o");
+    TORCH_CHECK(o.numel() >= rows * cv, "norm_gate: o");
+    chk_rows(out, f32, rows, cv, "out");
+    chk_rows(gate, f32, rows, cv, "gate");
+    TORCH_CHECK(out.stride(0) == out.size(1), "norm_gate: out must be contiguous");
+    c10::cuda::CUDAGuard guard(out.device());
+    mb::head_norm_gate(f32, s, o.data_ptr<float>(), fptr(gamma, s.vdim, "gamma"), gate.data_ptr(), gate.stride(0),
+                       out.data_ptr(), out.stride(0), (int)rows, cur_stream());
+  }
+};
+
+}  // namespace
+
+PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
+  m.doc() = "sm_100a kernels of layer-list models";
+  m.def("embed_pos_norm", &embed_pos_norm);
+  m.def("sandwich_norm", &sandwich_norm);
+  m.def("qk_norm_append", &qk_norm_append);
+  m.def("paged_attn_any", &paged_attn_any);
+  m.def("gemm_nt", &gemm_nt);
+  m.def("silu_gate", &silu_gate);
+  m.def("sample_tokens", &sample_tokens);
+  pybind11::class_<Recurrent>(m, "Recurrent")
+      .def(pybind11::init([](pybind11::dict spec, pybind11::dict tensors) {
+        Recurrent r;
+        auto geti = [&](const char* k, int d) { return spec.contains(k) ? spec[k].cast<int>() : d; };
+        auto getf = [&](const char* k, float d) { return spec.contains(k) ? spec[k].cast<float>() : d; };
+        auto gett = [&](const char* k) -> OptTensor {
+          if (!tensors.contains(k)) return c10::nullopt;
+          return tensors[k].cast<Tensor>();
+        };
+        r.s.heads = geti("heads", 0);
+        r.s.kv_heads = geti("kv_heads", r.s.heads);
+        r.s.dim = geti("dim", 0);
+        r.s.vdim = geti("vdim", 0);
+        r.s.taps = geti("taps", 0);
+        r.s.delta = geti("delta", 0);
+        r.s.unit_norm = geti("unit_norm", 0);
+        r.s.decay_kind = geti("decay_kind", 0);
+        r.s.gate_kind = geti("gate_kind", 0);
+        r.s.q_scale = getf("q_scale", 1.f);
+        r.s.inv_tau = getf("inv_tau", 1.f);
+        r.s.eps = getf("eps", 1e-6f);
+        r.q_off = geti("q_off", 0);
+        r.k_off = geti("k_off", 0);
+        r.v_off = geti("v_off", 0);
+        r.b_off = geti("b_off", 0);
+        r.z_bias = gett("z_bias");
+        r.a_log = gett("a_log");
+        r.conv_w = gett("conv_w");
+        r.conv_state = gett("conv_state");
+        r.gamma = gett("gamma");
+        r.a2 = gett("a2");
+        r.g2 = gett("g2");
+        r.state = tensors["state"].cast<Tensor>();
+        r.validate();
+        return r;
+      }))
+      .def("scan_seq", &Recurrent::scan_seq)
+      .def("norm_gate", &Recurrent::norm_gate);
+  m.def("launch_count", []() { return (int64_t)mb::launch_counter().load(); });
+}

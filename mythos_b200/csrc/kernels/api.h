@@ -347,7 +347,7 @@ struct SamplerArgs {
 };
 void sample_tokens(const void* logits, long long ld, int rows, int vocab, const int* history, int history_len,
                    const unsigned char* allow_mask, SamplerArgs a, int* out_tokens, float* out_logprob, float* scratch,
-                   cudaStream_t stream);
+                   cudaStream_t stream, bool f32 = false);   // f32: fp32 logits instead of bf16
 // y[n] = sum_k dequant(W)[n,k] * x[k] for one token (CUDA-core GEMV over packed I2_S trits).
 void i2s_gemv(const void* x, const DequantWeights& w, void* y, cudaStream_t stream);
 

@@ -1,0 +1,462 @@
+// Pointwise, normalisation and any-shape kernels of the layer-list models (hybrid_api.h).
+//
+// The residual stream is fp32. A sublayer's output is normalised before it is added ("sandwich"
+// norms), and the next sublayer's input norm reads the sum, so one kernel does post-norm, residual
+// add and pre-norm of a row; for two mixers side by side it also normalises and averages the two.
+#include "common.cuh"
+#include "hybrid_api.h"
+#include "hybrid_dev.cuh"
+#include "host_util.h"
+
+namespace mb {
+namespace {
+
+constexpr int SN_THREADS = 256;
+
+__device__ __forceinline__ float2 block_sum2(float2 v, float2* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+  v.x = warp_sum(v.x);
+  v.y = warp_sum(v.y);
+  __syncthreads();
+  if (lane == 0) scratch[warp] = v;
+  __syncthreads();
+  float2 t = (lane < nw) ? scratch[lane] : make_float2(0.f, 0.f);
+  t.x = warp_sum(t.x);
+  t.y = warp_sum(t.y);
+  return t;
+}
+
+// Four values per step when the row allows it (V = 4), else one.
+template <int V>
+__device__ __forceinline__ void ldv(const float* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    f[0] = t.x; f[1] = t.y; f[2] = t.z; f[3] = t.w;
+  } else {
+    f[0] = *p;
+  }
+}
+template <int V>
+__device__ __forceinline__ void ldv(const __nv_bfloat16* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.y));
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else {
+    f[0] = __bfloat162float(*p);
+  }
+}
+template <int V>
+__device__ __forceinline__ void stv(float* p, const float (&f)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *p = f[0];
+}
+template <int V>
+__device__ __forceinline__ void stv(__nv_bfloat16* p, const float (&f)[V]) {
+  if constexpr (V == 4) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    uint2 t;
+    t.x = *reinterpret_cast<uint32_t*>(&a);
+    t.y = *reinterpret_cast<uint32_t*>(&b);
+    *reinterpret_cast<uint2*>(p) = t;
+  } else {
+    *p = __float2bfloat16(f[0]);
+  }
+}
+
+// h = rms(row) * gamma for a row held in shared memory; columns [dim, ldh) are zeroed (GEMM padding).
+template <typename T, int V>
+__device__ __forceinline__ void write_normed(const float* row, float ss, const float* gamma, T* h, long long ldh,
+                                             int dim, float eps) {
+  const float r = 1.f / sqrtf(ss / (float)dim + eps);
+  for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
+    float x[V], g[V], y[V];
+    ldv<V>(row + i, x);
+    ldv<V>(gamma + i, g);
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] = x[j] * r * g[j];
+    stv<V>(h + i, y);
+  }
+  for (int i = dim + threadIdx.x; i < ldh; i += SN_THREADS) stf(h + i, 0.f);
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(SN_THREADS)
+embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ pos, const T* __restrict__ embed,
+                      const T* __restrict__ pos_table, int vocab, int max_pos, float scale,
+                      const float* __restrict__ gamma, float* __restrict__ x, T* __restrict__ h, long long ldh, int dim,
+                      float eps) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float scratch[32];
+  const long long t = blockIdx.x;
+  int id = ids[t];
+  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  int p = pos[t];
+  p = p < 0 ? 0 : (p >= max_pos ? max_pos - 1 : p);
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
+    float e[V], q[V], y[V];
+    ldv<V>(embed + (long long)id * dim + i, e);
+#pragma unroll
+    for (int j = 0; j < V; ++j) q[j] = 0.f;
+    if (pos_table) ldv<V>(pos_table + (long long)p * dim + i, q);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      y[j] = fmaf(e[j], scale, q[j]);
+      ss += y[j] * y[j];
+    }
+    stv<V>(row + i, y);
+    stv<V>(x + t * dim + i, y);
+  }
+  ss = block_sum(ss, scratch);
+  write_normed<T, V>(row, ss, gamma, h + t * ldh, ldh, dim, eps);
+}
+
+template <typename T, int V, bool TWO>
+__global__ void __launch_bounds__(SN_THREADS)
+sandwich_norm_kernel(const T* __restrict__ y1, const T* __restrict__ y2, long long ldy, const float* __restrict__ w1,
+                     const float* __restrict__ w2, const float* __restrict__ w_post, float* __restrict__ x,
+                     const float* __restrict__ w_next, T* __restrict__ h, long long ldh, int dim, float eps) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float2 scratch2[32];
+  __shared__ float scratch[32];
+  const long long t = blockIdx.x;
+  y1 += t * ldy;
+  float2 s2 = make_float2(0.f, 0.f);
+  for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
+    float a[V];
+    ldv<V>(y1 + i, a);
+#pragma unroll
+    for (int j = 0; j < V; ++j) s2.x += a[j] * a[j];
+    if constexpr (TWO) {
+      float b[V];
+      ldv<V>(y2 + t * ldy + i, b);
+#pragma unroll
+      for (int j = 0; j < V; ++j) s2.y += b[j] * b[j];
+    } else {
+      stv<V>(row + i, a);
+    }
+  }
+  s2 = block_sum2(s2, scratch2);
+  float ss = s2.x;
+  if constexpr (TWO) {
+    const float ra = 0.5f / sqrtf(s2.x / (float)dim + eps), rb = 0.5f / sqrtf(s2.y / (float)dim + eps);
+    ss = 0.f;
+    for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
+      float a[V], b[V], wa[V], wb[V];
+      ldv<V>(y1 + i, a);
+      ldv<V>(y2 + t * ldy + i, b);
+      ldv<V>(w1 + i, wa);
+      ldv<V>(w2 + i, wb);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        a[j] = a[j] * ra * wa[j] + b[j] * rb * wb[j];
+        ss += a[j] * a[j];
+      }
+      stv<V>(row + i, a);
+    }
+    ss = block_sum(ss, scratch);
+  }
+  const float r = 1.f / sqrtf(ss / (float)dim + eps);
+  float sx = 0.f;
+  for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
+    float a[V], w[V], xv[V];
+    ldv<V>(row + i, a);
+    ldv<V>(w_post + i, w);
+    ldv<V>(x + t * dim + i, xv);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      xv[j] += a[j] * r * w[j];
+      sx += xv[j] * xv[j];
+    }
+    stv<V>(x + t * dim + i, xv);
+    stv<V>(row + i, xv);
+  }
+  sx = block_sum(sx, scratch);
+  write_normed<T, V>(row, sx, w_next, h + t * ldh, ldh, dim, eps);
+}
+
+// One warp per (token, head slot): slots [0, H) are q, [H, H + G) k, [H + G, H + 2 G) v.
+template <typename T>
+__global__ void qk_norm_append_kernel(const T* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
+                                      const float* __restrict__ q_gamma, const float* __restrict__ k_gamma,
+                                      RaggedBatch rb, const int* __restrict__ block_table, int table_stride,
+                                      int page_size, T* __restrict__ q_out, T* __restrict__ k_cache,
+                                      T* __restrict__ v_cache, int heads, int kv_heads, int dk, int dv, float eps) {
+  const int lane = threadIdx.x & 31;
+  const int slots = heads + 2 * kv_heads;
+  const long long w = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (w >= (long long)rb.rows * slots) return;
+  const int t = (int)(w / slots), hs = (int)(w % slots);
+  const T* src = proj + (long long)t * ld;
+  if (hs < heads + kv_heads) {
+    const bool is_q = hs < heads;
+    src += is_q ? q_off + hs * dk : k_off + (hs - heads) * dk;
+    const float* gamma = is_q ? q_gamma : k_gamma;
+    float ss = 0.f;
+    for (int i = lane; i < dk; i += 32) {
+      const float v = ldf(src + i);
+      ss += v * v;
+    }
+    ss = warp_sum(ss);
+    const float r = 1.f / sqrtf(ss / (float)dk + eps);
+    T* dst;
+    if (is_q) {
+      dst = q_out + ((long long)t * heads + hs) * dk;
+    } else {
+      const int p = rb.pos[t];
+      const int page = block_table[(long long)rb.row_seq[t] * table_stride + p / page_size];
+      if (page < 0) return;
+      dst = k_cache + (((long long)page * page_size + p % page_size) * kv_heads + (hs - heads)) * dk;
+    }
+    for (int i = lane; i < dk; i += 32) stf(dst + i, ldf(src + i) * r * gamma[i]);
+  } else {
+    const int g = hs - heads - kv_heads, p = rb.pos[t];
+    const int page = block_table[(long long)rb.row_seq[t] * table_stride + p / page_size];
+    if (page < 0) return;
+    src += v_off + g * dv;
+    T* dst = v_cache + (((long long)page * page_size + p % page_size) * kv_heads + g) * dv;
+    for (int i = lane; i < dv; i += 32) dst[i] = src[i];
+  }
+}
+
+// One warp per (token, query head). Scores of 32 keys at a time (lane = key), then the value rows with
+// lane = channel: every product and the softmax are fp32 whatever the storage type.
+constexpr int PA_WARPS = 4;
+template <typename T, int ND>   // ND * 32 >= dv
+__global__ void __launch_bounds__(PA_WARPS * 32)
+paged_attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
+                      RaggedBatch rb, const int* __restrict__ block_table, int table_stride, int page_size,
+                      const T* __restrict__ gate, long long ld_gate, T* __restrict__ o, long long ldo, int heads,
+                      int kv_heads, int dk, int dv, float scale) {
+  extern __shared__ float sq_all[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long w = (long long)blockIdx.x * PA_WARPS + warp;
+  if (w >= (long long)rb.rows * heads) return;
+  // the last tokens have the longest contexts: start them first
+  const int t = rb.rows - 1 - (int)(w / heads), h = (int)(w % heads);
+  const int g = h / (heads / kv_heads);
+  float* sq = sq_all + warp * dk;
+  for (int i = lane; i < dk; i += 32) sq[i] = ldf(q + ((long long)t * heads + h) * dk + i) * scale;
+  __syncwarp();
+  const int* bt = block_table + (long long)rb.row_seq[t] * table_stride;
+  const int n = rb.pos[t] + 1;
+  float m = -INFINITY, l = 0.f, acc[ND];
+#pragma unroll
+  for (int j = 0; j < ND; ++j) acc[j] = 0.f;
+  for (int j0 = 0; j0 < n; j0 += 32) {
+    const int key = j0 + lane;
+    float s = -INFINITY;
+    long long tok = 0;
+    if (key < n) {
+      tok = (long long)bt[key / page_size] * page_size + key % page_size;
+      const T* kp = k_cache + (tok * kv_heads + g) * dk;
+      s = 0.f;
+      for (int i = 0; i < dk; ++i) s = fmaf(sq[i], ldf(kp + i), s);
+    }
+    const float mn = fmaxf(m, warp_max(s));
+    const float a = expf(m - mn), p = expf(s - mn);
+    l = l * a + warp_sum(p);
+    m = mn;
+#pragma unroll
+    for (int j = 0; j < ND; ++j) acc[j] *= a;
+    const int cnt = min(32, n - j0);
+    for (int jj = 0; jj < cnt; ++jj) {
+      const float pj = __shfl_sync(0xffffffffu, p, jj);
+      const long long tk = __shfl_sync(0xffffffffu, tok, jj);
+      const T* vp = v_cache + (tk * kv_heads + g) * dv;
+#pragma unroll
+      for (int j = 0; j < ND; ++j) {
+        const int d = lane + 32 * j;
+        if (d < dv) acc[j] = fmaf(pj, ldf(vp + d), acc[j]);
+      }
+    }
+  }
+  float r = 1.f / l;
+  if (gate) r *= sigmoid_f(ldf(gate + (long long)t * ld_gate + h));
+#pragma unroll
+  for (int j = 0; j < ND; ++j) {
+    const int d = lane + 32 * j;
+    if (d < dv) stf(o + (long long)t * ldo + (long long)h * dv + d, acc[j] * r);
+  }
+}
+
+// 64 x 64 tile, 16-deep steps, 4 x 4 outputs per thread.
+__global__ void __launch_bounds__(256)
+gemm_f32_kernel(const float* __restrict__ A, long long lda, const float* __restrict__ B, long long ldb,
+                float* __restrict__ C, long long ldc, int M, int N, int K, float alpha) {
+  __shared__ float sa[16][68], sb[16][68];
+  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+    for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+      const int r = i >> 4, c = i & 15;
+      sa[c][r] = (m0 + r < M && k0 + c < K) ? A[(long long)(m0 + r) * lda + k0 + c] : 0.f;
+      sb[c][r] = (n0 + r < N && k0 + c < K) ? B[(long long)(n0 + r) * ldb + k0 + c] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      float a[4], b[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        a[i] = sa[k][ty * 4 + i];
+        b[i] = sb[k][tx * 4 + i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
+      if (m < M && n < N) C[(long long)m * ldc + n] = alpha * acc[i][j];
+    }
+}
+
+template <typename T>
+__global__ void silu_gate_kernel(const T* __restrict__ gu, long long ldg, int f, int f_off, T* __restrict__ h,
+                                 long long ldh, long long rows) {
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < rows * ldh;
+       i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / ldh;
+    const int c = (int)(i % ldh);
+    float y = 0.f;
+    if (c < f) {
+      const float g = ldf(gu + r * ldg + c), u = ldf(gu + r * ldg + f_off + c);
+      y = g * sigmoid_f(g) * u;
+    }
+    stf(h + i, y);
+  }
+}
+
+inline int grid_for(long long n, int threads, int per_sm) {
+  long long g = (n + threads - 1) / threads;
+  const long long cap = (long long)sm_count() * per_sm;
+  return (int)(g < cap ? g : cap);
+}
+
+template <typename T, int V>
+void embed_launch(const int* ids, const int* pos, const void* embed, const void* pos_table, int vocab, int max_pos,
+                  float scale, const float* gamma, float* x, void* h, long long ldh, int rows, int dim, float eps,
+                  cudaStream_t stream) {
+  embed_pos_norm_kernel<T, V><<<rows, SN_THREADS, dim * 4, stream>>>(ids, pos, (const T*)embed, (const T*)pos_table,
+                                                                     vocab, max_pos, scale, gamma, x, (T*)h, ldh, dim,
+                                                                     eps);
+}
+template <typename T, int V>
+void sandwich_launch(const void* y1, const void* y2, long long ldy, const float* w1, const float* w2,
+                     const float* w_post, float* x, const float* w_next, void* h, long long ldh, int rows, int dim,
+                     float eps, cudaStream_t stream) {
+  if (y2)
+    sandwich_norm_kernel<T, V, true><<<rows, SN_THREADS, dim * 4, stream>>>(
+        (const T*)y1, (const T*)y2, ldy, w1, w2, w_post, x, w_next, (T*)h, ldh, dim, eps);
+  else
+    sandwich_norm_kernel<T, V, false><<<rows, SN_THREADS, dim * 4, stream>>>(
+        (const T*)y1, nullptr, ldy, w1, w2, w_post, x, w_next, (T*)h, ldh, dim, eps);
+}
+
+}  // namespace
+
+void embed_pos_norm(bool f32, const int* ids, const int* pos, const void* embed, const void* pos_table, int vocab,
+                    int max_pos, float scale, const float* gamma, float* x, void* h, long long ldh, int rows, int dim,
+                    float eps, cudaStream_t stream) {
+  MB_REQUIRE(dim > 0 && dim <= 12000 && ldh >= dim, "embed_pos_norm: row width out of range");
+  if (rows == 0) return;
+  const bool v4 = dim % 4 == 0 && ldh % 4 == 0;
+  auto go = [&](auto fn) {
+    fn(ids, pos, embed, pos_table, vocab, max_pos, scale, gamma, x, h, ldh, rows, dim, eps, stream);
+  };
+  if (f32) { if (v4) go(embed_launch<float, 4>); else go(embed_launch<float, 1>); }
+  else     { if (v4) go(embed_launch<__nv_bfloat16, 4>); else go(embed_launch<__nv_bfloat16, 1>); }
+  count_launch();
+  check_launch();
+}
+
+void sandwich_norm(bool f32, const void* y1, const void* y2, long long ldy, const float* w1, const float* w2,
+                   const float* w_post, float* x, const float* w_next, void* h, long long ldh, int rows, int dim,
+                   float eps, cudaStream_t stream) {
+  MB_REQUIRE(dim > 0 && dim <= 12000 && ldh >= dim && ldy >= dim, "sandwich_norm: row width out of range");
+  MB_REQUIRE(y2 == nullptr || (w1 && w2), "sandwich_norm: two inputs need their norm weights");
+  if (rows == 0) return;
+  const bool v4 = dim % 4 == 0 && ldh % 4 == 0 && ldy % 4 == 0;
+  auto go = [&](auto fn) { fn(y1, y2, ldy, w1, w2, w_post, x, w_next, h, ldh, rows, dim, eps, stream); };
+  if (f32) { if (v4) go(sandwich_launch<float, 4>); else go(sandwich_launch<float, 1>); }
+  else     { if (v4) go(sandwich_launch<__nv_bfloat16, 4>); else go(sandwich_launch<__nv_bfloat16, 1>); }
+  count_launch();
+  check_launch();
+}
+
+void qk_norm_append(bool f32, const void* proj, long long ld, int q_off, int k_off, int v_off, const float* q_gamma,
+                    const float* k_gamma, const RaggedBatch& rb, const int* block_table, int table_stride,
+                    int page_size, void* q_out, void* k_cache, void* v_cache, int heads, int kv_heads, int dk, int dv,
+                    float eps, cudaStream_t stream) {
+  if (rb.rows == 0) return;
+  const int grid = ceil_div((long long)rb.rows * (heads + 2 * kv_heads), 8);
+  if (f32)
+    qk_norm_append_kernel<float><<<grid, 256, 0, stream>>>(
+        (const float*)proj, ld, q_off, k_off, v_off, q_gamma, k_gamma, rb, block_table, table_stride, page_size,
+        (float*)q_out, (float*)k_cache, (float*)v_cache, heads, kv_heads, dk, dv, eps);
+  else
+    qk_norm_append_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(
+        (const __nv_bfloat16*)proj, ld, q_off, k_off, v_off, q_gamma, k_gamma, rb, block_table, table_stride,
+        page_size, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, heads, kv_heads, dk, dv,
+        eps);
+  count_launch();
+  check_launch();
+}
+
+void paged_attn_any(bool f32, const void* q, const void* k_cache, const void* v_cache, const RaggedBatch& rb,
+                    const int* block_table, int table_stride, int page_size, const void* gate, long long ld_gate,
+                    void* o, long long ldo, int heads, int kv_heads, int dk, int dv, float scale,
+                    cudaStream_t stream) {
+  MB_REQUIRE(heads % kv_heads == 0, "paged_attn_any: heads must be a multiple of kv_heads");
+  MB_REQUIRE(dk <= 1024 && dv <= 512, "paged_attn_any: head widths up to 1024 (keys) and 512 (values)");
+  if (rb.rows == 0) return;
+  const int grid = ceil_div((long long)rb.rows * heads, PA_WARPS);
+  const int smem = PA_WARPS * dk * 4;
+#define MB_PA(T, ND)                                                                                              \
+  paged_attn_any_kernel<T, ND><<<grid, PA_WARPS * 32, smem, stream>>>(                                            \
+      (const T*)q, (const T*)k_cache, (const T*)v_cache, rb, block_table, table_stride, page_size, (const T*)gate, \
+      ld_gate, (T*)o, ldo, heads, kv_heads, dk, dv, scale)
+  if (f32) {
+    if (dv <= 64) MB_PA(float, 2); else if (dv <= 128) MB_PA(float, 4); else if (dv <= 256) MB_PA(float, 8);
+    else MB_PA(float, 16);
+  } else {
+    if (dv <= 64) MB_PA(__nv_bfloat16, 2); else if (dv <= 128) MB_PA(__nv_bfloat16, 4);
+    else if (dv <= 256) MB_PA(__nv_bfloat16, 8); else MB_PA(__nv_bfloat16, 16);
+  }
+#undef MB_PA
+  count_launch();
+  check_launch();
+}
+
+void gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N,
+              int K, float alpha, cudaStream_t stream) {
+  if (M == 0 || N == 0) return;
+  gemm_f32_kernel<<<dim3((N + 63) / 64, (M + 63) / 64), 256, 0, stream>>>(A, lda, B, ldb, C, ldc, M, N, K, alpha);
+  count_launch();
+  check_launch();
+}
+
+void silu_gate(bool f32, const void* gu, long long ldg, int f, int f_off, void* h, long long ldh, int rows,
+               cudaStream_t stream) {
+  if (rows == 0) return;
+  const int grid = grid_for((long long)rows * ldh, 256, 16);
+  if (f32)
+    silu_gate_kernel<float><<<grid, 256, 0, stream>>>((const float*)gu, ldg, f, f_off, (float*)h, ldh, rows);
+  else
+    silu_gate_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)gu, ldg, f, f_off,
+                                                              (__nv_bfloat16*)h, ldh, rows);
+  count_launch();
+  check_launch();
+}
+
+}  // namespace mb

@@ -1,0 +1,267 @@
+// Linear recurrences with a decay per key channel: gated linear attention and the gated delta rule.
+//
+//   S <- diag(g_t) S;   u_t = v_t                        (gated linear attention)
+//                       u_t = beta_t (v_t - S^T k_t)     (delta rule)
+//   S <- S + k_t u_t^T; o_t = S^T q_t
+//
+// This file holds the token-by-token form, which works for every width and in both activation types
+// (it is what 32-bit engines and unusual widths use), and the steps around it: projections to 32-bit
+// q / k / v / log decay / beta (short convolution, silu, unit norms, decays), the convolution state,
+// and the per-head output norm with its gate. The columns of S belong to value channels and are
+// independent, so a warp owns a few of them (rows of S^T, lanes across the key channels).
+#include "common.cuh"
+#include "hybrid_api.h"
+#include "hybrid_dev.cuh"
+#include "host_util.h"
+
+namespace mb {
+namespace {
+
+struct PrepOut {
+  float *q, *k, *v, *lg, *beta;   // [rows, G, dim] x 2, [rows, H, vdim], [rows, H, dim], [rows, H]
+};
+
+// Input of channel c (within the concatenated q | k | v channels) j tokens before local token i.
+template <typename T>
+__device__ __forceinline__ float conv_tap(const T* __restrict__ col, long long ld, long long row, int i, int j,
+                                          const float* __restrict__ st, int channels, int taps, int c) {
+  if (i - j >= 0) return ldf(col + (row - j) * ld);
+  return st ? st[(long long)(taps - 1 + i - j) * channels + c] : 0.f;
+}
+
+template <typename T>
+__device__ __forceinline__ float conv_silu(const RecurrentSpec& s, const RecurrentInputs& in, const T* proj, long long row,
+                                           int i, const float* st, int channels, int c, int col) {
+  if (s.taps <= 0) return ldf(proj + row * in.ld + col);
+  float a = 0.f;
+  const float* w = in.conv_w + (long long)c * s.taps;
+  for (int j = 0; j < s.taps; ++j)
+    a = fmaf(w[s.taps - 1 - j], conv_tap(proj + col, in.ld, row, i, j, st, channels, s.taps, c), a);
+  return silu_f(a);
+}
+
+// One CTA per token.
+template <typename T>
+__global__ void __launch_bounds__(256)
+recurrent_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, PrepOut out) {
+  extern __shared__ float sm[];   // q then k of the token, after convolution
+  const long long row = blockIdx.x;
+  const int b = rb.row_seq[row];
+  const int i = (int)row - rb.cu_q[b];
+  const int base = rb.kv_lens[b] - (rb.cu_q[b + 1] - rb.cu_q[b]);
+  const int cq = s.kv_heads * s.dim, cv = s.heads * s.vdim, channels = 2 * cq + cv;
+  const T* proj = static_cast<const T*>(in.proj);
+  const float* st = (base > 0 && s.taps > 1) ? in.conv_state + (long long)rb.slots[b] * (s.taps - 1) * channels : nullptr;
+  for (int c = threadIdx.x; c < 2 * cq; c += blockDim.x) {
+    const int col = c < cq ? in.q_off + c : in.k_off + c - cq;
+    sm[c] = conv_silu(s, in, proj, row, i, st, channels, c, col);
+  }
+  for (int c = threadIdx.x; c < cv; c += blockDim.x)
+    out.v[row * cv + c] = conv_silu(s, in, proj, row, i, st, channels, 2 * cq + c, in.v_off + c);
+  for (int c = threadIdx.x; c < s.heads * s.dim; c += blockDim.x) {
+    const float z = in.z[row * in.ldz + c] + in.z_bias[c];
+    out.lg[row * s.heads * s.dim + c] =
+        s.decay_kind == 1 ? -expf(in.a_log[c / s.dim]) * softplus_f(z) : -softplus_f(-z) * s.inv_tau;
+  }
+  if (s.delta)
+    for (int h = threadIdx.x; h < s.heads; h += blockDim.x)
+      out.beta[row * s.heads + h] = sigmoid_f(ldf(proj + row * in.ld + in.b_off + h));
+  __syncthreads();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  for (int g = warp; g < 2 * s.kv_heads; g += nw) {
+    const float* x = sm + g * s.dim;
+    float r = 1.f;
+    if (s.unit_norm) {
+      float ss = 0.f;
+      for (int c = lane; c < s.dim; c += 32) ss += x[c] * x[c];
+      r = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
+    }
+    const bool is_q = g < s.kv_heads;
+    if (is_q) r *= s.q_scale;
+    float* dst = is_q ? out.q + row * cq + g * s.dim : out.k + row * cq + (g - s.kv_heads) * s.dim;
+    for (int c = lane; c < s.dim; c += 32) dst[c] = x[c] * r;
+  }
+}
+
+// grid (sequence, head, value block); a warp owns R rows of S^T in registers, lane l holds key channels
+// l, l + 32, ...
+constexpr int RS_WARPS = 4, RS_R = 4;
+template <int NI>
+__global__ void __launch_bounds__(RS_WARPS * 32)
+recurrent_scan_seq_kernel(RecurrentSpec s, RaggedBatch rb, PrepOut in, float* __restrict__ state, float* __restrict__ o) {
+  const int b = blockIdx.x, h = blockIdx.y;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int v0 = (blockIdx.z * RS_WARPS + warp) * RS_R;
+  if (v0 >= s.vdim) return;
+  const int r0 = rb.cu_q[b], r1 = rb.cu_q[b + 1];
+  if (r0 >= r1) return;
+  const bool fresh = rb.kv_lens[b] == r1 - r0;
+  const int g = h / (s.heads / s.kv_heads);
+  float* stp = state + (((long long)rb.slots[b] * s.heads + h) * s.vdim + v0) * s.dim;
+  float S[RS_R][NI];
+#pragma unroll
+  for (int r = 0; r < RS_R; ++r)
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int c = lane + 32 * n;
+      S[r][n] = (!fresh && c < s.dim && v0 + r < s.vdim) ? stp[(long long)r * s.dim + c] : 0.f;
+    }
+  for (long long t = r0; t < r1; ++t) {
+    float q[NI], k[NI], d[NI];
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int c = lane + 32 * n;
+      const bool ok = c < s.dim;
+      q[n] = ok ? in.q[(t * s.kv_heads + g) * s.dim + c] : 0.f;
+      k[n] = ok ? in.k[(t * s.kv_heads + g) * s.dim + c] : 0.f;
+      d[n] = ok ? expf(in.lg[(t * s.heads + h) * s.dim + c]) : 0.f;
+    }
+    float u[RS_R];
+#pragma unroll
+    for (int r = 0; r < RS_R; ++r) {
+      u[r] = v0 + r < s.vdim ? in.v[(t * s.heads + h) * s.vdim + v0 + r] : 0.f;
+#pragma unroll
+      for (int n = 0; n < NI; ++n) S[r][n] *= d[n];
+    }
+    if (s.delta) {
+      const float beta = in.beta[t * s.heads + h];
+#pragma unroll
+      for (int r = 0; r < RS_R; ++r) {
+        float a = 0.f;
+#pragma unroll
+        for (int n = 0; n < NI; ++n) a = fmaf(S[r][n], k[n], a);
+        u[r] = beta * (u[r] - warp_sum(a));
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < RS_R; ++r) {
+      float a = 0.f;
+#pragma unroll
+      for (int n = 0; n < NI; ++n) {
+        S[r][n] = fmaf(k[n], u[r], S[r][n]);
+        a = fmaf(S[r][n], q[n], a);
+      }
+      a = warp_sum(a);
+      if (lane == 0 && v0 + r < s.vdim) o[(t * s.heads + h) * s.vdim + v0 + r] = a;
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < RS_R; ++r)
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int c = lane + 32 * n;
+      if (c < s.dim && v0 + r < s.vdim) stp[(long long)r * s.dim + c] = S[r][n];
+    }
+}
+
+// One thread per (sequence, channel): the last taps - 1 inputs of the sequence become the state.
+template <typename T>
+__global__ void conv_state_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb) {
+  const int cq = s.kv_heads * s.dim, channels = 2 * cq + s.heads * s.vdim;
+  const int c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y;
+  if (c >= channels) return;
+  const int r0 = rb.cu_q[b], len = rb.cu_q[b + 1] - r0, n = s.taps - 1;
+  if (len <= 0) return;
+  const bool fresh = rb.kv_lens[b] == len;
+  const int col = c < cq ? in.q_off + c : (c < 2 * cq ? in.k_off + c - cq : in.v_off + c - 2 * cq);
+  float* st = in.conv_state + (long long)rb.slots[b] * n * channels + c;
+  const T* proj = static_cast<const T*>(in.proj) + col;
+  // entry j holds the input of token len - n + j; an entry moves down, never up, so in-place order is safe
+  for (int j = 0; j < n; ++j) {
+    const int i = len - n + j;
+    float v;
+    if (i >= 0) v = ldf(proj + (long long)(r0 + i) * in.ld);
+    else v = fresh ? 0.f : st[(long long)(n + i) * channels];
+    st[(long long)j * channels] = v;
+  }
+}
+
+// One warp per (token, head).
+template <typename T>
+__global__ void head_norm_gate_kernel(RecurrentSpec s, const float* __restrict__ o, const float* __restrict__ gamma,
+                                      const T* __restrict__ gate, long long ld_gate, T* __restrict__ out, long long ldo,
+                                      long long rows) {
+  const int lane = threadIdx.x & 31;
+  const long long w = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (w >= rows * s.heads) return;
+  const long long t = w / s.heads;
+  const int h = (int)(w % s.heads);
+  const float* x = o + w * s.vdim;
+  float ss = 0.f;
+  for (int i = lane; i < s.vdim; i += 32) ss += x[i] * x[i];
+  const float r = 1.f / sqrtf(warp_sum(ss) / (float)s.vdim + s.eps);
+  const T* gp = gate + t * ld_gate + h * s.vdim;
+  T* op = out + t * ldo + h * s.vdim;
+  for (int i = lane; i < s.vdim; i += 32) {
+    const float z = ldf(gp + i);
+    stf(op + i, x[i] * r * gamma[i] * (s.gate_kind == 1 ? sigmoid_f(z) : silu_f(z)));
+  }
+  if (h == s.heads - 1)
+    for (long long i = (long long)s.heads * s.vdim + lane; i < ldo; i += 32) stf(out + t * ldo + i, 0.f);
+}
+
+PrepOut carve(const RecurrentSpec& s, float* p, long long rows) {
+  PrepOut o;
+  o.q = p;
+  o.k = o.q + rows * s.kv_heads * s.dim;
+  o.v = o.k + rows * s.kv_heads * s.dim;
+  o.lg = o.v + rows * s.heads * s.vdim;
+  o.beta = o.lg + rows * s.heads * s.dim;
+  return o;
+}
+
+void check_spec(const RecurrentSpec& s) {
+  MB_REQUIRE(s.heads > 0 && s.kv_heads > 0 && s.heads % s.kv_heads == 0, "recurrent: heads must be a multiple of kv_heads");
+  MB_REQUIRE(s.dim > 0 && s.dim <= 256 && s.vdim > 0, "recurrent: key width up to 256");
+  MB_REQUIRE(s.taps >= 0 && s.taps <= 64, "recurrent: convolution taps out of range");
+}
+
+}  // namespace
+
+void recurrent_scan_seq(bool f32, const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb,
+                        float* scratch, float* o, cudaStream_t stream) {
+  check_spec(s);
+  if (rb.rows == 0) return;
+  const PrepOut p = carve(s, scratch, rb.rows);
+  const int smem = 2 * s.kv_heads * s.dim * 4;
+  MB_REQUIRE(smem <= 200 * 1024, "recurrent: q / k of one token exceed shared memory");
+  if (smem > 48 * 1024) {
+    if (f32) MB_CUDA_CHECK(cudaFuncSetAttribute(recurrent_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    else MB_CUDA_CHECK(cudaFuncSetAttribute(recurrent_prep_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  }
+  if (f32) recurrent_prep_kernel<float><<<rb.rows, 256, smem, stream>>>(s, in, rb, p);
+  else recurrent_prep_kernel<__nv_bfloat16><<<rb.rows, 256, smem, stream>>>(s, in, rb, p);
+  const dim3 grid(rb.n_seq, s.heads, (s.vdim + RS_WARPS * RS_R - 1) / (RS_WARPS * RS_R));
+  if (s.dim <= 32) recurrent_scan_seq_kernel<1><<<grid, RS_WARPS * 32, 0, stream>>>(s, rb, p, in.state, o);
+  else if (s.dim <= 64) recurrent_scan_seq_kernel<2><<<grid, RS_WARPS * 32, 0, stream>>>(s, rb, p, in.state, o);
+  else if (s.dim <= 128) recurrent_scan_seq_kernel<4><<<grid, RS_WARPS * 32, 0, stream>>>(s, rb, p, in.state, o);
+  else recurrent_scan_seq_kernel<8><<<grid, RS_WARPS * 32, 0, stream>>>(s, rb, p, in.state, o);
+  count_launch(2);
+  check_launch();
+}
+
+void conv_state_update(bool f32, const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb,
+                       cudaStream_t stream) {
+  if (s.taps <= 1 || rb.n_seq == 0) return;
+  const int channels = 2 * s.kv_heads * s.dim + s.heads * s.vdim;
+  const dim3 grid((channels + 255) / 256, rb.n_seq);
+  if (f32) conv_state_kernel<float><<<grid, 256, 0, stream>>>(s, in, rb);
+  else conv_state_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(s, in, rb);
+  count_launch();
+  check_launch();
+}
+
+void head_norm_gate(bool f32, const RecurrentSpec& s, const float* o, const float* gamma, const void* gate,
+                    long long ld_gate, void* out, long long ldo, int rows, cudaStream_t stream) {
+  if (rows == 0) return;
+  const int grid = ceil_div((long long)rows * s.heads, 8);
+  if (f32)
+    head_norm_gate_kernel<float><<<grid, 256, 0, stream>>>(s, o, gamma, (const float*)gate, ld_gate, (float*)out, ldo, rows);
+  else
+    head_norm_gate_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(s, o, gamma, (const __nv_bfloat16*)gate, ld_gate,
+                                                                   (__nv_bfloat16*)out, ldo, rows);
+  count_launch();
+  check_launch();
+}
+
+}  // namespace mb

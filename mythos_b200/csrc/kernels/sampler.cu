@@ -29,22 +29,28 @@ __device__ __forceinline__ unsigned long long splitmix64(unsigned long long x) {
   return x ^ (x >> 31);
 }
 
+__device__ __forceinline__ float logit(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float logit(const float* p) { return *p; }
+
+// Logits are bf16 or fp32 (T).
+template <typename T>
 struct RowView {
-  const __nv_bfloat16* logits;
+  const T* logits;
   const unsigned char* allow;
   const uint32_t* seen;  // bitmap of tokens subject to the repetition penalty (shared memory)
   float inv_temp, penalty;
   bool use_penalty;
   __device__ __forceinline__ float at(int i) const {
     if (allow && !allow[i]) return -INFINITY;
-    float v = __bfloat162float(logits[i]);
+    float v = logit(logits + i);
     if (use_penalty && (seen[i >> 5] >> (i & 31)) & 1u) v = v > 0.f ? v / penalty : v * penalty;
     return v * inv_temp;
   }
 };
 
+template <typename T>
 __global__ void __launch_bounds__(SAMP_THREADS)
-sampler_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int vocab, const int* __restrict__ history,
+sampler_kernel(const T* __restrict__ logits, long long ld, int vocab, const int* __restrict__ history,
                int history_len, const unsigned char* __restrict__ allow_mask, SamplerArgs a,
                int* __restrict__ out_tokens, float* __restrict__ out_logprob) {
   extern __shared__ uint32_t seen[];  // ceil(vocab/32) words
@@ -67,7 +73,7 @@ sampler_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int vocab
     }
     __syncthreads();
   }
-  RowView rv{logits + (long long)row * ld, allow_mask ? allow_mask + (long long)row * vocab : nullptr, seen,
+  RowView<T> rv{logits + (long long)row * ld, allow_mask ? allow_mask + (long long)row * vocab : nullptr, seen,
              greedy ? 1.f : 1.f / a.temperature, a.repetition_penalty, use_pen};
 
   // ---- max / argmax (first maximum wins)
@@ -196,24 +202,25 @@ __device__ __forceinline__ unsigned long long argmax_key(float v, int idx) {
   return ((unsigned long long)ord << 32) | (uint32_t)(0xFFFFFFFFu - (uint32_t)idx);
 }
 
+template <typename T>
 __global__ void __launch_bounds__(256)
-argmax_rows_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int vocab, int chunks,
+argmax_rows_kernel(const T* __restrict__ logits, long long ld, int vocab, int chunks,
                    int* __restrict__ out_tokens) {
   __shared__ unsigned long long s_key[8];
   const int row = blockIdx.x, chunk = blockIdx.y, tid = threadIdx.x;
-  const __nv_bfloat16* lp = logits + (long long)row * ld;
+  const T* lp = logits + (long long)row * ld;
   const int vec = vocab >> 3;                                   // whole 8-element groups
   const int per = (vec + chunks - 1) / chunks;
   const int v0 = chunk * per, v1 = min(vec, v0 + per);
   unsigned long long best = 0ull;
-  const bool aligned = ((reinterpret_cast<uintptr_t>(lp) & 15) == 0);
+  const bool aligned = sizeof(T) == 2 && ((reinterpret_cast<uintptr_t>(lp) & 15) == 0);
   for (int g = v0 + tid; g < v1; g += blockDim.x) {
     float f[8];
     if (aligned) {
       unpack8(ldg8(lp, (long long)g * 8), f);
     } else {
 #pragma unroll
-      for (int j = 0; j < 8; ++j) f[j] = __bfloat162float(lp[g * 8 + j]);
+      for (int j = 0; j < 8; ++j) f[j] = logit(lp + g * 8 + j);
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -223,7 +230,7 @@ argmax_rows_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int v
   }
   if (chunk == chunks - 1)                                      // ragged tail of the row
     for (int i = vec * 8 + tid; i < vocab; i += blockDim.x) {
-      const unsigned long long k = argmax_key(__bfloat162float(lp[i]), i);
+      const unsigned long long k = argmax_key(logit(lp + i), i);
       best = k > best ? k : best;
     }
 #pragma unroll
@@ -250,7 +257,7 @@ argmax_rows_kernel(const __nv_bfloat16* __restrict__ logits, long long ld, int v
 
 void sample_tokens(const void* logits, long long ld, int rows, int vocab, const int* history, int history_len,
                    const unsigned char* allow_mask, SamplerArgs a, int* out_tokens, float* out_logprob, float* scratch,
-                   cudaStream_t stream) {
+                   cudaStream_t stream, bool f32) {
   (void)scratch;
   if (rows == 0) return;
   const bool plain_greedy = a.temperature < 1e-5f && allow_mask == nullptr && out_logprob == nullptr &&
@@ -260,16 +267,23 @@ void sample_tokens(const void* logits, long long ld, int rows, int vocab, const 
     const int max_chunks = (vocab / 8 + 2047) / 2048;          // at least 8 vectors per thread
     if (chunks > max_chunks) chunks = max_chunks;
     if (chunks < 1) chunks = 1;
-    argmax_rows_kernel<<<dim3(rows, chunks), 256, 0, stream>>>((const __nv_bfloat16*)logits, ld, vocab, chunks,
-                                                               out_tokens);
+    if (f32)
+      argmax_rows_kernel<float><<<dim3(rows, chunks), 256, 0, stream>>>((const float*)logits, ld, vocab, chunks, out_tokens);
+    else
+      argmax_rows_kernel<__nv_bfloat16><<<dim3(rows, chunks), 256, 0, stream>>>((const __nv_bfloat16*)logits, ld, vocab,
+                                                                                chunks, out_tokens);
     count_launch();
     check_launch();
     return;
   }
   const size_t smem = (size_t)((vocab + 31) / 32) * 4;
   MB_REQUIRE(smem <= 48 * 1024, "sample_tokens: vocabulary too large for the repetition bitmap");
-  sampler_kernel<<<rows, SAMP_THREADS, smem, stream>>>((const __nv_bfloat16*)logits, ld, vocab, history, history_len,
-                                                       allow_mask, a, out_tokens, out_logprob);
+  if (f32)
+    sampler_kernel<float><<<rows, SAMP_THREADS, smem, stream>>>((const float*)logits, ld, vocab, history, history_len,
+                                                                allow_mask, a, out_tokens, out_logprob);
+  else
+    sampler_kernel<__nv_bfloat16><<<rows, SAMP_THREADS, smem, stream>>>((const __nv_bfloat16*)logits, ld, vocab, history,
+                                                                        history_len, allow_mask, a, out_tokens, out_logprob);
   count_launch();
   check_launch();
 }

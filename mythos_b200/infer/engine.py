@@ -182,6 +182,9 @@ class _Layer:
 
 
 class InferenceEngine:
+    # every prefill goes through the paged kernels (no contiguous form)
+    paged_prefill_only = False
+
     def __init__(self, cfg: TransformerConfig, device="cuda", max_batch: int = 64, max_seq_len: int | None = None,
                  page_size: int = 16, tp: TPContext | None = None, kv_pages: int | None = None,
                  kv_dtype: str = "bf16"):
@@ -237,6 +240,10 @@ class InferenceEngine:
         """Pack a (trained or random) ``DenseModel`` into inference weights. Under tensor
         parallelism every rank packs its own shard of each matrix."""
         cfg = model.cfg
+        if cls is InferenceEngine and not isinstance(cfg, TransformerConfig):
+            from .hybrid import HybridEngine      # layer-list designs
+
+            return HybridEngine.from_model(model, **kw)
         eng = cls(cfg, **kw)
         dev = eng.device
         W, r = eng.world, eng.rank
@@ -512,7 +519,7 @@ class InferenceEngine:
             else:
                 C.kv_append(k, v, self.cache.k[li], self.cache.v[li], table, pos, seq_ids)
             if paged is not None:
-                cu_q, kv_lens, rows, max_q = paged
+                cu_q, kv_lens, rows, max_q = paged[:4]
                 o = torch.empty(T, H, D, device=self.device, dtype=torch.bfloat16)
                 C.flash_attn_paged_prefill(q, self.cache.k[li], self.cache.v[li], rows, cu_q, kv_lens, o, max_q, scale,
                                            native.status_word(self.device))
@@ -578,7 +585,7 @@ class InferenceEngine:
         else:
             C.kv_append(k, v, self.cache.k[li], self.cache.v[li], table, pos, seq_ids)
         if paged is not None:
-            cu_q, kv_lens, rows, max_q = paged
+            cu_q, kv_lens, rows, max_q = paged[:4]
             o = torch.empty(T, H, D, device=self.device, dtype=torch.bfloat16)
             C.flash_attn_paged_prefill(q, self.cache.k[li], self.cache.v[li], rows, cu_q, kv_lens, o, max_q, scale,
                                        native.status_word(self.device))
@@ -670,16 +677,25 @@ class InferenceEngine:
         tokens, packed in the order given, and the row offsets of the sequences."""
         dev = self.device
         lens = [len(t) for t in token_lists]
-        ids = torch.tensor([x for t in token_lists for x in t], dtype=torch.int32, device=dev)
-        pos = torch.cat([torch.arange(b, b + n, dtype=torch.int32) for b, n in zip(bases, lens)]).to(dev)
-        sid = torch.cat([torch.full((n,), s, dtype=torch.int32) for s, n in zip(seqs, lens)]).to(dev)
+        n, T = len(lens), sum(lens)
         cu = [0]
-        for n in lens:
-            cu.append(cu[-1] + n)
-        cu_q = torch.tensor(cu, dtype=torch.int32, device=dev)
-        kv_lens = torch.tensor([b + n for b, n in zip(bases, lens)], dtype=torch.int32, device=dev)
-        rows = self.cache.block_table.index_select(0, torch.tensor(seqs, dtype=torch.long, device=dev)).contiguous()
-        h = self._forward(ids, pos, sid, None, paged=(cu_q, kv_lens, rows, max(lens)))
+        for k in lens:
+            cu.append(cu[-1] + k)
+        # one host buffer, one copy: ids | positions | slot per token | sequence per token | per-sequence arrays
+        host = torch.empty(4 * T + 3 * n + 1, dtype=torch.int32, pin_memory=dev.type == "cuda")
+        parts = host.split([T, T, T, T, n + 1, n, n])
+        for i, (s, base, toks) in enumerate(zip(seqs, bases, token_lists)):
+            lo, hi = cu[i], cu[i + 1]
+            parts[0][lo:hi] = torch.as_tensor(toks, dtype=torch.int32)
+            parts[1][lo:hi] = torch.arange(base, base + lens[i], dtype=torch.int32)
+            parts[2][lo:hi] = s
+            parts[3][lo:hi] = i
+        parts[4].copy_(torch.tensor(cu, dtype=torch.int32))
+        parts[5].copy_(torch.tensor([b + k for b, k in zip(bases, lens)], dtype=torch.int32))
+        parts[6].copy_(torch.tensor(seqs, dtype=torch.int32))
+        ids, pos, sid, row_seq, cu_q, kv_lens, slots = host.to(dev, non_blocking=True).split([T, T, T, T, n + 1, n, n])
+        rows = self.cache.block_table.index_select(0, slots.long()).contiguous()
+        h = self._forward(ids, pos, sid, None, paged=(cu_q, kv_lens, rows, max(lens), slots, row_seq))
         return h, cu
 
     @torch.no_grad()
@@ -748,7 +764,8 @@ class InferenceEngine:
         torch.cuda.synchronize(dev)
         t0 = time.perf_counter()
         # ---- prefill
-        chunked = (ragged or B * S > getattr(self, "prefill_chunk_threshold", 1 << 30)) and self._paged_prefill_ok()
+        chunked = self.paged_prefill_only or \
+            ((ragged or B * S > getattr(self, "prefill_chunk_threshold", 1 << 30)) and self._paged_prefill_ok())
         with trace.span("prefill", dev):
             if chunked:
                 last = self._prefill_chunked(seqs, lists)
@@ -831,8 +848,8 @@ class InferenceEngine:
     # ------------------------------------------------------------------ text-level API
     @classmethod
     def load(cls, path: str, device="cuda", **kw) -> "InferenceEngine":
-        """Engine from an ``.oil`` file and its sibling ``.vocab`` tokenizer (byte-level ids when the
-        vocabulary file is missing): the reference's ``engine::InferenceEngine::load`` + ``init``
+        """Engine from an ``.oil`` file or a checkpoint folder and its sibling ``.vocab`` tokenizer (byte-level
+        ids when the vocabulary file is missing): the reference's ``engine::InferenceEngine::load`` + ``init``
         (engines/inference/inference.cpp)."""
         import os
 
@@ -841,6 +858,7 @@ class InferenceEngine:
 
         model, _ = load_model(path, device=device)
         kw.setdefault("max_seq_len", model.cfg.max_seq_len)
+        path = path.rstrip("/")
         eng = cls.from_model(model, device=device, **kw)
         vocab = (path[:-4] if path.endswith(".oil") else path) + ".vocab"
         eng.tokenizer = BPETokenizer.load(vocab) if os.path.exists(vocab) else None
@@ -947,7 +965,7 @@ class InferenceEngine:
         dev = self.device
         self._prepare_decode_scratch(self.max_batch, self.max_seq_len)
         self.last_prefix_hit = covered
-        if covered == 0 and not (paged_ok and S > getattr(self, "prefill_chunk", 8192)):
+        if covered == 0 and not self.paged_prefill_only and not (paged_ok and S > getattr(self, "prefill_chunk", 8192)):
             t = torch.tensor(ids, dtype=torch.int32, device=dev)
             pos = torch.arange(S, device=dev, dtype=torch.int32)
             sid = torch.full((S,), seq, device=dev, dtype=torch.int32)
@@ -1000,17 +1018,57 @@ class InferenceEngine:
         ids = torch.as_tensor(tokens, dtype=torch.int32).to(dev).reshape(n)
         pos = torch.tensor([cache.lens[s] for s in seqs], dtype=torch.int32, device=dev)
         sid = torch.tensor(list(seqs), dtype=torch.int32, device=dev)
+        h = self._decode_rows(ids, pos, sid)
+        for s in seqs:
+            cache.advance(s, 1)
+        return self._logits(h)
+
+    def _decode_rows(self, ids, pos, sid):
+        """One token of each of the sequences ``sid`` at the positions ``pos`` -> hidden states."""
+        cache = self.cache
         # the decode kernel indexes block-table rows by position in the batch: gather the rows
         table_rows = cache.block_table.index_select(0, sid.long()).contiguous()
         saved = cache.block_table
         cache.block_table = table_rows
         try:
-            h = self._forward(ids, pos, torch.arange(n, device=dev, dtype=torch.int32), pos + 1, None)
+            return self._forward(ids, pos, torch.arange(ids.numel(), device=self.device, dtype=torch.int32), pos + 1, None)
         finally:
             cache.block_table = saved
-        for s in seqs:
-            cache.advance(s, 1)
-        return self._logits(h)
+
+    @torch.no_grad()
+    def step_hidden(self, seqs, token_lists):
+        """One batch over any mix of work: ``token_lists[i]`` are the next tokens of sequence ``seqs[i]``
+        (a whole prompt, a portion of one, or one decoded token), which run from what the cache holds
+        of it. Returns the packed hidden states of the new tokens and the row offset of every sequence."""
+        cache = self.cache
+        if len(set(seqs)) != len(seqs) or any(len(t) == 0 for t in token_lists):
+            raise ValueError("step: sequences must be distinct and bring at least one token each")
+        if not (self.paged_prefill_only or self._paged_prefill_ok()):
+            raise ValueError("step: this engine's cache has no paged prefill kernel (int8 pages or head width)")
+        bases = [cache.lens[s] for s in seqs]
+        for s, t in zip(seqs, token_lists):
+            if cache.lens[s] + len(t) > self.max_seq_len:
+                raise ValueError(f"sequence would exceed {self.max_seq_len} tokens")
+            cache.reserve(s, len(t))
+        cache.sync_tables()
+        h, cu = self._prefill_paged(list(seqs), token_lists, bases)
+        for s, t in zip(seqs, token_lists):
+            cache.advance(s, len(t))
+        return h, cu
+
+    @torch.no_grad()
+    def step(self, seqs, token_lists, want=None):
+        """:meth:`step_hidden`, then the logits of the places ``want[i]`` among the new tokens of each
+        sequence (default: its last one), in that order; ``None`` when nothing is wanted."""
+        h, cu = self.step_hidden(seqs, token_lists)
+        if want is None:
+            want = [[len(t) - 1] for t in token_lists]
+        rows = [cu[i] + int(p) for i, places in enumerate(want) for p in places]
+        if not rows:
+            return None
+        if len(rows) == h.shape[0] and rows == list(range(len(rows))):
+            return self._logits(h)
+        return self._logits(h.index_select(0, torch.tensor(rows, device=h.device)))
 
     def release(self, seq: int) -> None:
         self.cache.free_sequence(seq)

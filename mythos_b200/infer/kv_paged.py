@@ -47,15 +47,47 @@ class PageAllocator:
         return self.num_pages - len(self.free)
 
 
+class RecurrentStatePool:
+    """Per-sequence state of recurrent layers, one slot per sequence slot of the cache. ``add`` gives a
+    layer's tensor ``[slots, ...]`` (32-bit). A slot is not cleared when it changes hands: the kernels
+    start from zero for a sequence without earlier tokens."""
+
+    def __init__(self, slots: int, device="cuda"):
+        self.slots, self.device = slots, torch.device(device)
+        self.tensors: list[torch.Tensor] = []
+
+    def add(self, *shape: int) -> torch.Tensor:
+        t = torch.zeros((self.slots,) + shape, device=self.device, dtype=torch.float32)
+        self.tensors.append(t)
+        return t
+
+    def size_bytes(self) -> int:
+        return sum(t.numel() * 4 for t in self.tensors)
+
+    def save(self, slot: int):
+        return [t[slot].cpu() for t in self.tensors]
+
+    def restore(self, slot: int, saved) -> None:
+        for t, s in zip(self.tensors, saved):
+            t[slot].copy_(s)
+
+
 class PagedKVCache:
     def __init__(self, num_layers: int, kv_heads: int, head_dim: int, num_pages: int, page_size: int = 16,
-                 max_seqs: int = 64, max_pages_per_seq: int = 256, device="cuda", dtype=torch.bfloat16):
+                 max_seqs: int = 64, max_pages_per_seq: int = 256, device="cuda", dtype=torch.bfloat16,
+                 layer_shapes=None, states: RecurrentStatePool | None = None):
+        """``layer_shapes``: per attention layer ``(kv_heads, key width, value width)`` where the layers
+        differ or the two widths do; ``states``: the recurrent layers' per-sequence state, which follows
+        the sequence slots (a prefix is then never shared: its pages alone do not determine the rest)."""
         self.num_layers, self.kv_heads, self.head_dim = num_layers, kv_heads, head_dim
         self.page_size, self.max_seqs, self.max_pages = page_size, max_seqs, max_pages_per_seq
         self.device = torch.device(device)
-        shape = (num_pages, page_size, kv_heads, head_dim)
-        self.k = [torch.zeros(shape, device=self.device, dtype=dtype) for _ in range(num_layers)]
-        self.v = [torch.zeros(shape, device=self.device, dtype=dtype) for _ in range(num_layers)]
+        self.states = states
+        shapes = layer_shapes if layer_shapes is not None else [(kv_heads, head_dim, head_dim)] * num_layers
+        if len(shapes) != num_layers or (layer_shapes is not None and dtype == torch.int8):
+            raise ValueError("layer_shapes: one entry per layer, not with int8 pages")
+        self.k = [torch.zeros((num_pages, page_size, g, dk), device=self.device, dtype=dtype) for g, dk, _ in shapes]
+        self.v = [torch.zeros((num_pages, page_size, g, dv), device=self.device, dtype=dtype) for g, _, dv in shapes]
         # int8 pages carry one fp32 scale (max|x| / 127) per (token, kv head); the append kernel
         # writes them and the decode kernel folds them into the score and the probability
         self.int8 = dtype == torch.int8
@@ -120,6 +152,8 @@ class PagedKVCache:
     def share_prefix(self, seq: int, tokens) -> int:
         """If full pages holding a prefix of ``tokens`` are cached, map them into ``seq`` (their
         reference counts go up) and return the number of tokens covered; else 0."""
+        if self.states is not None:
+            return 0
         n_full = len(tokens) // self.page_size
         for n in range(n_full, 0, -1):
             entry = self.prefix_index.get(self._prefix_key(tokens[: n * self.page_size]))
@@ -137,7 +171,7 @@ class PagedKVCache:
 
     def publish_prefix(self, seq: int, tokens, max_entries: int = 1024) -> None:
         n_full = min(len(tokens), self.lens[seq]) // self.page_size
-        if n_full == 0:
+        if n_full == 0 or self.states is not None:
             return
         pages = [int(self.block_table_host[seq, i]) for i in range(n_full)]
         self.prefix_index[self._prefix_key(tokens[: n_full * self.page_size])] = [(p, self.alloc.gen[p]) for p in pages]
@@ -149,7 +183,9 @@ class PagedKVCache:
         return self.alloc.used / max(1, self.alloc.num_pages)
 
     def size_bytes(self) -> int:
-        n = 2 * self.num_layers * self.k[0].numel() * self.k[0].element_size()
+        n = sum(t.numel() * t.element_size() for t in self.k + self.v)
+        if self.states is not None:
+            n += self.states.size_bytes()
         if self.int8:
             n += 2 * self.num_layers * self.k_scale[0].numel() * 4
         return n
@@ -163,7 +199,8 @@ class PagedKVCache:
         for layer in range(self.num_layers):
             hk = torch.empty((len(pages),) + tuple(self.k[layer].shape[1:]), dtype=self.k[layer].dtype,
                              pin_memory=self.device.type == "cuda")
-            hv = torch.empty_like(hk, pin_memory=self.device.type == "cuda")
+            hv = torch.empty((len(pages),) + tuple(self.v[layer].shape[1:]), dtype=self.v[layer].dtype,
+                             pin_memory=self.device.type == "cuda")
             hk.copy_(self.k[layer][idx], non_blocking=True)
             hv.copy_(self.v[layer][idx], non_blocking=True)
             if self.int8:
@@ -172,11 +209,12 @@ class PagedKVCache:
                 host.append((hk, hv, ks, vs))
             else:
                 host.append((hk, hv))
+        state = self.states.save(seq) if self.states is not None else None
         if self.device.type == "cuda":
             torch.cuda.current_stream(self.device).synchronize()
         length = self.lens[seq]
         self.free_sequence(seq)
-        return {"len": length, "pages": host}
+        return {"len": length, "pages": host, "state": state}
 
     def restore_sequence(self, handle) -> int:
         seq = self.new_sequence()
@@ -189,13 +227,15 @@ class PagedKVCache:
             if self.int8:
                 self.k_scale[layer].view(-1, self.page_size, self.kv_heads)[idx] = rec[2].to(self.device)
                 self.v_scale[layer].view(-1, self.page_size, self.kv_heads)[idx] = rec[3].to(self.device)
+        if self.states is not None:
+            self.states.restore(seq, handle["state"])
         self.lens[seq] = handle["len"]
         return seq
 
     def save_pages(self, seq: int, path: str) -> None:
         """File tier: write a sequence's pages to ``path`` (torch.save of the offload handle)."""
         h = self.offload_sequence(seq)
-        torch.save({"len": h["len"], "pages": [tuple(t.clone() for t in rec) for rec in h["pages"]]}, path)
+        torch.save({"len": h["len"], "state": h["state"], "pages": [tuple(t.clone() for t in rec) for rec in h["pages"]]}, path)
 
     def load_pages(self, path: str) -> int:
         return self.restore_sequence(torch.load(path))

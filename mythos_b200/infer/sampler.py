@@ -72,11 +72,11 @@ def sample_reference(logits, history, cfg: SamplerConfig, allow_mask=None, gener
 
 
 def sample(logits, cfg: SamplerConfig, history=None, allow_mask=None, step: int = 0, out=None, logprobs=None):
-    """One token per row. logits: [rows, V] (bf16 on CUDA). Returns int32 [rows]."""
+    """One token per row. logits: [rows, V] (bf16 or fp32 on CUDA). Returns int32 [rows]."""
     if logits.is_cuda:
         if out is None:
             out = torch.empty(logits.shape[0], device=logits.device, dtype=torch.int32)
-        native.require().sample_tokens(logits, history, allow_mask, cfg.temperature, cfg.top_k, cfg.top_p,
+        native.require_sampler().sample_tokens(logits, history, allow_mask, cfg.temperature, cfg.top_k, cfg.top_p,
                                        cfg.repetition_penalty, (cfg.seed * 1000003 + step) & 0x7FFFFFFFFFFFFFFF, out,
                                        logprobs)
         return out

@@ -1,0 +1,139 @@
+"""Weights of a layer-list model (:mod:`.hybrid_config`) under their checkpoint names.
+
+The model object holds tensors; the computation is the inference engine's
+(:mod:`mythos_b200.infer.hybrid`), which packs them into the layouts its kernels read. ``forward`` runs
+whole sequences through such an engine, so the model-level helpers (log-probabilities, beam search,
+embeddings, reranking) work as they do for the other models. There is no CPU forward.
+"""
+from __future__ import annotations
+
+import torch
+import torch.nn as nn
+
+from .hybrid_config import AttentionMixer, HybridConfig, ParallelMixer, RecurrentMixer
+
+
+def _attention_shapes(p: str, m: AttentionMixer, d: int) -> dict:
+    return {p + "q": (m.heads * m.dim, d), p + "k": (m.kv_heads * m.dim, d), p + "v": (m.kv_heads * m.vdim, d),
+            p + "q.norm": (m.dim,), p + "k.norm": (m.dim,), p + "g": (m.heads, d), p + "o": (d, m.heads * m.vdim)}
+
+
+def _gla_shapes(p: str, m: RecurrentMixer, d: int) -> dict:
+    return {p + "q": (m.heads * m.dim, d), p + "k": (m.heads * m.dim, d), p + "v": (m.heads * m.vdim, d),
+            p + "g": (m.heads * m.vdim, d), p + "o": (d, m.heads * m.vdim), p + "norm": (m.vdim,),
+            p + "a1": (None, d), p + "a2": (m.heads * m.dim, None), p + "a2.b": (m.heads * m.dim,)}
+
+
+def _delta_shapes(p: str, m: RecurrentMixer, d: int) -> dict:
+    cq, cv = m.kv_heads * m.dim, m.heads * m.vdim
+    out = {p + "q": (cq, d), p + "k": (cq, d), p + "v": (cv, d), p + "b": (m.heads, d), p + "A_log": (m.heads,),
+           p + "norm": (m.vdim,), p + "a1": (None, d), p + "a2": (m.heads * m.dim, None),
+           p + "dt_bias": (m.heads * m.dim,), p + "g1": (None, d), p + "g2": (cv, None), p + "o": (d, cv)}
+    out.update({p + "q.conv": (cq, m.conv), p + "k.conv": (cq, m.conv), p + "v.conv": (cv, m.conv)})
+    return out
+
+
+def expected_shapes(cfg: HybridConfig) -> dict:
+    """Name -> shape of every tensor; ``None`` marks a low-rank width that the tensors themselves fix."""
+    d = cfg.hidden_size
+    out = {"embed": (cfg.vocab_size, d), "pos": (cfg.max_seq_len, d), "final.norm": (d,), "head": (cfg.vocab_size, d)}
+    for i, spec in enumerate(cfg.layers):
+        p = f"l{i}."
+        out[p + "norm1"] = out[p + "norm1b"] = (d,)
+        m = spec.mixer
+        if isinstance(m, ParallelMixer):
+            out.update(_attention_shapes(p + "mix.left.", m.left, d))
+            out.update(_delta_shapes(p + "mix.right.", m.right, d))
+            out[p + "mix.left.out"] = out[p + "mix.right.out"] = (d,)
+        else:
+            out.update(_gla_shapes(p + "mix.", m, d))
+        if spec.ff:
+            out[p + "norm2"] = out[p + "norm2b"] = (d,)
+            out.update({p + "mlp.gate": (spec.ff, d), p + "mlp.up": (spec.ff, d), p + "mlp.down": (d, spec.ff)})
+    return out
+
+
+def _key(name: str) -> str:
+    return name.replace(".", "/")
+
+
+class HybridModel(nn.Module):
+    def __init__(self, cfg: HybridConfig, tensors: dict):
+        super().__init__()
+        self.cfg = cfg
+        self._engine = None
+        for name, shape in expected_shapes(cfg).items():
+            if name not in tensors:
+                raise KeyError(f"checkpoint has no tensor {name!r}")
+            t = tensors[name]
+            if t.dim() != len(shape) or any(w is not None and int(w) != n for w, n in zip(shape, t.shape)):
+                raise ValueError(f"tensor {name!r} has shape {tuple(t.shape)}, the configuration wants {shape}")
+            self.register_parameter(_key(name), nn.Parameter(t, requires_grad=False))
+
+    def tensor(self, name: str) -> torch.Tensor:
+        return getattr(self, _key(name)).detach()
+
+    def named_tensors(self):
+        return [(n.replace("/", "."), p.detach()) for n, p in self.named_parameters()]
+
+    @classmethod
+    def random(cls, cfg: HybridConfig, seed: int = 0, device="cpu", dtype=torch.bfloat16, low_rank: int = 16,
+               std: float = 0.02) -> "HybridModel":
+        """Random weights of this configuration (benchmarks, tests)."""
+        g = torch.Generator(device=device).manual_seed(seed)
+        out = {}
+        for name, shape in expected_shapes(cfg).items():
+            shape = tuple(low_rank if n is None else n for n in shape)
+            leaf = name.rsplit(".", 1)[-1]
+            if leaf in ("norm", "norm1", "norm2", "norm1b", "norm2b", "out"):
+                t = torch.ones(shape, device=device)
+            elif leaf == "A_log":
+                t = torch.log(1.0 + 3.0 * torch.rand(shape, device=device, generator=g))
+            elif leaf == "dt_bias":
+                t = -4.0 + torch.rand(shape, device=device, generator=g)
+            elif leaf == "b":
+                t = (torch.rand(shape, device=device, generator=g) * 4 + 1 if len(shape) == 1
+                     else torch.randn(shape, device=device, generator=g) * std)
+            else:
+                t = torch.randn(shape, device=device, generator=g) * (0.5 if leaf == "conv" else std)
+            out[name] = t.to(dtype)
+        return cls(cfg, out)
+
+    def param_count(self) -> int:
+        return sum(p.numel() for p in self.parameters())
+
+    # ------------------------------------------------------------------ whole-sequence forward
+    def engine(self):
+        """Engine behind :meth:`forward` (built on first use, one sequence at a time)."""
+        dev = self.tensor("embed").device
+        if dev.type != "cuda":
+            raise RuntimeError("a layer-list model runs on the GPU only; move it to a CUDA device")
+        if self._engine is None:
+            from ..infer.engine import InferenceEngine
+
+            self._engine = InferenceEngine.from_model(self, device=dev, max_batch=1, max_seq_len=self.cfg.max_seq_len)
+        return self._engine
+
+    def _rows(self, ids, fn):
+        eng = self.engine()
+        out = []
+        for row in torch.as_tensor(ids).tolist():
+            seq = eng.cache.new_sequence()
+            try:
+                out.append(fn(eng, seq, row))
+            finally:
+                eng.release(seq)
+        return torch.stack(out)
+
+    def hidden_states(self, ids, pos=None):
+        """ids int [B, S] -> final normalised hidden states [B, S, d]."""
+        return self._rows(ids, lambda e, s, row: e.step_hidden([s], [row])[0][:, : self.cfg.hidden_size])
+
+    def forward(self, ids, targets=None, pos=None):
+        """Logits [B, S, V] (fp32)."""
+        if targets is not None:
+            raise NotImplementedError("layer-list models are inference only")
+        return self._rows(ids, lambda e, s, row: e.step([s], [row], [list(range(len(row)))]))
+
+    def logits(self, h):
+        return self.engine()._logits(h.reshape(-1, h.shape[-1])).view(*h.shape[:-1], -1)

@@ -48,11 +48,46 @@ def read_safetensors(path: str) -> dict:
     return out
 
 
+def read_safetensors_torch(path: str) -> dict:
+    """``{name: torch tensor}`` in the stored types (BF16, F16, F32, F64 and integer tables)."""
+    import torch
+
+    types = {"BF16": torch.bfloat16, "F16": torch.float16, "F32": torch.float32, "F64": torch.float64,
+             "I64": torch.int64, "I32": torch.int32, "I16": torch.int16, "I8": torch.int8, "U8": torch.uint8,
+             "BOOL": torch.bool}
+    with open(path, "rb") as f:
+        (n,) = struct.unpack("<Q", f.read(8))
+        header = json.loads(f.read(n).decode("utf-8"))
+        base = 8 + n
+        out = {}
+        for name, meta in header.items():
+            if name == "__metadata__":
+                continue
+            lo, hi = meta["data_offsets"]
+            f.seek(base + lo)
+            raw = bytearray(f.read(hi - lo))
+            if meta["dtype"] not in types or len(raw) != hi - lo:
+                raise ValueError(f"{path}: tensor {name!r} is truncated or has an unknown type {meta['dtype']}")
+            dt = types[meta["dtype"]]
+            t = torch.frombuffer(raw, dtype=dt) if raw else torch.empty(0, dtype=dt)
+            out[name] = t.reshape(meta["shape"])
+    return out
+
+
 def write_safetensors(path: str, tensors: dict) -> None:
+    """numpy arrays are stored as F32; torch tensors keep their type (BF16, F32 or I32)."""
+    import torch
+
+    names = {torch.bfloat16: "BF16", torch.float32: "F32", torch.int32: "I32"}
     header, blobs, off = {}, [], 0
     for name, a in tensors.items():
-        b = np.ascontiguousarray(a, dtype="<f4").tobytes()
-        header[name] = {"dtype": "F32", "shape": list(np.shape(a)), "data_offsets": [off, off + len(b)]}
+        if torch.is_tensor(a):
+            t = a.detach().cpu().contiguous()
+            dt, shape = names[t.dtype], list(t.shape)
+            b = t.view(torch.int16).numpy().tobytes() if t.dtype == torch.bfloat16 else t.numpy().tobytes()
+        else:
+            dt, shape, b = "F32", list(np.shape(a)), np.ascontiguousarray(a, dtype="<f4").tobytes()
+        header[name] = {"dtype": dt, "shape": shape, "data_offsets": [off, off + len(b)]}
         blobs.append(b)
         off += len(b)
     hj = json.dumps(header).encode("utf-8")

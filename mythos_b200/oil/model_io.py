@@ -171,8 +171,13 @@ def _assign_linear(mod, rd: OILReader, name: str, reference_layout: bool = False
 
 
 def load_model(path: str, device="cpu", model_cls=None):
-    """Returns ``(model, reader)``. Accepts files written by :func:`save_model` and files written by
+    """Returns ``(model, reader)``. A checkpoint folder (``config.json`` + ``model.safetensors``) gives the
+    model class its configuration names, and no reader. Accepts files written by :func:`save_model` and files written by
     the reference's ``DenseModel::save`` (FP32 blocks, separate q/k/v and gate/up tensors)."""
+    from ..models import registry
+
+    if registry.is_checkpoint_dir(path):
+        return registry.load_checkpoint(path, device), None
     from ..models.dense import DenseModel
     from ..models.layers import OILLinear
 

@@ -16,6 +16,7 @@ import torch
 _lock = threading.Lock()
 _ext = None
 _err: Exception | None = None
+_hybrid = None
 
 
 def _load():
@@ -45,10 +46,29 @@ def require():
     return ext
 
 
+def require_hybrid():
+    """The module with the layer-list model kernels (``mythos_b200._H``), or raise as :func:`require`."""
+    global _hybrid
+    with _lock:
+        if _hybrid is None:
+            try:
+                _hybrid = importlib.import_module("mythos_b200._H")
+            except Exception as e:  # noqa: BLE001
+                raise RuntimeError(f"mythos_b200._H is not built or failed to import ({e!r}). "
+                                   "Build it with `python -m mythos_b200.build`.") from e
+    return _hybrid
+
+
+def require_sampler():
+    """A module with the sampling kernels: the one that is loaded already, else the main library."""
+    return _hybrid if _ext is None and _hybrid is not None else require()
+
+
 def launch_count() -> int:
     """Number of kernels launched by this library in this process (0 if not loaded)."""
     ext = _load()
-    return int(ext.launch_count()) if ext is not None else 0
+    n = int(ext.launch_count()) if ext is not None else 0
+    return n + (int(_hybrid.launch_count()) if _hybrid is not None else 0)
 
 
 _status: dict = {}

@@ -1,0 +1,143 @@
+"""Plain, slow PyTorch statement of the hybrid designs (one function per mechanism, token by token where
+there is a recurrence). It is the yardstick of the hybrid tests and shares no code with the package."""
+import torch
+
+
+def rms(x, eps):
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
+
+
+def rms_norm(x, w, eps):
+    return rms(x, eps) * w
+
+
+def silu(x):
+    return x * torch.sigmoid(x)
+
+
+def softplus(x):
+    return torch.clamp(x, min=0) + torch.log1p(torch.exp(-x.abs()))
+
+
+def causal_attention(q, k, v, scale):
+    """q [T, H, dk]; k [T, G, dk]; v [T, G, dv]; query head h reads key head h // (H / G)."""
+    T, H, _ = q.shape
+    G = k.shape[1]
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for h in range(H):
+        g = h // (H // G)
+        s = (q[:, h] @ k[:, g].T) * scale
+        s = s.masked_fill(torch.triu(torch.ones(T, T, dtype=torch.bool), 1), float("-inf"))
+        s = torch.exp(s - s.max(-1, keepdim=True).values)
+        out[:, h] = (s / s.sum(-1, keepdim=True)) @ v[:, g]
+    return out
+
+
+def short_conv(x, w):
+    """Causal per-channel convolution, last tap = current token. x [T, C], w [C, taps]."""
+    T, C = x.shape
+    taps = w.shape[1]
+    out = torch.zeros_like(x)
+    for t in range(T):
+        for j in range(taps):
+            s = t - (taps - 1 - j)
+            if s >= 0:
+                out[t] += w[:, j] * x[s]
+    return out
+
+
+def unit(x):
+    return x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)
+
+
+def delta_recurrence(q, k, v, g, beta):
+    """q, k, g [T, H, dk]; v [T, H, dv]; beta [T, H] -> [T, H, dv]."""
+    T, H, dk = q.shape
+    S = torch.zeros(H, dk, v.shape[2], dtype=q.dtype)
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for t in range(T):
+        S = g[t][:, :, None] * S
+        u = beta[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", S, k[t]))
+        S = S + k[t][:, :, None] * u[:, None, :]
+        out[t] = torch.einsum("hkv,hk->hv", S, q[t])
+    return out
+
+
+def gla_recurrence(q, k, v, alpha):
+    T, H, dk = q.shape
+    S = torch.zeros(H, dk, v.shape[2], dtype=q.dtype)
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for t in range(T):
+        S = alpha[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        out[t] = torch.einsum("hkv,hk->hv", S, q[t])
+    return out
+
+
+def gated_attention(h, W, p, c, eps):
+    T = h.shape[0]
+    H, G, dk, dv = c["heads"], c["kv_heads"], c["dim"], c["vdim"]
+    q = rms_norm((h @ W[p + "q"].T).view(T, H, dk), W[p + "q.norm"], eps)
+    k = rms_norm((h @ W[p + "k"].T).view(T, G, dk), W[p + "k.norm"], eps)
+    v = (h @ W[p + "v"].T).view(T, G, dv)
+    o = causal_attention(q, k, v, c["scale"])
+    o = o * torch.sigmoid(h @ W[p + "g"].T)[:, :, None]
+    return o.reshape(T, H * dv) @ W[p + "o"].T
+
+
+def gated_delta(h, W, p, c, eps):
+    T = h.shape[0]
+    H, G, dk, dv = c["heads"], c["kv_heads"], c["dim"], c["vdim"]
+    q = silu(short_conv(h @ W[p + "q"].T, W[p + "q.conv"])).view(T, G, dk)
+    k = silu(short_conv(h @ W[p + "k"].T, W[p + "k.conv"])).view(T, G, dk)
+    v = silu(short_conv(h @ W[p + "v"].T, W[p + "v.conv"])).view(T, H, dv)
+    q, k = unit(q) * dk ** -0.5, unit(k)
+    q, k = q.repeat_interleave(H // G, 1), k.repeat_interleave(H // G, 1)
+    beta = torch.sigmoid(h @ W[p + "b"].T)
+    z = (h @ W[p + "a1"].T) @ W[p + "a2"].T + W[p + "dt_bias"]
+    g = torch.exp(-torch.exp(W[p + "A_log"])[None, :, None] * softplus(z).view(T, H, dk))
+    o = delta_recurrence(q, k, v, g, beta)
+    gate = torch.sigmoid((h @ W[p + "g1"].T) @ W[p + "g2"].T).view(T, H, dv)
+    return (rms_norm(o, W[p + "norm"], eps) * gate).reshape(T, H * dv) @ W[p + "o"].T
+
+
+def gla(h, W, p, c, eps):
+    T = h.shape[0]
+    H, dk, dv = c["heads"], c["dim"], c["vdim"]
+    q = (h @ W[p + "q"].T).view(T, H, dk) * dk ** -0.5
+    k = (h @ W[p + "k"].T).view(T, H, dk)
+    v = (h @ W[p + "v"].T).view(T, H, dv)
+    z = (h @ W[p + "a1"].T) @ W[p + "a2"].T + W[p + "a2.b"]
+    alpha = torch.sigmoid(z).pow(1.0 / c["tau"]).view(T, H, dk)
+    o = rms_norm(gla_recurrence(q, k, v, alpha), W[p + "norm"], eps)
+    return (o.reshape(T, H * dv) * silu(h @ W[p + "g"].T)) @ W[p + "o"].T
+
+
+def parallel(h, W, p, c, eps):
+    a = rms_norm(gated_attention(h, W, p + "left.", c["left"], eps), W[p + "left.out"], eps)
+    b = rms_norm(gated_delta(h, W, p + "right.", c["right"], eps), W[p + "right.out"], eps)
+    return 0.5 * (a + b)
+
+
+MIXERS = {"gla": gla, "parallel": parallel}
+
+
+def dense_ff(h, W, p):
+    return (silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
+
+
+def forward(cfg, W, tokens, dtype=torch.float64, trace=None):
+    """Logits [T, vocab] of one sequence; ``trace`` (a list) receives the stream after every layer."""
+    W = {k: v.to(dtype) for k, v in W.items()}
+    eps = cfg["norm"]["eps"]
+    tok = torch.as_tensor(tokens, dtype=torch.long)
+    x = W["embed"][tok] * cfg["embedding"]["scale"] + W["pos"][: tok.numel()]
+    for i, L in enumerate(cfg["layers"]):
+        p = f"l{i}."
+        y = MIXERS[L["type"]](rms_norm(x, W[p + "norm1"], eps), W, p + "mix.", L["mixer"], eps)
+        x = x + rms_norm(y, W[p + "norm1b"], eps)
+        if L["mlp"] is not None:
+            y = dense_ff(rms_norm(x, W[p + "norm2"], eps), W, p + "mlp.")
+            x = x + rms_norm(y, W[p + "norm2b"], eps)
+        if trace is not None:
+            trace.append(x)
+    return rms_norm(x, W["final.norm"], eps) @ W["head"].T * cfg["logit_scale"]
