@@ -27,8 +27,8 @@ CSRC = PKG / "csrc"
 OBJ = PKG / "csrc" / "build"
 
 # Sources of the layer-list model module: those it has to itself, and those it shares with ``_C``.
-HYBRID_ONLY = ["hybrid_ops", "recurrent"]
-HYBRID_SOURCES = HYBRID_ONLY + ["host_util", "gemm", "gemm_2cta", "sampler"]
+HYBRID_ONLY = ["hybrid_ops", "recurrent", "chunk_scan", "gemm_decode"]
+HYBRID_SOURCES = HYBRID_ONLY + ["host_util", "gemm", "gemm_2cta", "sampler", "attention_fwd", "attention_fwd2", "paged_attn"]
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

@@ -795,7 +795,7 @@ void paged_attn_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
   chk_c(counters, I32, "counters");
   const int64_t B = q.size(0), H = q.size(1), D = q.size(2), Hkv = k_cache.size(2);
   TORCH_CHECK(scratch.numel() >= B * H * splits * (D + 2), "paged_attn_decode: scratch too small");
-  TORCH_CHECK(counters.numel() >= B * Hkv, "paged_attn_decode: counters too small");
+  TORCH_CHECK(counters.numel() >= B * Hkv * ((H / Hkv + 7) / 8), "paged_attn_decode: counters too small");
   c10::cuda::CUDAGuard guard(q.device());
   mb::paged_attn_decode(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), block_table.data_ptr<int>(),
                         context_lens.data_ptr<int>(), out.data_ptr(), scratch.data_ptr<float>(),
@@ -826,7 +826,7 @@ void flash_attn_paged_prefill(const Tensor& q, const Tensor& k_cache, const Tens
   mb::flash_attn_paged_prefill(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), (int)k_cache.size(0),
                                block_table.data_ptr<int>(), (int)block_table.size(1), cu_q.data_ptr<int>(),
                                kv_lens.data_ptr<int>(), out.data_ptr(), out.stride(0), (int)B, (int)q.size(0),
-                               (int)max_q_len, (int)q.size(1), (int)k_cache.size(2), (int)q.size(2), (float)scale,
+                               (int)max_q_len, (int)q.size(1), (int)k_cache.size(2), (int)q.size(2), (int)q.size(2), nullptr, 0, (float)scale,
                                status_ptr(status), cur_stream());
 }
 

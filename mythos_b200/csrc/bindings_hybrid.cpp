@@ -124,6 +124,77 @@ void paged_attn_any(const Tensor& q, const Tensor& k_cache, const Tensor& v_cach
                      pg.dk, pg.dv, (float)scale, cur_stream());
 }
 
+// Tensor-core attention over the pages (key and value widths 64 or 128, 16-token pages): prompts and portions.
+void paged_attn_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const std::vector<Tensor>& batch,
+                        const Tensor& table, const OptTensor& gate, Tensor& o, int64_t max_q, double scale,
+                        const OptTensor& status) {
+  const auto rb = ragged(batch);
+  const Pages pg = pages(table, k_cache, v_cache, false, rb.n_seq);
+  chk_c(q, BF16, "q");
+  TORCH_CHECK(q.dim() == 3 && q.size(0) == rb.rows && q.size(2) == pg.dk && pg.page_size == 16, "paged_attn_prefill: q / pages");
+  const int heads = (int)q.size(1);
+  chk_rows(o, false, rb.rows, (int64_t)heads * pg.dv, "o");
+  if (gate.has_value()) chk_rows(*gate, false, rb.rows, heads, "gate");
+  c10::cuda::CUDAGuard guard(q.device());
+  mb::flash_attn_paged_prefill(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), (int)k_cache.size(0),
+                               pg.table, pg.stride, rb.cu_q, rb.kv_lens, o.data_ptr(), o.stride(0), rb.n_seq, rb.rows,
+                               (int)max_q, heads, pg.kv_heads, pg.dk, pg.dv, cptr(gate),
+                               gate.has_value() ? gate->stride(0) : 0, (float)scale, status_ptr(status), cur_stream());
+}
+
+// One token per sequence, split over the context.
+void paged_attn_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const std::vector<Tensor>& batch,
+                       const Tensor& table, const OptTensor& gate, Tensor& o, Tensor& scratch, Tensor& counters,
+                       int64_t splits, double scale, const OptTensor& status) {
+  const auto rb = ragged(batch);
+  const Pages pg = pages(table, k_cache, v_cache, false, rb.n_seq);
+  chk_c(q, BF16, "q");
+  TORCH_CHECK(q.dim() == 3 && q.size(0) == rb.rows && q.size(2) == pg.dk && rb.rows == rb.n_seq && pg.page_size == 16,
+              "paged_attn_decode: q / pages");
+  const int heads = (int)q.size(1);
+  chk_c(o, BF16, "o");
+  TORCH_CHECK(o.numel() == (int64_t)rb.rows * heads * pg.dv, "paged_attn_decode: o");
+  chk_c(scratch, F32, "scratch");
+  chk_c(counters, I32, "counters");
+  TORCH_CHECK(scratch.numel() >= (int64_t)rb.rows * heads * splits * (pg.dv + 2) &&
+                  counters.numel() >= (int64_t)rb.rows * pg.kv_heads * ((heads / pg.kv_heads + 7) / 8),
+              "paged_attn_decode: scratch");
+  if (gate.has_value()) chk_rows(*gate, false, rb.rows, heads, "gate");
+  c10::cuda::CUDAGuard guard(q.device());
+  mb::paged_attn_decode(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), pg.table, rb.kv_lens, o.data_ptr(),
+                        scratch.data_ptr<float>(), counters.data_ptr<int>(), rb.n_seq, heads, pg.kv_heads, pg.dk, 16,
+                        pg.stride, (int)k_cache.size(0), (int)splits, (float)scale, status_ptr(status), cur_stream(),
+                        q.stride(0), pg.dv, cptr(gate), gate.has_value() ? gate->stride(0) : 0);
+}
+
+// Few-token GEMM: out = alpha * x w^T, or with f > 0 silu(x w[:f]^T) * (x w[f_off : f_off + f]^T).
+void gemm_decode(const Tensor& x, const Tensor& w, Tensor& out, int64_t f, int64_t f_off, double alpha,
+                 const OptTensor& status) {
+  chk(x, BF16, "x");
+  chk(w, BF16, "w");
+  const bool of32 = is_f32(out, "out");
+  TORCH_CHECK(x.dim() == 2 && w.dim() == 2 && out.dim() == 2 && x.stride(1) == 1 && w.stride(1) == 1 && out.stride(1) == 1 &&
+                  x.size(1) == w.size(1), "gemm_decode: operands");
+  const int64_t n = f > 0 ? f : w.size(0);
+  TORCH_CHECK(out.size(0) == x.size(0) && out.size(1) >= n && (f == 0 || f_off + f <= w.size(0)), "gemm_decode: shapes");
+  c10::cuda::CUDAGuard guard(x.device());
+  mb::gemm_decode(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), of32, out.stride(0),
+                  (int)x.size(0), (int)n, (int)x.size(1), f > 0 ? (int)f_off : 0, (float)alpha, status_ptr(status),
+                  cur_stream());
+}
+
+// h = silu(x w[:f]^T) * (x w[f:2f]^T) in the GEMM's epilogue (prompt-sized batches, f a multiple of 128).
+void gemm_swiglu(const Tensor& x, const Tensor& w, Tensor& h, const OptTensor& status) {
+  chk(x, BF16, "x");
+  chk(w, BF16, "w");
+  chk(h, BF16, "h");
+  TORCH_CHECK(x.dim() == 2 && w.dim() == 2 && h.dim() == 2 && x.stride(1) == 1 && w.stride(1) == 1 && h.stride(1) == 1 &&
+                  x.size(1) == w.size(1) && h.size(0) == x.size(0) && h.size(1) * 2 == w.size(0), "gemm_swiglu: shapes");
+  c10::cuda::CUDAGuard guard(x.device());
+  mb::gemm_swiglu_fwd(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), nullptr, 0, h.data_ptr(), h.stride(0),
+                      (int)x.size(0), (int)h.size(1), (int)x.size(1), status_ptr(status), cur_stream());
+}
+
 // out = alpha * a b^T; bf16 operands run the tcgen05 GEMM (bf16 or fp32 output), fp32 operands the fp32 kernel.
 void gemm_nt(const Tensor& a, const Tensor& b, Tensor& out, double alpha, const OptTensor& status) {
   const bool f32 = is_f32(a, "a");
@@ -216,6 +287,50 @@ struct Recurrent {
     mb::recurrent_scan_seq(f32, s, in, rb, scratch.data_ptr<float>(), o.data_ptr<float>(), cur_stream());
     mb::conv_state_update(f32, s, in, rb, cur_stream());
   }
+  bool chunked_ok() const { return mb::recurrent_chunked_ok(s); }
+  int64_t chunked_scratch(int64_t rows, int64_t n_seq) const {
+    return mb::recurrent_chunked_scratch(s, (int)rows, (int)n_seq);
+  }
+  void scan_chunked(const Tensor& proj, const Tensor& z, const std::vector<Tensor>& batch, Tensor& scratch, Tensor& o,
+                    const OptTensor& status) {
+    const auto rb = ragged(batch);
+    chk(proj, BF16, "proj");
+    chk_c(scratch, U8, "scratch");
+    chk_c(o, F32, "o");
+    TORCH_CHECK(scratch.numel() >= chunked_scratch(rb.rows, rb.n_seq) &&
+                    o.numel() >= (int64_t)rb.rows * s.heads * s.vdim, "scan_chunked: buffers");
+    const auto in = inputs(proj, z, rb.rows);
+    c10::cuda::CUDAGuard guard(proj.device());
+    mb::recurrent_scan_chunked(s, in, rb, scratch.data_ptr(), o.data_ptr<float>(), status_ptr(status), cur_stream());
+    mb::conv_state_update(false, s, in, rb, cur_stream());
+  }
+  // One token per sequence in one launch; z / gate null: computed from the columns a_off / g_off of proj.
+  void decode(const Tensor& proj, const OptTensor& z, const OptTensor& gate, int64_t a_off, int64_t g_off,
+              const std::vector<Tensor>& batch, Tensor& out) {
+    const auto rb = ragged(batch);
+    const bool f32 = is_f32(out, "out");
+    const int64_t cv = (int64_t)s.heads * s.vdim;
+    chk_rows(out, f32, rb.rows, cv, "out");
+    TORCH_CHECK(out.stride(0) == out.size(1), "decode: out must be contiguous");
+    auto map = [&](const OptTensor& w, int64_t off, int64_t outputs, const char* name) {
+      mb::DecodeLowRank m{};
+      if (!w.has_value()) return m;
+      chk_c(*w, f32 ? F32 : BF16, name);
+      TORCH_CHECK(w->dim() == 2 && w->size(0) == outputs && off + w->size(1) <= proj.size(1), name);
+      m.w = w->data_ptr();
+      m.ld = w->stride(0);
+      m.off = (int)off;
+      m.rank = (int)w->size(1);
+      return m;
+    };
+    const auto ma = z.has_value() ? mb::DecodeLowRank{} : map(a2, a_off, (int64_t)s.heads * s.dim, "a2");
+    const auto mg = gate.has_value() ? mb::DecodeLowRank{} : map(g2, g_off, cv, "g2");
+    if (gate.has_value()) chk_rows(*gate, f32, rb.rows, cv, "gate");
+    const auto in = inputs(proj, z, rb.rows);
+    c10::cuda::CUDAGuard guard(out.device());
+    mb::recurrent_decode(f32, s, in, rb, ma, mg, fptr(gamma, s.vdim, "gamma"), cptr(gate),
+                         gate.has_value() ? gate->stride(0) : 0, out.data_ptr(), out.stride(0), cur_stream());
+  }
   void norm_gate(const Tensor& o, const Tensor& gate, Tensor& out) {
     const bool f32 = is_f32(out, "out");
     const int64_t rows = out.size(0), cv = (int64_t)s.heads * s.vdim;
@@ -238,6 +353,10 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("sandwich_norm", &sandwich_norm);
   m.def("qk_norm_append", &qk_norm_append);
   m.def("paged_attn_any", &paged_attn_any);
+  m.def("paged_attn_prefill", &paged_attn_prefill);
+  m.def("paged_attn_decode", &paged_attn_decode);
+  m.def("gemm_decode", &gemm_decode);
+  m.def("gemm_swiglu", &gemm_swiglu);
   m.def("gemm_nt", &gemm_nt);
   m.def("silu_gate", &silu_gate);
   m.def("sample_tokens", &sample_tokens);
@@ -278,6 +397,10 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         return r;
       }))
       .def("scan_seq", &Recurrent::scan_seq)
+      .def("chunked_ok", &Recurrent::chunked_ok)
+      .def("chunked_scratch", &Recurrent::chunked_scratch)
+      .def("scan_chunked", &Recurrent::scan_chunked)
+      .def("decode", &Recurrent::decode)
       .def("norm_gate", &Recurrent::norm_gate);
   m.def("launch_count", []() { return (int64_t)mb::launch_counter().load(); });
 }

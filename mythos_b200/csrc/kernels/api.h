@@ -175,7 +175,8 @@ int get_attn_fwd_mode();
 void flash_attn_paged_prefill(const void* q, long long q_tok_stride, const void* k_cache, const void* v_cache,
                               int n_pages, const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
                               void* o, long long o_tok_stride, int batch, int total_q, int max_q_len, int heads,
-                              int kv_heads, int head_dim, float scale, int* status, cudaStream_t stream);
+                              int kv_heads, int dk, int dv, const void* gate, long long ld_gate, float scale, int* status,
+                              cudaStream_t stream);   // gate: optional per-head output gate logits [total_q, heads]
 void flash_attn_bwd(const void* q, const void* k, const void* v, const void* o, const void* dout, const float* lse,
                     void* dq, void* dk, void* dv, float* dq_accum, float* delta, int batch, int seq, int heads,
                     int kv_heads, int head_dim, bool causal, float scale, int* status, cudaStream_t stream);
@@ -324,11 +325,14 @@ void kv_append(const void* k, const void* v, void* k_cache, void* v_cache, const
                const int* positions, const int* seq_ids, int tokens, int kv_heads, int head_dim, int page_size,
                int max_pages, long long kv_tok_stride, cudaStream_t stream);
 // One query token per sequence: q [batch, heads, head_dim]; context_lens [batch]. Split-KV flash
-// decoding: partials in `scratch` (>= batch*heads*splits*(head_dim+2) floats), combined in-kernel.
+// decoding: partials in `scratch` (>= batch*heads*splits*(value width+2) floats), combined in-kernel.
+// v_head_dim: value width (0: = head_dim); gate: optional per-head output gate logits [batch, heads], row
+// stride ld_gate. `counters`: one per (sequence, kv head, sub-group of 8 query heads).
 void paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                        const int* context_lens, void* out, float* scratch, int* counters, int batch, int heads,
                        int kv_heads, int head_dim, int page_size, int max_pages, int cache_pages, int splits,
-                       float scale, int* status, cudaStream_t stream, long long q_tok_stride = 0);
+                       float scale, int* status, cudaStream_t stream, long long q_tok_stride = 0, int v_head_dim = 0,
+                       const void* gate = nullptr, long long ld_gate = 0);
 // int8 pages: k_cache / v_cache [num_pages, page_size, kv_heads, head_dim] int8 with one fp32 scale
 // (max|x| / 127) per (token, kv head) in k_scale / v_scale [num_pages * page_size, kv_heads].
 void kv_append_int8(const void* k, const void* v, void* k_cache, void* v_cache, float* k_scale, float* v_scale,

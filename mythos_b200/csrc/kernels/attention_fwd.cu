@@ -23,11 +23,13 @@ constexpr int FA_BM = 128;  // query rows per tile (two tiles per CTA)
 constexpr int FA_BN = 64;   // kv rows per step
 constexpr int FA_STAGES = 3;
 
-template <int D>
+// DK: width of queries and keys, DV: width of values and outputs.
+template <int DK, int DV>
 struct FaFwdCfg {
-  static constexpr int Q_BYTES = FA_BM * D * 2;
-  static constexpr int KV_BYTES = FA_BN * D * 2;
-  static constexpr int STAGE_BYTES = 2 * KV_BYTES;
+  static constexpr int Q_BYTES = FA_BM * DK * 2;
+  static constexpr int K_BYTES = FA_BN * DK * 2;
+  static constexpr int V_BYTES = FA_BN * DV * 2;
+  static constexpr int STAGE_BYTES = K_BYTES + V_BYTES;
   static constexpr int P_BYTES = FA_BM * FA_BN * 2;
   static constexpr int OFF_Q = 0;
   static constexpr int OFF_KV = 2 * Q_BYTES;
@@ -35,9 +37,9 @@ struct FaFwdCfg {
   static constexpr int OFF_BAR = OFF_P + 2 * P_BYTES;
   static constexpr int NUM_BARS = 1 + 2 * FA_STAGES + 6;
   static constexpr int SMEM_BYTES = OFF_BAR + NUM_BARS * 8 + 16 + 1024;
-  static constexpr int TMEM_COLS = (D == 128) ? 512 : 256;
+  static constexpr int TMEM_COLS = (DV == 128) ? 512 : 256;
   static constexpr int COL_S = 0;    // S0 at 0, S1 at 64
-  static constexpr int COL_O = 128;  // O0 at 128, O1 at 128 + D
+  static constexpr int COL_O = 128;  // O0 at 128, O1 at 128 + DV
 };
 
 // PAGED: prefill attention whose K/V live in the paged cache. Queries are the new tokens of each
@@ -51,17 +53,19 @@ struct PagedPrefillArgs {
   const int* cu_q;          // [batch + 1] first query row of every sequence
   const int* kv_lens;       // [batch] keys visible to the LAST query of the sequence (prefix + new tokens)
   int table_stride;
+  const __nv_bfloat16* gate;   // [total_q, >= heads] logits of a per-head output gate (sigmoid), or null
+  long long ld_gate;
 };
 constexpr int FA_PAGE = 16;
 
-template <int D, bool PAGED>
+template <int DK, int DV, bool PAGED>
 __global__ void __launch_bounds__(FA_THREADS, 1)
 fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
               const __grid_constant__ CUtensorMap tm_v, __nv_bfloat16* __restrict__ o, float* __restrict__ lse,
               int seq, int heads, int kv_heads, long long o_tok_stride, int causal, float scale_log2, int* status,
               PagedPrefillArgs pa) {
-  using Cfg = FaFwdCfg<D>;
-  constexpr int DC = D / 64;  // 64-wide chunks of head_dim
+  using Cfg = FaFwdCfg<DK, DV>;
+  constexpr int DCK = DK / 64, DCV = DV / 64;  // 64-wide chunks of the head widths
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Cfg::OFF_BAR);
@@ -128,7 +132,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
     if (lane == 0) {
       mbar_arrive_expect_tx(q_full, 2 * Cfg::Q_BYTES);
       for (int t = 0; t < 2; ++t)
-        for (int c = 0; c < DC; ++c)
+        for (int c = 0; c < DCK; ++c)
           tma_load_4d(smem + Cfg::OFF_Q + t * Cfg::Q_BYTES + c * (FA_BM * 128), &tm_q, q_full, c * 64, h,
                       q_row0 + q0 + t * FA_BM, PAGED ? 0 : b);
       for (int j = 0; j < Jmax; ++j) {
@@ -137,7 +141,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
         if (!mbar_wait(&kv_empty[st], ph ^ 1, abort_flag, status, 11)) break;
         mbar_arrive_expect_tx(&kv_full[st], Cfg::STAGE_BYTES);
         uint8_t* sk = smem + Cfg::OFF_KV + st * Cfg::STAGE_BYTES;
-        uint8_t* sv = sk + Cfg::KV_BYTES;
+        uint8_t* sv = sk + Cfg::K_BYTES;
         if constexpr (PAGED) {
           // four pages of 16 tokens per kv tile; pages past the sequence's end (never visible: the
           // causal limit masks them) read page 0 so that the transaction count stays fixed
@@ -147,16 +151,16 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
             const int lp = j * (FA_BN / FA_PAGE) + p;
             int page = (lp * FA_PAGE < kv_len && lp < pa.table_stride) ? row[lp] : 0;
             if (page < 0) page = 0;
-            for (int c = 0; c < DC; ++c) {
+            for (int c = 0; c < DCK; ++c)
               tma_load_4d(sk + c * (FA_BN * 128) + p * (FA_PAGE * 128), &tm_k, &kv_full[st], c * 64, hkv, 0, page);
+            for (int c = 0; c < DCV; ++c)
               tma_load_4d(sv + c * (FA_BN * 128) + p * (FA_PAGE * 128), &tm_v, &kv_full[st], c * 64, hkv, 0, page);
-            }
           }
         } else {
-          for (int c = 0; c < DC; ++c) {
+          for (int c = 0; c < DCK; ++c)
             tma_load_4d(sk + c * (FA_BN * 128), &tm_k, &kv_full[st], c * 64, hkv, j * FA_BN, b);
+          for (int c = 0; c < DCV; ++c)
             tma_load_4d(sv + c * (FA_BN * 128), &tm_v, &kv_full[st], c * 64, hkv, j * FA_BN, b);
-          }
         }
       }
     }
@@ -164,7 +168,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
     // ------------------------------------------------------------------ MMA issuer
     if (lane == 0) {
       constexpr uint32_t IDESC_S = umma_idesc_bf16(FA_BM, FA_BN, false, false);
-      constexpr uint32_t IDESC_O = umma_idesc_bf16(FA_BM, D, false, true);
+      constexpr uint32_t IDESC_O = umma_idesc_bf16(FA_BM, DV, false, true);
       const uint32_t q_addr = smem_u32(smem + Cfg::OFF_Q);
       const uint32_t kv_addr = smem_u32(smem + Cfg::OFF_KV);
       const uint32_t p_addr = smem_u32(smem + Cfg::OFF_P);
@@ -172,7 +176,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
         const uint32_t qa = q_addr + t * Cfg::Q_BYTES;
         const uint32_t ka = kv_addr + (j % FA_STAGES) * Cfg::STAGE_BYTES;
 #pragma unroll
-        for (int k = 0; k < D / 16; ++k) {
+        for (int k = 0; k < DK / 16; ++k) {
           const int c = k >> 2, kk = k & 3;
           umma_f16(tmem_base + Cfg::COL_S + t * FA_BN, umma_desc_sw128(qa + c * (FA_BM * 128) + kk * 32, 0, 1024),
                    umma_desc_sw128(ka + c * (FA_BN * 128) + kk * 32, 0, 1024), IDESC_S, k > 0 ? 1u : 0u);
@@ -181,10 +185,10 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       };
       auto issue_pv = [&](int t, int j) {
         const uint32_t pa = p_addr + t * Cfg::P_BYTES;
-        const uint32_t va = kv_addr + (j % FA_STAGES) * Cfg::STAGE_BYTES + Cfg::KV_BYTES;
+        const uint32_t va = kv_addr + (j % FA_STAGES) * Cfg::STAGE_BYTES + Cfg::K_BYTES;
 #pragma unroll
         for (int k = 0; k < FA_BN / 16; ++k) {
-          umma_f16(tmem_base + Cfg::COL_O + t * D, umma_desc_sw128(pa + k * 32, 0, 1024),
+          umma_f16(tmem_base + Cfg::COL_O + t * DV, umma_desc_sw128(pa + k * 32, 0, 1024),
                    umma_desc_sw128(va + k * 2048, FA_BN * 128, 1024), IDESC_O, (j > 0 || k > 0) ? 1u : 0u);
         }
         umma_commit(&o_done[t]);
@@ -226,7 +230,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
     const int q_row = q0 + t * FA_BM + r;      // row within the sequence's queries
     const uint32_t lane_sel = (uint32_t)(quarter * 32) << 16;
     const uint32_t t_s = tmem_base + Cfg::COL_S + t * FA_BN + lane_sel;
-    const uint32_t t_o = tmem_base + Cfg::COL_O + t * D + lane_sel;
+    const uint32_t t_o = tmem_base + Cfg::COL_O + t * DV + lane_sel;
     uint8_t* p_tile = smem + Cfg::OFF_P + t * Cfg::P_BYTES;
     float m_ref = 0.f, l = 0.f;
     bool ok = true;
@@ -277,7 +281,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
         tc_fence_after();
         if (__any_sync(0xffffffffu, need)) {
 #pragma unroll 1
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             uint32_t orr[32];
             tmem_ld32(t_o + c * 32, orr);
             tmem_ld_wait();
@@ -306,11 +310,15 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       ok = __all_sync(0xffffffffu, ok);
       if (ok) {
         tc_fence_after();
-        const float inv_l = l > 0.f ? 1.f / l : 0.f;
+        float inv_l = l > 0.f ? 1.f / l : 0.f;
+        if constexpr (PAGED) {
+          if (pa.gate && q_row < q_len)
+            inv_l /= 1.f + expf(-__bfloat162float(pa.gate[(long long)(q_row0 + q_row) * pa.ld_gate + h]));
+        }
         __nv_bfloat16* orow = o + (PAGED ? (long long)(q_row0 + q_row) : (long long)b * seq + q_row) * o_tok_stride +
-                              (long long)h * D;
+                              (long long)h * DV;
 #pragma unroll 1
-        for (int c = 0; c < D / 32; ++c) {
+        for (int c = 0; c < DV / 32; ++c) {
           uint32_t orr[32];
           tmem_ld32(t_o + c * 32, orr);
           tmem_ld_wait();
@@ -380,21 +388,21 @@ void flash_attn_fwd_strided(const void* q, const void* k, const void* v, void* o
   if (head_dim == 128) {
     static bool configured = false;
     if (!configured) {
-      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         FaFwdCfg<128>::SMEM_BYTES));
+      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<128, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         FaFwdCfg<128, 128>::SMEM_BYTES));
       configured = true;
     }
-    fa_fwd_kernel<128, false><<<grid, FA_THREADS, FaFwdCfg<128>::SMEM_BYTES, stream>>>(
+    fa_fwd_kernel<128, 128, false><<<grid, FA_THREADS, FaFwdCfg<128, 128>::SMEM_BYTES, stream>>>(
         tq, tk, tv, (__nv_bfloat16*)o, lse, seq, heads, kv_heads, o_tok_stride, causal ? 1 : 0, scale_log2, status,
         PagedPrefillArgs{});
   } else {
     static bool configured = false;
     if (!configured) {
-      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<64, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         FaFwdCfg<64>::SMEM_BYTES));
+      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<64, 64, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         FaFwdCfg<64, 64>::SMEM_BYTES));
       configured = true;
     }
-    fa_fwd_kernel<64, false><<<grid, FA_THREADS, FaFwdCfg<64>::SMEM_BYTES, stream>>>(
+    fa_fwd_kernel<64, 64, false><<<grid, FA_THREADS, FaFwdCfg<64, 64>::SMEM_BYTES, stream>>>(
         tq, tk, tv, (__nv_bfloat16*)o, lse, seq, heads, kv_heads, o_tok_stride, causal ? 1 : 0, scale_log2, status,
         PagedPrefillArgs{});
   }
@@ -405,44 +413,34 @@ void flash_attn_fwd_strided(const void* q, const void* k, const void* v, void* o
 void flash_attn_paged_prefill(const void* q, long long q_tok_stride, const void* k_cache, const void* v_cache,
                               int n_pages, const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
                               void* o, long long o_tok_stride, int batch, int total_q, int max_q_len, int heads,
-                              int kv_heads, int head_dim, float scale, int* status, cudaStream_t stream) {
-  MB_REQUIRE(head_dim == 64 || head_dim == 128, "flash_attn_paged_prefill: head_dim must be 64 or 128");
+                              int kv_heads, int dk, int dv, const void* gate, long long ld_gate, float scale, int* status,
+                              cudaStream_t stream) {
+  MB_REQUIRE((dk == 64 || dk == 128) && (dv == 64 || dv == 128), "flash_attn_paged_prefill: head widths must be 64 or 128");
   MB_REQUIRE(heads % kv_heads == 0, "flash_attn_paged_prefill: heads must be a multiple of kv_heads");
   MB_REQUIRE(q_tok_stride % 8 == 0 && o_tok_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0,
              "flash_attn_paged_prefill: strides / alignment");
   if (batch == 0 || total_q == 0 || max_q_len == 0) return;
-  const CUtensorMap tq = make_bshd_map(q, 1, total_q, heads, head_dim, q_tok_stride, FA_BM);
-  // pages: [n_pages, 16 tokens, kv_heads, head_dim]; one box = 16 tokens x 64 columns of one head
-  auto page_map = [&](const void* base) {
-    uint64_t dims[4] = {(uint64_t)head_dim, (uint64_t)kv_heads, (uint64_t)FA_PAGE, (uint64_t)n_pages};
-    uint64_t strides[3] = {(uint64_t)head_dim * 2, (uint64_t)kv_heads * head_dim * 2,
-                           (uint64_t)FA_PAGE * kv_heads * head_dim * 2};
+  const CUtensorMap tq = make_bshd_map(q, 1, total_q, heads, dk, q_tok_stride, FA_BM);
+  // pages: [n_pages, 16 tokens, kv_heads, width]; one box = 16 tokens x 64 columns of one head
+  auto page_map = [&](const void* base, int width) {
+    uint64_t dims[4] = {(uint64_t)width, (uint64_t)kv_heads, (uint64_t)FA_PAGE, (uint64_t)n_pages};
+    uint64_t strides[3] = {(uint64_t)width * 2, (uint64_t)kv_heads * width * 2, (uint64_t)FA_PAGE * kv_heads * width * 2};
     uint32_t box[4] = {64, 1, (uint32_t)FA_PAGE, 1};
     return make_tensor_map(base, TmaDType::BF16, 4, dims, strides, box, true);
   };
-  const CUtensorMap tk = page_map(k_cache), tv = page_map(v_cache);
+  const CUtensorMap tk = page_map(k_cache, dk), tv = page_map(v_cache, dv);
   const dim3 grid((max_q_len + 2 * FA_BM - 1) / (2 * FA_BM), heads, batch);
   const float scale_log2 = scale * 1.4426950408889634f;
-  PagedPrefillArgs pa{block_table, cu_q, kv_lens, table_stride};
-  if (head_dim == 128) {
-    static bool configured = false;
-    if (!configured) {
-      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         FaFwdCfg<128>::SMEM_BYTES));
-      configured = true;
-    }
-    fa_fwd_kernel<128, true><<<grid, FA_THREADS, FaFwdCfg<128>::SMEM_BYTES, stream>>>(
-        tq, tk, tv, (__nv_bfloat16*)o, nullptr, total_q, heads, kv_heads, o_tok_stride, 1, scale_log2, status, pa);
-  } else {
-    static bool configured = false;
-    if (!configured) {
-      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<64, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         FaFwdCfg<64>::SMEM_BYTES));
-      configured = true;
-    }
-    fa_fwd_kernel<64, true><<<grid, FA_THREADS, FaFwdCfg<64>::SMEM_BYTES, stream>>>(
-        tq, tk, tv, (__nv_bfloat16*)o, nullptr, total_q, heads, kv_heads, o_tok_stride, 1, scale_log2, status, pa);
-  }
+  PagedPrefillArgs pa{block_table, cu_q, kv_lens, table_stride, (const __nv_bfloat16*)gate, ld_gate};
+  auto go = [&](auto kern, int smem) {
+    MB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    kern<<<grid, FA_THREADS, smem, stream>>>(tq, tk, tv, (__nv_bfloat16*)o, nullptr, total_q, heads, kv_heads,
+                                             o_tok_stride, 1, scale_log2, status, pa);
+  };
+  if (dk == 128 && dv == 128) go(fa_fwd_kernel<128, 128, true>, FaFwdCfg<128, 128>::SMEM_BYTES);
+  else if (dk == 64 && dv == 128) go(fa_fwd_kernel<64, 128, true>, FaFwdCfg<64, 128>::SMEM_BYTES);
+  else if (dk == 128 && dv == 64) go(fa_fwd_kernel<128, 64, true>, FaFwdCfg<128, 64>::SMEM_BYTES);
+  else go(fa_fwd_kernel<64, 64, true>, FaFwdCfg<64, 64>::SMEM_BYTES);
   count_launch();
   check_launch();
 }

@@ -44,6 +44,11 @@ void paged_attn_any(bool f32, const void* q, const void* k_cache, const void* v_
 void gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N,
               int K, float alpha, cudaStream_t stream);
 
+// y = alpha * x W^T for a few tokens (bf16 in, bf16 or fp32 out), reduction split over a cluster. f_off > 0: W holds
+// a gate matrix in rows [0, N) and an up matrix from row f_off; y = silu(gate) * up.
+void gemm_decode(const void* x, long long ldx, const void* W, long long ldw, void* out, bool out_f32, long long ldo, int M,
+                 int N, int K, int f_off, float alpha, int* status, cudaStream_t stream);
+
 // h = silu(gu[:, :f]) * gu[:, f_off : f_off + f]
 void silu_gate(bool f32, const void* gu, long long ldg, int f, int f_off, void* h, long long ldh, int rows,
                cudaStream_t stream);
@@ -75,6 +80,23 @@ struct RecurrentInputs {
 // floats per row: 2 * kv_heads * dim + heads * (vdim + dim + 1).
 void recurrent_scan_seq(bool f32, const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb,
                         float* scratch, float* o, cudaStream_t stream);
+// Chunked form on tensor cores (bf16 projections, dim <= 128): same result, for prompts and portions.
+bool recurrent_chunked_ok(const RecurrentSpec& s);
+long long recurrent_chunked_scratch(const RecurrentSpec& s, int rows, int n_seq);   // bytes
+void recurrent_scan_chunked(const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb, void* scratch,
+                            float* o, int* status, cudaStream_t stream);
+// One token per sequence (row b belongs to sequence b), everything in one launch: short convolution and its
+// state, norms, decay, state update, read-out, head norm and output gate -> out [rows, ldo]. The decay
+// pre-activations come from in.z, or are computed here from a1 (proj columns) and a2 [heads * dim, ld_a2];
+// the gate comes from `gate`, or from g1 and g2 [heads * vdim, ld_g2].
+struct DecodeLowRank {
+  const void* w;        // [outputs, ld]
+  long long ld;
+  int off, rank;        // columns of proj that hold the inner product
+};
+void recurrent_decode(bool f32, const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb,
+                      const DecodeLowRank& a, const DecodeLowRank& g, const float* gamma, const void* gate,
+                      long long ld_gate, void* out, long long ldo, cudaStream_t stream);
 // Shift the new inputs into the convolution state (after every reader of the old state has run).
 void conv_state_update(bool f32, const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb,
                        cudaStream_t stream);

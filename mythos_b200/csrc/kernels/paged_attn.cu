@@ -109,12 +109,14 @@ __device__ __forceinline__ void unpack8_int8(uint2 w, float (&f)[8]) {
 
 // Merge `nstate` online-softmax states of a CTA (s_m/s_l: [nstate][gstride]; s_acc: state s at
 // s_acc + s * acc_stride, laid out [gstride][D]) for the G heads of one (sequence, kv head), publish the partial result of
-// this split, and let the last CTA of the (sequence, kv head) combine all splits into `out`.
+// this split, and let the last CTA of the (sequence, kv head) combine all splits into `out`. h0: first query
+// head of the group, cidx: its counter. With `gate`, head h is multiplied by sigmoid(gate[b, h]).
 template <int D>
 __device__ __forceinline__ void merge_and_finish(const float* s_m, const float* s_l, const float* s_acc,
                                                  long long acc_stride, int nstate, int gstride, int G, int* s_last, float* __restrict__ scratch,
                                                  int* __restrict__ counters, __nv_bfloat16* __restrict__ out, int b,
-                                                 int hkv, int split, int heads, int kv_heads, int splits) {
+                                                 int h0, int cidx, int split, int heads, int splits,
+                                                 const __nv_bfloat16* __restrict__ gate = nullptr, long long ld_gate = 0) {
   const int stride = D + 2;
   for (int idx = threadIdx.x; idx < G * D; idx += blockDim.x) {
     const int g = idx / D, d = idx % D;
@@ -128,7 +130,7 @@ __device__ __forceinline__ void merge_and_finish(const float* s_m, const float* 
       L += w * s_l[s * gstride + g];
       A += w * s_acc[s * acc_stride + (long long)g * D + d];
     }
-    float* part = scratch + (((long long)b * heads + hkv * G + g) * splits + split) * stride;
+    float* part = scratch + (((long long)b * heads + h0 + g) * splits + split) * stride;
     part[d] = A;
     if (d == 0) {
       part[D] = M;
@@ -139,16 +141,16 @@ __device__ __forceinline__ void merge_and_finish(const float* s_m, const float* 
   __threadfence();
   __syncthreads();
   if (threadIdx.x == 0) {
-    const int prev = atomicAdd(&counters[b * kv_heads + hkv], 1);
+    const int prev = atomicAdd(&counters[cidx], 1);
     *s_last = (prev == splits - 1) ? 1 : 0;
-    if (*s_last) counters[b * kv_heads + hkv] = 0;  // ready for the next launch
+    if (*s_last) counters[cidx] = 0;  // ready for the next launch
   }
   __syncthreads();
   if (!*s_last) return;
   __threadfence();
   for (int idx = threadIdx.x; idx < G * D; idx += blockDim.x) {
     const int g = idx / D, d = idx % D;
-    const float* base = scratch + ((long long)b * heads + hkv * G + g) * splits * stride;
+    const float* base = scratch + ((long long)b * heads + h0 + g) * splits * stride;
     float M = -INFINITY;
     for (int s = 0; s < splits; ++s) M = fmaxf(M, base[s * stride + D]);
     float L = 0.f, A = 0.f;
@@ -159,7 +161,9 @@ __device__ __forceinline__ void merge_and_finish(const float* s_m, const float* 
       L += w * base[s * stride + D + 1];
       A += w * base[s * stride + d];
     }
-    out[((long long)b * heads + hkv * G + g) * D + d] = __float2bfloat16(L > 0.f ? A / L : 0.f);
+    float y = L > 0.f ? A / L : 0.f;
+    if (gate) y /= 1.f + expf(-__bfloat162float(gate[b * ld_gate + h0 + g]));
+    out[((long long)b * heads + h0 + g) * D + d] = __float2bfloat16(y);
   }
 }
 
@@ -279,8 +283,8 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
     for (int i = 0; i < 8; ++i) s_acc[st][g][li * 8 + i] = acc[g][i];
   }
   __syncthreads();
-  merge_and_finish<D>(&s_m[0][0], &s_l[0][0], &s_acc[0][0][0], (long long)G * D, NSTATE, G, G, &s_last, scratch, counters, out, b, hkv,
-                      split, heads, kv_heads, splits);
+  merge_and_finish<D>(&s_m[0][0], &s_l[0][0], &s_acc[0][0][0], (long long)G * D, NSTATE, G, G, &s_last, scratch, counters, out, b, hkv * G,
+                      b * kv_heads + hkv, split, heads, splits);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -309,39 +313,44 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&a
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <int D>
+// DK: width of queries and keys, DV: width of values.
+template <int DK, int DV = DK>
 struct PdSmem {
-  static constexpr int CHUNKS = D / 64;                 // 64-dim boxes per K or V page
+  static constexpr int CHUNKS = DK / 64, VCHUNKS = DV / 64;   // 64-dim boxes per K / V page
   static constexpr int TILE = 16 * 128;                 // one box: 16 tokens x 128 B
-  static constexpr int STAGE = 2 * CHUNKS * TILE;       // K + V
+  static constexpr int STAGE = (CHUNKS + VCHUNKS) * TILE;   // K + V
   static constexpr int WARP_BYTES = PD_STAGES * STAGE;
   static constexpr int OFF_BAR = 4 * WARP_BYTES;
   static constexpr int OFF_MERGE = OFF_BAR + 4 * PD_STAGES * 8 + 16;   // s_m[4][8], s_l[4][8]
   static constexpr int BYTES = OFF_MERGE + 64 * 4 + 1024;
-  static_assert(8 * D * 4 <= WARP_BYTES, "a warp's output state is staged in its own (drained) ring");
+  static_assert(8 * DV * 4 <= WARP_BYTES, "a warp's output state is staged in its own (drained) ring");
 };
 
-template <int D>
+template <int DK, int DV>
 __global__ void __launch_bounds__(128)
 paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                         const __nv_bfloat16* __restrict__ q, const int* __restrict__ block_table,
                         const int* __restrict__ context_lens, __nv_bfloat16* __restrict__ out,
                         float* __restrict__ scratch, int* __restrict__ counters, int heads, int kv_heads, int G,
-                        int max_pages, int splits, float scale_log2, long long q_tok_stride, int* status) {
-  using S = PdSmem<D>;
-  constexpr int KS = D / 16;   // k-steps of Q K^T
-  constexpr int NT = D / 8;    // n-tiles of P V
+                        int max_pages, int splits, float scale_log2, long long q_tok_stride, const __nv_bfloat16* __restrict__ gate,
+                        long long ld_gate, int* status) {
+  using S = PdSmem<DK, DV>;
+  constexpr int KS = DK / 16;   // k-steps of Q K^T
+  constexpr int NT = DV / 8;    // n-tiles of P V
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int b = blockIdx.x, hkv = blockIdx.y, split = blockIdx.z;
+  // grid.y: every kv head, in sub-groups of at most 8 query heads
+  const int subs = (G + 7) >> 3;
+  const int b = blockIdx.x, hkv = blockIdx.y / subs, split = blockIdx.z;
+  const int g0 = (blockIdx.y % subs) * 8, Gs = min(8, G - g0), h0 = hkv * G + g0;
   uint8_t* wsm = smem + warp * S::WARP_BYTES;
   uint64_t* full = reinterpret_cast<uint64_t*>(smem + S::OFF_BAR) + warp * PD_STAGES;
   volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + S::OFF_BAR + 4 * PD_STAGES * 8);
   int* s_last = const_cast<int*>(abort_flag) + 1;
   float* s_m = reinterpret_cast<float*>(smem + S::OFF_MERGE);
   float* s_l = s_m + 32;
-  float* w_acc = reinterpret_cast<float*>(wsm);   // this warp's [8][D] output state, written after its ring drained
+  float* w_acc = reinterpret_cast<float*>(wsm);   // this warp's [8][DV] output state, written after its ring drained
 
   if (threadIdx.x == 0) *abort_flag = 0;
   if (lane == 0) {
@@ -363,10 +372,10 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_c
     uint8_t* dst = wsm + st * S::STAGE;
     mbar_arrive_expect_tx(&full[st], S::STAGE);
 #pragma unroll
-    for (int c = 0; c < S::CHUNKS; ++c) {
-      tma_load_2d(dst + c * S::TILE, &tm_k, &full[st], hkv * D + c * 64, page * 16);
-      tma_load_2d(dst + (S::CHUNKS + c) * S::TILE, &tm_v, &full[st], hkv * D + c * 64, page * 16);
-    }
+    for (int c = 0; c < S::CHUNKS; ++c) tma_load_2d(dst + c * S::TILE, &tm_k, &full[st], hkv * DK + c * 64, page * 16);
+#pragma unroll
+    for (int c = 0; c < S::VCHUNKS; ++c)
+      tma_load_2d(dst + (S::CHUNKS + c) * S::TILE, &tm_v, &full[st], hkv * DV + c * 64, page * 16);
   };
   if (lane == 0)
     for (int i = 0; i < PD_STAGES && i < my_pages; ++i) issue(i);
@@ -377,8 +386,8 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_c
 #pragma unroll
   for (int ks = 0; ks < KS; ++ks) {
     qa[ks][0] = qa[ks][1] = qa[ks][2] = qa[ks][3] = 0u;
-    if (r < G) {
-      const __nv_bfloat16* qp = q + (long long)b * q_tok_stride + (long long)(hkv * G + r) * D + ks * 16 + 2 * t;
+    if (r < Gs) {
+      const __nv_bfloat16* qp = q + (long long)b * q_tok_stride + (long long)(h0 + r) * DK + ks * 16 + 2 * t;
       qa[ks][0] = *reinterpret_cast<const uint32_t*>(qp);
       qa[ks][2] = *reinterpret_cast<const uint32_t*>(qp + 8);
     }
@@ -469,11 +478,11 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_c
   if (ok) {   // every load this warp issued has landed and been consumed
 #pragma unroll
     for (int n = 0; n < NT; ++n)
-      *reinterpret_cast<float2*>(&w_acc[r * D + n * 8 + 2 * t]) = make_float2(o[n][0], o[n][1]);
+      *reinterpret_cast<float2*>(&w_acc[r * DV + n * 8 + 2 * t]) = make_float2(o[n][0], o[n][1]);
   }
   __syncthreads();
-  merge_and_finish<D>(s_m, s_l, reinterpret_cast<const float*>(smem), S::WARP_BYTES / 4, 4, 8, G, s_last, scratch, counters, out, b, hkv, split, heads, kv_heads,
-                      splits);
+  merge_and_finish<DV>(s_m, s_l, reinterpret_cast<const float*>(smem), S::WARP_BYTES / 4, 4, 8, Gs, s_last, scratch, counters, out, b, h0,
+                       b * gridDim.y + blockIdx.y, split, heads, splits, gate, ld_gate);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -700,8 +709,8 @@ paged_decode_mma_int8_kernel(const __grid_constant__ CUtensorMap tm_k, const __g
       *reinterpret_cast<float2*>(&w_acc[r * D + n * 8 + 2 * t]) = make_float2(o[n][0], o[n][1]);
   }
   __syncthreads();
-  merge_and_finish<D>(s_m, s_l, reinterpret_cast<const float*>(smem), S::WARP_BYTES / 4, 4, 8, G, s_last, scratch, counters, out, b, hkv,
-                      split, heads, kv_heads, splits);
+  merge_and_finish<D>(s_m, s_l, reinterpret_cast<const float*>(smem), S::WARP_BYTES / 4, 4, 8, G, s_last, scratch, counters, out, b, hkv * G,
+                      b * kv_heads + hkv, split, heads, splits);
 }
 
 // One warp per output row; x staged in shared memory as fp32.
@@ -755,7 +764,9 @@ void kv_append(const void* k, const void* v, void* k_cache, void* v_cache, const
 void paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                        const int* context_lens, void* out, float* scratch, int* counters, int batch, int heads,
                        int kv_heads, int head_dim, int page_size, int max_pages, int cache_pages, int splits,
-                       float scale, int* status, cudaStream_t stream, long long q_tok_stride) {
+                       float scale, int* status, cudaStream_t stream, long long q_tok_stride, int v_head_dim,
+                       const void* gate, long long ld_gate) {
+  const int dv = v_head_dim > 0 ? v_head_dim : head_dim;
   if (q_tok_stride <= 0) q_tok_stride = (long long)heads * head_dim;
   MB_REQUIRE(q_tok_stride % 8 == 0, "paged_attn_decode: query token stride must be a multiple of 8 elements");
   MB_REQUIRE(heads % kv_heads == 0, "paged_attn_decode: heads must be a multiple of kv_heads");
@@ -764,32 +775,38 @@ void paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, 
   const int G = heads / kv_heads;
   const dim3 grid(batch, kv_heads, splits);
   const float sl2 = scale * 1.4426950408889634f;
-  if (page_size == 16 && G <= 8 && (head_dim == 64 || head_dim == 128)) {
-    // K / V cache as [cache_pages * 16 tokens, kv_heads * head_dim]; one box = 16 tokens x 64 dims
-    uint64_t dims[2] = {(uint64_t)kv_heads * head_dim, (uint64_t)cache_pages * 16};
-    uint64_t strides[1] = {(uint64_t)kv_heads * head_dim * 2};
-    uint32_t box[2] = {64, 16};
-    const CUtensorMap tk = make_tensor_map(k_cache, TmaDType::BF16, 2, dims, strides, box, true);
-    const CUtensorMap tv = make_tensor_map(v_cache, TmaDType::BF16, 2, dims, strides, box, true);
-#define MB_PDM(DD)                                                                                                 \
+  if (page_size == 16 && (head_dim == 64 || head_dim == 128) && (dv == 64 || dv == 128)) {
+    // K / V cache as [cache_pages * 16 tokens, kv_heads * width]; one box = 16 tokens x 64 dims
+    auto page_map = [&](const void* base, int width) {
+      uint64_t dims[2] = {(uint64_t)kv_heads * width, (uint64_t)cache_pages * 16};
+      uint64_t strides[1] = {(uint64_t)kv_heads * width * 2};
+      uint32_t box[2] = {64, 16};
+      return make_tensor_map(base, TmaDType::BF16, 2, dims, strides, box, true);
+    };
+    const CUtensorMap tk = page_map(k_cache, head_dim), tv = page_map(v_cache, dv);
+    const dim3 mgrid(batch, kv_heads * ((G + 7) / 8), splits);
+#define MB_PDM(DD, VV)                                                                                             \
   do {                                                                                                             \
     static bool configured = false;                                                                                \
     if (!configured) {                                                                                             \
-      MB_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_mma_kernel<DD>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
-                                         PdSmem<DD>::BYTES));                                                      \
+      MB_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_mma_kernel<DD, VV>,                                          \
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, PdSmem<DD, VV>::BYTES));     \
       configured = true;                                                                                           \
     }                                                                                                              \
-    paged_decode_mma_kernel<DD><<<grid, 128, PdSmem<DD>::BYTES, stream>>>(                                         \
+    paged_decode_mma_kernel<DD, VV><<<mgrid, 128, PdSmem<DD, VV>::BYTES, stream>>>(                                \
         tk, tv, (const __nv_bfloat16*)q, block_table, context_lens, (__nv_bfloat16*)out, scratch, counters, heads, \
-        kv_heads, G, max_pages, splits, sl2, q_tok_stride, status);                                                              \
+        kv_heads, G, max_pages, splits, sl2, q_tok_stride, (const __nv_bfloat16*)gate, ld_gate, status);           \
   } while (0)
-    if (head_dim == 128) MB_PDM(128);
-    else MB_PDM(64);
+    if (head_dim == 128 && dv == 128) MB_PDM(128, 128);
+    else if (head_dim == 64 && dv == 128) MB_PDM(64, 128);
+    else if (head_dim == 128) MB_PDM(128, 64);
+    else MB_PDM(64, 64);
 #undef MB_PDM
     count_launch();
     check_launch();
     return;
   }
+  MB_REQUIRE(dv == head_dim && gate == nullptr, "paged_attn_decode: unequal widths and gates need 16-token pages");
 #define MB_PD(GG, DD)                                                                                         \
   paged_decode_kernel<GG, DD, false><<<grid, 128, 0, stream>>>(                                               \
       (const __nv_bfloat16*)q, k_cache, v_cache, nullptr, nullptr, block_table, context_lens,                 \

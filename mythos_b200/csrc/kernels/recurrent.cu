@@ -200,6 +200,152 @@ __global__ void head_norm_gate_kernel(RecurrentSpec s, const float* __restrict__
     for (long long i = (long long)s.heads * s.vdim + lane; i < ldo; i += 32) stf(out + t * ldo + i, 0.f);
 }
 
+// sum_r x[r] w[r] of one output channel, x in shared memory (fp32), w a row in the activation type.
+template <typename T>
+__device__ __forceinline__ float low_rank_dot(const float* x, const T* w, int rank) {
+  float a = 0.f;
+  int i = 0;
+  if constexpr (sizeof(T) == 2) {
+    for (; i + 8 <= rank; i += 8) {
+      float f[8];
+      unpack8(ldg8(w, i), f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a = fmaf(f[j], x[i + j], a);
+    }
+  }
+  for (; i < rank; ++i) a = fmaf(ldf(w + i), x[i], a);
+  return a;
+}
+
+// grid (head, sequence), RD_THREADS threads; one token per sequence.
+constexpr int RD_THREADS = 256, RD_R = 4;
+template <typename T, int NI>
+__global__ void __launch_bounds__(RD_THREADS)
+recurrent_decode_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, DecodeLowRank a, DecodeLowRank g2,
+                        const float* __restrict__ gamma, const T* __restrict__ gate, long long ld_gate,
+                        T* __restrict__ out, long long ldo, bool own_conv) {
+  extern __shared__ float sm[];   // q, k, decay [dim]; v, o [vdim]; inner products of the two low-rank maps
+  __shared__ float red[32];
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  constexpr int NW = RD_THREADS / 32;
+  const long long row = b;
+  const int slot = rb.slots[b];
+  const bool fresh = rb.kv_lens[b] <= 1;
+  float *q = sm, *k = q + s.dim, *d = k + s.dim, *v = d + s.dim, *o = v + s.vdim, *xa = o + s.vdim, *xg = xa + a.rank;
+  const int g = h / (s.heads / s.kv_heads), cq = s.kv_heads * s.dim, channels = 2 * cq + s.heads * s.vdim;
+  const T* proj = static_cast<const T*>(in.proj) + row * in.ld;
+  for (int c = tid; c < 2 * s.dim + s.vdim; c += RD_THREADS) {
+    int ch, col;
+    if (c < s.dim) { ch = g * s.dim + c; col = in.q_off + ch; }
+    else if (c < 2 * s.dim) { ch = cq + g * s.dim + c - s.dim; col = in.k_off + ch - cq; }
+    else { ch = 2 * cq + h * s.vdim + c - 2 * s.dim; col = in.v_off + ch - 2 * cq; }
+    float y = ldf(proj + col);
+    if (s.taps > 0) {
+      const float* w = in.conv_w + (long long)ch * s.taps;
+      float acc = w[s.taps - 1] * y, x = y;
+      if (s.taps > 1) {
+        float* st = in.conv_state + (long long)slot * (s.taps - 1) * channels + ch;
+        float nxt = x;                                // newest first: entry j moves to j - 1
+        for (int j = s.taps - 2; j >= 0; --j) {
+          const float old = fresh ? 0.f : st[(long long)j * channels];
+          acc = fmaf(w[j], old, acc);
+          if (own_conv) st[(long long)j * channels] = nxt;
+          nxt = old;
+        }
+      }
+      y = silu_f(acc);
+    }
+    sm[c < 2 * s.dim ? c : c + s.dim] = y;            // q | k, then past the decay: v
+  }
+  if (!in.z)
+    for (int i = tid; i < a.rank; i += RD_THREADS) xa[i] = ldf(proj + a.off + i);
+  if (!gate)
+    for (int i = tid; i < g2.rank; i += RD_THREADS) xg[i] = ldf(proj + g2.off + i);
+  __syncthreads();
+  for (int c = tid; c < s.dim; c += RD_THREADS) {
+    const int ch = h * s.dim + c;
+    const float z = in.z_bias[ch] + (in.z ? in.z[row * in.ldz + ch]
+                                          : low_rank_dot(xa, static_cast<const T*>(a.w) + ch * a.ld, a.rank));
+    d[c] = expf(s.decay_kind == 1 ? -expf(in.a_log[h]) * softplus_f(z) : -softplus_f(-z) * s.inv_tau);
+  }
+  if (warp >= NW - 2) {                               // unit norms on the last two warps
+    float* x = warp == NW - 2 ? q : k;
+    float r = 1.f;
+    if (s.unit_norm) {
+      float ss = 0.f;
+      for (int c = lane; c < s.dim; c += 32) ss += x[c] * x[c];
+      r = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
+    }
+    if (warp == NW - 2) r *= s.q_scale;
+    for (int c = lane; c < s.dim; c += 32) x[c] *= r;
+  }
+  const float beta = s.delta ? sigmoid_f(ldf(proj + in.b_off + h)) : 1.f;
+  __syncthreads();
+  float qr[NI], kr[NI], dr[NI];
+#pragma unroll
+  for (int n = 0; n < NI; ++n) {
+    const int c = lane + 32 * n;
+    const bool ok = c < s.dim;
+    qr[n] = ok ? q[c] : 0.f;
+    kr[n] = ok ? k[c] : 0.f;
+    dr[n] = ok ? d[c] : 0.f;
+  }
+  float* st = in.state + ((long long)slot * s.heads + h) * s.vdim * s.dim;
+  for (int v0 = warp * RD_R; v0 < s.vdim; v0 += NW * RD_R) {
+    float S[RD_R][NI];
+#pragma unroll
+    for (int r = 0; r < RD_R; ++r)
+#pragma unroll
+      for (int n = 0; n < NI; ++n) {
+        const int c = lane + 32 * n;
+        S[r][n] = (!fresh && c < s.dim && v0 + r < s.vdim) ? st[(long long)(v0 + r) * s.dim + c] : 0.f;
+      }
+    float u[RD_R];
+#pragma unroll
+    for (int r = 0; r < RD_R; ++r) {
+      float acc = 0.f;
+#pragma unroll
+      for (int n = 0; n < NI; ++n) {
+        S[r][n] *= dr[n];
+        acc = fmaf(S[r][n], kr[n], acc);
+      }
+      u[r] = v0 + r < s.vdim ? v[v0 + r] : 0.f;
+      if (s.delta) u[r] = beta * (u[r] - warp_sum(acc));
+    }
+#pragma unroll
+    for (int r = 0; r < RD_R; ++r) {
+      float acc = 0.f;
+#pragma unroll
+      for (int n = 0; n < NI; ++n) {
+        S[r][n] = fmaf(kr[n], u[r], S[r][n]);
+        acc = fmaf(S[r][n], qr[n], acc);
+      }
+      acc = warp_sum(acc);
+      if (lane == 0 && v0 + r < s.vdim) o[v0 + r] = acc;
+    }
+#pragma unroll
+    for (int r = 0; r < RD_R; ++r)
+#pragma unroll
+      for (int n = 0; n < NI; ++n) {
+        const int c = lane + 32 * n;
+        if (c < s.dim && v0 + r < s.vdim) st[(long long)(v0 + r) * s.dim + c] = S[r][n];
+      }
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int i = tid; i < s.vdim; i += RD_THREADS) ss += o[i] * o[i];
+  ss = block_sum(ss, red);
+  const float r = 1.f / sqrtf(ss / (float)s.vdim + s.eps);
+  for (int i = tid; i < s.vdim; i += RD_THREADS) {
+    const int ch = h * s.vdim + i;
+    const float z = gate ? ldf(gate + row * ld_gate + ch)
+                         : low_rank_dot(xg, static_cast<const T*>(g2.w) + ch * g2.ld, g2.rank);
+    stf(out + row * ldo + ch, o[i] * r * gamma[i] * (s.gate_kind == 1 ? sigmoid_f(z) : silu_f(z)));
+  }
+  if (h == s.heads - 1)
+    for (long long i = (long long)s.heads * s.vdim + tid; i < ldo; i += RD_THREADS) stf(out + row * ldo + i, 0.f);
+}
+
 PrepOut carve(const RecurrentSpec& s, float* p, long long rows) {
   PrepOut o;
   o.q = p;
@@ -238,6 +384,38 @@ void recurrent_scan_seq(bool f32, const RecurrentSpec& s, const RecurrentInputs&
   else recurrent_scan_seq_kernel<8><<<grid, RS_WARPS * 32, 0, stream>>>(s, rb, p, in.state, o);
   count_launch(2);
   check_launch();
+}
+
+void recurrent_decode(bool f32, const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb,
+                      const DecodeLowRank& a, const DecodeLowRank& g, const float* gamma, const void* gate,
+                      long long ld_gate, void* out, long long ldo, cudaStream_t stream) {
+  check_spec(s);
+  MB_REQUIRE(in.z || a.w, "recurrent_decode: decay pre-activations or their low-rank map");
+  MB_REQUIRE(gate || g.w, "recurrent_decode: output gate or its low-rank map");
+  MB_REQUIRE((!a.w || a.ld % 8 == 0) && (!g.w || g.ld % 8 == 0), "recurrent_decode: low-rank maps need 16-byte rows");
+  if (rb.n_seq == 0) return;
+  MB_REQUIRE(rb.rows == rb.n_seq, "recurrent_decode: one token per sequence");
+  const bool own_conv = s.heads == s.kv_heads;      // otherwise several heads read one channel's convolution state
+  const int smem = (3 * s.dim + 2 * s.vdim + (in.z ? 0 : a.rank) + (gate ? 0 : g.rank)) * 4;
+  MB_REQUIRE(smem <= 48 * 1024, "recurrent_decode: head too wide");
+  DecodeLowRank aa = a, gg = g;
+  if (in.z) aa.rank = 0;
+  if (gate) gg.rank = 0;
+  const dim3 grid(s.heads, rb.n_seq);
+#define MB_RD(T, NI)                                                                                              \
+  recurrent_decode_kernel<T, NI><<<grid, RD_THREADS, smem, stream>>>(s, in, rb, aa, gg, gamma, (const T*)gate, ld_gate, \
+                                                                     (T*)out, ldo, own_conv)
+  if (f32) {
+    if (s.dim <= 32) MB_RD(float, 1); else if (s.dim <= 64) MB_RD(float, 2); else if (s.dim <= 128) MB_RD(float, 4);
+    else MB_RD(float, 8);
+  } else {
+    if (s.dim <= 32) MB_RD(__nv_bfloat16, 1); else if (s.dim <= 64) MB_RD(__nv_bfloat16, 2);
+    else if (s.dim <= 128) MB_RD(__nv_bfloat16, 4); else MB_RD(__nv_bfloat16, 8);
+  }
+#undef MB_RD
+  count_launch();
+  check_launch();
+  if (!own_conv) conv_state_update(f32, s, in, rb, stream);
 }
 
 void conv_state_update(bool f32, const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb,

@@ -695,7 +695,8 @@ class InferenceEngine:
         parts[6].copy_(torch.tensor(seqs, dtype=torch.int32))
         ids, pos, sid, row_seq, cu_q, kv_lens, slots = host.to(dev, non_blocking=True).split([T, T, T, T, n + 1, n, n])
         rows = self.cache.block_table.index_select(0, slots.long()).contiguous()
-        h = self._forward(ids, pos, sid, None, paged=(cu_q, kv_lens, rows, max(lens), slots, row_seq))
+        h = self._forward(ids, pos, sid, None, paged=(cu_q, kv_lens, rows, max(lens), slots, row_seq,
+                                                        max(b + k for b, k in zip(bases, lens))))
         return h, cu
 
     @torch.no_grad()

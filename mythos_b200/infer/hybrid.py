@@ -55,14 +55,23 @@ class _Sublayer:
 
 
 class _Ctx:
-    """One pass: the ragged batch (cu_q, kv_lens, slots, row_seq, pos), its block-table rows and sizes."""
+    """One pass: the ragged batch (cu_q, kv_lens, slots, row_seq, pos), its block-table rows and sizes.
+    ``decode``: one token of every sequence."""
 
-    def __init__(self, batch, table, rows, n_seq, max_q):
-        self.batch, self.table, self.rows, self.n_seq, self.max_q = batch, table, rows, n_seq, max_q
+    def __init__(self, batch, table, rows, n_seq, max_q, max_kv):
+        self.batch, self.table, self.rows, self.n_seq, self.max_q, self.max_kv = batch, table, rows, n_seq, max_q, max_kv
+        self.decode = max_q == 1
+
+
+DECODE_GEMM_ROWS = 128     # up to this many tokens a product goes through the few-token GEMM
+LOW_RANK_FUSE_ROWS = 16    # decode batches up to this size evaluate the low-rank maps inside the recurrence kernel
 
 
 class HybridEngine(InferenceEngine):
     paged_prefill_only = True
+    # False: every step runs the plain any-shape kernels (token-by-token recurrence, scalar attention, one
+    # kernel per step). Same results beyond rounding; for comparison and for 32-bit engines.
+    tensor_kernels = True
 
     def __init__(self, cfg: HybridConfig, device="cuda", max_batch: int = 64, max_seq_len: int | None = None,
                  page_size: int = 16, tp=None, kv_pages: int | None = None, kv_dtype: str | None = None,
@@ -93,6 +102,9 @@ class HybridEngine(InferenceEngine):
         self._sms = torch.cuda.get_device_properties(self.device).multi_processor_count if self.device.type == "cuda" else 1
         self.H = native.require_hybrid() if self.device.type == "cuda" else None
         self._status = native.status_word(self.device)
+        groups = max([m.kv_heads * ((m.heads // m.kv_heads + 7) // 8) for m in att] or [1])
+        self._counters = torch.zeros(max_batch * groups, device=self.device, dtype=torch.int32)
+        self._max_ctx = self.max_seq_len
 
     # ------------------------------------------------------------------ weights
     @classmethod
@@ -160,7 +172,7 @@ class HybridEngine(InferenceEngine):
         L.a2, L.rank = self._matrix(t(p + "a2")), _pad8(t(p + "a1").shape[0])
         off = L.proj.off
         L.rec = self._recurrent(m, {"q": off["q"], "k": off["k"], "v": off["v"]},
-                                {"z_bias": self._vector(t(p + "a2.b")), "gamma": self._vector(t(p + "norm"))})
+                                {"z_bias": self._vector(t(p + "a2.b")), "gamma": self._vector(t(p + "norm")), "a2": L.a2})
         L.out = self._matrix(t(p + "o"))
 
     def _pack_parallel(self, L, t, p: str, att_index: int) -> None:
@@ -177,7 +189,7 @@ class HybridEngine(InferenceEngine):
         L.g2, L.g_rank = self._matrix(t(right + "g2")), _pad8(t(right + "g1").shape[0])
         off = L.proj.off
         tensors = {"z_bias": self._vector(t(right + "dt_bias")), "a_log": self._vector(t(right + "A_log")),
-                   "gamma": self._vector(t(right + "norm"))}
+                   "gamma": self._vector(t(right + "norm")), "a2": L.a2, "g2": L.g2}
         if r.conv > 0:
             tensors["conv_w"] = self._vector(torch.cat([t(right + n + ".conv") for n in ("q", "k", "v")]))
         L.rec = self._recurrent(r, {"q": off["rq"], "k": off["rk"], "v": off["rv"], "b": off["rb"]}, tensors)
@@ -197,25 +209,46 @@ class HybridEngine(InferenceEngine):
     def _gemm(self, x, w, out=None, dtype=None, alpha: float = 1.0):
         if out is None:
             out = self._new(x.shape[0], w.shape[0], dtype)
-        self.H.gemm_nt(x, w, out, alpha, self._status)
+        if self._fast and x.shape[0] <= DECODE_GEMM_ROWS:
+            self.H.gemm_decode(x, w, out, 0, 0, alpha, self._status)
+        else:
+            self.H.gemm_nt(x, w, out, alpha, self._status)
         return out
 
-    def _recurrence(self, L, proj, z, gate, ctx):
-        """Recurrence of a layer over the batch, head norm and output gate -> [rows, pad8(heads * vdim)]."""
-        m = L.spec.recurrent
-        o = torch.empty(ctx.rows, m.heads, m.vdim, device=self.device, dtype=torch.float32)
-        scratch = torch.empty(ctx.rows * (2 * m.kv_heads * m.dim + m.heads * (m.vdim + m.dim + 1)),
-                              device=self.device, dtype=torch.float32)
-        L.rec.scan_seq(proj, z, ctx.batch, scratch, o)
+    @property
+    def _fast(self) -> bool:
+        return self.tensor_kernels and not self.f32
+
+    def _recurrence(self, L, proj, a_off: int, gate, g_off: int, ctx):
+        """Recurrence of a layer over the batch, head norm and output gate -> [rows, pad8(heads * vdim)].
+        ``a_off`` / ``g_off``: columns of ``proj`` with the inner products of the low-rank maps of the decay
+        and (where ``gate`` is None) of the output gate."""
+        m, rec = L.spec.recurrent, L.rec
         out = self._new(ctx.rows, _pad8(m.heads * m.vdim))
-        L.rec.norm_gate(o, gate, out)
+        fuse = ctx.decode and self.tensor_kernels and ctx.rows <= LOW_RANK_FUSE_ROWS
+        z = None
+        if not fuse:
+            z = self._gemm(proj[:, a_off:a_off + L.rank], L.a2, dtype=torch.float32)
+            if gate is None:
+                gate = self._gemm(proj[:, g_off:g_off + L.g_rank], L.g2)
+        if ctx.decode and self.tensor_kernels:
+            rec.decode(proj, z, gate, a_off, g_off, ctx.batch, out)
+            return out
+        o = torch.empty(ctx.rows, m.heads, m.vdim, device=self.device, dtype=torch.float32)
+        if self._fast and rec.chunked_ok():
+            scratch = torch.empty(rec.chunked_scratch(ctx.rows, ctx.n_seq), device=self.device, dtype=torch.uint8)
+            rec.scan_chunked(proj, z, ctx.batch, scratch, o, self._status)
+        else:
+            scratch = torch.empty(ctx.rows * (2 * m.kv_heads * m.dim + m.heads * (m.vdim + m.dim + 1)),
+                                  device=self.device, dtype=torch.float32)
+            rec.scan_seq(proj, z, ctx.batch, scratch, o)
+        rec.norm_gate(o, gate, out)
         return out
 
     def _gla(self, L, h, ctx):
         off = L.proj.off
         proj = self._gemm(h, L.proj.weight)
-        z = self._gemm(proj[:, off["a1"]:off["a1"] + L.rank], L.a2, dtype=torch.float32)
-        y = self._recurrence(L, proj, z, proj[:, off["g"]:], ctx)
+        y = self._recurrence(L, proj, off["a1"], proj[:, off["g"]:], 0, ctx)
         return self._gemm(y, L.out), None
 
     def _attention(self, L, proj, ctx):
@@ -230,22 +263,35 @@ class HybridEngine(InferenceEngine):
         if o.shape[1] != width:
             o[:, width:].zero_()
         gate = proj[:, off["lg"]:off["lg"] + m.heads]
-        self.H.paged_attn_any(q, kc, vc, ctx.batch, ctx.table, gate, o, m.scale)
+        if not (self._fast and self.page_size == 16 and m.dim in (64, 128) and m.vdim in (64, 128)):
+            self.H.paged_attn_any(q, kc, vc, ctx.batch, ctx.table, gate, o, m.scale)
+        elif ctx.decode:
+            pairs = ctx.n_seq * m.kv_heads * ((m.heads // m.kv_heads + 7) // 8)
+            splits = max(1, min(32, (6 * self._sms + pairs - 1) // pairs, (ctx.max_kv + 255) // 256))
+            scratch = torch.empty(ctx.rows * m.heads * splits * (m.vdim + 2), device=self.device, dtype=torch.float32)
+            self.H.paged_attn_decode(q, kc, vc, ctx.batch, ctx.table, gate, o, scratch, self._counters, splits, m.scale,
+                                     self._status)
+        else:
+            self.H.paged_attn_prefill(q, kc, vc, ctx.batch, ctx.table, gate, o, ctx.max_q, m.scale, self._status)
         return o
 
     def _parallel(self, L, h, ctx):
         off = L.proj.off
         proj = self._gemm(h, L.proj.weight)
-        z = self._gemm(proj[:, off["ra1"]:off["ra1"] + L.rank], L.a2, dtype=torch.float32)
-        gate = self._gemm(proj[:, off["rg1"]:off["rg1"] + L.g_rank], L.g2)
-        y_right = self._gemm(self._recurrence(L, proj, z, gate, ctx), L.right_out)
+        y_right = self._gemm(self._recurrence(L, proj, off["ra1"], None, off["rg1"], ctx), L.right_out)
         y_left = self._gemm(self._attention(L, proj, ctx), L.left_out)
         return y_left, y_right
 
     def _feed_forward(self, L, h, ctx):
-        gu = self._gemm(h, L.gate_up.weight)
         f = L.spec.ff
         a = self._new(ctx.rows, L.down.shape[1])
+        if self._fast and f % 8 == 0 and ctx.rows <= DECODE_GEMM_ROWS:
+            self.H.gemm_decode(h, L.gate_up.weight, a, f, L.gate_up.off["up"], 1.0, self._status)
+            return self._gemm(a, L.down)
+        if self._fast and f % 128 == 0 and ctx.rows >= 256:
+            self.H.gemm_swiglu(h, L.gate_up.weight, a, self._status)
+            return self._gemm(a, L.down)
+        gu = self._gemm(h, L.gate_up.weight)
         self.H.silu_gate(gu, f, L.gate_up.off["up"], a)
         return self._gemm(a, L.down)
 
@@ -260,13 +306,13 @@ class HybridEngine(InferenceEngine):
         """``paged`` as in the base class; without it every row is one token of the sequence ``seq_ids[row]``
         with ``ctx_lens[row]`` tokens including it (a decode step)."""
         if paged is not None:
-            cu_q, kv_lens, table, max_q, slots, row_seq = paged
+            cu_q, kv_lens, table, max_q, slots, row_seq, max_kv = paged
         else:
             n = ids.numel()
             cu_q = torch.arange(n + 1, device=self.device, dtype=torch.int32)
-            row_seq, slots, kv_lens, max_q = cu_q[:n], seq_ids, ctx_lens, 1
+            row_seq, slots, kv_lens, max_q, max_kv = cu_q[:n], seq_ids, ctx_lens, 1, self._max_ctx
             table = self.cache.block_table.index_select(0, slots)
-        ctx = _Ctx([cu_q, kv_lens, slots, row_seq, pos], table, ids.numel(), kv_lens.numel(), max_q)
+        ctx = _Ctx([cu_q, kv_lens, slots, row_seq, pos], table, ids.numel(), kv_lens.numel(), max_q, max_kv)
         return self._run_layers(ids, pos, ctx)
 
     def _run_layers(self, ids, pos, ctx, trace=None):

@@ -65,7 +65,7 @@ class RecurrentStatePool:
         return sum(t.numel() * 4 for t in self.tensors)
 
     def save(self, slot: int):
-        return [t[slot].cpu() for t in self.tensors]
+        return [t[slot].to("cpu", copy=True) for t in self.tensors]
 
     def restore(self, slot: int, saved) -> None:
         for t, s in zip(self.tensors, saved):

@@ -167,11 +167,17 @@ class ModelZoo:
         self.loaded = {}
 
     def scan(self) -> dict[str, str]:
+        """Name -> path of the ``.oil`` files and checkpoint folders of the directory."""
+        from ..models.registry import is_checkpoint_dir
+
         out = {}
         if os.path.isdir(self.directory):
             for fn in sorted(os.listdir(self.directory)):
+                path = os.path.join(self.directory, fn)
                 if fn.endswith(".oil"):
-                    out[fn[:-4]] = os.path.join(self.directory, fn)
+                    out[fn[:-4]] = path
+                elif is_checkpoint_dir(path):
+                    out[fn] = path
         return out
 
     def load(self, name: str, device="cpu"):
@@ -238,7 +244,9 @@ class GenerationBackend:
         # that reads slowly stalls only its own request; other requests interleave token by token.
         with self._lock, torch.no_grad():
             dev = next(self.model.parameters()).device
-            engine = self._engine(dev) if (self.use_engine and dev.type == "cuda") else None
+            # layer-list models always run in their engine
+            wants = self.use_engine or getattr(self.model.cfg, "layers", None) is not None
+            engine = self._engine(dev) if (wants and dev.type == "cuda") else None
             room = self.model.cfg.max_seq_len - len(ids)
             kv_seq = None
             logits = None

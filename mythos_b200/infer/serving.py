@@ -90,8 +90,14 @@ class DynamicBatcher:
 
 
 class ContinuousBatcher:
-    def __init__(self, engine, max_batch: int | None = None):
+    def __init__(self, engine, max_batch: int | None = None, chunk_tokens: int | None = None):
+        """``chunk_tokens``: run prompts in portions inside the decode steps. A step is then one engine batch
+        of at most about that many tokens: one token of every running request and, with what is left of
+        the budget, the next portions of the prompts being read (first come, first served). Without it a
+        prompt is prefilled as a whole when its request is admitted."""
         self.engine = engine
+        self.chunk_tokens = chunk_tokens
+        self.prefilling: list[list] = []          # [request, prompt tokens already run]
         self.max_batch = max_batch or engine.max_batch
         self.scheduler = RequestScheduler()
         self.running: list[Request] = []
@@ -119,6 +125,8 @@ class ContinuousBatcher:
     def step(self) -> int:
         """Admit waiting requests, decode one token for every running one. Returns the number of
         tokens produced."""
+        if self.chunk_tokens is not None:
+            return self._step_mixed()
         self._admit()
         live = [r for r in self.running if not self._done(r)]
         produced = 0
@@ -129,6 +137,10 @@ class ContinuousBatcher:
                 r.output.append(tok)
                 self._next_token[r.request_id] = tok
                 produced += 1
+        self._retire()
+        return produced
+
+    def _retire(self) -> None:
         for r in list(self.running):
             if self._done(r):
                 self.engine.release(r.seq)
@@ -136,7 +148,59 @@ class ContinuousBatcher:
                 self.running.remove(r)
                 self.finished.append(r)
                 self._next_token.pop(r.request_id, None)
-        return produced
+
+    def _admit_chunked(self) -> None:
+        """Give waiting requests a sequence slot and all the pages they can need, while there are any."""
+        cache = self.engine.cache
+        while len(self.running) + len(self.prefilling) < self.max_batch and len(self.scheduler):
+            req = self.scheduler.pop()
+            if req is None:
+                break
+            need = len(req.prompt) + req.max_new_tokens
+            pages = (need + cache.page_size - 1) // cache.page_size
+            if pages > len(cache.alloc.free):
+                if not self.running and not self.prefilling:
+                    raise MemoryError(f"request of {need} tokens does not fit the page pool")
+                self.scheduler.push(req)
+                break
+            req.seq = cache.new_sequence()
+            cache.reserve(req.seq, need)
+            self.prefilling.append([req, 0])
+
+    def _step_mixed(self) -> int:
+        self._admit_chunked()
+        live = [r for r in self.running if not self._done(r)]
+        seqs = [r.seq for r in live]
+        lists = [[self._next_token[r.request_id]] for r in live]
+        want = [[0] for _ in live]
+        budget = max(1, self.chunk_tokens - len(live))
+        takers = list(live)
+        for item in self.prefilling:
+            req, done = item
+            part = req.prompt[done:done + budget]
+            if not part:
+                break
+            budget -= len(part)
+            item[1] = done + len(part)
+            seqs.append(req.seq)
+            lists.append(part)
+            complete = item[1] == len(req.prompt)
+            want.append([len(part) - 1] if complete else [])
+            if complete:
+                takers.append(req)
+        if not seqs:
+            return 0
+        logits = self.engine.step(seqs, lists, want)
+        for i, r in enumerate(takers):
+            tok = int(sample(logits[i:i + 1], r.sampler, step=len(r.output))[0])
+            if not r.output:
+                r.first_token_at = time.time()
+                self.running.append(r)
+            r.output.append(tok)
+            self._next_token[r.request_id] = tok
+        self.prefilling = [it for it in self.prefilling if it[1] < len(it[0].prompt)]
+        self._retire()
+        return len(takers)
 
     @staticmethod
     def _done(r: Request) -> bool:
@@ -144,7 +208,7 @@ class ContinuousBatcher:
 
     def run_until_idle(self, max_steps: int = 1 << 20) -> list[Request]:
         for _ in range(max_steps):
-            if not self.running and not len(self.scheduler):
+            if not self.running and not self.prefilling and not len(self.scheduler):
                 break
             self.step()
         return self.finished

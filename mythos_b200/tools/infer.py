@@ -1,4 +1,4 @@
-"""oil-infer: generate text from a ``.oil`` model.
+"""oil-infer: generate text from a ``.oil`` model or a checkpoint folder.
 
 Reference spelling (tools/infer.cpp): ``oil-infer <model.oil> [prompt]`` with temperature 0.7,
 top-k 40, top-p 0.9, 512 tokens, a sibling ``.vocab`` tokenizer (byte tokens without it) and tok/s
@@ -33,7 +33,8 @@ def build_parser():
     ap.add_argument("--gpu", "--device", dest="device", default="auto")
     ap.add_argument("--precision", default="auto", choices=["auto", "fp32", "fp16", "bf16", "int8"],
                     help="int8: int8 KV pages on the GPU engine, int8 activations on the CPU path; the other "
-                         "values keep the engine's bf16 compute (GPU) / fp32 reference ops (CPU)")
+                         "values keep the engine's bf16 compute (GPU) / fp32 reference ops (CPU). Layer-list models: fp32 runs "
+                         "everything in 32-bit floats, other values bf16")
     ap.add_argument("--verbose", action="store_true")
     return ap
 
@@ -48,10 +49,18 @@ def generate_text(model, tokenizer, prompt: str, max_tokens: int, sampler, devic
     if device.type == "cuda":
         from ..infer.engine import InferenceEngine
 
+        from ..models.config import TransformerConfig
+
         S = len(ids)
-        eng = InferenceEngine.from_model(model, device=device, max_batch=1,
-                                         max_seq_len=min(model.cfg.max_seq_len, S + max_tokens) + 16,
-                                         kv_dtype="int8" if precision == "int8" else "bf16")
+        if isinstance(model.cfg, TransformerConfig):
+            kw = {"max_seq_len": min(model.cfg.max_seq_len, S + max_tokens) + 16,
+                  "kv_dtype": "int8" if precision == "int8" else "bf16"}
+        else:
+            if precision == "int8":
+                raise ValueError("int8 pages are not available for layer-list models")
+            kw = {"max_seq_len": min(model.cfg.max_seq_len, S + max_tokens + 16),
+                  "dtype": "float32" if precision == "fp32" else "bfloat16"}
+        eng = InferenceEngine.from_model(model, device=device, max_batch=1, **kw)
         room = eng.max_seq_len - S
         res = eng.generate([ids], max_new_tokens=max(1, min(max_tokens, room)), sampler=sampler,
                            use_graph=sampler.greedy)
@@ -102,7 +111,7 @@ def main(argv=None) -> int:
     device = pick_device(args.device)
     model, _ = load_model(path, device=device)
     model.eval()
-    vocab = (path[:-4] if path.endswith(".oil") else path) + ".vocab"
+    vocab = (path[:-4] if path.endswith(".oil") else path.rstrip("/")) + ".vocab"
     tokenizer = None
     if os.path.exists(vocab):
         tokenizer = BPETokenizer.load(vocab)

@@ -1,4 +1,4 @@
-"""oil-info: describe a ``.oil`` file (header, architecture, tensors with formats, average bits per
+"""oil-info: describe a ``.oil`` file or a checkpoint folder (for the file: header, architecture, tensors with formats, average bits per
 weight, per-format share, codebook bytes). ``oil-info <model.oil>`` as in the reference
 (tools/info.cpp); ``--json`` and ``--verify`` (check the sidecar digests) are additions."""
 from __future__ import annotations
@@ -44,6 +44,21 @@ def describe(path: str) -> dict:
     return info
 
 
+def describe_checkpoint(path: str) -> dict:
+    """Configuration, layer list and tensors of a checkpoint folder (``config.json`` + ``model.safetensors``)."""
+    import os
+
+    from ..models import registry
+    from ..oil.importers import read_safetensors_torch
+
+    arch, cfg = registry.load_config(path)
+    tensors = read_safetensors_torch(os.path.join(path, "model.safetensors"))
+    return {"path": path, "architecture": arch.name, "config": cfg.to_dict(),
+            "params": sum(t.numel() for t in tensors.values()),
+            "tensors": [{"name": n, "shape": list(t.shape), "dtype": str(t.dtype).removeprefix("torch.")}
+                        for n, t in tensors.items()]}
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="oil-info", description=__doc__)
     ap.add_argument("model_pos", nargs="?")
@@ -56,6 +71,19 @@ def main(argv=None) -> int:
     if not path:
         ap.print_usage(sys.stderr)
         return 2
+    from ..models.registry import is_checkpoint_dir
+
+    if is_checkpoint_dir(path):
+        info = describe_checkpoint(path)
+        if a.json:
+            print(json.dumps(info, indent=2))
+            return 0
+        c = info["config"]
+        print(f"{path}: {info['architecture']}, {info['params']:,} parameters in {len(info['tensors'])} tensors, "
+              f"{len(c['layers'])} layers ({', '.join(x['type'] for x in c['layers'])}), width {c['width']}, vocabulary {c['vocab']}")
+        for t in info["tensors"]:
+            print(f"  {t['name']:40s} {str(t['shape']):18s} {t['dtype']}")
+        return 0
     info = describe(path)
     if a.verify:
         from ..oil.container import verify

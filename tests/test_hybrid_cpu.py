@@ -1,0 +1,209 @@
+"""Layer-list models without a GPU: configuration, registry, checkpoint folders, caches with unequal key
+and value widths, request handling of the trace replay, and the sensitivity of the oracle."""
+import json
+import os
+
+import pytest
+import torch
+
+import hybrid_oracle as oracle
+import hybrid_util as hu
+from mythos_b200.infer.kv_paged import PagedKVCache, RecurrentStatePool
+from mythos_b200.models import registry
+from mythos_b200.models.hybrid import HybridModel
+from mythos_b200.models.hybrid_config import HybridConfig, teganex_config
+from mythos_b200.oil.importers import read_safetensors_torch, write_safetensors
+from mythos_b200.oil.model_io import load_model
+
+
+@pytest.mark.parametrize("name", sorted(hu.CONFIGS))
+def test_config_round_trip(name):
+    cfg = HybridConfig.from_dict(hu.CONFIGS[name])
+    assert cfg.to_dict() == hu.CONFIGS[name]
+    assert HybridConfig.from_dict(cfg.to_dict()).to_dict() == cfg.to_dict()
+
+
+@pytest.mark.parametrize("change", [
+    lambda c: c["layers"][0].update(type="other"),
+    lambda c: c["layers"][0]["mixer"].update(heads=0),
+    lambda c: c["layers"][1]["mixer"]["left"].update(kv_heads=4),
+    lambda c: c["layers"][0]["mlp"].update(kind="sparse"),
+    lambda c: c.update(architecture="Unheard"),
+])
+def test_bad_configurations_are_refused(tmp_path, change):
+    raw = json.loads(json.dumps(hu.CONFIGS["ragged"]))
+    change(raw)
+    (tmp_path / "config.json").write_text(json.dumps(raw))
+    with pytest.raises((ValueError, KeyError)):
+        registry.load_config(str(tmp_path))
+
+
+def _write(folder, cfg, w):
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    write_safetensors(os.path.join(folder, "model.safetensors"), w)
+
+
+def test_checkpoint_folder_loads_through_the_registry(tmp_path):
+    cfg = hu.CONFIGS["ragged"]
+    w = hu.weights(cfg, 3)
+    w["table"] = torch.arange(5, dtype=torch.int32)
+    _write(str(tmp_path), cfg, w)
+    back = read_safetensors_torch(str(tmp_path / "model.safetensors"))
+    assert all(back[n].dtype == t.dtype and torch.equal(back[n], t) for n, t in w.items())
+    m, rd = load_model(str(tmp_path))
+    assert rd is None and isinstance(m, HybridModel) and m.cfg.num_layers == len(cfg["layers"])
+    assert torch.equal(m.tensor("l1.mix.right.q.conv"), w["l1.mix.right.q.conv"])
+    with pytest.raises(RuntimeError):
+        m(torch.zeros(1, 4, dtype=torch.int32))           # no CPU forward
+    from mythos_b200.infer.server import ModelZoo
+
+    assert ModelZoo(str(tmp_path.parent)).scan()[tmp_path.name] == str(tmp_path)
+    from mythos_b200.tools.info import main as info_main
+
+    assert info_main([str(tmp_path)]) == 0
+
+
+def test_missing_and_misshapen_tensors_are_refused():
+    cfg = hu.CONFIGS["single"]
+    hc = HybridConfig.from_dict(cfg)
+    w = hu.weights(cfg)
+    short = {k: v for k, v in w.items() if k != "l1.mix.a2.b"}
+    with pytest.raises(KeyError):
+        HybridModel(hc, short)
+    w["l0.mlp.down"] = w["l0.mlp.down"][:, :-1]
+    with pytest.raises(ValueError):
+        HybridModel(hc, w)
+
+
+def test_named_configuration_has_consistent_shapes():
+    cfg = teganex_config(width=256, layers=4, vocab=64, max_positions=32)
+    m = HybridModel.random(cfg, low_rank=8)
+    assert m.param_count() == sum(t.numel() for _, t in m.named_tensors())
+    assert [s.type for s in cfg.layers] == ["gla", "gla", "gla", "parallel"]
+
+
+def test_cache_with_unequal_widths_and_state_slots():
+    states = RecurrentStatePool(3, "cpu")
+    s0 = states.add(2, 4, 5)
+    c = PagedKVCache(2, 0, 0, num_pages=6, page_size=4, max_seqs=3, max_pages_per_seq=4, device="cpu",
+                     layer_shapes=[(1, 8, 16), (2, 4, 8)], states=states)
+    assert c.k[0].shape == (6, 4, 1, 8) and c.v[1].shape == (6, 4, 2, 8)
+    a = c.new_sequence()
+    c.reserve(a, 9)
+    c.advance(a, 9)
+    c.k[1][int(c.block_table_host[a, 2]), 0] = 7.0
+    s0[a] = 3.0
+    toks = list(range(9))
+    c.publish_prefix(a, toks)
+    b = c.new_sequence()
+    assert c.share_prefix(b, toks) == 0                    # pages alone do not determine the states
+    c.free_sequence(b)
+    h = c.offload_sequence(a)
+    assert c.alloc.used == 0
+    s0.zero_()
+    other = c.new_sequence()
+    a2 = c.restore_sequence(h)
+    assert a2 != other and c.lens[a2] == 9 and float(s0[a2].min()) == 3.0
+    assert float(c.k[1][int(c.block_table_host[a2, 2]), 0].min()) == 7.0
+    assert c.size_bytes() == sum(t.numel() * 2 for t in c.k + c.v) + s0.numel() * 4
+
+
+class _FakeEngine:
+    """Counts tokens of every sequence; the logits of a place are its position."""
+
+    def __init__(self, slots=2, pages=8):
+        self.cache = PagedKVCache(1, 1, 1, pages, 4, slots, pages, device="cpu")
+        self.max_batch = slots
+        self.batches = []
+
+    def step(self, seqs, lists, want=None):
+        c = self.cache
+        out = []
+        self.batches.append([len(t) for t in lists])
+        want = want if want is not None else [[len(t) - 1] for t in lists]
+        for s, t, w in zip(seqs, lists, want):
+            c.reserve(s, len(t))
+            for p in w:
+                row = torch.zeros(16)
+                row[(c.lens[s] + p) % 16] = 1.0
+                out.append(row)
+            c.advance(s, len(t))
+        return torch.stack(out) if out else None
+
+    def release(self, s):
+        self.cache.free_sequence(s)
+
+
+def test_trace_replay_admits_continues_and_releases():
+    from mythos_b200.tools.trace_run import TraceReplay
+
+    eng = _FakeEngine()
+    r = TraceReplay(eng)
+    out = r.run({"step": 0, "entries": [{"id": "a", "tokens": [1, 2, 3], "want": [0, 2]},
+                                        {"id": "b", "tokens": [4], "want": []}], "end": []})
+    assert out.argmax(-1).tolist() == [0, 2]
+    assert r.run({"step": 1, "entries": [{"id": "b", "tokens": [5, 6], "want": []}], "end": ["b"]}) is None
+    out = r.run({"step": 2, "entries": [{"id": "c", "tokens": [9, 9], "want": [1]}, {"id": "a", "tokens": [7], "want": [0]}],
+                 "end": ["a", "c"]})
+    assert out.argmax(-1).tolist() == [1, 3] and eng.cache.alloc.used == 0 and not any(eng.cache.active)
+
+
+def test_batcher_mixes_portions_with_decoded_tokens():
+    from mythos_b200.infer.serving import ContinuousBatcher
+
+    eng = _FakeEngine(slots=2, pages=8)
+    cb = ContinuousBatcher(eng, chunk_tokens=4)
+    reqs = [cb.submit([1] * n, max_new_tokens=3) for n in (2, 11, 5)]
+    done = cb.run_until_idle()
+    assert len(done) == 3 and eng.cache.alloc.used == 0
+    for r, n in zip(reqs, (2, 11, 5)):
+        assert r.output == [n - 1, n, n + 1]               # logits named the positions n - 1, n, n + 1
+    assert any(1 in b and max(b) > 1 for b in eng.batches)  # a decoded token beside a portion
+    assert max(sum(b) for b in eng.batches) <= 5
+    with pytest.raises(MemoryError):
+        cb.submit([1] * 100)
+        cb.run_until_idle()
+
+
+# ------------------------------------------------------------------ the oracle notices mistakes
+def _slip(name):
+    """A copy of one mechanism with a mistake in it."""
+    def late_write(q, k, v, g, beta):                      # read-out before the current token's write
+        T, H, dk = q.shape
+        S = torch.zeros(H, dk, v.shape[2], dtype=q.dtype)
+        out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+        for t in range(T):
+            S = g[t][:, :, None] * S
+            out[t] = torch.einsum("hkv,hk->hv", S, q[t])
+            u = beta[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", S, k[t]))
+            S = S + k[t][:, :, None] * u[:, None, :]
+        return out
+
+    def no_decay(q, k, v, alpha):
+        return oracle_gla(q, k, v, torch.ones_like(alpha))
+
+    def shifted_conv(x, w):
+        return oracle_conv(torch.cat([torch.zeros_like(x[:1]), x[:-1]]), w)
+
+    def blind(q, k, v, scale):                             # the newest key is left out
+        T = q.shape[0]
+        keep = oracle_att(q[:-1], k[:-1], v[:-1], scale)
+        return torch.cat([v[:1].repeat_interleave(q.shape[1] // v.shape[1], 1), keep[: T - 1]])
+
+    return {"late_write": ("delta_recurrence", late_write), "no_decay": ("gla_recurrence", no_decay),
+            "shifted_conv": ("short_conv", shifted_conv), "blind": ("causal_attention", blind)}[name]
+
+
+oracle_gla, oracle_conv, oracle_att = oracle.gla_recurrence, oracle.short_conv, oracle.causal_attention
+
+
+@pytest.mark.parametrize("slip", ["late_write", "no_decay", "shifted_conv", "blind"])
+def test_a_mistake_in_a_mechanism_is_larger_than_the_tolerance(slip, monkeypatch):
+    cfg = hu.CONFIGS["ragged"]
+    w, toks = hu.weights(cfg, 5), hu.tokens(cfg, 24)
+    right = oracle.forward(cfg, w, toks)
+    fn, wrong = _slip(slip)
+    monkeypatch.setattr(oracle, fn, wrong)
+    assert hu.rel(oracle.forward(cfg, w, toks), right) > 0.15   # bf16 comparisons allow 0.06
