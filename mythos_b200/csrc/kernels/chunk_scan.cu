@@ -16,14 +16,16 @@
 // the recurrence at 32-bit accuracy although the tensor cores take 16-bit operands: the state, the
 // decays, the unit norms and the chunk matrices never see a plain bf16 rounding.
 //
-// No exponent above is positive. P and A are formed as (q e^{b_t - m}) (k e^{m - b_s}) around the middle
-// m of the chunk's decay, where the factors stay in range; a channel that decays by more than e^-80
-// inside one chunk sends the chunk to a pairwise evaluation instead.
+// No exponent above is positive. P and A are formed as (q e^{b_t}) (k e^{-b_s}), whose second factor grows
+// with the decay inside the chunk: a channel that decays by more than e^-60 in one chunk sends the chunk to
+// a pairwise evaluation instead.
 #include "common.cuh"
 #include "hybrid_api.h"
 #include "hybrid_dev.cuh"
 #include "host_util.h"
 #include "tc.cuh"
+
+#include <type_traits>
 
 namespace mb {
 namespace {
@@ -34,7 +36,7 @@ constexpr int CS_V = 16 * CS_WARPS;
 constexpr int CP_THREADS = 128;
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
                "{%0, %1, %2, %3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
@@ -80,28 +82,115 @@ __device__ __forceinline__ int chunk_base(const int* cu_q, int b) { return cu_q[
 
 using T = __nv_bfloat16;   // projections (32-bit engines use the token-by-token form)
 
-__device__ __forceinline__ float raw_tap(const T* col, long long ld, long long r0, int i, const float* st, int channels,
-                                         int taps, int n) {
-  // input at local token i (i < 0: the convolution state, i >= n: past the end)
-  if (i >= n) return 0.f;
-  if (i >= 0) return ldf(col + (r0 + i) * ld);
-  return st ? st[(long long)(taps - 1 + i) * channels] : 0.f;
+// Activation of the short convolution. The projections are bf16 and the convolution need not be better, so
+// the fast exponential and divide will do here (unlike in the decays).
+__device__ __forceinline__ float conv_act(float y) { return __fdividef(y, 1.f + __expf(-y)); }
+// log(1 + e^x), small arguments of the logarithm from its series
+__device__ __forceinline__ float softplus_fast(float x) {
+  const float e = __expf(-fabsf(x));
+  const float l = e < 0.015625f ? e * (1.f + e * (-0.5f + e * (1.f / 3.f))) : logf(1.f + e);
+  return fmaxf(x, 0.f) + l;
+}
+
+// Input of a channel at local token i < 0: the convolution state, or 0 at a sequence's start.
+__device__ __forceinline__ float conv_past(const float* st, int i, int taps, int channels) {
+  return st && i + taps - 1 >= 0 ? st[(long long)(taps - 1 + i) * channels] : 0.f;
+}
+
+// W adjacent channels (2 when every offset is even, else 1) of the chunk's 16 tokens through the short
+// convolution; `put(t, y)` takes the result. col: the channel's column of the projection; ch: its index.
+template <int W, class Put>
+__device__ __forceinline__ void conv_column(const RecurrentSpec& s, const RecurrentInputs& in, const T* __restrict__ col, int q0,
+                                            int i0, int n, const float* __restrict__ st, int channels, int ch, Put put) {
+  const T* p = col + (long long)(q0 + i0) * in.ld;
+  float x[CK][W];
+#pragma unroll
+  for (int t = 0; t < CK; ++t) {
+    if constexpr (W == 2) {
+      float2 f = make_float2(0.f, 0.f);
+      if (t < n) f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p + t * in.ld));
+      x[t][0] = f.x;
+      x[t][1] = f.y;
+    } else {
+      x[t][0] = t < n ? __bfloat162float(p[t * in.ld]) : 0.f;
+    }
+  }
+  if (s.taps == 0) {
+#pragma unroll
+    for (int t = 0; t < CK; ++t) put(t, x[t]);
+    return;
+  }
+  auto before = [&](int i, int w) {        // input i of the portion
+    return i >= 0 ? __bfloat162float(col[(long long)(q0 + i) * in.ld + w]) : conv_past(st ? st + w : nullptr, i, s.taps, channels);
+  };
+  if (s.taps == 4) {
+    float w4[4][W], h1[W], h2[W], h3[W];
+#pragma unroll
+    for (int w = 0; w < W; ++w) {
+      h3[w] = before(i0 - 3, w);
+      h2[w] = before(i0 - 2, w);
+      h1[w] = before(i0 - 1, w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) w4[j][w] = in.conv_w[(long long)(ch + w) * 4 + j];
+    }
+#pragma unroll
+    for (int t = 0; t < CK; ++t) {
+      float y[W];
+#pragma unroll
+      for (int w = 0; w < W; ++w) {
+        const float a = fmaf(w4[0][w], h3[w], fmaf(w4[1][w], h2[w], fmaf(w4[2][w], h1[w], w4[3][w] * x[t][w])));
+        y[w] = t < n ? conv_act(a) : 0.f;
+        h3[w] = h2[w];
+        h2[w] = h1[w];
+        h1[w] = x[t][w];
+      }
+      put(t, y);
+    }
+  } else {
+    for (int t = 0; t < CK; ++t) {         // any number of taps: inputs are read again
+      float y[W] = {};
+      if (t < n) {
+        for (int w = 0; w < W; ++w) {
+          for (int j = 0; j < s.taps; ++j)
+            y[w] = fmaf(in.conv_w[(long long)(ch + w) * s.taps + s.taps - 1 - j], before(i0 + t - j, w), y[w]);
+          y[w] = conv_act(y[w]);
+        }
+      }
+      put(t, y);
+    }
+  }
 }
 
 template <int DP, bool DELTA>
-__global__ void __launch_bounds__(CP_THREADS)
+struct PrepSmem {
+  using R = Rec<DP, DELTA>;
+  static constexpr int LD = DP + 8;                        // fp32 rows
+  static constexpr int F32 = 3 * CK * LD * 4;              // q, k, running log decay
+  static constexpr int KHAT = R::BYTES;                    // k e^{-b}, head and tail, behind the record image
+  static constexpr int IMG = KHAT + 2 * R::MAT;
+  static constexpr int OFF_MISC = IMG > F32 ? IMG : F32;   // the record image replaces the fp32 rows
+  // norms [32], beta [16], e^{-b_16} [DP], partial P / A [4][512], P / A [512]
+  static constexpr int BYTES = OFF_MISC + (48 + DP + 2048 + 512) * 4;
+};
+
+// One CTA per (chunk, head).
+template <int DP, bool DELTA>
+__global__ void __launch_bounds__(CP_THREADS, 4)
 chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* __restrict__ records,
                   float* __restrict__ vbuf, int vblocks) {
   using R = Rec<DP, DELTA>;
-  constexpr int LD = DP + 1;
-  extern __shared__ float sm[];
-  float* sq = sm;                     // [16][LD]
+  using PS = PrepSmem<DP, DELTA>;
+  constexpr int LD = PS::LD;
+  extern __shared__ __align__(128) uint8_t psm[];
+  float* sq = reinterpret_cast<float*>(psm);     // [16][LD]
   float* sk = sq + CK * LD;
-  float* sb = sk + CK * LD;           // running log decay
-  float* sP = sb + CK * LD;           // [16][16]
+  float* sb = sk + CK * LD;
+  float* s_norm = reinterpret_cast<float*>(psm + PS::OFF_MISC);   // [32] scales of the q and k rows
+  float* sbeta = s_norm + 32;
+  float* s_inv = sbeta + CK;                     // [DP] e^{-b_16}
+  float* part = s_inv + DP;                      // [4 warps][P, A][256]
+  float* sP = part + 2048;                       // [16][16]
   float* sA = sP + 256;
-  float* sbeta = sA + 256;            // [16]
-  float* part = sbeta + CK;           // [warps][2][256] partial P and A
   const int slot = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   int b = 0;
   {
@@ -121,56 +210,39 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
   const int g = h / (s.heads / s.kv_heads);
   const int cq = s.kv_heads * s.dim, channels = 2 * cq + s.heads * s.vdim;
   const T* proj = static_cast<const T*>(in.proj);
-  // ---- q, k, v: short convolution + silu, channel by channel
-  const int tasks = 2 * s.dim + s.vdim;
+  const float* st = (has_state && s.taps > 1) ? in.conv_state + (long long)rb.slots[b] * (s.taps - 1) * channels : nullptr;
+  // ---- q, k, v: short convolution + silu
   float* vrow = vbuf + ((long long)slot * s.heads + h) * vblocks * (CK * CS_V);
-  for (int c = tid; c < tasks; c += CP_THREADS) {
-    int ch, col;                                           // channel within q | k | v, column of the projection
-    if (c < s.dim) { ch = g * s.dim + c; col = in.q_off + ch; }
-    else if (c < 2 * s.dim) { ch = cq + g * s.dim + c - s.dim; col = in.k_off + ch - cq; }
-    else { ch = 2 * cq + h * s.vdim + c - 2 * s.dim; col = in.v_off + ch - 2 * cq; }
-    const T* p = proj + col;
-    float y[CK];
-    if (s.taps > 0) {
-      const float* st = (has_state && s.taps > 1)
-                            ? in.conv_state + (long long)rb.slots[b] * (s.taps - 1) * channels + ch : nullptr;
-      const float* w = in.conv_w + (long long)ch * s.taps;
-#pragma unroll
-      for (int t = 0; t < CK; ++t) y[t] = 0.f;
-      // input i of the portion feeds outputs i .. i + taps - 1
-      if (s.taps == 4) {
-        float x[CK + 3];
-#pragma unroll
-        for (int j = 0; j < CK + 3; ++j) x[j] = raw_tap(p, in.ld, q0, i0 + j - 3, st, channels, 4, len);
-        const float w0 = w[0], w1 = w[1], w2 = w[2], w3 = w[3];
-#pragma unroll
-        for (int t = 0; t < CK; ++t) y[t] = fmaf(w0, x[t], fmaf(w1, x[t + 1], fmaf(w2, x[t + 2], w3 * x[t + 3])));
+  auto columns = [&](auto wide) {
+    constexpr int W = decltype(wide)::value;
+    const int tasks = (2 * s.dim + s.vdim) / W;
+    for (int i = tid; i < tasks; i += CP_THREADS) {
+      const int c = i * W;
+      if (c < 2 * s.dim) {
+        const bool is_q = c < s.dim;
+        const int cc = is_q ? c : c - s.dim, at = g * s.dim + cc;
+        const int ch = is_q ? at : cq + at;
+        float* dst = (is_q ? sq : sk) + cc;
+        conv_column<W>(s, in, proj + (is_q ? in.q_off : in.k_off) + at, q0, i0, n, st ? st + ch : nullptr, channels, ch,
+                       [&](int t, const float (&y)[W]) {
+                         if constexpr (W == 2) *reinterpret_cast<float2*>(dst + t * LD) = make_float2(y[0], y[1]);
+                         else dst[t * LD] = y[0];
+                       });
       } else {
-        for (int j = 0; j < s.taps; ++j) {
-          const float wj = w[s.taps - 1 - j];
-#pragma unroll
-          for (int t = 0; t < CK; ++t) y[t] = fmaf(wj, raw_tap(p, in.ld, q0, i0 + t - j, st, channels, s.taps, len), y[t]);
-        }
+        const int v = c - 2 * s.dim, at = h * s.vdim + v, ch = 2 * cq + at;
+        float* dst = vrow + (v / CS_V) * (CK * CS_V);
+        conv_column<W>(s, in, proj + in.v_off + at, q0, i0, n, st ? st + ch : nullptr, channels, ch,
+                       [&](int t, const float (&y)[W]) {
+                         float* d = dst + t * CS_V + ((v % CS_V) ^ (((t >> 1) & 3) << 3));
+                         if constexpr (W == 2) *reinterpret_cast<float2*>(d) = make_float2(y[0], y[1]);
+                         else *d = y[0];
+                       });
       }
-#pragma unroll
-      for (int t = 0; t < CK; ++t) y[t] = silu_f(y[t]);
-    } else {
-#pragma unroll
-      for (int t = 0; t < CK; ++t) y[t] = t < n ? ldf(p + (r0 + t) * in.ld) : 0.f;
     }
-    if (c < 2 * s.dim) {
-      float* dst = c < s.dim ? sq + c : sk + c - s.dim;
-#pragma unroll
-      for (int t = 0; t < CK; ++t) dst[t * LD] = t < n ? y[t] : 0.f;
-    } else {
-      const int v = c - 2 * s.dim;
-      float* dst = vrow + (v / CS_V) * (CK * CS_V);
-#pragma unroll
-      for (int t = 0; t < CK; ++t) dst[t * CS_V + ((v % CS_V) ^ (((t >> 1) & 3) << 3))] = t < n ? y[t] : 0.f;
-    }
-  }
+  };
+  if (((s.dim | s.vdim | (int)in.ld) & 1) == 0) columns(std::integral_constant<int, 2>{});
+  else columns(std::integral_constant<int, 1>{});
   for (int v = s.vdim + tid; v < vblocks * CS_V; v += CP_THREADS)
-#pragma unroll
     for (int t = 0; t < CK; ++t) vrow[(v / CS_V) * (CK * CS_V) + t * CS_V + ((v % CS_V) ^ (((t >> 1) & 3) << 3))] = 0.f;
   // ---- log decays and their running sum; channels past dim are empty
   float range = 0.f;
@@ -178,129 +250,159 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
     float run = 0.f;
     if (c < s.dim) {
       const float bias = in.z_bias[h * s.dim + c];
-      const float ea = DELTA ? expf(in.a_log[h]) : 0.f;
+      const float ea = DELTA ? -expf(in.a_log[h]) : -s.inv_tau;
+      const float* zp = in.z + r0 * in.ldz + h * s.dim + c;
       float z[CK];
 #pragma unroll
-      for (int t = 0; t < CK; ++t) z[t] = t < n ? in.z[(r0 + t) * in.ldz + h * s.dim + c] : 0.f;
+      for (int t = 0; t < CK; ++t) z[t] = t < n ? zp[t * in.ldz] : 0.f;
 #pragma unroll
       for (int t = 0; t < CK; ++t) {
-        if (t < n) run += DELTA ? -ea * softplus_f(z[t] + bias) : -softplus_f(-(z[t] + bias)) * s.inv_tau;
+        if (t < n) run = fmaf(ea, softplus_fast(DELTA ? z[t] + bias : -(z[t] + bias)), run);
         sb[t * LD + c] = run;
       }
     } else {
 #pragma unroll
       for (int t = 0; t < CK; ++t) { sb[t * LD + c] = 0.f; sq[t * LD + c] = 0.f; sk[t * LD + c] = 0.f; }
     }
+    s_inv[c] = __expf(-run);
     range = fmaxf(range, -run);
   }
   if (DELTA && tid < CK) sbeta[tid] = tid < n ? sigmoid_f(ldf(proj + (r0 + tid) * in.ld + in.b_off + h)) : 0.f;
-  const bool pairwise = __syncthreads_or(!(range <= 80.f)) != 0;
-  // ---- unit norms
+  const bool pairwise = __syncthreads_or(!(range <= 60.f)) != 0;
+  // ---- unit norms (as one scale per row) and the query scale
   for (int j = warp; j < 2 * CK; j += CP_THREADS / 32) {
-    float* x = (j < CK ? sq : sk) + (j & (CK - 1)) * LD;
+    const float* x = (j < CK ? sq : sk) + (j & (CK - 1)) * LD;
     float r = 1.f;
     if (s.unit_norm) {
       float ss = 0.f;
-      for (int c = lane; c < s.dim; c += 32) ss += x[c] * x[c];
+#pragma unroll
+      for (int c = lane; c < DP; c += 32) ss = fmaf(x[c], x[c], ss);
       r = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
     }
-    if (j < CK) r *= s.q_scale;
-    for (int c = lane; c < s.dim; c += 32) x[c] *= r;
+    if (lane == 0) s_norm[j] = j < CK ? r * s.q_scale : r;
   }
-  for (int i = tid; i < 512; i += CP_THREADS) sP[i] = 0.f;   // P and A (the pairwise form leaves their upper triangles)
   __syncthreads();
-  // ---- decayed operands of the scan
-  uint8_t* rec = records + ((long long)slot * s.heads + h) * R::BYTES;
-  for (int i = tid; i < CK * (DP / 8); i += CP_THREADS) {
-    const int t = i / (DP / 8), u = i % (DP / 8);
-    uint32_t qh[4], ql[4], kh[4], kl[4], bh[4], bl[4];
+  if (pairwise) {
+    for (int i = tid; i < CK * CK; i += CP_THREADS) {
+      const int t = i / CK, c = i % CK;
+      float p = 0.f, a = 0.f;
+      if (c <= t)
+        for (int k = 0; k < s.dim; ++k) {
+          const float w = sk[c * LD + k] * __expf(sb[t * LD + k] - sb[c * LD + k]);
+          p = fmaf(sq[t * LD + k], w, p);
+          a = fmaf(sk[t * LD + k], w, a);
+        }
+      sP[i] = p * s_norm[t] * s_norm[CK + c];
+      sA[i] = DELTA && c < t ? a * s_norm[CK + t] * s_norm[CK + c] : 0.f;
+    }
+  }
+  // ---- decayed operands: a thread takes units of 8 channels of one token through registers, because the
+  // record image takes the place of the fp32 rows
+  constexpr int UPR = DP / 8, UNITS = (CK * UPR + CP_THREADS - 1) / CP_THREADS;
+  const int u = tid % UPR;
+  float qv[UNITS][8], kv[UNITS][8], bv[UNITS][8], be[8];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      float qv[2], kv[2], bv[2];
+  for (int m = 0; m < UNITS; ++m) {
+    const int t = (tid + m * CP_THREADS) / UPR;
+    if (t < CK) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int c = u * 8 + 2 * j + e;
-        const float bt = sb[t * LD + c], d = __expf(bt);
-        qv[e] = sq[t * LD + c] * d;
-        if (DELTA) kv[e] = sk[t * LD + c] * d;
-        bv[e] = sk[t * LD + c] * __expf(sb[(CK - 1) * LD + c] - bt);
+        const float4 q4 = *reinterpret_cast<const float4*>(sq + t * LD + u * 8 + 4 * e);
+        const float4 k4 = *reinterpret_cast<const float4*>(sk + t * LD + u * 8 + 4 * e);
+        const float4 b4 = *reinterpret_cast<const float4*>(sb + t * LD + u * 8 + 4 * e);
+        qv[m][4 * e] = q4.x; qv[m][4 * e + 1] = q4.y; qv[m][4 * e + 2] = q4.z; qv[m][4 * e + 3] = q4.w;
+        kv[m][4 * e] = k4.x; kv[m][4 * e + 1] = k4.y; kv[m][4 * e + 2] = k4.z; kv[m][4 * e + 3] = k4.w;
+        bv[m][4 * e] = b4.x; bv[m][4 * e + 1] = b4.y; bv[m][4 * e + 2] = b4.z; bv[m][4 * e + 3] = b4.w;
       }
-      split2(qv[0], qv[1], qh[j], ql[j]);
-      if (DELTA) split2(kv[0], kv[1], kh[j], kl[j]);
-      split2(bv[0], bv[1], bh[j], bl[j]);
-    }
-    const int o = unit_off<DP>(t, u);
-    *reinterpret_cast<uint4*>(rec + R::Q_HI + o) = make_uint4(qh[0], qh[1], qh[2], qh[3]);
-    *reinterpret_cast<uint4*>(rec + R::Q_LO + o) = make_uint4(ql[0], ql[1], ql[2], ql[3]);
-    *reinterpret_cast<uint4*>(rec + R::B_HI + o) = make_uint4(bh[0], bh[1], bh[2], bh[3]);
-    *reinterpret_cast<uint4*>(rec + R::B_LO + o) = make_uint4(bl[0], bl[1], bl[2], bl[3]);
-    if (DELTA) {
-      *reinterpret_cast<uint4*>(rec + R::K_HI + o) = make_uint4(kh[0], kh[1], kh[2], kh[3]);
-      *reinterpret_cast<uint4*>(rec + R::K_LO + o) = make_uint4(kl[0], kl[1], kl[2], kl[3]);
     }
   }
-  for (int c = tid; c < DP; c += CP_THREADS) reinterpret_cast<float*>(rec + R::DEC)[c] = __expf(sb[(CK - 1) * LD + c]);
-  // ---- P and A
+#pragma unroll
+  for (int e = 0; e < 8; ++e) be[e] = sb[(CK - 1) * LD + u * 8 + e];
+  __syncthreads();
+#pragma unroll
+  for (int m = 0; m < UNITS; ++m) {
+    const int t = (tid + m * CP_THREADS) / UPR;
+    if (t < CK) {
+      const float nq = s_norm[t], nk = s_norm[CK + t];
+      uint32_t qh[4], ql[4], kh[4], kl[4], bh[4], bl[4], gh[4], gl[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        float q2[2], k2[2], b2[2], g2[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int i = 2 * j + e;
+          const float d = __expf(bv[m][i]), k0 = kv[m][i] * nk;
+          q2[e] = qv[m][i] * nq * d;
+          k2[e] = k0 * d;
+          b2[e] = k0 * __expf(be[i] - bv[m][i]);
+          g2[e] = b2[e] * s_inv[u * 8 + i];
+        }
+        split2(q2[0], q2[1], qh[j], ql[j]);
+        if (DELTA) split2(k2[0], k2[1], kh[j], kl[j]);
+        split2(b2[0], b2[1], bh[j], bl[j]);
+        split2(g2[0], g2[1], gh[j], gl[j]);
+      }
+      const int o = unit_off<DP>(t, u);
+      *reinterpret_cast<uint4*>(psm + R::Q_HI + o) = make_uint4(qh[0], qh[1], qh[2], qh[3]);
+      *reinterpret_cast<uint4*>(psm + R::Q_LO + o) = make_uint4(ql[0], ql[1], ql[2], ql[3]);
+      *reinterpret_cast<uint4*>(psm + R::B_HI + o) = make_uint4(bh[0], bh[1], bh[2], bh[3]);
+      *reinterpret_cast<uint4*>(psm + R::B_LO + o) = make_uint4(bl[0], bl[1], bl[2], bl[3]);
+      *reinterpret_cast<uint4*>(psm + PS::KHAT + o) = make_uint4(gh[0], gh[1], gh[2], gh[3]);
+      *reinterpret_cast<uint4*>(psm + PS::KHAT + R::MAT + o) = make_uint4(gl[0], gl[1], gl[2], gl[3]);
+      if constexpr (DELTA) {
+        *reinterpret_cast<uint4*>(psm + R::K_HI + o) = make_uint4(kh[0], kh[1], kh[2], kh[3]);
+        *reinterpret_cast<uint4*>(psm + R::K_LO + o) = make_uint4(kl[0], kl[1], kl[2], kl[3]);
+      }
+    }
+  }
+  if (tid < UPR)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) reinterpret_cast<float*>(psm + R::DEC)[u * 8 + e] = __expf(be[e]);
+  __syncthreads();
+  // ---- P = tril(q~ k^^T) and A = tril(k~ k^^T, -1): the warps share the channels
   if (!pairwise) {
-    const int r = lane >> 2, tq = lane & 3;
+    const int n_row = (lane & 7) + ((lane >> 4) << 3), n_unit = (lane >> 3) & 1;      // B fragments (row = token)
+    const int a_row = (lane & 7) + (((lane >> 3) & 1) << 3), a_unit = lane >> 4;      // A fragments
+    const uint32_t base = smem_u32(psm);
     float p[2][4] = {}, a[2][4] = {};
     for (int ks = warp; ks < DP / 16; ks += CP_THREADS / 32) {
-      uint32_t qh[4], ql[4], kh[4], kl[4], bh[2][2], bl[2][2];
-#pragma unroll
-      for (int f = 0; f < 4; ++f) {       // A fragments: rows r, r + 8; columns 2 tq (+ 8)
-        const int t = r + 8 * (f & 1), c = ks * 16 + 2 * tq + 8 * (f >> 1);
-        const float d0 = __expf(sb[t * LD + c] - 0.5f * sb[(CK - 1) * LD + c]);
-        const float d1 = __expf(sb[t * LD + c + 1] - 0.5f * sb[(CK - 1) * LD + c + 1]);
-        split2(sq[t * LD + c] * d0, sq[t * LD + c + 1] * d1, qh[f], ql[f]);
-        if (DELTA) split2(sk[t * LD + c] * d0, sk[t * LD + c + 1] * d1, kh[f], kl[f]);
-      }
-#pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-        for (int f = 0; f < 2; ++f) {     // B fragments: k = 2 tq (+ 8), n = r
-          const int t = nt * 8 + r, c = ks * 16 + 2 * tq + 8 * f;
-          const float d0 = __expf(0.5f * sb[(CK - 1) * LD + c] - sb[t * LD + c]);
-          const float d1 = __expf(0.5f * sb[(CK - 1) * LD + c + 1] - sb[t * LD + c + 1]);
-          split2(sk[t * LD + c] * d0, sk[t * LD + c + 1] * d1, bh[nt][f], bl[nt][f]);
-        }
+      uint32_t xh[4], xl[4], bh[4], bl[4];
+      const int bo = unit_off<DP>(n_row, 2 * ks + n_unit), ao = unit_off<DP>(a_row, 2 * ks + a_unit);
+      ldm_x4(base + PS::KHAT + bo, bh);
+      ldm_x4(base + PS::KHAT + R::MAT + bo, bl);
+      ldm_x4(base + R::Q_HI + ao, xh);
+      ldm_x4(base + R::Q_LO + ao, xl);
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) {
-        mma_bf16(p[nt], qh, bh[nt][0], bh[nt][1]);
-        mma_bf16(p[nt], qh, bl[nt][0], bl[nt][1]);
-        mma_bf16(p[nt], ql, bh[nt][0], bh[nt][1]);
-        if (DELTA) {
-          mma_bf16(a[nt], kh, bh[nt][0], bh[nt][1]);
-          mma_bf16(a[nt], kh, bl[nt][0], bl[nt][1]);
-          mma_bf16(a[nt], kl, bh[nt][0], bh[nt][1]);
+        mma_bf16(p[nt], xh, bh[2 * nt], bh[2 * nt + 1]);
+        mma_bf16(p[nt], xh, bl[2 * nt], bl[2 * nt + 1]);
+        mma_bf16(p[nt], xl, bh[2 * nt], bh[2 * nt + 1]);
+      }
+      if constexpr (DELTA) {
+        ldm_x4(base + R::K_HI + ao, xh);
+        ldm_x4(base + R::K_LO + ao, xl);
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          mma_bf16(a[nt], xh, bh[2 * nt], bh[2 * nt + 1]);
+          mma_bf16(a[nt], xh, bl[2 * nt], bl[2 * nt + 1]);
+          mma_bf16(a[nt], xl, bh[2 * nt], bh[2 * nt + 1]);
         }
       }
     }
+    const int r = lane >> 2, tq = lane & 3;
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int t = r + 8 * (e >> 1), c = nt * 8 + 2 * tq + (e & 1);
         part[warp * 512 + t * CK + c] = c <= t ? p[nt][e] : 0.f;     // above the diagonal: may be out of range
-        part[warp * 512 + 256 + t * CK + c] = DELTA && c < t ? a[nt][e] : 0.f;
+        if (DELTA) part[warp * 512 + 256 + t * CK + c] = c < t ? a[nt][e] : 0.f;
       }
     __syncthreads();
-    for (int i = tid; i < 512; i += CP_THREADS)
+    for (int i = tid; i < (DELTA ? 512 : 256); i += CP_THREADS)
       sP[i] = (part[i] + part[512 + i]) + (part[1024 + i] + part[1536 + i]);
-  } else {
-    for (int i = tid; i < CK * CK; i += CP_THREADS) {
-      const int t = i / CK, c = i % CK;
-      if (c > t) continue;
-      float p = 0.f, a = 0.f;
-      for (int k = 0; k < s.dim; ++k) {
-        const float w = sk[c * LD + k] * __expf(sb[t * LD + k] - sb[c * LD + k]);
-        p = fmaf(sq[t * LD + k], w, p);
-        a = fmaf(sk[t * LD + k], w, a);
-      }
-      sP[i] = p;
-      if (DELTA && c < t) sA[i] = a;
-    }
+    __syncthreads();
   }
-  __syncthreads();
   // ---- T = (I + diag(beta) A)^-1 diag(beta): lane j solves column j by forward substitution
   if (DELTA && warp == 0 && lane < CK) {
     float x[CK];
@@ -316,15 +418,24 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
     for (int t = 0; t < CK; ++t) {
       const float v = x[t] * beta;
       const __nv_bfloat16 hi = __float2bfloat16(v);
-      reinterpret_cast<__nv_bfloat16*>(rec + R::T_HI)[t * CK + lane] = hi;
-      reinterpret_cast<__nv_bfloat16*>(rec + R::T_LO)[t * CK + lane] = __float2bfloat16(v - __bfloat162float(hi));
+      reinterpret_cast<__nv_bfloat16*>(psm + R::T_HI)[t * CK + lane] = hi;
+      reinterpret_cast<__nv_bfloat16*>(psm + R::T_LO)[t * CK + lane] = __float2bfloat16(v - __bfloat162float(hi));
     }
   }
-  for (int i = tid - 32; i >= 0 && i < CK * CK; i += CP_THREADS - 32) {
-    const float v = sP[i];
-    const __nv_bfloat16 hi = __float2bfloat16(v);
-    reinterpret_cast<__nv_bfloat16*>(rec + R::P_HI)[i] = hi;
-    reinterpret_cast<__nv_bfloat16*>(rec + R::P_LO)[i] = __float2bfloat16(v - __bfloat162float(hi));
+  if (warp > 0)
+    for (int i = tid - 32; i < CK * CK; i += CP_THREADS - 32) {
+      const float v = sP[i];
+      const __nv_bfloat16 hi = __float2bfloat16(v);
+      reinterpret_cast<__nv_bfloat16*>(psm + R::P_HI)[i] = hi;
+      reinterpret_cast<__nv_bfloat16*>(psm + R::P_LO)[i] = __float2bfloat16(v - __bfloat162float(hi));
+    }
+  fence_proxy_async_smem();
+  __syncthreads();
+  if (tid == 0) {
+    asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;"
+                 ::"l"(records + ((long long)slot * s.heads + h) * R::BYTES), "r"(smem_u32(psm)), "r"((uint32_t)R::BYTES) : "memory");
+    tma_store_commit();
+    tma_store_wait0();
   }
 }
 
@@ -407,35 +518,32 @@ chunk_scan_kernel(RecurrentSpec s, RaggedBatch rb, const uint8_t* __restrict__ r
     const uint8_t* rec = smem + stg * SM::STAGE;
     const uint32_t ra = smem_u32(rec);
     const float* sv = reinterpret_cast<const float*>(rec + R::BYTES);
-    float O[2][4] = {}, W[2][4] = {};
-    // ---- read the old state: O^T = S^T q~^T, W^T = S^T k~^T
+    // The chain from one chunk to the next is S -> W -> U -> S; O hangs off it. So the products of W go
+    // first and those of O fill the waits on U. The three parts of a split product have accumulators of
+    // their own: a chain of dependent MMAs is then as short as the number of k-steps.
+    uint32_t ah[KS][4], al[KS][4];
 #pragma unroll
     for (int j = 0; j < KS; ++j) {
-      uint32_t ah[4], al[4], bh[4], bl[4];
-      split2(S[2 * j][0], S[2 * j][1], ah[0], al[0]);
-      split2(S[2 * j][2], S[2 * j][3], ah[1], al[1]);
-      split2(S[2 * j + 1][0], S[2 * j + 1][1], ah[2], al[2]);
-      split2(S[2 * j + 1][2], S[2 * j + 1][3], ah[3], al[3]);
-      const int off = unit_off<DP>(n_row, 2 * j + n_unit);
-      ldm_x4(ra + R::Q_HI + off, bh);
-      ldm_x4(ra + R::Q_LO + off, bl);
+      split2(S[2 * j][0], S[2 * j][1], ah[j][0], al[j][0]);
+      split2(S[2 * j][2], S[2 * j][3], ah[j][1], al[j][1]);
+      split2(S[2 * j + 1][0], S[2 * j + 1][1], ah[j][2], al[j][2]);
+      split2(S[2 * j + 1][2], S[2 * j + 1][3], ah[j][3], al[j][3]);
+    }
+    auto read_out = [&](int hi_off, int lo_off, float (&acc)[3][2][4]) {   // S^T x^T, x = q~ or k~
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt) {
-        mma_bf16(O[nt], ah, bh[2 * nt], bh[2 * nt + 1]);
-        mma_bf16(O[nt], ah, bl[2 * nt], bl[2 * nt + 1]);
-        mma_bf16(O[nt], al, bh[2 * nt], bh[2 * nt + 1]);
-      }
-      if (DELTA) {
-        ldm_x4(ra + R::K_HI + off, bh);
-        ldm_x4(ra + R::K_LO + off, bl);
+      for (int j = 0; j < KS; ++j) {
+        uint32_t bh[4], bl[4];
+        const int off = unit_off<DP>(n_row, 2 * j + n_unit);
+        ldm_x4(ra + hi_off + off, bh);
+        ldm_x4(ra + lo_off + off, bl);
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
-          mma_bf16(W[nt], ah, bh[2 * nt], bh[2 * nt + 1]);
-          mma_bf16(W[nt], ah, bl[2 * nt], bl[2 * nt + 1]);
-          mma_bf16(W[nt], al, bh[2 * nt], bh[2 * nt + 1]);
+          mma_bf16(acc[0][nt], ah[j], bh[2 * nt], bh[2 * nt + 1]);
+          mma_bf16(acc[1][nt], ah[j], bl[2 * nt], bl[2 * nt + 1]);
+          mma_bf16(acc[2][nt], al[j], bh[2 * nt], bh[2 * nt + 1]);
         }
       }
-    }
+    };
     // ---- U^T (16 channels x 16 tokens) as accumulator fragments
     float U[2][4];
 #pragma unroll
@@ -443,41 +551,48 @@ chunk_scan_kernel(RecurrentSpec s, RaggedBatch rb, const uint8_t* __restrict__ r
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int t = nt * 8 + 2 * tq + (e & 1), col = warp * 16 + r + 8 * (e >> 1);
-        U[nt][e] = sv[t * CS_V + (col ^ (((t >> 1) & 3) << 3))] - (DELTA ? W[nt][e] : 0.f);
+        U[nt][e] = sv[t * CS_V + (col ^ (((t >> 1) & 3) << 3))];
       }
     uint32_t uh[4], ul[4];
-    split2(U[0][0], U[0][1], uh[0], ul[0]);
-    split2(U[0][2], U[0][3], uh[1], ul[1]);
-    split2(U[1][0], U[1][1], uh[2], ul[2]);
-    split2(U[1][2], U[1][3], uh[3], ul[3]);
-    if (DELTA) {
-      uint32_t th[4], tl[4];
-      ldm_x4(ra + R::T_HI + n_row * 32 + n_unit * 16, th);
-      ldm_x4(ra + R::T_LO + n_row * 32 + n_unit * 16, tl);
-#pragma unroll
-      for (int nt = 0; nt < 2; ++nt) {
-        U[nt][0] = U[nt][1] = U[nt][2] = U[nt][3] = 0.f;
-        mma_bf16(U[nt], uh, th[2 * nt], th[2 * nt + 1]);
-        mma_bf16(U[nt], uh, tl[2 * nt], tl[2 * nt + 1]);
-        mma_bf16(U[nt], ul, th[2 * nt], th[2 * nt + 1]);
-      }
+    auto split_u = [&]() {
       split2(U[0][0], U[0][1], uh[0], ul[0]);
       split2(U[0][2], U[0][3], uh[1], ul[1]);
       split2(U[1][0], U[1][1], uh[2], ul[2]);
       split2(U[1][2], U[1][3], uh[3], ul[3]);
-    }
-    // ---- O^T += U^T P^T
-    {
-      uint32_t phh[4], pll[4];
-      ldm_x4(ra + R::P_HI + n_row * 32 + n_unit * 16, phh);
-      ldm_x4(ra + R::P_LO + n_row * 32 + n_unit * 16, pll);
+    };
+    float Oa[3][2][4] = {};
+    if constexpr (DELTA) {
+      float Wa[3][2][4] = {};
+      read_out(R::K_HI, R::K_LO, Wa);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) U[nt][e] -= Wa[0][nt][e] + (Wa[1][nt][e] + Wa[2][nt][e]);
+      split_u();
+      uint32_t th[4], tl[4];
+      ldm_x4(ra + R::T_HI + n_row * 32 + n_unit * 16, th);
+      ldm_x4(ra + R::T_LO + n_row * 32 + n_unit * 16, tl);
+      float Ua[3][2][4] = {};
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) {
-        mma_bf16(O[nt], uh, phh[2 * nt], phh[2 * nt + 1]);
-        mma_bf16(O[nt], uh, pll[2 * nt], pll[2 * nt + 1]);
-        mma_bf16(O[nt], ul, phh[2 * nt], phh[2 * nt + 1]);
+        mma_bf16(Ua[0][nt], uh, th[2 * nt], th[2 * nt + 1]);
+        mma_bf16(Ua[1][nt], uh, tl[2 * nt], tl[2 * nt + 1]);
+        mma_bf16(Ua[2][nt], ul, th[2 * nt], th[2 * nt + 1]);
       }
+      read_out(R::Q_HI, R::Q_LO, Oa);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) U[nt][e] = Ua[0][nt][e] + (Ua[1][nt][e] + Ua[2][nt][e]);
+    } else {
+      read_out(R::Q_HI, R::Q_LO, Oa);
     }
+    split_u();
+    float O[2][4];
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) O[nt][e] = Oa[0][nt][e] + (Oa[1][nt][e] + Oa[2][nt][e]);
     // ---- S^T = S^T diag(e^b) + U^T K-
     const float* dec = reinterpret_cast<const float*>(rec + R::DEC);
 #pragma unroll
@@ -496,7 +611,19 @@ chunk_scan_kernel(RecurrentSpec s, RaggedBatch rb, const uint8_t* __restrict__ r
         acc[3] *= d.y;
         mma_bf16(acc, uh, bh[2 * nt], bh[2 * nt + 1]);
         mma_bf16(acc, uh, bl[2 * nt], bl[2 * nt + 1]);
-        mma_bf16(acc, ul, bh[2 * nt], bh[2 * nt + 1]);
+        if (DELTA) mma_bf16(acc, ul, bh[2 * nt], bh[2 * nt + 1]);   // without the delta rule U = V is exact in bf16
+      }
+    }
+    // ---- O^T += U^T P^T
+    {
+      uint32_t phh[4], pll[4];
+      ldm_x4(ra + R::P_HI + n_row * 32 + n_unit * 16, phh);
+      ldm_x4(ra + R::P_LO + n_row * 32 + n_unit * 16, pll);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) {
+        mma_bf16(O[nt], uh, phh[2 * nt], phh[2 * nt + 1]);
+        mma_bf16(O[nt], uh, pll[2 * nt], pll[2 * nt + 1]);
+        if (DELTA) mma_bf16(O[nt], ul, phh[2 * nt], phh[2 * nt + 1]);
       }
     }
     // ---- the warp is done with the stage; thread 0 refills it once all warps are
@@ -537,13 +664,14 @@ void launch_chunked(const RecurrentSpec& s, const RecurrentInputs& in, const Rag
   using SM = ScanSmem<DP, DELTA>;
   const int vblocks = (s.vdim + CS_V - 1) / CS_V;
   const int slots = rb.rows / CK + rb.n_seq;
-  const int prep_smem = (3 * CK * (DP + 1) + 512 + CK + 2048) * 4;
+  using PS = PrepSmem<DP, DELTA>;
   static bool configured = false;
   if (!configured) {
     MB_CUDA_CHECK(cudaFuncSetAttribute(chunk_scan_kernel<DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, SM::BYTES));
+    MB_CUDA_CHECK(cudaFuncSetAttribute(chunk_prep_kernel<DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, PS::BYTES));
     configured = true;
   }
-  chunk_prep_kernel<DP, DELTA><<<dim3(slots, s.heads), CP_THREADS, prep_smem, stream>>>(s, in, rb, records, vbuf, vblocks);
+  chunk_prep_kernel<DP, DELTA><<<dim3(slots, s.heads), CP_THREADS, PS::BYTES, stream>>>(s, in, rb, records, vbuf, vblocks);
   check_launch();
   chunk_scan_kernel<DP, DELTA><<<dim3(vblocks, s.heads, rb.n_seq), CS_WARPS * 32, SM::BYTES, stream>>>(
       s, rb, records, vbuf, vblocks, in.state, o, status);
@@ -559,7 +687,9 @@ long long record_bytes(const RecurrentSpec& s) {
 
 }  // namespace
 
-bool recurrent_chunked_ok(const RecurrentSpec& s) { return s.dim <= 128; }
+bool recurrent_chunked_ok(const RecurrentSpec& s) {
+  return s.dim <= 128 && (s.delta ? s.decay_kind == 1 : s.decay_kind == 0 && s.taps == 0);
+}
 
 long long recurrent_chunked_scratch(const RecurrentSpec& s, int rows, int n_seq) {
   const long long recs = ((long long)rows / CK + n_seq) * s.heads;
@@ -568,8 +698,8 @@ long long recurrent_chunked_scratch(const RecurrentSpec& s, int rows, int n_seq)
 
 void recurrent_scan_chunked(const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb,
                             void* scratch, float* o, int* status, cudaStream_t stream) {
-  MB_REQUIRE(recurrent_chunked_ok(s), "recurrent_scan_chunked: key width up to 128");
-  MB_REQUIRE((s.delta != 0) == (s.decay_kind == 1), "recurrent_scan_chunked: decay kind and rule come in pairs");
+  MB_REQUIRE(recurrent_chunked_ok(s), "recurrent_scan_chunked: key width up to 128; the delta rule with its own decay, "
+                                      "or gated linear attention without a convolution");
   MB_REQUIRE((reinterpret_cast<uintptr_t>(scratch) & 15) == 0, "recurrent_scan_chunked: scratch must be 16-byte aligned");
   if (rb.rows == 0) return;
   uint8_t* rec = static_cast<uint8_t*>(scratch);

@@ -221,6 +221,54 @@ __global__ void qk_norm_append_kernel(const T* __restrict__ proj, long long ld, 
   }
 }
 
+// bf16 form for widths that are multiples of 8 up to 128: 16 lanes per (token, head slot), 16-byte accesses.
+__global__ void __launch_bounds__(256)
+qk_norm_append8_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
+                       const float* __restrict__ q_gamma, const float* __restrict__ k_gamma, RaggedBatch rb,
+                       const int* __restrict__ block_table, int table_stride, int page_size,
+                       __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_cache,
+                       __nv_bfloat16* __restrict__ v_cache, int heads, int kv_heads, int dk, int dv, float eps) {
+  const int l = threadIdx.x & 15, slots = heads + 2 * kv_heads;
+  const long long total = (long long)rb.rows * slots;
+  const long long stride = (long long)gridDim.x * (blockDim.x >> 4);
+  // both halves of a warp run the same number of iterations: the shuffles need the whole warp
+  for (long long w0 = ((long long)blockIdx.x * (blockDim.x >> 4) + (threadIdx.x >> 4)) & ~1ll; w0 < total; w0 += stride) {
+    const long long w = w0 + ((threadIdx.x >> 4) & 1);
+    const bool live = w < total;
+    const int t = live ? (int)(w / slots) : 0, hs = live ? (int)(w % slots) : 0;
+    const bool is_q = hs < heads, is_v = hs >= heads + kv_heads;
+    const int width = is_v ? dv : dk, j = is_q ? hs : (is_v ? hs - heads - kv_heads : hs - heads);
+    const bool on = live && l * 8 < width;
+    bf16x8 raw;
+    float f[8];
+    float ss = 0.f;
+    if (on) {
+      raw = ldg8(proj, (long long)t * ld + (is_q ? q_off : (is_v ? v_off : k_off)) + j * width + l * 8);
+      unpack8(raw, f);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ss = fmaf(f[i], f[i], ss);
+    }
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!on) continue;
+    if (!is_v) {
+      const float r = 1.f / sqrtf(ss / (float)dk + eps);
+      const float* gm = (is_q ? q_gamma : k_gamma) + l * 8;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] *= r * gm[i];
+      raw = pack8(f);
+    }
+    if (is_q) {
+      stg8(q_out, ((long long)t * heads + j) * dk + l * 8, raw);
+    } else {
+      const int p = rb.pos[t];
+      const int page = block_table[(long long)rb.row_seq[t] * table_stride + p / page_size];
+      if (page >= 0)
+        stg8(is_v ? v_cache : k_cache, (((long long)page * page_size + p % page_size) * kv_heads + j) * width + l * 8, raw);
+    }
+  }
+}
+
 // One warp per (token, query head). Scores of 32 keys at a time (lane = key), then the value rows with
 // lane = channel: every product and the softmax are fp32 whatever the storage type.
 constexpr int PA_WARPS = 4;
@@ -400,6 +448,14 @@ void qk_norm_append(bool f32, const void* proj, long long ld, int q_off, int k_o
                     float eps, cudaStream_t stream) {
   if (rb.rows == 0) return;
   const int grid = ceil_div((long long)rb.rows * (heads + 2 * kv_heads), 8);
+  if (!f32 && dk % 8 == 0 && dv % 8 == 0 && dk <= 128 && dv <= 128 && ((ld | q_off | k_off | v_off) & 7) == 0) {
+    qk_norm_append8_kernel<<<grid_for((long long)rb.rows * (heads + 2 * kv_heads) * 16, 256, 16), 256, 0, stream>>>(
+        (const __nv_bfloat16*)proj, ld, q_off, k_off, v_off, q_gamma, k_gamma, rb, block_table, table_stride, page_size,
+        (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, heads, kv_heads, dk, dv, eps);
+    count_launch();
+    check_launch();
+    return;
+  }
   if (f32)
     qk_norm_append_kernel<float><<<grid, 256, 0, stream>>>(
         (const float*)proj, ld, q_off, k_off, v_off, q_gamma, k_gamma, rb, block_table, table_stride, page_size,

@@ -176,6 +176,56 @@ __global__ void conv_state_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBat
   }
 }
 
+template <typename T>
+__device__ __forceinline__ void ld4(const T* p, float (&f)[4]) {
+  if constexpr (sizeof(T) == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  } else {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  }
+}
+template <typename T>
+__device__ __forceinline__ void st4(T* p, const float (&f)[4]) {
+  if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  }
+}
+
+// The same for value widths up to 128 that are multiples of 4: four channels per lane, one pass.
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_norm_gate4_kernel(RecurrentSpec s, const float* __restrict__ o, const float* __restrict__ gamma,
+                       const T* __restrict__ gate, long long ld_gate, T* __restrict__ out, long long ldo, long long rows) {
+  const int lane = threadIdx.x & 31, nw = (int)(gridDim.x * (blockDim.x >> 5));
+  const bool on = lane * 4 < s.vdim;
+  float g[4] = {};
+  if (on) ld4(gamma + lane * 4, g);
+  const long long total = rows * s.heads;
+  for (long long w = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5); w < total; w += nw) {
+    const long long t = w / s.heads;
+    const int h = (int)(w % s.heads);
+    float x[4] = {}, z[4] = {};
+    if (on) {
+      ld4(o + w * s.vdim + lane * 4, x);
+      ld4(gate + t * ld_gate + h * s.vdim + lane * 4, z);
+    }
+    const float r = 1.f / sqrtf(warp_sum(x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3]) / (float)s.vdim + s.eps);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float e = __fdividef(1.f, 1.f + __expf(-z[j]));
+      x[j] *= r * g[j] * (s.gate_kind == 1 ? e : z[j] * e);
+    }
+    if (on) st4(out + t * ldo + h * s.vdim + lane * 4, x);
+  }
+}
+
 // One warp per (token, head).
 template <typename T>
 __global__ void head_norm_gate_kernel(RecurrentSpec s, const float* __restrict__ o, const float* __restrict__ gamma,
@@ -433,6 +483,15 @@ void head_norm_gate(bool f32, const RecurrentSpec& s, const float* o, const floa
                     long long ld_gate, void* out, long long ldo, int rows, cudaStream_t stream) {
   if (rows == 0) return;
   const int grid = ceil_div((long long)rows * s.heads, 8);
+  if (!f32 && s.vdim <= 128 && s.vdim % 4 == 0 && ld_gate % 4 == 0 && ldo == (long long)s.heads * s.vdim &&
+      (reinterpret_cast<uintptr_t>(gate) & 7) == 0) {
+    const int cap = sm_count() * 16;
+    head_norm_gate4_kernel<__nv_bfloat16><<<grid < cap ? grid : cap, 256, 0, stream>>>(
+        s, o, gamma, (const __nv_bfloat16*)gate, ld_gate, (__nv_bfloat16*)out, ldo, rows);
+    count_launch();
+    check_launch();
+    return;
+  }
   if (f32)
     head_norm_gate_kernel<float><<<grid, 256, 0, stream>>>(s, o, gamma, (const float*)gate, ld_gate, (float*)out, ldo, rows);
   else
