@@ -99,7 +99,7 @@ __device__ __forceinline__ float conv_past(const float* st, int i, int taps, int
 
 // W adjacent channels (2 when every offset is even, else 1) of the chunk's 16 tokens through the short
 // convolution; `put(t, y)` takes the result. col: the channel's column of the projection; ch: its index.
-template <int W, class Put>
+template <int W, bool FULL, class Put>
 __device__ __forceinline__ void conv_column(const RecurrentSpec& s, const RecurrentInputs& in, const T* __restrict__ col, int q0,
                                             int i0, int n, const float* __restrict__ st, int channels, int ch, Put put) {
   const T* p = col + (long long)(q0 + i0) * in.ld;
@@ -108,11 +108,11 @@ __device__ __forceinline__ void conv_column(const RecurrentSpec& s, const Recurr
   for (int t = 0; t < CK; ++t) {
     if constexpr (W == 2) {
       float2 f = make_float2(0.f, 0.f);
-      if (t < n) f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p + t * in.ld));
+      if (FULL || t < n) f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p + t * in.ld));
       x[t][0] = f.x;
       x[t][1] = f.y;
     } else {
-      x[t][0] = t < n ? __bfloat162float(p[t * in.ld]) : 0.f;
+      x[t][0] = FULL || t < n ? __bfloat162float(p[t * in.ld]) : 0.f;
     }
   }
   if (s.taps == 0) {
@@ -139,7 +139,7 @@ __device__ __forceinline__ void conv_column(const RecurrentSpec& s, const Recurr
 #pragma unroll
       for (int w = 0; w < W; ++w) {
         const float a = fmaf(w4[0][w], h3[w], fmaf(w4[1][w], h2[w], fmaf(w4[2][w], h1[w], w4[3][w] * x[t][w])));
-        y[w] = t < n ? conv_act(a) : 0.f;
+        y[w] = FULL || t < n ? conv_act(a) : 0.f;
         h3[w] = h2[w];
         h2[w] = h1[w];
         h1[w] = x[t][w];
@@ -169,13 +169,13 @@ struct PrepSmem {
   static constexpr int KHAT = R::BYTES;                    // k e^{-b}, head and tail, behind the record image
   static constexpr int IMG = KHAT + 2 * R::MAT;
   static constexpr int OFF_MISC = IMG > F32 ? IMG : F32;   // the record image replaces the fp32 rows
-  // norms [32], beta [16], e^{-b_16} [DP], partial P / A [4][512], P / A [512]
-  static constexpr int BYTES = OFF_MISC + (48 + DP + 2048 + 512) * 4;
+  // norms [32], beta [16], e^{-b_16} [DP], P / A [512]
+  static constexpr int BYTES = OFF_MISC + (48 + DP + 512) * 4;
 };
 
 // One CTA per (chunk, head).
 template <int DP, bool DELTA>
-__global__ void __launch_bounds__(CP_THREADS, 4)
+__global__ void __launch_bounds__(CP_THREADS, 5)
 chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* __restrict__ records,
                   float* __restrict__ vbuf, int vblocks) {
   using R = Rec<DP, DELTA>;
@@ -188,8 +188,7 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
   float* s_norm = reinterpret_cast<float*>(psm + PS::OFF_MISC);   // [32] scales of the q and k rows
   float* sbeta = s_norm + 32;
   float* s_inv = sbeta + CK;                     // [DP] e^{-b_16}
-  float* part = s_inv + DP;                      // [4 warps][P, A][256]
-  float* sP = part + 2048;                       // [16][16]
+  float* sP = s_inv + DP;                        // [16][16], pairwise form only
   float* sA = sP + 256;
   const int slot = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   int b = 0;
@@ -213,8 +212,9 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
   const float* st = (has_state && s.taps > 1) ? in.conv_state + (long long)rb.slots[b] * (s.taps - 1) * channels : nullptr;
   // ---- q, k, v: short convolution + silu
   float* vrow = vbuf + ((long long)slot * s.heads + h) * vblocks * (CK * CS_V);
-  auto columns = [&](auto wide) {
+  auto columns = [&](auto wide, auto full) {
     constexpr int W = decltype(wide)::value;
+    constexpr bool FULL = decltype(full)::value;
     const int tasks = (2 * s.dim + s.vdim) / W;
     for (int i = tid; i < tasks; i += CP_THREADS) {
       const int c = i * W;
@@ -223,7 +223,7 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
         const int cc = is_q ? c : c - s.dim, at = g * s.dim + cc;
         const int ch = is_q ? at : cq + at;
         float* dst = (is_q ? sq : sk) + cc;
-        conv_column<W>(s, in, proj + (is_q ? in.q_off : in.k_off) + at, q0, i0, n, st ? st + ch : nullptr, channels, ch,
+        conv_column<W, FULL>(s, in, proj + (is_q ? in.q_off : in.k_off) + at, q0, i0, n, st ? st + ch : nullptr, channels, ch,
                        [&](int t, const float (&y)[W]) {
                          if constexpr (W == 2) *reinterpret_cast<float2*>(dst + t * LD) = make_float2(y[0], y[1]);
                          else dst[t * LD] = y[0];
@@ -231,7 +231,7 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
       } else {
         const int v = c - 2 * s.dim, at = h * s.vdim + v, ch = 2 * cq + at;
         float* dst = vrow + (v / CS_V) * (CK * CS_V);
-        conv_column<W>(s, in, proj + in.v_off + at, q0, i0, n, st ? st + ch : nullptr, channels, ch,
+        conv_column<W, FULL>(s, in, proj + in.v_off + at, q0, i0, n, st ? st + ch : nullptr, channels, ch,
                        [&](int t, const float (&y)[W]) {
                          float* d = dst + t * CS_V + ((v % CS_V) ^ (((t >> 1) & 3) << 3));
                          if constexpr (W == 2) *reinterpret_cast<float2*>(d) = make_float2(y[0], y[1]);
@@ -240,8 +240,9 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
       }
     }
   };
-  if (((s.dim | s.vdim | (int)in.ld) & 1) == 0) columns(std::integral_constant<int, 2>{});
-  else columns(std::integral_constant<int, 1>{});
+  if (((s.dim | s.vdim | (int)in.ld) & 1) != 0) columns(std::integral_constant<int, 1>{}, std::false_type{});
+  else if (n == CK) columns(std::integral_constant<int, 2>{}, std::true_type{});
+  else columns(std::integral_constant<int, 2>{}, std::false_type{});
   for (int v = s.vdim + tid; v < vblocks * CS_V; v += CP_THREADS)
     for (int t = 0; t < CK; ++t) vrow[(v / CS_V) * (CK * CS_V) + t * CS_V + ((v % CS_V) ^ (((t >> 1) & 3) << 3))] = 0.f;
   // ---- log decays and their running sum; channels past dim are empty
@@ -359,76 +360,76 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
 #pragma unroll
     for (int e = 0; e < 8; ++e) reinterpret_cast<float*>(psm + R::DEC)[u * 8 + e] = __expf(be[e]);
   __syncthreads();
-  // ---- P = tril(q~ k^^T) and A = tril(k~ k^^T, -1): the warps share the channels
-  if (!pairwise) {
-    const int n_row = (lane & 7) + ((lane >> 4) << 3), n_unit = (lane >> 3) & 1;      // B fragments (row = token)
-    const int a_row = (lane & 7) + (((lane >> 3) & 1) << 3), a_unit = lane >> 4;      // A fragments
-    const uint32_t base = smem_u32(psm);
-    float p[2][4] = {}, a[2][4] = {};
-    for (int ks = warp; ks < DP / 16; ks += CP_THREADS / 32) {
-      uint32_t xh[4], xl[4], bh[4], bl[4];
-      const int bo = unit_off<DP>(n_row, 2 * ks + n_unit), ao = unit_off<DP>(a_row, 2 * ks + a_unit);
-      ldm_x4(base + PS::KHAT + bo, bh);
-      ldm_x4(base + PS::KHAT + R::MAT + bo, bl);
-      ldm_x4(base + R::Q_HI + ao, xh);
-      ldm_x4(base + R::Q_LO + ao, xl);
+  // ---- warp 0: P = tril(q~ k^^T); warp 1: A = tril(k~ k^^T, -1) and T
+  if (warp < (DELTA ? 2 : 1)) {
+    const int r = lane >> 2, tq = lane & 3;
+    const int x_hi = warp == 0 ? R::Q_HI : (DELTA ? R::K_HI : 0), x_lo = warp == 0 ? R::Q_LO : (DELTA ? R::K_LO : 0);
+    float* dst = warp == 0 ? sP : sA;
+    float acc[3][2][4] = {};
+    if (!pairwise) {
+      const int n_row = (lane & 7) + ((lane >> 4) << 3), n_unit = (lane >> 3) & 1;      // B fragments (row = token)
+      const int a_row = (lane & 7) + (((lane >> 3) & 1) << 3), a_unit = lane >> 4;      // A fragments
+      const uint32_t base = smem_u32(psm);
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt) {
-        mma_bf16(p[nt], xh, bh[2 * nt], bh[2 * nt + 1]);
-        mma_bf16(p[nt], xh, bl[2 * nt], bl[2 * nt + 1]);
-        mma_bf16(p[nt], xl, bh[2 * nt], bh[2 * nt + 1]);
-      }
-      if constexpr (DELTA) {
-        ldm_x4(base + R::K_HI + ao, xh);
-        ldm_x4(base + R::K_LO + ao, xl);
+      for (int ks = 0; ks < DP / 16; ++ks) {
+        uint32_t xh[4], xl[4], bh[4], bl[4];
+        const int bo = unit_off<DP>(n_row, 2 * ks + n_unit), ao = unit_off<DP>(a_row, 2 * ks + a_unit);
+        ldm_x4(base + PS::KHAT + bo, bh);
+        ldm_x4(base + PS::KHAT + R::MAT + bo, bl);
+        ldm_x4(base + x_hi + ao, xh);
+        ldm_x4(base + x_lo + ao, xl);
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
-          mma_bf16(a[nt], xh, bh[2 * nt], bh[2 * nt + 1]);
-          mma_bf16(a[nt], xh, bl[2 * nt], bl[2 * nt + 1]);
-          mma_bf16(a[nt], xl, bh[2 * nt], bh[2 * nt + 1]);
+          mma_bf16(acc[0][nt], xh, bh[2 * nt], bh[2 * nt + 1]);
+          mma_bf16(acc[1][nt], xh, bl[2 * nt], bl[2 * nt + 1]);
+          mma_bf16(acc[2][nt], xl, bh[2 * nt], bh[2 * nt + 1]);
         }
       }
     }
-    const int r = lane >> 2, tq = lane & 3;
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int t = r + 8 * (e >> 1), c = nt * 8 + 2 * tq + (e & 1);
-        part[warp * 512 + t * CK + c] = c <= t ? p[nt][e] : 0.f;     // above the diagonal: may be out of range
-        if (DELTA) part[warp * 512 + 256 + t * CK + c] = c < t ? a[nt][e] : 0.f;
+      for (int e = 0; e < 4; e += 2) {
+        const int t = r + 4 * e, c = nt * 8 + 2 * tq;
+        float v[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const float y = pairwise ? dst[t * CK + c + i] : acc[0][nt][e + i] + (acc[1][nt][e + i] + acc[2][nt][e + i]);
+          // past the diagonal the factors may be out of range: select, do not multiply
+          v[i] = (warp == 0 ? c + i <= t : c + i < t) ? y : 0.f;
+        }
+        if (warp == 0) {
+          uint32_t hi, lo;
+          split2(v[0], v[1], hi, lo);
+          *reinterpret_cast<uint32_t*>(psm + R::P_HI + (t * CK + c) * 2) = hi;
+          *reinterpret_cast<uint32_t*>(psm + R::P_LO + (t * CK + c) * 2) = lo;
+        } else {
+          *reinterpret_cast<float2*>(sA + t * CK + c) = make_float2(v[0], v[1]);
+        }
       }
-    __syncthreads();
-    for (int i = tid; i < (DELTA ? 512 : 256); i += CP_THREADS)
-      sP[i] = (part[i] + part[512 + i]) + (part[1024 + i] + part[1536 + i]);
-    __syncthreads();
+    __syncwarp();
+    // T = (I + diag(beta) A)^-1 diag(beta): lane j solves column j by forward substitution
+    if constexpr (DELTA) {
+      if (warp == 1 && lane < CK) {
+        float x[CK];
+#pragma unroll
+        for (int t = 0; t < CK; ++t) {
+          float y = 0.f;
+#pragma unroll
+          for (int c = 0; c < t; ++c) y = fmaf(sA[t * CK + c], x[c], y);
+          x[t] = t == lane ? 1.f : (t > lane ? -sbeta[t] * y : 0.f);
+        }
+        const float beta = sbeta[lane];
+#pragma unroll
+        for (int t = 0; t < CK; ++t) {
+          const float v = x[t] * beta;
+          const __nv_bfloat16 hi = __float2bfloat16(v);
+          reinterpret_cast<__nv_bfloat16*>(psm + R::T_HI)[t * CK + lane] = hi;
+          reinterpret_cast<__nv_bfloat16*>(psm + R::T_LO)[t * CK + lane] = __float2bfloat16(v - __bfloat162float(hi));
+        }
+      }
+    }
   }
-  // ---- T = (I + diag(beta) A)^-1 diag(beta): lane j solves column j by forward substitution
-  if (DELTA && warp == 0 && lane < CK) {
-    float x[CK];
-#pragma unroll
-    for (int t = 0; t < CK; ++t) {
-      float y = 0.f;
-#pragma unroll
-      for (int c = 0; c < t; ++c) y = fmaf(sA[t * CK + c], x[c], y);
-      x[t] = t == lane ? 1.f : (t > lane ? -sbeta[t] * y : 0.f);
-    }
-    const float beta = sbeta[lane];
-#pragma unroll
-    for (int t = 0; t < CK; ++t) {
-      const float v = x[t] * beta;
-      const __nv_bfloat16 hi = __float2bfloat16(v);
-      reinterpret_cast<__nv_bfloat16*>(psm + R::T_HI)[t * CK + lane] = hi;
-      reinterpret_cast<__nv_bfloat16*>(psm + R::T_LO)[t * CK + lane] = __float2bfloat16(v - __bfloat162float(hi));
-    }
-  }
-  if (warp > 0)
-    for (int i = tid - 32; i < CK * CK; i += CP_THREADS - 32) {
-      const float v = sP[i];
-      const __nv_bfloat16 hi = __float2bfloat16(v);
-      reinterpret_cast<__nv_bfloat16*>(psm + R::P_HI)[i] = hi;
-      reinterpret_cast<__nv_bfloat16*>(psm + R::P_LO)[i] = __float2bfloat16(v - __bfloat162float(hi));
-    }
   fence_proxy_async_smem();
   __syncthreads();
   if (tid == 0) {
