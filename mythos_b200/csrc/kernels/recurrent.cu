@@ -284,6 +284,20 @@ recurrent_decode_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, Dec
   float *q = sm, *k = q + s.dim, *d = k + s.dim, *v = d + s.dim, *o = v + s.vdim, *xa = o + s.vdim, *xg = xa + a.rank;
   const int g = h / (s.heads / s.kv_heads), cq = s.kv_heads * s.dim, channels = 2 * cq + s.heads * s.vdim;
   const T* proj = static_cast<const T*>(in.proj) + row * in.ld;
+  // the state rows of the warp's first group are on their way while q, k, v and the decays are prepared,
+  // those of every next group while the one before is worked on
+  float* st = in.state + ((long long)slot * s.heads + h) * s.vdim * s.dim;
+  float nextS[RD_R][NI];
+  auto fetch = [&](int v0) {
+#pragma unroll
+    for (int r = 0; r < RD_R; ++r)
+#pragma unroll
+      for (int n = 0; n < NI; ++n) {
+        const int c = lane + 32 * n;
+        nextS[r][n] = (!fresh && c < s.dim && v0 + r < s.vdim) ? st[(long long)(v0 + r) * s.dim + c] : 0.f;
+      }
+  };
+  fetch(warp * RD_R);
   for (int c = tid; c < 2 * s.dim + s.vdim; c += RD_THREADS) {
     int ch, col;
     if (c < s.dim) { ch = g * s.dim + c; col = in.q_off + ch; }
@@ -295,12 +309,25 @@ recurrent_decode_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, Dec
       float acc = w[s.taps - 1] * y, x = y;
       if (s.taps > 1) {
         float* st = in.conv_state + (long long)slot * (s.taps - 1) * channels + ch;
-        float nxt = x;                                // newest first: entry j moves to j - 1
-        for (int j = s.taps - 2; j >= 0; --j) {
-          const float old = fresh ? 0.f : st[(long long)j * channels];
-          acc = fmaf(w[j], old, acc);
-          if (own_conv) st[(long long)j * channels] = nxt;
-          nxt = old;
+        if (s.taps == 4) {                            // all loads before the stores
+          float old[3];
+#pragma unroll
+          for (int j = 0; j < 3; ++j) old[j] = fresh ? 0.f : st[(long long)j * channels];
+#pragma unroll
+          for (int j = 0; j < 3; ++j) acc = fmaf(w[j], old[j], acc);
+          if (own_conv) {
+            st[0] = old[1];
+            st[channels] = old[2];
+            st[2ll * channels] = x;
+          }
+        } else {
+          float nxt = x;                              // newest first: entry j moves to j - 1
+          for (int j = s.taps - 2; j >= 0; --j) {
+            const float old = fresh ? 0.f : st[(long long)j * channels];
+            acc = fmaf(w[j], old, acc);
+            if (own_conv) st[(long long)j * channels] = nxt;
+            nxt = old;
+          }
         }
       }
       y = silu_f(acc);
@@ -340,16 +367,13 @@ recurrent_decode_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, Dec
     kr[n] = ok ? k[c] : 0.f;
     dr[n] = ok ? d[c] : 0.f;
   }
-  float* st = in.state + ((long long)slot * s.heads + h) * s.vdim * s.dim;
   for (int v0 = warp * RD_R; v0 < s.vdim; v0 += NW * RD_R) {
     float S[RD_R][NI];
 #pragma unroll
     for (int r = 0; r < RD_R; ++r)
 #pragma unroll
-      for (int n = 0; n < NI; ++n) {
-        const int c = lane + 32 * n;
-        S[r][n] = (!fresh && c < s.dim && v0 + r < s.vdim) ? st[(long long)(v0 + r) * s.dim + c] : 0.f;
-      }
+      for (int n = 0; n < NI; ++n) S[r][n] = nextS[r][n];
+    if (v0 + NW * RD_R < s.vdim) fetch(v0 + NW * RD_R);
     float u[RD_R];
 #pragma unroll
     for (int r = 0; r < RD_R; ++r) {
