@@ -33,7 +33,9 @@ namespace {
 constexpr int CK = 16;            // tokens per chunk
 constexpr int CS_WARPS = 4;       // scan warps per CTA
 constexpr int CS_V = 16 * CS_WARPS;
-constexpr int CP_THREADS = 128;
+// threads and resident CTAs per SM of chunk_prep by key width
+__host__ __device__ constexpr int cp_threads(int dp) { return dp == 128 ? 256 : 128; }
+__host__ __device__ constexpr int cp_blocks(int dp) { return dp == 128 ? 4 : 8; }
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
@@ -175,12 +177,12 @@ struct PrepSmem {
 
 // One CTA per (chunk, head).
 template <int DP, bool DELTA>
-__global__ void __launch_bounds__(CP_THREADS, 5)
+__global__ void __launch_bounds__(cp_threads(DP), cp_blocks(DP))
 chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* __restrict__ records,
                   float* __restrict__ vbuf, int vblocks) {
   using R = Rec<DP, DELTA>;
   using PS = PrepSmem<DP, DELTA>;
-  constexpr int LD = PS::LD;
+  constexpr int LD = PS::LD, CP_THREADS = cp_threads(DP);
   extern __shared__ __align__(128) uint8_t psm[];
   float* sq = reinterpret_cast<float*>(psm);     // [16][LD]
   float* sk = sq + CK * LD;
@@ -672,7 +674,7 @@ void launch_chunked(const RecurrentSpec& s, const RecurrentInputs& in, const Rag
     MB_CUDA_CHECK(cudaFuncSetAttribute(chunk_prep_kernel<DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, PS::BYTES));
     configured = true;
   }
-  chunk_prep_kernel<DP, DELTA><<<dim3(slots, s.heads), CP_THREADS, PS::BYTES, stream>>>(s, in, rb, records, vbuf, vblocks);
+  chunk_prep_kernel<DP, DELTA><<<dim3(slots, s.heads), cp_threads(DP), PS::BYTES, stream>>>(s, in, rb, records, vbuf, vblocks);
   check_launch();
   chunk_scan_kernel<DP, DELTA><<<dim3(vblocks, s.heads, rb.n_seq), CS_WARPS * 32, SM::BYTES, stream>>>(
       s, rb, records, vbuf, vblocks, in.state, o, status);
