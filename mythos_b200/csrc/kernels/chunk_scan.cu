@@ -171,8 +171,8 @@ struct PrepSmem {
   static constexpr int KHAT = R::BYTES;                    // k e^{-b}, head and tail, behind the record image
   static constexpr int IMG = KHAT + 2 * R::MAT;
   static constexpr int OFF_MISC = IMG > F32 ? IMG : F32;   // the record image replaces the fp32 rows
-  // norms [32], beta [16], e^{-b_16} [DP], P / A [512]
-  static constexpr int BYTES = OFF_MISC + (48 + DP + 512) * 4;
+  // norms [32], beta [16], e^{-b_16} [DP], P / A [512], blocks of the inverse [256]
+  static constexpr int BYTES = OFF_MISC + (48 + DP + 512 + 256) * 4;
 };
 
 // One CTA per (chunk, head).
@@ -191,7 +191,8 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
   float* sbeta = s_norm + 32;
   float* s_inv = sbeta + CK;                     // [DP] e^{-b_16}
   float* sP = s_inv + DP;                        // [16][16], pairwise form only
-  float* sA = sP + 256;
+  float* sA = sP + 256;                          // A, then diag(beta) A
+  float* sD = sA + 256;                          // inverses of the two diagonal 8 x 8 blocks, two products [8][8] each
   const int slot = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   int b = 0;
   {
@@ -406,29 +407,59 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
           *reinterpret_cast<uint32_t*>(psm + R::P_HI + (t * CK + c) * 2) = hi;
           *reinterpret_cast<uint32_t*>(psm + R::P_LO + (t * CK + c) * 2) = lo;
         } else {
-          *reinterpret_cast<float2*>(sA + t * CK + c) = make_float2(v[0], v[1]);
+          *reinterpret_cast<float2*>(sA + t * CK + c) = make_float2(sbeta[t] * v[0], sbeta[t] * v[1]);
         }
       }
     __syncwarp();
-    // T = (I + diag(beta) A)^-1 diag(beta): lane j solves column j by forward substitution
+    // T = (I + N)^-1 diag(beta), N = diag(beta) A: the two diagonal 8 x 8 blocks by forward substitution (a lane
+    // per column), the block below them as -D22 N21 D11
     if constexpr (DELTA) {
-      if (warp == 1 && lane < CK) {
-        float x[CK];
+      if (warp == 1) {
+        if (lane < CK) {
+          const int j = lane & 7;
+          const float* nb = sA + (lane & 8) * (CK + 1);
+          float x[8];
 #pragma unroll
-        for (int t = 0; t < CK; ++t) {
-          float y = 0.f;
+          for (int t = 0; t < 8; ++t) {
+            float y = 0.f;
 #pragma unroll
-          for (int c = 0; c < t; ++c) y = fmaf(sA[t * CK + c], x[c], y);
-          x[t] = t == lane ? 1.f : (t > lane ? -sbeta[t] * y : 0.f);
+            for (int c = 0; c < t; ++c) y = fmaf(nb[t * CK + c], x[c], y);
+            x[t] = t == j ? 1.f : (t > j ? -y : 0.f);
+            sD[(lane & 8) * 8 + t * 8 + j] = x[t];
+          }
         }
-        const float beta = sbeta[lane];
+        __syncwarp();
+        float m[2] = {};
 #pragma unroll
-        for (int t = 0; t < CK; ++t) {
-          const float v = x[t] * beta;
-          const __nv_bfloat16 hi = __float2bfloat16(v);
-          reinterpret_cast<__nv_bfloat16*>(psm + R::T_HI)[t * CK + lane] = hi;
-          reinterpret_cast<__nv_bfloat16*>(psm + R::T_LO)[t * CK + lane] = __float2bfloat16(v - __bfloat162float(hi));
+        for (int c = 0; c < 8; ++c) {
+          const float d = sD[c * 8 + (lane & 7)];
+          m[0] = fmaf(sA[(8 + (lane >> 3)) * CK + c], d, m[0]);
+          m[1] = fmaf(sA[(12 + (lane >> 3)) * CK + c], d, m[1]);
         }
+        sD[128 + lane] = m[0];
+        sD[160 + lane] = m[1];
+        __syncwarp();
+        m[0] = m[1] = 0.f;
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+          const float d = sD[128 + c * 8 + (lane & 7)];
+          m[0] = fmaf(-sD[64 + (lane >> 3) * 8 + c], d, m[0]);
+          m[1] = fmaf(-sD[96 + (lane >> 3) * 8 + c], d, m[1]);
+        }
+        sD[192 + lane] = m[0];
+        sD[224 + lane] = m[1];
+        __syncwarp();
+        const int t = lane >> 1, half = lane & 1;      // 8 columns of a row per lane
+        const float* row = t < 8 ? sD + t * 8 : (half ? sD + 64 + (t - 8) * 8 : sD + 192 + (t - 8) * 8);
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const bool zero = t < 8 && half;
+          split2(zero ? 0.f : row[2 * i] * sbeta[half * 8 + 2 * i], zero ? 0.f : row[2 * i + 1] * sbeta[half * 8 + 2 * i + 1], hi[i],
+                 lo[i]);
+        }
+        *reinterpret_cast<uint4*>(psm + R::T_HI + t * 32 + half * 16) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(psm + R::T_LO + t * 32 + half * 16) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
       }
     }
   }
@@ -438,7 +469,7 @@ chunk_prep_kernel(RecurrentSpec s, RecurrentInputs in, RaggedBatch rb, uint8_t* 
     asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;"
                  ::"l"(records + ((long long)slot * s.heads + h) * R::BYTES), "r"(smem_u32(psm)), "r"((uint32_t)R::BYTES) : "memory");
     tma_store_commit();
-    tma_store_wait0();
+    tma_store_wait_read0();          // shared memory has been read; the grid's end covers the rest
   }
 }
 
