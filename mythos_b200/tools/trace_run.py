@@ -42,7 +42,7 @@ class TraceReplay:
 
     def run(self, step: dict):
         """Logits [wanted, vocab] of one step, or None when nothing is wanted."""
-        eng, entries = self.engine, step["entries"]
+        eng, entries = self.engine, [e for e in step["entries"] if e["tokens"]]
         for e in entries:
             if e["id"] not in self.seqs:
                 self.seqs[e["id"]] = eng.cache.new_sequence()

@@ -163,7 +163,7 @@ def _run_attention(case, kernel, gamma_q, gamma_k, scale):
 
 
 def _attention_want(case, q, scale):
-    """From the pages as the append left them (bf16 pages are part of the contract)."""
+    """From the pages as the append left them (they hold the activation type)."""
     c, out, row = case, [], 0
     d = lambda t: t.double().cpu()
     kc, vc, table = d(c["kc"]), d(c["vc"]), c["table"].cpu()
@@ -294,7 +294,7 @@ def _scan(case, how, rows, lens, bases, slots):
     return o, out[:, : s["heads"] * s["vdim"]].view(n, s["heads"], s["vdim"])
 
 
-RECURRENT = [("delta", 2, 2, 64, 64, 4, False), ("delta", 6, 2, 44, 28, 3, True), ("delta", 3, 1, 128, 96, 2, True),
+RECURRENT = [("delta", 3, 3, 64, 80, 4, False), ("delta", 6, 2, 44, 28, 3, True), ("delta", 3, 1, 128, 96, 2, True),
              ("delta", 1, 1, 32, 130, 1, False), ("gla", 3, 3, 24, 40, 0, False), ("gla", 2, 2, 128, 128, 0, False),
              ("gla", 2, 2, 64, 17, 0, False), ("delta", 2, 2, 16, 16, 6, True)]
 
