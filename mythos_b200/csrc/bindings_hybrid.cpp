@@ -37,7 +37,7 @@ mb::RaggedBatch ragged(const std::vector<Tensor>& batch) {
 }
 
 void embed_pos_norm(const Tensor& ids, const Tensor& pos, const Tensor& embed, const OptTensor& pos_table, double scale,
-                    const Tensor& gamma, Tensor& x, Tensor& h, double eps) {
+                    const OptTensor& gamma, Tensor& x, Tensor& h, double eps) {
   const bool f32 = is_f32(h, "h");
   const int64_t rows = ids.numel(), dim = embed.size(1);
   chk_c(ids, I32, "ids");
@@ -58,7 +58,7 @@ void embed_pos_norm(const Tensor& ids, const Tensor& pos, const Tensor& embed, c
 }
 
 void sandwich_norm(const Tensor& y1, const OptTensor& y2, const OptTensor& w1, const OptTensor& w2, const Tensor& w_post,
-                   Tensor& x, const Tensor& w_next, Tensor& h, double eps) {
+                   Tensor& x, const OptTensor& w_next, Tensor& h, double eps, double mult) {
   const bool f32 = is_f32(h, "h");
   chk_c(x, F32, "x");
   const int64_t rows = x.size(0), dim = x.size(1);
@@ -69,9 +69,27 @@ void sandwich_norm(const Tensor& y1, const OptTensor& y2, const OptTensor& w1, c
     TORCH_CHECK(y2->stride(0) == y1.stride(0), "sandwich_norm: y1 and y2 need the same row stride");
   }
   c10::cuda::CUDAGuard guard(h.device());
-  mb::sandwich_norm(f32, y1.data_ptr(), cptr(y2), y1.stride(0), fptr(w1, dim, "w1"), fptr(w2, dim, "w2"),
-                    fptr(w_post, dim, "w_post"), x.data_ptr<float>(), fptr(w_next, dim, "w_next"), h.data_ptr(),
-                    h.stride(0), (int)rows, (int)dim, (float)eps, cur_stream());
+  const mb::SublayerOut y{y1.data_ptr(), cptr(y2), y1.stride(0), fptr(w1, dim, "w1"), fptr(w2, dim, "w2"), nullptr, nullptr, 0};
+  mb::sandwich_norm(f32, y, fptr(w_post, dim, "w_post"), (float)mult, x.data_ptr<float>(), fptr(w_next, dim, "w_next"),
+                    h.data_ptr(), h.stride(0), (int)rows, (int)dim, (float)eps, cur_stream());
+}
+
+// The same with the weighted sum of a token's experts as the sublayer's output: y [pairs, dim], row and weight [rows, top].
+void expert_norm(const Tensor& y, const Tensor& row, const Tensor& weight, const Tensor& w_post, Tensor& x,
+                 const OptTensor& w_next, Tensor& h, double eps, double mult) {
+  const bool f32 = is_f32(h, "h");
+  chk_c(x, F32, "x");
+  const int64_t rows = x.size(0), dim = x.size(1), top = row.size(1);
+  chk_c(row, I32, "row");
+  chk_c(weight, F32, "weight");
+  TORCH_CHECK(row.dim() == 2 && row.size(0) == rows && weight.sizes() == row.sizes(), "expert_norm: row / weight");
+  chk_rows(y, f32, rows * top, dim, "y");
+  chk_rows(h, f32, rows, dim, "h");
+  c10::cuda::CUDAGuard guard(h.device());
+  const mb::SublayerOut s{y.data_ptr(), nullptr, y.stride(0), nullptr, nullptr, row.data_ptr<int>(), weight.data_ptr<float>(),
+                          (int)top};
+  mb::sandwich_norm(f32, s, fptr(w_post, dim, "w_post"), (float)mult, x.data_ptr<float>(), fptr(w_next, dim, "w_next"),
+                    h.data_ptr(), h.stride(0), (int)rows, (int)dim, (float)eps, cur_stream());
 }
 
 struct Pages {
@@ -167,9 +185,14 @@ void paged_attn_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_c
                         q.stride(0), pg.dv, cptr(gate), gate.has_value() ? gate->stride(0) : 0);
 }
 
-// Few-token GEMM: out = alpha * x w^T, or with f > 0 silu(x w[:f]^T) * (x w[f_off : f_off + f]^T).
+// Gated activation (kind, limit, alpha); see GateAct.
+using Act = std::tuple<int64_t, double, double>;
+mb::GateAct gate(const Act& a) { return mb::GateAct{(int)std::get<0>(a), (float)std::get<1>(a), (float)std::get<2>(a)}; }
+
+// Few-token GEMM: out = alpha * x w^T, or with f > 0 act(x w[:f]^T, x w[f_off : f_off + f]^T), or with mul
+// gelu_tanh(x w^T) * mul[ids, :].
 void gemm_decode(const Tensor& x, const Tensor& w, Tensor& out, int64_t f, int64_t f_off, double alpha,
-                 const OptTensor& status) {
+                 const OptTensor& status, const Act& act, const OptTensor& mul, const OptTensor& ids) {
   chk(x, BF16, "x");
   chk(w, BF16, "w");
   const bool of32 = is_f32(out, "out");
@@ -177,11 +200,243 @@ void gemm_decode(const Tensor& x, const Tensor& w, Tensor& out, int64_t f, int64
                   x.size(1) == w.size(1), "gemm_decode: operands");
   const int64_t n = f > 0 ? f : w.size(0);
   TORCH_CHECK(out.size(0) == x.size(0) && out.size(1) >= n && (f == 0 || f_off + f <= w.size(0)), "gemm_decode: shapes");
+  mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0};
+  if (mul.has_value()) {
+    TORCH_CHECK(ids.has_value() && mul->dim() == 2 && mul->stride(1) == 1 && mul->size(1) >= n, "gemm_decode: mul");
+    chk(*mul, BF16, "mul");
+    chk_c(*ids, I32, "ids");
+    TORCH_CHECK(ids->numel() == x.size(0), "gemm_decode: one id per row");
+    tail.mul = mul->data_ptr();
+    tail.mul_ids = ids->data_ptr<int>();
+    tail.ld_mul = mul->stride(0);
+    tail.vocab = (int)mul->size(0);
+  }
   c10::cuda::CUDAGuard guard(x.device());
   mb::gemm_decode(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), of32, out.stride(0),
-                  (int)x.size(0), (int)n, (int)x.size(1), f > 0 ? (int)f_off : 0, (float)alpha, status_ptr(status),
-                  cur_stream());
+                  (int)x.size(0), (int)n, (int)x.size(1), (float)alpha, tail, mb::GemmGroup{}, status_ptr(status), cur_stream());
 }
+
+// out[:, b] = x[:, b] w[b]^T for every b: x [rows, b, K], w [b, N, K], out [rows, b, N], inner strides 1.
+void gemm_heads(const Tensor& x, const Tensor& w, Tensor& out, const OptTensor& status) {
+  const bool f32 = is_f32(x, "x");
+  for (const Tensor* t : {&x, &w, (const Tensor*)&out}) {
+    chk(*t, f32 ? F32 : BF16, "gemm_heads operand");
+    TORCH_CHECK(t->dim() == 3 && t->stride(2) == 1, "gemm_heads: 3-D operands with unit inner stride");
+  }
+  const int64_t rows = x.size(0), b = x.size(1), K = x.size(2), N = w.size(1);
+  TORCH_CHECK(w.size(0) == b && w.size(2) == K && out.size(0) == rows && out.size(1) == b && out.size(2) == N, "gemm_heads: shapes");
+  if (rows == 0) return;
+  c10::cuda::CUDAGuard guard(x.device());
+  if (f32)
+    mb::gemm_f32(x.data_ptr<float>(), x.stride(0), w.data_ptr<float>(), w.stride(1), out.data_ptr<float>(), out.stride(0), (int)rows,
+                 (int)N, (int)K, 1.f, cur_stream(), (int)b, x.stride(1), w.stride(0), out.stride(1));
+  else
+    mb::gemm_decode(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(1), out.data_ptr(), false, out.stride(0), (int)rows, (int)N,
+                    (int)K, 1.f, mb::GemmTail{}, mb::GemmGroup{(int)b, x.stride(1), w.stride(0), out.stride(1), nullptr, 0},
+                    status_ptr(status), cur_stream());
+}
+
+mb::TileList tile_list(const Tensor& tiles, const Tensor& count) {
+  chk_c(tiles, I32, "tiles");
+  chk_c(count, I32, "tile count");
+  TORCH_CHECK(tiles.dim() == 2 && tiles.size(1) == 3 && tiles.size(0) > 0 && count.numel() == 1, "tile list");
+  return mb::TileList{tiles.data_ptr<int>(), count.data_ptr<int>(), (int)tiles.size(0)};
+}
+
+// Row segments that meet a matrix each: out rows = x rows times w[matrix]^T (w [matrices, rows, K]), tiles of tile_rows
+// rows. f > 0: act of the halves (bf16; fp32 operands take the plain product only). 128-row tiles run the prompt-sized
+// kernel, smaller ones the few-token kernel, fp32 operands the fp32 kernel (64-row tiles).
+void gemm_tiles(const Tensor& x, const Tensor& w, Tensor& out, const Tensor& tiles, const Tensor& count, int64_t tile_rows,
+                int64_t f, int64_t f_off, const Act& act, const OptTensor& status) {
+  const bool f32 = is_f32(x, "x");
+  chk(w, f32 ? F32 : BF16, "w");
+  chk(out, f32 ? F32 : BF16, "out");
+  TORCH_CHECK(x.dim() == 2 && x.stride(1) == 1 && w.dim() == 3 && w.stride(2) == 1 && x.size(1) == w.size(2) && out.dim() == 2 &&
+                  out.stride(1) == 1 && out.size(0) == x.size(0), "gemm_tiles: operands");
+  const int64_t n = f > 0 ? f : w.size(1);
+  TORCH_CHECK(out.size(1) >= n && (f == 0 || f_off + f <= w.size(1)), "gemm_tiles: shapes");
+  const mb::TileList list = tile_list(tiles, count);
+  const mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0};
+  c10::cuda::CUDAGuard guard(x.device());
+  if (f32) {
+    TORCH_CHECK(f == 0 && tile_rows == 64, "gemm_tiles: fp32 takes 64-row tiles and no tail");
+    mb::gemm_f32(x.data_ptr<float>(), x.stride(0), w.data_ptr<float>(), w.stride(1), out.data_ptr<float>(), out.stride(0),
+                 (int)x.size(0), (int)n, (int)x.size(1), 1.f, cur_stream(), 1, 0, w.stride(0), 0, &list);
+  } else if (tile_rows == 128) {
+    mb::gemm_segments(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(1), w.stride(0), (int)w.size(0), out.data_ptr(),
+                      out.stride(0), (int)x.size(0), (int)n, (int)x.size(1), tail, list, status_ptr(status), cur_stream());
+  } else {
+    mb::gemm_decode(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(1), out.data_ptr(), false, out.stride(0), (int)x.size(0),
+                    (int)n, (int)x.size(1), 1.f, tail,
+                    mb::GemmGroup{(int)w.size(0), 0, w.stride(0), 0, &list, (int)tile_rows}, status_ptr(status), cur_stream());
+  }
+}
+
+// ---- routed experts: spec = (experts, top, groups, keep)
+using Router = std::tuple<int64_t, int64_t, int64_t, int64_t>;
+struct Routing {
+  mb::RouterSpec s;
+  mb::RouterBuffers b;
+};
+// idx, weight, slot [rows, top]; state: counts [experts + 1] (zeroed once); plan: offset [experts] | tile count
+Routing routing(const Router& r, const Tensor& idx, const Tensor& weight, const Tensor& slot, const Tensor& counts, const Tensor& offset,
+                const Tensor& tiles, const Tensor& count) {
+  for (const Tensor* t : {&idx, &slot, &counts, &offset}) chk_c(*t, I32, "routing buffer");
+  chk_c(weight, F32, "weight");
+  const mb::TileList l = tile_list(tiles, count);
+  Routing out{{(int)std::get<0>(r), (int)std::get<1>(r), (int)std::get<2>(r), (int)std::get<3>(r)}, {}};
+  TORCH_CHECK(idx.dim() == 2 && idx.size(1) == out.s.top && slot.sizes() == idx.sizes() && weight.sizes() == idx.sizes() &&
+                  counts.numel() > out.s.experts && offset.numel() >= out.s.experts, "routing buffers");
+  out.b = {idx.data_ptr<int>(), weight.data_ptr<float>(), slot.data_ptr<int>(), counts.data_ptr<int>(), offset.data_ptr<int>(),
+           const_cast<int*>(l.tiles), const_cast<int*>(l.count), l.max_tiles};
+  return out;
+}
+void expert_select(const Tensor& logits, const Tensor& correction, const Router& r, int64_t tile_rows, Tensor& idx, Tensor& weight,
+                   Tensor& slot, Tensor& counts, Tensor& offset, Tensor& tiles, Tensor& count) {
+  const Routing rt = routing(r, idx, weight, slot, counts, offset, tiles, count);
+  const int64_t rows = idx.size(0);
+  chk_rows(logits, true, rows, rt.s.experts, "logits");
+  TORCH_CHECK(tile_rows > 0 && tiles.size(0) >= std::min<int64_t>(rows * rt.s.top, rt.s.experts + rows * rt.s.top / tile_rows),
+              "expert_select: tile list too short");
+  c10::cuda::CUDAGuard guard(logits.device());
+  mb::expert_select(logits.data_ptr<float>(), logits.stride(0), fptr(correction, rt.s.experts, "correction"), rt.s, rt.b,
+                    (int)tile_rows, (int)rows, cur_stream());
+}
+void expert_gather(const Tensor& h, const Router& r, const Tensor& idx, const Tensor& weight, const Tensor& slot, const Tensor& counts,
+                   const Tensor& offset, const Tensor& tiles, const Tensor& count, Tensor& out, Tensor& row) {
+  const Routing rt = routing(r, idx, weight, slot, counts, offset, tiles, count);
+  const bool f32 = is_f32(h, "h");
+  const int64_t rows = idx.size(0), es = f32 ? 4 : 2;
+  chk_rows(h, f32, rows, 1, "h");
+  chk_c(out, f32 ? F32 : BF16, "out");
+  chk_c(row, I32, "row");
+  TORCH_CHECK(out.dim() == 2 && out.size(0) >= rows * rt.s.top && out.size(1) <= h.size(1) && row.numel() == rows * rt.s.top,
+              "expert_gather: shapes");
+  c10::cuda::CUDAGuard guard(h.device());
+  mb::expert_gather(h.data_ptr(), h.stride(0) * es, rt.s, rt.b, out.data_ptr(), row.data_ptr<int>(), out.size(1) * es, (int)rows,
+                    cur_stream());
+}
+
+void gelu_mul(Tensor& y, const Tensor& table, const Tensor& ids) {
+  const bool f32 = is_f32(y, "y");
+  chk_rows(y, f32, y.size(0), y.size(1), "y");
+  chk_c(ids, I32, "ids");
+  TORCH_CHECK(ids.numel() == y.size(0), "gelu_mul: one id per row");
+  chk(table, f32 ? F32 : BF16, "table");
+  TORCH_CHECK(table.dim() == 2 && table.stride(1) == 1, "gelu_mul: table");
+  c10::cuda::CUDAGuard guard(y.device());
+  mb::gelu_mul(f32, y.data_ptr(), y.stride(0), table.data_ptr(), table.stride(0), ids.data_ptr<int>(), (int)table.size(0),
+               (int)y.size(0), (int)std::min(y.size(1), table.size(1)), cur_stream());
+}
+
+// ---- latent attention of one layer: sizes, offsets in the projection and parameters, built once per layer
+struct Latent {
+  mb::LatentSpec s{};
+  int qr_off = 0, c_off = 0, kr_off = 0;
+  float scale = 1.f, eps = 1e-6f;
+  Tensor gamma, turns, sink;
+
+  mb::LatentPages pages(const Tensor& table, const Tensor& cache, bool f32, int64_t n_seq) const {
+    chk_c(table, I32, "block_table");
+    chk_c(cache, f32 ? F32 : BF16, "cache");
+    TORCH_CHECK(table.dim() == 2 && table.size(0) >= n_seq, "block_table: one row per sequence of the batch");
+    TORCH_CHECK(cache.dim() == 4 && cache.size(2) == 1 && cache.size(3) == s.row(), "cache: [pages, page_size, 1, latent row]");
+    return mb::LatentPages{cache.data_ptr(), table.data_ptr<int>(), (int)table.size(1), (int)cache.size(1), (int)cache.size(0)};
+  }
+  void prep(Tensor& proj, const std::vector<Tensor>& batch, const Tensor& table, const Tensor& cache) const {
+    const auto rb = ragged(batch);
+    const bool f32 = is_f32(proj, "proj");
+    chk_rows(proj, f32, rb.rows, std::max({qr_off + s.heads * s.rot_p, c_off + s.rank_p, kr_off + s.rot_p}), "proj");
+    c10::cuda::CUDAGuard guard(proj.device());
+    mb::latent_prep(f32, proj.data_ptr(), proj.stride(0), qr_off, c_off, kr_off, gamma.data_ptr<float>(),
+                    turns.data_ptr<double>(), s, rb, pages(table, cache, f32, rb.n_seq), eps, cur_stream());
+  }
+  void gather(const Tensor& table, const Tensor& cache, const Tensor& cu_k, int64_t max_kv, Tensor& out) const {
+    chk_c(out, BF16, "out");
+    chk_c(cu_k, I32, "cu_k");
+    TORCH_CHECK(out.dim() == 2 && out.size(1) == s.row(), "gather: out");
+    const int n_seq = (int)cu_k.numel() - 1;
+    c10::cuda::CUDAGuard guard(out.device());
+    mb::latent_gather(s, pages(table, cache, false, n_seq), cu_k.data_ptr<int>(), n_seq, (int)max_kv, out.data_ptr(), cur_stream());
+  }
+  mb::LatentQuery query(const Tensor& q_lat, const Tensor& proj, const Tensor& row_seq, const Tensor& pos, const Tensor& o,
+                        bool f32) const {
+    const int64_t rows = q_lat.size(0);
+    for (const Tensor* t : {&q_lat, &o}) {
+      chk_c(*t, f32 ? F32 : BF16, "q_lat / o");
+      TORCH_CHECK(t->dim() == 3 && t->size(0) == rows && t->size(1) == s.heads && t->size(2) == s.rank_p, "q_lat / o: [rows, heads, rank]");
+    }
+    chk_rows(proj, f32, rows, qr_off + s.heads * s.rot_p, "proj");
+    chk_c(row_seq, I32, "row_seq");
+    chk_c(pos, I32, "pos");
+    TORCH_CHECK(row_seq.numel() == rows && pos.numel() == rows, "row_seq / pos");
+    return mb::LatentQuery{q_lat.data_ptr(), static_cast<const char*>(proj.data_ptr()) + (int64_t)qr_off * (f32 ? 4 : 2), proj.stride(0),
+                           row_seq.data_ptr<int>(), pos.data_ptr<int>(), (int)rows};
+  }
+  void attn_any(const Tensor& q_lat, const Tensor& proj, const Tensor& row_seq, const Tensor& pos, const Tensor& table,
+                const Tensor& cache, Tensor& o) const {
+    const bool f32 = is_f32(q_lat, "q_lat");
+    const auto q = query(q_lat, proj, row_seq, pos, o, f32);
+    c10::cuda::CUDAGuard guard(o.device());
+    mb::latent_attn_any(f32, q, s, pages(table, cache, f32, 0), sink.data_ptr<float>(), o.data_ptr(), scale, cur_stream());
+  }
+  bool decode_ok(int64_t page_size) const { return mb::latent_decode_ok(s, (int)page_size); }
+  void attn_decode(const Tensor& q_lat, const Tensor& proj, const Tensor& row_seq, const Tensor& pos, const Tensor& table,
+                   const Tensor& cache, Tensor& o, Tensor& scratch, Tensor& counters, int64_t splits, const OptTensor& status) const {
+    const auto q = query(q_lat, proj, row_seq, pos, o, false);
+    chk_c(scratch, F32, "scratch");
+    chk_c(counters, I32, "counters");
+    TORCH_CHECK(scratch.numel() >= (int64_t)q.rows * s.heads * splits * (s.rank_p + 2) &&
+                    counters.numel() >= (int64_t)q.rows * ((s.heads + 15) / 16), "attn_decode: scratch");
+    c10::cuda::CUDAGuard guard(o.device());
+    mb::latent_attn_decode(q, s, pages(table, cache, false, 0), sink.data_ptr<float>(), o.data_ptr(), scratch.data_ptr<float>(),
+                           counters.data_ptr<int>(), (int)splits, scale, status_ptr(status), cur_stream());
+  }
+  bool prefill_ok(int64_t dim_p, int64_t vdim_p) const { return mb::flash_attn_ragged_ok((int)dim_p, s.rot_p, (int)vdim_p); }
+  // q, kv: [rows, heads, width] views (unrotated queries; expanded keys and values), latents [keys, row], o [rows, heads, vdim]
+  void attn_prefill(const Tensor& q, const Tensor& proj, const Tensor& k, const Tensor& v, const Tensor& latents,
+                    const std::vector<Tensor>& batch, const Tensor& cu_k, int64_t max_q, int64_t min_q, Tensor& o,
+                    const OptTensor& status) const {
+    const auto rb = ragged(batch);
+    for (const Tensor* t : {&q, &k, &v, (const Tensor*)&o}) {
+      chk(*t, BF16, "attn_prefill operand");
+      TORCH_CHECK(t->dim() == 3 && t->size(1) == s.heads && t->stride(2) == 1 && t->stride(1) == t->size(2), "attn_prefill: [rows, heads, width]");
+    }
+    chk_rows(proj, false, rb.rows, qr_off + s.heads * s.rot_p, "proj");
+    chk_c(latents, BF16, "latents");
+    chk_c(cu_k, I32, "cu_k");
+    TORCH_CHECK(q.size(0) == rb.rows && o.size(0) == rb.rows && k.size(0) == v.size(0) && k.stride(0) == v.stride(0) &&
+                    q.size(2) == k.size(2) && v.size(2) == o.size(2) && proj.stride(0) == q.stride(0) && latents.size(0) == k.size(0) &&
+                    latents.size(1) == s.row() && cu_k.numel() == rb.n_seq + 1, "attn_prefill: shapes");
+    mb::RaggedAttn a{};
+    a.q = q.data_ptr();
+    a.q_rot = static_cast<const char*>(proj.data_ptr()) + (int64_t)qr_off * 2;
+    a.k = k.data_ptr();
+    a.k_rot = static_cast<const char*>(latents.data_ptr()) + (int64_t)s.rank_p * 2;
+    a.v = v.data_ptr();
+    a.o = o.data_ptr();
+    a.ldq = q.stride(0);
+    a.ldkv = k.stride(0);
+    a.ldk_rot = latents.stride(0);
+    a.ldo = o.stride(0);
+    a.cu_q = rb.cu_q;
+    a.cu_k = cu_k.data_ptr<int>();
+    a.kv_lens = rb.kv_lens;
+    a.sink = sink.data_ptr<float>();
+    a.batch = rb.n_seq;
+    a.total_q = rb.rows;
+    a.total_k = (int)k.size(0);
+    a.max_q = (int)max_q;
+    a.min_q = (int)min_q;
+    a.heads = s.heads;
+    a.dim = (int)q.size(2);
+    a.rot = s.rot_p;
+    a.vdim = (int)v.size(2);
+    a.scale = scale;
+    c10::cuda::CUDAGuard guard(o.device());
+    mb::flash_attn_ragged(a, status_ptr(status), cur_stream());
+  }
+};
 
 // h = silu(x w[:f]^T) * (x w[f:2f]^T) in the GEMM's epilogue (prompt-sized batches, f a multiple of 128).
 void gemm_swiglu(const Tensor& x, const Tensor& w, Tensor& h, const OptTensor& status) {
@@ -215,13 +470,13 @@ void gemm_nt(const Tensor& a, const Tensor& b, Tensor& out, double alpha, const 
   }
 }
 
-void silu_gate(const Tensor& gu, int64_t f, int64_t f_off, Tensor& h) {
+void gate_pair(const Tensor& gu, int64_t f, int64_t f_off, const Act& act, Tensor& h) {
   const bool f32 = is_f32(h, "h");
   chk_rows(h, f32, h.size(0), f, "h");
   chk_rows(gu, f32, h.size(0), f_off + f, "gu");
-  TORCH_CHECK(h.stride(0) == h.size(1), "silu_gate: h must be contiguous");
+  TORCH_CHECK(h.stride(0) == h.size(1), "gate_pair: h must be contiguous");
   c10::cuda::CUDAGuard guard(h.device());
-  mb::silu_gate(f32, gu.data_ptr(), gu.stride(0), (int)f, (int)f_off, h.data_ptr(), h.stride(0), (int)h.size(0),
+  mb::gate_pair(f32, gu.data_ptr(), gu.stride(0), (int)f, (int)f_off, gate(act), h.data_ptr(), h.stride(0), (int)h.size(0),
                 cur_stream());
 }
 
@@ -350,15 +605,24 @@ struct Recurrent {
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.doc() = "sm_100a kernels of layer-list models";
   m.def("embed_pos_norm", &embed_pos_norm);
-  m.def("sandwich_norm", &sandwich_norm);
+  namespace py = pybind11;
+  m.def("sandwich_norm", &sandwich_norm, py::arg("y1"), py::arg("y2"), py::arg("w1"), py::arg("w2"), py::arg("w_post"), py::arg("x"),
+        py::arg("w_next"), py::arg("h"), py::arg("eps"), py::arg("mult") = 1.0);
+  m.def("expert_norm", &expert_norm);
   m.def("qk_norm_append", &qk_norm_append);
   m.def("paged_attn_any", &paged_attn_any);
   m.def("paged_attn_prefill", &paged_attn_prefill);
   m.def("paged_attn_decode", &paged_attn_decode);
-  m.def("gemm_decode", &gemm_decode);
+  m.def("gemm_decode", &gemm_decode, py::arg("x"), py::arg("w"), py::arg("out"), py::arg("f"), py::arg("f_off"), py::arg("alpha"),
+        py::arg("status"), py::arg("act") = Act(0, 0.0, 0.0), py::arg("mul") = OptTensor(), py::arg("ids") = OptTensor());
+  m.def("gemm_heads", &gemm_heads);
+  m.def("gemm_tiles", &gemm_tiles);
+  m.def("expert_select", &expert_select);
+  m.def("expert_gather", &expert_gather);
+  m.def("gelu_mul", &gelu_mul);
+  m.def("gate_pair", &gate_pair);
   m.def("gemm_swiglu", &gemm_swiglu);
   m.def("gemm_nt", &gemm_nt);
-  m.def("silu_gate", &silu_gate);
   m.def("sample_tokens", &sample_tokens);
   pybind11::class_<Recurrent>(m, "Recurrent")
       .def(pybind11::init([](pybind11::dict spec, pybind11::dict tensors) {
@@ -402,5 +666,34 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
       .def("scan_chunked", &Recurrent::scan_chunked)
       .def("decode", &Recurrent::decode)
       .def("norm_gate", &Recurrent::norm_gate);
+  py::class_<Latent>(m, "Latent")
+      .def(py::init([](py::dict d, const Tensor& gamma, const Tensor& turns, const Tensor& sink) {
+        Latent l;
+        auto geti = [&](const char* k) { return d[k].cast<int>(); };
+        l.s = mb::LatentSpec{geti("heads"), geti("rank"), geti("rot"), geti("rank_p"), geti("rot_p")};
+        TORCH_CHECK(l.s.heads > 0 && l.s.rank > 0 && l.s.rot > 0 && l.s.rank_p >= l.s.rank && l.s.rot_p >= l.s.rot &&
+                        l.s.rank_p % 8 == 0 && l.s.rot_p % 8 == 0, "latent: sizes");
+        l.qr_off = geti("qr_off");
+        l.c_off = geti("c_off");
+        l.kr_off = geti("kr_off");
+        TORCH_CHECK((l.qr_off | l.c_off | l.kr_off) % 8 == 0, "latent: offsets");
+        l.scale = d["scale"].cast<float>();
+        l.eps = d["eps"].cast<float>();
+        fptr(gamma, l.s.rank, "gamma");
+        fptr(sink, l.s.heads, "sink");
+        chk_c(turns, torch::kFloat64, "turns");
+        TORCH_CHECK(turns.numel() >= l.s.rot / 2, "latent: turns");
+        l.gamma = gamma;
+        l.turns = turns;
+        l.sink = sink;
+        return l;
+      }))
+      .def("prep", &Latent::prep)
+      .def("gather", &Latent::gather)
+      .def("attn_any", &Latent::attn_any)
+      .def("decode_ok", &Latent::decode_ok)
+      .def("attn_decode", &Latent::attn_decode)
+      .def("prefill_ok", &Latent::prefill_ok)
+      .def("attn_prefill", &Latent::attn_prefill);
   m.def("launch_count", []() { return (int64_t)mb::launch_counter().load(); });
 }

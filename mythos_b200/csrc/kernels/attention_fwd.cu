@@ -21,11 +21,11 @@ namespace {
 constexpr int FA_THREADS = 320;
 constexpr int FA_BM = 128;  // query rows per tile (two tiles per CTA)
 constexpr int FA_BN = 64;   // kv rows per step
-constexpr int FA_STAGES = 3;
 
 // DK: width of queries and keys, DV: width of values and outputs.
 template <int DK, int DV>
 struct FaFwdCfg {
+  static constexpr int STAGES = DK > 128 ? 2 : 3;
   static constexpr int Q_BYTES = FA_BM * DK * 2;
   static constexpr int K_BYTES = FA_BN * DK * 2;
   static constexpr int V_BYTES = FA_BN * DV * 2;
@@ -33,21 +33,29 @@ struct FaFwdCfg {
   static constexpr int P_BYTES = FA_BM * FA_BN * 2;
   static constexpr int OFF_Q = 0;
   static constexpr int OFF_KV = 2 * Q_BYTES;
-  static constexpr int OFF_P = OFF_KV + FA_STAGES * STAGE_BYTES;
+  static constexpr int OFF_P = OFF_KV + STAGES * STAGE_BYTES;
   static constexpr int OFF_BAR = OFF_P + 2 * P_BYTES;
-  static constexpr int NUM_BARS = 1 + 2 * FA_STAGES + 6;
+  static constexpr int NUM_BARS = 1 + 2 * STAGES + 6;
   static constexpr int SMEM_BYTES = OFF_BAR + NUM_BARS * 8 + 16 + 1024;
   static constexpr int TMEM_COLS = (DV == 128) ? 512 : 256;
   static constexpr int COL_S = 0;    // S0 at 0, S1 at 64
   static constexpr int COL_O = 128;  // O0 at 128, O1 at 128 + DV
 };
 
-// PAGED: prefill attention whose K/V live in the paged cache. Queries are the new tokens of each
+// MODE FA_PAGED: prefill attention whose K/V live in the paged cache. Queries are the new tokens of each
 // sequence, packed one sequence after another ([total_q, heads, D], sequence b = rows cu_q[b] ..
 // cu_q[b+1]); keys / values are read page by page (16 tokens each) through the block table, one TMA
 // box per page and 64-wide chunk, landing in the same swizzled tiles as the contiguous loads. The
 // first query of sequence b sits at position kv_lens[b] - q_len, so the kernel serves a whole prompt
 // (offset 0), one chunk of a long prompt, the remainder after a cached prefix, and ragged batches.
+//
+// MODE FA_RAGGED: the same packed queries over packed keys and values (sequence b at rows cu_k[b] ..), keys
+// and values per query head. The last DR columns of queries and keys are a second pair of tensors: a part
+// of the key that all heads share (one row per token). Widths below a multiple of 64 are filled with zeros
+// by TMA. Sequences with fewer than min_q new tokens are left out.
+//
+// sink (FA_PAGED and FA_RAGGED, may be null): one more logit per head in the softmax denominator.
+enum { FA_DENSE = 0, FA_PAGED = 1, FA_RAGGED = 2 };
 struct PagedPrefillArgs {
   const int* block_table;   // [batch, table_stride] page ids
   const int* cu_q;          // [batch + 1] first query row of every sequence
@@ -55,24 +63,29 @@ struct PagedPrefillArgs {
   int table_stride;
   const __nv_bfloat16* gate;   // [total_q, >= heads] logits of a per-head output gate (sigmoid), or null
   long long ld_gate;
+  const float* sink;           // [heads]
+  const int* cu_k;             // FA_RAGGED: first key row of every sequence
+  int min_q, o_cols;           // FA_RAGGED: see above; output columns of a head
 };
 constexpr int FA_PAGE = 16;
 
-template <int DK, int DV, bool PAGED>
+template <int DK, int DV, int MODE, int DR = 0>
 __global__ void __launch_bounds__(FA_THREADS, 1)
 fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
               const __grid_constant__ CUtensorMap tm_v, __nv_bfloat16* __restrict__ o, float* __restrict__ lse,
               int seq, int heads, int kv_heads, long long o_tok_stride, int causal, float scale_log2, int* status,
-              PagedPrefillArgs pa) {
+              PagedPrefillArgs pa, const __grid_constant__ CUtensorMap tm_q2, const __grid_constant__ CUtensorMap tm_k2) {
   using Cfg = FaFwdCfg<DK, DV>;
-  constexpr int DCK = DK / 64, DCV = DV / 64;  // 64-wide chunks of the head widths
+  constexpr bool PAGED = MODE != FA_DENSE;     // packed queries
+  constexpr int STAGES = Cfg::STAGES;
+  constexpr int DCK = (DK - DR) / 64, DCR = DR / 64, DCV = DV / 64;  // 64-wide chunks of the head widths
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Cfg::OFF_BAR);
   uint64_t* q_full = bars;
   uint64_t* kv_full = bars + 1;
-  uint64_t* kv_empty = kv_full + FA_STAGES;
-  uint64_t* s_full = kv_empty + FA_STAGES;
+  uint64_t* kv_empty = kv_full + STAGES;
+  uint64_t* s_full = kv_empty + STAGES;
   uint64_t* p_full = s_full + 2;
   uint64_t* o_done = p_full + 2;
   uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(o_done + 2);
@@ -91,6 +104,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
     kv_len = pa.kv_lens[b];
     q_off = kv_len - q_len;
     if (q0 >= q_len) return;                     // uniform over the CTA, before any barrier exists
+    if (MODE == FA_RAGGED && q_len < pa.min_q) return;
   }
   const int n_qt = (q0 + FA_BM < q_len) ? 2 : 1;
   int J[2];
@@ -103,7 +117,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
-    for (int s = 0; s < FA_STAGES; ++s) {
+    for (int s = 0; s < STAGES; ++s) {
       mbar_init(&kv_full[s], 1);
       mbar_init(&kv_empty[s], 1);
     }
@@ -135,14 +149,24 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
         for (int c = 0; c < DCK; ++c)
           tma_load_4d(smem + Cfg::OFF_Q + t * Cfg::Q_BYTES + c * (FA_BM * 128), &tm_q, q_full, c * 64, h,
                       q_row0 + q0 + t * FA_BM, PAGED ? 0 : b);
+      if constexpr (DCR > 0)
+        for (int t = 0; t < 2; ++t)
+          for (int c = 0; c < DCR; ++c)
+            tma_load_4d(smem + Cfg::OFF_Q + t * Cfg::Q_BYTES + (DCK + c) * (FA_BM * 128), &tm_q2, q_full, c * 64, h,
+                        q_row0 + q0 + t * FA_BM, 0);
       for (int j = 0; j < Jmax; ++j) {
-        const int st = j % FA_STAGES;
-        const uint32_t ph = (j / FA_STAGES) & 1;
+        const int st = j % STAGES;
+        const uint32_t ph = (j / STAGES) & 1;
         if (!mbar_wait(&kv_empty[st], ph ^ 1, abort_flag, status, 11)) break;
         mbar_arrive_expect_tx(&kv_full[st], Cfg::STAGE_BYTES);
         uint8_t* sk = smem + Cfg::OFF_KV + st * Cfg::STAGE_BYTES;
         uint8_t* sv = sk + Cfg::K_BYTES;
-        if constexpr (PAGED) {
+        if constexpr (MODE == FA_RAGGED) {
+          const int row = pa.cu_k[b] + j * FA_BN;
+          for (int c = 0; c < DCK; ++c) tma_load_4d(sk + c * (FA_BN * 128), &tm_k, &kv_full[st], c * 64, h, row, 0);
+          for (int c = 0; c < DCR; ++c) tma_load_4d(sk + (DCK + c) * (FA_BN * 128), &tm_k2, &kv_full[st], c * 64, 0, row, 0);
+          for (int c = 0; c < DCV; ++c) tma_load_4d(sv + c * (FA_BN * 128), &tm_v, &kv_full[st], c * 64, h, row, 0);
+        } else if constexpr (PAGED) {
           // four pages of 16 tokens per kv tile; pages past the sequence's end (never visible: the
           // causal limit masks them) read page 0 so that the transaction count stays fixed
           const int* row = pa.block_table + (long long)b * pa.table_stride;
@@ -174,7 +198,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       const uint32_t p_addr = smem_u32(smem + Cfg::OFF_P);
       auto issue_s = [&](int t, int j) {
         const uint32_t qa = q_addr + t * Cfg::Q_BYTES;
-        const uint32_t ka = kv_addr + (j % FA_STAGES) * Cfg::STAGE_BYTES;
+        const uint32_t ka = kv_addr + (j % STAGES) * Cfg::STAGE_BYTES;
 #pragma unroll
         for (int k = 0; k < DK / 16; ++k) {
           const int c = k >> 2, kk = k & 3;
@@ -185,7 +209,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       };
       auto issue_pv = [&](int t, int j) {
         const uint32_t pa = p_addr + t * Cfg::P_BYTES;
-        const uint32_t va = kv_addr + (j % FA_STAGES) * Cfg::STAGE_BYTES + Cfg::K_BYTES;
+        const uint32_t va = kv_addr + (j % STAGES) * Cfg::STAGE_BYTES + Cfg::K_BYTES;
 #pragma unroll
         for (int k = 0; k < FA_BN / 16; ++k) {
           umma_f16(tmem_base + Cfg::COL_O + t * DV, umma_desc_sw128(pa + k * 32, 0, 1024),
@@ -209,11 +233,11 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
           tc_fence_after();
           issue_pv(t, j);
           const bool last_user = (t == 1) || (j >= J[1]);
-          if (last_user) umma_commit(&kv_empty[j % FA_STAGES]);
+          if (last_user) umma_commit(&kv_empty[j % STAGES]);
           if (j + 1 < J[t]) {
             if (have_next && !next_ready) {
-              const int st = (j + 1) % FA_STAGES;
-              if (!mbar_wait(&kv_full[st], ((j + 1) / FA_STAGES) & 1, abort_flag, status, 15)) { ok = false; break; }
+              const int st = (j + 1) % STAGES;
+              if (!mbar_wait(&kv_full[st], ((j + 1) / STAGES) & 1, abort_flag, status, 15)) { ok = false; break; }
               tc_fence_after();
               next_ready = true;
             }
@@ -310,13 +334,16 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       ok = __all_sync(0xffffffffu, ok);
       if (ok) {
         tc_fence_after();
+        if constexpr (PAGED) {
+          if (pa.sink) l += exp2f(pa.sink[h] * 1.4426950408889634f - m_ref);
+        }
         float inv_l = l > 0.f ? 1.f / l : 0.f;
         if constexpr (PAGED) {
           if (pa.gate && q_row < q_len)
             inv_l /= 1.f + expf(-__bfloat162float(pa.gate[(long long)(q_row0 + q_row) * pa.ld_gate + h]));
         }
         __nv_bfloat16* orow = o + (PAGED ? (long long)(q_row0 + q_row) : (long long)b * seq + q_row) * o_tok_stride +
-                              (long long)h * DV;
+                              (long long)h * (MODE == FA_RAGGED ? pa.o_cols : DV);
 #pragma unroll 1
         for (int c = 0; c < DV / 32; ++c) {
           uint32_t orr[32];
@@ -331,7 +358,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
               v.y = pack_bf16x2(__uint_as_float(orr[8 * i + 2]) * inv_l, __uint_as_float(orr[8 * i + 3]) * inv_l);
               v.z = pack_bf16x2(__uint_as_float(orr[8 * i + 4]) * inv_l, __uint_as_float(orr[8 * i + 5]) * inv_l);
               v.w = pack_bf16x2(__uint_as_float(orr[8 * i + 6]) * inv_l, __uint_as_float(orr[8 * i + 7]) * inv_l);
-              p4[i] = v;
+              if (MODE != FA_RAGGED || c * 32 + i * 8 < pa.o_cols) p4[i] = v;
             }
           }
         }
@@ -388,23 +415,23 @@ void flash_attn_fwd_strided(const void* q, const void* k, const void* v, void* o
   if (head_dim == 128) {
     static bool configured = false;
     if (!configured) {
-      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<128, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<128, 128, FA_DENSE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          FaFwdCfg<128, 128>::SMEM_BYTES));
       configured = true;
     }
-    fa_fwd_kernel<128, 128, false><<<grid, FA_THREADS, FaFwdCfg<128, 128>::SMEM_BYTES, stream>>>(
+    fa_fwd_kernel<128, 128, FA_DENSE><<<grid, FA_THREADS, FaFwdCfg<128, 128>::SMEM_BYTES, stream>>>(
         tq, tk, tv, (__nv_bfloat16*)o, lse, seq, heads, kv_heads, o_tok_stride, causal ? 1 : 0, scale_log2, status,
-        PagedPrefillArgs{});
+        PagedPrefillArgs{}, tq, tk);
   } else {
     static bool configured = false;
     if (!configured) {
-      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<64, 64, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+      MB_CUDA_CHECK(cudaFuncSetAttribute(fa_fwd_kernel<64, 64, FA_DENSE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          FaFwdCfg<64, 64>::SMEM_BYTES));
       configured = true;
     }
-    fa_fwd_kernel<64, 64, false><<<grid, FA_THREADS, FaFwdCfg<64, 64>::SMEM_BYTES, stream>>>(
+    fa_fwd_kernel<64, 64, FA_DENSE><<<grid, FA_THREADS, FaFwdCfg<64, 64>::SMEM_BYTES, stream>>>(
         tq, tk, tv, (__nv_bfloat16*)o, lse, seq, heads, kv_heads, o_tok_stride, causal ? 1 : 0, scale_log2, status,
-        PagedPrefillArgs{});
+        PagedPrefillArgs{}, tq, tk);
   }
   count_launch();
   check_launch();
@@ -431,16 +458,51 @@ void flash_attn_paged_prefill(const void* q, long long q_tok_stride, const void*
   const CUtensorMap tk = page_map(k_cache, dk), tv = page_map(v_cache, dv);
   const dim3 grid((max_q_len + 2 * FA_BM - 1) / (2 * FA_BM), heads, batch);
   const float scale_log2 = scale * 1.4426950408889634f;
-  PagedPrefillArgs pa{block_table, cu_q, kv_lens, table_stride, (const __nv_bfloat16*)gate, ld_gate};
+  PagedPrefillArgs pa{block_table, cu_q, kv_lens, table_stride, (const __nv_bfloat16*)gate, ld_gate, nullptr, nullptr, 0, dv};
   auto go = [&](auto kern, int smem) {
     MB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     kern<<<grid, FA_THREADS, smem, stream>>>(tq, tk, tv, (__nv_bfloat16*)o, nullptr, total_q, heads, kv_heads,
-                                             o_tok_stride, 1, scale_log2, status, pa);
+                                             o_tok_stride, 1, scale_log2, status, pa, tq, tk);
   };
-  if (dk == 128 && dv == 128) go(fa_fwd_kernel<128, 128, true>, FaFwdCfg<128, 128>::SMEM_BYTES);
-  else if (dk == 64 && dv == 128) go(fa_fwd_kernel<64, 128, true>, FaFwdCfg<64, 128>::SMEM_BYTES);
-  else if (dk == 128 && dv == 64) go(fa_fwd_kernel<128, 64, true>, FaFwdCfg<128, 64>::SMEM_BYTES);
-  else go(fa_fwd_kernel<64, 64, true>, FaFwdCfg<64, 64>::SMEM_BYTES);
+  if (dk == 128 && dv == 128) go(fa_fwd_kernel<128, 128, FA_PAGED>, FaFwdCfg<128, 128>::SMEM_BYTES);
+  else if (dk == 64 && dv == 128) go(fa_fwd_kernel<64, 128, FA_PAGED>, FaFwdCfg<64, 128>::SMEM_BYTES);
+  else if (dk == 128 && dv == 64) go(fa_fwd_kernel<128, 64, FA_PAGED>, FaFwdCfg<128, 64>::SMEM_BYTES);
+  else go(fa_fwd_kernel<64, 64, FA_PAGED>, FaFwdCfg<64, 64>::SMEM_BYTES);
+  count_launch();
+  check_launch();
+}
+
+bool flash_attn_ragged_ok(int dim, int rot, int vdim) { return dim <= 128 && rot <= 64 && vdim <= 128; }
+
+void flash_attn_ragged(const RaggedAttn& a, int* status, cudaStream_t stream) {
+  MB_REQUIRE(flash_attn_ragged_ok(a.dim, a.rot, a.vdim), "flash_attn_ragged: head widths up to 128 + 64 and 128");
+  MB_REQUIRE((a.dim | a.rot | a.vdim) % 8 == 0 && a.dim > 0 && a.rot > 0 && a.vdim > 0, "flash_attn_ragged: widths in units of 8");
+  MB_REQUIRE((reinterpret_cast<uintptr_t>(a.o) & 15) == 0 && a.ldo % 8 == 0, "flash_attn_ragged: output alignment");
+  if (a.batch == 0 || a.total_q == 0 || a.total_k == 0 || a.max_q == 0) return;
+  // token-major [rows, heads, width] views: one box = 64 columns of one head
+  auto map = [](const void* base, int rows, int heads, int width, long long ld, int box_rows) {
+    uint64_t dims[4] = {(uint64_t)width, (uint64_t)heads, (uint64_t)rows, 1};
+    uint64_t strides[3] = {(uint64_t)(heads > 1 ? width : ld) * 2, (uint64_t)ld * 2, (uint64_t)rows * ld * 2};
+    uint32_t box[4] = {64, 1, (uint32_t)box_rows, 1};
+    return make_tensor_map(base, TmaDType::BF16, 4, dims, strides, box, true);
+  };
+  const CUtensorMap tq = map(a.q, a.total_q, a.heads, a.dim, a.ldq, FA_BM), tq2 = map(a.q_rot, a.total_q, a.heads, a.rot, a.ldq, FA_BM);
+  const CUtensorMap tk = map(a.k, a.total_k, a.heads, a.dim, a.ldkv, FA_BN), tv = map(a.v, a.total_k, a.heads, a.vdim, a.ldkv, FA_BN);
+  const CUtensorMap tk2 = map(a.k_rot, a.total_k, 1, a.rot, a.ldk_rot, FA_BN);
+  const dim3 grid((a.max_q + 2 * FA_BM - 1) / (2 * FA_BM), a.heads, a.batch);
+  PagedPrefillArgs pa{nullptr, a.cu_q, a.kv_lens, 0, nullptr, 0, a.sink, a.cu_k, a.min_q, a.vdim};
+  auto go = [&](auto kern, int smem) {
+    MB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    kern<<<grid, FA_THREADS, smem, stream>>>(tq, tk, tv, (__nv_bfloat16*)a.o, nullptr, a.total_q, a.heads, a.heads, a.ldo, 1,
+                                             a.scale * 1.4426950408889634f, status, pa, tq2, tk2);
+  };
+#define MB_FR(DK, DV) go(fa_fwd_kernel<DK, DV, FA_RAGGED, 64>, FaFwdCfg<DK, DV>::SMEM_BYTES)
+  if (a.dim <= 64) {
+    if (a.vdim <= 64) MB_FR(128, 64); else MB_FR(128, 128);
+  } else {
+    if (a.vdim <= 64) MB_FR(192, 64); else MB_FR(192, 128);
+  }
+#undef MB_FR
   count_launch();
   check_launch();
 }

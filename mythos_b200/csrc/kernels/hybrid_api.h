@@ -1,6 +1,7 @@
 // Launch API of the kernels behind layer-list ("hybrid") models: gated linear attention and gated
-// delta-rule recurrences, attention with unequal key / value widths and per-head output gates,
-// sandwich RMSNorms on a 32-bit residual stream, and the GEMMs those models need beside gemm.cu.
+// delta-rule recurrences, attention with unequal key / value widths and per-head output gates, attention
+// over a cached latent, routed experts, RMSNorms around sublayers on a 32-bit residual stream, and the
+// GEMMs those models need beside gemm.cu.
 // Same conventions as api.h (raw pointers, asynchronous on `stream`, exceptions on bad arguments).
 // `f32` selects the activation type: false = bf16 (serving), true = 32-bit floats throughout.
 #pragma once
@@ -17,15 +18,25 @@ struct RaggedBatch {
   int n_seq, rows;
 };
 
-// x[t] = embed[id] * scale + pos_table[pos] (fp32 stream), h[t] = rmsnorm(x[t]) * gamma.
+// x[t] = embed[id] * scale + pos_table[pos] (fp32 stream; the table may be null),
+// h[t] = rmsnorm(x[t]) * gamma, or x[t] with gamma null.
 void embed_pos_norm(bool f32, const int* ids, const int* pos, const void* embed, const void* pos_table, int vocab,
                     int max_pos, float scale, const float* gamma, float* x, void* h, long long ldh, int rows, int dim,
                     float eps, cudaStream_t stream);
 
-// y = y1, or with y2: (rms(y1) * w1 + rms(y2) * w2) / 2.  x += rms(y) * w_post;  h = rms(x) * w_next.
-void sandwich_norm(bool f32, const void* y1, const void* y2, long long ldy, const float* w1, const float* w2,
-                   const float* w_post, float* x, const float* w_next, void* h, long long ldh, int rows, int dim,
-                   float eps, cudaStream_t stream);
+// Output of a sublayer: y1 alone; (rms(y1) * w1 + rms(y2) * w2) / 2; or the sum over j < top of
+// weight[t, j] * y1[row[t, j]] (routed experts).
+struct SublayerOut {
+  const void *y1, *y2;
+  long long ld;
+  const float *w1, *w2;
+  const int* row;
+  const float* weight;
+  int top;
+};
+// x += mult * rms(y) * w_post;  h = rms(x) * w_next, or x with w_next null.
+void sandwich_norm(bool f32, const SublayerOut& y, const float* w_post, float mult, float* x, const float* w_next, void* h,
+                   long long ldh, int rows, int dim, float eps, cudaStream_t stream);
 
 // Per-head RMSNorm of q and k, q written out, k and v stored into their pages (key width dk, value width dv).
 void qk_norm_append(bool f32, const void* proj, long long ld, int q_off, int k_off, int v_off, const float* q_gamma,
@@ -40,18 +51,112 @@ void paged_attn_any(bool f32, const void* q, const void* k_cache, const void* v_
                     const int* block_table, int table_stride, int page_size, const void* gate, long long ld_gate,
                     void* o, long long ldo, int heads, int kv_heads, int dk, int dv, float scale, cudaStream_t stream);
 
-// C[M, N] = alpha * A[M, K] B[N, K]^T, all fp32, no reduced-precision mode.
+// Segments of rows that meet a weight matrix each: tiles[i] = (matrix, first row, rows), *count of them.
+struct TileList {
+  const int *tiles, *count;
+  int max_tiles;
+};
+
+// C[M, N] = alpha * A[M, K] B[N, K]^T, all fp32, no reduced-precision mode. batch > 1: that many products, the
+// operands of each `*_batch` elements further. With `list` (64-row tiles) row segments meet the matrix they name.
 void gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N,
-              int K, float alpha, cudaStream_t stream);
+              int K, float alpha, cudaStream_t stream, int batch = 1, long long a_batch = 0, long long b_batch = 0,
+              long long c_batch = 0, const TileList* list = nullptr);
 
-// y = alpha * x W^T for a few tokens (bf16 in, bf16 or fp32 out), reduction split over a cluster. f_off > 0: W holds
-// a gate matrix in rows [0, N) and an up matrix from row f_off; y = silu(gate) * up.
+// Gated feed-forward activations: what a gate value g does to its up value u.
+struct GateAct {
+  int kind;                 // 0: silu(g) u   1: relu(g) u   2: g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit),
+  float limit, alpha;       //    u' = u clamped to [-limit, limit]
+};
+// What a few-token GEMM does with the products of a row: nothing; a gated activation of two halves of W; or
+// gelu_tanh(y) * mul[mul_ids[t] * ld_mul + n].
+struct GemmTail {
+  int f_off;                // > 0: W holds a gate matrix in rows [0, N) and an up matrix from row f_off
+  GateAct act;
+  const void* mul;
+  const int* mul_ids;
+  long long ld_mul;
+  int vocab;                // rows of mul
+};
+// Several products in one launch: `batch` of them side by side (x, W and out advance by *_batch elements), or with
+// `list` (tile rows = mt: 16, 32, 64 or 128) rows grouped by matrix, W advancing by w_batch elements.
+struct GemmGroup {
+  int batch;
+  long long x_batch, w_batch, out_batch;
+  const TileList* list;
+  int mt;
+};
+// y = alpha * x W^T for a few tokens (bf16 in, bf16 or fp32 out), reduction split over a cluster.
 void gemm_decode(const void* x, long long ldx, const void* W, long long ldw, void* out, bool out_f32, long long ldo, int M,
-                 int N, int K, int f_off, float alpha, int* status, cudaStream_t stream);
+                 int N, int K, float alpha, const GemmTail& tail, const GemmGroup& group, int* status, cudaStream_t stream);
 
-// h = silu(gu[:, :f]) * gu[:, f_off : f_off + f]
-void silu_gate(bool f32, const void* gu, long long ldg, int f, int f_off, void* h, long long ldh, int rows,
+// The same products for prompt-sized row segments: persistent 128-token x 256-weight-row tiles (128 of each half with
+// a gated tail), bf16 out. `list` has 128-row tiles; total_rows: rows of x.
+void gemm_segments(const void* x, long long ldx, const void* W, long long ldw, long long w_batch, int matrices, void* out,
+                   long long ldo, int total_rows, int N, int K, const GemmTail& tail, const TileList& list, int* status,
+                   cudaStream_t stream);
+
+// h = act(gu[:, :f], gu[:, f_off : f_off + f])
+void gate_pair(bool f32, const void* gu, long long ldg, int f, int f_off, const GateAct& act, void* h, long long ldh, int rows,
                cudaStream_t stream);
+// y[t, n] = gelu_tanh(y[t, n]) * table[ids[t] * ld_table + n], n < width
+void gelu_mul(bool f32, void* y, long long ldy, const void* table, long long ld_table, const int* ids, int vocab, int rows,
+              int width, cudaStream_t stream);
+
+// ---- routed experts (expert_route.cu)
+struct RouterSpec {
+  int experts, top, groups, keep;
+};
+struct RouterBuffers {
+  int* idx;                 // [rows, top] chosen expert
+  float* weight;            // [rows, top] its score
+  int* slot;                // [rows, top] place within the expert's segment
+  int* counts;              // [experts + 1], zero before the first launch and left zero by every launch
+  int* offset;              // [experts] first row of the segment
+  int *tiles, *tile_count;  // tile list for `tile_rows` rows a tile
+  int max_tiles;
+};
+// Softmax scores of fp32 logits, choice by score + correction within the best groups, row segments per expert.
+void expert_select(const float* logits, long long ldz, const float* correction, const RouterSpec& s, const RouterBuffers& b,
+                   int tile_rows, int rows, cudaStream_t stream);
+// Rows of h (row_bytes each, a multiple of 16) into their segments; row[t, j] = where (t, j) went.
+void expert_gather(const void* h, long long ldh_bytes, const RouterSpec& s, const RouterBuffers& b, void* out, int* row,
+                   long long row_bytes, int rows, cudaStream_t stream);
+
+// ---- attention over a cached latent (latent.cu): a page row holds [latent | rotated key part], each padded to a
+// multiple of 8 values with zeros; all heads read the same rows.
+struct LatentSpec {
+  int heads, rank, rot, rank_p, rot_p;   // widths and their padded forms
+  __host__ __device__ int row() const { return rank_p + rot_p; }
+};
+struct LatentPages {
+  void* cache;              // [pages, page_size, row]
+  const int* table;
+  int stride, page_size, pages;
+};
+// Latent norm, rotation of the key part and of the queries' rotated columns (in place), append to the pages.
+// turns[i]: revolutions per position of pair i.
+void latent_prep(bool f32, void* proj, long long ld, int qr_off, int c_off, int kr_off, const float* gamma,
+                 const double* turns, const LatentSpec& s, const RaggedBatch& rb, const LatentPages& pg, float eps,
+                 cudaStream_t stream);
+// Latent rows of the sequences' pages, packed: sequence b at rows cu_k[b] .. cu_k[b + 1] of out.
+void latent_gather(const LatentSpec& s, const LatentPages& pg, const int* cu_k, int n_seq, int max_kv, void* out,
+                   cudaStream_t stream);
+// Queries of single tokens: q_lat [rows, heads, rank_p] (unrotated part taken into the latent's space) and the rotated
+// part at qr + t * ld_qr + h * rot_p; token t sees positions 0 .. pos[t] of sequence row_seq[t].
+struct LatentQuery {
+  const void* q_lat;
+  const void* qr;
+  long long ld_qr;
+  const int *row_seq, *pos;
+  int rows;
+};
+// out [rows, heads, rank_p]: softmax-weighted latents, with exp(sink[h]) in the denominator.
+void latent_attn_any(bool f32, const LatentQuery& q, const LatentSpec& s, const LatentPages& pg, const float* sink, void* out,
+                     float scale, cudaStream_t stream);
+bool latent_decode_ok(const LatentSpec& s, int page_size);
+void latent_attn_decode(const LatentQuery& q, const LatentSpec& s, const LatentPages& pg, const float* sink, void* out,
+                        float* scratch, int* counters, int splits, float scale, int* status, cudaStream_t stream);
 
 // ---- recurrences: S <- diag(g) S ; u = beta (v - S^T k) or u = v ; S <- S + k u^T ; o = S^T q
 // State layout: [slot][head][vdim][dim] fp32 (a row of S^T is contiguous).

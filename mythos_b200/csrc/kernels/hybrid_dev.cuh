@@ -2,6 +2,8 @@
 #pragma once
 #include <cuda_bf16.h>
 
+#include "hybrid_api.h"
+
 namespace mb {
 
 __device__ __forceinline__ float ldf(const float* p) { return *p; }
@@ -12,5 +14,16 @@ __device__ __forceinline__ void stf(__nv_bfloat16* p, float v) { *p = __float2bf
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
+__device__ __forceinline__ float gate_act(const GateAct& a, float g, float u) {
+  if (a.kind == 0) return silu_f(g) * u;
+  if (a.kind == 1) return fmaxf(g, 0.f) * u;
+  g = fminf(g, a.limit);
+  u = fminf(fmaxf(u, -a.limit), a.limit);
+  return g * sigmoid_f(a.alpha * g) * (u + 1.f);
+}
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
 
 }  // namespace mb

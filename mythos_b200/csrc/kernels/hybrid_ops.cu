@@ -1,8 +1,9 @@
 // Pointwise, normalisation and any-shape kernels of the layer-list models (hybrid_api.h).
 //
 // The residual stream is fp32. A sublayer's output is normalised before it is added ("sandwich"
-// norms), and the next sublayer's input norm reads the sum, so one kernel does post-norm, residual
-// add and pre-norm of a row; for two mixers side by side it also normalises and averages the two.
+// norms), and the next sublayer reads the sum (through a norm of its own, or as it is), so one kernel
+// does post-norm, residual add and pre-norm of a row; for two mixers side by side it also normalises and
+// averages the two, and for routed experts it forms the weighted sum of their outputs.
 #include "common.cuh"
 #include "hybrid_api.h"
 #include "hybrid_dev.cuh"
@@ -65,18 +66,20 @@ __device__ __forceinline__ void stv(__nv_bfloat16* p, const float (&f)[V]) {
   }
 }
 
-// h = rms(row) * gamma for a row held in shared memory; columns [dim, ldh) are zeroed (GEMM padding).
+// h = rms(row) * gamma (or the row itself) for a row held in shared memory; columns [dim, ldh) are zeroed (GEMM padding).
 template <typename T, int V>
 __device__ __forceinline__ void write_normed(const float* row, float ss, const float* gamma, T* h, long long ldh,
                                              int dim, float eps) {
   const float r = 1.f / sqrtf(ss / (float)dim + eps);
   for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
-    float x[V], g[V], y[V];
+    float x[V], g[V];
     ldv<V>(row + i, x);
-    ldv<V>(gamma + i, g);
+    if (gamma) {
+      ldv<V>(gamma + i, g);
 #pragma unroll
-    for (int j = 0; j < V; ++j) y[j] = x[j] * r * g[j];
-    stv<V>(h + i, y);
+      for (int j = 0; j < V; ++j) x[j] *= r * g[j];
+    }
+    stv<V>(h + i, x);
   }
   for (int i = dim + threadIdx.x; i < ldh; i += SN_THREADS) stf(h + i, 0.f);
 }
@@ -113,25 +116,51 @@ embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ pos, 
   write_normed<T, V>(row, ss, gamma, h + t * ldh, ldh, dim, eps);
 }
 
-template <typename T, int V, bool TWO>
+enum { SUB_ONE, SUB_TWO, SUB_EXPERTS };
+constexpr int SN_MAX_TOP = 32;
+
+template <typename T, int V, int SRC>
 __global__ void __launch_bounds__(SN_THREADS)
-sandwich_norm_kernel(const T* __restrict__ y1, const T* __restrict__ y2, long long ldy, const float* __restrict__ w1,
-                     const float* __restrict__ w2, const float* __restrict__ w_post, float* __restrict__ x,
+sandwich_norm_kernel(SublayerOut src, const float* __restrict__ w_post, float mult, float* __restrict__ x,
                      const float* __restrict__ w_next, T* __restrict__ h, long long ldh, int dim, float eps) {
   extern __shared__ __align__(16) float row[];
   __shared__ float2 scratch2[32];
   __shared__ float scratch[32];
+  __shared__ long long s_row[SN_MAX_TOP];
+  __shared__ float s_weight[SN_MAX_TOP];
   const long long t = blockIdx.x;
-  y1 += t * ldy;
+  const T* y1 = static_cast<const T*>(src.y1);
+  const T* y2 = static_cast<const T*>(src.y2);
+  if constexpr (SRC == SUB_EXPERTS) {
+    if (threadIdx.x < src.top) {
+      s_row[threadIdx.x] = (long long)src.row[t * src.top + threadIdx.x] * src.ld;
+      s_weight[threadIdx.x] = src.weight[t * src.top + threadIdx.x];
+    }
+    __syncthreads();
+  } else {
+    y1 += t * src.ld;
+    y2 += t * src.ld;
+  }
   float2 s2 = make_float2(0.f, 0.f);
   for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
     float a[V];
-    ldv<V>(y1 + i, a);
+    if constexpr (SRC == SUB_EXPERTS) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) a[j] = 0.f;
+      for (int e = 0; e < src.top; ++e) {
+        float b[V];
+        ldv<V>(y1 + s_row[e] + i, b);
+#pragma unroll
+        for (int j = 0; j < V; ++j) a[j] = fmaf(s_weight[e], b[j], a[j]);
+      }
+    } else {
+      ldv<V>(y1 + i, a);
+    }
 #pragma unroll
     for (int j = 0; j < V; ++j) s2.x += a[j] * a[j];
-    if constexpr (TWO) {
+    if constexpr (SRC == SUB_TWO) {
       float b[V];
-      ldv<V>(y2 + t * ldy + i, b);
+      ldv<V>(y2 + i, b);
 #pragma unroll
       for (int j = 0; j < V; ++j) s2.y += b[j] * b[j];
     } else {
@@ -140,15 +169,15 @@ sandwich_norm_kernel(const T* __restrict__ y1, const T* __restrict__ y2, long lo
   }
   s2 = block_sum2(s2, scratch2);
   float ss = s2.x;
-  if constexpr (TWO) {
+  if constexpr (SRC == SUB_TWO) {
     const float ra = 0.5f / sqrtf(s2.x / (float)dim + eps), rb = 0.5f / sqrtf(s2.y / (float)dim + eps);
     ss = 0.f;
     for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
       float a[V], b[V], wa[V], wb[V];
       ldv<V>(y1 + i, a);
-      ldv<V>(y2 + t * ldy + i, b);
-      ldv<V>(w1 + i, wa);
-      ldv<V>(w2 + i, wb);
+      ldv<V>(y2 + i, b);
+      ldv<V>(src.w1 + i, wa);
+      ldv<V>(src.w2 + i, wb);
 #pragma unroll
       for (int j = 0; j < V; ++j) {
         a[j] = a[j] * ra * wa[j] + b[j] * rb * wb[j];
@@ -158,7 +187,7 @@ sandwich_norm_kernel(const T* __restrict__ y1, const T* __restrict__ y2, long lo
     }
     ss = block_sum(ss, scratch);
   }
-  const float r = 1.f / sqrtf(ss / (float)dim + eps);
+  const float r = mult / sqrtf(ss / (float)dim + eps);
   float sx = 0.f;
   for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
     float a[V], w[V], xv[V];
@@ -173,7 +202,7 @@ sandwich_norm_kernel(const T* __restrict__ y1, const T* __restrict__ y2, long lo
     stv<V>(x + t * dim + i, xv);
     stv<V>(row + i, xv);
   }
-  sx = block_sum(sx, scratch);
+  if (w_next) sx = block_sum(sx, scratch);
   write_normed<T, V>(row, sx, w_next, h + t * ldh, ldh, dim, eps);
 }
 
@@ -330,12 +359,27 @@ paged_attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
   }
 }
 
-// 64 x 64 tile, 16-deep steps, 4 x 4 outputs per thread.
+// 64 x 64 tile, 16-deep steps, 4 x 4 outputs per thread. blockIdx.z: product of a batch, or entry of a tile list.
 __global__ void __launch_bounds__(256)
 gemm_f32_kernel(const float* __restrict__ A, long long lda, const float* __restrict__ B, long long ldb,
-                float* __restrict__ C, long long ldc, int M, int N, int K, float alpha) {
+                float* __restrict__ C, long long ldc, int M, int N, int K, float alpha, long long a_batch,
+                long long b_batch, long long c_batch, TileList list) {
   __shared__ float sa[16][68], sb[16][68];
-  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  int m0 = blockIdx.y * 64;
+  const int n0 = blockIdx.x * 64;
+  if (list.tiles) {
+    if ((int)blockIdx.z >= *list.count) return;
+    const int* tile = list.tiles + 3 * blockIdx.z;
+    m0 = 0;
+    M = tile[2];
+    A += tile[1] * lda;
+    C += tile[1] * ldc;
+    B += tile[0] * b_batch;
+  } else {
+    A += blockIdx.z * a_batch;
+    B += blockIdx.z * b_batch;
+    C += blockIdx.z * c_batch;
+  }
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += 16) {
@@ -370,18 +414,24 @@ gemm_f32_kernel(const float* __restrict__ A, long long lda, const float* __restr
 }
 
 template <typename T>
-__global__ void silu_gate_kernel(const T* __restrict__ gu, long long ldg, int f, int f_off, T* __restrict__ h,
+__global__ void gate_pair_kernel(const T* __restrict__ gu, long long ldg, int f, int f_off, GateAct act, T* __restrict__ h,
                                  long long ldh, long long rows) {
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < rows * ldh;
        i += (long long)gridDim.x * blockDim.x) {
     const long long r = i / ldh;
     const int c = (int)(i % ldh);
-    float y = 0.f;
-    if (c < f) {
-      const float g = ldf(gu + r * ldg + c), u = ldf(gu + r * ldg + f_off + c);
-      y = g * sigmoid_f(g) * u;
-    }
-    stf(h + i, y);
+    stf(h + i, c < f ? gate_act(act, ldf(gu + r * ldg + c), ldf(gu + r * ldg + f_off + c)) : 0.f);
+  }
+}
+
+template <typename T>
+__global__ void gelu_mul_kernel(T* __restrict__ y, long long ldy, const T* __restrict__ table, long long ld_table,
+                                const int* __restrict__ ids, int vocab, long long rows, int width) {
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < rows * width;
+       i += (long long)gridDim.x * blockDim.x) {
+    const long long r = i / width;
+    const int c = (int)(i % width), id = min(max(ids[r], 0), vocab - 1);
+    stf(y + r * ldy + c, gelu_tanh_f(ldf(y + r * ldy + c)) * ldf(table + id * ld_table + c));
   }
 }
 
@@ -400,15 +450,14 @@ void embed_launch(const int* ids, const int* pos, const void* embed, const void*
                                                                      eps);
 }
 template <typename T, int V>
-void sandwich_launch(const void* y1, const void* y2, long long ldy, const float* w1, const float* w2,
-                     const float* w_post, float* x, const float* w_next, void* h, long long ldh, int rows, int dim,
-                     float eps, cudaStream_t stream) {
-  if (y2)
-    sandwich_norm_kernel<T, V, true><<<rows, SN_THREADS, dim * 4, stream>>>(
-        (const T*)y1, (const T*)y2, ldy, w1, w2, w_post, x, w_next, (T*)h, ldh, dim, eps);
-  else
-    sandwich_norm_kernel<T, V, false><<<rows, SN_THREADS, dim * 4, stream>>>(
-        (const T*)y1, nullptr, ldy, w1, w2, w_post, x, w_next, (T*)h, ldh, dim, eps);
+void sandwich_launch(const SublayerOut& y, const float* w_post, float mult, float* x, const float* w_next, void* h,
+                     long long ldh, int rows, int dim, float eps, cudaStream_t stream) {
+#define MB_SN(SRC) \
+  sandwich_norm_kernel<T, V, SRC><<<rows, SN_THREADS, dim * 4, stream>>>(y, w_post, mult, x, w_next, (T*)h, ldh, dim, eps)
+  if (y.row) MB_SN(SUB_EXPERTS);
+  else if (y.y2) MB_SN(SUB_TWO);
+  else MB_SN(SUB_ONE);
+#undef MB_SN
 }
 
 }  // namespace
@@ -428,14 +477,14 @@ void embed_pos_norm(bool f32, const int* ids, const int* pos, const void* embed,
   check_launch();
 }
 
-void sandwich_norm(bool f32, const void* y1, const void* y2, long long ldy, const float* w1, const float* w2,
-                   const float* w_post, float* x, const float* w_next, void* h, long long ldh, int rows, int dim,
-                   float eps, cudaStream_t stream) {
-  MB_REQUIRE(dim > 0 && dim <= 12000 && ldh >= dim && ldy >= dim, "sandwich_norm: row width out of range");
-  MB_REQUIRE(y2 == nullptr || (w1 && w2), "sandwich_norm: two inputs need their norm weights");
+void sandwich_norm(bool f32, const SublayerOut& y, const float* w_post, float mult, float* x, const float* w_next, void* h,
+                   long long ldh, int rows, int dim, float eps, cudaStream_t stream) {
+  MB_REQUIRE(dim > 0 && dim <= 12000 && ldh >= dim && y.ld >= dim, "sandwich_norm: row width out of range");
+  MB_REQUIRE(y.y2 == nullptr || (y.w1 && y.w2), "sandwich_norm: two inputs need their norm weights");
+  MB_REQUIRE(y.row == nullptr || (y.weight && y.top > 0 && y.top <= SN_MAX_TOP), "sandwich_norm: at most 32 experts a token");
   if (rows == 0) return;
-  const bool v4 = dim % 4 == 0 && ldh % 4 == 0 && ldy % 4 == 0;
-  auto go = [&](auto fn) { fn(y1, y2, ldy, w1, w2, w_post, x, w_next, h, ldh, rows, dim, eps, stream); };
+  const bool v4 = dim % 4 == 0 && ldh % 4 == 0 && y.ld % 4 == 0;
+  auto go = [&](auto fn) { fn(y, w_post, mult, x, w_next, h, ldh, rows, dim, eps, stream); };
   if (f32) { if (v4) go(sandwich_launch<float, 4>); else go(sandwich_launch<float, 1>); }
   else     { if (v4) go(sandwich_launch<__nv_bfloat16, 4>); else go(sandwich_launch<__nv_bfloat16, 1>); }
   count_launch();
@@ -495,22 +544,38 @@ void paged_attn_any(bool f32, const void* q, const void* k_cache, const void* v_
 }
 
 void gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N,
-              int K, float alpha, cudaStream_t stream) {
-  if (M == 0 || N == 0) return;
-  gemm_f32_kernel<<<dim3((N + 63) / 64, (M + 63) / 64), 256, 0, stream>>>(A, lda, B, ldb, C, ldc, M, N, K, alpha);
+              int K, float alpha, cudaStream_t stream, int batch, long long a_batch, long long b_batch, long long c_batch,
+              const TileList* list) {
+  if (M == 0 || N == 0 || batch == 0) return;
+  const dim3 grid((N + 63) / 64, list ? 1 : (M + 63) / 64, list ? list->max_tiles : batch);
+  gemm_f32_kernel<<<grid, 256, 0, stream>>>(A, lda, B, ldb, C, ldc, M, N, K, alpha, a_batch, b_batch, c_batch,
+                                            list ? *list : TileList{nullptr, nullptr, 0});
   count_launch();
   check_launch();
 }
 
-void silu_gate(bool f32, const void* gu, long long ldg, int f, int f_off, void* h, long long ldh, int rows,
+void gate_pair(bool f32, const void* gu, long long ldg, int f, int f_off, const GateAct& act, void* h, long long ldh, int rows,
                cudaStream_t stream) {
   if (rows == 0) return;
   const int grid = grid_for((long long)rows * ldh, 256, 16);
   if (f32)
-    silu_gate_kernel<float><<<grid, 256, 0, stream>>>((const float*)gu, ldg, f, f_off, (float*)h, ldh, rows);
+    gate_pair_kernel<float><<<grid, 256, 0, stream>>>((const float*)gu, ldg, f, f_off, act, (float*)h, ldh, rows);
   else
-    silu_gate_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)gu, ldg, f, f_off,
+    gate_pair_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)gu, ldg, f, f_off, act,
                                                               (__nv_bfloat16*)h, ldh, rows);
+  count_launch();
+  check_launch();
+}
+
+void gelu_mul(bool f32, void* y, long long ldy, const void* table, long long ld_table, const int* ids, int vocab, int rows,
+              int width, cudaStream_t stream) {
+  if (rows == 0 || width == 0) return;
+  const int grid = grid_for((long long)rows * width, 256, 16);
+  if (f32)
+    gelu_mul_kernel<float><<<grid, 256, 0, stream>>>((float*)y, ldy, (const float*)table, ld_table, ids, vocab, rows, width);
+  else
+    gelu_mul_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((__nv_bfloat16*)y, ldy, (const __nv_bfloat16*)table, ld_table, ids,
+                                                             vocab, rows, width);
   count_launch();
   check_launch();
 }

@@ -681,9 +681,11 @@ class InferenceEngine:
         cu = [0]
         for k in lens:
             cu.append(cu[-1] + k)
-        # one host buffer, one copy: ids | positions | slot per token | sequence per token | per-sequence arrays
-        host = torch.empty(4 * T + 3 * n + 1, dtype=torch.int32, pin_memory=dev.type == "cuda")
-        parts = host.split([T, T, T, T, n + 1, n, n])
+        extra, build = self._batch_plan(lens, bases)
+        # one host buffer, one copy: ids | positions | slot per token | sequence per token | per-sequence arrays | extras
+        sizes = [T, T, T, T, n + 1, n, n] + [len(e) for e in extra]
+        host = torch.empty(sum(sizes), dtype=torch.int32, pin_memory=dev.type == "cuda")
+        parts = host.split(sizes)
         for i, (s, base, toks) in enumerate(zip(seqs, bases, token_lists)):
             lo, hi = cu[i], cu[i + 1]
             parts[0][lo:hi] = torch.as_tensor(toks, dtype=torch.int32)
@@ -693,11 +695,20 @@ class InferenceEngine:
         parts[4].copy_(torch.tensor(cu, dtype=torch.int32))
         parts[5].copy_(torch.tensor([b + k for b, k in zip(bases, lens)], dtype=torch.int32))
         parts[6].copy_(torch.tensor(seqs, dtype=torch.int32))
-        ids, pos, sid, row_seq, cu_q, kv_lens, slots = host.to(dev, non_blocking=True).split([T, T, T, T, n + 1, n, n])
+        for part, e in zip(parts[7:], extra):
+            part.copy_(torch.tensor(e, dtype=torch.int32))
+        ids, pos, sid, row_seq, cu_q, kv_lens, slots, *more = host.to(dev, non_blocking=True).split(sizes)
         rows = self.cache.block_table.index_select(0, slots.long()).contiguous()
         h = self._forward(ids, pos, sid, None, paged=(cu_q, kv_lens, rows, max(lens), slots, row_seq,
-                                                        max(b + k for b, k in zip(bases, lens))))
+                                                        max(b + k for b, k in zip(bases, lens)),
+                                                        build(*more) if build is not None else None))
         return h, cu
+
+    def _batch_plan(self, lens, bases):
+        """What an engine wants to know about a ragged batch (new tokens and earlier tokens of every sequence)
+        beyond the arrays above: int lists that are uploaded with them, and a function that makes the last
+        entry of ``paged`` from their device copies."""
+        return [], None
 
     @torch.no_grad()
     def _prefill_chunked(self, seqs, token_lists, bases=None):

@@ -11,14 +11,23 @@ gated-linear-attention layer: projections -> decay GEMM -> recurrence -> head no
 GEMM -> (post-norm + residual + next pre-norm). A parallel layer runs the delta-rule recurrence and
 paged attention side by side and averages their normalised outputs inside that last kernel.
 
+Latent attention caches one row per token (latent | rotated key part) that all heads share. Tokens of
+sequences that bring few of them at once (decoding, short portions) attend in the latent's space: queries go
+through W_uk, the result through W_uv. Longer portions expand the latents of their sequence to keys and
+values once per pass and run the tensor-core prompt attention. A batch with both runs both. Routed experts:
+router GEMM -> selection and row segments -> row gather -> two grouped GEMMs -> (weighted sum + norm +
+residual).
+
 ``dtype``: "bfloat16" (matrix products and activations in bf16 with 32-bit accumulation; residual,
 norms, decays, states and scores in 32-bit) or "float32" (everything in 32-bit).
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
-from ..models.hybrid_config import HybridConfig, ParallelMixer, RecurrentMixer
+from ..models.hybrid_config import HybridConfig, LatentAttentionMixer, MoeFF, ParallelMixer, RecurrentMixer
 from ..ops import native
 from .engine import InferenceEngine
 from .kv_paged import PagedKVCache, RecurrentStatePool
@@ -55,15 +64,29 @@ class _Sublayer:
 
 
 class _Ctx:
-    """One pass: the ragged batch (cu_q, kv_lens, slots, row_seq, pos), its block-table rows and sizes.
-    ``decode``: one token of every sequence."""
+    """One pass: token ids, the ragged batch (cu_q, kv_lens, slots, row_seq, pos), its block-table rows and sizes.
+    ``decode``: one token of every sequence. ``split`` (passes with a long portion and latent layers):
+    ``_LatentSplit``, else every token attends in the latent's space."""
 
-    def __init__(self, batch, table, rows, n_seq, max_q, max_kv):
-        self.batch, self.table, self.rows, self.n_seq, self.max_q, self.max_kv = batch, table, rows, n_seq, max_q, max_kv
+    def __init__(self, ids, batch, table, rows, n_seq, max_q, max_kv, split=None):
+        self.ids, self.batch, self.table, self.rows, self.n_seq = ids, batch, table, rows, n_seq
+        self.max_q, self.max_kv, self.split = max_q, max_kv, split
         self.decode = max_q == 1
 
 
+class _LatentSplit:
+    """Which tokens attend how: ``cu_k`` first expanded row of every sequence with a long portion (``keys`` in all,
+    at most ``max_k`` of one), ``short`` the rows of the other sequences (None: there are none)."""
+
+    def __init__(self, cu_k, keys, max_k, short, short_seq, short_pos):
+        self.cu_k, self.keys, self.max_k = cu_k, keys, max_k
+        self.short, self.short_seq, self.short_pos = short, short_seq, short_pos
+
+
 DECODE_GEMM_ROWS = 128     # up to this many tokens a product goes through the few-token GEMM
+EXPAND_TOKENS = 16         # portions of at least this many tokens expand the latents of their sequence
+EXPAND_BYTES = 4 << 30     # unless the expanded keys and values would need more than this
+SEGMENT_GEMM_ROWS = 48     # mean rows per expert from which the prompt-sized grouped GEMM runs
 LOW_RANK_FUSE_ROWS = 16    # decode batches up to this size evaluate the low-rank maps inside the recurrence kernel
 
 
@@ -86,15 +109,21 @@ class HybridEngine(InferenceEngine):
         self.dtype = DTYPES[dtype]
         self.f32 = self.dtype == torch.float32
         self.max_batch = max_batch
-        self.max_seq_len = min(max_seq_len or cfg.max_seq_len, cfg.max_seq_len)
+        self.max_seq_len = min(max_seq_len or cfg.max_seq_len, cfg.context_limit)
         self.page_size = page_size
         self.world, self.rank = 1, 0
         pages_per_seq = (self.max_seq_len + page_size - 1) // page_size
         att = [s.attention for s in cfg.layers if s.attention is not None]
-        self.states = RecurrentStatePool(max_batch, self.device)
-        self.cache = PagedKVCache(len(att), 0, 0, kv_pages or max_batch * pages_per_seq, page_size, max_batch,
-                                  pages_per_seq, self.device, dtype=self.dtype,
-                                  layer_shapes=[(m.kv_heads, m.dim, m.vdim) for m in att], states=self.states)
+        recurrent = any(s.recurrent is not None for s in cfg.layers)
+        self.states = RecurrentStatePool(max_batch, self.device) if recurrent else None
+        shapes = []                # per caching layer; a latent layer's rows are keys and values at once
+        for s in cfg.layers:
+            if s.attention is not None:
+                shapes.append((s.attention.kv_heads, s.attention.dim, s.attention.vdim))
+            elif s.latent is not None:
+                shapes.append((1, _pad8(s.latent.kv_rank) + _pad8(s.latent.rot_dim), 0))
+        self.cache = PagedKVCache(len(shapes), 0, 0, kv_pages or max_batch * pages_per_seq, page_size, max_batch,
+                                  pages_per_seq, self.device, dtype=self.dtype, layer_shapes=shapes, states=self.states)
         self.layers = []
         self.prefill_chunk = 8192
         self.prefill_chunk_threshold = 0
@@ -103,7 +132,12 @@ class HybridEngine(InferenceEngine):
         self.H = native.require_hybrid() if self.device.type == "cuda" else None
         self._status = native.status_word(self.device)
         groups = max([m.kv_heads * ((m.heads // m.kv_heads + 7) // 8) for m in att] or [1])
-        self._counters = torch.zeros(max_batch * groups, device=self.device, dtype=torch.int32)
+        latent_groups = max([(s.latent.heads + 15) // 16 for s in cfg.layers if s.latent is not None] or [0])
+        # tokens that can attend in the latent's space in one pass: short portions only
+        self._counters = torch.zeros(max(max_batch * groups, max_batch * EXPAND_TOKENS * latent_groups), device=self.device,
+                                     dtype=torch.int32)
+        experts = max([s.mlp.experts for s in cfg.layers if isinstance(s.mlp, MoeFF)] or [0])
+        self._expert_counts = torch.zeros(experts + 1, device=self.device, dtype=torch.int32)
         self._max_ctx = self.max_seq_len
 
     # ------------------------------------------------------------------ weights
@@ -132,25 +166,48 @@ class HybridEngine(InferenceEngine):
 
     def _pack(self, model) -> None:
         t = model.tensor
+        cfg = self.cfg
         self.embed_table = t("embed").to(self.device, self.dtype).contiguous()
-        self.pos_table = t("pos").to(self.device, self.dtype).contiguous()
+        self.pos_table = t("pos").to(self.device, self.dtype).contiguous() if cfg.position_table else None
+        self.side_table = t("side.embed").to(self.device, self.dtype).contiguous() if cfg.token_side else None
         self.final_norm = self._vector(t("final.norm"))
         self.head = self._matrix(t("head"))
         n_att = 0
-        for i, spec in enumerate(self.cfg.layers):
+
+        def norms(p: str, n: int) -> _Sublayer:
+            if cfg.pre_norm:
+                return _Sublayer(self._vector(t(p + f"norm{n}")), self._vector(t(p + f"norm{n}b")))
+            return _Sublayer(None, self._vector(t(p + f"norm{n}")))
+
+        for i, spec in enumerate(cfg.layers):
             p = f"l{i}."
             L = _HybridLayer()
             L.spec = spec
-            L.norms = _Sublayer(self._vector(t(p + "norm1")), self._vector(t(p + "norm1b")))
+            L.norms = norms(p, 1)
             if isinstance(spec.mixer, ParallelMixer):
-                self._pack_parallel(L, t, p + "mix.", n_att)
+                L.run, L.att_index = self._parallel, n_att
+                self._pack_parallel(L, t, p + "mix.")
+                n_att += 1
+            elif isinstance(spec.mixer, LatentAttentionMixer):
+                L.run, L.att_index = self._latent, n_att
+                self._pack_latent(L, t, p + "mix.")
                 n_att += 1
             else:
+                L.run = self._gla
                 self._pack_gla(L, t, p + "mix.")
-            if spec.ff:
-                L.ff_norms = _Sublayer(self._vector(t(p + "norm2")), self._vector(t(p + "norm2b")))
-                L.gate_up = FusedProjection([("gate", t(p + "mlp.gate")), ("up", t(p + "mlp.up"))], self.dtype, self.device)
-                L.down = self._matrix(t(p + "mlp.down"))
+            if spec.mlp is not None:
+                L.ff_norms = norms(p, 2)
+                if isinstance(spec.mlp, MoeFF):
+                    self._pack_experts(L, t, p + "mlp.")
+                else:
+                    L.act = ({"silu": 0, "relu": 1}[spec.mlp.act], 0.0, 0.0)
+                    L.gate_up = FusedProjection([("gate", t(p + "mlp.gate")), ("up", t(p + "mlp.up"))], self.dtype, self.device)
+                    L.down = self._matrix(t(p + "mlp.down"))
+            if cfg.token_side:
+                n = cfg.token_side
+                L.side_gate, L.side_proj = self._matrix(t(p + "side.gate")), self._matrix(t(p + "side.proj"))
+                L.side_embed = self.side_table[:, i * n:(i + 1) * n]
+                L.side_norms = _Sublayer(None, self._vector(t(p + "side.norm")))
             self.layers.append(L)
 
     def _recurrent(self, m: RecurrentMixer, off: dict, tensors: dict):
@@ -175,13 +232,12 @@ class HybridEngine(InferenceEngine):
                                 {"z_bias": self._vector(t(p + "a2.b")), "gamma": self._vector(t(p + "norm")), "a2": L.a2})
         L.out = self._matrix(t(p + "o"))
 
-    def _pack_parallel(self, L, t, p: str, att_index: int) -> None:
+    def _pack_parallel(self, L, t, p: str) -> None:
         a, r = L.spec.mixer.left, L.spec.mixer.right
         left, right = p + "left.", p + "right."
         L.proj = FusedProjection(
             [("lq", t(left + "q")), ("lk", t(left + "k")), ("lv", t(left + "v")), ("lg", t(left + "g"))]
             + [("r" + n, t(right + n)) for n in ("q", "k", "v", "b", "a1", "g1")], self.dtype, self.device)
-        L.att_index = att_index
         L.q_gamma, L.k_gamma = self._vector(t(left + "q.norm")), self._vector(t(left + "k.norm"))
         L.left_out, L.right_out = self._matrix(t(left + "o")), self._matrix(t(right + "o"))
         L.left_norm, L.right_norm = self._vector(t(left + "out")), self._vector(t(right + "out"))
@@ -194,11 +250,62 @@ class HybridEngine(InferenceEngine):
             tensors["conv_w"] = self._vector(torch.cat([t(right + n + ".conv") for n in ("q", "k", "v")]))
         L.rec = self._recurrent(r, {"q": off["rq"], "k": off["rk"], "v": off["rv"], "b": off["rb"]}, tensors)
 
+    def _pack_latent(self, L, t, p: str) -> None:
+        """Projection columns: unrotated queries per head | rotated queries per head | latent | rotated key part, each
+        part of a head padded to a multiple of 8."""
+        m = L.spec.mixer
+        H, dn, dr, dv, r = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank
+        dn_p, dr_p, dv_p, r_p = _pad8(dn), _pad8(dr), _pad8(dv), _pad8(r)
+
+        def heads(w, width, padded):                   # [heads * width, K] -> [heads * padded, K]
+            out = w.new_zeros(H, padded, w.shape[1])
+            out[:, :width] = w.view(H, width, -1)
+            return out.view(H * padded, -1)
+
+        q = t(p + "q").view(H, dn + dr, -1)
+        dkv = t(p + "dkv")
+        L.proj = FusedProjection([("q", heads(q[:, :dn].reshape(H * dn, -1), dn, dn_p)),
+                                  ("qr", heads(q[:, dn:].reshape(H * dr, -1), dr, dr_p)),
+                                  ("c", dkv[:r]), ("kr", dkv[r:])], self.dtype, self.device)
+        uk, uv = t(p + "uk").view(H, dn, r), t(p + "uv").view(H, dv, r)
+        L.uk_t = torch.zeros(H, r_p, dn_p, dtype=self.dtype, device=self.device)       # queries into the latent's space
+        L.uk_t[:, :r, :dn] = uk.transpose(1, 2).to(self.device, self.dtype)
+        L.uv = torch.zeros(H, dv_p, r_p, dtype=self.dtype, device=self.device)         # latents to a head's values
+        L.uv[:, :dv, :r] = uv.to(self.device, self.dtype)
+        off = L.proj.off
+        turns = torch.tensor([m.rot_base ** (-2.0 * i / dr) / (2.0 * math.pi) for i in range(dr // 2)], dtype=torch.float64)
+        L.lat = self.H.Latent({"heads": H, "rank": r, "rot": dr, "rank_p": r_p, "rot_p": dr_p, "qr_off": off["qr"],
+                               "c_off": off["c"], "kr_off": off["kr"], "scale": m.scale, "eps": self.cfg.norm_eps},
+                              self._vector(t(p + "dkv.norm")), turns.to(self.device), self._vector(t(p + "sink")))
+        L.expand = None
+        if self.tensor_kernels and not self.f32 and L.lat.prefill_ok(dn_p, dv_p):      # keys and values of all heads
+            L.expand = torch.zeros(H * (dn_p + dv_p), r_p, dtype=self.dtype, device=self.device)
+            L.expand[: H * dn_p].view(H, dn_p, r_p)[:, :dn, :r] = uk.to(self.device, self.dtype)
+            L.expand[H * dn_p:].view(H, dv_p, r_p).copy_(L.uv)
+        out = t(p + "o")
+        w = out.new_zeros(out.shape[0], H, dv_p)
+        w[:, :, :dv] = out.view(-1, H, dv)
+        L.out = self._matrix(w.view(-1, H * dv_p))
+
+    def _pack_experts(self, L, t, p: str) -> None:
+        """Gate and up rows of an expert in one matrix [2 * ff, d], all experts stacked; ff padded to a multiple of 8."""
+        m, d = L.spec.mlp, self.cfg.hidden_size
+        f = _pad8(m.ff)
+        L.act = (2, m.limit, m.alpha)
+        L.router, L.correction = self._matrix(t(p + "router")), self._vector(t(p + "correction"))
+        L.w_in = torch.zeros(m.experts, 2 * f, _pad8(d), dtype=self.dtype, device=self.device)
+        L.w_out = torch.zeros(m.experts, _pad8(d), f, dtype=self.dtype, device=self.device)
+        for e in range(m.experts):
+            L.w_in[e, : m.ff, :d] = t(p + f"e{e}.gate").to(self.device, self.dtype)
+            L.w_in[e, f:f + m.ff, :d] = t(p + f"e{e}.up").to(self.device, self.dtype)
+            L.w_out[e, :d, : m.ff] = t(p + f"e{e}.down").to(self.device, self.dtype)
+
     def weight_bytes(self) -> int:
-        n = sum(x.numel() * x.element_size() for x in (self.embed_table, self.pos_table, self.head))
+        tables = (self.embed_table, self.pos_table, self.side_table, self.head)
+        n = sum(x.numel() * x.element_size() for x in tables if x is not None)
         for L in self.layers:
-            mats = [L.proj.weight, L.a2, L.g2, L.out, L.left_out, L.right_out, L.down,
-                    L.gate_up.weight if L.gate_up is not None else None]
+            mats = [L.proj.weight, L.a2, L.g2, L.out, L.left_out, L.right_out, L.down, L.uk_t, L.uv, L.router, L.w_in, L.w_out,
+                    L.side_gate, L.side_proj, L.gate_up.weight if L.gate_up is not None else None]
             n += sum(x.numel() * x.element_size() for x in mats if x is not None)
         return n
 
@@ -282,18 +389,106 @@ class HybridEngine(InferenceEngine):
         y_left = self._gemm(self._attention(L, proj, ctx), L.left_out)
         return y_left, y_right
 
+    # ---- latent attention
+    def _latent_tokens(self, L, proj, row_seq, pos, ctx):
+        """Tokens that attend in the latent's space -> [rows, heads, padded value width]."""
+        m, H = L.spec.mixer, L.spec.mixer.heads
+        n, cache = proj.shape[0], self.cache.k[L.att_index]
+        r_p, dn_p = L.uk_t.shape[1:]
+        q = proj[:, : H * dn_p].unflatten(1, (H, dn_p))
+        q_lat = torch.empty(n, H, r_p, device=self.device, dtype=self.dtype)
+        o_lat = torch.empty_like(q_lat)
+        self.H.gemm_heads(q, L.uk_t, q_lat, self._status)
+        groups = (H + 15) // 16
+        if self._fast and n * groups <= self._counters.numel() and L.lat.decode_ok(self.page_size):
+            splits = max(1, min(64, (self._sms + n * groups - 1) // (n * groups), (ctx.max_kv + 127) // 128))
+            scratch = torch.empty(n * H * splits * (r_p + 2), device=self.device, dtype=torch.float32)
+            L.lat.attn_decode(q_lat, proj, row_seq, pos, ctx.table, cache, o_lat, scratch, self._counters, splits, self._status)
+        else:
+            L.lat.attn_any(q_lat, proj, row_seq, pos, ctx.table, cache, o_lat)
+        out = torch.empty(n, H, L.uv.shape[1], device=self.device, dtype=self.dtype)
+        self.H.gemm_heads(o_lat, L.uv, out, self._status)
+        return out
+
+    def _latent(self, L, h, ctx):
+        m, H = L.spec.mixer, L.spec.mixer.heads
+        proj = self._gemm(h, L.proj.weight)
+        cache = self.cache.k[L.att_index]
+        L.lat.prep(proj, ctx.batch, ctx.table, cache)
+        sp = ctx.split
+        if sp is None or L.expand is None or not self._fast or sp.keys * L.expand.shape[0] * 2 > EXPAND_BYTES:
+            o = self._latent_tokens(L, proj, ctx.batch[3], ctx.batch[4], ctx)
+            return self._gemm(o.flatten(1), L.out), None
+        dn_p, dv_p = L.uk_t.shape[2], L.uv.shape[1]
+        latents = self._new(sp.keys, cache.shape[3])
+        L.lat.gather(ctx.table, cache, sp.cu_k, sp.max_k, latents)
+        kv = self._gemm(latents[:, : L.expand.shape[1]], L.expand)
+        o = torch.empty(ctx.rows, H, dv_p, device=self.device, dtype=self.dtype)
+        L.lat.attn_prefill(proj[:, : H * dn_p].unflatten(1, (H, dn_p)), proj, kv[:, : H * dn_p].unflatten(1, (H, dn_p)),
+                           kv[:, H * dn_p:].unflatten(1, (H, dv_p)), latents, ctx.batch, sp.cu_k, ctx.max_q, EXPAND_TOKENS, o,
+                           self._status)
+        if sp.short is not None:
+            o.index_copy_(0, sp.short, self._latent_tokens(L, proj.index_select(0, sp.short), sp.short_seq, sp.short_pos, ctx))
+        return self._gemm(o.flatten(1), L.out), None
+
+    # ---- feed-forwards
+    def _experts(self, L, h, ctx):
+        """Outputs of the chosen experts [rows * top, d], where each (token, choice) lies and its weight."""
+        m, T, C = L.spec.mlp, ctx.rows, self.H
+        z = self._gemm(h, L.router, dtype=torch.float32)
+        pairs = T * m.top
+        if self.f32:
+            tile = 64
+        elif pairs >= SEGMENT_GEMM_ROWS * m.experts:
+            tile = 128
+        else:
+            tile = max(16, min(64, 1 << (2 * pairs // m.experts).bit_length()))
+        i32 = dict(device=self.device, dtype=torch.int32)
+        idx, slot, row = (torch.empty(T, m.top, **i32) for _ in range(3))
+        weight = torch.empty(T, m.top, device=self.device, dtype=torch.float32)
+        offset, count = torch.empty(m.experts, **i32), torch.empty(1, **i32)
+        tiles = torch.empty(min(pairs, m.experts + pairs // tile), 3, **i32)
+        route = (m.experts, m.top, m.groups, m.keep)
+        plan = (idx, weight, slot, self._expert_counts[: m.experts + 1], offset, tiles, count)
+        C.expert_select(z, L.correction, route, tile, *plan)
+        d_p, f = L.w_in.shape[2], L.w_out.shape[2]
+        x = self._new(pairs, d_p)
+        C.expert_gather(h, route, *plan, x, row)
+        a, y = self._new(pairs, f), self._new(pairs, d_p)
+        if self.f32:
+            gu = self._new(pairs, 2 * f)
+            C.gemm_tiles(x, L.w_in, gu, tiles, count, tile, 0, 0, L.act, self._status)
+            C.gate_pair(gu, f, f, L.act, a)
+        else:
+            C.gemm_tiles(x, L.w_in, a, tiles, count, tile, f, f, L.act, self._status)
+        C.gemm_tiles(a, L.w_out, y, tiles, count, tile, 0, 0, L.act, self._status)
+        return y, row, weight
+
     def _feed_forward(self, L, h, ctx):
-        f = L.spec.ff
+        f = L.spec.mlp.ff
         a = self._new(ctx.rows, L.down.shape[1])
         if self._fast and f % 8 == 0 and ctx.rows <= DECODE_GEMM_ROWS:
-            self.H.gemm_decode(h, L.gate_up.weight, a, f, L.gate_up.off["up"], 1.0, self._status)
+            self.H.gemm_decode(h, L.gate_up.weight, a, f, L.gate_up.off["up"], 1.0, self._status, L.act)
             return self._gemm(a, L.down)
-        if self._fast and f % 128 == 0 and ctx.rows >= 256:
+        if self._fast and L.act[0] == 0 and f % 128 == 0 and ctx.rows >= 256:
             self.H.gemm_swiglu(h, L.gate_up.weight, a, self._status)
             return self._gemm(a, L.down)
         gu = self._gemm(h, L.gate_up.weight)
-        self.H.silu_gate(gu, f, L.gate_up.off["up"], a)
+        self.H.gate_pair(gu, f, L.gate_up.off["up"], L.act, a)
         return self._gemm(a, L.down)
+
+    def _token_side(self, L, h, ctx):
+        """proj(gelu(gate x) * side embedding of the token)"""
+        g = self._new(ctx.rows, L.side_proj.shape[1])
+        n = L.side_gate.shape[0]
+        if g.shape[1] != n:
+            g[:, n:].zero_()
+        if self._fast:
+            self.H.gemm_decode(h, L.side_gate, g, 0, 0, 1.0, self._status, (0, 0.0, 0.0), L.side_embed, ctx.ids)
+        else:
+            self.H.gemm_nt(h, L.side_gate, g[:, :n], 1.0, self._status)
+            self.H.gelu_mul(g[:, :n], L.side_embed, ctx.ids)
+        return self._gemm(g, L.side_proj)
 
     # ------------------------------------------------------------------ the pass
     def _paged_prefill_ok(self) -> bool:
@@ -306,14 +501,34 @@ class HybridEngine(InferenceEngine):
         """``paged`` as in the base class; without it every row is one token of the sequence ``seq_ids[row]``
         with ``ctx_lens[row]`` tokens including it (a decode step)."""
         if paged is not None:
-            cu_q, kv_lens, table, max_q, slots, row_seq, max_kv = paged
+            cu_q, kv_lens, table, max_q, slots, row_seq, max_kv, split = paged
         else:
             n = ids.numel()
             cu_q = torch.arange(n + 1, device=self.device, dtype=torch.int32)
-            row_seq, slots, kv_lens, max_q, max_kv = cu_q[:n], seq_ids, ctx_lens, 1, self._max_ctx
+            row_seq, slots, kv_lens, max_q, max_kv, split = cu_q[:n], seq_ids, ctx_lens, 1, self._max_ctx, None
             table = self.cache.block_table.index_select(0, slots)
-        ctx = _Ctx([cu_q, kv_lens, slots, row_seq, pos], table, ids.numel(), kv_lens.numel(), max_q, max_kv)
+        ctx = _Ctx(ids, [cu_q, kv_lens, slots, row_seq, pos], table, ids.numel(), kv_lens.numel(), max_q, max_kv, split)
         return self._run_layers(ids, pos, ctx)
+
+    def _batch_plan(self, lens, bases):
+        if not any(s.latent is not None for s in self.cfg.layers) or max(lens) < EXPAND_TOKENS:
+            return [], None
+        cu_k, short, short_seq, short_pos, at, max_k = [0], [], [], [], 0, 0
+        for i, (n, base) in enumerate(zip(lens, bases)):
+            if n >= EXPAND_TOKENS:
+                cu_k.append(cu_k[-1] + base + n)
+                max_k = max(max_k, base + n)
+            else:
+                cu_k.append(cu_k[-1])
+                short += range(at, at + n)
+                short_seq += [i] * n
+                short_pos += range(base, base + n)
+            at += n
+
+        def build(cu, rows, seq, pos):
+            return _LatentSplit(cu, cu_k[-1], max_k, rows.long() if short else None, seq, pos)
+
+        return [cu_k, short, short_seq, short_pos], build
 
     def _run_layers(self, ids, pos, ctx, trace=None):
         cfg, H = self.cfg, self.H
@@ -322,18 +537,21 @@ class HybridEngine(InferenceEngine):
         h = self._new(ctx.rows, _pad8(d))
         subs = []                                    # (layer, sublayer function, its norms)
         for L in self.layers:
-            subs.append((L, self._parallel if L.spec.attention is not None else self._gla, L.norms))
-            if L.spec.ff:
-                subs.append((L, None, L.ff_norms))
+            subs.append((L, L.run, L.norms))
+            if L.spec.mlp is not None:
+                subs.append((L, self._experts if L.router is not None else self._feed_forward, L.ff_norms))
+            if L.side_gate is not None:
+                subs.append((L, self._token_side, L.side_norms))
         H.embed_pos_norm(ids, pos, self.embed_table, self.pos_table, cfg.embed_scale,
                          subs[0][2].pre if subs else self.final_norm, x, h, eps)
         for j, (L, fn, norms) in enumerate(subs):
             nxt = subs[j + 1][2].pre if j + 1 < len(subs) else self.final_norm
-            if fn is None:
-                H.sandwich_norm(self._feed_forward(L, h, ctx), None, None, None, norms.post, x, nxt, h, eps)
+            y = fn(L, h, ctx)
+            if fn == self._experts:
+                H.expert_norm(*y, norms.post, x, nxt, h, eps, cfg.residual_mult)
             else:
-                y1, y2 = fn(L, h, ctx)
-                H.sandwich_norm(y1, y2, L.left_norm, L.right_norm, norms.post, x, nxt, h, eps)
+                y1, y2 = y if isinstance(y, tuple) else (y, None)
+                H.sandwich_norm(y1, y2, L.left_norm, L.right_norm, norms.post, x, nxt, h, eps, cfg.residual_mult)
             if trace is not None and (j + 1 == len(subs) or subs[j + 1][0] is not L):
                 trace.append(x.clone())
         return h
@@ -351,5 +569,7 @@ class HybridEngine(InferenceEngine):
 
 class _HybridLayer:
     spec = norms = ff_norms = proj = a2 = g2 = out = left_out = right_out = left_norm = right_norm = rec = None
-    gate_up = down = None
+    gate_up = down = act = router = correction = w_in = w_out = None
+    lat = uk_t = uv = expand = run = None
+    side_gate = side_proj = side_embed = side_norms = None
     rank = g_rank = att_index = 0

@@ -10,7 +10,8 @@ from __future__ import annotations
 import torch
 import torch.nn as nn
 
-from .hybrid_config import AttentionMixer, HybridConfig, ParallelMixer, RecurrentMixer
+from .hybrid_config import (AttentionMixer, HybridConfig, LatentAttentionMixer, MoeFF, ParallelMixer,
+                            RecurrentMixer)
 
 
 def _attention_shapes(p: str, m: AttentionMixer, d: int) -> dict:
@@ -33,23 +34,57 @@ def _delta_shapes(p: str, m: RecurrentMixer, d: int) -> dict:
     return out
 
 
+def _latent_shapes(p: str, m: LatentAttentionMixer, d: int) -> dict:
+    return {p + "q": (m.heads * (m.dim + m.rot_dim), d), p + "dkv": (m.kv_rank + m.rot_dim, d), p + "dkv.norm": (m.kv_rank,),
+            p + "uk": (m.heads * m.dim, m.kv_rank), p + "uv": (m.heads * m.vdim, m.kv_rank), p + "sink": (m.heads,),
+            p + "o": (d, m.heads * m.vdim)}
+
+
+def _gated_shapes(p: str, ff: int, d: int) -> dict:
+    return {p + "gate": (ff, d), p + "up": (ff, d), p + "down": (d, ff)}
+
+
+def _mlp_shapes(p: str, f, d: int) -> dict:
+    if not isinstance(f, MoeFF):
+        return _gated_shapes(p, f.ff, d)
+    out = {p + "router": (f.experts, d), p + "correction": (f.experts,)}
+    for e in range(f.experts):
+        out.update(_gated_shapes(p + f"e{e}.", f.ff, d))
+    return out
+
+
 def expected_shapes(cfg: HybridConfig) -> dict:
     """Name -> shape of every tensor; ``None`` marks a low-rank width that the tensors themselves fix."""
     d = cfg.hidden_size
-    out = {"embed": (cfg.vocab_size, d), "pos": (cfg.max_seq_len, d), "final.norm": (d,), "head": (cfg.vocab_size, d)}
+    out = {"embed": (cfg.vocab_size, d)}
+    if cfg.position_table:
+        out["pos"] = (cfg.max_seq_len, d)
+    out.update({"final.norm": (d,), "head": (cfg.vocab_size, d)})
+    if cfg.token_side:
+        out["side.embed"] = (cfg.vocab_size, cfg.num_layers * cfg.token_side)
+
+    def norms(p: str, n: int) -> None:                 # a sublayer's norms: before (if the design has one), after
+        out[p + f"norm{n}"] = (d,)
+        if cfg.pre_norm:
+            out[p + f"norm{n}b"] = (d,)
+
     for i, spec in enumerate(cfg.layers):
         p = f"l{i}."
-        out[p + "norm1"] = out[p + "norm1b"] = (d,)
+        norms(p, 1)
         m = spec.mixer
         if isinstance(m, ParallelMixer):
             out.update(_attention_shapes(p + "mix.left.", m.left, d))
             out.update(_delta_shapes(p + "mix.right.", m.right, d))
             out[p + "mix.left.out"] = out[p + "mix.right.out"] = (d,)
+        elif isinstance(m, LatentAttentionMixer):
+            out.update(_latent_shapes(p + "mix.", m, d))
         else:
             out.update(_gla_shapes(p + "mix.", m, d))
-        if spec.ff:
-            out[p + "norm2"] = out[p + "norm2b"] = (d,)
-            out.update({p + "mlp.gate": (spec.ff, d), p + "mlp.up": (spec.ff, d), p + "mlp.down": (d, spec.ff)})
+        if spec.mlp is not None:
+            norms(p, 2)
+            out.update(_mlp_shapes(p + "mlp.", spec.mlp, d))
+        if cfg.token_side:
+            out.update({p + "side.gate": (cfg.token_side, d), p + "side.proj": (d, cfg.token_side), p + "side.norm": (d,)})
     return out
 
 
@@ -89,6 +124,8 @@ class HybridModel(nn.Module):
                 t = torch.ones(shape, device=device)
             elif leaf == "A_log":
                 t = torch.log(1.0 + 3.0 * torch.rand(shape, device=device, generator=g))
+            elif leaf in ("sink", "correction"):
+                t = torch.randn(shape, device=device, generator=g) * (1.0 if leaf == "sink" else 0.01)
             elif leaf == "dt_bias":
                 t = -4.0 + torch.rand(shape, device=device, generator=g)
             elif leaf == "b":

@@ -70,7 +70,7 @@ def main(argv=None) -> int:
     model = registry.load_checkpoint(args.model, device=args.device)
     pages = (args.max_tokens + PAGE - 1) // PAGE
     engine = InferenceEngine.from_model(model, device=args.device, dtype=args.dtype, max_batch=SLOTS,
-                                        max_seq_len=model.cfg.max_seq_len, page_size=PAGE, kv_pages=pages)
+                                        max_seq_len=min(model.cfg.context_limit, pages * PAGE), page_size=PAGE, kv_pages=pages)
     del model
     replay = TraceReplay(engine)
     for line in sys.stdin:

@@ -125,8 +125,113 @@ def dense_ff(h, W, p):
     return (silu(h @ W[p + "gate"].T) * (h @ W[p + "up"].T)) @ W[p + "down"].T
 
 
+# ------------------------------------------------------------------ Lebedra
+def rotate_pairs(x, pos, base):
+    """Interleaved rotation: components 2i and 2i + 1 of x [T, ..., n] turn by pos * base^(-2i / n)."""
+    n = x.shape[-1]
+    out = x.clone()
+    for i in range(n // 2):
+        a = pos.to(torch.float64) * float(base) ** (-2.0 * i / n)
+        c, s = torch.cos(a).to(x.dtype), torch.sin(a).to(x.dtype)
+        shape = [-1] + [1] * (x.dim() - 2)
+        c, s = c.view(shape), s.view(shape)
+        u, v = x[..., 2 * i], x[..., 2 * i + 1]
+        out[..., 2 * i], out[..., 2 * i + 1] = u * c - v * s, v * c + u * s
+    return out
+
+
+def sink_attention(q, k, v, scale, sink):
+    """Causal attention with one more term exp(sink[h]) in the denominator. q [T, H, dk]; k [T, H, dk]; v [T, H, dv]."""
+    T, H, _ = q.shape
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for h in range(H):
+        for t in range(T):
+            s = (k[: t + 1, h] @ q[t, h]) * scale
+            m = torch.maximum(s.max(), sink[h])
+            e = torch.exp(s - m)
+            out[t, h] = (e @ v[: t + 1, h]) / (e.sum() + torch.exp(sink[h] - m))
+    return out
+
+
+def latent_parts(h, W, p, c, eps, pos):
+    """(queries [T, H, dim + rot], latent [T, rank], shared rotated key [T, rot])."""
+    T, H, dn, dr, r = h.shape[0], c["heads"], c["dim"], c["rot_dim"], c["kv_rank"]
+    base = c["rot"]["base"]
+    q = (h @ W[p + "q"].T).view(T, H, dn + dr)
+    q = torch.cat([q[..., :dn], rotate_pairs(q[..., dn:], pos, base)], -1)
+    kv = h @ W[p + "dkv"].T
+    return q, rms_norm(kv[:, :r], W[p + "dkv.norm"], eps), rotate_pairs(kv[:, r:], pos, base)
+
+
+def latent_attention(h, W, p, c, eps):
+    T, H, dn, dv = h.shape[0], c["heads"], c["dim"], c["vdim"]
+    q, lat, kr = latent_parts(h, W, p, c, eps, torch.arange(T))
+    k = torch.cat([(lat @ W[p + "uk"].T).view(T, H, dn), kr[:, None, :].expand(T, H, kr.shape[1])], -1)
+    v = (lat @ W[p + "uv"].T).view(T, H, dv)
+    return sink_attention(q, k, v, c["scale"], W[p + "sink"]).reshape(T, H * dv) @ W[p + "o"].T
+
+
+def relu_ff(h, W, p):
+    return (torch.clamp(h @ W[p + "gate"].T, min=0) * (h @ W[p + "up"].T)) @ W[p + "down"].T
+
+
+def clamped_expert(h, W, p, limit):
+    g = torch.clamp(h @ W[p + "gate"].T, max=limit)
+    u = torch.clamp(h @ W[p + "up"].T, min=-limit, max=limit)
+    return (g * torch.sigmoid(1.702 * g) * (u + 1)) @ W[p + "down"].T
+
+
+def choose_experts(z, correction, r):
+    """Router logits of one token -> list of (expert, weight)."""
+    E, n, keep = r["experts"], r["groups"]["count"], r["groups"]["keep"]
+    s = torch.exp(z - z.max())
+    s = s / s.sum()
+    choice = (s + correction).tolist()
+    size = E // n
+    best = sorted(range(n), key=lambda g: -max(choice[g * size:(g + 1) * size]))[:keep]
+    allowed = [e for e in range(E) if e // size in best]
+    picked = sorted(allowed, key=lambda e: -choice[e])[: r["top"]]
+    return [(e, s[e]) for e in picked]
+
+
+def moe(h, W, p, c):
+    z = h @ W[p + "router"].T
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, w in choose_experts(z[t], W[p + "correction"], c["router"]):
+            out[t] += w * clamped_expert(h[t:t + 1], W, p + f"e{e}.", c["expert"]["limit"])[0]
+    return out
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1 + torch.tanh((2 / torch.pi) ** 0.5 * (z + 0.044715 * z ** 3)))
+
+
+def token_side(x, W, p, e, eps):
+    return rms_norm((gelu_tanh(x @ W[p + "gate"].T) * e) @ W[p + "proj"].T, W[p + "norm"], eps)
+
+
+def forward_lebedra(cfg, W, tokens, dtype=torch.float64, trace=None):
+    W = {k: v.to(dtype) for k, v in W.items()}
+    eps, m, n = cfg["norm"]["eps"], cfg["residual_mult"], cfg["token_side"]["dim"]
+    tok = torch.as_tensor(tokens, dtype=torch.long)
+    x = W["embed"][tok]
+    for i, L in enumerate(cfg["layers"]):
+        p = f"l{i}."
+        x = x + m * rms_norm(latent_attention(x, W, p + "mix.", L["mixer"], eps), W[p + "norm1"], eps)
+        if L["mlp"] is not None:
+            y = moe(x, W, p + "mlp.", L["mlp"]) if L["mlp"]["kind"] == "moe" else relu_ff(x, W, p + "mlp.")
+            x = x + m * rms_norm(y, W[p + "norm2"], eps)
+        x = x + m * token_side(x, W, p + "side.", W["side.embed"][tok][:, i * n:(i + 1) * n], eps)
+        if trace is not None:
+            trace.append(x)
+    return rms_norm(x, W["final.norm"], eps) @ W["head"].T
+
+
 def forward(cfg, W, tokens, dtype=torch.float64, trace=None):
     """Logits [T, vocab] of one sequence; ``trace`` (a list) receives the stream after every layer."""
+    if cfg["architecture"] == "Lebedra":
+        return forward_lebedra(cfg, W, tokens, dtype, trace)
     W = {k: v.to(dtype) for k, v in W.items()}
     eps = cfg["norm"]["eps"]
     tok = torch.as_tensor(tokens, dtype=torch.long)
