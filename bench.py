@@ -164,7 +164,7 @@ def run_reference_arm():
     return 0
 
 
-def run_hybrid() -> int:
+def run_hybrid(design: str) -> int:
     """Layer-list models beside the dense engine (mythos_b200/tools/hybrid_bench.py)."""
     from mythos_b200.tools import hybrid_bench
 
@@ -176,7 +176,7 @@ def run_hybrid() -> int:
         pass
     sampler = ClockSampler(0)
     sampler.start()
-    models, kernels = hybrid_bench.run_models(), hybrid_bench.run_kernels(peaks)
+    models, kernels = hybrid_bench.run_models(design), hybrid_bench.run_kernels(peaks, design=design)
     print(json.dumps({"metric": "hybrid prefill / decode throughput", "n_gpus": 1, "dtype": "bf16", "models": models,
                       "kernels": kernels, "clocks": sampler.stop(), "data": "random-init weights, uniform-random prompts"}))
     return 0
@@ -194,9 +194,9 @@ def main() -> int:
                     help="data-parallel gradient path: fused peer-memory kernels or plain NCCL collectives")
     ap.add_argument("--activation-checkpointing", action="store_true",
                     help="recompute block activations in the backward pass (memory for one extra forward)")
-    ap.add_argument("--hybrid", action="store_true",
-                    help="instead of the headline workload: prefill / decode throughput and kernel times of layer-list "
-                         "(Teganex) layers beside the dense engine of equal size, one JSON line (1 GPU)")
+    ap.add_argument("--hybrid", nargs="?", const="teganex", default=None, choices=["teganex", "lebedra"],
+                    help="instead of the headline workload: prefill / decode throughput and kernel times of layer-list layers "
+                         "of this design (default: teganex) beside the dense engine of equal size, one JSON line (1 GPU)")
     ap.add_argument("--no-decode", action="store_true", help="skip the tensor-parallel decode measurement")
     ap.add_argument("--decode-batch", type=int, default=64)
     ap.add_argument("--decode-prompt", type=int, default=1024)
@@ -210,7 +210,7 @@ def main() -> int:
 
     sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
     if args.hybrid:
-        return run_hybrid()
+        return run_hybrid(args.hybrid)
     from mythos_b200.models import DenseModel
     from mythos_b200.models.config import llama_1p3b_config
     from mythos_b200.ops import native

@@ -382,15 +382,13 @@ struct Latent {
   }
   bool decode_ok(int64_t page_size) const { return mb::latent_decode_ok(s, (int)page_size); }
   void attn_decode(const Tensor& q_lat, const Tensor& proj, const Tensor& row_seq, const Tensor& pos, const Tensor& table,
-                   const Tensor& cache, Tensor& o, Tensor& scratch, Tensor& counters, int64_t splits, const OptTensor& status) const {
+                   const Tensor& cache, Tensor& o, Tensor& scratch, int64_t splits, const OptTensor& status) const {
     const auto q = query(q_lat, proj, row_seq, pos, o, false);
     chk_c(scratch, F32, "scratch");
-    chk_c(counters, I32, "counters");
-    TORCH_CHECK(scratch.numel() >= (int64_t)q.rows * s.heads * splits * (s.rank_p + 2) &&
-                    counters.numel() >= (int64_t)q.rows * ((s.heads + 15) / 16), "attn_decode: scratch");
+    TORCH_CHECK(splits == 1 || scratch.numel() >= (int64_t)q.rows * s.heads * splits * (s.rank_p + 4), "attn_decode: scratch");
     c10::cuda::CUDAGuard guard(o.device());
     mb::latent_attn_decode(q, s, pages(table, cache, false, 0), sink.data_ptr<float>(), o.data_ptr(), scratch.data_ptr<float>(),
-                           counters.data_ptr<int>(), (int)splits, scale, status_ptr(status), cur_stream());
+                           (int)splits, scale, status_ptr(status), cur_stream());
   }
   bool prefill_ok(int64_t dim_p, int64_t vdim_p) const { return mb::flash_attn_ragged_ok((int)dim_p, s.rot_p, (int)vdim_p); }
   // q, kv: [rows, heads, width] views (unrotated queries; expanded keys and values), latents [keys, row], o [rows, heads, vdim]

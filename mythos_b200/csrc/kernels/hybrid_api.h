@@ -155,8 +155,9 @@ struct LatentQuery {
 void latent_attn_any(bool f32, const LatentQuery& q, const LatentSpec& s, const LatentPages& pg, const float* sink, void* out,
                      float scale, cudaStream_t stream);
 bool latent_decode_ok(const LatentSpec& s, int page_size);
+// scratch: rows * heads * splits * (rank_p + 4) floats (none with one split).
 void latent_attn_decode(const LatentQuery& q, const LatentSpec& s, const LatentPages& pg, const float* sink, void* out,
-                        float* scratch, int* counters, int splits, float scale, int* status, cudaStream_t stream);
+                        float* scratch, int splits, float scale, int* status, cudaStream_t stream);
 
 // ---- recurrences: S <- diag(g) S ; u = beta (v - S^T k) or u = v ; S <- S + k u^T ; o = S^T q
 // State layout: [slot][head][vdim][dim] fp32 (a row of S^T is contiguous).

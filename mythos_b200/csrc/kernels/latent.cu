@@ -6,7 +6,8 @@
 //                       them by one GEMM, and the attention kernel of attention_fwd.cu takes over)
 //   latent_attn_any     any widths, fp32 arithmetic, one warp per (token, head)
 //   latent_attn_decode  single tokens: 16 heads share every cached row that is read; the row serves as key
-//                       and, its latent columns, as value. Split over the context.
+//                       and, its latent columns, as value. Split over the context,
+//                       the splits' states merged by a second kernel.
 //
 // In the single-token forms the queries have been taken into the latent's space beforehand
 // (q_lat = W_uk^T q) and the output leaves it afterwards (W_uv), so nothing per head is cached.
@@ -19,44 +20,92 @@
 namespace mb {
 namespace {
 
-// One CTA per token. Angles: position x revolutions, reduced to a fraction of a turn in double precision.
+// 16 bytes of a row as floats.
 template <typename T>
-__global__ void __launch_bounds__(128)
+struct Vec16 {
+  static constexpr int N = 16 / (int)sizeof(T);
+  float v[N];
+  __device__ __forceinline__ void load(const T* p) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = ldf(e + i);
+  }
+  __device__ __forceinline__ void store(T* p) const {
+    uint4 raw;
+    T* e = reinterpret_cast<T*>(&raw);
+#pragma unroll
+    for (int i = 0; i < N; ++i) stf(e + i, v[i]);
+    *reinterpret_cast<uint4*>(p) = raw;
+  }
+  // Pairs (2i, 2i + 1) turned by the (cos, sin) entries cs[0 ..]
+  __device__ __forceinline__ void rotate(const float2* cs) {
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i) {
+      const float u = v[2 * i], w = v[2 * i + 1];
+      v[2 * i] = u * cs[i].x - w * cs[i].y;
+      v[2 * i + 1] = w * cs[i].x + u * cs[i].y;
+    }
+  }
+};
+
+// One warp per token. Angles: position x revolutions, reduced to a fraction of a turn in double precision. Padded
+// columns of the projection are zero, and so are those of a page row.
+constexpr int LP_WARPS = 4;
+template <typename T>
+__global__ void __launch_bounds__(LP_WARPS * 32)
 latent_prep_kernel(T* __restrict__ proj, long long ld, int qr_off, int c_off, int kr_off, const float* __restrict__ gamma,
                    const double* __restrict__ turns, LatentSpec s, RaggedBatch rb, LatentPages pg, float eps) {
-  extern __shared__ float2 cs[];
-  __shared__ float scratch[32];
-  const int t = blockIdx.x, half = s.rot / 2, pos = rb.pos[t];
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    const double a = pos * turns[i];
-    float sn, co;
-    sincospif(2.f * (float)(a - rint(a)), &sn, &co);
+  constexpr int N = Vec16<T>::N;
+  extern __shared__ float2 cs_all[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * LP_WARPS + warp;
+  if (t >= rb.rows) return;
+  float2* cs = cs_all + warp * (s.rot_p / 2);
+  const int pos = rb.pos[t];
+  const int page = pg.table[(long long)rb.row_seq[t] * pg.stride + pos / pg.page_size];
+  for (int i = lane; i < s.rot_p / 2; i += 32) {
+    float sn = 0.f, co = 1.f;
+    if (i < s.rot / 2) {
+      const double a = pos * turns[i];
+      sincospif(2.f * (float)(a - rint(a)), &sn, &co);
+    }
     cs[i] = make_float2(co, sn);
   }
   T* row = proj + (long long)t * ld;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < s.rank; i += blockDim.x) {
-    const float v = ldf(row + c_off + i);
-    ss += v * v;
+  for (int i = lane * N; i < s.rank_p; i += 32 * N) {
+    Vec16<T> x;
+    x.load(row + c_off + i);
+#pragma unroll
+    for (int j = 0; j < N; ++j) ss = fmaf(x.v[j], x.v[j], ss);
   }
-  ss = block_sum(ss, scratch);               // also orders cs
-  const int page = pg.table[(long long)rb.row_seq[t] * pg.stride + pos / pg.page_size];
+  ss = warp_sum(ss);
+  __syncwarp();                              // cs is complete
   if (page >= 0) {
     T* dst = static_cast<T*>(pg.cache) + ((long long)page * pg.page_size + pos % pg.page_size) * s.row();
     const float r = 1.f / sqrtf(ss / (float)s.rank + eps);
-    for (int i = threadIdx.x; i < s.rank; i += blockDim.x) stf(dst + i, ldf(row + c_off + i) * r * gamma[i]);
-    for (int i = threadIdx.x; i < half; i += blockDim.x) {
-      const float u = ldf(row + kr_off + 2 * i), v = ldf(row + kr_off + 2 * i + 1);
-      stf(dst + s.rank_p + 2 * i, u * cs[i].x - v * cs[i].y);
-      stf(dst + s.rank_p + 2 * i + 1, v * cs[i].x + u * cs[i].y);
+    for (int i = lane * N; i < s.rank_p; i += 32 * N) {
+      Vec16<T> x;
+      x.load(row + c_off + i);
+#pragma unroll
+      for (int j = 0; j < N; ++j) x.v[j] *= i + j < s.rank ? r * gamma[i + j] : 0.f;
+      x.store(dst + i);
+    }
+    for (int i = lane * N; i < s.rot_p; i += 32 * N) {
+      Vec16<T> x;
+      x.load(row + kr_off + i);
+      x.rotate(cs + i / 2);
+      x.store(dst + s.rank_p + i);
     }
   }
-  for (int j = threadIdx.x; j < s.heads * half; j += blockDim.x) {
-    const int h = j / half, i = j % half;
-    T* q = row + qr_off + h * s.rot_p + 2 * i;
-    const float u = ldf(q), v = ldf(q + 1);
-    stf(q, u * cs[i].x - v * cs[i].y);
-    stf(q + 1, v * cs[i].x + u * cs[i].y);
+  const int per = s.rot_p / N;               // vectors per head
+  for (int j = lane; j < s.heads * per; j += 32) {
+    Vec16<T> x;
+    T* q = row + qr_off + j * N;
+    x.load(q);
+    x.rotate(cs + (j % per) * (N / 2));
+    x.store(q);
   }
 }
 
@@ -149,14 +198,14 @@ struct LdLayout {
 __host__ __device__ inline LdLayout ld_layout(int row) {
   LdLayout l;
   l.chunks = (row + 63) / 64;
-  const int fixed = l.chunks * 16 * 128 + 2 * 16 * LD_SLD * 4 + 16 * 128 + 16 * (LD_MAX_SPLITS + 2) * 4 + 1024;
+  const int fixed = l.chunks * 16 * 128 + 2 * 16 * LD_SLD * 4 + 16 * 128 + 64 + 1024;
   l.stages = (220 * 1024 - fixed) / (l.chunks * LD_CHUNK);
   if (l.stages > LD_MAX_STAGES) l.stages = LD_MAX_STAGES;
   l.off_q = l.stages * l.chunks * LD_CHUNK;
   l.off_p = l.off_q + l.chunks * 16 * 128;
   l.off_s = l.off_p + 16 * 128;
   l.off_w = l.off_s + 2 * 16 * LD_SLD * 4;
-  l.bytes = l.off_w + 16 * (LD_MAX_SPLITS + 2) * 4 + 1024;
+  l.bytes = l.off_w + 64 + 1024;
   return l;
 }
 
@@ -179,16 +228,15 @@ template <int NT>
 __global__ void __launch_bounds__(LD_THREADS, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tm_c, LatentQuery q, LatentSpec s, LatentPages pg,
                      const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, float* __restrict__ scratch,
-                     int* __restrict__ counters, int splits, float scale_log2, int* status) {
+                     int splits, float scale_log2, int* status) {
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t full[LD_MAX_STAGES];
-  __shared__ int abort_word, s_last;
+  __shared__ int abort_word;
   volatile int* abort_flag = &abort_word;
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
   const LdLayout L = ld_layout(s.row());
   float* s_part = reinterpret_cast<float*>(smem + L.off_s);
   float* s_alpha = reinterpret_cast<float*>(smem + L.off_w);        // [16]
-  float* s_w = s_alpha + 32;                                        // [16][splits]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int b = blockIdx.x, h0 = blockIdx.y * 16, G = min(16, s.heads - h0), split = blockIdx.z;
   if (threadIdx.x == 0) {
@@ -247,24 +295,28 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_c, LatentQuery q, La
     ok = mbar_wait(&full[st], (j / L.stages) & 1, abort_flag, status, 110);
     if (!__syncthreads_and(ok)) { ok = false; break; }
     const uint32_t tile = kv_addr + st * L.chunks * LD_CHUNK;
-    // ---- scores
-    float sc[2][4];
+    // ---- scores: two independent chains of products
+    float sc[2][2][4];
 #pragma unroll
-    for (int i = 0; i < 2; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
+    for (int i = 0; i < 8; ++i) sc[i >> 2][(i >> 1) & 1][(i & 1) * 2] = sc[i >> 2][(i >> 1) & 1][(i & 1) * 2 + 1] = 0.f;
     const int half = L.chunks * 2;                                  // 16-column steps per half
-    for (int ks = kh * half; ks < (kh + 1) * half; ++ks) {
-      const int c = ks >> 2, u = (ks & 3) << 1;
-      uint32_t qa[4], kb[4];
-      ld_matrix4(q_addr + c * 2048 + sw128_offset(a_row, u + a_unit), qa);
-      ld_matrix4(tile + c * LD_CHUNK + sw128_offset(k_tok, u + k_unit), kb);
-      ld_mma(sc[0], qa, kb[0], kb[1]);
-      ld_mma(sc[1], qa, kb[2], kb[3]);
+#pragma unroll 2
+    for (int k0 = kh * half; k0 < (kh + 1) * half; k0 += 2) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int c = (k0 + e) >> 2, u = ((k0 + e) & 3) << 1;
+        uint32_t qa[4], kb[4];
+        ld_matrix4(q_addr + c * 2048 + sw128_offset(a_row, u + a_unit), qa);
+        ld_matrix4(tile + c * LD_CHUNK + sw128_offset(k_tok, u + k_unit), kb);
+        ld_mma(sc[e][0], qa, kb[0], kb[1]);
+        ld_mma(sc[e][1], qa, kb[2], kb[3]);
+      }
     }
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       float* dst = s_part + (kh * 16 + (lane >> 2)) * LD_SLD + tq * 16 + i * 8 + 2 * (lane & 3);
-      *reinterpret_cast<float2*>(dst) = make_float2(sc[i][0], sc[i][1]);
-      *reinterpret_cast<float2*>(dst + 8 * LD_SLD) = make_float2(sc[i][2], sc[i][3]);
+      *reinterpret_cast<float2*>(dst) = make_float2(sc[0][i][0] + sc[1][i][0], sc[0][i][1] + sc[1][i][1]);
+      *reinterpret_cast<float2*>(dst + 8 * LD_SLD) = make_float2(sc[0][i][2] + sc[1][i][2], sc[0][i][3] + sc[1][i][3]);
     }
     __syncthreads();
     // ---- softmax of the tile
@@ -329,63 +381,90 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_c, LatentQuery q, La
     while (clock64() - t0 < 10000000LL) {}
     __syncthreads();
   }
-  // ---- this split's state, then the last CTA of the (token, head group) merges
-  const int stride = s.rank_p + 2;
 #pragma unroll
   for (int d = 8; d > 0; d >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, d);
-  float* part = scratch + (((long long)b * s.heads + h0) * splits + split) * stride;     // head h: + h * splits * stride
-  if (slane == 0 && srow < G) {
-    part[(long long)srow * splits * stride + s.rank_p] = ok ? m_run : -INFINITY;
-    part[(long long)srow * splits * stride + s.rank_p + 1] = l_run;
-  }
+  const int r0 = lane >> 2;
+  if (splits == 1) {                            // nothing to merge: the sink, then the quotient
+    if (slane == 0) {
+      const float sk = srow < G ? sink[h0 + srow] * 1.4426950408889634f : -INFINITY, M = fmaxf(m_run, sk);
+      const float w = exp2f(m_run - M);
+      s_alpha[srow] = w / (w * l_run + exp2f(sk - M));
+    }
+    __syncthreads();
+    const float w0 = s_alpha[r0], w1 = s_alpha[r0 + 8];
+    __nv_bfloat16* dst = out + ((long long)b * s.heads + h0) * s.rank_p;
 #pragma unroll
-  for (int n = 0; n < NT; ++n) {
-    const int col = col0 + n * 8 + 2 * (lane & 3), r = lane >> 2;
-    if (col < s.rank_p) {
-      if (r < G) *reinterpret_cast<float2*>(part + (long long)r * splits * stride + col) = make_float2(o[n][0], o[n][1]);
-      if (r + 8 < G)
-        *reinterpret_cast<float2*>(part + (long long)(r + 8) * splits * stride + col) = make_float2(o[n][2], o[n][3]);
-    }
-  }
-  __threadfence();
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    int* c = &counters[b * gridDim.y + blockIdx.y];
-    s_last = atomicAdd(c, 1) == splits - 1;
-    if (s_last) *c = 0;
-  }
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
-  const float* base = scratch + ((long long)b * s.heads + h0) * splits * stride;
-  if (threadIdx.x < G) {
-    const int h = threadIdx.x;
-    const float* p = base + (long long)h * splits * stride + s.rank_p;
-    const float sk = sink[h0 + h] * 1.4426950408889634f;
-    float M = sk;
-    for (int i = 0; i < splits; ++i) M = fmaxf(M, p[(long long)i * stride]);
-    float sum = exp2f(sk - M);
-    for (int i = 0; i < splits; ++i) {
-      const float w = exp2f(p[(long long)i * stride] - M);
-      s_w[h * splits + i] = w;
-      sum += w * p[(long long)i * stride + 1];
-    }
-    for (int i = 0; i < splits; ++i) s_w[h * splits + i] /= sum;
-  }
-  __syncthreads();
-  for (int i = threadIdx.x; i < G * (s.rank_p / 2); i += LD_THREADS) {
-    const int h = i / (s.rank_p / 2), d = (i % (s.rank_p / 2)) * 2;
-    const float* p = base + (long long)h * splits * stride + d;
-    float y0 = 0.f, y1 = 0.f;
-    for (int k = 0; k < splits; ++k) {
-      const float w = s_w[h * splits + k];
-      const float2 v = *reinterpret_cast<const float2*>(p + (long long)k * stride);
-      if (w > 0.f) {                                                // an empty split's numbers are never used
-        y0 = fmaf(w, v.x, y0);
-        y1 = fmaf(w, v.y, y1);
+    for (int n = 0; n < NT; ++n) {
+      const int col = col0 + n * 8 + 2 * (lane & 3);
+      if (col < s.rank_p) {
+        if (r0 < G) *reinterpret_cast<uint32_t*>(dst + r0 * s.rank_p + col) = pack_bf16x2(o[n][0] * w0, o[n][1] * w0);
+        if (r0 + 8 < G) *reinterpret_cast<uint32_t*>(dst + (r0 + 8) * s.rank_p + col) = pack_bf16x2(o[n][2] * w1, o[n][3] * w1);
       }
     }
-    *reinterpret_cast<uint32_t*>(out + ((long long)b * s.heads + h0 + h) * s.rank_p + d) = pack_bf16x2(y0, y1);
+    return;
+  }
+  // this split's state: the weighted latents, then maximum and sum
+  const int stride = s.rank_p + 4;
+  float* part = scratch + (((long long)b * s.heads + h0) * splits + split) * stride;     // head h: + h * splits * stride
+  if (slane == 0 && srow < G)
+    *reinterpret_cast<float2*>(part + (long long)srow * splits * stride + s.rank_p) = make_float2(ok ? m_run : -INFINITY, l_run);
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    const int col = col0 + n * 8 + 2 * (lane & 3);
+    if (col < s.rank_p) {
+      if (r0 < G) *reinterpret_cast<float2*>(part + (long long)r0 * splits * stride + col) = make_float2(o[n][0], o[n][1]);
+      if (r0 + 8 < G)
+        *reinterpret_cast<float2*>(part + (long long)(r0 + 8) * splits * stride + col) = make_float2(o[n][2], o[n][3]);
+    }
+  }
+}
+
+// One CTA per (token, head): the splits' states and the sink into one result.
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(const float* __restrict__ scratch, const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int heads,
+                    int rank_p, int splits) {
+  __shared__ float s_w[LD_MAX_SPLITS], s_sum;
+  const int stride = rank_p + 4;
+  const float* base = scratch + (long long)blockIdx.x * splits * stride;
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    float2 ml[2];
+    const float sk = sink[blockIdx.x % heads] * 1.4426950408889634f;
+    float M = sk;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int k = lane + 32 * i;
+      ml[i] = k < splits ? *reinterpret_cast<const float2*>(base + (long long)k * stride + rank_p) : make_float2(-INFINITY, 0.f);
+      M = fmaxf(M, ml[i].x);
+    }
+    M = warp_max(M);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const float w = exp2f(ml[i].x - M);
+      s_w[lane + 32 * i] = w;
+      if (w > 0.f) sum += w * ml[i].y;
+    }
+    sum = warp_sum(sum) + exp2f(sk - M);
+    if (lane == 0) s_sum = 1.f / sum;
+  }
+  __syncthreads();
+  const float inv = s_sum;
+  for (int d = threadIdx.x * 4; d < rank_p; d += 512) {
+    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int k = 0; k < splits; ++k) {
+      const float4 v = *reinterpret_cast<const float4*>(base + (long long)k * stride + d);
+      const float w = s_w[k];
+      if (w > 0.f) {                            // an empty split's numbers are never used
+        y.x = fmaf(w, v.x, y.x);
+        y.y = fmaf(w, v.y, y.y);
+        y.z = fmaf(w, v.z, y.z);
+        y.w = fmaf(w, v.w, y.w);
+      }
+    }
+    *reinterpret_cast<uint2*>(out + (long long)blockIdx.x * rank_p + d) =
+        make_uint2(pack_bf16x2(y.x * inv, y.y * inv), pack_bf16x2(y.z * inv, y.w * inv));
   }
 }
 
@@ -394,14 +473,16 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_c, LatentQuery q, La
 void latent_prep(bool f32, void* proj, long long ld, int qr_off, int c_off, int kr_off, const float* gamma,
                  const double* turns, const LatentSpec& s, const RaggedBatch& rb, const LatentPages& pg, float eps,
                  cudaStream_t stream) {
-  MB_REQUIRE(s.rot > 0 && s.rot % 2 == 0 && s.rot <= 4096, "latent_prep: rotated width");
+  MB_REQUIRE(s.rot > 0 && s.rot % 2 == 0 && s.rot <= 2048, "latent_prep: rotated width");
+  MB_REQUIRE(ld % 8 == 0 && ((qr_off | c_off | kr_off) & 7) == 0, "latent_prep: columns in units of 8");
   if (rb.rows == 0) return;
-  const int smem = s.rot / 2 * (int)sizeof(float2);
+  const int smem = LP_WARPS * (s.rot_p / 2) * (int)sizeof(float2), grid = (rb.rows + LP_WARPS - 1) / LP_WARPS;
   if (f32)
-    latent_prep_kernel<float><<<rb.rows, 128, smem, stream>>>((float*)proj, ld, qr_off, c_off, kr_off, gamma, turns, s, rb, pg, eps);
+    latent_prep_kernel<float><<<grid, LP_WARPS * 32, smem, stream>>>((float*)proj, ld, qr_off, c_off, kr_off, gamma, turns, s, rb,
+                                                                     pg, eps);
   else
-    latent_prep_kernel<__nv_bfloat16><<<rb.rows, 128, smem, stream>>>((__nv_bfloat16*)proj, ld, qr_off, c_off, kr_off, gamma,
-                                                                       turns, s, rb, pg, eps);
+    latent_prep_kernel<__nv_bfloat16><<<grid, LP_WARPS * 32, smem, stream>>>((__nv_bfloat16*)proj, ld, qr_off, c_off, kr_off, gamma,
+                                                                             turns, s, rb, pg, eps);
   count_launch();
   check_launch();
 }
@@ -440,7 +521,7 @@ bool latent_decode_ok(const LatentSpec& s, int page_size) {
 }
 
 void latent_attn_decode(const LatentQuery& q, const LatentSpec& s, const LatentPages& pg, const float* sink, void* out,
-                        float* scratch, int* counters, int splits, float scale, int* status, cudaStream_t stream) {
+                        float* scratch, int splits, float scale, int* status, cudaStream_t stream) {
   MB_REQUIRE(latent_decode_ok(s, pg.page_size), "latent_attn_decode: widths or page size");
   MB_REQUIRE(splits >= 1 && splits <= LD_MAX_SPLITS && q.ld_qr % 8 == 0, "latent_attn_decode: splits / stride");
   if (q.rows == 0) return;
@@ -451,7 +532,7 @@ void latent_attn_decode(const LatentQuery& q, const LatentSpec& s, const LatentP
   const dim3 grid(q.rows, (s.heads + 15) / 16, splits);
   auto go = [&](auto kern) {
     MB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    kern<<<grid, LD_THREADS, smem, stream>>>(tc, q, s, pg, sink, (__nv_bfloat16*)out, scratch, counters, splits,
+    kern<<<grid, LD_THREADS, smem, stream>>>(tc, q, s, pg, sink, (__nv_bfloat16*)out, scratch, splits,
                                              scale * 1.4426950408889634f, status);
   };
   if (s.rank_p <= 128) go(latent_decode_kernel<2>);
@@ -459,6 +540,11 @@ void latent_attn_decode(const LatentQuery& q, const LatentSpec& s, const LatentP
   else go(latent_decode_kernel<8>);
   count_launch();
   check_launch();
+  if (splits > 1) {
+    latent_merge_kernel<<<q.rows * s.heads, 128, 0, stream>>>(scratch, sink, (__nv_bfloat16*)out, s.heads, s.rank_p, splits);
+    count_launch();
+    check_launch();
+  }
 }
 
 }  // namespace mb

@@ -132,10 +132,7 @@ class HybridEngine(InferenceEngine):
         self.H = native.require_hybrid() if self.device.type == "cuda" else None
         self._status = native.status_word(self.device)
         groups = max([m.kv_heads * ((m.heads // m.kv_heads + 7) // 8) for m in att] or [1])
-        latent_groups = max([(s.latent.heads + 15) // 16 for s in cfg.layers if s.latent is not None] or [0])
-        # tokens that can attend in the latent's space in one pass: short portions only
-        self._counters = torch.zeros(max(max_batch * groups, max_batch * EXPAND_TOKENS * latent_groups), device=self.device,
-                                     dtype=torch.int32)
+        self._counters = torch.zeros(max_batch * groups, device=self.device, dtype=torch.int32)
         experts = max([s.mlp.experts for s in cfg.layers if isinstance(s.mlp, MoeFF)] or [0])
         self._expert_counts = torch.zeros(experts + 1, device=self.device, dtype=torch.int32)
         self._max_ctx = self.max_seq_len
@@ -399,16 +396,20 @@ class HybridEngine(InferenceEngine):
         q_lat = torch.empty(n, H, r_p, device=self.device, dtype=self.dtype)
         o_lat = torch.empty_like(q_lat)
         self.H.gemm_heads(q, L.uk_t, q_lat, self._status)
-        groups = (H + 15) // 16
-        if self._fast and n * groups <= self._counters.numel() and L.lat.decode_ok(self.page_size):
-            splits = max(1, min(64, (self._sms + n * groups - 1) // (n * groups), (ctx.max_kv + 127) // 128))
-            scratch = torch.empty(n * H * splits * (r_p + 2), device=self.device, dtype=torch.float32)
-            L.lat.attn_decode(q_lat, proj, row_seq, pos, ctx.table, cache, o_lat, scratch, self._counters, splits, self._status)
+        if self._fast and L.lat.decode_ok(self.page_size):
+            splits = self._latent_splits(n, H, ctx.max_kv)
+            scratch = torch.empty(n * H * splits * (r_p + 4) if splits > 1 else 0, device=self.device, dtype=torch.float32)
+            L.lat.attn_decode(q_lat, proj, row_seq, pos, ctx.table, cache, o_lat, scratch, splits, self._status)
         else:
             L.lat.attn_any(q_lat, proj, row_seq, pos, ctx.table, cache, o_lat)
         out = torch.empty(n, H, L.uv.shape[1], device=self.device, dtype=self.dtype)
         self.H.gemm_heads(o_lat, L.uv, out, self._status)
         return out
+
+    def _latent_splits(self, rows: int, heads: int, max_kv: int) -> int:
+        """At most one CTA per SM (a CTA fills one), and two 64-token tiles of work for each."""
+        pairs = rows * ((heads + 15) // 16)
+        return max(1, min(64, self._sms // pairs, (max_kv + 127) // 128))
 
     def _latent(self, L, h, ctx):
         m, H = L.spec.mixer, L.spec.mixer.heads
@@ -432,17 +433,18 @@ class HybridEngine(InferenceEngine):
         return self._gemm(o.flatten(1), L.out), None
 
     # ---- feed-forwards
+    def _expert_tile(self, rows: int, m) -> int:
+        """Rows of a tile of the grouped GEMMs, from the mean rows per expert."""
+        mean = rows * m.top // m.experts
+        if self.f32:
+            return 64
+        return 128 if mean >= SEGMENT_GEMM_ROWS else max(16, min(64, 1 << (2 * mean).bit_length()))
+
     def _experts(self, L, h, ctx):
         """Outputs of the chosen experts [rows * top, d], where each (token, choice) lies and its weight."""
         m, T, C = L.spec.mlp, ctx.rows, self.H
         z = self._gemm(h, L.router, dtype=torch.float32)
-        pairs = T * m.top
-        if self.f32:
-            tile = 64
-        elif pairs >= SEGMENT_GEMM_ROWS * m.experts:
-            tile = 128
-        else:
-            tile = max(16, min(64, 1 << (2 * pairs // m.experts).bit_length()))
+        pairs, tile = T * m.top, self._expert_tile(T, m)
         i32 = dict(device=self.device, dtype=torch.int32)
         idx, slot, row = (torch.empty(T, m.top, **i32) for _ in range(3))
         weight = torch.empty(T, m.top, device=self.device, dtype=torch.float32)

@@ -1,5 +1,6 @@
-"""Speed of layer-list models (Teganex layers at the sizes of a real model, random weights) beside the
-dense transformer engine of equal width, depth and feed-forward, both with bf16 weights.
+"""Speed of layer-list models (Teganex or Lebedra layers at the sizes of a real model, random weights) beside
+the dense transformer engine of equal width, depth and feed-forward (Lebedra: the dense layer's, and the experts of
+a token together about as wide), both with bf16 weights.
 
 ``run_models``: prefill and decode throughput of both engines. ``run_kernels``: every kernel of the new
 design next to the like kernel of the dense model, with the fraction of its roofline (bytes over the
@@ -24,13 +25,14 @@ def _dense_config(width, layers, vocab, max_len):
                              weight_format="bf16", embed_format="bf16")
 
 
-def _engines(width, layers, vocab, batch, max_len):
+def _engines(design, width, layers, vocab, batch, max_len):
     from ..infer.engine import InferenceEngine
     from ..infer.hybrid import HybridEngine
-    from ..models.hybrid_config import teganex_config
+    from ..models import hybrid_config as hc
 
     kw = dict(seed=1, device="cuda", max_batch=batch, max_seq_len=max_len)
-    yield "teganex", HybridEngine.random(teganex_config(width, layers, vocab, max_len), **kw)
+    make = {"teganex": hc.teganex_config, "lebedra": hc.lebedra_config}[design]
+    yield design, HybridEngine.random(make(width, layers, vocab, max_len), **kw)
     yield "dense", InferenceEngine.random(_dense_config(width, layers, vocab, max_len), **kw)
 
 
@@ -70,13 +72,13 @@ def _prefill_ms(eng, batch, length, iters=4):
     return statistics.median(ms)
 
 
-def run_models(sizes=((2048, 8), (4096, 8)), vocab: int = 32000, prefill=((4, 2048), (1, 8192)),
+def run_models(design: str = "teganex", sizes=((2048, 8), (4096, 8)), vocab: int = 32000, prefill=((4, 2048), (1, 8192)),
                decode=((1, 1024), (16, 1024), (64, 1024)), new_tokens: int = 64) -> list[dict]:
     out = []
     for width, layers in sizes:
         max_len = max(max(n for _, n in prefill), max(n for _, n in decode) + new_tokens) + PAGE
         max_batch = max(max(b for b, _ in prefill), max(b for b, _ in decode))
-        for name, eng in _engines(width, layers, vocab, max_batch, max_len):
+        for name, eng in _engines(design, width, layers, vocab, max_batch, max_len):
             rec = {"model": name, "width": width, "layers": layers, "weight_mb": round(eng.weight_bytes() / 1e6), "prefill": [],
                    "decode": []}
             for b, n in prefill:
@@ -154,7 +156,136 @@ def _recurrent_rows(K, H, st, kind, heads, dim, vdim, lens, decode):
     K.add("chunked recurrence + norm + gate", sizes, fn, nbytes=io + state, like="paged prefill attention (dense)")
 
 
-def run_kernels(peaks: dict, width: int = 2048) -> list[dict]:
+def _dense_attention_rows(K, H, C, st, rnd, h, kv):
+    """Prefill and decode attention of the dense engine, for comparison."""
+    bf, B, S = torch.bfloat16, 4, 2048
+    pages = B * S // PAGE
+    table = torch.randperm(pages, device="cuda").to(torch.int32).view(B, -1)
+    kc, vc, q, o = rnd(pages, PAGE, kv, 128), rnd(pages, PAGE, kv, 128), rnd(B * S, h, 128), rnd(B * S, h, 128)
+    b = _batch([S] * B, [0] * B)
+    K.add("paged prefill attention (dense)", f"{B} x {S}, {h}/{kv} heads, 128",
+          lambda: C.flash_attn_paged_prefill(q, kc, vc, table, b[0], b[1], o, S, 128 ** -0.5, st),
+          flops=2.0 * B * h * (S * (S + 1) / 2) * 256)
+    sms = torch.cuda.get_device_properties(0).multi_processor_count
+    for NB, ctx in ((16, 4096), (64, 1024)):
+        pages = NB * ctx // PAGE
+        table = torch.randperm(pages, device="cuda").to(torch.int32).view(NB, -1)
+        kc, vc, q, o = rnd(pages, PAGE, kv, 128), rnd(pages, PAGE, kv, 128), rnd(NB, h, 128), rnd(NB, h, 128)
+        splits = max(1, min(32, (6 * sms + NB * kv - 1) // (NB * kv), (ctx + 255) // 256))
+        b = _batch([1] * NB, [ctx - 1] * NB)
+        scratch, cnt = torch.empty(NB * h * splits * 130, device="cuda"), torch.zeros(NB * kv, device="cuda", dtype=torch.int32)
+        K.add("paged decode attention (dense)", f"{NB} x {ctx}, {h}/{kv} heads, 128",
+              lambda: C.paged_attn_decode(q, kc, vc, table, b[1], o, scratch, cnt, splits, 128 ** -0.5, st),
+              nbytes=4.0 * NB * ctx * kv * 128)
+
+
+def run_lebedra_kernels(peaks: dict, width: int = 2048) -> list[dict]:
+    """Latent attention (latents of 512, heads of 128 + 64 rotated), routed experts and the norms around them."""
+    from ..infer.hybrid import HybridEngine
+    from ..models.hybrid_config import lebedra_config
+    from ..ops import functional as F, native
+
+    H, C, st = native.require_hybrid(), native.require(), native.status_word("cuda")
+    K, bf, d = _Kernels(peaks), torch.bfloat16, width
+    rnd = lambda *s: torch.randn(*s, device="cuda").to(bf)
+    cfg = lebedra_config(width, 2, 1024)
+    eng = HybridEngine.random(cfg, device="cuda", max_batch=64, max_seq_len=4096, kv_pages=64)
+    L, m, e = eng.layers[1], cfg.layers[1].mixer, cfg.layers[1].mlp
+    h, r, W = m.heads, m.kv_rank, m.kv_rank + m.rot_dim
+    _dense_attention_rows(K, H, C, st, rnd, h, max(1, h // 8))
+    # ---- attention
+    def pages(B, S):
+        return torch.randperm(B * S // PAGE, device="cuda").to(torch.int32).view(B, -1), rnd(B * S // PAGE, PAGE, 1, W)
+
+    for B, S in ((4, 2048), (1, 8192)):
+        table, cache = pages(B, S)
+        b, n = _batch([S] * B, [0] * B), B * S
+        proj, o = rnd(n, L.proj.N), torch.empty(n, h, m.vdim, device="cuda", dtype=bf)
+        lat, kv = torch.empty(n, W, device="cuda", dtype=bf), rnd(n, h * (m.dim + m.vdim))
+        q, k, v = (t.unflatten(1, (h, 128)) for t in (proj[:, : h * m.dim], kv[:, : h * m.dim], kv[:, h * m.dim:]))
+        K.add("latent_prep", f"{n} tokens, {h} heads", lambda: L.lat.prep(proj, b, table, cache),
+              nbytes=2.0 * n * (2 * h * m.rot_dim + 2 * W), like="rope (dense)")
+        K.add("latent_gather", f"{n} tokens", lambda: L.lat.gather(table, cache, b[0], S, lat), nbytes=4.0 * n * W, like="rope (dense)")
+        K.add("expand latents (GEMM)", f"{n} x {L.expand.shape[0]} x {r}", lambda: H.gemm_nt(lat[:, :r], L.expand, kv, 1.0, st),
+              flops=2.0 * n * L.expand.shape[0] * r, like="gemm (dense bf16)")
+        K.add("latent prefill attention", f"{B} x {S}, {h} heads, 128 + 64 / 128",
+              lambda: L.lat.attn_prefill(q, proj, k, v, lat, b, b[0], S, 16, o, st),
+              flops=2.0 * B * h * (S * (S + 1) / 2) * (m.dim + m.rot_dim + m.vdim), like="paged prefill attention (dense)")
+    qkv, pos = rnd(8192, h + 2, 128), torch.arange(2048, device="cuda", dtype=torch.int32).repeat(4)
+    K.add("rope (dense)", f"8192 tokens, {h} heads, 128", lambda: C.rope(qkv[:, :h], pos, 10000.0, False), nbytes=4.0 * 8192 * h * 128)
+    for NB, ctx in ((1, 4096), (16, 4096), (64, 1024)):
+        table, cache = pages(NB, ctx)
+        b, proj = _batch([1] * NB, [ctx - 1] * NB), rnd(NB, L.proj.N)
+        ql, ol, out = rnd(NB, h, r), rnd(NB, h, r), rnd(NB, h, m.vdim)
+        q = proj[:, : h * m.dim].unflatten(1, (h, m.dim))
+        K.add("W_uk per head", f"{NB} tokens, {h} heads", lambda: H.gemm_heads(q, L.uk_t, ql, st),
+              nbytes=2.0 * (L.uk_t.numel() + NB * h * (m.dim + r)), like="gemm_decode")
+        splits = eng._latent_splits(NB, h, ctx)
+        sc = torch.empty(NB * h * splits * (r + 4), device="cuda")
+        K.add("latent decode attention", f"{NB} x {ctx}, {h} heads", lambda: L.lat.attn_decode(
+            ql, proj, b[3], b[4], table, cache, ol, sc, splits, st),
+            nbytes=2.0 * NB * (ctx * W + h * (W + r)), flops=2.0 * NB * h * ctx * (W + r), like="paged decode attention (dense)")
+        K.add("W_uv per head", f"{NB} tokens, {h} heads", lambda: H.gemm_heads(ol, L.uv, out, st),
+              nbytes=2.0 * (L.uv.numel() + NB * h * (m.vdim + r)), like="gemm_decode")
+        N = h * r
+        x, w, y = rnd(NB, m.dim * 4), rnd(N // 4, m.dim * 4), rnd(NB, N // 4)
+        K.add("gemm_decode", f"{NB} x {N // 4} x {m.dim * 4}", lambda: H.gemm_decode(x, w, y, 0, 0, 1.0, st),
+              nbytes=2.0 * (w.numel() + x.numel() + y.numel()))
+    # ---- experts
+    route = (e.experts, e.top, e.groups, e.keep)
+    i32 = dict(device="cuda", dtype=torch.int32)
+    f, gen = e.ff, torch.Generator().manual_seed(5)
+    for T in (1, 16, 64, 1024, 8192):
+        pairs, tile = T * e.top, eng._expert_tile(T, e)
+        z = torch.randn(T, e.experts, generator=gen).cuda()
+        idx, slot, row = (torch.empty(T, e.top, **i32) for _ in range(3))
+        wt, off, cnt = torch.empty(T, e.top, device="cuda"), torch.empty(e.experts, **i32), torch.empty(1, **i32)
+        tiles = torch.empty(min(pairs, e.experts + pairs // tile), 3, **i32)
+        plan = (idx, wt, slot, eng._expert_counts, off, tiles, cnt)
+        x, hid, a, y = rnd(pairs, d), rnd(T, d), rnd(pairs, f), rnd(pairs, d)
+        sizes = f"{T} tokens, {e.top} of {e.experts}, {d} x {f}"
+        K.add("expert_select", sizes, lambda: H.expert_select(z, L.correction, route, tile, *plan), nbytes=4.0 * T * e.experts,
+              like="moe_route (training)")
+        probs, psum, lg = torch.empty(T, e.experts, device="cuda"), torch.zeros(e.experts, device="cuda"), z.to(bf)
+        cn = torch.zeros(e.experts, **i32)
+        K.add("moe_route (training)", sizes, lambda: C.moe_route(lg, e.experts, probs, idx, slot, wt, cn, psum), nbytes=2.0 * T * e.experts)
+        H.expert_select(z, L.correction, route, tile, *plan)
+        used = int((torch.bincount(idx.flatten().long(), minlength=e.experts) > 0).sum())
+        K.add("expert_gather", sizes, lambda: H.expert_gather(hid, route, *plan, x, row), nbytes=2.0 * d * (T + pairs), like="rope (dense)")
+        K.add("experts in (gate, up)", sizes, lambda: H.gemm_tiles(x, L.w_in, a, tiles, cnt, tile, f, f, L.act, st),
+              nbytes=2.0 * (used * 2 * f * d + pairs * (d + f)), flops=4.0 * pairs * f * d, like="gemm (dense bf16)")
+        K.add("experts out (down)", sizes, lambda: H.gemm_tiles(a, L.w_out, y, tiles, cnt, tile, 0, 0, L.act, st),
+              nbytes=2.0 * (used * f * d + pairs * (d + f)), flops=2.0 * pairs * f * d, like="gemm (dense bf16)")
+        for N, Kd in ((2 * f * e.top, d), (d, f * e.top)):         # the dense layer of the same width
+            xx, ww, o1 = rnd(T, Kd), rnd(N, Kd), torch.empty(T, N, device="cuda", dtype=bf)
+            K.add("gemm (dense bf16)", f"{T} x {N} x {Kd}", lambda: F.gemm(xx, ww, out=o1), nbytes=2.0 * (N * Kd + T * (N + Kd)),
+                  flops=2.0 * T * N * Kd)
+        xs, w32, hh = torch.randn(T, d, device="cuda"), torch.ones(d, device="cuda"), rnd(T, d)
+        K.add("expert_norm", f"{T} x {d}, {e.top} outputs", lambda: H.expert_norm(y, row, wt, w32, xs, None, hh, 1e-6, 0.5),
+              nbytes=T * d * (2.0 * e.top + 10), like="rmsnorm + residual (dense)")
+        K.add("norm + residual", f"{T} x {d}", lambda: H.sandwich_norm(hh, None, None, None, w32, xs, None, x[:T], 1e-6, 0.5),
+              nbytes=T * d * 12.0, like="rmsnorm + residual (dense)")
+        g, res = torch.ones(d, device="cuda", dtype=bf), rnd(T, d)
+        K.add("rmsnorm + residual (dense)", f"{T} x {d}", lambda: F.rmsnorm(hh, g, 1e-6, res), nbytes=T * d * 8.0)
+        # ---- token side and router
+        n, ids = cfg.token_side, torch.zeros(T, **i32)
+        sg = torch.empty(T, n, device="cuda", dtype=bf)
+        K.add("side gate", f"{T} x {n} x {d}", lambda: H.gemm_decode(hid, L.side_gate, sg, 0, 0, 1.0, st, (0, 0.0, 0.0), L.side_embed, ids),
+              nbytes=2.0 * (n * d + T * (d + 2 * n)), flops=2.0 * T * n * d, like="gemm (dense bf16), narrow")
+        K.add("gemm (dense bf16), narrow", f"{T} x {n} x {d}", lambda: F.gemm(hid, L.side_gate, out=sg), nbytes=2.0 * (n * d + T * (d + n)),
+              flops=2.0 * T * n * d)
+        K.add("side projection", f"{T} x {d} x {n}", lambda: eng._gemm(sg, L.side_proj, out=hh), nbytes=2.0 * (n * d + T * (d + n)),
+              flops=2.0 * T * n * d, like="gemm (dense bf16), narrow")
+        zz = torch.empty(T, e.experts, device="cuda")
+        K.add("router", f"{T} x {e.experts} x {d}", lambda: eng._gemm(hid, L.router, out=zz),
+              nbytes=2.0 * (e.experts * d + T * (d + 2 * e.experts)), flops=2.0 * T * e.experts * d, like="gemm (dense bf16), narrow")
+    native.check_status("cuda")
+    return K.rows
+
+
+def run_kernels(peaks: dict, width: int = 2048, design: str = "teganex") -> list[dict]:
+    if design == "lebedra":
+        return run_lebedra_kernels(peaks, width)
     from ..ops import functional as F, native
 
     H, C, st = native.require_hybrid(), native.require(), native.status_word("cuda")
@@ -241,6 +372,7 @@ def main(argv=None) -> int:
     ap.add_argument("--kernels", action="store_true")
     ap.add_argument("--models", action="store_true")
     ap.add_argument("--width", type=int, default=2048)
+    ap.add_argument("--design", default="teganex", choices=["teganex", "lebedra"])
     a = ap.parse_args(argv)
     peaks = {}
     path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
@@ -248,10 +380,10 @@ def main(argv=None) -> int:
         with open(path) as f:
             peaks = json.load(f)
     if a.kernels or not a.models:
-        for r in run_kernels(peaks, a.width):
+        for r in run_kernels(peaks, a.width, a.design):
             print(json.dumps(r), flush=True)
     if a.models or not a.kernels:
-        for r in run_models():
+        for r in run_models(a.design):
             print(json.dumps(r), flush=True)
     return 0
 

@@ -144,12 +144,12 @@ def sink_attention(q, k, v, scale, sink):
     """Causal attention with one more term exp(sink[h]) in the denominator. q [T, H, dk]; k [T, H, dk]; v [T, H, dv]."""
     T, H, _ = q.shape
     out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    future = torch.triu(torch.ones(T, T, dtype=torch.bool), 1)
     for h in range(H):
-        for t in range(T):
-            s = (k[: t + 1, h] @ q[t, h]) * scale
-            m = torch.maximum(s.max(), sink[h])
-            e = torch.exp(s - m)
-            out[t, h] = (e @ v[: t + 1, h]) / (e.sum() + torch.exp(sink[h] - m))
+        s = ((q[:, h] @ k[:, h].T) * scale).masked_fill(future, float("-inf"))
+        m = torch.clamp(s.max(-1, keepdim=True).values, min=float(sink[h]))
+        e = torch.exp(s - m)
+        out[:, h] = (e @ v[:, h]) / (e.sum(-1, keepdim=True) + torch.exp(sink[h] - m))
     return out
 
 

@@ -27,6 +27,26 @@ def config(width, vocab, layers, eps=1e-5, embed_scale=1.5, logit_scale=0.7, max
             "embedding": {"scale": embed_scale}, "norm": {"eps": eps}, "logit_scale": logit_scale, "layers": layers}
 
 
+def latent(heads, dim, rot, vdim, rank, base=10000.0, scale=None):
+    return {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "rot": {"base": base, "dims": rot},
+            "scale": (dim + rot) ** -0.5 if scale is None else scale}
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts, top, ff, limit, groups=1, keep=1):
+    return {"kind": "moe", "expert": {"ff": ff, "limit": limit},
+            "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}}
+
+
+def lebedra(width, vocab, layers, side, mult=0.5, eps=1e-5):
+    return {"architecture": "Lebedra", "vocab": vocab, "width": width, "norm": {"eps": eps}, "residual_mult": mult,
+            "token_side": {"dim": side},
+            "layers": [{"type": "latent_attention", "mixer": m, "mlp": f} for m, f in layers]}
+
+
 CONFIGS = {
     # unaligned widths everywhere, grouped heads, three taps
     "ragged": config(100, 211, [gla_layer(3, 24, 40, 8.0, ff=52),
@@ -42,12 +62,28 @@ CONFIGS = {
     "deep": config(128, 160, [parallel_layer(attention(4, 2, 64, 128), delta(6, 3, 64, 48, 2), ff=96),
                               gla_layer(5, 16, 32, 32.0), gla_layer(2, 96, 96, 4.0, ff=72),
                               parallel_layer(attention(8, 4, 128, 128), delta(3, 1, 96, 64, 5))], eps=1e-6),
+    # Lebedra: unaligned widths, layers of different sizes, a layer without feed-forward
+    "latent_ragged": lebedra(100, 211, [(latent(3, 20, 6, 36, 44), dense(52)), (latent(5, 12, 10, 20, 28, 500.0, 0.3), moe(6, 3, 20, 0.7, 3, 2)),
+                                        (latent(2, 40, 14, 12, 60), None)], 12, 0.7),
+    # widths of the tensor-core paths, more than 16 heads, no groups
+    "latent_wide": lebedra(256, 384, [(latent(20, 128, 64, 128, 256), moe(8, 2, 64, 5.0)), (latent(2, 64, 32, 64, 512), dense(256)),
+                                      (latent(4, 72, 40, 104, 128), moe(12, 4, 72, 1.5, 4, 2))], 32, 0.4),
+    # one head, one expert, the narrowest rotation, whole residuals
+    "latent_single": lebedra(64, 96, [(latent(1, 64, 2, 64, 64, 100.0), moe(1, 1, 64, 2.0)), (latent(1, 8, 8, 8, 8), moe(4, 1, 16, 1.0, 4, 1))],
+                             8, 1.0, 1e-3),
+    # widths beyond the prompt attention's, a token side wider than a tile
+    "latent_plain": lebedra(136, 130, [(latent(2, 160, 72, 136, 40), moe(9, 5, 24, 3.0, 3, 3)), (latent(17, 16, 4, 24, 520), dense(40))], 136, 0.6),
 }
+TEGANEX = [n for n in CONFIGS if not n.startswith("latent")]
+LEBEDRA = [n for n in CONFIGS if n.startswith("latent")]
 
 
-def weights(cfg: dict, seed: int = 0, low_rank: int = 12) -> dict:
+def weights(cfg: dict, seed: int = 0, low_rank: int = 12, sure_routes: bool = False) -> dict:
     """Random bf16 weights with visible effects: decays from nearly one to nearly zero, write strengths and
-    gates spread over their range, norm weights away from one."""
+    gates spread over their range, norm weights away from one.
+
+    ``sure_routes``: routers read only the first columns of the stream and no sublayer writes those, so that the
+    choice of experts depends on the token alone and rounding in bf16 cannot change it."""
     g = torch.Generator().manual_seed(seed)
     hc = HybridConfig.from_dict(cfg)
     out = {}
@@ -60,16 +96,28 @@ def weights(cfg: dict, seed: int = 0, low_rank: int = 12) -> dict:
                 t = torch.linspace(-3.0, 2.7, shape[0]) if shape[0] > 1 else torch.zeros(1)
             elif leaf == "dt_bias":
                 t = r * 1.5 - 1.0
+            elif leaf == "sink":
+                t = r * 1.5
+            elif leaf == "correction":
+                t = r * 0.15
             elif leaf == "b":
                 t = r + 2.0
             else:
                 t = 1.0 + 0.3 * r
         elif leaf == "conv":
             t = r * 0.5
+        elif leaf in ("q", "router") and cfg["architecture"] == "Lebedra":
+            t = r * ((1.0 if leaf == "q" else 2.0) / shape[1] ** 0.5)
         elif leaf in ("embed", "pos"):
             t = r * (1.0 if leaf == "embed" else 0.4)
         else:
             t = r * (1.5 / shape[1] ** 0.5)
+        if sure_routes and cfg["architecture"] == "Lebedra":
+            n = max([x["mlp"]["router"]["experts"] for x in cfg["layers"] if (x["mlp"] or {}).get("kind") == "moe"] or [0])
+            if leaf == "router":
+                t = torch.cat([r[:, :n] * 2.0 / n ** 0.5, torch.zeros(shape[0], shape[1] - n)], 1)
+            elif leaf in ("o", "down", "proj"):
+                t[:n] = 0.0
         out[name] = t.to(torch.bfloat16)
     return out
 
@@ -80,6 +128,12 @@ def model(cfg: dict, seed: int = 0, device="cuda", w=None) -> HybridModel:
 
 def tokens(cfg: dict, n: int, seed: int = 1):
     return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+def row_errors(a, b, scale=None):
+    """Root-mean-square error of every row relative to the rms of the reference (or of ``scale``)."""
+    a, b = a.double().cpu(), b.double().cpu()
+    return (a - b).pow(2).mean(-1).sqrt() / (b if scale is None else scale).double().pow(2).mean().sqrt()
 
 
 def rel(a, b):

@@ -33,6 +33,7 @@ def engine(cfg, dtype="bfloat16", seed=0, w=None, **kw):
     from mythos_b200.infer.engine import InferenceEngine
 
     kw.setdefault("max_batch", 4)
+    kw.setdefault("max_seq_len", 640)
     return InferenceEngine.from_model(hu.model(cfg, seed, w=w), device="cuda", dtype=dtype, **kw)
 
 
@@ -55,6 +56,26 @@ def close(a, b, tol):
     assert torch.isfinite(a).all()
     err = float((a - b).abs().max()) / max(1e-9, float(b.abs().max()))
     assert err <= tol, f"{err} > {tol}"
+
+
+class Truth:
+    """The oracle's logits and streams for one sequence."""
+
+    def __init__(self, cfg, w, toks):
+        self.layers, self.lebedra = [], cfg["architecture"] == "Lebedra"
+        self.logits = oracle.forward(cfg, w, toks, trace=self.layers)
+
+    def agrees(self, got, dtype, rows=slice(None), layer=None):
+        """Every row within the tolerance; in bf16, with norms on the outputs of sublayers only, up to one row in
+        thirty may be a small output whose rounding its norm enlarges."""
+        want = self.logits if layer is None else self.layers[layer]
+        e = hu.row_errors(got, want[rows], want)
+        over = int((e >= TOL[dtype]).sum())
+        return bool(torch.isfinite(got).all()) and over <= (max(1, e.numel() // 30) if self.lebedra and dtype == "bfloat16" else 0)
+
+
+def model_weights(cfg, seed, dtype):
+    return hu.weights(cfg, seed, sure_routes=dtype == "bfloat16")
 
 
 # ------------------------------------------------------------------------------- single kernels
@@ -369,26 +390,25 @@ def test_sampler_takes_fp32_logits():
 @pytest.mark.parametrize("name", sorted(hu.CONFIGS))
 def test_whole_prompt_and_layers(name, dtype):
     cfg = hu.CONFIGS[name]
-    w, toks = hu.weights(cfg, 2), hu.tokens(cfg, 75)
-    trace = []
-    want = oracle.forward(cfg, w, toks, trace=trace)
+    w, toks = model_weights(cfg, 2, dtype), hu.tokens(cfg, 75)
+    truth = Truth(cfg, w, toks)
     eng = engine(cfg, dtype, w=w)
     seen, run = [], eng._run_layers
     eng._run_layers = lambda i, p, c: run(i, p, c, seen)
     s = eng.cache.new_sequence()
     got = eng.step([s], [toks], [list(range(75))])
-    for a, b in zip(seen, trace):
-        assert hu.rel(a, b) < TOL[dtype]
-    assert len(seen) == len(trace) and hu.rel(got, want) < TOL[dtype]
+    assert len(seen) == len(truth.layers) and all(truth.agrees(x, dtype, layer=i) for i, x in enumerate(seen))
+    assert truth.agrees(got, dtype)
 
 
 @pytest.mark.parametrize("name", sorted(hu.CONFIGS))
 @pytest.mark.parametrize("tensor_kernels", [True, False])
 def test_portions_and_single_tokens_give_the_whole_prompt(name, tensor_kernels):
     cfg = hu.CONFIGS[name]
-    w, toks = hu.weights(cfg, 4), hu.tokens(cfg, 150, 7)
-    want = oracle.forward(cfg, w, toks)
+    toks = hu.tokens(cfg, 150, 7)
     for dtype in ("float32", "bfloat16"):
+        w = model_weights(cfg, 4, dtype)
+        truth = Truth(cfg, w, toks)
         eng = engine(cfg, dtype, w=w)
         eng.tensor_kernels = tensor_kernels
         for cuts in ([2, 3, 2, 17, 15, 1, 64, 33, 13], [1] * 40 + [110], [149, 1], [16] * 9 + [6]):
@@ -397,16 +417,16 @@ def test_portions_and_single_tokens_give_the_whole_prompt(name, tensor_kernels):
                 out.append(eng.step([s], [toks[at:at + n]], [list(range(n))]))
                 at += n
             eng.release(s)
-            assert hu.rel(torch.cat(out), want) < TOL[dtype], (dtype, cuts)
+            assert truth.agrees(torch.cat(out), dtype), (dtype, cuts)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_mixed_batches_reuse_pages_and_slots(dtype):
     """Requests of unequal length come and go in a pool that holds two or three of them at a time; portions
     run beside decoded tokens and a request is left out of some steps."""
-    for name in ("deep", "ragged"):
+    for name in ("deep", "ragged", "latent_ragged", "latent_wide", "latent_plain"):
         cfg = hu.CONFIGS[name]
-        w = hu.weights(cfg, 9)
+        w = model_weights(cfg, 9, dtype)
         eng = engine(cfg, dtype, w=w, kv_pages=22)
         g = torch.Generator().manual_seed(3)
         waiting = [(hu.tokens(cfg, n, n), []) for n in (70, 5, 131, 33, 90, 2, 64, 17)]
@@ -440,26 +460,29 @@ def test_mixed_batches_reuse_pages_and_slots(dtype):
             live = [r for r in live if r[3] < len(r[0])]
         assert eng.cache.alloc.used == 0 and len(finished) == 8
         for t, o, *_ in finished:
-            assert hu.rel(torch.cat(o), oracle.forward(cfg, w, t)) < TOL[dtype], (name, len(t))
+            assert Truth(cfg, w, t).agrees(torch.cat(o), dtype), (name, len(t))
 
 
-def test_long_decoding_does_not_drift():
-    cfg = hu.CONFIGS["wide"]
-    w, toks = hu.weights(cfg, 6), hu.tokens(cfg, 420, 5)
-    want = oracle.forward(cfg, w, toks)
+@pytest.mark.parametrize("name", ["wide", "latent_wide"])
+def test_long_decoding_does_not_drift(name):
+    cfg = hu.CONFIGS[name]
+    toks = hu.tokens(cfg, 420, 5)
     for dtype in ("float32", "bfloat16"):
+        w = model_weights(cfg, 6, dtype)
+        truth = Truth(cfg, w, toks)
         eng = engine(cfg, dtype, w=w)
         s, twin = eng.cache.new_sequence(), eng.cache.new_sequence()
         out = [eng.step([s, twin], [toks[:20], toks[:35]], [[19], []])]
         for t in toks[20:]:
             out.append(eng.decode([s], [t]))
-        assert hu.rel(torch.cat(out), want[19:]) < TOL[dtype]
+        assert truth.agrees(torch.cat(out), dtype, slice(19, None))
         lg = eng.step([twin], [toks[35:]])                 # the sequence that waited meanwhile
-        assert hu.rel(lg, want[-1:]) < TOL[dtype]
+        assert truth.agrees(lg, dtype, slice(-1, None))
 
 
-def test_offloaded_sequence_continues_in_another_slot():
-    cfg = hu.CONFIGS["deep"]
+@pytest.mark.parametrize("name", ["deep", "latent_ragged"])
+def test_offloaded_sequence_continues_in_another_slot(name):
+    cfg = hu.CONFIGS[name]
     w, toks = hu.weights(cfg, 8), hu.tokens(cfg, 60)
     eng = engine(cfg, "float32", w=w)
     a = eng.cache.new_sequence()
@@ -482,11 +505,12 @@ def _greedy(cfg, w, prompt, n):
     return seq[len(prompt):], gaps
 
 
-def test_greedy_generation_and_scheduler():
+@pytest.mark.parametrize("name,wide", [("ragged", "wide"), ("latent_ragged", "latent_wide")])
+def test_greedy_generation_and_scheduler(name, wide):
     from mythos_b200.infer.sampler import SamplerConfig
     from mythos_b200.infer.serving import ContinuousBatcher
 
-    cfg = hu.CONFIGS["ragged"]
+    cfg = hu.CONFIGS[name]
     w = hu.weights(cfg, 1)
     prompts = [hu.tokens(cfg, n, 20 + n) for n in (9, 1, 30)]
     want = []
@@ -507,25 +531,27 @@ def test_greedy_generation_and_scheduler():
         assert [r.output for r in reqs] == want
         assert eng.cache.alloc.used == 0
     # bf16: the captured decode graph follows the same path as single steps
-    e16 = engine(hu.CONFIGS["wide"], seed=3)
-    ps = [hu.tokens(hu.CONFIGS["wide"], n, n) for n in (40, 40)]
+    e16 = engine(hu.CONFIGS[wide], seed=3, max_seq_len=640)
+    ps = [hu.tokens(hu.CONFIGS[wide], n, n) for n in (40, 40)]
     assert e16.generate(ps, max_new_tokens=20).tokens == e16.generate(ps, max_new_tokens=20, use_graph=False).tokens
 
 
-def test_model_helpers_and_command_line(tmp_path):
+@pytest.mark.parametrize("name", ["ragged", "latent_ragged"])
+def test_model_helpers_and_command_line(tmp_path, name):
     from mythos_b200.infer.engine import InferenceEngine
     from mythos_b200.infer.serving import compute_logprobs
     from mythos_b200.oil.importers import write_safetensors
     from mythos_b200.oil.model_io import load_model
     from mythos_b200.tools.infer import main as infer_main
 
-    cfg = json.loads(json.dumps(hu.CONFIGS["ragged"]))
-    w, toks = hu.weights(cfg, 11), hu.tokens(cfg, 25)
+    cfg = json.loads(json.dumps(hu.CONFIGS[name]))
+    w, toks = model_weights(cfg, 11, "bfloat16"), hu.tokens(cfg, 25)
     (tmp_path / "config.json").write_text(json.dumps(cfg))
     write_safetensors(str(tmp_path / "model.safetensors"), w)
     m, _ = load_model(str(tmp_path), device="cuda")
-    want = oracle.forward(cfg, w, toks)
-    assert hu.rel(m(torch.tensor([toks]))[0], want) < TOL["bfloat16"]
+    truth = Truth(cfg, w, toks)
+    want = truth.logits
+    assert truth.agrees(m(torch.tensor([toks]))[0], "bfloat16")
     lp = torch.log_softmax(want, -1)[:-1].gather(1, torch.tensor(toks[1:])[:, None])[:, 0]
     assert float((compute_logprobs(m, toks) - lp).abs().max()) < 0.5
     eng = InferenceEngine.load(str(tmp_path), device="cuda", max_batch=1)

@@ -11,7 +11,7 @@ import hybrid_util as hu
 from mythos_b200.infer.kv_paged import PagedKVCache, RecurrentStatePool
 from mythos_b200.models import registry
 from mythos_b200.models.hybrid import HybridModel
-from mythos_b200.models.hybrid_config import HybridConfig, teganex_config
+from mythos_b200.models.hybrid_config import HybridConfig, lebedra_config, teganex_config
 from mythos_b200.oil.importers import read_safetensors_torch, write_safetensors
 from mythos_b200.oil.model_io import load_model
 
@@ -29,6 +29,7 @@ def test_config_round_trip(name):
     lambda c: c["layers"][1]["mixer"]["left"].update(kv_heads=4),
     lambda c: c["layers"][0]["mlp"].update(kind="sparse"),
     lambda c: c.update(architecture="Unheard"),
+    lambda c: c["layers"][0].update(type="latent_attention"),
 ])
 def test_bad_configurations_are_refused(tmp_path, change):
     raw = json.loads(json.dumps(hu.CONFIGS["ragged"]))
@@ -36,6 +37,22 @@ def test_bad_configurations_are_refused(tmp_path, change):
     (tmp_path / "config.json").write_text(json.dumps(raw))
     with pytest.raises((ValueError, KeyError)):
         registry.load_config(str(tmp_path))
+
+
+@pytest.mark.parametrize("change", [
+    lambda c: c["layers"][0]["mixer"].update(rot_dim=7, rot={"base": 10.0, "dims": 7}),
+    lambda c: c["layers"][0]["mixer"]["rot"].update(dims=4),
+    lambda c: c["layers"][1]["mlp"]["router"]["groups"].update(count=4),
+    lambda c: c["layers"][1]["mlp"]["router"]["groups"].update(keep=4),
+    lambda c: c["layers"][1]["mlp"]["router"].update(top=5),
+    lambda c: c["layers"][1]["mlp"].update(kind="other"),
+    lambda c: c["layers"][0].update(type="gla"),
+])
+def test_bad_latent_configurations_are_refused(change):
+    raw = json.loads(json.dumps(hu.CONFIGS["latent_ragged"]))
+    change(raw)
+    with pytest.raises((ValueError, KeyError)):
+        HybridConfig.from_dict(raw)
 
 
 def _write(folder, cfg, w):
@@ -65,6 +82,19 @@ def test_checkpoint_folder_loads_through_the_registry(tmp_path):
     assert info_main([str(tmp_path)]) == 0
 
 
+def test_lebedra_folder_loads_through_the_registry(tmp_path):
+    cfg = hu.CONFIGS["latent_ragged"]
+    w = hu.weights(cfg, 3)
+    _write(str(tmp_path), cfg, w)
+    m, _ = load_model(str(tmp_path))
+    assert isinstance(m, HybridModel) and m.cfg.architecture == "Lebedra" and not m.cfg.pre_norm
+    assert torch.equal(m.tensor("l1.mlp.e5.down"), w["l1.mlp.e5.down"]) and torch.equal(m.tensor("l0.mix.sink"), w["l0.mix.sink"])
+    assert m.cfg.context_limit > m.cfg.max_seq_len and "l2.norm2" not in dict(m.named_tensors())
+    del w["l1.mlp.correction"]
+    with pytest.raises(KeyError):
+        HybridModel(HybridConfig.from_dict(cfg), w)
+
+
 def test_missing_and_misshapen_tensors_are_refused():
     cfg = hu.CONFIGS["single"]
     hc = HybridConfig.from_dict(cfg)
@@ -82,6 +112,8 @@ def test_named_configuration_has_consistent_shapes():
     m = HybridModel.random(cfg, low_rank=8)
     assert m.param_count() == sum(t.numel() for _, t in m.named_tensors())
     assert [s.type for s in cfg.layers] == ["gla", "gla", "gla", "parallel"]
+    m = HybridModel.random(lebedra_config(width=256, layers=2, vocab=64, experts=8, top=2))
+    assert m.param_count() == sum(t.numel() for _, t in m.named_tensors()) and m.tensor("l1.mlp.e7.gate").shape[1] == 256
 
 
 def test_cache_with_unequal_widths_and_state_slots():
@@ -108,6 +140,37 @@ def test_cache_with_unequal_widths_and_state_slots():
     assert a2 != other and c.lens[a2] == 9 and float(s0[a2].min()) == 3.0
     assert float(c.k[1][int(c.block_table_host[a2, 2]), 0].min()) == 7.0
     assert c.size_bytes() == sum(t.numel() * 2 for t in c.k + c.v) + s0.numel() * 4
+
+
+def test_pages_of_rows_without_separate_values():
+    c = PagedKVCache(2, 0, 0, num_pages=5, page_size=4, max_seqs=2, max_pages_per_seq=4, device="cpu",
+                     layer_shapes=[(1, 24, 0), (1, 16, 0)])
+    assert c.k[0].shape == (5, 4, 1, 24) and c.v[0].numel() == 0 and c.size_bytes() == 5 * 4 * 40 * 2
+    a = c.new_sequence()
+    c.reserve(a, 6)
+    c.advance(a, 6)
+    c.k[1][int(c.block_table_host[a, 1]), 1] = 3.0
+    b = c.restore_sequence(c.offload_sequence(a))
+    assert c.lens[b] == 6 and float(c.k[1][int(c.block_table_host[b, 1]), 1].min()) == 3.0
+    c.publish_prefix(b, list(range(6)))
+    other = c.new_sequence()
+    assert c.share_prefix(other, list(range(9))) == 4      # pages alone determine such a prefix
+
+
+def test_batch_plan_separates_long_and_short_portions():
+    from mythos_b200.infer.hybrid import EXPAND_TOKENS, HybridEngine
+
+    class Cfg:
+        cfg = HybridConfig.from_dict(hu.CONFIGS["latent_ragged"])
+
+    n = EXPAND_TOKENS
+    assert HybridEngine._batch_plan(Cfg, [1, n - 1], [5, 0]) == ([], None)
+    lists, build = HybridEngine._batch_plan(Cfg, [2, n, 1, n + 3], [7, 0, 0, 100])
+    assert lists == [[0, 0, n, n, 2 * n + 103], [0, 1, n + 2], [0, 0, 2], [7, 8, 0]]
+    sp = build(*[torch.tensor(x, dtype=torch.int32) for x in lists])
+    assert sp.keys == 2 * n + 103 and sp.max_k == n + 103 and sp.short.dtype == torch.int64
+    lists, build = HybridEngine._batch_plan(Cfg, [n], [3])
+    assert lists == [[0, n + 3], [], [], []] and build(*[torch.tensor(x) for x in lists]).short is None
 
 
 class _FakeEngine:
@@ -207,3 +270,67 @@ def test_a_mistake_in_a_mechanism_is_larger_than_the_tolerance(slip, monkeypatch
     fn, wrong = _slip(slip)
     monkeypatch.setattr(oracle, fn, wrong)
     assert hu.rel(oracle.forward(cfg, w, toks), right) > 0.15   # bf16 comparisons allow 0.06
+
+
+def _latent_slips():
+    """Mistakes in Lebedra's mechanisms: name -> (function of the oracle, wrong version)."""
+    att, rot, choose, expert, side, norm = (oracle.sink_attention, oracle.rotate_pairs, oracle.choose_experts, oracle.clamped_expert,
+                                            oracle.token_side, oracle.rms_norm)
+
+    def half_split(x, pos, base):
+        n = x.shape[-1]
+        order = torch.tensor([i // 2 + (i % 2) * (n // 2) for i in range(n)])
+        out = torch.empty_like(x)
+        out[..., order] = rot(x[..., order], pos, base)
+        return out
+
+    def renormalised(z, c, r, *_):
+        p = choose(z, c, r)
+        total = sum(w for _, w in p)
+        return [(e, w / total) for e, w in p]
+
+    def zero_mask(z, c, r, *_):                                 # other groups count as zero instead of never
+        E, n, keep = r["experts"], r["groups"]["count"], r["groups"]["keep"]
+        s = torch.softmax(z, -1)
+        choice, size = s + c, E // n
+        best = torch.topk(choice.view(n, size).amax(1), keep).indices
+        ok = torch.zeros(n, dtype=torch.bool)
+        ok[best] = True
+        masked = torch.where(ok.repeat_interleave(size), choice, torch.zeros_like(choice))
+        return [(int(e), s[e]) for e in torch.topk(masked, r["top"]).indices]
+
+    def groups_by_sum(z, c, r, *_):
+        E, n, keep = r["experts"], r["groups"]["count"], r["groups"]["keep"]
+        s = torch.softmax(z, -1)
+        choice, size = s + c, E // n
+        best = torch.topk(choice.view(n, size).sum(1), keep).indices.tolist()
+        allowed = [e for e in range(E) if e // size in best]
+        return [(e, s[e]) for e in sorted(allowed, key=lambda e: -float(choice[e]))[: r["top"]]]
+
+    return {"no_sink": ("sink_attention", lambda q, k, v, sc, sink: att(q, k, v, sc, torch.full_like(sink, -1e9))),
+            "scaled_sink": ("sink_attention", lambda q, k, v, sc, sink: att(q, k, v, sc, sink * sc)),
+            "no_rotation": ("rotate_pairs", lambda x, pos, base: x),
+            "half_split": ("rotate_pairs", half_split),
+            "late_positions": ("rotate_pairs", lambda x, pos, base: rot(x, pos if x.dim() == 3 else pos + 1, base)),
+            "renormalised": ("choose_experts", renormalised),
+            "weights_with_correction": ("choose_experts", lambda z, c, r, *_: [(e, w + c[e]) for e, w in choose(z, c, r)]),
+            "no_correction": ("choose_experts", lambda z, c, r, *_: choose(z, torch.zeros_like(c), r)),
+            "no_groups": ("choose_experts", lambda z, c, r, *_: choose(z, c, {**r, "groups": {"count": 1, "keep": 1}})),
+            "groups_by_sum": ("choose_experts", groups_by_sum), "zero_mask": ("choose_experts", zero_mask),
+            "no_limit": ("clamped_expert", lambda h, W, p, limit: expert(h, W, p, 1e9)),
+            "no_token_input": ("token_side", lambda x, W, p, e, eps: side(x, W, p, e, eps) * 0)}
+
+
+@pytest.mark.parametrize("slip", sorted(_latent_slips()))
+def test_a_mistake_in_a_latent_or_expert_mechanism_shows(slip, monkeypatch):
+    """Far above what 32-bit comparisons allow (5e-5), and on most rows above the bf16 tolerance as well."""
+    cfg = json.loads(json.dumps(hu.CONFIGS["latent_ragged"]))
+    cfg["layers"][1]["mlp"] = hu.moe(12, 3, 20, 0.7, 3, 1)
+    cfg["norm"]["eps"] = 0.05                               # the scale of a sublayer's output shows
+    w, toks = hu.weights(cfg, 5), hu.tokens(cfg, 40)
+    w["l1.mlp.correction"] = (w["l1.mlp.correction"].float() - 0.5).to(torch.bfloat16)      # negative choice scores
+    right = oracle.forward(cfg, w, toks)
+    fn, wrong = _latent_slips()[slip]
+    monkeypatch.setattr(oracle, fn, wrong)
+    e = hu.row_errors(oracle.forward(cfg, w, toks), right)
+    assert float(e.max()) > 0.06 and float((e > 1e-3).double().mean()) > 0.3, (float(e.max()), float(e.median()))
