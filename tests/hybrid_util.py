@@ -69,7 +69,7 @@ CONFIGS = {
     "latent_wide": lebedra(256, 384, [(latent(20, 128, 64, 128, 256), moe(8, 2, 64, 5.0)), (latent(2, 64, 32, 64, 512), dense(256)),
                                       (latent(4, 72, 40, 104, 128), moe(12, 4, 72, 1.5, 4, 2))], 32, 0.4),
     # one head, one expert, the narrowest rotation, whole residuals
-    "latent_single": lebedra(64, 96, [(latent(1, 64, 2, 64, 64, 100.0), moe(1, 1, 64, 2.0)), (latent(1, 8, 8, 8, 8), moe(4, 1, 16, 1.0, 4, 1))],
+    "latent_single": lebedra(64, 96, [(latent(1, 64, 2, 64, 64, 100.0), moe(1, 1, 64, 2.0)), (latent(1, 24, 8, 40, 40), moe(4, 1, 32, 1.0, 4, 1))],
                              8, 1.0, 1e-3),
     # widths beyond the prompt attention's, a token side wider than a tile
     "latent_plain": lebedra(136, 130, [(latent(2, 160, 72, 136, 40), moe(9, 5, 24, 3.0, 3, 3)), (latent(17, 16, 4, 24, 520), dense(40))], 136, 0.6),
