@@ -826,7 +826,7 @@ void flash_attn_paged_prefill(const Tensor& q, const Tensor& k_cache, const Tens
   mb::flash_attn_paged_prefill(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), (int)k_cache.size(0),
                                block_table.data_ptr<int>(), (int)block_table.size(1), cu_q.data_ptr<int>(),
                                kv_lens.data_ptr<int>(), out.data_ptr(), out.stride(0), (int)B, (int)q.size(0),
-                               (int)max_q_len, (int)q.size(1), (int)k_cache.size(2), (int)q.size(2), (int)q.size(2), nullptr, 0, (float)scale,
+                               (int)max_q_len, (int)q.size(1), (int)k_cache.size(2), (int)q.size(2), (int)q.size(2), mb::AttnExtras{}, (float)scale,
                                status_ptr(status), cur_stream());
 }
 

@@ -74,8 +74,9 @@ void sandwich_norm(const Tensor& y1, const OptTensor& y2, const OptTensor& w1, c
                     h.data_ptr(), h.stride(0), (int)rows, (int)dim, (float)eps, cur_stream());
 }
 
-// The same with the weighted sum of a token's experts as the sublayer's output: y [pairs, dim], row and weight [rows, top].
-void expert_norm(const Tensor& y, const Tensor& row, const Tensor& weight, const Tensor& w_post, Tensor& x,
+// The same with the weighted sum of a token's experts as the sublayer's output: y [pairs, dim], row and weight [rows, top];
+// shared [rows, dim] (may be null) is added.
+void expert_norm(const Tensor& y, const OptTensor& shared, const Tensor& row, const Tensor& weight, const Tensor& w_post, Tensor& x,
                  const OptTensor& w_next, Tensor& h, double eps, double mult) {
   const bool f32 = is_f32(h, "h");
   chk_c(x, F32, "x");
@@ -85,8 +86,12 @@ void expert_norm(const Tensor& y, const Tensor& row, const Tensor& weight, const
   TORCH_CHECK(row.dim() == 2 && row.size(0) == rows && weight.sizes() == row.sizes(), "expert_norm: row / weight");
   chk_rows(y, f32, rows * top, dim, "y");
   chk_rows(h, f32, rows, dim, "h");
+  if (shared.has_value()) {
+    chk_rows(*shared, f32, rows, dim, "shared");
+    TORCH_CHECK(shared->stride(0) == y.stride(0), "expert_norm: y and shared need the same row stride");
+  }
   c10::cuda::CUDAGuard guard(h.device());
-  const mb::SublayerOut s{y.data_ptr(), nullptr, y.stride(0), nullptr, nullptr, row.data_ptr<int>(), weight.data_ptr<float>(),
+  const mb::SublayerOut s{y.data_ptr(), cptr(shared), y.stride(0), nullptr, nullptr, row.data_ptr<int>(), weight.data_ptr<float>(),
                           (int)top};
   mb::sandwich_norm(f32, s, fptr(w_post, dim, "w_post"), (float)mult, x.data_ptr<float>(), fptr(w_next, dim, "w_next"),
                     h.data_ptr(), h.stride(0), (int)rows, (int)dim, (float)eps, cur_stream());
@@ -108,91 +113,104 @@ Pages pages(const Tensor& table, const Tensor& k_cache, const Tensor& v_cache, b
                (int)k_cache.size(3), (int)v_cache.size(3)};
 }
 
-void qk_norm_append(const Tensor& proj, int64_t q_off, int64_t k_off, int64_t v_off, const Tensor& q_gamma,
-                    const Tensor& k_gamma, const std::vector<Tensor>& batch, const Tensor& table, Tensor& q_out,
-                    Tensor& k_cache, Tensor& v_cache, double eps) {
-  const bool f32 = is_f32(q_out, "q_out");
-  const auto rb = ragged(batch);
-  const Pages pg = pages(table, k_cache, v_cache, f32, rb.n_seq);
-  chk_c(q_out, f32 ? F32 : BF16, "q_out");
-  TORCH_CHECK(q_out.dim() == 3 && q_out.size(0) == rb.rows && q_out.size(2) == pg.dk, "q_out: [rows, heads, dk]");
-  const int heads = (int)q_out.size(1);
-  chk_rows(proj, f32, rb.rows, std::max({q_off + heads * pg.dk, k_off + pg.kv_heads * pg.dk, v_off + pg.kv_heads * pg.dv}),
-           "proj");
-  c10::cuda::CUDAGuard guard(q_out.device());
-  mb::qk_norm_append(f32, proj.data_ptr(), proj.stride(0), (int)q_off, (int)k_off, (int)v_off,
-                     fptr(q_gamma, pg.dk, "q_gamma"), fptr(k_gamma, pg.dk, "k_gamma"), rb, pg.table, pg.stride,
-                     pg.page_size, q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), heads, pg.kv_heads, pg.dk,
-                     pg.dv, (float)eps, cur_stream());
-}
+// Softmax attention over the pages of one layer: sizes, offsets in the projection and parameters, built once per layer.
+// Head widths are the stored ones (dk, dv); norm_dim, the true key width, counts where heads are normalised.
+struct Attention {
+  mb::HeadPrep p{};
+  float scale = 1.f, out_scale = 1.f;
+  int window = 0;
+  bool gate_channels = false;
+  OptTensor q_bias, k_bias, v_bias, q_gamma, k_gamma, turns, sink;
 
-void paged_attn_any(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const std::vector<Tensor>& batch,
-                    const Tensor& table, const OptTensor& gate, Tensor& o, double scale) {
-  const bool f32 = is_f32(q, "q");
-  const auto rb = ragged(batch);
-  const Pages pg = pages(table, k_cache, v_cache, f32, rb.n_seq);
-  chk_c(q, f32 ? F32 : BF16, "q");
-  TORCH_CHECK(q.dim() == 3 && q.size(0) == rb.rows && q.size(2) == pg.dk, "q: [rows, heads, dk]");
-  const int heads = (int)q.size(1);
-  chk_rows(o, f32, rb.rows, (int64_t)heads * pg.dv, "o");
-  if (gate.has_value()) chk_rows(*gate, f32, rb.rows, heads, "gate");
-  c10::cuda::CUDAGuard guard(q.device());
-  mb::paged_attn_any(f32, q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), rb, pg.table, pg.stride, pg.page_size,
-                     cptr(gate), gate.has_value() ? gate->stride(0) : 0, o.data_ptr(), o.stride(0), heads, pg.kv_heads,
-                     pg.dk, pg.dv, (float)scale, cur_stream());
-}
-
-// Tensor-core attention over the pages (key and value widths 64 or 128, 16-token pages): prompts and portions.
-void paged_attn_prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const std::vector<Tensor>& batch,
-                        const Tensor& table, const OptTensor& gate, Tensor& o, int64_t max_q, double scale,
-                        const OptTensor& status) {
-  const auto rb = ragged(batch);
-  const Pages pg = pages(table, k_cache, v_cache, false, rb.n_seq);
-  chk_c(q, BF16, "q");
-  TORCH_CHECK(q.dim() == 3 && q.size(0) == rb.rows && q.size(2) == pg.dk && pg.page_size == 16, "paged_attn_prefill: q / pages");
-  const int heads = (int)q.size(1);
-  chk_rows(o, false, rb.rows, (int64_t)heads * pg.dv, "o");
-  if (gate.has_value()) chk_rows(*gate, false, rb.rows, heads, "gate");
-  c10::cuda::CUDAGuard guard(q.device());
-  mb::flash_attn_paged_prefill(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), (int)k_cache.size(0),
-                               pg.table, pg.stride, rb.cu_q, rb.kv_lens, o.data_ptr(), o.stride(0), rb.n_seq, rb.rows,
-                               (int)max_q, heads, pg.kv_heads, pg.dk, pg.dv, cptr(gate),
-                               gate.has_value() ? gate->stride(0) : 0, (float)scale, status_ptr(status), cur_stream());
-}
-
-// One token per sequence, split over the context.
-void paged_attn_decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const std::vector<Tensor>& batch,
-                       const Tensor& table, const OptTensor& gate, Tensor& o, Tensor& scratch, Tensor& counters,
-                       int64_t splits, double scale, const OptTensor& status) {
-  const auto rb = ragged(batch);
-  const Pages pg = pages(table, k_cache, v_cache, false, rb.n_seq);
-  chk_c(q, BF16, "q");
-  TORCH_CHECK(q.dim() == 3 && q.size(0) == rb.rows && q.size(2) == pg.dk && rb.rows == rb.n_seq && pg.page_size == 16,
-              "paged_attn_decode: q / pages");
-  const int heads = (int)q.size(1);
-  chk_c(o, BF16, "o");
-  TORCH_CHECK(o.numel() == (int64_t)rb.rows * heads * pg.dv, "paged_attn_decode: o");
-  chk_c(scratch, F32, "scratch");
-  chk_c(counters, I32, "counters");
-  TORCH_CHECK(scratch.numel() >= (int64_t)rb.rows * heads * splits * (pg.dv + 2) &&
-                  counters.numel() >= (int64_t)rb.rows * pg.kv_heads * ((heads / pg.kv_heads + 7) / 8),
-              "paged_attn_decode: scratch");
-  if (gate.has_value()) chk_rows(*gate, false, rb.rows, heads, "gate");
-  c10::cuda::CUDAGuard guard(q.device());
-  mb::paged_attn_decode(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), pg.table, rb.kv_lens, o.data_ptr(),
-                        scratch.data_ptr<float>(), counters.data_ptr<int>(), rb.n_seq, heads, pg.kv_heads, pg.dk, 16,
-                        pg.stride, (int)k_cache.size(0), (int)splits, (float)scale, status_ptr(status), cur_stream(),
-                        q.stride(0), pg.dv, cptr(gate), gate.has_value() ? gate->stride(0) : 0);
-}
+  mb::AttnExtras extras(const OptTensor& gate, bool f32, int64_t rows) const {
+    mb::AttnExtras ex;
+    if (gate.has_value()) {
+      chk_rows(*gate, f32, rows, gate_channels ? (int64_t)p.heads * p.dv : p.heads, "gate");
+      ex.gate = gate->data_ptr();
+      ex.ld_gate = gate->stride(0);
+      ex.gate_channels = gate_channels;
+    }
+    ex.sink = fptr(sink, p.heads, "sink");
+    ex.window = window;
+    ex.out_scale = out_scale;
+    return ex;
+  }
+  Pages layer_pages(const Tensor& table, const Tensor& k_cache, const Tensor& v_cache, bool f32, int n_seq) const {
+    const Pages pg = pages(table, k_cache, v_cache, f32, n_seq);
+    TORCH_CHECK(pg.kv_heads == p.kv_heads && pg.dk == p.dk && pg.dv == p.dv, "attention: the pages have other heads");
+    return pg;
+  }
+  void check_q(const Tensor& q, bool f32, int64_t rows) const {
+    chk_c(q, f32 ? F32 : BF16, "q");
+    TORCH_CHECK(q.dim() == 3 && q.size(0) == rows && q.size(1) == p.heads && q.size(2) == p.dk, "q: [rows, heads, dk]");
+  }
+  void prep(const Tensor& proj, const std::vector<Tensor>& batch, const Tensor& table, Tensor& q, Tensor& k_cache, Tensor& v_cache) const {
+    const bool f32 = is_f32(q, "q");
+    const auto rb = ragged(batch);
+    const Pages pg = layer_pages(table, k_cache, v_cache, f32, rb.n_seq);
+    check_q(q, f32, rb.rows);
+    int cols = p.q_off + p.heads * p.dk;
+    if (p.k_off >= 0) cols = std::max({cols, p.k_off + p.kv_heads * p.dk, p.v_off + p.kv_heads * p.dv});
+    chk_rows(proj, f32, rb.rows, cols, "proj");
+    c10::cuda::CUDAGuard guard(q.device());
+    mb::attn_prep(f32, proj.data_ptr(), proj.stride(0), p, rb, pg.table, pg.stride, pg.page_size, q.data_ptr(), k_cache.data_ptr(),
+                  v_cache.data_ptr(), cur_stream());
+  }
+  // Any widths, scalar arithmetic in 32-bit.
+  void any(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const std::vector<Tensor>& batch, const Tensor& table,
+           const OptTensor& gate, Tensor& o) const {
+    const bool f32 = is_f32(q, "q");
+    const auto rb = ragged(batch);
+    const Pages pg = layer_pages(table, k_cache, v_cache, f32, rb.n_seq);
+    check_q(q, f32, rb.rows);
+    chk_rows(o, f32, rb.rows, (int64_t)p.heads * p.dv, "o");
+    c10::cuda::CUDAGuard guard(q.device());
+    mb::paged_attn_any(f32, q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), rb, pg.table, pg.stride, pg.page_size,
+                       extras(gate, f32, rb.rows), o.data_ptr(), o.stride(0), p.heads, p.kv_heads, p.dk, p.dv, scale, cur_stream());
+  }
+  bool tensor_ok(int64_t page_size) const { return page_size == 16 && p.dk % 8 == 0 && p.dv % 8 == 0 && p.dk <= 128 && p.dv <= 128; }
+  // Tensor cores: prompts and portions.
+  void prefill(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const std::vector<Tensor>& batch, const Tensor& table,
+               const OptTensor& gate, Tensor& o, int64_t max_q, const OptTensor& status) const {
+    const auto rb = ragged(batch);
+    const Pages pg = layer_pages(table, k_cache, v_cache, false, rb.n_seq);
+    check_q(q, false, rb.rows);
+    TORCH_CHECK(tensor_ok(pg.page_size), "attention prefill: widths / page size");
+    chk_rows(o, false, rb.rows, (int64_t)p.heads * p.dv, "o");
+    c10::cuda::CUDAGuard guard(q.device());
+    mb::flash_attn_paged_prefill(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), (int)k_cache.size(0), pg.table,
+                                 pg.stride, rb.cu_q, rb.kv_lens, o.data_ptr(), o.stride(0), rb.n_seq, rb.rows, (int)max_q, p.heads,
+                                 p.kv_heads, p.dk, p.dv, extras(gate, false, rb.rows), scale, status_ptr(status), cur_stream());
+  }
+  // One token per sequence, split over the context.
+  void decode(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache, const std::vector<Tensor>& batch, const Tensor& table,
+              const OptTensor& gate, Tensor& o, Tensor& scratch, Tensor& counters, int64_t splits, const OptTensor& status) const {
+    const auto rb = ragged(batch);
+    const Pages pg = layer_pages(table, k_cache, v_cache, false, rb.n_seq);
+    check_q(q, false, rb.rows);
+    TORCH_CHECK(tensor_ok(pg.page_size) && rb.rows == rb.n_seq, "attention decode: widths / page size / one token per sequence");
+    chk_rows(o, false, rb.rows, (int64_t)p.heads * p.dv, "o");
+    chk_c(scratch, F32, "scratch");
+    chk_c(counters, I32, "counters");
+    TORCH_CHECK(scratch.numel() >= decode_scratch(rb.rows, splits) &&
+                    counters.numel() >= (int64_t)rb.rows * p.kv_heads * ((p.heads / p.kv_heads + 7) / 8), "attention decode: scratch");
+    c10::cuda::CUDAGuard guard(q.device());
+    mb::paged_attn_decode(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), pg.table, rb.kv_lens, o.data_ptr(),
+                          scratch.data_ptr<float>(), counters.data_ptr<int>(), rb.n_seq, p.heads, p.kv_heads, p.dk, 16, pg.stride,
+                          (int)k_cache.size(0), (int)splits, scale, status_ptr(status), cur_stream(), q.stride(0), p.dv,
+                          extras(gate, false, rb.rows), o.stride(0));
+  }
+  int64_t decode_scratch(int64_t rows, int64_t splits) const { return rows * p.heads * splits * ((p.dv + 63) / 64 * 64 + 2); }
+};
 
 // Gated activation (kind, limit, alpha); see GateAct.
 using Act = std::tuple<int64_t, double, double>;
 mb::GateAct gate(const Act& a) { return mb::GateAct{(int)std::get<0>(a), (float)std::get<1>(a), (float)std::get<2>(a)}; }
 
 // Few-token GEMM: out = alpha * x w^T, or with f > 0 act(x w[:f]^T, x w[f_off : f_off + f]^T), or with mul
-// gelu_tanh(x w^T) * mul[ids, :].
+// gelu_tanh(x w^T) * mul[ids, :], or with cap > 0 the soft-capped product.
 void gemm_decode(const Tensor& x, const Tensor& w, Tensor& out, int64_t f, int64_t f_off, double alpha,
-                 const OptTensor& status, const Act& act, const OptTensor& mul, const OptTensor& ids) {
+                 const OptTensor& status, const Act& act, const OptTensor& mul, const OptTensor& ids, double cap) {
   chk(x, BF16, "x");
   chk(w, BF16, "w");
   const bool of32 = is_f32(out, "out");
@@ -200,7 +218,7 @@ void gemm_decode(const Tensor& x, const Tensor& w, Tensor& out, int64_t f, int64
                   x.size(1) == w.size(1), "gemm_decode: operands");
   const int64_t n = f > 0 ? f : w.size(0);
   TORCH_CHECK(out.size(0) == x.size(0) && out.size(1) >= n && (f == 0 || f_off + f <= w.size(0)), "gemm_decode: shapes");
-  mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0};
+  mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0, (float)cap};
   if (mul.has_value()) {
     TORCH_CHECK(ids.has_value() && mul->dim() == 2 && mul->stride(1) == 1 && mul->size(1) >= n, "gemm_decode: mul");
     chk(*mul, BF16, "mul");
@@ -256,7 +274,7 @@ void gemm_tiles(const Tensor& x, const Tensor& w, Tensor& out, const Tensor& til
   const int64_t n = f > 0 ? f : w.size(1);
   TORCH_CHECK(out.size(1) >= n && (f == 0 || f_off + f <= w.size(1)), "gemm_tiles: shapes");
   const mb::TileList list = tile_list(tiles, count);
-  const mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0};
+  const mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0, 0.f};
   c10::cuda::CUDAGuard guard(x.device());
   if (f32) {
     TORCH_CHECK(f == 0 && tile_rows == 64, "gemm_tiles: fp32 takes 64-row tiles and no tail");
@@ -272,8 +290,9 @@ void gemm_tiles(const Tensor& x, const Tensor& w, Tensor& out, const Tensor& til
   }
 }
 
-// ---- routed experts: spec = (experts, top, groups, keep)
+// ---- routed experts: spec = (experts, top, groups, keep), rule = (sigmoid, group_best, normalise, scale)
 using Router = std::tuple<int64_t, int64_t, int64_t, int64_t>;
+using RouterRule = std::tuple<int64_t, int64_t, int64_t, double>;
 struct Routing {
   mb::RouterSpec s;
   mb::RouterBuffers b;
@@ -284,16 +303,20 @@ Routing routing(const Router& r, const Tensor& idx, const Tensor& weight, const 
   for (const Tensor* t : {&idx, &slot, &counts, &offset}) chk_c(*t, I32, "routing buffer");
   chk_c(weight, F32, "weight");
   const mb::TileList l = tile_list(tiles, count);
-  Routing out{{(int)std::get<0>(r), (int)std::get<1>(r), (int)std::get<2>(r), (int)std::get<3>(r)}, {}};
+  Routing out{{(int)std::get<0>(r), (int)std::get<1>(r), (int)std::get<2>(r), (int)std::get<3>(r), 0, 1, 0, 1.f}, {}};
   TORCH_CHECK(idx.dim() == 2 && idx.size(1) == out.s.top && slot.sizes() == idx.sizes() && weight.sizes() == idx.sizes() &&
                   counts.numel() > out.s.experts && offset.numel() >= out.s.experts, "routing buffers");
   out.b = {idx.data_ptr<int>(), weight.data_ptr<float>(), slot.data_ptr<int>(), counts.data_ptr<int>(), offset.data_ptr<int>(),
            const_cast<int*>(l.tiles), const_cast<int*>(l.count), l.max_tiles};
   return out;
 }
-void expert_select(const Tensor& logits, const Tensor& correction, const Router& r, int64_t tile_rows, Tensor& idx, Tensor& weight,
-                   Tensor& slot, Tensor& counts, Tensor& offset, Tensor& tiles, Tensor& count) {
-  const Routing rt = routing(r, idx, weight, slot, counts, offset, tiles, count);
+void expert_select(const Tensor& logits, const OptTensor& correction, const Router& r, int64_t tile_rows, Tensor& idx, Tensor& weight,
+                   Tensor& slot, Tensor& counts, Tensor& offset, Tensor& tiles, Tensor& count, const RouterRule& rule) {
+  Routing rt = routing(r, idx, weight, slot, counts, offset, tiles, count);
+  rt.s.sigmoid = (int)std::get<0>(rule);
+  rt.s.group_best = (int)std::get<1>(rule);
+  rt.s.normalise = (int)std::get<2>(rule);
+  rt.s.scale = (float)std::get<3>(rule);
   const int64_t rows = idx.size(0);
   chk_rows(logits, true, rows, rt.s.experts, "logits");
   TORCH_CHECK(tile_rows > 0 && tiles.size(0) >= std::min<int64_t>(rows * rt.s.top, rt.s.experts + rows * rt.s.top / tile_rows),
@@ -598,6 +621,95 @@ struct Recurrent {
   }
 };
 
+// The selective scan of one layer with its parameters and state, built once per layer.
+struct Selective {
+  mb::SelectiveSpec s{};
+  int x_off = 0, z_off = 0, b_off = 0, c_off = 0;
+  Tensor conv_w, conv_b, a, d, dt_b, state, w_dt;
+  OptTensor conv_state;
+
+  void validate() const {
+    const int64_t sp = mb::selective_padded_state(s.state);
+    TORCH_CHECK(s.inner > 0 && s.state > 0 && s.rank > 0 && s.taps > 0, "selective: sizes");
+    chk_c(state, F32, "state");
+    TORCH_CHECK(state.dim() == 3 && state.size(1) == s.inner && state.size(2) == sp, "state: [slots, inner, padded state]");
+    fptr(conv_w, (int64_t)s.taps * s.inner, "conv_w");
+    for (const Tensor* t : {&conv_b, &d, &dt_b}) fptr(*t, s.inner, "selective: channel parameters");
+    fptr(a, s.inner * sp, "a");
+    TORCH_CHECK(s.taps == 1 || conv_state.has_value(), "selective: conv_state");
+    fptr(conv_state, state.size(0) * (s.taps - 1) * s.inner, "conv_state");
+    is_f32(w_dt, "w_dt");
+    TORCH_CHECK(w_dt.dim() == 2 && w_dt.size(0) == s.inner && w_dt.stride(1) == 1 && w_dt.size(1) >= (s.rank + 7) / 8 * 8, "w_dt");
+  }
+  mb::SelectiveInputs inputs(const Tensor& proj, bool f32, int64_t rows) const {
+    chk_rows(proj, f32, rows, std::max(x_off, z_off) + s.inner, "proj");
+    mb::SelectiveInputs in{};
+    in.proj = proj.data_ptr();
+    in.ld = proj.stride(0);
+    in.x_off = x_off;
+    in.z_off = z_off;
+    in.conv_w = conv_w.data_ptr<float>();
+    in.conv_b = conv_b.data_ptr<float>();
+    in.a = a.data_ptr<float>();
+    in.d = d.data_ptr<float>();
+    in.dt_bias = dt_b.data_ptr<float>();
+    in.conv_state = const_cast<float*>(fptr(conv_state, 0, "conv_state"));
+    in.state = state.data_ptr<float>();
+    in.b_off = b_off;
+    in.c_off = c_off;
+    return in;
+  }
+  mb::SelectiveInputs inputs(const Tensor& proj, const Tensor& x, const Tensor& low, bool f32, int64_t rows) const {
+    mb::SelectiveInputs in = inputs(proj, f32, rows);
+    chk_rows(x, f32, rows, s.inner, "x");
+    chk_rows(low, f32, rows, std::max({b_off + s.state, c_off + s.state, (s.rank + 7) / 8 * 8}), "low");
+    in.x = x.data_ptr();
+    in.ld_x = x.stride(0);
+    in.low = low.data_ptr();
+    in.ld_low = low.stride(0);
+    return in;
+  }
+  void conv(const Tensor& proj, const std::vector<Tensor>& batch, bool one_token, Tensor& x) const {
+    const auto rb = ragged(batch);
+    const bool f32 = is_f32(x, "x");
+    chk_rows(x, f32, rb.rows, s.inner, "x");
+    TORCH_CHECK(x.stride(0) == x.size(1), "conv: x must be contiguous");
+    c10::cuda::CUDAGuard guard(x.device());
+    mb::selective_conv(f32, s, inputs(proj, f32, rb.rows), rb, one_token, x.data_ptr(), x.stride(0), cur_stream());
+  }
+  int64_t scratch_floats(int64_t n_seq, int64_t max_q) const { return mb::selective_scratch(s, (int)n_seq, (int)max_q); }
+  void scan(const Tensor& proj, const Tensor& x, const Tensor& low, const Tensor& dt, const std::vector<Tensor>& batch, int64_t max_q,
+            Tensor& scratch, Tensor& out) const {
+    const auto rb = ragged(batch);
+    const bool f32 = is_f32(out, "out");
+    chk_rows(out, f32, rb.rows, s.inner, "out");
+    chk_rows(dt, true, rb.rows, s.inner, "dt");
+    chk_c(scratch, F32, "scratch");
+    TORCH_CHECK(scratch.numel() >= scratch_floats(rb.n_seq, max_q), "scan: scratch");
+    c10::cuda::CUDAGuard guard(out.device());
+    mb::selective_scan(f32, s, inputs(proj, x, low, f32, rb.rows), rb, (int)max_q, dt.data_ptr<float>(), dt.stride(0),
+                       scratch.data_ptr<float>(), out.data_ptr(), out.stride(0), cur_stream());
+  }
+  // One token per sequence; dt null: computed from the first columns of low.
+  void step(const Tensor& proj, const Tensor& x, const Tensor& low, const OptTensor& dt, const std::vector<Tensor>& batch,
+            Tensor& out) const {
+    const auto rb = ragged(batch);
+    const bool f32 = is_f32(out, "out");
+    chk_rows(out, f32, rb.rows, s.inner, "out");
+    if (dt.has_value()) chk_rows(*dt, true, rb.rows, s.inner, "dt");
+    TORCH_CHECK(is_f32(w_dt, "w_dt") == f32, "step: w_dt and the activations differ in type");
+    c10::cuda::CUDAGuard guard(out.device());
+    mb::selective_step(f32, s, inputs(proj, x, low, f32, rb.rows), rb, dt.has_value() ? dt->data_ptr<float>() : nullptr,
+                       dt.has_value() ? dt->stride(0) : 0, w_dt.data_ptr(), w_dt.stride(0), out.data_ptr(), out.stride(0), cur_stream());
+  }
+};
+
+void soft_cap(Tensor& y, double cap) {
+  chk_rows(y, true, y.size(0), y.size(1), "y");
+  c10::cuda::CUDAGuard guard(y.device());
+  mb::soft_cap(y.data_ptr<float>(), y.stride(0), (int)y.size(0), (int)y.size(1), (float)cap, cur_stream());
+}
+
 }  // namespace
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
@@ -606,16 +718,18 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   namespace py = pybind11;
   m.def("sandwich_norm", &sandwich_norm, py::arg("y1"), py::arg("y2"), py::arg("w1"), py::arg("w2"), py::arg("w_post"), py::arg("x"),
         py::arg("w_next"), py::arg("h"), py::arg("eps"), py::arg("mult") = 1.0);
-  m.def("expert_norm", &expert_norm);
-  m.def("qk_norm_append", &qk_norm_append);
-  m.def("paged_attn_any", &paged_attn_any);
-  m.def("paged_attn_prefill", &paged_attn_prefill);
-  m.def("paged_attn_decode", &paged_attn_decode);
+  m.def("expert_norm", &expert_norm, py::arg("y"), py::arg("shared"), py::arg("row"), py::arg("weight"), py::arg("w_post"), py::arg("x"),
+        py::arg("w_next"), py::arg("h"), py::arg("eps"), py::arg("mult") = 1.0);
   m.def("gemm_decode", &gemm_decode, py::arg("x"), py::arg("w"), py::arg("out"), py::arg("f"), py::arg("f_off"), py::arg("alpha"),
-        py::arg("status"), py::arg("act") = Act(0, 0.0, 0.0), py::arg("mul") = OptTensor(), py::arg("ids") = OptTensor());
+        py::arg("status"), py::arg("act") = Act(0, 0.0, 0.0), py::arg("mul") = OptTensor(), py::arg("ids") = OptTensor(),
+        py::arg("cap") = 0.0);
   m.def("gemm_heads", &gemm_heads);
   m.def("gemm_tiles", &gemm_tiles);
-  m.def("expert_select", &expert_select);
+  m.def("expert_select", &expert_select, py::arg("logits"), py::arg("correction"), py::arg("spec"), py::arg("tile_rows"), py::arg("idx"),
+        py::arg("weight"), py::arg("slot"), py::arg("counts"), py::arg("offset"), py::arg("tiles"), py::arg("count"),
+        py::arg("rule") = RouterRule(0, 1, 0, 1.0));
+  m.def("soft_cap", &soft_cap);
+  m.def("selective_padded_state", [](int64_t state) { return mb::selective_padded_state((int)state); });
   m.def("expert_gather", &expert_gather);
   m.def("gelu_mul", &gelu_mul);
   m.def("gate_pair", &gate_pair);
@@ -693,5 +807,85 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
       .def("attn_decode", &Latent::attn_decode)
       .def("prefill_ok", &Latent::prefill_ok)
       .def("attn_prefill", &Latent::attn_prefill);
+  py::class_<Attention>(m, "Attention")
+      .def(py::init([](py::dict spec, py::dict tensors) {
+        Attention t;
+        auto geti = [&](const char* k, int v) { return spec.contains(k) ? spec[k].cast<int>() : v; };
+        auto getf = [&](const char* k, float v) { return spec.contains(k) ? spec[k].cast<float>() : v; };
+        auto gett = [&](const char* k) -> OptTensor {
+          if (!tensors.contains(k)) return c10::nullopt;
+          return tensors[k].cast<Tensor>();
+        };
+        t.p.heads = geti("heads", 0);
+        t.p.kv_heads = geti("kv_heads", t.p.heads);
+        t.p.dk = geti("dk", 0);
+        t.p.dv = geti("dv", 0);
+        TORCH_CHECK(t.p.heads > 0 && t.p.kv_heads > 0 && t.p.heads % t.p.kv_heads == 0 && t.p.dk > 0 && t.p.dv > 0, "attention: sizes");
+        t.p.q_off = geti("q_off", 0);
+        t.p.k_off = geti("k_off", -1);
+        t.p.v_off = geti("v_off", 0);
+        t.p.norm_dim = geti("norm_dim", 0);
+        t.p.rot = geti("rot", 0);
+        t.p.temp_coef = getf("temp_coef", 0.f);
+        t.p.temp_every = getf("temp_every", 1.f);
+        t.p.eps = getf("eps", 1e-6f);
+        t.scale = getf("scale", 1.f);
+        t.out_scale = getf("out_scale", 1.f);
+        t.window = geti("window", 0);
+        t.gate_channels = geti("gate_channels", 0) != 0;
+        t.q_bias = gett("q_bias");
+        t.k_bias = gett("k_bias");
+        t.v_bias = gett("v_bias");
+        t.q_gamma = gett("q_gamma");
+        t.k_gamma = gett("k_gamma");
+        t.turns = gett("turns");
+        t.sink = gett("sink");
+        TORCH_CHECK(t.window >= 0 && t.p.norm_dim >= 0 && t.p.norm_dim <= t.p.dk && t.p.rot >= 0 && t.p.rot <= t.p.dk && t.p.rot % 2 == 0,
+                    "attention: window / norm / rotation");
+        t.p.q_bias = fptr(t.q_bias, (int64_t)t.p.heads * t.p.dk, "q_bias");
+        t.p.k_bias = fptr(t.k_bias, (int64_t)t.p.kv_heads * t.p.dk, "k_bias");
+        t.p.v_bias = fptr(t.v_bias, (int64_t)t.p.kv_heads * t.p.dv, "v_bias");
+        t.p.q_gamma = fptr(t.q_gamma, t.p.dk, "q_gamma");
+        t.p.k_gamma = fptr(t.k_gamma, t.p.dk, "k_gamma");
+        fptr(t.sink, t.p.heads, "sink");
+        if (t.p.rot > 0) {
+          TORCH_CHECK(t.turns.has_value(), "attention: turns");
+          chk_c(*t.turns, torch::kFloat64, "turns");
+          TORCH_CHECK(t.turns->numel() >= t.p.rot / 2, "attention: turns");
+          t.p.turns = t.turns->data_ptr<double>();
+        }
+        return t;
+      }))
+      .def("prep", &Attention::prep)
+      .def("any", &Attention::any)
+      .def("tensor_ok", &Attention::tensor_ok)
+      .def("prefill", &Attention::prefill)
+      .def("decode", &Attention::decode)
+      .def("decode_scratch", &Attention::decode_scratch);
+  py::class_<Selective>(m, "Selective")
+      .def(py::init([](py::dict spec, py::dict tensors) {
+        Selective t;
+        auto geti = [&](const char* k) { return spec[k].cast<int>(); };
+        auto gett = [&](const char* k) { return tensors[k].cast<Tensor>(); };
+        t.s = mb::SelectiveSpec{geti("inner"), geti("state"), geti("rank"), geti("taps"), spec["out_scale"].cast<float>()};
+        t.x_off = geti("x_off");
+        t.z_off = geti("z_off");
+        t.b_off = geti("b_off");
+        t.c_off = geti("c_off");
+        t.conv_w = gett("conv_w");
+        t.conv_b = gett("conv_b");
+        t.a = gett("a");
+        t.d = gett("d");
+        t.dt_b = gett("dt_b");
+        t.state = gett("state");
+        t.w_dt = gett("w_dt");
+        if (tensors.contains("conv_state")) t.conv_state = gett("conv_state");
+        t.validate();
+        return t;
+      }))
+      .def("conv", &Selective::conv)
+      .def("scratch_floats", &Selective::scratch_floats)
+      .def("scan", &Selective::scan)
+      .def("step", &Selective::step);
   m.def("launch_count", []() { return (int64_t)mb::launch_counter().load(); });
 }

@@ -168,14 +168,24 @@ void flash_attn_fwd2_strided(const void* q, const void* k, const void* v, void* 
                              long long o_tok_stride, bool causal, float scale, int* status, cudaStream_t stream);
 void set_attn_fwd_mode(int mode);
 int get_attn_fwd_mode();
+// What attention over the pages does besides softmax(scale q k) v.
+struct AttnExtras {
+  const void* gate = nullptr;   // logits of a sigmoid output gate: one per head, or (gate_channels) one per output value
+  long long ld_gate = 0;        // row stride of the gate
+  bool gate_channels = false;
+  const float* sink = nullptr;  // [heads] one more logit per head in the softmax denominator
+  int window = 0;               // keys a query sees, its own included (0: all earlier ones)
+  float out_scale = 1.f;        // factor of the output
+};
 // Prefill attention over the paged KV cache (tcgen05, causal): q holds the NEW tokens of `batch` sequences
 // packed back to back (sequence b = rows cu_q[b] .. cu_q[b+1]); k_cache / v_cache are bf16 pages
 // [n_pages, 16, kv_heads, head_dim] addressed through block_table [batch, table_stride]; kv_lens[b] counts the
-// keys the last query of b sees (cached prefix + new tokens, which must already be in the pages).
+// keys the last query of b sees (cached prefix + new tokens, which must already be in the pages). Head widths (keys dk,
+// values dv): multiples of 8 up to 128.
 void flash_attn_paged_prefill(const void* q, long long q_tok_stride, const void* k_cache, const void* v_cache,
                               int n_pages, const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
                               void* o, long long o_tok_stride, int batch, int total_q, int max_q_len, int heads,
-                              int kv_heads, int dk, int dv, const void* gate, long long ld_gate, float scale, int* status,
+                              int kv_heads, int dk, int dv, const AttnExtras& ex, float scale, int* status,
                               cudaStream_t stream);
 // Causal attention of packed queries over packed keys and values of their own heads, with a second query / key part
 // whose key is shared by all heads and one more denominator logit per head (attention_fwd.cu, FA_RAGGED). Queries
@@ -342,13 +352,14 @@ void kv_append(const void* k, const void* v, void* k_cache, void* v_cache, const
                int max_pages, long long kv_tok_stride, cudaStream_t stream);
 // One query token per sequence: q [batch, heads, head_dim]; context_lens [batch]. Split-KV flash
 // decoding: partials in `scratch` (>= batch*heads*splits*(value width+2) floats), combined in-kernel.
-// v_head_dim: value width (0: = head_dim); gate: optional per-head output gate logits [batch, heads], row
-// stride ld_gate. `counters`: one per (sequence, kv head, sub-group of 8 query heads).
+// v_head_dim: value width (0: = head_dim); ldo: row stride of out (0: contiguous). Unequal widths, widths other than
+// 64 and 128 (multiples of 8 up to 128) and `ex` need 16-token pages. `counters`: one per (sequence, kv head,
+// sub-group of 8 query heads).
 void paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
                        const int* context_lens, void* out, float* scratch, int* counters, int batch, int heads,
                        int kv_heads, int head_dim, int page_size, int max_pages, int cache_pages, int splits,
                        float scale, int* status, cudaStream_t stream, long long q_tok_stride = 0, int v_head_dim = 0,
-                       const void* gate = nullptr, long long ld_gate = 0);
+                       const AttnExtras& ex = AttnExtras{}, long long ldo = 0);
 // int8 pages: k_cache / v_cache [num_pages, page_size, kv_heads, head_dim] int8 with one fp32 scale
 // (max|x| / 127) per (token, kv head) in k_scale / v_scale [num_pages * page_size, kv_heads].
 void kv_append_int8(const void* k, const void* v, void* k_cache, void* v_cache, float* k_scale, float* v_scale,

@@ -12,6 +12,7 @@
 // without a transpose. Replaces the reference's materialised S x S attention
 // (src/autograd.cpp:361-461) and its CPU tiled kernel (src/flash_attention.cpp:37-159).
 #include "api.h"
+#include "common.cuh"
 #include "host_util.h"
 #include "tc.cuh"
 
@@ -51,19 +52,23 @@ struct FaFwdCfg {
 //
 // MODE FA_RAGGED: the same packed queries over packed keys and values (sequence b at rows cu_k[b] ..), keys
 // and values per query head. The last DR columns of queries and keys are a second pair of tensors: a part
-// of the key that all heads share (one row per token). Widths below a multiple of 64 are filled with zeros
-// by TMA. Sequences with fewer than min_q new tokens are left out.
+// of the key that all heads share (one row per token). Sequences with fewer than min_q new tokens are left out.
 //
-// sink (FA_PAGED and FA_RAGGED, may be null): one more logit per head in the softmax denominator.
+// FA_PAGED and FA_RAGGED: widths below a multiple of 64 are filled with zeros by TMA; sink (may be null): one more
+// logit per head in the softmax denominator; window (0: none): keys a query sees, its own included. A CTA starts at
+// the first key tile its first query sees, so a later row may meet tiles in which it sees nothing yet.
 enum { FA_DENSE = 0, FA_PAGED = 1, FA_RAGGED = 2 };
 struct PagedPrefillArgs {
   const int* block_table;   // [batch, table_stride] page ids
   const int* cu_q;          // [batch + 1] first query row of every sequence
   const int* kv_lens;       // [batch] keys visible to the LAST query of the sequence (prefix + new tokens)
   int table_stride;
-  const __nv_bfloat16* gate;   // [total_q, >= heads] logits of a per-head output gate (sigmoid), or null
-  long long ld_gate;
+  const __nv_bfloat16* gate;   // logits of an output gate (sigmoid), or null: [total_q, >= heads], or
+  long long ld_gate;           // [total_q, heads * o_cols] with gate_channels
+  bool gate_channels;
   const float* sink;           // [heads]
+  int window;
+  float out_scale;             // factor of the output
   const int* cu_k;             // FA_RAGGED: first key row of every sequence
   int min_q, o_cols;           // FA_RAGGED: see above; output columns of a head
 };
@@ -107,11 +112,15 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
     if (MODE == FA_RAGGED && q_len < pa.min_q) return;
   }
   const int n_qt = (q0 + FA_BM < q_len) ? 2 : 1;
-  int J[2];
+  int jb = 0;                                    // first key tile
+  if constexpr (PAGED) {
+    if (pa.window > 0) jb = max(0, q_off + q0 - pa.window + 1) / FA_BN;
+  }
+  int J[2];                                      // key tiles from jb on
 #pragma unroll
   for (int t = 0; t < 2; ++t) {
     const int hi = causal ? min(kv_len, q_off + min(q_len, q0 + (t + 1) * FA_BM)) : kv_len;
-    J[t] = (t < n_qt) ? (hi + FA_BN - 1) / FA_BN : 0;
+    J[t] = (t < n_qt) ? (hi + FA_BN - 1) / FA_BN - jb : 0;
   }
   const int Jmax = max(J[0], J[1]);
 
@@ -162,7 +171,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
         uint8_t* sk = smem + Cfg::OFF_KV + st * Cfg::STAGE_BYTES;
         uint8_t* sv = sk + Cfg::K_BYTES;
         if constexpr (MODE == FA_RAGGED) {
-          const int row = pa.cu_k[b] + j * FA_BN;
+          const int row = pa.cu_k[b] + (jb + j) * FA_BN;
           for (int c = 0; c < DCK; ++c) tma_load_4d(sk + c * (FA_BN * 128), &tm_k, &kv_full[st], c * 64, h, row, 0);
           for (int c = 0; c < DCR; ++c) tma_load_4d(sk + (DCK + c) * (FA_BN * 128), &tm_k2, &kv_full[st], c * 64, 0, row, 0);
           for (int c = 0; c < DCV; ++c) tma_load_4d(sv + c * (FA_BN * 128), &tm_v, &kv_full[st], c * 64, h, row, 0);
@@ -172,7 +181,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
           const int* row = pa.block_table + (long long)b * pa.table_stride;
 #pragma unroll
           for (int p = 0; p < FA_BN / FA_PAGE; ++p) {
-            const int lp = j * (FA_BN / FA_PAGE) + p;
+            const int lp = (jb + j) * (FA_BN / FA_PAGE) + p;
             int page = (lp * FA_PAGE < kv_len && lp < pa.table_stride) ? row[lp] : 0;
             if (page < 0) page = 0;
             for (int c = 0; c < DCK; ++c)
@@ -258,6 +267,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
     uint8_t* p_tile = smem + Cfg::OFF_P + t * Cfg::P_BYTES;
     float m_ref = 0.f, l = 0.f;
     bool ok = true;
+    bool first = true;              // no visible key so far (PAGED): O and l are zero and m_ref is free
     for (int j = 0; j < J[t] && ok; ++j) {
       ok = mbar_wait(&s_full[t], j & 1, abort_flag, status, 16);
       ok = __all_sync(0xffffffffu, ok);
@@ -268,12 +278,20 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       tmem_ld32(t_s + 32, sr[1]);
       tmem_ld_wait();
       float* s = reinterpret_cast<float*>(&sr[0][0]);
-      const int kv0 = j * FA_BN;
+      const int kv0 = (jb + j) * FA_BN;
       const int limit = causal ? min(kv_len - 1, q_off + q_row) : kv_len - 1;  // last visible kv index
       if (kv0 + FA_BN - 1 > limit) {
 #pragma unroll
         for (int i = 0; i < FA_BN; ++i)
           if (kv0 + i > limit) s[i] = -INFINITY;
+      }
+      if constexpr (PAGED) {
+        const int lo = pa.window > 0 ? q_off + q_row - pa.window + 1 : 0;   // first visible kv index
+        if (kv0 < lo) {
+#pragma unroll
+          for (int i = 0; i < FA_BN; ++i)
+            if (kv0 + i < lo) s[i] = -INFINITY;
+        }
       }
       float mx4[4] = {s[0], s[1], s[2], s[3]};  // four independent chains instead of one of length 64
 #pragma unroll
@@ -282,8 +300,9 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       const float m_new = mx * scale_log2;
       float alpha = 1.f;
       bool need = false;
-      if (j == 0) {
+      if (PAGED ? first : j == 0) {
         m_ref = (m_new == -INFINITY) ? 0.f : m_new;
+        first = m_new == -INFINITY;
       } else if (m_new - m_ref > 8.f) {
         need = true;
         alpha = fast_exp2(m_ref - m_new);
@@ -338,12 +357,17 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
           if (pa.sink) l += exp2f(pa.sink[h] * 1.4426950408889634f - m_ref);
         }
         float inv_l = l > 0.f ? 1.f / l : 0.f;
+        const __nv_bfloat16* grow = nullptr;      // the row's gate logits of this head's channels
         if constexpr (PAGED) {
-          if (pa.gate && q_row < q_len)
-            inv_l /= 1.f + expf(-__bfloat162float(pa.gate[(long long)(q_row0 + q_row) * pa.ld_gate + h]));
+          inv_l *= pa.out_scale;
+          if (pa.gate && q_row < q_len) {
+            const __nv_bfloat16* gp = pa.gate + (long long)(q_row0 + q_row) * pa.ld_gate;
+            if (pa.gate_channels) grow = gp + (long long)h * pa.o_cols;
+            else inv_l /= 1.f + expf(-__bfloat162float(gp[h]));
+          }
         }
         __nv_bfloat16* orow = o + (PAGED ? (long long)(q_row0 + q_row) : (long long)b * seq + q_row) * o_tok_stride +
-                              (long long)h * (MODE == FA_RAGGED ? pa.o_cols : DV);
+                              (long long)h * (PAGED ? pa.o_cols : DV);
 #pragma unroll 1
         for (int c = 0; c < DV / 32; ++c) {
           uint32_t orr[32];
@@ -353,12 +377,22 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
             uint4* p4 = reinterpret_cast<uint4*>(orow + c * 32);
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
+              if (PAGED && c * 32 + i * 8 >= pa.o_cols) break;
+              if constexpr (MODE == FA_PAGED) {
+                if (grow) {
+                  float g[8];
+                  unpack8(ldg8(grow, c * 32 + i * 8), g);
+#pragma unroll
+                  for (int e = 0; e < 8; ++e)
+                    orr[8 * i + e] = __float_as_uint(__fdividef(__uint_as_float(orr[8 * i + e]), 1.f + __expf(-g[e])));
+                }
+              }
               uint4 v;
               v.x = pack_bf16x2(__uint_as_float(orr[8 * i + 0]) * inv_l, __uint_as_float(orr[8 * i + 1]) * inv_l);
               v.y = pack_bf16x2(__uint_as_float(orr[8 * i + 2]) * inv_l, __uint_as_float(orr[8 * i + 3]) * inv_l);
               v.z = pack_bf16x2(__uint_as_float(orr[8 * i + 4]) * inv_l, __uint_as_float(orr[8 * i + 5]) * inv_l);
               v.w = pack_bf16x2(__uint_as_float(orr[8 * i + 6]) * inv_l, __uint_as_float(orr[8 * i + 7]) * inv_l);
-              if (MODE != FA_RAGGED || c * 32 + i * 8 < pa.o_cols) p4[i] = v;
+              p4[i] = v;
             }
           }
         }
@@ -440,15 +474,18 @@ void flash_attn_fwd_strided(const void* q, const void* k, const void* v, void* o
 void flash_attn_paged_prefill(const void* q, long long q_tok_stride, const void* k_cache, const void* v_cache,
                               int n_pages, const int* block_table, int table_stride, const int* cu_q, const int* kv_lens,
                               void* o, long long o_tok_stride, int batch, int total_q, int max_q_len, int heads,
-                              int kv_heads, int dk, int dv, const void* gate, long long ld_gate, float scale, int* status,
+                              int kv_heads, int dk, int dv, const AttnExtras& ex, float scale, int* status,
                               cudaStream_t stream) {
-  MB_REQUIRE((dk == 64 || dk == 128) && (dv == 64 || dv == 128), "flash_attn_paged_prefill: head widths must be 64 or 128");
+  MB_REQUIRE(dk > 0 && dk <= 128 && dk % 8 == 0 && dv > 0 && dv <= 128 && dv % 8 == 0,
+             "flash_attn_paged_prefill: head widths must be multiples of 8 up to 128");
+  MB_REQUIRE(ex.window >= 0 && (!ex.gate_channels || (ex.ld_gate % 8 == 0 && (reinterpret_cast<uintptr_t>(ex.gate) & 15) == 0)),
+             "flash_attn_paged_prefill: window / gate alignment");
   MB_REQUIRE(heads % kv_heads == 0, "flash_attn_paged_prefill: heads must be a multiple of kv_heads");
   MB_REQUIRE(q_tok_stride % 8 == 0 && o_tok_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0,
              "flash_attn_paged_prefill: strides / alignment");
   if (batch == 0 || total_q == 0 || max_q_len == 0) return;
   const CUtensorMap tq = make_bshd_map(q, 1, total_q, heads, dk, q_tok_stride, FA_BM);
-  // pages: [n_pages, 16 tokens, kv_heads, width]; one box = 16 tokens x 64 columns of one head
+  // pages: [n_pages, 16 tokens, kv_heads, width]; one box = 16 tokens x 64 columns of one head (zeros past its width)
   auto page_map = [&](const void* base, int width) {
     uint64_t dims[4] = {(uint64_t)width, (uint64_t)kv_heads, (uint64_t)FA_PAGE, (uint64_t)n_pages};
     uint64_t strides[3] = {(uint64_t)width * 2, (uint64_t)kv_heads * width * 2, (uint64_t)FA_PAGE * kv_heads * width * 2};
@@ -458,15 +495,16 @@ void flash_attn_paged_prefill(const void* q, long long q_tok_stride, const void*
   const CUtensorMap tk = page_map(k_cache, dk), tv = page_map(v_cache, dv);
   const dim3 grid((max_q_len + 2 * FA_BM - 1) / (2 * FA_BM), heads, batch);
   const float scale_log2 = scale * 1.4426950408889634f;
-  PagedPrefillArgs pa{block_table, cu_q, kv_lens, table_stride, (const __nv_bfloat16*)gate, ld_gate, nullptr, nullptr, 0, dv};
+  PagedPrefillArgs pa{block_table, cu_q, kv_lens, table_stride, (const __nv_bfloat16*)ex.gate, ex.ld_gate, ex.gate_channels,
+                      ex.sink, ex.window, ex.out_scale, nullptr, 0, dv};
   auto go = [&](auto kern, int smem) {
     MB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     kern<<<grid, FA_THREADS, smem, stream>>>(tq, tk, tv, (__nv_bfloat16*)o, nullptr, total_q, heads, kv_heads,
                                              o_tok_stride, 1, scale_log2, status, pa, tq, tk);
   };
-  if (dk == 128 && dv == 128) go(fa_fwd_kernel<128, 128, FA_PAGED>, FaFwdCfg<128, 128>::SMEM_BYTES);
-  else if (dk == 64 && dv == 128) go(fa_fwd_kernel<64, 128, FA_PAGED>, FaFwdCfg<64, 128>::SMEM_BYTES);
-  else if (dk == 128 && dv == 64) go(fa_fwd_kernel<128, 64, FA_PAGED>, FaFwdCfg<128, 64>::SMEM_BYTES);
+  if (dk > 64 && dv > 64) go(fa_fwd_kernel<128, 128, FA_PAGED>, FaFwdCfg<128, 128>::SMEM_BYTES);
+  else if (dv > 64) go(fa_fwd_kernel<64, 128, FA_PAGED>, FaFwdCfg<64, 128>::SMEM_BYTES);
+  else if (dk > 64) go(fa_fwd_kernel<128, 64, FA_PAGED>, FaFwdCfg<128, 64>::SMEM_BYTES);
   else go(fa_fwd_kernel<64, 64, FA_PAGED>, FaFwdCfg<64, 64>::SMEM_BYTES);
   count_launch();
   check_launch();
@@ -490,7 +528,7 @@ void flash_attn_ragged(const RaggedAttn& a, int* status, cudaStream_t stream) {
   const CUtensorMap tk = map(a.k, a.total_k, a.heads, a.dim, a.ldkv, FA_BN), tv = map(a.v, a.total_k, a.heads, a.vdim, a.ldkv, FA_BN);
   const CUtensorMap tk2 = map(a.k_rot, a.total_k, 1, a.rot, a.ldk_rot, FA_BN);
   const dim3 grid((a.max_q + 2 * FA_BM - 1) / (2 * FA_BM), a.heads, a.batch);
-  PagedPrefillArgs pa{nullptr, a.cu_q, a.kv_lens, 0, nullptr, 0, a.sink, a.cu_k, a.min_q, a.vdim};
+  PagedPrefillArgs pa{nullptr, a.cu_q, a.kv_lens, 0, nullptr, 0, false, a.sink, 0, 1.f, a.cu_k, a.min_q, a.vdim};
   auto go = [&](auto kern, int smem) {
     MB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     kern<<<grid, FA_THREADS, smem, stream>>>(tq, tk, tv, (__nv_bfloat16*)a.o, nullptr, a.total_q, a.heads, a.heads, a.ldo, 1,

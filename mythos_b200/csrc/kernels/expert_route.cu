@@ -1,7 +1,7 @@
 // Routing of tokens to experts for serving (hybrid_api.h).
 //
-//   expert_select  one warp per token: softmax over all router logits, choice scores (score + correction),
-//                  the best groups of neighbouring experts, the best experts in them, a place inside each
+//   expert_select  one warp per token: scores of all router logits (softmax or sigmoid), choice scores (score +
+//                  correction), the best groups of neighbouring experts, the best experts in them, a place inside each
 //                  chosen expert's row segment. The last CTA to finish turns the counts into segments and a
 //                  tile list for the grouped GEMMs and clears the counts for the next launch.
 //   expert_gather  token rows into their segments.
@@ -11,6 +11,7 @@
 #include "common.cuh"
 #include "host_util.h"
 #include "hybrid_api.h"
+#include "hybrid_dev.cuh"
 
 namespace mb {
 namespace {
@@ -43,27 +44,39 @@ expert_select_kernel(const float* __restrict__ logits, long long ldz, const floa
   const int t = blockIdx.x * ER_WARPS + warp;
   if (t < rows) {
     const float* z = logits + (long long)t * ldz;
-    float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-    mx = warp_max(mx);
-    float sum = 0.f;
-    for (int e = lane; e < E; e += 32) {
-      const float p = expf(z[e] - mx);
-      score[e] = p;
-      sum += p;
-    }
-    sum = warp_sum(sum);
-    for (int e = lane; e < E; e += 32) {
-      const float p = score[e] / sum;
-      score[e] = p;
-      choice[e] = p + correction[e];
+    if (s.sigmoid) {
+      for (int e = lane; e < E; e += 32) {
+        const float p = sigmoid_f(z[e]);
+        score[e] = p;
+        choice[e] = p + (correction ? correction[e] : 0.f);
+      }
+    } else {
+      float mx = -INFINITY;
+      for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+      mx = warp_max(mx);
+      float sum = 0.f;
+      for (int e = lane; e < E; e += 32) {
+        const float p = expf(z[e] - mx);
+        score[e] = p;
+        sum += p;
+      }
+      sum = warp_sum(sum);
+      for (int e = lane; e < E; e += 32) {
+        const float p = score[e] / sum;
+        score[e] = p;
+        choice[e] = p + (correction ? correction[e] : 0.f);
+      }
     }
     __syncwarp();
     if (s.keep < s.groups) {
       for (int g = lane; g < s.groups; g += 32) {
-        float m = choice[g * size];
-        for (int i = 1; i < size; ++i) m = fmaxf(m, choice[g * size + i]);
-        best[g] = m;
+        float m = choice[g * size], m2 = -INFINITY;     // the two largest
+        for (int i = 1; i < size; ++i) {
+          const float c = choice[g * size + i];
+          m2 = fmaxf(m2, fminf(m, c));
+          m = fmaxf(m, c);
+        }
+        best[g] = s.group_best == 2 && size > 1 ? m + m2 : m;
       }
       __syncwarp();
       for (int j = 0; j < s.groups - s.keep; ++j) {      // strike out the worst groups
@@ -86,6 +99,7 @@ expert_select_kernel(const float* __restrict__ logits, long long ldz, const floa
         __syncwarp();
       }
     }
+    float mine = 0.f, total = 0.f;                      // lane j keeps the score of choice j
     for (int j = 0; j < s.top; ++j) {
       float v = -INFINITY;
       int at = 0x7fffffff;
@@ -96,15 +110,18 @@ expert_select_kernel(const float* __restrict__ logits, long long ldz, const floa
         }
       warp_argmax(v, at);
       at = min(at, E - 1);
+      const float p = score[at];
+      total += p;
+      if (lane == j) mine = p;
       if (lane == 0) {
         choice[at] = -INFINITY;
         const long long o = (long long)t * s.top + j;
         b.idx[o] = at;
-        b.weight[o] = score[at];
         b.slot[o] = atomicAdd(&b.counts[at], 1);
       }
       __syncwarp();
     }
+    if (lane < s.top) b.weight[(long long)t * s.top + lane] = s.normalise ? mine / (total + 1e-20f) * s.scale : mine;
   }
   // ---- the last CTA plans the segments
   __threadfence();
@@ -170,7 +187,8 @@ void expert_select(const float* logits, long long ldz, const float* correction, 
                    int tile_rows, int rows, cudaStream_t stream) {
   MB_REQUIRE(s.experts > 0 && s.experts <= ER_MAX_EXPERTS, "expert_select: at most 1024 experts");
   MB_REQUIRE(s.groups > 0 && s.experts % s.groups == 0 && s.keep > 0 && s.keep <= s.groups &&
-                 s.top > 0 && s.top <= s.experts / s.groups * s.keep, "expert_select: groups / top");
+                 s.top > 0 && s.top <= 32 && s.top <= s.experts / s.groups * s.keep && (s.group_best == 1 || s.group_best == 2),
+             "expert_select: groups / top");
   MB_REQUIRE(tile_rows > 0, "expert_select: tile rows");
   if (rows == 0) return;
   const int smem = ER_WARPS * (2 * s.experts + s.groups) * 4;

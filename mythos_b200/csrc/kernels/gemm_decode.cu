@@ -47,6 +47,7 @@ __device__ __forceinline__ float gd_ld_cluster(uint32_t addr) {
 
 // Value of one output element before it is stored.
 __device__ __forceinline__ float gd_tail(const GemmTail& tail, float y, int token, int n) {
+  if (tail.cap > 0.f) return soft_cap_f(y, tail.cap);
   if (tail.mul == nullptr) return y;
   const int id = min(max(tail.mul_ids[token], 0), tail.vocab - 1);
   return gelu_tanh_f(y) * __bfloat162float(static_cast<const __nv_bfloat16*>(tail.mul)[id * tail.ld_mul + n]);
@@ -391,7 +392,7 @@ void gemm_decode(const void* x, long long ldx, const void* W, long long ldw, voi
   MB_REQUIRE(ldx % 8 == 0 && ldw % 8 == 0 && (!many || (group.x_batch % 8 == 0 && group.w_batch % 8 == 0)),
              "gemm_decode: strides must be multiples of 8 elements");
   MB_REQUIRE(f_off == 0 || f_off >= N, "gemm_decode: the up half starts after the gate half");
-  MB_REQUIRE(!(tail.mul && f_off), "gemm_decode: one tail at a time");
+  MB_REQUIRE((tail.mul != nullptr) + (f_off > 0) + (tail.cap > 0.f) <= 1, "gemm_decode: one tail at a time");
   int mt = (M + 15) / 16 * 16;
   if (mt > 128) mt = 128;
   if (group.list) mt = group.mt;
@@ -431,7 +432,7 @@ void gemm_segments(const void* x, long long ldx, const void* W, long long ldw, l
   MB_REQUIRE(ldx % 8 == 0 && ldw % 8 == 0 && w_batch % 8 == 0 && ldo % 8 == 0 && N % 8 == 0 &&
                  (reinterpret_cast<uintptr_t>(out) & 15) == 0, "gemm_segments: alignment");
   MB_REQUIRE(tail.f_off == 0 || tail.f_off >= N, "gemm_segments: the up half starts after the gate half");
-  MB_REQUIRE(tail.mul == nullptr, "gemm_segments: gated tail only");
+  MB_REQUIRE(tail.mul == nullptr && tail.cap <= 0.f, "gemm_segments: gated tail only");
   static bool configured = false;
   if (!configured) {
     MB_CUDA_CHECK(cudaFuncSetAttribute(gemm_segments_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, GS_SMEM));

@@ -1,6 +1,6 @@
 // Launch API of the kernels behind layer-list ("hybrid") models: gated linear attention and gated
-// delta-rule recurrences, attention with unequal key / value widths and per-head output gates, attention
-// over a cached latent, routed experts, RMSNorms around sublayers on a 32-bit residual stream, and the
+// delta-rule recurrences, selective scans, attention with unequal key / value widths, windows, sinks and output
+// gates, attention over a cached latent, routed experts, RMSNorms around sublayers on a 32-bit residual stream, and the
 // GEMMs those models need beside gemm.cu.
 // Same conventions as api.h (raw pointers, asynchronous on `stream`, exceptions on bad arguments).
 // `f32` selects the activation type: false = bf16 (serving), true = 32-bit floats throughout.
@@ -10,6 +10,8 @@
 #include <stdint.h>
 
 namespace mb {
+
+struct AttnExtras;   // api.h
 
 // A ragged batch of new tokens: sequence b owns rows cu_q[b] .. cu_q[b+1]; kv_lens[b] counts its
 // tokens including the new ones; slots[b] is its state slot; row_seq[t] = b; pos[t] = position.
@@ -25,7 +27,7 @@ void embed_pos_norm(bool f32, const int* ids, const int* pos, const void* embed,
                     float eps, cudaStream_t stream);
 
 // Output of a sublayer: y1 alone; (rms(y1) * w1 + rms(y2) * w2) / 2; or the sum over j < top of
-// weight[t, j] * y1[row[t, j]] (routed experts).
+// weight[t, j] * y1[row[t, j]] (routed experts), plus y2[t] if there is one (their shared expert).
 struct SublayerOut {
   const void *y1, *y2;
   long long ld;
@@ -38,18 +40,28 @@ struct SublayerOut {
 void sandwich_norm(bool f32, const SublayerOut& y, const float* w_post, float mult, float* x, const float* w_next, void* h,
                    long long ldh, int rows, int dim, float eps, cudaStream_t stream);
 
-// Per-head RMSNorm of q and k, q written out, k and v stored into their pages (key width dk, value width dv).
-void qk_norm_append(bool f32, const void* proj, long long ld, int q_off, int k_off, int v_off, const float* q_gamma,
-                    const float* k_gamma, const RaggedBatch& rb, const int* block_table, int table_stride,
-                    int page_size, void* q_out, void* k_cache, void* v_cache, int heads, int kv_heads, int dk, int dv,
-                    float eps, cudaStream_t stream);
+// How projected heads become queries, keys and values: bias, RMS norm of every q and k head, rotation, query
+// temperature. q [rows, heads, dk] is written out, k and v go to their pages. dk and dv are the stored widths;
+// columns past a head's true width are zero in the projection and stay zero.
+struct HeadPrep {
+  int heads, kv_heads, dk, dv;
+  int q_off, k_off, v_off;          // columns of the projection; k_off < 0: queries only
+  const float *q_bias, *k_bias, *v_bias;      // [heads * dk], [kv_heads * dk], [kv_heads * dv], or null
+  int norm_dim;                     // columns the norm averages over; 0: no norm
+  const float *q_gamma, *k_gamma;   // [dk] norm weights, or null
+  const double* turns;              // revolutions per position of the pair (i, i + rot / 2)
+  int rot;                          // rotated columns (0: none)
+  float temp_coef, temp_every;      // queries times 1 + coef ln(floor((pos + 1) / every) + 1); coef 0: none
+  float eps;
+};
+void attn_prep(bool f32, const void* proj, long long ld, const HeadPrep& p, const RaggedBatch& rb, const int* block_table,
+               int table_stride, int page_size, void* q_out, void* k_cache, void* v_cache, cudaStream_t stream);
 
-// Causal attention of every new token over its sequence's pages, any widths, 32-bit arithmetic.
-// gate (may be null): logits [rows, heads] with row stride ld_gate; head h is multiplied by sigmoid(gate[t, h]).
-// block_table row b belongs to sequence b of the batch.
+// Causal attention of every new token over its sequence's pages, any widths, 32-bit arithmetic. The gate of `ex` is in
+// the activation type. block_table row b belongs to sequence b of the batch.
 void paged_attn_any(bool f32, const void* q, const void* k_cache, const void* v_cache, const RaggedBatch& rb,
-                    const int* block_table, int table_stride, int page_size, const void* gate, long long ld_gate,
-                    void* o, long long ldo, int heads, int kv_heads, int dk, int dv, float scale, cudaStream_t stream);
+                    const int* block_table, int table_stride, int page_size, const AttnExtras& ex, void* o, long long ldo,
+                    int heads, int kv_heads, int dk, int dv, float scale, cudaStream_t stream);
 
 // Segments of rows that meet a weight matrix each: tiles[i] = (matrix, first row, rows), *count of them.
 struct TileList {
@@ -68,8 +80,8 @@ struct GateAct {
   int kind;                 // 0: silu(g) u   1: relu(g) u   2: g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit),
   float limit, alpha;       //    u' = u clamped to [-limit, limit]
 };
-// What a few-token GEMM does with the products of a row: nothing; a gated activation of two halves of W; or
-// gelu_tanh(y) * mul[mul_ids[t] * ld_mul + n].
+// What a few-token GEMM does with the products of a row: nothing; a gated activation of two halves of W;
+// gelu_tanh(y) * mul[mul_ids[t] * ld_mul + n]; or a soft cap.
 struct GemmTail {
   int f_off;                // > 0: W holds a gate matrix in rows [0, N) and an up matrix from row f_off
   GateAct act;
@@ -77,6 +89,7 @@ struct GemmTail {
   const int* mul_ids;
   long long ld_mul;
   int vocab;                // rows of mul
+  float cap;                // > 0: y <- cap tanh(y / cap)
 };
 // Several products in one launch: `batch` of them side by side (x, W and out advance by *_batch elements), or with
 // `list` (tile rows = mt: 16, 32, 64 or 128) rows grouped by matrix, W advancing by w_batch elements.
@@ -103,20 +116,27 @@ void gate_pair(bool f32, const void* gu, long long ldg, int f, int f_off, const 
 void gelu_mul(bool f32, void* y, long long ldy, const void* table, long long ld_table, const int* ids, int vocab, int rows,
               int width, cudaStream_t stream);
 
+// y[t, n] = cap * tanh(y[t, n] / cap) in place, n < width
+void soft_cap(float* y, long long ldy, int rows, int width, float cap, cudaStream_t stream);
+
 // ---- routed experts (expert_route.cu)
 struct RouterSpec {
   int experts, top, groups, keep;
+  int sigmoid;              // scores: 0 softmax over all experts, 1 sigmoid of each logit
+  int group_best;           // a group counts the sum of its 1 or 2 largest choice scores
+  int normalise;            // 1: the chosen scores are divided by their sum (+ 1e-20) and multiplied by scale
+  float scale;
 };
 struct RouterBuffers {
   int* idx;                 // [rows, top] chosen expert
-  float* weight;            // [rows, top] its score
+  float* weight;            // [rows, top] its score, normalised if the router says so
   int* slot;                // [rows, top] place within the expert's segment
   int* counts;              // [experts + 1], zero before the first launch and left zero by every launch
   int* offset;              // [experts] first row of the segment
   int *tiles, *tile_count;  // tile list for `tile_rows` rows a tile
   int max_tiles;
 };
-// Softmax scores of fp32 logits, choice by score + correction within the best groups, row segments per expert.
+// Scores of fp32 logits, choice by score + correction (may be null) within the best groups, row segments per expert.
 void expert_select(const float* logits, long long ldz, const float* correction, const RouterSpec& s, const RouterBuffers& b,
                    int tile_rows, int rows, cudaStream_t stream);
 // Rows of h (row_bytes each, a multiple of 16) into their segments; row[t, j] = where (t, j) went.
@@ -206,6 +226,42 @@ void recurrent_decode(bool f32, const RecurrentSpec& s, const RecurrentInputs& i
 // Shift the new inputs into the convolution state (after every reader of the old state has run).
 void conv_state_update(bool f32, const RecurrentSpec& s, const RecurrentInputs& in, const RaggedBatch& rb,
                        cudaStream_t stream);
+// ---- selective scan (selective_scan.cu), per channel c and state value n:
+// S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n;  out_c = (sum_n S[c, n] C_n + D_c x_c) silu(z_c) out_scale
+// with x = silu(short convolution of the projection's x columns + bias) and dt = softplus(pre-activation + bias).
+struct SelectiveSpec {
+  int inner, state, rank, taps;     // channels, state values per channel, width of the map to dt, convolution taps
+  float out_scale;
+};
+int selective_padded_state(int state);   // state values per channel as stored
+struct SelectiveInputs {
+  const void* proj;                 // [rows, ld]: x | z columns at the offsets below
+  long long ld;
+  int x_off, z_off;
+  const float *conv_w, *conv_b;     // [taps, inner] (last row: the current token's), [inner]
+  const float* a;                   // [inner, padded state]: A log2(e), zero in the padding
+  const float *d, *dt_bias;         // [inner]
+  float* conv_state;                // [slots][taps - 1][inner]
+  float* state;                     // [slots][inner][padded state]
+  const void* low;                  // [rows, ld_low]: x's maps, dt columns from 0, B and C columns at the offsets below
+  long long ld_low;
+  int b_off, c_off;
+  const void* x;                    // [rows, ld_x] the convolved channels
+  long long ld_x;
+};
+// x = silu(conv) of a ragged batch, columns [inner, ldx) zeroed; the convolution state advances.
+void selective_conv(bool f32, const SelectiveSpec& s, const SelectiveInputs& in, const RaggedBatch& rb, bool one_token,
+                    void* x, long long ldx, cudaStream_t stream);
+// Prompts and portions; dt [rows, ld_dt]: pre-activations without bias. Long portions are cut into chunks that run side
+// by side: a first kernel forms every chunk's own state and summed step sizes, the second starts each chunk from
+// the states before it. Scratch: selective_scratch floats.
+long long selective_scratch(const SelectiveSpec& s, int n_seq, int max_q);
+void selective_scan(bool f32, const SelectiveSpec& s, const SelectiveInputs& in, const RaggedBatch& rb, int max_q,
+                    const float* dt, long long ld_dt, float* scratch, void* out, long long ldo, cudaStream_t stream);
+// One token per sequence. The pre-activations come from dt, or from the dt columns of `low` and w_dt [inner, ld_w].
+void selective_step(bool f32, const SelectiveSpec& s, const SelectiveInputs& in, const RaggedBatch& rb, const float* dt,
+                    long long ld_dt, const void* w_dt, long long ld_w, void* out, long long ldo, cudaStream_t stream);
+
 // out = rms_over_vdim(o) * gamma * act(gate)
 void head_norm_gate(bool f32, const RecurrentSpec& s, const float* o, const float* gamma, const void* gate,
                     long long ld_gate, void* out, long long ldo, int rows, cudaStream_t stream);

@@ -22,6 +22,7 @@ __device__ __forceinline__ float gate_act(const GateAct& a, float g, float u) {
   u = fminf(fmaxf(u, -a.limit), a.limit);
   return g * sigmoid_f(a.alpha * g) * (u + 1.f);
 }
+__device__ __forceinline__ float soft_cap_f(float y, float cap) { return cap * tanhf(y / cap); }
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }

@@ -4,6 +4,7 @@
 // norms), and the next sublayer reads the sum (through a norm of its own, or as it is), so one kernel
 // does post-norm, residual add and pre-norm of a row; for two mixers side by side it also normalises and
 // averages the two, and for routed experts it forms the weighted sum of their outputs.
+#include "api.h"
 #include "common.cuh"
 #include "hybrid_api.h"
 #include "hybrid_dev.cuh"
@@ -153,6 +154,12 @@ sandwich_norm_kernel(SublayerOut src, const float* __restrict__ w_post, float mu
 #pragma unroll
         for (int j = 0; j < V; ++j) a[j] = fmaf(s_weight[e], b[j], a[j]);
       }
+      if (y2) {
+        float b[V];
+        ldv<V>(y2 + t * src.ld + i, b);
+#pragma unroll
+        for (int j = 0; j < V; ++j) a[j] += b[j];
+      }
     } else {
       ldv<V>(y1 + i, a);
     }
@@ -206,94 +213,154 @@ sandwich_norm_kernel(SublayerOut src, const float* __restrict__ w_post, float mu
   write_normed<T, V>(row, sx, w_next, h + t * ldh, ldh, dim, eps);
 }
 
+// Cosine and sine of a position's turn: position x revolutions, reduced to a fraction of a turn in double precision.
+__device__ __forceinline__ float2 turn(int pos, double revolutions) {
+  const double a = pos * revolutions;
+  float sn, co;
+  sincospif(2.f * (float)(a - rint(a)), &sn, &co);
+  return make_float2(co, sn);
+}
+__device__ __forceinline__ float query_factor(const HeadPrep& p, int pos) {
+  return p.temp_coef == 0.f ? 1.f : 1.f + p.temp_coef * logf(floorf((float)(pos + 1) / p.temp_every) + 1.f);
+}
+
 // One warp per (token, head slot): slots [0, H) are q, [H, H + G) k, [H + G, H + 2 G) v.
 template <typename T>
-__global__ void qk_norm_append_kernel(const T* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
-                                      const float* __restrict__ q_gamma, const float* __restrict__ k_gamma,
-                                      RaggedBatch rb, const int* __restrict__ block_table, int table_stride,
-                                      int page_size, T* __restrict__ q_out, T* __restrict__ k_cache,
-                                      T* __restrict__ v_cache, int heads, int kv_heads, int dk, int dv, float eps) {
+__global__ void attn_prep_kernel(const T* __restrict__ proj, long long ld, HeadPrep p, RaggedBatch rb,
+                                 const int* __restrict__ block_table, int table_stride, int page_size, T* __restrict__ q_out,
+                                 T* __restrict__ k_cache, T* __restrict__ v_cache) {
   const int lane = threadIdx.x & 31;
-  const int slots = heads + 2 * kv_heads;
+  const int slots = p.heads + (p.k_off < 0 ? 0 : 2 * p.kv_heads);
   const long long w = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (w >= (long long)rb.rows * slots) return;
-  const int t = (int)(w / slots), hs = (int)(w % slots);
-  const T* src = proj + (long long)t * ld;
-  if (hs < heads + kv_heads) {
-    const bool is_q = hs < heads;
-    src += is_q ? q_off + hs * dk : k_off + (hs - heads) * dk;
-    const float* gamma = is_q ? q_gamma : k_gamma;
+  const int t = (int)(w / slots), hs = (int)(w % slots), pos = rb.pos[t];
+  const bool is_q = hs < p.heads, is_v = hs >= p.heads + p.kv_heads;
+  const int j = is_q ? hs : (is_v ? hs - p.heads - p.kv_heads : hs - p.heads), width = is_v ? p.dv : p.dk;
+  const T* src = proj + (long long)t * ld + (is_q ? p.q_off : (is_v ? p.v_off : p.k_off)) + j * width;
+  const float* bias = is_q ? p.q_bias : (is_v ? p.v_bias : p.k_bias);
+  if (bias) bias += j * width;
+  T* dst;
+  if (is_q) {
+    dst = q_out + ((long long)t * p.heads + j) * width;
+  } else {
+    const int page = block_table[(long long)rb.row_seq[t] * table_stride + pos / page_size];
+    if (page < 0) return;
+    dst = (is_v ? v_cache : k_cache) + (((long long)page * page_size + pos % page_size) * p.kv_heads + j) * width;
+  }
+  auto raw = [&](int i) { return ldf(src + i) + (bias ? bias[i] : 0.f); };
+  if (is_v) {
+    for (int i = lane; i < width; i += 32) stf(dst + i, raw(i));
+    return;
+  }
+  float r = 1.f;
+  if (p.norm_dim > 0) {
     float ss = 0.f;
-    for (int i = lane; i < dk; i += 32) {
-      const float v = ldf(src + i);
+    for (int i = lane; i < width; i += 32) {
+      const float v = raw(i);
       ss += v * v;
     }
-    ss = warp_sum(ss);
-    const float r = 1.f / sqrtf(ss / (float)dk + eps);
-    T* dst;
-    if (is_q) {
-      dst = q_out + ((long long)t * heads + hs) * dk;
-    } else {
-      const int p = rb.pos[t];
-      const int page = block_table[(long long)rb.row_seq[t] * table_stride + p / page_size];
-      if (page < 0) return;
-      dst = k_cache + (((long long)page * page_size + p % page_size) * kv_heads + (hs - heads)) * dk;
+    r = 1.f / sqrtf(warp_sum(ss) / (float)p.norm_dim + p.eps);
+  }
+  const float* gamma = is_q ? p.q_gamma : p.k_gamma;
+  auto normed = [&](int i) { return raw(i) * r * (gamma ? gamma[i] : 1.f); };
+  const float f = is_q ? query_factor(p, pos) : 1.f;
+  const int half = p.rot / 2;
+  for (int i = lane; i < width; i += 32) {
+    float x = normed(i);
+    if (i < p.rot) {
+      const float2 cs = turn(pos, p.turns[i < half ? i : i - half]);
+      x = i < half ? x * cs.x - normed(i + half) * cs.y : x * cs.x + normed(i - half) * cs.y;
     }
-    for (int i = lane; i < dk; i += 32) stf(dst + i, ldf(src + i) * r * gamma[i]);
-  } else {
-    const int g = hs - heads - kv_heads, p = rb.pos[t];
-    const int page = block_table[(long long)rb.row_seq[t] * table_stride + p / page_size];
-    if (page < 0) return;
-    src += v_off + g * dv;
-    T* dst = v_cache + (((long long)page * page_size + p % page_size) * kv_heads + g) * dv;
-    for (int i = lane; i < dv; i += 32) dst[i] = src[i];
+    stf(dst + i, x * f);
   }
 }
 
-// bf16 form for widths that are multiples of 8 up to 128: 16 lanes per (token, head slot), 16-byte accesses.
-__global__ void __launch_bounds__(256)
-qk_norm_append8_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
-                       const float* __restrict__ q_gamma, const float* __restrict__ k_gamma, RaggedBatch rb,
-                       const int* __restrict__ block_table, int table_stride, int page_size,
-                       __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_cache,
-                       __nv_bfloat16* __restrict__ v_cache, int heads, int kv_heads, int dk, int dv, float eps) {
-  const int l = threadIdx.x & 15, slots = heads + 2 * kv_heads;
-  const long long total = (long long)rb.rows * slots;
-  const long long stride = (long long)gridDim.x * (blockDim.x >> 4);
+// bf16 form for widths that are multiples of 8 up to 128: 16 lanes per (token, head slot), 16-byte accesses, `tokens`
+// tokens per block, whose angles are evaluated once for all heads.
+constexpr int AP_THREADS = 256;
+__global__ void __launch_bounds__(AP_THREADS)
+attn_prep8_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, HeadPrep p, RaggedBatch rb,
+                  const int* __restrict__ block_table, int table_stride, int page_size, int tokens,
+                  __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache) {
+  extern __shared__ float2 cs_all[];         // [tokens][rot / 2]
+  const int l = threadIdx.x & 15, slots = p.heads + (p.k_off < 0 ? 0 : 2 * p.kv_heads), half = p.rot / 2;
+  const int t0 = blockIdx.x * tokens, nt = min(tokens, rb.rows - t0);
+  if (half > 0) {
+    for (int i = threadIdx.x; i < nt * half; i += AP_THREADS) cs_all[i] = turn(rb.pos[t0 + i / half], p.turns[i % half]);
+    __syncthreads();
+  }
+  const int total = nt * slots;
   // both halves of a warp run the same number of iterations: the shuffles need the whole warp
-  for (long long w0 = ((long long)blockIdx.x * (blockDim.x >> 4) + (threadIdx.x >> 4)) & ~1ll; w0 < total; w0 += stride) {
-    const long long w = w0 + ((threadIdx.x >> 4) & 1);
+  for (int w0 = (threadIdx.x >> 4) & ~1; w0 < total; w0 += AP_THREADS >> 4) {
+    const int w = w0 + ((threadIdx.x >> 4) & 1);
     const bool live = w < total;
-    const int t = live ? (int)(w / slots) : 0, hs = live ? (int)(w % slots) : 0;
-    const bool is_q = hs < heads, is_v = hs >= heads + kv_heads;
-    const int width = is_v ? dv : dk, j = is_q ? hs : (is_v ? hs - heads - kv_heads : hs - heads);
-    const bool on = live && l * 8 < width;
-    bf16x8 raw;
+    const int tl = live ? w / slots : 0, hs = live ? w % slots : 0, t = t0 + tl;
+    const bool is_q = hs < p.heads, is_v = hs >= p.heads + p.kv_heads;
+    const int width = is_v ? p.dv : p.dk, j = is_q ? hs : (is_v ? hs - p.heads - p.kv_heads : hs - p.heads), c = l * 8;
+    const bool on = live && c < width;
+    const __nv_bfloat16* src = proj + (long long)t * ld + (is_q ? p.q_off : (is_v ? p.v_off : p.k_off)) + j * width;
+    const float* bias = is_q ? p.q_bias : (is_v ? p.v_bias : p.k_bias);
+    if (bias) bias += j * width;
+    const float* gamma = is_q ? p.q_gamma : p.k_gamma;
     float f[8];
     float ss = 0.f;
     if (on) {
-      raw = ldg8(proj, (long long)t * ld + (is_q ? q_off : (is_v ? v_off : k_off)) + j * width + l * 8);
-      unpack8(raw, f);
+      unpack8(ldg8(src, c), f);
+      if (bias) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] += bias[c + i];
+      }
 #pragma unroll
       for (int i = 0; i < 8; ++i) ss = fmaf(f[i], f[i], ss);
     }
 #pragma unroll
     for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if (!on) continue;
+    const int pos = rb.pos[t];
     if (!is_v) {
-      const float r = 1.f / sqrtf(ss / (float)dk + eps);
-      const float* gm = (is_q ? q_gamma : k_gamma) + l * 8;
+      const float r = p.norm_dim > 0 ? 1.f / sqrtf(ss / (float)p.norm_dim + p.eps) : 1.f;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] *= r * gm[i];
-      raw = pack8(f);
+      for (int i = 0; i < 8; ++i) f[i] *= gamma ? r * gamma[c + i] : r;
+      if (c < p.rot) {
+        // column i < half turns with i + half; the partner's value is read again
+        float g[8];
+        if (half % 8 == 0) {
+          const int at = c < half ? c + half : c - half;
+          unpack8(ldg8(src, at), g);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) g[i] = (g[i] + (bias ? bias[at + i] : 0.f)) * (gamma ? r * gamma[at + i] : r);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const int col = c + i;
+            if (col < p.rot) {
+              const int at = col < half ? col + half : col - half;
+              g[i] = (__bfloat162float(src[at]) + (bias ? bias[at] : 0.f)) * (gamma ? r * gamma[at] : r);
+            }
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int col = c + i;
+          if (col < p.rot) {
+            const float2 cs = cs_all[tl * half + (col < half ? col : col - half)];
+            f[i] = col < half ? f[i] * cs.x - g[i] * cs.y : f[i] * cs.x + g[i] * cs.y;
+          }
+        }
+      }
+      if (is_q && p.temp_coef != 0.f) {
+        const float q = query_factor(p, pos);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] *= q;
+      }
     }
+    const bf16x8 out = pack8(f);
     if (is_q) {
-      stg8(q_out, ((long long)t * heads + j) * dk + l * 8, raw);
+      stg8(q_out, ((long long)t * p.heads + j) * width + c, out);
     } else {
-      const int p = rb.pos[t];
-      const int page = block_table[(long long)rb.row_seq[t] * table_stride + p / page_size];
+      const int page = block_table[(long long)rb.row_seq[t] * table_stride + pos / page_size];
       if (page >= 0)
-        stg8(is_v ? v_cache : k_cache, (((long long)page * page_size + p % page_size) * kv_heads + j) * width + l * 8, raw);
+        stg8(is_v ? v_cache : k_cache, (((long long)page * page_size + pos % page_size) * p.kv_heads + j) * width + c, out);
     }
   }
 }
@@ -305,8 +372,7 @@ template <typename T, int ND>   // ND * 32 >= dv
 __global__ void __launch_bounds__(PA_WARPS * 32)
 paged_attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                       RaggedBatch rb, const int* __restrict__ block_table, int table_stride, int page_size,
-                      const T* __restrict__ gate, long long ld_gate, T* __restrict__ o, long long ldo, int heads,
-                      int kv_heads, int dk, int dv, float scale) {
+                      AttnExtras ex, T* __restrict__ o, long long ldo, int heads, int kv_heads, int dk, int dv, float scale) {
   extern __shared__ float sq_all[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long w = (long long)blockIdx.x * PA_WARPS + warp;
@@ -318,11 +384,11 @@ paged_attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
   for (int i = lane; i < dk; i += 32) sq[i] = ldf(q + ((long long)t * heads + h) * dk + i) * scale;
   __syncwarp();
   const int* bt = block_table + (long long)rb.row_seq[t] * table_stride;
-  const int n = rb.pos[t] + 1;
+  const int n = rb.pos[t] + 1, first = ex.window > 0 ? max(0, n - ex.window) : 0;
   float m = -INFINITY, l = 0.f, acc[ND];
 #pragma unroll
   for (int j = 0; j < ND; ++j) acc[j] = 0.f;
-  for (int j0 = 0; j0 < n; j0 += 32) {
+  for (int j0 = first; j0 < n; j0 += 32) {
     const int key = j0 + lane;
     float s = -INFINITY;
     long long tok = 0;
@@ -350,12 +416,17 @@ paged_attn_any_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, co
       }
     }
   }
-  float r = 1.f / l;
-  if (gate) r *= sigmoid_f(ldf(gate + (long long)t * ld_gate + h));
+  if (ex.sink) l += expf(ex.sink[h] - m);
+  float r = ex.out_scale / l;
+  const T* gate = ex.gate ? static_cast<const T*>(ex.gate) + (long long)t * ex.ld_gate : nullptr;
+  if (gate && !ex.gate_channels) r *= sigmoid_f(ldf(gate + h));
 #pragma unroll
   for (int j = 0; j < ND; ++j) {
     const int d = lane + 32 * j;
-    if (d < dv) stf(o + (long long)t * ldo + (long long)h * dv + d, acc[j] * r);
+    if (d >= dv) continue;
+    float y = acc[j] * r;
+    if (gate && ex.gate_channels) y *= sigmoid_f(ldf(gate + h * dv + d));
+    stf(o + (long long)t * ldo + (long long)h * dv + d, y);
   }
 }
 
@@ -435,6 +506,14 @@ __global__ void gelu_mul_kernel(T* __restrict__ y, long long ldy, const T* __res
   }
 }
 
+__global__ void soft_cap_kernel(float* __restrict__ y, long long ldy, long long rows, int width, float cap) {
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < rows * width;
+       i += (long long)gridDim.x * blockDim.x) {
+    float* p = y + i / width * ldy + i % width;
+    *p = soft_cap_f(*p, cap);
+  }
+}
+
 inline int grid_for(long long n, int threads, int per_sm) {
   long long g = (n + threads - 1) / threads;
   const long long cap = (long long)sm_count() * per_sm;
@@ -480,7 +559,7 @@ void embed_pos_norm(bool f32, const int* ids, const int* pos, const void* embed,
 void sandwich_norm(bool f32, const SublayerOut& y, const float* w_post, float mult, float* x, const float* w_next, void* h,
                    long long ldh, int rows, int dim, float eps, cudaStream_t stream) {
   MB_REQUIRE(dim > 0 && dim <= 12000 && ldh >= dim && y.ld >= dim, "sandwich_norm: row width out of range");
-  MB_REQUIRE(y.y2 == nullptr || (y.w1 && y.w2), "sandwich_norm: two inputs need their norm weights");
+  MB_REQUIRE(y.y2 == nullptr || y.row || (y.w1 && y.w2), "sandwich_norm: two inputs need their norm weights");
   MB_REQUIRE(y.row == nullptr || (y.weight && y.top > 0 && y.top <= SN_MAX_TOP), "sandwich_norm: at most 32 experts a token");
   if (rows == 0) return;
   const bool v4 = dim % 4 == 0 && ldh % 4 == 0 && y.ld % 4 == 0;
@@ -491,37 +570,42 @@ void sandwich_norm(bool f32, const SublayerOut& y, const float* w_post, float mu
   check_launch();
 }
 
-void qk_norm_append(bool f32, const void* proj, long long ld, int q_off, int k_off, int v_off, const float* q_gamma,
-                    const float* k_gamma, const RaggedBatch& rb, const int* block_table, int table_stride,
-                    int page_size, void* q_out, void* k_cache, void* v_cache, int heads, int kv_heads, int dk, int dv,
-                    float eps, cudaStream_t stream) {
+void attn_prep(bool f32, const void* proj, long long ld, const HeadPrep& p, const RaggedBatch& rb, const int* block_table,
+               int table_stride, int page_size, void* q_out, void* k_cache, void* v_cache, cudaStream_t stream) {
+  MB_REQUIRE(p.rot >= 0 && p.rot % 2 == 0 && p.rot <= p.dk && (p.rot == 0 || p.turns), "attn_prep: rotated columns");
+  MB_REQUIRE(p.temp_coef == 0.f || p.temp_every > 0.f, "attn_prep: query temperature");
   if (rb.rows == 0) return;
-  const int grid = ceil_div((long long)rb.rows * (heads + 2 * kv_heads), 8);
-  if (!f32 && dk % 8 == 0 && dv % 8 == 0 && dk <= 128 && dv <= 128 && ((ld | q_off | k_off | v_off) & 7) == 0) {
-    qk_norm_append8_kernel<<<grid_for((long long)rb.rows * (heads + 2 * kv_heads) * 16, 256, 16), 256, 0, stream>>>(
-        (const __nv_bfloat16*)proj, ld, q_off, k_off, v_off, q_gamma, k_gamma, rb, block_table, table_stride, page_size,
-        (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, heads, kv_heads, dk, dv, eps);
+  const int slots = p.heads + (p.k_off < 0 ? 0 : 2 * p.kv_heads);
+  const bool kv = p.k_off >= 0;
+  if (!f32 && p.dk % 8 == 0 && p.dv % 8 == 0 && p.dk <= 128 && p.dv <= 128 &&
+      ((ld | p.q_off | (kv ? p.k_off | p.v_off : 0)) & 7) == 0 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0) {
+    // enough head slots for a few rounds of a block's 16 groups, but no fewer blocks than SMs
+    int tokens = (64 + slots - 1) / slots;
+    const int most = rb.rows / (2 * sm_count());
+    if (tokens > most) tokens = most;
+    if (tokens < 1) tokens = 1;
+    attn_prep8_kernel<<<(rb.rows + tokens - 1) / tokens, AP_THREADS, tokens * (p.rot / 2) * 8, stream>>>(
+        (const __nv_bfloat16*)proj, ld, p, rb, block_table, table_stride, page_size, tokens, (__nv_bfloat16*)q_out,
+        (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache);
     count_launch();
     check_launch();
     return;
   }
+  const int grid = ceil_div((long long)rb.rows * slots, 8);
   if (f32)
-    qk_norm_append_kernel<float><<<grid, 256, 0, stream>>>(
-        (const float*)proj, ld, q_off, k_off, v_off, q_gamma, k_gamma, rb, block_table, table_stride, page_size,
-        (float*)q_out, (float*)k_cache, (float*)v_cache, heads, kv_heads, dk, dv, eps);
+    attn_prep_kernel<float><<<grid, 256, 0, stream>>>((const float*)proj, ld, p, rb, block_table, table_stride, page_size,
+                                                      (float*)q_out, (float*)k_cache, (float*)v_cache);
   else
-    qk_norm_append_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(
-        (const __nv_bfloat16*)proj, ld, q_off, k_off, v_off, q_gamma, k_gamma, rb, block_table, table_stride,
-        page_size, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, heads, kv_heads, dk, dv,
-        eps);
+    attn_prep_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)proj, ld, p, rb, block_table, table_stride,
+                                                              page_size, (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache,
+                                                              (__nv_bfloat16*)v_cache);
   count_launch();
   check_launch();
 }
 
 void paged_attn_any(bool f32, const void* q, const void* k_cache, const void* v_cache, const RaggedBatch& rb,
-                    const int* block_table, int table_stride, int page_size, const void* gate, long long ld_gate,
-                    void* o, long long ldo, int heads, int kv_heads, int dk, int dv, float scale,
-                    cudaStream_t stream) {
+                    const int* block_table, int table_stride, int page_size, const AttnExtras& ex, void* o, long long ldo,
+                    int heads, int kv_heads, int dk, int dv, float scale, cudaStream_t stream) {
   MB_REQUIRE(heads % kv_heads == 0, "paged_attn_any: heads must be a multiple of kv_heads");
   MB_REQUIRE(dk <= 1024 && dv <= 512, "paged_attn_any: head widths up to 1024 (keys) and 512 (values)");
   if (rb.rows == 0) return;
@@ -529,8 +613,8 @@ void paged_attn_any(bool f32, const void* q, const void* k_cache, const void* v_
   const int smem = PA_WARPS * dk * 4;
 #define MB_PA(T, ND)                                                                                              \
   paged_attn_any_kernel<T, ND><<<grid, PA_WARPS * 32, smem, stream>>>(                                            \
-      (const T*)q, (const T*)k_cache, (const T*)v_cache, rb, block_table, table_stride, page_size, (const T*)gate, \
-      ld_gate, (T*)o, ldo, heads, kv_heads, dk, dv, scale)
+      (const T*)q, (const T*)k_cache, (const T*)v_cache, rb, block_table, table_stride, page_size, ex, (T*)o, ldo, \
+      heads, kv_heads, dk, dv, scale)
   if (f32) {
     if (dv <= 64) MB_PA(float, 2); else if (dv <= 128) MB_PA(float, 4); else if (dv <= 256) MB_PA(float, 8);
     else MB_PA(float, 16);
@@ -576,6 +660,14 @@ void gelu_mul(bool f32, void* y, long long ldy, const void* table, long long ld_
   else
     gelu_mul_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((__nv_bfloat16*)y, ldy, (const __nv_bfloat16*)table, ld_table, ids,
                                                              vocab, rows, width);
+  count_launch();
+  check_launch();
+}
+
+void soft_cap(float* y, long long ldy, int rows, int width, float cap, cudaStream_t stream) {
+  MB_REQUIRE(cap > 0.f && ldy >= width, "soft_cap: arguments");
+  if (rows == 0 || width == 0) return;
+  soft_cap_kernel<<<grid_for((long long)rows * width, 256, 16), 256, 0, stream>>>(y, ldy, rows, width, cap);
   count_launch();
   check_launch();
 }

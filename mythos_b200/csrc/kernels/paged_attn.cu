@@ -110,13 +110,13 @@ __device__ __forceinline__ void unpack8_int8(uint2 w, float (&f)[8]) {
 // Merge `nstate` online-softmax states of a CTA (s_m/s_l: [nstate][gstride]; s_acc: state s at
 // s_acc + s * acc_stride, laid out [gstride][D]) for the G heads of one (sequence, kv head), publish the partial result of
 // this split, and let the last CTA of the (sequence, kv head) combine all splits into `out`. h0: first query
-// head of the group, cidx: its counter. With `gate`, head h is multiplied by sigmoid(gate[b, h]).
+// head of the group, cidx: its counter. dv: values of a head in `out` (at most D), whose rows are ldo apart.
 template <int D>
 __device__ __forceinline__ void merge_and_finish(const float* s_m, const float* s_l, const float* s_acc,
                                                  long long acc_stride, int nstate, int gstride, int G, int* s_last, float* __restrict__ scratch,
                                                  int* __restrict__ counters, __nv_bfloat16* __restrict__ out, int b,
-                                                 int h0, int cidx, int split, int heads, int splits,
-                                                 const __nv_bfloat16* __restrict__ gate = nullptr, long long ld_gate = 0) {
+                                                 int h0, int cidx, int split, int heads, int splits, int dv, long long ldo,
+                                                 const AttnExtras& ex) {
   const int stride = D + 2;
   for (int idx = threadIdx.x; idx < G * D; idx += blockDim.x) {
     const int g = idx / D, d = idx % D;
@@ -148,8 +148,10 @@ __device__ __forceinline__ void merge_and_finish(const float* s_m, const float* 
   __syncthreads();
   if (!*s_last) return;
   __threadfence();
+  const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(ex.gate);
   for (int idx = threadIdx.x; idx < G * D; idx += blockDim.x) {
     const int g = idx / D, d = idx % D;
+    if (d >= dv) continue;
     const float* base = scratch + ((long long)b * heads + h0 + g) * splits * stride;
     float M = -INFINITY;
     for (int s = 0; s < splits; ++s) M = fmaxf(M, base[s * stride + D]);
@@ -161,9 +163,13 @@ __device__ __forceinline__ void merge_and_finish(const float* s_m, const float* 
       L += w * base[s * stride + D + 1];
       A += w * base[s * stride + d];
     }
-    float y = L > 0.f ? A / L : 0.f;
-    if (gate) y /= 1.f + expf(-__bfloat162float(gate[b * ld_gate + h0 + g]));
-    out[((long long)b * heads + h0 + g) * D + d] = __float2bfloat16(y);
+    if (ex.sink) L += exp2f(ex.sink[h0 + g] * 1.4426950408889634f - M);
+    float y = L > 0.f ? A / L * ex.out_scale : 0.f;
+    if (gate) {
+      const __nv_bfloat16* gp = gate + b * ex.ld_gate;
+      y /= 1.f + expf(-__bfloat162float(ex.gate_channels ? gp[(h0 + g) * dv + d] : gp[h0 + g]));
+    }
+    out[b * ldo + (long long)(h0 + g) * dv + d] = __float2bfloat16(y);
   }
 }
 
@@ -284,7 +290,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
   }
   __syncthreads();
   merge_and_finish<D>(&s_m[0][0], &s_l[0][0], &s_acc[0][0][0], (long long)G * D, NSTATE, G, G, &s_last, scratch, counters, out, b, hkv * G,
-                      b * kv_heads + hkv, split, heads, splits);
+                      b * kv_heads + hkv, split, heads, splits, D, (long long)heads * D, AttnExtras{});
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -313,7 +319,7 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&a
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// DK: width of queries and keys, DV: width of values.
+// DK: width of queries and keys, DV: width of values, as multiples of 64 (narrower heads are filled with zeros by TMA).
 template <int DK, int DV = DK>
 struct PdSmem {
   static constexpr int CHUNKS = DK / 64, VCHUNKS = DV / 64;   // 64-dim boxes per K / V page
@@ -332,8 +338,8 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_c
                         const __nv_bfloat16* __restrict__ q, const int* __restrict__ block_table,
                         const int* __restrict__ context_lens, __nv_bfloat16* __restrict__ out,
                         float* __restrict__ scratch, int* __restrict__ counters, int heads, int kv_heads, int G,
-                        int max_pages, int splits, float scale_log2, long long q_tok_stride, const __nv_bfloat16* __restrict__ gate,
-                        long long ld_gate, int* status) {
+                        int max_pages, int splits, float scale_log2, long long q_tok_stride, int dk, int dv, long long ldo,
+                        const __grid_constant__ AttnExtras ex, int* status) {
   using S = PdSmem<DK, DV>;
   constexpr int KS = DK / 16;   // k-steps of Q K^T
   constexpr int NT = DV / 8;    // n-tiles of P V
@@ -360,9 +366,10 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_c
   __syncthreads();
 
   const int ctx = context_lens[b];
-  const int n_pages = (ctx + 15) >> 4;
-  const int per = (n_pages + splits - 1) / splits;
-  const int p0 = split * per, p1 = min(n_pages, p0 + per);
+  const int lo = ex.window > 0 ? max(0, ctx - ex.window) : 0;   // first visible token
+  const int first_page = lo >> 4, end_page = (ctx + 15) >> 4;
+  const int per = (end_page - first_page + splits - 1) / splits;
+  const int p0 = first_page + split * per, p1 = min(end_page, p0 + per);
   const int my_pages = (p1 - p0 - warp + 3) >> 2;   // pages p0 + warp, p0 + warp + 4, ... (<= 0: none)
   const int* bt = block_table + (long long)b * max_pages;
 
@@ -372,10 +379,10 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_c
     uint8_t* dst = wsm + st * S::STAGE;
     mbar_arrive_expect_tx(&full[st], S::STAGE);
 #pragma unroll
-    for (int c = 0; c < S::CHUNKS; ++c) tma_load_2d(dst + c * S::TILE, &tm_k, &full[st], hkv * DK + c * 64, page * 16);
+    for (int c = 0; c < S::CHUNKS; ++c) tma_load_3d(dst + c * S::TILE, &tm_k, &full[st], c * 64, hkv, page * 16);
 #pragma unroll
     for (int c = 0; c < S::VCHUNKS; ++c)
-      tma_load_2d(dst + (S::CHUNKS + c) * S::TILE, &tm_v, &full[st], hkv * DV + c * 64, page * 16);
+      tma_load_3d(dst + (S::CHUNKS + c) * S::TILE, &tm_v, &full[st], c * 64, hkv, page * 16);
   };
   if (lane == 0)
     for (int i = 0; i < PD_STAGES && i < my_pages; ++i) issue(i);
@@ -387,9 +394,9 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_c
   for (int ks = 0; ks < KS; ++ks) {
     qa[ks][0] = qa[ks][1] = qa[ks][2] = qa[ks][3] = 0u;
     if (r < Gs) {
-      const __nv_bfloat16* qp = q + (long long)b * q_tok_stride + (long long)(h0 + r) * DK + ks * 16 + 2 * t;
-      qa[ks][0] = *reinterpret_cast<const uint32_t*>(qp);
-      qa[ks][2] = *reinterpret_cast<const uint32_t*>(qp + 8);
+      const __nv_bfloat16* qp = q + (long long)b * q_tok_stride + (long long)(h0 + r) * dk + ks * 16 + 2 * t;
+      if (ks * 16 < dk) qa[ks][0] = *reinterpret_cast<const uint32_t*>(qp);        // dk is a multiple of 8
+      if (ks * 16 + 8 < dk) qa[ks][2] = *reinterpret_cast<const uint32_t*>(qp + 8);
     }
   }
   float o[NT][4];
@@ -428,7 +435,8 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_c
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const float v = (tok0 + j * 8 + e < ctx) ? sc[j][e] * scale_log2 : -INFINITY;
+        const int tok = tok0 + j * 8 + e;
+        const float v = (tok < ctx && tok >= lo) ? sc[j][e] * scale_log2 : -INFINITY;
         pv[j][e] = v;
         mx = fmaxf(mx, v);
       }
@@ -482,7 +490,7 @@ paged_decode_mma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_c
   }
   __syncthreads();
   merge_and_finish<DV>(s_m, s_l, reinterpret_cast<const float*>(smem), S::WARP_BYTES / 4, 4, 8, Gs, s_last, scratch, counters, out, b, h0,
-                       b * gridDim.y + blockIdx.y, split, heads, splits, gate, ld_gate);
+                       b * gridDim.y + blockIdx.y, split, heads, splits, dv, ldo, ex);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -710,7 +718,7 @@ paged_decode_mma_int8_kernel(const __grid_constant__ CUtensorMap tm_k, const __g
   }
   __syncthreads();
   merge_and_finish<D>(s_m, s_l, reinterpret_cast<const float*>(smem), S::WARP_BYTES / 4, 4, 8, G, s_last, scratch, counters, out, b, hkv * G,
-                      b * kv_heads + hkv, split, heads, splits);
+                      b * kv_heads + hkv, split, heads, splits, D, (long long)heads * D, AttnExtras{});
 }
 
 // One warp per output row; x staged in shared memory as fp32.
@@ -765,7 +773,7 @@ void paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, 
                        const int* context_lens, void* out, float* scratch, int* counters, int batch, int heads,
                        int kv_heads, int head_dim, int page_size, int max_pages, int cache_pages, int splits,
                        float scale, int* status, cudaStream_t stream, long long q_tok_stride, int v_head_dim,
-                       const void* gate, long long ld_gate) {
+                       const AttnExtras& ex, long long ldo) {
   const int dv = v_head_dim > 0 ? v_head_dim : head_dim;
   if (q_tok_stride <= 0) q_tok_stride = (long long)heads * head_dim;
   MB_REQUIRE(q_tok_stride % 8 == 0, "paged_attn_decode: query token stride must be a multiple of 8 elements");
@@ -775,13 +783,14 @@ void paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, 
   const int G = heads / kv_heads;
   const dim3 grid(batch, kv_heads, splits);
   const float sl2 = scale * 1.4426950408889634f;
-  if (page_size == 16 && (head_dim == 64 || head_dim == 128) && (dv == 64 || dv == 128)) {
-    // K / V cache as [cache_pages * 16 tokens, kv_heads * width]; one box = 16 tokens x 64 dims
+  if (ldo <= 0) ldo = (long long)heads * dv;
+  if (page_size == 16 && head_dim % 8 == 0 && dv % 8 == 0 && head_dim <= 128 && dv <= 128) {
+    // K / V cache as [cache_pages * 16 tokens, kv_heads, width]; one box = 16 tokens x 64 dims of one head
     auto page_map = [&](const void* base, int width) {
-      uint64_t dims[2] = {(uint64_t)kv_heads * width, (uint64_t)cache_pages * 16};
-      uint64_t strides[1] = {(uint64_t)kv_heads * width * 2};
-      uint32_t box[2] = {64, 16};
-      return make_tensor_map(base, TmaDType::BF16, 2, dims, strides, box, true);
+      uint64_t dims[3] = {(uint64_t)width, (uint64_t)kv_heads, (uint64_t)cache_pages * 16};
+      uint64_t strides[2] = {(uint64_t)width * 2, (uint64_t)kv_heads * width * 2};
+      uint32_t box[3] = {64, 1, 16};
+      return make_tensor_map(base, TmaDType::BF16, 3, dims, strides, box, true);
     };
     const CUtensorMap tk = page_map(k_cache, head_dim), tv = page_map(v_cache, dv);
     const dim3 mgrid(batch, kv_heads * ((G + 7) / 8), splits);
@@ -795,18 +804,19 @@ void paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, 
     }                                                                                                              \
     paged_decode_mma_kernel<DD, VV><<<mgrid, 128, PdSmem<DD, VV>::BYTES, stream>>>(                                \
         tk, tv, (const __nv_bfloat16*)q, block_table, context_lens, (__nv_bfloat16*)out, scratch, counters, heads, \
-        kv_heads, G, max_pages, splits, sl2, q_tok_stride, (const __nv_bfloat16*)gate, ld_gate, status);           \
+        kv_heads, G, max_pages, splits, sl2, q_tok_stride, head_dim, dv, ldo, ex, status);                         \
   } while (0)
-    if (head_dim == 128 && dv == 128) MB_PDM(128, 128);
-    else if (head_dim == 64 && dv == 128) MB_PDM(64, 128);
-    else if (head_dim == 128) MB_PDM(128, 64);
+    if (head_dim > 64 && dv > 64) MB_PDM(128, 128);
+    else if (dv > 64) MB_PDM(64, 128);
+    else if (head_dim > 64) MB_PDM(128, 64);
     else MB_PDM(64, 64);
 #undef MB_PDM
     count_launch();
     check_launch();
     return;
   }
-  MB_REQUIRE(dv == head_dim && gate == nullptr, "paged_attn_decode: unequal widths and gates need 16-token pages");
+  MB_REQUIRE(dv == head_dim && !ex.gate && !ex.sink && ex.window == 0 && ex.out_scale == 1.f && ldo == (long long)heads * dv,
+             "paged_attn_decode: unequal widths, gates, sinks and windows need 16-token pages");
 #define MB_PD(GG, DD)                                                                                         \
   paged_decode_kernel<GG, DD, false><<<grid, 128, 0, stream>>>(                                               \
       (const __nv_bfloat16*)q, k_cache, v_cache, nullptr, nullptr, block_table, context_lens,                 \

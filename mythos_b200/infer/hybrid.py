@@ -8,15 +8,21 @@ A pass takes a ragged batch (new tokens of several sequences, packed; prompts, p
 single decoded tokens in any mix). The residual stream is fp32; a sublayer reads its normalised copy in
 the engine's activation type. All projections of a mixer that read the same input are one GEMM. Per
 gated-linear-attention layer: projections -> decay GEMM -> recurrence -> head norm * gate -> output
-GEMM -> (post-norm + residual + next pre-norm). A parallel layer runs the delta-rule recurrence and
-paged attention side by side and averages their normalised outputs inside that last kernel.
+GEMM -> (post-norm + residual + next pre-norm). A parallel layer runs a recurrence and paged attention side by
+side: with norms of their own their outputs are averaged inside that last kernel, with constant scales both write
+into one row and share one output GEMM.
+
+Attention: one kernel turns the projection into queries and cached keys and values (bias, head norm, rotation,
+query temperature), one attends (window, sink, output gate). Heads are stored padded to a multiple of 8 columns. A
+layer that shares another's keys and values only forms queries. Selective scan: convolution -> GEMM to step sizes
+and input / read-out maps -> GEMM to the channels' step sizes -> scan with its output gate.
 
 Latent attention caches one row per token (latent | rotated key part) that all heads share. Tokens of
 sequences that bring few of them at once (decoding, short portions) attend in the latent's space: queries go
 through W_uk, the result through W_uv. Longer portions expand the latents of their sequence to keys and
 values once per pass and run the tensor-core prompt attention. A batch with both runs both. Routed experts:
-router GEMM -> selection and row segments -> row gather -> two grouped GEMMs -> (weighted sum + norm +
-residual).
+router GEMM -> selection and row segments -> row gather -> two grouped GEMMs -> (weighted sum + shared expert +
+norm + residual).
 
 ``dtype``: "bfloat16" (matrix products and activations in bf16 with 32-bit accumulation; residual,
 norms, decays, states and scores in 32-bit) or "float32" (everything in 32-bit).
@@ -27,7 +33,8 @@ import math
 
 import torch
 
-from ..models.hybrid_config import HybridConfig, LatentAttentionMixer, MoeFF, ParallelMixer, RecurrentMixer
+from ..models.hybrid_config import (AttentionMixer, HybridConfig, LatentAttentionMixer, MoeFF, ParallelMixer, RecurrentMixer,
+                                    SelectiveMixer)
 from ..ops import native
 from .engine import InferenceEngine
 from .kv_paged import PagedKVCache, RecurrentStatePool
@@ -37,6 +44,14 @@ DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.f
 
 def _pad8(n: int) -> int:
     return (n + 7) // 8 * 8
+
+
+def _pad_heads(w: torch.Tensor, heads: int) -> torch.Tensor:
+    """Rows (or values) of every head padded with zeros to a multiple of 8."""
+    width = w.shape[0] // heads
+    out = w.new_zeros(heads, _pad8(width), *w.shape[1:])
+    out[:, :width] = w.reshape(heads, width, *w.shape[1:])
+    return out.flatten(0, 1)
 
 
 class FusedProjection:
@@ -83,6 +98,7 @@ class _LatentSplit:
         self.short, self.short_seq, self.short_pos = short, short_seq, short_pos
 
 
+ACT_KINDS = {"silu": 0, "relu": 1, "clamped": 2}
 DECODE_GEMM_ROWS = 128     # up to this many tokens a product goes through the few-token GEMM
 EXPAND_TOKENS = 16         # portions of at least this many tokens expand the latents of their sequence
 EXPAND_BYTES = 4 << 30     # unless the expanded keys and values would need more than this
@@ -119,7 +135,8 @@ class HybridEngine(InferenceEngine):
         shapes = []                # per caching layer; a latent layer's rows are keys and values at once
         for s in cfg.layers:
             if s.attention is not None:
-                shapes.append((s.attention.kv_heads, s.attention.dim, s.attention.vdim))
+                if s.attention.kv_from is None:
+                    shapes.append((s.attention.kv_heads, _pad8(s.attention.dim), _pad8(s.attention.vdim)))
             elif s.latent is not None:
                 shapes.append((1, _pad8(s.latent.kv_rank) + _pad8(s.latent.rot_dim), 0))
         self.cache = PagedKVCache(len(shapes), 0, 0, kv_pages or max_batch * pages_per_seq, page_size, max_batch,
@@ -161,34 +178,51 @@ class HybridEngine(InferenceEngine):
     def _vector(self, w: torch.Tensor) -> torch.Tensor:
         return w.to(device=self.device, dtype=torch.float32).contiguous()
 
+    def _norm(self, w: torch.Tensor) -> torch.Tensor:
+        return self._vector(w) + self.cfg.norm_offset
+
     def _pack(self, model) -> None:
         t = model.tensor
         cfg = self.cfg
         self.embed_table = t("embed").to(self.device, self.dtype).contiguous()
         self.pos_table = t("pos").to(self.device, self.dtype).contiguous() if cfg.position_table else None
         self.side_table = t("side.embed").to(self.device, self.dtype).contiguous() if cfg.token_side else None
-        self.final_norm = self._vector(t("final.norm"))
-        self.head = self._matrix(t("head"))
-        n_att = 0
+        self.final_norm = self._norm(t("final.norm"))
+        if not cfg.tied_head:
+            self.head = self._matrix(t("head"))
+        else:
+            self.head = self.embed_table if cfg.hidden_size % 8 == 0 else self._matrix(self.embed_table)
+        pages_of = {}                                 # layer -> its entry of the cache
+        for i, spec in enumerate(cfg.layers):
+            share = spec.attention.kv_from if spec.attention is not None else None
+            if share is not None:
+                pages_of[i] = pages_of[share]
+            elif spec.attention is not None or spec.latent is not None:
+                pages_of[i] = len(set(pages_of.values()))
 
         def norms(p: str, n: int) -> _Sublayer:
             if cfg.pre_norm:
-                return _Sublayer(self._vector(t(p + f"norm{n}")), self._vector(t(p + f"norm{n}b")))
-            return _Sublayer(None, self._vector(t(p + f"norm{n}")))
+                return _Sublayer(self._norm(t(p + f"norm{n}")), self._norm(t(p + f"norm{n}b")))
+            return _Sublayer(None, self._norm(t(p + f"norm{n}")))
 
         for i, spec in enumerate(cfg.layers):
             p = f"l{i}."
             L = _HybridLayer()
             L.spec = spec
             L.norms = norms(p, 1)
-            if isinstance(spec.mixer, ParallelMixer):
-                L.run, L.att_index = self._parallel, n_att
+            L.att_index = pages_of.get(i, 0)
+            if isinstance(spec.mixer, ParallelMixer) and isinstance(spec.mixer.right, SelectiveMixer):
+                L.run = self._parallel_selective
+                self._pack_parallel_selective(L, t, p + "mix.")
+            elif isinstance(spec.mixer, ParallelMixer):
+                L.run = self._parallel
                 self._pack_parallel(L, t, p + "mix.")
-                n_att += 1
+            elif isinstance(spec.mixer, AttentionMixer):
+                L.run = self._attention_layer
+                self._pack_attention(L, t, p + "mix.")
             elif isinstance(spec.mixer, LatentAttentionMixer):
-                L.run, L.att_index = self._latent, n_att
+                L.run = self._latent
                 self._pack_latent(L, t, p + "mix.")
-                n_att += 1
             else:
                 L.run = self._gla
                 self._pack_gla(L, t, p + "mix.")
@@ -197,9 +231,8 @@ class HybridEngine(InferenceEngine):
                 if isinstance(spec.mlp, MoeFF):
                     self._pack_experts(L, t, p + "mlp.")
                 else:
-                    L.act = ({"silu": 0, "relu": 1}[spec.mlp.act], 0.0, 0.0)
-                    L.gate_up = FusedProjection([("gate", t(p + "mlp.gate")), ("up", t(p + "mlp.up"))], self.dtype, self.device)
-                    L.down = self._matrix(t(p + "mlp.down"))
+                    L.act = (ACT_KINDS[spec.mlp.act], 0.0, 0.0)
+                    self._pack_gated(L, t, p + "mlp.")
             if cfg.token_side:
                 n = cfg.token_side
                 L.side_gate, L.side_proj = self._matrix(t(p + "side.gate")), self._matrix(t(p + "side.proj"))
@@ -229,15 +262,81 @@ class HybridEngine(InferenceEngine):
                                 {"z_bias": self._vector(t(p + "a2.b")), "gamma": self._vector(t(p + "norm")), "a2": L.a2})
         L.out = self._matrix(t(p + "o"))
 
+    # ---- attention: projection parts under a prefix, then the kernel-side object over their offsets
+    def _attention_parts(self, m: AttentionMixer, t, p: str, prefix: str = "") -> list:
+        parts = [("q", m.heads)] + ([("k", m.kv_heads), ("v", m.kv_heads)] if m.kv_from is None else [])
+        parts = [(prefix + n, _pad_heads(t(p + n), heads)) for n, heads in parts]
+        if m.gate is not None:
+            parts.append((prefix + "g", _pad_heads(t(p + "g"), m.heads) if m.gate == "channel" else t(p + "g")))
+        return parts
+
+    def _attention_object(self, m: AttentionMixer, t, p: str, off: dict, prefix: str = "", out_scale: float = 1.0):
+        own = m.kv_from is None
+        spec = {"heads": m.heads, "kv_heads": m.kv_heads, "dk": _pad8(m.dim), "dv": _pad8(m.vdim), "q_off": off[prefix + "q"],
+                "scale": m.scale, "out_scale": out_scale, "window": m.window, "gate_channels": int(m.gate == "channel"),
+                "norm_dim": m.dim if m.qk_norm else 0, "eps": self.cfg.norm_eps}
+        if own:
+            spec.update(k_off=off[prefix + "k"], v_off=off[prefix + "v"])
+        tensors = {}
+        if m.bias:
+            for n, heads in [("q", m.heads)] + ([("k", m.kv_heads), ("v", m.kv_heads)] if own else []):
+                tensors[n + "_bias"] = self._vector(_pad_heads(t(p + n + ".b"), heads))
+        if m.qk_norm == "weighted":
+            for n in ("q", "k") if own else ("q",):
+                tensors[n + "_gamma"] = self._vector(_pad_heads(t(p + n + ".norm"), 1))
+        if m.sink:
+            tensors["sink"] = self._vector(t(p + "sink"))
+        if m.rotation is not None:
+            spec["rot"] = m.rotation.dims
+            tensors["turns"] = torch.tensor(m.rotation.turns(), dtype=torch.float64, device=self.device)
+        if m.q_temp is not None:
+            spec.update(temp_coef=m.q_temp.coef, temp_every=m.q_temp.every)
+        return self.H.Attention(spec, tensors)
+
+    @staticmethod
+    def _attention_out(m: AttentionMixer, w: torch.Tensor) -> torch.Tensor:
+        """Output matrix over padded value heads."""
+        return _pad_heads(w.t(), m.heads).t()
+
+    def _pack_attention(self, L, t, p: str) -> None:
+        m = L.spec.attention
+        L.proj = FusedProjection(self._attention_parts(m, t, p), self.dtype, self.device)
+        L.att = self._attention_object(m, t, p, L.proj.off)
+        L.out = self._matrix(self._attention_out(m, t(p + "o")))
+
+    def _pack_parallel_selective(self, L, t, p: str) -> None:
+        """Both mixers project from one GEMM and write their scaled outputs side by side for another."""
+        a, r = L.spec.mixer.left, L.spec.mixer.right
+        scale_l, scale_r = L.spec.mixer.scales
+        left, right = p + "left.", p + "right."
+        w_in, w_x = t(right + "in"), t(right + "x")
+        L.proj = FusedProjection(self._attention_parts(a, t, left, "l") + [("rx", w_in[: r.inner]), ("rz", w_in[r.inner:])],
+                                 self.dtype, self.device)
+        L.att = self._attention_object(a, t, left, L.proj.off, "l", scale_l)
+        n, k = r.state, r.dt_rank
+        L.x_maps = FusedProjection([("dt", w_x[:k]), ("B", w_x[k:k + n]), ("C", w_x[k + n:])], self.dtype, self.device)
+        L.w_dt = self._matrix(t(right + "dt"))
+        padded = self.H.selective_padded_state(n)
+        decay = torch.zeros(r.inner, padded, dtype=torch.float64)
+        decay[:, :n] = -torch.exp(t(right + "A_log").double().cpu()) / math.log(2.0)
+        tensors = {"conv_w": self._vector(t(right + "conv").t()), "conv_b": self._vector(t(right + "conv.b")),
+                   "a": self._vector(decay), "d": self._vector(t(right + "D")), "dt_b": self._vector(t(right + "dt.b")),
+                   "w_dt": L.w_dt, "state": self.states.add(r.inner, padded)}
+        if r.conv > 1:
+            tensors["conv_state"] = self.states.add(r.conv - 1, r.inner)
+        L.sel = self.H.Selective({"inner": r.inner, "state": n, "rank": k, "taps": r.conv, "out_scale": scale_r,
+                                  "x_off": L.proj.off["rx"], "z_off": L.proj.off["rz"], "b_off": L.x_maps.off["B"],
+                                  "c_off": L.x_maps.off["C"]}, tensors)
+        L.out = self._matrix(torch.cat([self._attention_out(a, t(left + "o")), t(right + "o")], 1))
+
     def _pack_parallel(self, L, t, p: str) -> None:
         a, r = L.spec.mixer.left, L.spec.mixer.right
         left, right = p + "left.", p + "right."
-        L.proj = FusedProjection(
-            [("lq", t(left + "q")), ("lk", t(left + "k")), ("lv", t(left + "v")), ("lg", t(left + "g"))]
-            + [("r" + n, t(right + n)) for n in ("q", "k", "v", "b", "a1", "g1")], self.dtype, self.device)
-        L.q_gamma, L.k_gamma = self._vector(t(left + "q.norm")), self._vector(t(left + "k.norm"))
-        L.left_out, L.right_out = self._matrix(t(left + "o")), self._matrix(t(right + "o"))
-        L.left_norm, L.right_norm = self._vector(t(left + "out")), self._vector(t(right + "out"))
+        L.proj = FusedProjection(self._attention_parts(a, t, left, "l")
+                                 + [("r" + n, t(right + n)) for n in ("q", "k", "v", "b", "a1", "g1")], self.dtype, self.device)
+        L.att = self._attention_object(a, t, left, L.proj.off, "l")
+        L.left_out, L.right_out = self._matrix(self._attention_out(a, t(left + "o"))), self._matrix(t(right + "o"))
+        L.left_norm, L.right_norm = self._norm(t(left + "out")), self._norm(t(right + "out"))
         L.a2, L.rank = self._matrix(t(right + "a2")), _pad8(t(right + "a1").shape[0])
         L.g2, L.g_rank = self._matrix(t(right + "g2")), _pad8(t(right + "g1").shape[0])
         off = L.proj.off
@@ -284,12 +383,19 @@ class HybridEngine(InferenceEngine):
         w[:, :, :dv] = out.view(-1, H, dv)
         L.out = self._matrix(w.view(-1, H * dv_p))
 
+    def _pack_gated(self, L, t, p: str) -> None:
+        L.gate_up = FusedProjection([("gate", t(p + "gate")), ("up", t(p + "up"))], self.dtype, self.device)
+        L.down = self._matrix(t(p + "down"))
+
     def _pack_experts(self, L, t, p: str) -> None:
         """Gate and up rows of an expert in one matrix [2 * ff, d], all experts stacked; ff padded to a multiple of 8."""
         m, d = L.spec.mlp, self.cfg.hidden_size
         f = _pad8(m.ff)
-        L.act = (2, m.limit, m.alpha)
-        L.router, L.correction = self._matrix(t(p + "router")), self._vector(t(p + "correction"))
+        L.act = (ACT_KINDS[m.act], m.limit, m.alpha)
+        L.router, L.correction = self._matrix(t(p + "router")), self._vector(t(p + "correction")) if m.correction else None
+        L.rule = (int(m.score == "sigmoid"), m.group_best, int(m.normalise), m.scale)
+        if m.shared:
+            self._pack_gated(L, t, p + "shared.")
         L.w_in = torch.zeros(m.experts, 2 * f, _pad8(d), dtype=self.dtype, device=self.device)
         L.w_out = torch.zeros(m.experts, _pad8(d), f, dtype=self.dtype, device=self.device)
         for e in range(m.experts):
@@ -298,11 +404,11 @@ class HybridEngine(InferenceEngine):
             L.w_out[e, :d, : m.ff] = t(p + f"e{e}.down").to(self.device, self.dtype)
 
     def weight_bytes(self) -> int:
-        tables = (self.embed_table, self.pos_table, self.side_table, self.head)
+        tables = (self.embed_table, self.pos_table, self.side_table, self.head if self.head is not self.embed_table else None)
         n = sum(x.numel() * x.element_size() for x in tables if x is not None)
         for L in self.layers:
             mats = [L.proj.weight, L.a2, L.g2, L.out, L.left_out, L.right_out, L.down, L.uk_t, L.uv, L.router, L.w_in, L.w_out,
-                    L.side_gate, L.side_proj, L.gate_up.weight if L.gate_up is not None else None]
+                    L.side_gate, L.side_proj, L.w_dt] + [f.weight for f in (L.gate_up, L.x_maps) if f is not None]
             n += sum(x.numel() * x.element_size() for x in mats if x is not None)
         return n
 
@@ -310,13 +416,16 @@ class HybridEngine(InferenceEngine):
     def _new(self, rows: int, cols: int, dtype=None) -> torch.Tensor:
         return torch.empty(rows, cols, device=self.device, dtype=dtype or self.dtype)
 
-    def _gemm(self, x, w, out=None, dtype=None, alpha: float = 1.0):
+    def _gemm(self, x, w, out=None, dtype=None, alpha: float = 1.0, cap: float = 0.0):
+        """alpha * x w^T; with ``cap`` (fp32 results) the soft-capped product."""
         if out is None:
             out = self._new(x.shape[0], w.shape[0], dtype)
         if self._fast and x.shape[0] <= DECODE_GEMM_ROWS:
-            self.H.gemm_decode(x, w, out, 0, 0, alpha, self._status)
+            self.H.gemm_decode(x, w, out, 0, 0, alpha, self._status, cap=cap)
         else:
             self.H.gemm_nt(x, w, out, alpha, self._status)
+            if cap > 0.0:
+                self.H.soft_cap(out, cap)
         return out
 
     @property
@@ -355,35 +464,64 @@ class HybridEngine(InferenceEngine):
         y = self._recurrence(L, proj, off["a1"], proj[:, off["g"]:], 0, ctx)
         return self._gemm(y, L.out), None
 
-    def _attention(self, L, proj, ctx):
-        """Left mixer of a parallel layer up to its output projection."""
-        m, off, li = L.spec.attention, L.proj.off, L.att_index
-        kc, vc = self.cache.k[li], self.cache.v[li]
-        q = torch.empty(ctx.rows, m.heads, m.dim, device=self.device, dtype=self.dtype)
-        self.H.qk_norm_append(proj, off["lq"], off["lk"], off["lv"], L.q_gamma, L.k_gamma, ctx.batch, ctx.table, q, kc, vc,
-                              self.cfg.norm_eps)
-        width = m.heads * m.vdim
-        o = self._new(ctx.rows, _pad8(width))
-        if o.shape[1] != width:
-            o[:, width:].zero_()
-        gate = proj[:, off["lg"]:off["lg"] + m.heads]
-        if not (self._fast and self.page_size == 16 and m.dim in (64, 128) and m.vdim in (64, 128)):
-            self.H.paged_attn_any(q, kc, vc, ctx.batch, ctx.table, gate, o, m.scale)
+    def _attention(self, L, proj, ctx, prefix: str = "", out=None):
+        """Attention up to its output projection -> [rows, heads * padded value width]."""
+        m, att = L.spec.attention, L.att
+        kc, vc = self.cache.k[L.att_index], self.cache.v[L.att_index]
+        dk, dv = kc.shape[3], vc.shape[3]
+        q = torch.empty(ctx.rows, m.heads, dk, device=self.device, dtype=self.dtype)
+        att.prep(proj, ctx.batch, ctx.table, q, kc, vc)
+        o = self._new(ctx.rows, m.heads * dv) if out is None else out
+        gate = None
+        if m.gate is not None:
+            g = L.proj.off[prefix + "g"]
+            gate = proj[:, g:g + m.heads * (dv if m.gate == "channel" else 1)]
+        if not (self._fast and att.tensor_ok(self.page_size)):
+            att.any(q, kc, vc, ctx.batch, ctx.table, gate, o)
         elif ctx.decode:
+            keys = min(ctx.max_kv, m.window + self.page_size) if m.window else ctx.max_kv
             pairs = ctx.n_seq * m.kv_heads * ((m.heads // m.kv_heads + 7) // 8)
-            splits = max(1, min(32, (6 * self._sms + pairs - 1) // pairs, (ctx.max_kv + 255) // 256))
-            scratch = torch.empty(ctx.rows * m.heads * splits * (m.vdim + 2), device=self.device, dtype=torch.float32)
-            self.H.paged_attn_decode(q, kc, vc, ctx.batch, ctx.table, gate, o, scratch, self._counters, splits, m.scale,
-                                     self._status)
+            splits = max(1, min(32, (6 * self._sms + pairs - 1) // pairs, (keys + 255) // 256))
+            scratch = torch.empty(att.decode_scratch(ctx.rows, splits), device=self.device, dtype=torch.float32)
+            att.decode(q, kc, vc, ctx.batch, ctx.table, gate, o, scratch, self._counters, splits, self._status)
         else:
-            self.H.paged_attn_prefill(q, kc, vc, ctx.batch, ctx.table, gate, o, ctx.max_q, m.scale, self._status)
+            att.prefill(q, kc, vc, ctx.batch, ctx.table, gate, o, ctx.max_q, self._status)
         return o
+
+    def _attention_layer(self, L, h, ctx):
+        return self._gemm(self._attention(L, self._gemm(h, L.proj.weight), ctx), L.out), None
+
+    def _selective(self, L, proj, ctx, out):
+        """Selective scan of a layer over the batch with its output gate -> out [rows, padded channels]."""
+        m, sel = L.spec.recurrent, L.sel
+        one = ctx.decode and self.tensor_kernels
+        x = self._new(ctx.rows, _pad8(m.inner))
+        sel.conv(proj, ctx.batch, one, x)
+        low = self._gemm(x, L.x_maps.weight)
+        dt = None
+        if not (one and ctx.rows <= LOW_RANK_FUSE_ROWS):
+            dt = self._gemm(low[:, : L.w_dt.shape[1]], L.w_dt, dtype=torch.float32)
+        if out.shape[1] != m.inner:
+            out[:, m.inner:].zero_()
+        if one:
+            sel.step(proj, x, low, dt, ctx.batch, out)
+        else:
+            scratch = torch.empty(sel.scratch_floats(ctx.n_seq, ctx.max_q), device=self.device, dtype=torch.float32)
+            sel.scan(proj, x, low, dt, ctx.batch, ctx.max_q, scratch, out)
+
+    def _parallel_selective(self, L, h, ctx):
+        proj = self._gemm(h, L.proj.weight)
+        y = self._new(ctx.rows, L.out.shape[1])
+        n = L.spec.attention.heads * self.cache.v[L.att_index].shape[3]
+        self._attention(L, proj, ctx, "l", y[:, :n])
+        self._selective(L, proj, ctx, y[:, n:])
+        return self._gemm(y, L.out), None
 
     def _parallel(self, L, h, ctx):
         off = L.proj.off
         proj = self._gemm(h, L.proj.weight)
         y_right = self._gemm(self._recurrence(L, proj, off["ra1"], None, off["rg1"], ctx), L.right_out)
-        y_left = self._gemm(self._attention(L, proj, ctx), L.left_out)
+        y_left = self._gemm(self._attention(L, proj, ctx, "l"), L.left_out)
         return y_left, y_right
 
     # ---- latent attention
@@ -441,7 +579,8 @@ class HybridEngine(InferenceEngine):
         return 128 if mean >= SEGMENT_GEMM_ROWS else max(16, min(64, 1 << (2 * mean).bit_length()))
 
     def _experts(self, L, h, ctx):
-        """Outputs of the chosen experts [rows * top, d], where each (token, choice) lies and its weight."""
+        """Outputs of the chosen experts [rows * top, d], of the shared expert, where each (token, choice) lies and its
+        weight."""
         m, T, C = L.spec.mlp, ctx.rows, self.H
         z = self._gemm(h, L.router, dtype=torch.float32)
         pairs, tile = T * m.top, self._expert_tile(T, m)
@@ -452,7 +591,7 @@ class HybridEngine(InferenceEngine):
         tiles = torch.empty(min(pairs, m.experts + pairs // tile), 3, **i32)
         route = (m.experts, m.top, m.groups, m.keep)
         plan = (idx, weight, slot, self._expert_counts[: m.experts + 1], offset, tiles, count)
-        C.expert_select(z, L.correction, route, tile, *plan)
+        C.expert_select(z, L.correction, route, tile, *plan, L.rule)
         d_p, f = L.w_in.shape[2], L.w_out.shape[2]
         x = self._new(pairs, d_p)
         C.expert_gather(h, route, *plan, x, row)
@@ -464,20 +603,26 @@ class HybridEngine(InferenceEngine):
         else:
             C.gemm_tiles(x, L.w_in, a, tiles, count, tile, f, f, L.act, self._status)
         C.gemm_tiles(a, L.w_out, y, tiles, count, tile, 0, 0, L.act, self._status)
-        return y, row, weight
+        shared = None
+        if m.shared:
+            shared = self._new(T, d_p)
+            self._gated(L, m.shared, h, ctx, shared[:, : self.cfg.hidden_size])
+        return y, shared, row, weight
 
-    def _feed_forward(self, L, h, ctx):
-        f = L.spec.mlp.ff
+    def _gated(self, L, f: int, h, ctx, out=None):
+        """Gated feed-forward of width ``f`` for every token."""
         a = self._new(ctx.rows, L.down.shape[1])
         if self._fast and f % 8 == 0 and ctx.rows <= DECODE_GEMM_ROWS:
             self.H.gemm_decode(h, L.gate_up.weight, a, f, L.gate_up.off["up"], 1.0, self._status, L.act)
-            return self._gemm(a, L.down)
-        if self._fast and L.act[0] == 0 and f % 128 == 0 and ctx.rows >= 256:
+        elif self._fast and L.act[0] == 0 and f % 128 == 0 and ctx.rows >= 256:
             self.H.gemm_swiglu(h, L.gate_up.weight, a, self._status)
-            return self._gemm(a, L.down)
-        gu = self._gemm(h, L.gate_up.weight)
-        self.H.gate_pair(gu, f, L.gate_up.off["up"], L.act, a)
-        return self._gemm(a, L.down)
+        else:
+            gu = self._gemm(h, L.gate_up.weight)
+            self.H.gate_pair(gu, f, L.gate_up.off["up"], L.act, a)
+        return self._gemm(a, L.down, out)
+
+    def _feed_forward(self, L, h, ctx):
+        return self._gated(L, L.spec.mlp.ff, h, ctx)
 
     def _token_side(self, L, h, ctx):
         """proj(gelu(gate x) * side embedding of the token)"""
@@ -566,12 +711,13 @@ class HybridEngine(InferenceEngine):
             full = torch.zeros(h.shape[0], self.head.shape[1], device=self.device, dtype=self.dtype)
             full[:, : h.shape[1]] = h
             h = full
-        return self._gemm(h, self.head, dtype=torch.float32, alpha=self.cfg.logit_scale)
+        return self._gemm(h, self.head, dtype=torch.float32, alpha=self.cfg.logit_scale, cap=self.cfg.logit_softcap)
 
 
 class _HybridLayer:
     spec = norms = ff_norms = proj = a2 = g2 = out = left_out = right_out = left_norm = right_norm = rec = None
-    gate_up = down = act = router = correction = w_in = w_out = None
+    att = sel = x_maps = w_dt = None
+    gate_up = down = act = router = correction = rule = w_in = w_out = None
     lat = uk_t = uv = expand = run = None
     side_gate = side_proj = side_embed = side_norms = None
     rank = g_rank = att_index = 0

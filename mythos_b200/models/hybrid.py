@@ -11,12 +11,31 @@ import torch
 import torch.nn as nn
 
 from .hybrid_config import (AttentionMixer, HybridConfig, LatentAttentionMixer, MoeFF, ParallelMixer,
-                            RecurrentMixer)
+                            RecurrentMixer, SelectiveMixer)
 
 
 def _attention_shapes(p: str, m: AttentionMixer, d: int) -> dict:
-    return {p + "q": (m.heads * m.dim, d), p + "k": (m.kv_heads * m.dim, d), p + "v": (m.kv_heads * m.vdim, d),
-            p + "q.norm": (m.dim,), p + "k.norm": (m.dim,), p + "g": (m.heads, d), p + "o": (d, m.heads * m.vdim)}
+    out = {p + "q": (m.heads * m.dim, d)}
+    if m.kv_from is None:
+        out.update({p + "k": (m.kv_heads * m.dim, d), p + "v": (m.kv_heads * m.vdim, d)})
+    if m.bias:
+        out.update({name + ".b": shape[:1] for name, shape in out.items()})
+    if m.qk_norm == "weighted":
+        out[p + "q.norm"] = (m.dim,)
+        if m.kv_from is None:
+            out[p + "k.norm"] = (m.dim,)
+    if m.gate is not None:
+        out[p + "g"] = (m.heads * (m.vdim if m.gate == "channel" else 1), d)
+    if m.sink:
+        out[p + "sink"] = (m.heads,)
+    out[p + "o"] = (d, m.heads * m.vdim)
+    return out
+
+
+def _selective_shapes(p: str, m: SelectiveMixer, d: int) -> dict:
+    c = m.inner
+    return {p + "in": (2 * c, d), p + "conv": (c, m.conv), p + "conv.b": (c,), p + "x": (m.dt_rank + 2 * m.state, c),
+            p + "dt": (c, m.dt_rank), p + "dt.b": (c,), p + "A_log": (c, m.state), p + "D": (c,), p + "o": (d, c)}
 
 
 def _gla_shapes(p: str, m: RecurrentMixer, d: int) -> dict:
@@ -47,7 +66,11 @@ def _gated_shapes(p: str, ff: int, d: int) -> dict:
 def _mlp_shapes(p: str, f, d: int) -> dict:
     if not isinstance(f, MoeFF):
         return _gated_shapes(p, f.ff, d)
-    out = {p + "router": (f.experts, d), p + "correction": (f.experts,)}
+    out = {p + "router": (f.experts, d)}
+    if f.correction:
+        out[p + "correction"] = (f.experts,)
+    if f.shared:
+        out.update(_gated_shapes(p + "shared.", f.shared, d))
     for e in range(f.experts):
         out.update(_gated_shapes(p + f"e{e}.", f.ff, d))
     return out
@@ -59,7 +82,9 @@ def expected_shapes(cfg: HybridConfig) -> dict:
     out = {"embed": (cfg.vocab_size, d)}
     if cfg.position_table:
         out["pos"] = (cfg.max_seq_len, d)
-    out.update({"final.norm": (d,), "head": (cfg.vocab_size, d)})
+    out["final.norm"] = (d,)
+    if not cfg.tied_head:
+        out["head"] = (cfg.vocab_size, d)
     if cfg.token_side:
         out["side.embed"] = (cfg.vocab_size, cfg.num_layers * cfg.token_side)
 
@@ -73,9 +98,13 @@ def expected_shapes(cfg: HybridConfig) -> dict:
         norms(p, 1)
         m = spec.mixer
         if isinstance(m, ParallelMixer):
+            right = _selective_shapes if isinstance(m.right, SelectiveMixer) else _delta_shapes
             out.update(_attention_shapes(p + "mix.left.", m.left, d))
-            out.update(_delta_shapes(p + "mix.right.", m.right, d))
-            out[p + "mix.left.out"] = out[p + "mix.right.out"] = (d,)
+            out.update(right(p + "mix.right.", m.right, d))
+            if m.scales is None:
+                out[p + "mix.left.out"] = out[p + "mix.right.out"] = (d,)
+        elif isinstance(m, AttentionMixer):
+            out.update(_attention_shapes(p + "mix.", m, d))
         elif isinstance(m, LatentAttentionMixer):
             out.update(_latent_shapes(p + "mix.", m, d))
         else:
@@ -121,7 +150,15 @@ class HybridModel(nn.Module):
             shape = tuple(low_rank if n is None else n for n in shape)
             leaf = name.rsplit(".", 1)[-1]
             if leaf in ("norm", "norm1", "norm2", "norm1b", "norm2b", "out"):
+                t = torch.full(shape, 1.0 - cfg.norm_offset, device=device)
+            elif leaf == "A_log" and len(shape) == 2:
+                t = torch.log(torch.arange(1, shape[1] + 1, device=device, dtype=torch.float32)).expand(shape)
+            elif leaf == "D":
                 t = torch.ones(shape, device=device)
+            elif name.endswith(".dt.b"):
+                t = -5.0 + 3.0 * torch.rand(shape, device=device, generator=g)
+            elif name.endswith((".q.b", ".k.b", ".v.b", ".conv.b")):
+                t = torch.randn(shape, device=device, generator=g) * std
             elif leaf == "A_log":
                 t = torch.log(1.0 + 3.0 * torch.rand(shape, device=device, generator=g))
             elif leaf in ("sink", "correction"):

@@ -4,24 +4,70 @@ Mixers (``LayerSpec.mixer``):
 
 * ``RecurrentMixer`` kind ``gla``: gated linear attention, decay ``sigmoid(z)^(1/tau)`` per key channel;
 * ``RecurrentMixer`` kind ``delta``: gated delta rule with short convolutions and unit-norm q / k;
-* ``AttentionMixer``: causal softmax attention without rotation, q / k norms, per-head output gate,
-  key and value widths of their own;
-* ``ParallelMixer``: an attention and a delta mixer on the same input, averaged after their own norms;
+* ``AttentionMixer``: causal softmax attention with key and value widths of their own; q / k norms, biases,
+  rotation, query temperature, sliding window, sink and output gate as its fields say. A layer may use the
+  keys and values of an earlier one (``kv_from``);
+* ``SelectiveMixer``: selective scan, a diagonal recurrence per channel with step sizes, input and output maps
+  that depend on the token, behind a short convolution;
+* ``ParallelMixer``: an attention and a recurrent mixer on the same input, averaged after their own norms or
+  added with constant scales;
 * ``LatentAttentionMixer``: attention whose keys and values are linear maps of one normalised latent per
   token, plus a rotated key part that all heads share; only the latent and that part are cached. A
   learned sink per head enters the softmax denominator.
 
-Feed-forwards (``LayerSpec.mlp``): ``DenseFF`` (gated, with its activation) and ``MoeFF`` (softmax router
-with a choice correction and expert groups over gated experts).
+Feed-forwards (``LayerSpec.mlp``): ``DenseFF`` (gated, with its activation) and ``MoeFF`` (a router that
+scores by softmax or sigmoid, with expert groups, over gated experts, and optionally a shared expert).
 
 The designs served under this configuration are Teganex (norms before and after every sublayer, learned
-positions) and Lebedra (norms on the sublayer outputs only, latent attention, experts, per-layer token input).
+positions), Lebedra (norms on the sublayer outputs only, latent attention, experts, per-layer token input) and
+Dogozen (norms around sublayers with weights stored around zero, tempered full attention with shared caches,
+window attention beside a selective scan, sigmoid-routed experts, tied and soft-capped output).
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 
 from .registry import register
+
+
+@dataclass
+class FrequencyScaling:
+    """Slows the rotation of pairs that turn fewer than ``low`` times within ``original`` positions by ``factor``,
+    leaves those that turn more than ``high`` times, and blends between."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+    def apply(self, f: float) -> float:
+        turns = self.original * f / (2.0 * math.pi)
+        if turns > self.high:
+            return f
+        if turns < self.low:
+            return f / self.factor
+        s = (turns - self.low) / (self.high - self.low) if self.high != self.low else 1.0
+        return (1.0 - s) * f / self.factor + s * f
+
+
+@dataclass
+class Rotation:
+    """Rotary positions on the first ``dims`` columns of a head, column i paired with i + dims / 2."""
+    base: float
+    dims: int
+    scaling: FrequencyScaling | None = None
+
+    def turns(self) -> list:
+        """Revolutions per position of every pair."""
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        return [(self.scaling.apply(x) if self.scaling else x) / (2.0 * math.pi) for x in f]
+
+
+@dataclass
+class QueryTemperature:
+    """Queries at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
+    coef: float
+    every: float
 
 
 @dataclass
@@ -31,11 +77,28 @@ class AttentionMixer:
     dim: int
     vdim: int
     scale: float
+    qk_norm: str | None = "weighted"   # RMS norm of every q / k head: "weighted", "plain" (no weight) or None
+    gate: str | None = "head"          # sigmoid output gate: one value per head, per "channel", or None
+    bias: bool = False                 # on q, k and v
+    rotation: Rotation | None = None
+    window: int = 0                    # keys a query sees, itself included; 0: all earlier ones
+    sink: bool = False                 # one more logit per head in the softmax denominator
+    q_temp: QueryTemperature | None = None
+    kv_from: int | None = None         # layer whose cached keys and values are used
 
     def __post_init__(self):
         _positive(self, "heads", "kv_heads", "dim", "vdim")
         if self.heads % self.kv_heads:
             raise ValueError(f"attention: {self.heads} heads do not divide by {self.kv_heads} key/value heads")
+        if self.qk_norm not in ("weighted", "plain", None) or self.gate not in ("head", "channel", None):
+            raise ValueError(f"attention: unknown norm {self.qk_norm!r} or gate {self.gate!r}")
+        if self.window < 0:
+            raise ValueError(f"attention: negative window {self.window}")
+        r = self.rotation
+        if r is not None and (r.dims <= 0 or r.dims % 2 or r.dims > self.dim):
+            raise ValueError(f"attention: {r.dims} rotated columns of {self.dim}")
+        if self.q_temp is not None and self.q_temp.every <= 0:
+            raise ValueError("attention: the query temperature's period must be positive")
 
 
 @dataclass
@@ -61,9 +124,22 @@ class RecurrentMixer:
 
 
 @dataclass
+class SelectiveMixer:
+    """S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n, y_c = sum_n S[c, n] C_n + D_c x_c, times silu(z)."""
+    inner: int                 # channels
+    state: int                 # state values per channel
+    dt_rank: int               # width of the low-rank map to the step sizes
+    conv: int                  # taps of the short convolution on x
+
+    def __post_init__(self):
+        _positive(self, "inner", "state", "dt_rank", "conv")
+
+
+@dataclass
 class ParallelMixer:
     left: AttentionMixer
-    right: RecurrentMixer
+    right: RecurrentMixer | SelectiveMixer
+    scales: tuple | None = None        # (left, right) factors of the sum; None: mean of the normalised outputs
 
 
 @dataclass
@@ -96,20 +172,33 @@ class DenseFF:
 
 @dataclass
 class MoeFF:
-    """``top`` of ``experts`` clamped gated experts of width ``ff``: g = min(gate h, limit),
-    u = clamp(up h, -limit, limit), ``down(g sigmoid(alpha g) (u + 1))``. Scores are the softmax over all
-    experts and weigh the outputs as they are; scores + correction choose, first the ``keep`` best of
-    ``groups`` groups of neighbours (by their best expert), then the experts in them."""
+    """``top`` of ``experts`` gated experts of width ``ff``. Scores (softmax over all experts, or the sigmoid of each)
+    choose, plus a correction per expert if there is one: first the ``keep`` best of ``groups`` groups of neighbours
+    (by the sum of their ``group_best`` largest), then the experts in them. The chosen scores, without
+    correction, weigh the outputs: as they are, or normalised to the sum ``scale``. A shared expert of width
+    ``shared`` runs for every token.
+
+    Experts: ``act`` "clamped": g = min(gate h, limit), u = clamp(up h, -limit, limit),
+    ``down(g sigmoid(alpha g) (u + 1))``; "silu" / "relu": as ``DenseFF``."""
     experts: int
     top: int
     ff: int
-    limit: float
+    limit: float = 0.0
     groups: int = 1
     keep: int = 1
     alpha: float = 1.702
+    act: str = "clamped"
+    score: str = "softmax"     # "softmax" | "sigmoid"
+    correction: bool = True
+    group_best: int = 1        # scores of a group that are added (1 or 2)
+    normalise: bool = False
+    scale: float = 1.0
+    shared: int = 0
 
     def __post_init__(self):
         _positive(self, "experts", "top", "ff", "groups", "keep")
+        if self.act not in ("clamped", "silu", "relu") or self.score not in ("softmax", "sigmoid") or self.group_best not in (1, 2):
+            raise ValueError(f"experts: unknown activation {self.act!r}, score {self.score!r} or group rule {self.group_best!r}")
         if self.experts % self.groups or self.keep > self.groups:
             raise ValueError(f"experts: {self.experts} do not form {self.groups} equal groups, or more are kept ({self.keep})")
         if self.top > self.experts // self.groups * self.keep:
@@ -124,17 +213,17 @@ class LayerSpec:
 
     @property
     def attention(self) -> AttentionMixer | None:
-        return self.mixer.left if isinstance(self.mixer, ParallelMixer) else None
+        m = self.mixer.left if isinstance(self.mixer, ParallelMixer) else self.mixer
+        return m if isinstance(m, AttentionMixer) else None
 
     @property
     def latent(self) -> LatentAttentionMixer | None:
         return self.mixer if isinstance(self.mixer, LatentAttentionMixer) else None
 
     @property
-    def recurrent(self) -> RecurrentMixer | None:
-        if isinstance(self.mixer, ParallelMixer):
-            return self.mixer.right
-        return self.mixer if isinstance(self.mixer, RecurrentMixer) else None
+    def recurrent(self) -> RecurrentMixer | SelectiveMixer | None:
+        m = self.mixer.right if isinstance(self.mixer, ParallelMixer) else self.mixer
+        return m if isinstance(m, (RecurrentMixer, SelectiveMixer)) else None
 
 
 DEFAULT_CONTEXT = 8192        # of designs without a position table, where the caller names no length
@@ -155,10 +244,20 @@ class HybridConfig:
     pre_norm: bool = True          # sublayers read a normalised copy of the stream (else the stream itself)
     residual_mult: float = 1.0     # x <- x + residual_mult * norm(sublayer)
     token_side: int = 0            # width of the per-layer token input, 0: none
+    norm_offset: float = 0.0       # added to every stored norm weight
+    tied_head: bool = False        # the embedding table is the output matrix
+    logit_softcap: float = 0.0     # logits <- cap tanh(logits / cap); 0: none
     extras: dict = field(default_factory=dict)
 
     def __post_init__(self):
         _positive(self, "vocab_size", "hidden_size", "max_seq_len")
+        for i, x in enumerate(self.layers):
+            a = x.attention
+            if a is None or a.kv_from is None:
+                continue
+            b = self.layers[a.kv_from].attention if 0 <= a.kv_from < i else None
+            if b is None or b.kv_from is not None or (b.kv_heads, b.dim, b.vdim) != (a.kv_heads, a.dim, a.vdim):
+                raise ValueError(f"layer {i}: layer {a.kv_from} has no keys and values of its shape to share")
 
     @property
     def num_layers(self) -> int:
@@ -178,17 +277,25 @@ class HybridConfig:
             return cls(layers=[_layer_from_dict(i, x, ("latent_attention",), "relu") for i, x in enumerate(d["layers"])],
                        position_table=False, pre_norm=False, residual_mult=float(d["residual_mult"]),
                        token_side=int(side["dim"]) if side else 0, **common)
+        if arch == "Dogozen":
+            return cls(layers=[_dogozen_layer(i, x) for i, x in enumerate(d["layers"])],
+                       position_table=False, norm_offset=1.0, tied_head=True, logit_softcap=float(d.get("logit_softcap") or 0.0),
+                       **common)
         return cls(layers=[_layer_from_dict(i, x, ("gla", "parallel"), "silu") for i, x in enumerate(d["layers"])],
                    embed_scale=float(d["embedding"]["scale"]), logit_scale=float(d["logit_scale"]),
                    max_seq_len=int(d["max_positions"]), **common)
 
     def to_dict(self) -> dict:
+        layer = _dogozen_layer_to_dict if self.architecture == "Dogozen" else _layer_to_dict
         d = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
-             "norm": {"eps": self.norm_eps}, "layers": [_layer_to_dict(x) for x in self.layers]}
+             "norm": {"eps": self.norm_eps}, "layers": [layer(x) for x in self.layers]}
         if self.architecture == "Lebedra":
             d["residual_mult"] = self.residual_mult
             if self.token_side:
                 d["token_side"] = {"dim": self.token_side}
+        elif self.architecture == "Dogozen":
+            if self.logit_softcap:
+                d["logit_softcap"] = self.logit_softcap
         else:
             d.update(max_positions=self.max_seq_len, embedding={"scale": self.embed_scale}, logit_scale=self.logit_scale)
         return d
@@ -253,6 +360,70 @@ def _layer_to_dict(x: LayerSpec) -> dict:
     return {"type": x.type, "mixer": mixer, "mlp": mlp}
 
 
+# ---- Dogozen
+def _dogozen_attention(a: dict, **fixed) -> AttentionMixer:
+    rot, temp = a.get("rot"), a.get("q_temp")
+    scaling = rot.get("scaling") if rot else None
+    return AttentionMixer(
+        int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), int(a["vdim"]), float(a["scale"]),
+        rotation=Rotation(float(rot["base"]), int(rot["dims"]),
+                          FrequencyScaling(*(float(scaling[n]) for n in ("factor", "low", "high", "original"))) if scaling else None)
+        if rot else None,
+        window=int((a.get("mask") or {}).get("size", 0)),
+        q_temp=QueryTemperature(float(temp["coef"]), float(temp["every"])) if temp else None,
+        kv_from=int(a["kv_from"]) if a.get("kv_from") is not None else None, **fixed)
+
+
+def _dogozen_layer(index: int, d: dict) -> LayerSpec:
+    kind, m, mlp = d["type"], d["mixer"], d.get("mlp")
+    if kind == "attention":
+        mixer = _dogozen_attention(m, qk_norm="plain", gate="channel", bias=True)
+    elif kind == "parallel":
+        r = m["right"]
+        mixer = ParallelMixer(_dogozen_attention(m["left"], qk_norm=None, gate=None, sink=True),
+                              SelectiveMixer(int(r["inner"]), int(r["state"]), int(r["dt_rank"]), int(r["conv"])),
+                              (float(m["left_scale"]), float(m["right_scale"])))
+    else:
+        raise ValueError(f"layer {index}: unknown mixer type {kind!r}")
+    if mlp is not None and mlp.get("kind") == "moe":
+        r, shared = mlp["router"], mlp.get("shared")
+        g = r.get("groups") or {"count": 1, "keep": 1}
+        ff = MoeFF(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), groups=int(g["count"]), keep=int(g["keep"]), act="silu",
+                   score="sigmoid", correction=False, group_best=2, normalise=True, scale=float(r["scale"]),
+                   shared=int(shared["ff"]) if shared else 0)
+        return LayerSpec(kind, mixer, ff)
+    return LayerSpec(kind, mixer, _mlp_from_dict(index, mlp, "silu"))
+
+
+def _dogozen_layer_to_dict(x: LayerSpec) -> dict:
+    def attention(a: AttentionMixer) -> dict:
+        d = {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale}
+        if a.rotation:
+            d["rot"] = {"base": a.rotation.base, "dims": a.rotation.dims}
+            if a.rotation.scaling:
+                d["rot"]["scaling"] = dict(vars(a.rotation.scaling))
+        if a.window:
+            d["mask"] = {"size": a.window}
+        if a.q_temp:
+            d["q_temp"] = dict(vars(a.q_temp))
+        if a.kv_from is not None:
+            d["kv_from"] = a.kv_from
+        return d
+
+    m, f = x.mixer, x.mlp
+    if isinstance(m, ParallelMixer):
+        mixer = {"left": attention(m.left), "right": dict(vars(m.right)), "left_scale": m.scales[0], "right_scale": m.scales[1]}
+    else:
+        mixer = attention(m)
+    mlp = {"kind": "dense", "ff": f.ff} if f is not None else None
+    if isinstance(f, MoeFF):
+        mlp = {"kind": "moe", "expert": {"ff": f.ff},
+               "router": {"experts": f.experts, "top": f.top, "scale": f.scale, "groups": {"count": f.groups, "keep": f.keep}}}
+        if f.shared:
+            mlp["shared"] = {"ff": f.shared}
+    return {"type": x.type, "mixer": mixer, "mlp": mlp}
+
+
 # ------------------------------------------------------------------ named configurations
 def teganex_config(width: int = 2048, layers: int = 8, vocab: int = 32000, max_positions: int = 8192,
                    parallel_every: int = 4) -> HybridConfig:
@@ -282,5 +453,33 @@ def lebedra_config(width: int = 2048, layers: int = 8, vocab: int = 32000, max_p
                         pre_norm=False, residual_mult=0.5, token_side=128)
 
 
+def dogozen_config(width: int = 2048, layers: int = 8, vocab: int = 32000, max_positions: int = 8192, experts: int = 64,
+                   top: int = 6, window: int = 1024) -> HybridConfig:
+    """Dogozen at the layer sizes of a real model: full attention and window attention beside a selective scan of
+    twice the width alternate; dense feed-forwards and experts whose ``top`` and shared one together are about as
+    wide. The last full-attention layer uses the keys and values of the one before."""
+    h = width // 128
+    dense = width * 11 // 4 // 128 * 128
+    one = max(128, dense // (top + 2) // 128 * 128)
+    moe = MoeFF(experts, top, one, groups=8, keep=4, act="silu", score="sigmoid", correction=False, group_best=2, normalise=True,
+                scale=2.5, shared=2 * one)
+    full = [i for i in range(layers) if i % 2 == 0]
+    out = []
+    for i in range(layers):
+        if i % 2 == 0:
+            share = full[-2] if len(full) > 2 and i == full[-1] else None
+            out.append(LayerSpec("attention", AttentionMixer(
+                h, max(1, h // 8), 128, 128, 128 ** -0.5, qk_norm="plain", gate="channel", bias=True,
+                q_temp=QueryTemperature(0.1, 8192), kv_from=share), DenseFF(dense)))
+        else:
+            out.append(LayerSpec("parallel", ParallelMixer(
+                AttentionMixer(h, max(1, h // 8), 128, 128, 128 ** -0.5, qk_norm=None, gate=None, sink=True, window=window,
+                               rotation=Rotation(500000.0, 128, FrequencyScaling(8.0, 1.0, 4.0, 8192))),
+                SelectiveMixer(2 * width, 16, max(8, width // 16), 4), (1.0, 1.0)), moe))
+    return HybridConfig(vocab, width, out, 1e-6, max_seq_len=max_positions, architecture="Dogozen", position_table=False,
+                        norm_offset=1.0, tied_head=True, logit_softcap=30.0)
+
+
+register("Dogozen", HybridConfig.from_dict, "mythos_b200.models.hybrid:HybridModel")
 register("Lebedra", HybridConfig.from_dict, "mythos_b200.models.hybrid:HybridModel")
 register("Teganex", HybridConfig.from_dict, "mythos_b200.models.hybrid:HybridModel")

@@ -228,10 +228,170 @@ def forward_lebedra(cfg, W, tokens, dtype=torch.float64, trace=None):
     return rms_norm(x, W["final.norm"], eps) @ W["head"].T
 
 
+# ------------------------------------------------------------------ Dogozen
+def rms_norm_around_zero(x, w, eps):
+    return rms(x, eps) * (1 + w)
+
+
+def frequencies(r):
+    """Angle per position of every rotated pair, with the optional stretching of long wavelengths: pairs that turn
+    fewer than ``low`` times within ``original`` positions are slowed by ``factor``, those that turn more than ``high``
+    times are not, and those between are blended linearly in the number of turns."""
+    out = []
+    for i in range(r["dims"] // 2):
+        f = float(r["base"]) ** (-2.0 * i / r["dims"])
+        sc = r.get("scaling")
+        if sc:
+            turns = sc["original"] * f / (2 * torch.pi)
+            if turns < sc["low"]:
+                f = f / sc["factor"]
+            elif turns <= sc["high"]:
+                s = (turns - sc["low"]) / (sc["high"] - sc["low"])
+                f = (1 - s) * f / sc["factor"] + s * f
+        out.append(f)
+    return out
+
+
+def rotate_halves(x, pos, r):
+    """Components i and i + dims / 2 of x [T, heads, n] turn together; those from ``dims`` on stay."""
+    out, half = x.clone(), r["dims"] // 2
+    for i, f in enumerate(frequencies(r)):
+        a = pos.to(torch.float64) * f
+        c, s = torch.cos(a).to(x.dtype)[:, None], torch.sin(a).to(x.dtype)[:, None]
+        u, v = x[..., i], x[..., i + half]
+        out[..., i], out[..., i + half] = u * c - v * s, v * c + u * s
+    return out
+
+
+def query_temperature(pos, c):
+    return 1 + c["coef"] * torch.log(torch.floor((pos + 1).to(torch.float64) / c["every"]) + 1)
+
+
+def window_sink_attention(q, k, v, scale, window=None, sink=None):
+    """Query i sees keys j <= i, with ``window`` only those with i - j < window; with ``sink`` the denominator has one
+    more term per query head. q [T, H, dk]; k [T, G, dk]; v [T, G, dv]."""
+    T, H, _ = q.shape
+    G = k.shape[1]
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for h in range(H):
+        g = h // (H // G)
+        for i in range(T):
+            lo = 0 if window is None else max(0, i - window + 1)
+            s = (k[lo:i + 1, g] @ q[i, h]) * scale
+            m = s.max() if sink is None else torch.maximum(s.max(), sink[h])
+            e = torch.exp(s - m)
+            out[i, h] = (e @ v[lo:i + 1, g]) / (e.sum() + (0 if sink is None else torch.exp(sink[h] - m)))
+    return out
+
+
+def tempered_attention(h, W, p, c, eps, kv):
+    """Attention with unit-rms queries and keys, query temperature and a gate per channel; ``kv`` (layer -> keys and
+    values) receives the layer's own and gives those of a layer that shares them."""
+    T, H, G = h.shape[0], c["heads"], c["kv_heads"]
+    pos = torch.arange(T)
+    q = rms((h @ W[p + "q"].T + W[p + "q.b"]).view(T, H, c["dim"]), eps)
+    if c.get("q_temp"):
+        q = q * query_temperature(pos, c["q_temp"]).to(q.dtype)[:, None, None]
+    if c.get("kv_from") is None:
+        k = rms((h @ W[p + "k"].T + W[p + "k.b"]).view(T, G, c["dim"]), eps)
+        v = (h @ W[p + "v"].T + W[p + "v.b"]).view(T, G, c["vdim"])
+        kv[p] = (k, v)
+    else:
+        k, v = kv[f"l{c['kv_from']}.mix."]
+    o = window_sink_attention(q, k, v, c["scale"]).reshape(T, H * c["vdim"])
+    return (o * torch.sigmoid(h @ W[p + "g"].T)) @ W[p + "o"].T
+
+
+def window_attention(h, W, p, c):
+    T, H, G = h.shape[0], c["heads"], c["kv_heads"]
+    pos = torch.arange(T)
+    q = rotate_halves((h @ W[p + "q"].T).view(T, H, c["dim"]), pos, c["rot"])
+    k = rotate_halves((h @ W[p + "k"].T).view(T, G, c["dim"]), pos, c["rot"])
+    v = (h @ W[p + "v"].T).view(T, G, c["vdim"])
+    o = window_sink_attention(q, k, v, c["scale"], c["mask"]["size"], W[p + "sink"])
+    return o.reshape(T, H * c["vdim"]) @ W[p + "o"].T
+
+
+def selective_scan(x, dt, A, B, C, D):
+    """x, dt [T, channels]; A [channels, n]; B, C [T, n]; D [channels] -> y [T, channels]."""
+    S = torch.zeros_like(A)
+    out = torch.zeros_like(x)
+    for t in range(x.shape[0]):
+        S = torch.exp(dt[t][:, None] * A) * S + (dt[t] * x[t])[:, None] * B[t][None, :]
+        out[t] = S @ C[t] + D * x[t]
+    return out
+
+
+def mamba(h, W, p, c):
+    n, r = c["state"], c["dt_rank"]
+    xz = h @ W[p + "in"].T
+    x, z = xz[:, : c["inner"]], xz[:, c["inner"]:]
+    x = silu(short_conv(x, W[p + "conv"]) + W[p + "conv.b"])
+    low = x @ W[p + "x"].T
+    dt = softplus(low[:, :r] @ W[p + "dt"].T + W[p + "dt.b"])
+    y = selective_scan(x, dt, -torch.exp(W[p + "A_log"]), low[:, r:r + n], low[:, r + n:], W[p + "D"])
+    return (y * silu(z)) @ W[p + "o"].T
+
+
+def scaled_parallel(h, W, p, c):
+    return (c["left_scale"] * window_attention(h, W, p + "left.", c["left"])
+            + c["right_scale"] * mamba(h, W, p + "right.", c["right"]))
+
+
+def choose_by_sigmoid(z, r):
+    """Router logits of one token -> list of (expert, weight): groups by the sum of their two best scores, weights
+    normalised over the chosen experts."""
+    s = torch.sigmoid(z)
+    g = r.get("groups") or {"count": 1, "keep": 1}
+    size = r["experts"] // g["count"]
+    score = s.tolist()
+    rank = lambda i: sum(sorted(score[i * size:(i + 1) * size])[-2:])
+    best = sorted(range(g["count"]), key=lambda i: -rank(i))[: g["keep"]]
+    allowed = [e for e in range(r["experts"]) if e // size in best]
+    picked = sorted(allowed, key=lambda e: -score[e])[: r["top"]]
+    total = sum(s[e] for e in picked) + 1e-20
+    return [(e, s[e] / total * r["scale"]) for e in picked]
+
+
+def sigmoid_moe(h, W, p, c):
+    z = h @ W[p + "router"].T
+    out = dense_ff(h, W, p + "shared.") if c.get("shared") else torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, w in choose_by_sigmoid(z[t], c["router"]):
+            out[t] += w * dense_ff(h[t:t + 1], W, p + f"e{e}.")[0]
+    return out
+
+
+def soft_cap(x, cap):
+    return cap * torch.tanh(x / cap)
+
+
+def forward_dogozen(cfg, W, tokens, dtype=torch.float64, trace=None):
+    W = {k: v.to(dtype) for k, v in W.items()}
+    eps = cfg["norm"]["eps"]
+    x = W["embed"][torch.as_tensor(tokens, dtype=torch.long)]
+    kv = {}
+    for i, L in enumerate(cfg["layers"]):
+        p = f"l{i}."
+        h = rms_norm_around_zero(x, W[p + "norm1"], eps)
+        y = (tempered_attention(h, W, p + "mix.", L["mixer"], eps, kv) if L["type"] == "attention"
+             else scaled_parallel(h, W, p + "mix.", L["mixer"]))
+        x = x + rms_norm_around_zero(y, W[p + "norm1b"], eps)
+        if L["mlp"] is not None:
+            h = rms_norm_around_zero(x, W[p + "norm2"], eps)
+            y = sigmoid_moe(h, W, p + "mlp.", L["mlp"]) if L["mlp"]["kind"] == "moe" else dense_ff(h, W, p + "mlp.")
+            x = x + rms_norm_around_zero(y, W[p + "norm2b"], eps)
+        if trace is not None:
+            trace.append(x)
+    return soft_cap(rms_norm_around_zero(x, W["final.norm"], eps) @ W["embed"].T, cfg["logit_softcap"])
+
+
 def forward(cfg, W, tokens, dtype=torch.float64, trace=None):
     """Logits [T, vocab] of one sequence; ``trace`` (a list) receives the stream after every layer."""
     if cfg["architecture"] == "Lebedra":
         return forward_lebedra(cfg, W, tokens, dtype, trace)
+    if cfg["architecture"] == "Dogozen":
+        return forward_dogozen(cfg, W, tokens, dtype, trace)
     W = {k: v.to(dtype) for k, v in W.items()}
     eps = cfg["norm"]["eps"]
     tok = torch.as_tensor(tokens, dtype=torch.long)

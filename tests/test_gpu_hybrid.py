@@ -167,18 +167,20 @@ def _run_attention(case, kernel, gamma_q, gamma_k, scale):
     c, dt = case, case["proj"].dtype
     rows = c["proj"].shape[0]
     q = torch.empty(rows, c["heads"], c["dk"], device="cuda", dtype=dt)
-    H().qk_norm_append(c["proj"], *c["off"], gamma_q, gamma_k, c["batch"], c["table"], q, c["kc"], c["vc"], 1e-5)
+    att = H().Attention({"heads": c["heads"], "kv_heads": c["kv"], "dk": c["dk"], "dv": c["dv"], "q_off": c["off"][0], "k_off": c["off"][1],
+                         "v_off": c["off"][2], "norm_dim": c["dk"], "eps": 1e-5, "scale": scale}, {"q_gamma": gamma_q, "k_gamma": gamma_k})
+    att.prep(c["proj"], c["batch"], c["table"], q, c["kc"], c["vc"])
     o = torch.full((rows, c["heads"] * c["dv"]), float("nan"), device="cuda", dtype=dt)
     args = (q, c["kc"], c["vc"], c["batch"], c["table"], c["gate"], o)
     if kernel == "any":
-        H().paged_attn_any(*args, scale)
+        att.any(*args)
     elif kernel == "prefill":
-        H().paged_attn_prefill(*args, max(c["lens"]), scale, status())
+        att.prefill(*args, max(c["lens"]), status())
     else:
         counters = torch.zeros(4096, dtype=torch.int32, device="cuda")
         for splits in (1, 3):
-            scratch = torch.empty(rows * c["heads"] * splits * (c["dv"] + 2), device="cuda")
-            H().paged_attn_decode(*args, scratch, counters, splits, scale, status())
+            scratch = torch.empty(att.decode_scratch(rows, splits), device="cuda")
+            att.decode(*args, scratch, counters, splits, status())
             assert int(counters.abs().sum()) == 0
     return q, o.view(rows, c["heads"], c["dv"])
 

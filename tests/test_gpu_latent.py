@@ -295,7 +295,7 @@ def test_experts_of_a_batch(dtype, tile, T, E, top, dim, ff, limit):
     close(y, want, tol)
     out, xs = torch.empty(T, dim, device="cuda", dtype=dtype), torch.randn(T, dim, device="cuda")
     wp, x0 = 1 + 0.3 * torch.randn(dim, device="cuda"), d(xs)
-    C.expert_norm(y, row, weight, wp, xs, None, out, 1e-4, 0.7)
+    C.expert_norm(y, None, row, weight, wp, xs, None, out, 1e-4, 0.7)
     total = (d(y)[rc.long()] * d(weight)[..., None]).sum(1)
     ref = x0 + 0.7 * oracle.rms_norm(total, d(wp), 1e-4)
     close(xs, ref, 1e-5)
