@@ -1,6 +1,6 @@
-"""Speed of layer-list models (Teganex or Lebedra layers at the sizes of a real model, random weights) beside
-the dense transformer engine of equal width, depth and feed-forward (Lebedra: the dense layer's, and the experts of
-a token together about as wide), both with bf16 weights.
+"""Speed of layer-list models (Teganex, Lebedra or Dogozen layers at the sizes of a real model, random weights) beside
+the dense transformer engine of equal width, depth and feed-forward (Lebedra, Dogozen: the dense layers', and the
+experts of a token together about as wide), both with bf16 weights.
 
 ``run_models``: prefill and decode throughput of both engines. ``run_kernels``: every kernel of the new
 design next to the like kernel of the dense model, with the fraction of its roofline (bytes over the
@@ -31,7 +31,7 @@ def _engines(design, width, layers, vocab, batch, max_len):
     from ..models import hybrid_config as hc
 
     kw = dict(seed=1, device="cuda", max_batch=batch, max_seq_len=max_len)
-    make = {"teganex": hc.teganex_config, "lebedra": hc.lebedra_config}[design]
+    make = {"teganex": hc.teganex_config, "lebedra": hc.lebedra_config, "dogozen": hc.dogozen_config}[design]
     yield design, HybridEngine.random(make(width, layers, vocab, max_len), **kw)
     yield "dense", InferenceEngine.random(_dense_config(width, layers, vocab, max_len), **kw)
 
@@ -179,6 +179,153 @@ def _dense_attention_rows(K, H, C, st, rnd, h, kv):
               nbytes=4.0 * NB * ctx * kv * 128)
 
 
+EXPERT_TOKENS = (1, 16, 64, 1024, 8192)
+
+
+def _expert_rows(K, H, C, rnd, eng, L, T):
+    """Routed experts of a layer for T tokens and the norms around them; gives two [T, width] activations."""
+    from ..ops import functional as F
+
+    e, d, bf, st = L.spec.mlp, eng.cfg.hidden_size, torch.bfloat16, eng._status
+    route = (e.experts, e.top, e.groups, e.keep)
+    i32 = dict(device="cuda", dtype=torch.int32)
+    f, gen = e.ff, torch.Generator().manual_seed(5)
+    pairs, tile = T * e.top, eng._expert_tile(T, e)
+    z = torch.randn(T, e.experts, generator=gen).cuda()
+    idx, slot, row = (torch.empty(T, e.top, **i32) for _ in range(3))
+    wt, off, cnt = torch.empty(T, e.top, device="cuda"), torch.empty(e.experts, **i32), torch.empty(1, **i32)
+    tiles = torch.empty(min(pairs, e.experts + pairs // tile), 3, **i32)
+    plan = (idx, wt, slot, eng._expert_counts, off, tiles, cnt)
+    x, hid, a, y = rnd(pairs, d), rnd(T, d), rnd(pairs, f), rnd(pairs, d)
+    sizes = f"{T} tokens, {e.top} of {e.experts}, {d} x {f}"
+    K.add("expert_select", sizes, lambda: H.expert_select(z, L.correction, route, tile, *plan, L.rule), nbytes=4.0 * T * e.experts,
+          like="moe_route (training)")
+    probs, psum, lg = torch.empty(T, e.experts, device="cuda"), torch.zeros(e.experts, device="cuda"), z.to(bf)
+    cn = torch.zeros(e.experts, **i32)
+    K.add("moe_route (training)", sizes, lambda: C.moe_route(lg, e.experts, probs, idx, slot, wt, cn, psum), nbytes=2.0 * T * e.experts)
+    H.expert_select(z, L.correction, route, tile, *plan, L.rule)
+    used = int((torch.bincount(idx.flatten().long(), minlength=e.experts) > 0).sum())
+    K.add("expert_gather", sizes, lambda: H.expert_gather(hid, route, *plan, x, row), nbytes=2.0 * d * (T + pairs), like="rope (dense)")
+    K.add("experts in (gate, up)", sizes, lambda: H.gemm_tiles(x, L.w_in, a, tiles, cnt, tile, f, f, L.act, st),
+          nbytes=2.0 * (used * 2 * f * d + pairs * (d + f)), flops=4.0 * pairs * f * d, like="gemm (dense bf16)")
+    K.add("experts out (down)", sizes, lambda: H.gemm_tiles(a, L.w_out, y, tiles, cnt, tile, 0, 0, L.act, st),
+          nbytes=2.0 * (used * f * d + pairs * (d + f)), flops=2.0 * pairs * f * d, like="gemm (dense bf16)")
+    for N, Kd in ((2 * f * e.top, d), (d, f * e.top)):         # the dense layer of the same width
+        xx, ww, o1 = rnd(T, Kd), rnd(N, Kd), torch.empty(T, N, device="cuda", dtype=bf)
+        K.add("gemm (dense bf16)", f"{T} x {N} x {Kd}", lambda: F.gemm(xx, ww, out=o1), nbytes=2.0 * (N * Kd + T * (N + Kd)),
+              flops=2.0 * T * N * Kd)
+    shared = rnd(T, d) if e.shared else None
+    xs, w32, hh = torch.randn(T, d, device="cuda"), torch.ones(d, device="cuda"), rnd(T, d)
+    nxt = w32 if eng.cfg.pre_norm else None
+    K.add("expert_norm", f"{T} x {d}, {e.top} outputs", lambda: H.expert_norm(y, shared, row, wt, w32, xs, nxt, hh, 1e-6, 0.5),
+          nbytes=T * d * (2.0 * e.top + 10 + 2 * (shared is not None)), like="rmsnorm + residual (dense)")
+    K.add("norm + residual", f"{T} x {d}", lambda: H.sandwich_norm(hh, None, None, None, w32, xs, nxt, x[:T], 1e-6, 0.5),
+          nbytes=T * d * 12.0, like="rmsnorm + residual (dense)")
+    g, res = torch.ones(d, device="cuda", dtype=bf), rnd(T, d)
+    K.add("rmsnorm + residual (dense)", f"{T} x {d}", lambda: F.rmsnorm(hh, g, 1e-6, res), nbytes=T * d * 8.0)
+    return hid, hh
+
+
+def run_dogozen_kernels(peaks: dict, width: int = 2048) -> list[dict]:
+    """Tempered and window attention (heads of 128), selective scan, routed and shared experts, soft-capped output."""
+    from ..infer.hybrid import LOW_RANK_FUSE_ROWS, HybridEngine
+    from ..models.hybrid_config import dogozen_config
+    from ..ops import functional as F, native
+
+    H, C, st = native.require_hybrid(), native.require(), native.status_word("cuda")
+    K, bf, d = _Kernels(peaks), torch.bfloat16, width
+    rnd = lambda *s: torch.randn(*s, device="cuda").to(bf)
+    cfg = dogozen_config(width, 2, 32000)
+    eng = HybridEngine.random(cfg, device="cuda", max_batch=64, max_seq_len=4096, kv_pages=64)
+    full, par = eng.layers
+    h, kv, r = full.spec.mixer.heads, full.spec.mixer.kv_heads, par.spec.mixer.right
+    win, sms = par.spec.mixer.left.window, torch.cuda.get_device_properties(0).multi_processor_count
+    _dense_attention_rows(K, H, C, st, rnd, h, kv)
+
+    def visible(S, w):                                 # query-key pairs of a sequence
+        return S * (S + 1) / 2 if not w or w >= S else w * (w + 1) / 2 + (S - w) * w
+
+    def pages(B, S):
+        n = B * S // PAGE
+        return torch.randperm(n, device="cuda").to(torch.int32).view(B, -1), rnd(n, PAGE, kv, 128), rnd(n, PAGE, kv, 128)
+
+    # ---- attention
+    kinds = (("tempered, gated", full, 0), (f"window {win}, sink", par, win))
+    for B, S in ((4, 2048), (1, 8192)):
+        (table, kc, vc), b, n = pages(B, S), _batch([S] * B, [0] * B), B * S
+        q, o = rnd(n, h, 128), torch.empty(n, h * 128, device="cuda", dtype=bf)
+        for name, L, w in kinds:
+            proj = rnd(n, L.proj.N)
+            gate = proj[:, L.proj.off["g"]:][:, : h * 128] if "g" in L.proj.off else None
+            K.add(f"attn_prep, {name}", f"{n} tokens, {h}/{kv} heads, 128", lambda: L.att.prep(proj, b, table, q, kc, vc),
+                  nbytes=4.0 * n * (h + 2 * kv) * 128, like="rope (dense)")
+            K.add(f"paged prefill attention, {name}", f"{B} x {S}, {h}/{kv} heads, 128",
+                  lambda: L.att.prefill(q, kc, vc, b, table, gate, o, S, st), flops=2.0 * B * h * visible(S, w) * 256,
+                  nbytes=n * (h * 128 * (4.0 + 2 * (gate is not None)) + 512 * kv), like="paged prefill attention (dense)")
+    qkv, pos = rnd(8192, h + 2 * kv, 128), torch.arange(2048, device="cuda", dtype=torch.int32).repeat(4)
+    K.add("rope (dense)", f"8192 tokens, {h}/{kv} heads, 128", lambda: C.rope(qkv[:, : h + kv], pos, 10000.0, False),
+          nbytes=4.0 * 8192 * (h + kv) * 128)
+    for NB, ctx in ((16, 4096), (64, 1024), (64, 4096)):
+        (table, kc, vc), b = pages(NB, ctx), _batch([1] * NB, [ctx - 1] * NB)
+        q, o = rnd(NB, h, 128), torch.empty(NB, h * 128, device="cuda", dtype=bf)
+        for name, L, w in kinds:
+            proj, keys = rnd(NB, L.proj.N), min(ctx, w or ctx)
+            gate = proj[:, L.proj.off["g"]:][:, : h * 128] if "g" in L.proj.off else None
+            splits = max(1, min(32, (6 * sms + NB * kv - 1) // (NB * kv), (keys + (PAGE if w else 0) + 255) // 256))
+            scratch = torch.empty(L.att.decode_scratch(NB, splits), device="cuda")
+            K.add(f"paged decode attention, {name}", f"{NB} x {ctx}, {h}/{kv} heads, 128",
+                  lambda: L.att.decode(q, kc, vc, b, table, gate, o, scratch, eng._counters, splits, st), nbytes=4.0 * NB * keys * kv * 128,
+                  like="paged decode attention (dense)")
+    # ---- selective scan
+    c, ns, sel, N = r.inner, r.state, par.sel, par.proj.N
+    for B, S in ((16, 512), (4, 2048), (1, 8192)):
+        n, b = B * S, _batch([S] * B, [0] * B)
+        proj, x, low, out = rnd(n, N), rnd(n, c), rnd(n, par.x_maps.N), torch.empty(n, c, device="cuda", dtype=bf)
+        dt, sizes = torch.randn(n, c, device="cuda") - 3.0, f"{B} x {S}, {c} channels, {ns} state values"
+        scratch = torch.empty(sel.scratch_floats(B, S), device="cuda")
+        K.add("selective_conv", sizes, lambda: sel.conv(proj, b, False, x), nbytes=4.0 * n * c, like="rope (dense)")
+        K.add("selective_scan", sizes, lambda: sel.scan(proj, x, low, dt, b, S, scratch, out),
+              nbytes=n * (c * 10.0 + 4 * ns) + 8.0 * B * c * ns, like="chunked recurrence + norm + gate")
+        _recurrent_rows(K, H, st, "delta", h, 128, 128, [S] * B, False)
+        _recurrent_rows(K, H, st, "gla", h, 64, 128, [S] * B, False)
+    for T in (1, 16, 64):
+        b = _batch([1] * T, [99] * T)
+        proj, x, low, out = rnd(T, N), rnd(T, c), rnd(T, par.x_maps.N), torch.empty(T, c, device="cuda", dtype=bf)
+        dt = torch.randn(T, c, device="cuda") if T > LOW_RANK_FUSE_ROWS else None
+        sizes = f"{T} tokens, {c} channels, {ns} state values"
+        K.add("selective_conv, one token", sizes, lambda: sel.conv(proj, b, True, x), nbytes=T * c * (4.0 + 24), like="recurrent_decode")
+        K.add("selective_step", sizes, lambda: sel.step(proj, x, low, dt, b, out),
+              nbytes=T * c * (8.0 * ns + 6 + 4 * (dt is not None)) + 2.0 * c * r.dt_rank * (dt is None), like="recurrent_decode")
+        _recurrent_rows(K, H, st, "delta", h, 128, 128, [1] * T, True)
+        _recurrent_rows(K, H, st, "gla", h, 64, 128, [1] * T, True)
+    for T in EXPERT_TOKENS:
+        proj, x, low = rnd(T, N), rnd(T, c), rnd(T, par.x_maps.N)
+        dt, y, z = torch.empty(T, c, device="cuda"), rnd(T, par.out.shape[1]), rnd(T, d)
+        R = par.w_dt.shape[1]
+        for name, xx, ww, oo, like in (
+                ("mixer in", z, par.proj.weight, proj, "gemm (dense bf16)"), ("mixer out, both mixers", y, par.out, z, "gemm (dense bf16)"),
+                ("maps of the scan", x, par.x_maps.weight, low, "gemm (dense bf16), narrow"),
+                ("step sizes", low[:, :R], par.w_dt, dt, "gemm (dense bf16), narrow")):
+            n_out, k_in = ww.shape
+            nb = 2.0 * (n_out * k_in + T * (k_in + n_out * oo.element_size() / 2))
+            K.add(f"{name} (GEMM)", f"{T} x {n_out} x {k_in}", lambda: eng._gemm(xx, ww, out=oo), nbytes=nb, flops=2.0 * T * n_out * k_in,
+                  like=like)
+            x2, o2 = rnd(T, k_in), torch.empty(T, n_out, device="cuda", dtype=bf)
+            K.add(like, f"{T} x {n_out} x {k_in}", lambda: F.gemm(x2, ww, out=o2), nbytes=2.0 * (n_out * k_in + T * (k_in + n_out)),
+                  flops=2.0 * T * n_out * k_in)
+    # ---- experts, output
+    for T in EXPERT_TOKENS:
+        hid, _ = _expert_rows(K, H, C, rnd, eng, par, T)
+    for T in (1, 64):
+        x, lg, lb = rnd(T, d), torch.empty(T, 32000, device="cuda"), torch.empty(T, 32000, device="cuda", dtype=bf)
+        nb = 2.0 * (32000 * d + T * (d + 64000))
+        K.add("soft-capped output (GEMM)", f"{T} x 32000 x {d}", lambda: eng._gemm(x, eng.head, out=lg, cap=30.0), nbytes=nb,
+              flops=2.0 * T * 32000 * d, like="gemm (dense bf16)")
+        K.add("gemm (dense bf16)", f"{T} x 32000 x {d}", lambda: F.gemm(x, eng.head, out=lb), nbytes=nb, flops=2.0 * T * 32000 * d)
+    native.check_status("cuda")
+    return K.rows
+
+
 def run_lebedra_kernels(peaks: dict, width: int = 2048) -> list[dict]:
     """Latent attention (latents of 512, heads of 128 + 64 rotated), routed experts and the norms around them."""
     from ..infer.hybrid import HybridEngine
@@ -232,43 +379,10 @@ def run_lebedra_kernels(peaks: dict, width: int = 2048) -> list[dict]:
         K.add("gemm_decode", f"{NB} x {N // 4} x {m.dim * 4}", lambda: H.gemm_decode(x, w, y, 0, 0, 1.0, st),
               nbytes=2.0 * (w.numel() + x.numel() + y.numel()))
     # ---- experts
-    route = (e.experts, e.top, e.groups, e.keep)
-    i32 = dict(device="cuda", dtype=torch.int32)
-    f, gen = e.ff, torch.Generator().manual_seed(5)
-    for T in (1, 16, 64, 1024, 8192):
-        pairs, tile = T * e.top, eng._expert_tile(T, e)
-        z = torch.randn(T, e.experts, generator=gen).cuda()
-        idx, slot, row = (torch.empty(T, e.top, **i32) for _ in range(3))
-        wt, off, cnt = torch.empty(T, e.top, device="cuda"), torch.empty(e.experts, **i32), torch.empty(1, **i32)
-        tiles = torch.empty(min(pairs, e.experts + pairs // tile), 3, **i32)
-        plan = (idx, wt, slot, eng._expert_counts, off, tiles, cnt)
-        x, hid, a, y = rnd(pairs, d), rnd(T, d), rnd(pairs, f), rnd(pairs, d)
-        sizes = f"{T} tokens, {e.top} of {e.experts}, {d} x {f}"
-        K.add("expert_select", sizes, lambda: H.expert_select(z, L.correction, route, tile, *plan), nbytes=4.0 * T * e.experts,
-              like="moe_route (training)")
-        probs, psum, lg = torch.empty(T, e.experts, device="cuda"), torch.zeros(e.experts, device="cuda"), z.to(bf)
-        cn = torch.zeros(e.experts, **i32)
-        K.add("moe_route (training)", sizes, lambda: C.moe_route(lg, e.experts, probs, idx, slot, wt, cn, psum), nbytes=2.0 * T * e.experts)
-        H.expert_select(z, L.correction, route, tile, *plan)
-        used = int((torch.bincount(idx.flatten().long(), minlength=e.experts) > 0).sum())
-        K.add("expert_gather", sizes, lambda: H.expert_gather(hid, route, *plan, x, row), nbytes=2.0 * d * (T + pairs), like="rope (dense)")
-        K.add("experts in (gate, up)", sizes, lambda: H.gemm_tiles(x, L.w_in, a, tiles, cnt, tile, f, f, L.act, st),
-              nbytes=2.0 * (used * 2 * f * d + pairs * (d + f)), flops=4.0 * pairs * f * d, like="gemm (dense bf16)")
-        K.add("experts out (down)", sizes, lambda: H.gemm_tiles(a, L.w_out, y, tiles, cnt, tile, 0, 0, L.act, st),
-              nbytes=2.0 * (used * f * d + pairs * (d + f)), flops=2.0 * pairs * f * d, like="gemm (dense bf16)")
-        for N, Kd in ((2 * f * e.top, d), (d, f * e.top)):         # the dense layer of the same width
-            xx, ww, o1 = rnd(T, Kd), rnd(N, Kd), torch.empty(T, N, device="cuda", dtype=bf)
-            K.add("gemm (dense bf16)", f"{T} x {N} x {Kd}", lambda: F.gemm(xx, ww, out=o1), nbytes=2.0 * (N * Kd + T * (N + Kd)),
-                  flops=2.0 * T * N * Kd)
-        xs, w32, hh = torch.randn(T, d, device="cuda"), torch.ones(d, device="cuda"), rnd(T, d)
-        K.add("expert_norm", f"{T} x {d}, {e.top} outputs", lambda: H.expert_norm(y, row, wt, w32, xs, None, hh, 1e-6, 0.5),
-              nbytes=T * d * (2.0 * e.top + 10), like="rmsnorm + residual (dense)")
-        K.add("norm + residual", f"{T} x {d}", lambda: H.sandwich_norm(hh, None, None, None, w32, xs, None, x[:T], 1e-6, 0.5),
-              nbytes=T * d * 12.0, like="rmsnorm + residual (dense)")
-        g, res = torch.ones(d, device="cuda", dtype=bf), rnd(T, d)
-        K.add("rmsnorm + residual (dense)", f"{T} x {d}", lambda: F.rmsnorm(hh, g, 1e-6, res), nbytes=T * d * 8.0)
+    for T in EXPERT_TOKENS:
+        hid, hh = _expert_rows(K, H, C, rnd, eng, L, T)
         # ---- token side and router
-        n, ids = cfg.token_side, torch.zeros(T, **i32)
+        n, ids = cfg.token_side, torch.zeros(T, device="cuda", dtype=torch.int32)
         sg = torch.empty(T, n, device="cuda", dtype=bf)
         K.add("side gate", f"{T} x {n} x {d}", lambda: H.gemm_decode(hid, L.side_gate, sg, 0, 0, 1.0, st, (0, 0.0, 0.0), L.side_embed, ids),
               nbytes=2.0 * (n * d + T * (d + 2 * n)), flops=2.0 * T * n * d, like="gemm (dense bf16), narrow")
@@ -286,6 +400,8 @@ def run_lebedra_kernels(peaks: dict, width: int = 2048) -> list[dict]:
 def run_kernels(peaks: dict, width: int = 2048, design: str = "teganex") -> list[dict]:
     if design == "lebedra":
         return run_lebedra_kernels(peaks, width)
+    if design == "dogozen":
+        return run_dogozen_kernels(peaks, width)
     from ..ops import functional as F, native
 
     H, C, st = native.require_hybrid(), native.require(), native.status_word("cuda")
@@ -320,16 +436,17 @@ def run_kernels(peaks: dict, width: int = 2048, design: str = "teganex") -> list
         kc, vc = rnd(pages, PAGE, kv, dk), rnd(pages, PAGE, kv, dv)
         b = _batch([S] * B, [0] * B)
         q, gate, o = rnd(B * S, h, dk), rnd(B * S, h), torch.empty(B * S, h * dv, device="cuda", dtype=bf)
+        proj, ones = rnd(B * S, h * dk + kv * (dk + dv)), torch.ones(dk, device="cuda")
+        att = H.Attention({"heads": h, "kv_heads": kv, "dk": dk, "dv": dv, "k_off": h * dk, "v_off": (h + kv) * dk, "norm_dim": dk,
+                           "scale": dk ** -0.5}, {"q_gamma": ones, "k_gamma": ones})
         fl = 2.0 * B * h * (S * (S + 1) / 2) * (dk + dv)
         K.add("gated paged prefill attention", f"{B} x {S}, {h}/{kv} heads, {dk} / {dv}",
-              lambda: H.paged_attn_prefill(q, kc, vc, b, table, gate, o, S, dk ** -0.5, st), flops=fl, like="paged prefill attention (dense)")
+              lambda: att.prefill(q, kc, vc, b, table, gate, o, S, st), flops=fl, like="paged prefill attention (dense)")
         if dk == dv:
             o3 = o.view(B * S, h, dv)
             K.add("paged prefill attention (dense)", f"{B} x {S}, {h}/{kv} heads, {dk}",
                   lambda: C.flash_attn_paged_prefill(q, kc, vc, table, b[0], b[1], o3, S, dk ** -0.5, st), flops=fl)
-        proj, ones = rnd(B * S, h * dk + kv * (dk + dv)), torch.ones(dk, device="cuda")
-        K.add("qk_norm_append", f"{B * S} tokens, {h}/{kv} heads, {dk} / {dv}",
-              lambda: H.qk_norm_append(proj, 0, h * dk, (h + kv) * dk, ones, ones, b, table, q, kc, vc, 1e-6),
+        K.add("attn_prep, norm", f"{B * S} tokens, {h}/{kv} heads, {dk} / {dv}", lambda: att.prep(proj, b, table, q, kc, vc),
               nbytes=4.0 * B * S * (h * dk + kv * (dk + dv)), like="rope (dense)")
     qkv, pos = rnd(B * S, h + 2 * kv, 128), torch.arange(S, device="cuda", dtype=torch.int32).repeat(B)
     K.add("rope (dense)", f"{B * S} tokens, {h}/{kv} heads, 128", lambda: C.rope(qkv[:, : h + kv], pos, 10000.0, False),
@@ -343,10 +460,11 @@ def run_kernels(peaks: dict, width: int = 2048, design: str = "teganex") -> list
             kc, vc = rnd(pages, PAGE, kv, dk), rnd(pages, PAGE, kv, dv)
             q, gate, o = rnd(NB, h, dk), rnd(NB, h), torch.empty(NB, h * dv, device="cuda", dtype=bf)
             b = _batch([1] * NB, [ctx - 1] * NB)
+            att = H.Attention({"heads": h, "kv_heads": kv, "dk": dk, "dv": dv, "scale": dk ** -0.5}, {})
             scratch, cnt = torch.empty(NB * h * splits * (dv + 2), device="cuda"), torch.zeros(NB * kv, device="cuda", dtype=torch.int32)
             nb = 2.0 * NB * ctx * kv * (dk + dv)
             K.add("gated paged decode attention", f"{NB} x {ctx}, {h}/{kv} heads, {dk} / {dv}",
-                  lambda: H.paged_attn_decode(q, kc, vc, b, table, gate, o, scratch, cnt, splits, dk ** -0.5, st), nbytes=nb,
+                  lambda: att.decode(q, kc, vc, b, table, gate, o, scratch, cnt, splits, st), nbytes=nb,
                   like="paged decode attention (dense)")
             if dk == dv:
                 o3 = o.view(NB, h, dv)
@@ -372,7 +490,7 @@ def main(argv=None) -> int:
     ap.add_argument("--kernels", action="store_true")
     ap.add_argument("--models", action="store_true")
     ap.add_argument("--width", type=int, default=2048)
-    ap.add_argument("--design", default="teganex", choices=["teganex", "lebedra"])
+    ap.add_argument("--design", default="teganex", choices=["teganex", "lebedra", "dogozen"])
     a = ap.parse_args(argv)
     peaks = {}
     path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
