@@ -662,7 +662,7 @@ struct Selective {
   mb::SelectiveInputs inputs(const Tensor& proj, const Tensor& x, const Tensor& low, bool f32, int64_t rows) const {
     mb::SelectiveInputs in = inputs(proj, f32, rows);
     chk_rows(x, f32, rows, s.inner, "x");
-    chk_rows(low, f32, rows, std::max({b_off + s.state, c_off + s.state, (s.rank + 7) / 8 * 8}), "low");
+    chk_rows(low, f32, rows, std::max({std::max(b_off, c_off) + (s.state + 7) / 8 * 8, (s.rank + 7) / 8 * 8}), "low");
     in.x = x.data_ptr();
     in.ld_x = x.stride(0);
     in.low = low.data_ptr();
@@ -677,18 +677,20 @@ struct Selective {
     c10::cuda::CUDAGuard guard(x.device());
     mb::selective_conv(f32, s, inputs(proj, f32, rb.rows), rb, one_token, x.data_ptr(), x.stride(0), cur_stream());
   }
-  int64_t scratch_floats(int64_t n_seq, int64_t max_q) const { return mb::selective_scratch(s, (int)n_seq, (int)max_q); }
+  int64_t scratch_floats(int64_t n_seq, int64_t rows, int64_t max_q) const {
+    return mb::selective_scratch(s, (int)n_seq, (int)rows, (int)max_q);
+  }
   void scan(const Tensor& proj, const Tensor& x, const Tensor& low, const Tensor& dt, const std::vector<Tensor>& batch, int64_t max_q,
-            Tensor& scratch, Tensor& out) const {
+            Tensor& scratch, Tensor& out, const OptTensor& status) const {
     const auto rb = ragged(batch);
     const bool f32 = is_f32(out, "out");
     chk_rows(out, f32, rb.rows, s.inner, "out");
     chk_rows(dt, true, rb.rows, s.inner, "dt");
     chk_c(scratch, F32, "scratch");
-    TORCH_CHECK(scratch.numel() >= scratch_floats(rb.n_seq, max_q), "scan: scratch");
+    TORCH_CHECK(scratch.numel() >= scratch_floats(rb.n_seq, rb.rows, max_q), "scan: scratch");
     c10::cuda::CUDAGuard guard(out.device());
     mb::selective_scan(f32, s, inputs(proj, x, low, f32, rb.rows), rb, (int)max_q, dt.data_ptr<float>(), dt.stride(0),
-                       scratch.data_ptr<float>(), out.data_ptr(), out.stride(0), cur_stream());
+                       scratch.data_ptr<float>(), out.data_ptr(), out.stride(0), status_ptr(status), cur_stream());
   }
   // One token per sequence; dt null: computed from the first columns of low.
   void step(const Tensor& proj, const Tensor& x, const Tensor& low, const OptTensor& dt, const std::vector<Tensor>& batch,

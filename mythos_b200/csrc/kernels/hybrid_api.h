@@ -255,9 +255,9 @@ void selective_conv(bool f32, const SelectiveSpec& s, const SelectiveInputs& in,
 // Prompts and portions; dt [rows, ld_dt]: pre-activations without bias. Long portions are cut into chunks that run side
 // by side: a first kernel forms every chunk's own state and summed step sizes, the second starts each chunk from
 // the states before it. Scratch: selective_scratch floats.
-long long selective_scratch(const SelectiveSpec& s, int n_seq, int max_q);
+long long selective_scratch(const SelectiveSpec& s, int n_seq, int rows, int max_q);
 void selective_scan(bool f32, const SelectiveSpec& s, const SelectiveInputs& in, const RaggedBatch& rb, int max_q,
-                    const float* dt, long long ld_dt, float* scratch, void* out, long long ldo, cudaStream_t stream);
+                    const float* dt, long long ld_dt, float* scratch, void* out, long long ldo, int* status, cudaStream_t stream);
 // One token per sequence. The pre-activations come from dt, or from the dt columns of `low` and w_dt [inner, ld_w].
 void selective_step(bool f32, const SelectiveSpec& s, const SelectiveInputs& in, const RaggedBatch& rb, const float* dt,
                     long long ld_dt, const void* w_dt, long long ld_w, void* out, long long ldo, cudaStream_t stream);

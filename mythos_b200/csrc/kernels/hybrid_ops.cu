@@ -275,93 +275,131 @@ __global__ void attn_prep_kernel(const T* __restrict__ proj, long long ld, HeadP
   }
 }
 
+__device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
 // bf16 form for widths that are multiples of 8 up to 128: 16 lanes per (token, head slot), 16-byte accesses, `tokens`
-// tokens per block, whose angles are evaluated once for all heads.
-constexpr int AP_THREADS = 256;
+// tokens per block. What depends on the token alone (page row, query factor, angles) is evaluated once for all heads.
+constexpr int AP_THREADS = 256, AP_TOKENS = 16;
 __global__ void __launch_bounds__(AP_THREADS)
-attn_prep8_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, HeadPrep p, RaggedBatch rb,
-                  const int* __restrict__ block_table, int table_stride, int page_size, int tokens,
-                  __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache) {
-  extern __shared__ float2 cs_all[];         // [tokens][rot / 2]
-  const int l = threadIdx.x & 15, slots = p.heads + (p.k_off < 0 ? 0 : 2 * p.kv_heads), half = p.rot / 2;
-  const int t0 = blockIdx.x * tokens, nt = min(tokens, rb.rows - t0);
-  if (half > 0) {
-    for (int i = threadIdx.x; i < nt * half; i += AP_THREADS) cs_all[i] = turn(rb.pos[t0 + i / half], p.turns[i % half]);
-    __syncthreads();
-  }
-  const int total = nt * slots;
+attn_prep8_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, const __grid_constant__ HeadPrep p,
+                  const __grid_constant__ RaggedBatch rb, const int* __restrict__ block_table, int table_stride, int page_size,
+                  int tokens, __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ k_cache,
+                  __nv_bfloat16* __restrict__ v_cache) {
+  extern __shared__ __align__(16) float2 cs_all[];         // [tokens][rot / 2], pair 8 a + b at place b * (rot / 16) + a
+  __shared__ int s_page_row[AP_TOKENS];                    // row of the pages, or -1
+  __shared__ float s_factor[AP_TOKENS];
+  const int l = threadIdx.x & 15, c = l * 8, slots = p.heads + (p.k_off < 0 ? 0 : 2 * p.kv_heads), half = p.rot / 2;
+  const int t0 = blockIdx.x * tokens, nt = min(tokens, rb.rows - t0), total = nt * slots;
+  const float per = 1.f / (float)slots;
+  struct Item {                                            // one head of one token
+    int tl, j, width;
+    bool live, is_q, is_v;
+    const __nv_bfloat16* src;
+  };
+  auto item = [&](int w) {
+    Item it;
+    it.live = w < total;
+    if (!it.live) w = 0;
+    it.tl = (int)(((float)w + 0.5f) * per);                // exact: w is far below 2^23
+    const int hs = w - it.tl * slots;
+    it.is_q = hs < p.heads;
+    it.is_v = hs >= p.heads + p.kv_heads;
+    it.j = it.is_q ? hs : (it.is_v ? hs - p.heads - p.kv_heads : hs - p.heads);
+    it.width = it.is_v ? p.dv : p.dk;
+    it.src = proj + (long long)(t0 + it.tl) * ld + (it.is_q ? p.q_off : (it.is_v ? p.v_off : p.k_off)) + it.j * it.width;
+    it.live = it.live && c < it.width;
+    return it;
+  };
   // both halves of a warp run the same number of iterations: the shuffles need the whole warp
-  for (int w0 = (threadIdx.x >> 4) & ~1; w0 < total; w0 += AP_THREADS >> 4) {
-    const int w = w0 + ((threadIdx.x >> 4) & 1);
-    const bool live = w < total;
-    const int tl = live ? w / slots : 0, hs = live ? w % slots : 0, t = t0 + tl;
-    const bool is_q = hs < p.heads, is_v = hs >= p.heads + p.kv_heads;
-    const int width = is_v ? p.dv : p.dk, j = is_q ? hs : (is_v ? hs - p.heads - p.kv_heads : hs - p.heads), c = l * 8;
-    const bool on = live && c < width;
-    const __nv_bfloat16* src = proj + (long long)t * ld + (is_q ? p.q_off : (is_v ? p.v_off : p.k_off)) + j * width;
-    const float* bias = is_q ? p.q_bias : (is_v ? p.v_bias : p.k_bias);
-    if (bias) bias += j * width;
-    const float* gamma = is_q ? p.q_gamma : p.k_gamma;
-    float f[8];
-    float ss = 0.f;
-    if (on) {
-      unpack8(ldg8(src, c), f);
-      if (bias) {
+  const int first = (threadIdx.x >> 4) & ~1, side = (threadIdx.x >> 4) & 1;
+  Item next = item(first + side);
+  bf16x8 raw_next{};
+  if (next.live) raw_next = ldg8(next.src, c);
+  for (int i = threadIdx.x; i < nt; i += AP_THREADS) {
+    const int pos = rb.pos[t0 + i];
+    const int page = block_table[(long long)rb.row_seq[t0 + i] * table_stride + pos / page_size];
+    s_page_row[i] = page < 0 ? -1 : page * page_size + pos % page_size;
+    s_factor[i] = query_factor(p, pos);
+  }
+  const bool spread = half % 8 == 0;                       // neighbouring lanes then read neighbouring entries
+  for (int i = threadIdx.x; i < nt * half; i += AP_THREADS) {
+    const int tl = i / half, k = i - tl * half;
+    cs_all[tl * half + (spread ? (k & 7) * (half >> 3) + (k >> 3) : k)] = turn(rb.pos[t0 + tl], p.turns[k]);
+  }
+  __syncthreads();
+  for (int w0 = first; w0 < total; w0 += AP_THREADS >> 4) {
+    const Item it = next;
+    const bf16x8 raw = raw_next;
+    next = item(w0 + (AP_THREADS >> 4) + side);            // the next item's values are on their way meanwhile
+    if (next.live) raw_next = ldg8(next.src, c);
+    const float* bias = it.is_q ? p.q_bias : (it.is_v ? p.v_bias : p.k_bias);
+    const float* gamma = it.is_q ? p.q_gamma : p.k_gamma;
+    float f[8], ss = 0.f;
+    unpack8(raw, f);
+    if (bias) bias += it.j * it.width;
+    if (bias && it.live) {
+      float g[8];
+      load8(bias + c, g);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] += bias[c + i];
+      for (int i = 0; i < 8; ++i) f[i] += g[i];
+    }
+    float r = 1.f;
+    if (p.norm_dim > 0) {
+      if (it.live) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) ss = fmaf(f[i], f[i], ss);
       }
 #pragma unroll
-      for (int i = 0; i < 8; ++i) ss = fmaf(f[i], f[i], ss);
+      for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      r = rsqrtf(__fdividef(ss, (float)p.norm_dim) + p.eps);
     }
+    if (!it.live) continue;
+    if (!it.is_v) {
+      const float q = it.is_q ? r * s_factor[it.tl] : r;   // the factor commutes with the rotation
+      if (gamma) {
+        float g[8];
+        load8(gamma + c, g);
 #pragma unroll
-    for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if (!on) continue;
-    const int pos = rb.pos[t];
-    if (!is_v) {
-      const float r = p.norm_dim > 0 ? 1.f / sqrtf(ss / (float)p.norm_dim + p.eps) : 1.f;
+        for (int i = 0; i < 8; ++i) f[i] *= q * g[i];
+      } else {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] *= gamma ? r * gamma[c + i] : r;
+        for (int i = 0; i < 8; ++i) f[i] *= q;
+      }
       if (c < p.rot) {
         // column i < half turns with i + half; the partner's value is read again
-        float g[8];
-        if (half % 8 == 0) {
-          const int at = c < half ? c + half : c - half;
-          unpack8(ldg8(src, at), g);
+        const float2* cs = cs_all + it.tl * half;
+        if (spread) {
+          const int at = c < half ? c + half : c - half, k = (c < half ? c : at) >> 3, lanes = half >> 3;
+          float g[8];
+          unpack8(ldg8(it.src, at), g);
+          const float sign = c < half ? -q : q;
 #pragma unroll
-          for (int i = 0; i < 8; ++i) g[i] = (g[i] + (bias ? bias[at + i] : 0.f)) * (gamma ? r * gamma[at + i] : r);
+          for (int i = 0; i < 8; ++i) {
+            const float v = (g[i] + (bias ? bias[at + i] : 0.f)) * (gamma ? sign * gamma[at + i] : sign);
+            const float2 t = cs[i * lanes + k];
+            f[i] = f[i] * t.x + v * t.y;
+          }
         } else {
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             const int col = c + i;
             if (col < p.rot) {
-              const int at = col < half ? col + half : col - half;
-              g[i] = (__bfloat162float(src[at]) + (bias ? bias[at] : 0.f)) * (gamma ? r * gamma[at] : r);
+              const int at = col < half ? col + half : col - half, k = col < half ? col : at;
+              const float v = (__bfloat162float(it.src[at]) + (bias ? bias[at] : 0.f)) * (gamma ? q * gamma[at] : q);
+              f[i] = f[i] * cs[k].x + (col < half ? -v : v) * cs[k].y;
             }
           }
         }
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          const int col = c + i;
-          if (col < p.rot) {
-            const float2 cs = cs_all[tl * half + (col < half ? col : col - half)];
-            f[i] = col < half ? f[i] * cs.x - g[i] * cs.y : f[i] * cs.x + g[i] * cs.y;
-          }
-        }
-      }
-      if (is_q && p.temp_coef != 0.f) {
-        const float q = query_factor(p, pos);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] *= q;
       }
     }
     const bf16x8 out = pack8(f);
-    if (is_q) {
-      stg8(q_out, ((long long)t * p.heads + j) * width + c, out);
-    } else {
-      const int page = block_table[(long long)rb.row_seq[t] * table_stride + pos / page_size];
-      if (page >= 0)
-        stg8(is_v ? v_cache : k_cache, (((long long)page * page_size + pos % page_size) * p.kv_heads + j) * width + c, out);
-    }
+    const int row = s_page_row[it.tl];
+    if (it.is_q) stg8(q_out, ((long long)(t0 + it.tl) * p.heads + it.j) * it.width + c, out);
+    else if (row >= 0) stg8(it.is_v ? v_cache : k_cache, ((long long)row * p.kv_heads + it.j) * it.width + c, out);
   }
 }
 
@@ -580,9 +618,10 @@ void attn_prep(bool f32, const void* proj, long long ld, const HeadPrep& p, cons
   if (!f32 && p.dk % 8 == 0 && p.dv % 8 == 0 && p.dk <= 128 && p.dv <= 128 &&
       ((ld | p.q_off | (kv ? p.k_off | p.v_off : 0)) & 7) == 0 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0) {
     // enough head slots for a few rounds of a block's 16 groups, but no fewer blocks than SMs
-    int tokens = (64 + slots - 1) / slots;
-    const int most = rb.rows / (2 * sm_count());
+    int tokens = (128 + slots - 1) / slots;
+    const int most = rb.rows / (4 * sm_count());
     if (tokens > most) tokens = most;
+    if (tokens > AP_TOKENS) tokens = AP_TOKENS;
     if (tokens < 1) tokens = 1;
     attn_prep8_kernel<<<(rb.rows + tokens - 1) / tokens, AP_THREADS, tokens * (p.rot / 2) * 8, stream>>>(
         (const __nv_bfloat16*)proj, ld, p, rb, block_table, table_stride, page_size, tokens, (__nv_bfloat16*)q_out,

@@ -148,23 +148,30 @@ __device__ __forceinline__ void merge_and_finish(const float* s_m, const float* 
   __syncthreads();
   if (!*s_last) return;
   __threadfence();
+  // one warp per head forms the weights of the splits (at most 32, one per lane); the accumulators' memory is free now
+  float* w = const_cast<float*>(s_acc);               // [G][32]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int g = warp; g < G; g += blockDim.x >> 5) {
+    const float* base = scratch + ((long long)b * heads + h0 + g) * splits * stride + D;
+    const float ms = lane < splits ? base[lane * stride] : -INFINITY, ls = lane < splits ? base[lane * stride + 1] : 0.f;
+    const float M = warp_max(ms);
+    const float e = ms == -INFINITY ? 0.f : exp2f(ms - M);
+    float L = warp_sum(e == 0.f ? 0.f : e * ls);
+    if (ex.sink) L += exp2f(ex.sink[h0 + g] * 1.4426950408889634f - M);
+    w[g * 32 + lane] = L > 0.f ? e / L * ex.out_scale : 0.f;
+  }
+  __syncthreads();
   const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(ex.gate);
   for (int idx = threadIdx.x; idx < G * D; idx += blockDim.x) {
     const int g = idx / D, d = idx % D;
     if (d >= dv) continue;
-    const float* base = scratch + ((long long)b * heads + h0 + g) * splits * stride;
-    float M = -INFINITY;
-    for (int s = 0; s < splits; ++s) M = fmaxf(M, base[s * stride + D]);
-    float L = 0.f, A = 0.f;
+    const float* base = scratch + ((long long)b * heads + h0 + g) * splits * stride + d;
+    float y = 0.f;
+#pragma unroll 8
     for (int s = 0; s < splits; ++s) {
-      const float ms = base[s * stride + D];
-      if (ms == -INFINITY) continue;
-      const float w = exp2f(ms - M);
-      L += w * base[s * stride + D + 1];
-      A += w * base[s * stride + d];
+      const float v = base[s * stride], ws = w[g * 32 + s];
+      y += ws == 0.f ? 0.f : ws * v;                  // an empty split's accumulator may hold anything
     }
-    if (ex.sink) L += exp2f(ex.sink[h0 + g] * 1.4426950408889634f - M);
-    float y = L > 0.f ? A / L * ex.out_scale : 0.f;
     if (gate) {
       const __nv_bfloat16* gp = gate + b * ex.ld_gate;
       y /= 1.f + expf(-__bfloat162float(ex.gate_channels ? gp[(h0 + g) * dv + d] : gp[h0 + g]));
@@ -778,7 +785,7 @@ void paged_attn_decode(const void* q, const void* k_cache, const void* v_cache, 
   if (q_tok_stride <= 0) q_tok_stride = (long long)heads * head_dim;
   MB_REQUIRE(q_tok_stride % 8 == 0, "paged_attn_decode: query token stride must be a multiple of 8 elements");
   MB_REQUIRE(heads % kv_heads == 0, "paged_attn_decode: heads must be a multiple of kv_heads");
-  MB_REQUIRE(splits >= 1, "paged_attn_decode: splits must be positive");
+  MB_REQUIRE(splits >= 1 && splits <= 32, "paged_attn_decode: 1 to 32 splits");
   if (batch == 0) return;
   const int G = heads / kv_heads;
   const dim3 grid(batch, kv_heads, splits);
@@ -865,7 +872,7 @@ void paged_attn_decode_int8(const void* q, const void* k_cache, const void* v_ca
   if (q_tok_stride <= 0) q_tok_stride = (long long)heads * head_dim;
   MB_REQUIRE(q_tok_stride % 8 == 0, "paged_attn_decode_int8: query token stride must be a multiple of 8 elements");
   MB_REQUIRE(heads % kv_heads == 0, "paged_attn_decode_int8: heads must be a multiple of kv_heads");
-  MB_REQUIRE(splits >= 1, "paged_attn_decode_int8: splits must be positive");
+  MB_REQUIRE(splits >= 1 && splits <= 32, "paged_attn_decode_int8: 1 to 32 splits");
   if (batch == 0) return;
   const int G = heads / kv_heads;
   const dim3 grid(batch, kv_heads, splits);

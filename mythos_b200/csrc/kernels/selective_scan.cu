@@ -3,7 +3,8 @@
 //
 //   selective_conv  short causal convolution + silu of the channels, and its state
 //   selective_scan  prompts and portions: a thread owns NR state values of a channel in registers and walks the
-//                   tokens of a chunk; B and C of a tile of tokens lie in shared memory and are read by all channels.
+//                   tokens of a chunk; tiles of inputs pass through shared memory by TMA, B and C of a token are read
+//                   by all channels.
 //                   Chunks of a long portion run side by side: kernel 1 forms each chunk's state from zero and the sum
 //                   of its step sizes (the decay over a chunk is exp(A sum dt)), kernel 2 composes the states before
 //                   a chunk, walks it again and reads out.
@@ -12,6 +13,8 @@
 //
 // Step sizes, decays, states and the read-out are fp32 in both activation types. A is stored times log2(e), so a
 // decay is one exp2.
+#include <type_traits>
+
 #include "common.cuh"
 #include "host_util.h"
 #include "hybrid_api.h"
@@ -22,9 +25,11 @@ namespace mb {
 namespace {
 
 constexpr int SS_THREADS = 128;
-constexpr int SS_GROUP = 4;            // tokens whose inputs are loaded together
-constexpr int SS_TILE = 32;            // tokens whose B and C are staged together (fewer for wide states)
-constexpr int SS_TILE_VALUES = 4096;   // at most this many values of B (and of C) in shared memory
+constexpr int SS_TILE = 16;            // tokens of a tile (fewer for wide states)
+constexpr int SS_BLOCKS = 4;           // blocks of a scan that fit into an SM
+constexpr int SS_STAGES = 3;           // tiles in flight
+constexpr int SS_GROUP = 4;            // tokens handled together
+constexpr int SS_TILE_VALUES = 2048;   // at most this many values of B (and of C) in a tile
 constexpr int SS_CHUNK = 64;           // shortest chunk
 
 // A channel's state values lie on `lanes` neighbouring threads, nr on each.
@@ -39,8 +44,13 @@ StateMap state_map(int state) {
 }
 
 // ln(1 + e) for 0 <= e <= 1 as 2 artanh(e / (2 + e)), series in t^2 <= 1/9.
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ float log1p_unit(float e) {
-  const float t = __fdividef(e, 2.f + e), t2 = t * t;
+  const float t = e * fast_rcp(2.f + e), t2 = t * t;
   float p = fmaf(t2, 1.f / 15.f, 1.f / 13.f);
   p = fmaf(p, t2, 1.f / 11.f);
   p = fmaf(p, t2, 1.f / 9.f);
@@ -50,7 +60,9 @@ __device__ __forceinline__ float log1p_unit(float e) {
   p = fmaf(p, t2, 1.f);
   return 2.f * t * p;
 }
-__device__ __forceinline__ float softplus_fast(float z) { return fmaxf(z, 0.f) + log1p_unit(expf(-fabsf(z))); }
+__device__ __forceinline__ float softplus_fast(float z) { return fmaxf(z, 0.f) + log1p_unit(fast_exp2(-1.4426950408889634f * fabsf(z))); }
+// z / (1 + e^-z)
+__device__ __forceinline__ float silu_fast(float z) { return z * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * z)); }
 
 template <int V>
 __device__ __forceinline__ void load_v(const float* p, float (&f)[V]) {
@@ -69,6 +81,11 @@ template <int V>
 __device__ __forceinline__ void load_v(const __nv_bfloat16* p, float (&f)[V]) {
   if constexpr (V == 8) {
     unpack8(*reinterpret_cast<const bf16x8*>(p), f);
+  } else if constexpr (V == 4) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.y));
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
   } else {
 #pragma unroll
     for (int i = 0; i < V; ++i) f[i] = __bfloat162float(p[i]);
@@ -86,8 +103,8 @@ __device__ __forceinline__ void store_v(float* p, const float (&f)[V]) {
 }
 template <int V>
 __device__ __forceinline__ void store_v(__nv_bfloat16* p, const float (&f)[V]) {
-  if constexpr (V == 8) {
-    *reinterpret_cast<bf16x8*>(p) = pack8(f);
+  if constexpr (V == 4) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
   } else {
 #pragma unroll
     for (int i = 0; i < V; ++i) p[i] = __float2bfloat16(f[i]);
@@ -95,80 +112,110 @@ __device__ __forceinline__ void store_v(__nv_bfloat16* p, const float (&f)[V]) {
 }
 
 // ---------------------------------------------------------------------------------------------
-// V channels and SC_ROWS neighbouring rows per thread, so that a row's input is read about twice and not once per tap.
-// TAPS: number of taps, weights held in registers (0: any number, weights read from the cache).
-constexpr int SC_ROWS = 4;
+// V channels of SC_ROWS neighbouring rows per thread; the rows' inputs pass through registers (TAPS > 0), so each is read
+// once. TAPS: number of taps, 0: any number, read from the cache.
+constexpr int SC_ROWS = 16, SC_STEP = 4;
+template <typename T>
+__device__ __forceinline__ float silu_t(float z) {
+  if constexpr (sizeof(T) == 2) return silu_fast(z);
+  else return silu_f(z);
+}
 template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(256)
 selective_conv_kernel(SelectiveSpec s, SelectiveInputs in, RaggedBatch rb, T* __restrict__ x, long long ldx) {
+  __shared__ int s_index[SC_ROWS];                 // row within its sequence's portion
+  __shared__ long long s_state[SC_ROWS];           // its sequence's convolution state, -1: it has no earlier tokens
   const long long c = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
   const int r0 = blockIdx.y * SC_ROWS, n = min(SC_ROWS, rb.rows - r0), taps = TAPS > 0 ? TAPS : s.taps;
+  if (threadIdx.x < n) {
+    const int b = rb.row_seq[r0 + threadIdx.x], lo = rb.cu_q[b];
+    s_index[threadIdx.x] = r0 + threadIdx.x - lo;
+    s_state[threadIdx.x] = rb.kv_lens[b] > rb.cu_q[b + 1] - lo ? (long long)rb.slots[b] * (taps - 1) * s.inner : -1;
+  }
+  __syncthreads();
   if (c >= ldx) return;
   if (c >= s.inner) {                              // padding (V = 1)
     for (int r = 0; r < n; ++r) stf(x + (r0 + r) * ldx + c, 0.f);
     return;
   }
-  float acc[SC_ROWS][V], wr[TAPS > 0 ? TAPS : 1][V];
-  if constexpr (TAPS > 0) {
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) load_v<V>(in.conv_w + (long long)j * s.inner + c, wr[j]);
-  }
-  int lo[SC_ROWS];
-#pragma unroll
-  for (int r = 0; r < SC_ROWS; ++r) {
-    lo[r] = r < n ? rb.cu_q[rb.row_seq[r0 + r]] : 0x7fffffff;
-    load_v<V>(in.conv_b + c, acc[r]);
-  }
-  const T* col = static_cast<const T*>(in.proj) + in.x_off + c;
-  auto add = [&](int j, const float (&v)[V], float (&a)[V]) {   // input v, j tokens before the current one
-    if constexpr (TAPS > 0) {
-#pragma unroll
-      for (int k = 0; k < TAPS; ++k)
-        if (k == j)
-#pragma unroll
-          for (int i = 0; i < V; ++i) a[i] = fmaf(wr[TAPS - 1 - k][i], v[i], a[i]);
+  const T* col = static_cast<const T*>(in.proj) + (long long)r0 * in.ld + in.x_off + c;
+  T* dst = x + (long long)r0 * ldx + c;
+  const float* w = in.conv_w + c;
+  float bias[V];
+  load_v<V>(in.conv_b + c, bias);
+  // inputs j tokens before row r that lie before its portion: from the state, zeros before the start
+  auto early = [&](int r, int j, float (&v)[V]) {
+    const long long st = s_state[r];
+    if (st >= 0) {
+      load_v<V>(in.conv_state + st + (long long)(taps - 1 + s_index[r] - j) * s.inner + c, v);
     } else {
-      float w[V];
-      load_v<V>(in.conv_w + (long long)(taps - 1 - j) * s.inner + c, w);
 #pragma unroll
-      for (int i = 0; i < V; ++i) a[i] = fmaf(w[i], v[i], a[i]);
-    }
-  };
-  auto source = [&](int k) {                       // row r0 - (taps - 1) + k
-    const int src = r0 - (taps - 1) + k;
-    if (src < 0 || src >= r0 + n) return;
-    float v[V];
-    load_v<V>(col + src * in.ld, v);
-#pragma unroll
-    for (int r = 0; r < SC_ROWS; ++r) {
-      const int j = r + taps - 1 - k;
-      if (j >= 0 && j < taps && src >= lo[r]) add(j, v, acc[r]);
+      for (int i = 0; i < V; ++i) v[i] = 0.f;
     }
   };
   if constexpr (TAPS > 0) {
+    float wr[TAPS][V], h[TAPS - 1 + SC_STEP][V];   // h: inputs from row r - (TAPS - 1) on
 #pragma unroll
-    for (int k = 0; k < TAPS - 1 + SC_ROWS; ++k) source(k);
-  } else {
-    for (int k = 0; k < taps - 1 + SC_ROWS; ++k) source(k);
-  }
+    for (int j = 0; j < TAPS; ++j) load_v<V>(w + (long long)j * s.inner, wr[j]);
 #pragma unroll
-  for (int r = 0; r < SC_ROWS; ++r) {
-    if (r >= n) break;
-    const int i = r0 + r - lo[r];
-    if (i < taps - 1) {                            // inputs before this portion: from the state, zeros before the start
-      const int b = rb.row_seq[r0 + r];
-      if (rb.kv_lens[b] > rb.cu_q[b + 1] - lo[r]) {
-        const float* st = in.conv_state + (long long)rb.slots[b] * (taps - 1) * s.inner + c;
-        for (int j = i + 1; j < taps; ++j) {
-          float v[V];
-          load_v<V>(st + (long long)(taps - 1 + i - j) * s.inner, v);
-          add(j, v, acc[r]);
-        }
+    for (int j = 0; j < TAPS - 1; ++j) {
+      if (r0 - (TAPS - 1) + j >= 0) {
+        load_v<V>(col + (long long)(j - (TAPS - 1)) * in.ld, h[j]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; ++i) h[j][i] = 0.f;
       }
     }
+#pragma unroll 1
+    for (int r = 0; r < n; r += SC_STEP) {
 #pragma unroll
-    for (int q = 0; q < V; ++q) acc[r][q] = silu_f(acc[r][q]);
-    store_v<V>(x + (r0 + r) * ldx + c, acc[r]);
+      for (int u = 0; u < SC_STEP; ++u)
+        if (r + u < n) load_v<V>(col + (long long)(r + u) * in.ld, h[TAPS - 1 + u]);
+#pragma unroll
+      for (int u = 0; u < SC_STEP; ++u) {
+        if (r + u >= n) break;
+        const int i0 = s_index[r + u];
+        float acc[V];
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] = fmaf(wr[TAPS - 1][i], h[TAPS - 1 + u][i], bias[i]);
+#pragma unroll
+        for (int j = 1; j < TAPS; ++j) {
+          if (j <= i0) {                           // the same for the whole block
+#pragma unroll
+            for (int i = 0; i < V; ++i) acc[i] = fmaf(wr[TAPS - 1 - j][i], h[TAPS - 1 + u - j][i], acc[i]);
+          } else {
+            float v[V];
+            early(r + u, j, v);
+#pragma unroll
+            for (int i = 0; i < V; ++i) acc[i] = fmaf(wr[TAPS - 1 - j][i], v[i], acc[i]);
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] = silu_t<T>(acc[i]);
+        store_v<V>(dst + (long long)(r + u) * ldx, acc);
+      }
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+        for (int i = 0; i < V; ++i) h[j][i] = h[j + SC_STEP][i];
+    }
+  } else {
+    for (int r = 0; r < n; ++r) {
+      float acc[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) acc[i] = bias[i];
+      for (int j = 0; j < taps; ++j) {
+        float v[V], wj[V];
+        if (j <= s_index[r]) load_v<V>(col + (long long)(r - j) * in.ld, v);
+        else early(r, j, v);
+        load_v<V>(w + (long long)(taps - 1 - j) * s.inner, wj);
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] = fmaf(wj[i], v[i], acc[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) acc[i] = silu_t<T>(acc[i]);
+      store_v<V>(dst + (long long)r * ldx, acc);
+    }
   }
 }
 
@@ -235,129 +282,242 @@ struct ChunkScratch {
   float *init, *ends, *sums;       // [n_seq][inner][state], [n_seq][chunks][inner][state], [n_seq][chunks][inner]
 };
 
-// State update of one token; the read-out is formed when Y.
+// State update of one token on packed pairs of state values; the read-out is formed when Y.
 template <int NR, bool Y>
-__device__ __forceinline__ float advance(float (&S)[NR], const float (&a)[NR], float dt, float x, const float* sB, const float* sC) {
-  const float dx = dt * x;
-  float y[2] = {0.f, 0.f};
+__device__ __forceinline__ float advance(uint64_t (&S)[NR / 2], const uint64_t (&a)[NR / 2], float dt, float x, const float* sB,
+                                         const float* sC) {
+  const uint64_t dt2 = f32x2(dt, dt), dx2 = f32x2(dt * x, dt * x);
+  uint64_t y[2] = {0ull, 0ull};
 #pragma unroll
   for (int i = 0; i < NR / 4; ++i) {
-    const float4 B = reinterpret_cast<const float4*>(sB)[i];
-    const float bv[4] = {B.x, B.y, B.z, B.w};
-    float cv[4];
-    if constexpr (Y) {
-      const float4 C = reinterpret_cast<const float4*>(sC)[i];
-      cv[0] = C.x; cv[1] = C.y; cv[2] = C.z; cv[3] = C.w;
-    }
+    const ulonglong2 B = reinterpret_cast<const ulonglong2*>(sB)[i];
+    ulonglong2 C{};
+    if constexpr (Y) C = reinterpret_cast<const ulonglong2*>(sC)[i];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int n = 4 * i + j;
-      S[n] = fmaf(fast_exp2(dt * a[n]), S[n], dx * bv[j]);
-      if constexpr (Y) y[j & 1] = fmaf(S[n], cv[j], y[j & 1]);
+    for (int j = 0; j < 2; ++j) {
+      const int n = 2 * i + j;
+      float e0, e1;
+      f32x2_unpack(mul_f32x2(dt2, a[n]), e0, e1);
+      S[n] = fma_f32x2(f32x2(fast_exp2(e0), fast_exp2(e1)), S[n], mul_f32x2(dx2, j ? B.y : B.x));
+      if constexpr (Y) y[j] = fma_f32x2(S[n], j ? C.y : C.x, y[j]);
     }
   }
-  return y[0] + y[1];
+  if constexpr (!Y) return 0.f;
+  float y0, y1;
+  f32x2_unpack(add_f32x2(y[0], y[1]), y0, y1);
+  return y0 + y1;
+}
+template <int NR>
+__device__ __forceinline__ void load_pairs(const float* p, uint64_t (&v)[NR / 2]) {
+#pragma unroll
+  for (int i = 0; i < NR / 4; ++i) {
+    const ulonglong2 t = reinterpret_cast<const ulonglong2*>(p)[i];
+    v[2 * i] = t.x;
+    v[2 * i + 1] = t.y;
+  }
+}
+template <int NR>
+__device__ __forceinline__ void store_pairs(float* p, const uint64_t (&v)[NR / 2]) {
+#pragma unroll
+  for (int i = 0; i < NR / 4; ++i) reinterpret_cast<ulonglong2*>(p)[i] = make_ulonglong2(v[2 * i], v[2 * i + 1]);
 }
 
-// grid (channel blocks, chunks, sequences). OUT: read out and store; else form the chunk's summary.
-template <typename T, int NR, bool OUT>
-__global__ void __launch_bounds__(SS_THREADS)
-selective_scan_kernel(SelectiveSpec s, SelectiveInputs in, RaggedBatch rb, int lanes, int chunk, int chunks,
-                      const float* __restrict__ dt, long long ld_dt, ChunkScratch sc, T* __restrict__ out, long long ldo) {
-  extern __shared__ __align__(16) float sm[];
+// Inputs of a tile of tokens in shared memory: [token][channel of the block] x, z (T) and pre-activations, and
+// [token][row] B and C as they lie in memory (T). SS_STAGES of them form a ring.
+template <typename T>
+struct TileLayout {
+  int tokens, channels, row;       // row: state values of B (and of C) per token, a whole number of 16-byte units
+  static __host__ __device__ int up(int n) { return (n + 127) / 128 * 128; }
+  __host__ __device__ int x() const { return 0; }
+  __host__ __device__ int z() const { return up(tokens * channels * (int)sizeof(T)); }
+  __host__ __device__ int dt() const { return 2 * z(); }
+  __host__ __device__ int b() const { return dt() + up(tokens * channels * 4); }
+  __host__ __device__ int c() const { return b() + up(tokens * row * (int)sizeof(T)); }
+  __host__ __device__ int bytes() const { return c() + up(tokens * row * (int)sizeof(T)); }
+  // bytes of a tile's copies
+  __host__ __device__ int loaded(bool out) const {
+    return tokens * ((out ? 2 : 1) * (channels + row) * (int)sizeof(T) + channels * 4);
+  }
+};
+struct TileMaps {
+  CUtensorMap x, z, dt, b, c, out;
+};
+
+// Quotients of small numbers by one that is not a constant (exact below 2^22).
+struct Quotient {
+  float inv;
+  __device__ __forceinline__ explicit Quotient(int d) : inv(1.f / (float)d) {}
+  __device__ __forceinline__ int operator()(int i) const { return (int)(((float)i + 0.5f) * inv); }
+};
+// n rows of `cols` values: dst (row stride dst_ld) <- src (row stride ld)
+template <typename E>
+__device__ __forceinline__ void copy_rows(E* dst, long long dst_ld, const E* src, long long ld, int n, int cols) {
+  const Quotient by(cols);
+  for (int i = threadIdx.x; i < n * cols; i += SS_THREADS) {
+    const int r = by(i), c = i - r * cols;
+    dst[r * dst_ld + c] = src[r * ld + c];
+  }
+}
+
+// grid (channel blocks, chunks, sequences). OUT: read out and store; else form the chunk's summary. tma: tiles arrive
+// and leave by TMA (rows of whole 16-byte units), else by plain copies. LANES: threads per channel (0: `lanes_`).
+template <typename T, int NR, bool OUT, int LANES>
+__global__ void __launch_bounds__(SS_THREADS, SS_BLOCKS)
+selective_scan_kernel(const __grid_constant__ SelectiveSpec s, const __grid_constant__ SelectiveInputs in,
+                      const __grid_constant__ RaggedBatch rb, int lanes_, int chunk, int chunks, const float* __restrict__ dt,
+                      long long ld_dt, ChunkScratch sc, T* __restrict__ out, long long ldo, TileLayout<T> lay, bool tma,
+                      const __grid_constant__ TileMaps maps, int* status) {
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ uint64_t full[SS_STAGES];
+  __shared__ int abort_word;
+  volatile int* abort_flag = &abort_word;
+  uint8_t* smem = smem_raw + ((128u - (smem_u32(smem_raw) & 127u)) & 127u);
+  const int lanes = LANES > 0 ? LANES : lanes_, channels = SS_THREADS / lanes;
   const int b = blockIdx.z, k = blockIdx.y;
   const int row0 = rb.cu_q[b], len = rb.cu_q[b + 1] - row0, t0 = k * chunk;
   if (t0 >= len) return;
   const int t1 = min(len, t0 + chunk), state_p = NR * lanes;
   const bool last = t1 == len;
   if (!OUT && last) return;                        // nothing starts from the last chunk's state
-  const int idx = blockIdx.x * SS_THREADS + threadIdx.x, sub = idx % lanes;
-  const bool live = idx / lanes < s.inner;
-  const int ch = live ? idx / lanes : s.inner - 1;
+  const int cl = threadIdx.x / lanes, sub = threadIdx.x % lanes, c0 = blockIdx.x * channels;
+  const bool live = c0 + cl < s.inner;
+  const int ch = live ? c0 + cl : s.inner - 1, width = min(channels, s.inner - c0);
+  const int tile = lay.tokens, tiles = (t1 - t0 + tile - 1) / tile;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < SS_STAGES; ++i) mbar_init(&full[i], 1);
+    *abort_flag = 0;
+    fence_mbar_init();
+  }
+  __syncthreads();
+  auto fetch = [&](int i) {                        // by TMA: one thread
+    const int st = i % SS_STAGES, row = row0 + t0 + i * tile;
+    uint8_t* buf = smem + st * lay.bytes();
+    mbar_arrive_expect_tx(&full[st], (uint32_t)lay.loaded(OUT));
+    tma_load_2d(buf + lay.x(), &maps.x, &full[st], c0, row);
+    tma_load_2d(buf + lay.dt(), &maps.dt, &full[st], c0, row);
+    tma_load_2d(buf + lay.b(), &maps.b, &full[st], 0, row);
+    if constexpr (OUT) {
+      tma_load_2d(buf + lay.z(), &maps.z, &full[st], c0, row);
+      tma_load_2d(buf + lay.c(), &maps.c, &full[st], 0, row);
+    }
+  };
+  if (tma && threadIdx.x == 0)
+    for (int i = 0; i < SS_STAGES - 1 && i < tiles; ++i) fetch(i);
   const bool fresh = rb.kv_lens[b] == len;
   float* slot = in.state + ((long long)rb.slots[b] * s.inner + ch) * state_p + sub * NR;
-  float a[NR], S[NR];
-  load_v<NR>(in.a + (long long)ch * state_p + sub * NR, a);
+  uint64_t a[NR / 2], S[NR / 2];                   // pairs of state values
+  load_pairs<NR>(in.a + (long long)ch * state_p + sub * NR, a);
   if (OUT && (k > 0 || !last)) {                   // several chunks: the slot may already hold the final state
-    load_v<NR>(sc.init + ((long long)b * s.inner + ch) * state_p + sub * NR, S);
+    load_pairs<NR>(sc.init + ((long long)b * s.inner + ch) * state_p + sub * NR, S);
     for (int i = 0; i < k; ++i) {
       const long long at = ((long long)b * chunks + i) * s.inner + ch;
       const float sum = sc.sums[at];
-      float e[NR];
-      load_v<NR>(sc.ends + at * state_p + sub * NR, e);
+      uint64_t e[NR / 2];
+      load_pairs<NR>(sc.ends + at * state_p + sub * NR, e);
 #pragma unroll
-      for (int n = 0; n < NR; ++n) S[n] = fmaf(fast_exp2(sum * a[n]), S[n], e[n]);
+      for (int n = 0; n < NR / 2; ++n) {
+        float d0, d1;
+        f32x2_unpack(mul_f32x2(f32x2(sum, sum), a[n]), d0, d1);
+        S[n] = fma_f32x2(f32x2(fast_exp2(d0), fast_exp2(d1)), S[n], e[n]);
+      }
     }
   } else {
 #pragma unroll
-    for (int n = 0; n < NR; ++n) S[n] = 0.f;
-    if ((OUT || k == 0) && !fresh) load_v<NR>(slot, S);
+    for (int n = 0; n < NR / 2; ++n) S[n] = 0ull;
+    if ((OUT || k == 0) && !fresh) load_pairs<NR>(slot, S);
     if (!OUT && k == 0) {
-      if (live) store_v<NR>(sc.init + ((long long)b * s.inner + ch) * state_p + sub * NR, S);
+      if (live) store_pairs<NR>(sc.init + ((long long)b * s.inner + ch) * state_p + sub * NR, S);
 #pragma unroll
-      for (int n = 0; n < NR; ++n) S[n] = 0.f;
+      for (int n = 0; n < NR / 2; ++n) S[n] = 0ull;
     }
   }
-  const float bias = in.dt_bias[ch], D = OUT ? in.d[ch] : 0.f;
-  const T* xp = static_cast<const T*>(in.x) + (long long)row0 * in.ld_x + ch;
-  const T* zp = static_cast<const T*>(in.proj) + (long long)row0 * in.ld + in.z_off + ch;
-  const float* dp = dt + (long long)row0 * ld_dt + ch;
-  const T* low = static_cast<const T*>(in.low) + (long long)row0 * in.ld_low;
-  const int tile = min(SS_TILE, SS_TILE_VALUES / state_p / SS_GROUP * SS_GROUP);
-  float *sB = sm, *sC = sm + tile * state_p;
+  const float bias = in.dt_bias[ch], D = OUT ? in.d[ch] : 0.f, scale = s.out_scale;
+  // B, then C, of the tile in fp32, zeros in the padding
+  float* sB = reinterpret_cast<float*>(smem + (tma ? SS_STAGES : 1) * lay.bytes());
+  float* sC = sB + tile * state_p;
   float total = 0.f;
-  float nx[SS_GROUP], nd[SS_GROUP], nz[SS_GROUP];  // inputs of the next group
-  auto fetch = [&](int t) {
-#pragma unroll
-    for (int u = 0; u < SS_GROUP; ++u) {
-      const bool on = t + u < t1;
-      nx[u] = on ? ldf(xp + (long long)(t + u) * in.ld_x) : 0.f;
-      nd[u] = on ? dp[(long long)(t + u) * ld_dt] : 0.f;
-      if constexpr (OUT) nz[u] = on ? ldf(zp + (long long)(t + u) * in.ld) : 0.f;
-    }
-  };
-  fetch(t0);
-  for (int tt = t0; tt < t1; tt += tile) {
-    const int n = min(tile, t1 - tt);
-    __syncthreads();
-    for (int i = threadIdx.x; i < n * state_p; i += SS_THREADS) {
-      const int u = i / state_p, v = i % state_p;
-      const T* row = low + (long long)(tt + u) * in.ld_low;
-      sB[i] = v < s.state ? ldf(row + in.b_off + v) : 0.f;
-      if constexpr (OUT) sC[i] = v < s.state ? ldf(row + in.c_off + v) : 0.f;
-    }
-    __syncthreads();
-    for (int g = 0; g < n; g += SS_GROUP) {
-      float x[SS_GROUP], d[SS_GROUP], z[SS_GROUP];
-#pragma unroll
-      for (int u = 0; u < SS_GROUP; ++u) {
-        x[u] = nx[u];
-        d[u] = softplus_fast(nd[u] + bias);
-        if constexpr (OUT) z[u] = nz[u];
+  for (int i = 0; i < tiles; ++i) {
+    const int tt = t0 + i * tile, n = min(tile, t1 - tt), st = tma ? i % SS_STAGES : 0;
+    uint8_t* buf = smem + st * lay.bytes();
+    if (tma) {
+      const bool ok = mbar_wait(&full[st], (i / SS_STAGES) & 1, abort_flag, status, 110);
+      if (!__syncthreads_and(ok)) break;           // also: nobody reads B and C of the tile before any more
+    } else {
+      __syncthreads();
+      const long long row = row0 + tt;
+      copy_rows((T*)(buf + lay.x()), channels, static_cast<const T*>(in.x) + row * in.ld_x + c0, in.ld_x, n, width);
+      copy_rows((float*)(buf + lay.dt()), channels, dt + row * ld_dt + c0, ld_dt, n, width);
+      copy_rows((T*)(buf + lay.b()), lay.row, static_cast<const T*>(in.low) + row * in.ld_low + in.b_off, in.ld_low, n, s.state);
+      if constexpr (OUT) {
+        copy_rows((T*)(buf + lay.z()), channels, static_cast<const T*>(in.proj) + row * in.ld + in.z_off + c0, in.ld, n, width);
+        copy_rows((T*)(buf + lay.c()), lay.row, static_cast<const T*>(in.low) + row * in.ld_low + in.c_off, in.ld_low, n, s.state);
       }
-      fetch(tt + g + SS_GROUP);
+      __syncthreads();
+    }
+    const Quotient by_state(state_p);
+    for (int j = threadIdx.x; j < n * state_p; j += SS_THREADS) {
+      const int u = by_state(j), v = j - u * state_p;
+      sB[j] = v < s.state ? ldf((const T*)(buf + lay.b()) + u * lay.row + v) : 0.f;
+      if constexpr (OUT) sC[j] = v < s.state ? ldf((const T*)(buf + lay.c()) + u * lay.row + v) : 0.f;
+    }
+    __syncthreads();
+    T* sx = (T*)(buf + lay.x()) + cl;
+    const T* sz = (const T*)(buf + lay.z()) + cl;
+    const float* sd = (const float*)(buf + lay.dt()) + cl;
+    const float *pB = sB + sub * NR, *pC = sC + sub * NR;
+    // G tokens at a time: their step sizes and gates overlap, and no store lies between their state updates
+    auto run = [&](auto group, int u0) {
+      constexpr int G = decltype(group)::value;
+      float x[G], d[G], y[G];
 #pragma unroll
-      for (int u = 0; u < SS_GROUP; ++u) {
-        if (g + u >= n) break;                     // the same for the whole block
-        const int at = (g + u) * state_p + sub * NR;
-        float y = advance<NR, OUT>(S, a, d[u], x[u], sB + at, sC + at);
-        if constexpr (OUT) {
-          for (int o = 1; o < lanes; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-          if (live && sub == 0)
-            stf(out + (long long)(row0 + tt + g + u) * ldo + ch,
-                fmaf(D, x[u], y) * __fdividef(z[u], 1.f + __expf(-z[u])) * s.out_scale);
-        } else {
-          total += d[u];
+      for (int g = 0; g < G; ++g) {
+        x[g] = ldf(sx + (u0 + g) * channels);
+        d[g] = softplus_fast(sd[(u0 + g) * channels] + bias);
+        if constexpr (!OUT) total += d[g];
+      }
+#pragma unroll
+      for (int g = 0; g < G; ++g) y[g] = advance<NR, OUT>(S, a, d[g], x[g], pB + (u0 + g) * state_p, pC + (u0 + g) * state_p);
+      if constexpr (OUT) {
+        for (int o = 1; o < lanes; o <<= 1)
+#pragma unroll
+          for (int g = 0; g < G; ++g) y[g] += __shfl_xor_sync(0xffffffffu, y[g], o);
+#pragma unroll
+        for (int g = 0; g < G; ++g) y[g] = fmaf(D, x[g], y[g]) * scale * silu_fast(ldf(sz + (u0 + g) * channels));
+        if (sub == 0) {                            // the output takes x's place
+#pragma unroll
+          for (int g = 0; g < G; ++g) stf(sx + (u0 + g) * channels, y[g]);
         }
       }
+    };
+    int u = 0;
+    for (; u + SS_GROUP <= n; u += SS_GROUP) run(std::integral_constant<int, SS_GROUP>{}, u);
+    for (; u < n; ++u) run(std::integral_constant<int, 1>{}, u);
+    if (OUT && tma) fence_proxy_async_smem();
+    __syncthreads();
+    if (tma && threadIdx.x == 0) {
+      // the tile before has long been read by its store: its place takes the tile after the next
+      if constexpr (OUT) tma_store_wait_read0();
+      if (i + SS_STAGES - 1 < tiles) fetch(i + SS_STAGES - 1);
+      if (OUT && n == tile) {
+        tma_store_2d(&maps.out, buf + lay.x(), c0, row0 + tt);
+        tma_store_commit();
+      }
     }
+    if (OUT && !(tma && n == tile))
+      copy_rows(out + (long long)(row0 + tt) * ldo + c0, ldo, (const T*)(buf + lay.x()), channels, n, width);
   }
+  if (tma && *abort_flag) {        // copies in flight land in this CTA's memory: give them time
+    const long long c = clock64();
+    while (clock64() - c < 10000000LL) {}
+    return;
+  }
+  if (OUT && tma && threadIdx.x == 0) tma_store_wait_read0();
   if (!live) return;
   if constexpr (OUT) {
-    if (last) store_v<NR>(slot, S);
+    if (last) store_pairs<NR>(slot, S);
   } else {
     const long long at = ((long long)b * chunks + k) * s.inner + ch;
-    store_v<NR>(sc.ends + at * state_p + sub * NR, S);
+    store_pairs<NR>(sc.ends + at * state_p + sub * NR, S);
     if (sub == 0) sc.sums[at] = total;
   }
 }
@@ -373,11 +533,11 @@ selective_step_kernel(SelectiveSpec s, SelectiveInputs in, RaggedBatch rb, int l
   const bool live = idx / lanes < s.inner;
   const int ch = live ? idx / lanes : s.inner - 1;
   float* slot = in.state + ((long long)rb.slots[b] * s.inner + ch) * state_p + sub * NR;
-  float a[NR], S[NR];
+  uint64_t a[NR / 2], S[NR / 2];
 #pragma unroll
-  for (int n = 0; n < NR; ++n) S[n] = 0.f;
-  if (rb.kv_lens[b] > 1) load_v<NR>(slot, S);
-  load_v<NR>(in.a + (long long)ch * state_p + sub * NR, a);
+  for (int n = 0; n < NR / 2; ++n) S[n] = 0ull;
+  if (rb.kv_lens[b] > 1) load_pairs<NR>(slot, S);
+  load_pairs<NR>(in.a + (long long)ch * state_p + sub * NR, a);
   const T* low = static_cast<const T*>(in.low) + b * in.ld_low;
   float *sB = sm, *sC = sm + state_p, *sR = sC + state_p;
   for (int v = threadIdx.x; v < state_p; v += SS_THREADS) {
@@ -407,8 +567,8 @@ selective_step_kernel(SelectiveSpec s, SelectiveInputs in, RaggedBatch rb, int l
   float y = advance<NR, true>(S, a, d, x, sB + sub * NR, sC + sub * NR);
   for (int o = 1; o < lanes; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
   if (!live) return;
-  store_v<NR>(slot, S);
-  if (sub == 0) stf(out + b * ldo + ch, fmaf(in.d[ch], x, y) * __fdividef(z, 1.f + __expf(-z)) * s.out_scale);
+  store_pairs<NR>(slot, S);
+  if (sub == 0) stf(out + b * ldo + ch, fmaf(in.d[ch], x, y) * silu_fast(z) * s.out_scale);
 }
 
 void check_spec(const SelectiveSpec& s) {
@@ -416,18 +576,20 @@ void check_spec(const SelectiveSpec& s) {
   MB_REQUIRE(s.state > 0 && s.state <= 512, "selective scan: at most 512 state values per channel");
 }
 
-// Chunks of the longest portion: enough blocks for the machine, unless a single pass already gives half of them.
+// Chunks of the longest portion. Chunks cost a second pass, so a portion is cut only where its blocks leave SMs idle, and
+// then into enough of them to fill every SM (measured: 4 blocks on an SM run twice as fast as one).
 struct ChunkPlan {
   int chunk, chunks;
 };
-ChunkPlan plan_chunks(const SelectiveSpec& s, int n_seq, int max_q) {
+ChunkPlan plan_chunks(const SelectiveSpec& s, int rows, int max_q) {
   const StateMap m = state_map(s.state);
-  const long long blocks = ((long long)s.inner * m.lanes + SS_THREADS - 1) / SS_THREADS * n_seq;
-  long long chunks = 6ll * sm_count() / (blocks > 0 ? blocks : 1);
+  if (max_q <= 0) return ChunkPlan{1, 1};
+  const long long blocks = ((long long)s.inner * m.lanes + SS_THREADS - 1) / SS_THREADS * ((rows + max_q - 1) / max_q);
+  long long chunks = blocks * 5 >= sm_count() * 4ll ? 1 : 6ll * sm_count() / blocks;
   const long long most = (max_q + SS_CHUNK - 1) / SS_CHUNK;
   if (chunks > most) chunks = most;
   if (chunks > 64) chunks = 64;
-  if (chunks < 2) return ChunkPlan{max_q > 0 ? max_q : 1, 1};
+  if (chunks < 2) return ChunkPlan{max_q, 1};
   const int chunk = (int)((max_q + chunks - 1) / chunks);
   return ChunkPlan{chunk, (max_q + chunk - 1) / chunk};
 }
@@ -453,17 +615,17 @@ void selective_conv(bool f32, const SelectiveSpec& s, const SelectiveInputs& in,
     check_launch();
     return;
   }
-  const int es = f32 ? 4 : 2, V = 16 / es;
+  const int V = 4;
   const bool vec = s.inner % V == 0 && ldx == s.inner && in.ld % V == 0 && in.x_off % V == 0 &&
                    ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(in.proj)) & 15) == 0;
-  const int units = (int)(vec ? ldx / V : ldx), threads = units >= 256 ? 256 : (units + 31) / 32 * 32;
+  const int units = (int)(vec ? ldx / V : ldx), threads = units >= 128 ? 128 : (units + 31) / 32 * 32;
   const dim3 grid((units + threads - 1) / threads, (rb.rows + SC_ROWS - 1) / SC_ROWS);
   MB_REQUIRE(grid.y <= 65535, "selective_conv: too many rows in one batch");
 #define MB_SC(T, V, TAPS) selective_conv_kernel<T, V, TAPS><<<grid, threads, 0, stream>>>(s, in, rb, (T*)x, ldx)
   if (f32) {
     if (vec && s.taps == 4) MB_SC(float, 4, 4); else if (vec) MB_SC(float, 4, 0); else MB_SC(float, 1, 0);
   } else {
-    if (vec && s.taps == 4) MB_SC(__nv_bfloat16, 8, 4); else if (vec) MB_SC(__nv_bfloat16, 8, 0); else MB_SC(__nv_bfloat16, 1, 0);
+    if (vec && s.taps == 4) MB_SC(__nv_bfloat16, 4, 4); else if (vec) MB_SC(__nv_bfloat16, 4, 0); else MB_SC(__nv_bfloat16, 1, 0);
   }
 #undef MB_SC
   count_launch();
@@ -477,8 +639,8 @@ void selective_conv(bool f32, const SelectiveSpec& s, const SelectiveInputs& in,
   }
 }
 
-long long selective_scratch(const SelectiveSpec& s, int n_seq, int max_q) {
-  const ChunkPlan p = plan_chunks(s, n_seq, max_q);
+long long selective_scratch(const SelectiveSpec& s, int n_seq, int rows, int max_q) {
+  const ChunkPlan p = plan_chunks(s, rows, max_q);
   if (p.chunks <= 1) return 0;
   const long long state = (long long)s.inner * selective_padded_state(s.state);
   return n_seq * (state + p.chunks * (state + s.inner));
@@ -488,27 +650,62 @@ long long selective_scratch(const SelectiveSpec& s, int n_seq, int max_q) {
   if (m.nr == 4) GO(4); else if (m.nr == 8) GO(8); else if (m.nr == 12) GO(12); else GO(16)
 
 void selective_scan(bool f32, const SelectiveSpec& s, const SelectiveInputs& in, const RaggedBatch& rb, int max_q,
-                    const float* dt, long long ld_dt, float* scratch, void* out, long long ldo, cudaStream_t stream) {
+                    const float* dt, long long ld_dt, float* scratch, void* out, long long ldo, int* status,
+                    cudaStream_t stream) {
   check_spec(s);
   if (rb.rows == 0) return;
   MB_REQUIRE(max_q > 0 && rb.n_seq <= 65535, "selective_scan: batch");
   const StateMap m = state_map(s.state);
-  const ChunkPlan p = plan_chunks(s, rb.n_seq, max_q);
+  const ChunkPlan p = plan_chunks(s, rb.rows, max_q);
   const int state_p = m.nr * m.lanes;
   const long long state = (long long)s.inner * state_p;
   ChunkScratch sc{scratch, scratch + rb.n_seq * state, scratch + rb.n_seq * state * (1 + p.chunks)};
   const dim3 grid((int)(((long long)s.inner * m.lanes + SS_THREADS - 1) / SS_THREADS), p.chunks, rb.n_seq);
-  const int per = SS_TILE_VALUES / state_p / SS_GROUP * SS_GROUP, tile = per < SS_TILE ? per : SS_TILE;
-  const int smem = 2 * tile * state_p * 4;
-#define MB_SS(T, NR, OUT)                                                                                           \
-  selective_scan_kernel<T, NR, OUT><<<grid, SS_THREADS, smem, stream>>>(s, in, rb, m.lanes, p.chunk, p.chunks, dt, ld_dt, sc, \
-                                                                        (T*)out, ldo)
-#define MB_SS_BF(NR) do { if (p.chunks > 1) MB_SS(__nv_bfloat16, NR, false); MB_SS(__nv_bfloat16, NR, true); } while (0)
-#define MB_SS_F(NR) do { if (p.chunks > 1) MB_SS(float, NR, false); MB_SS(float, NR, true); } while (0)
+  const int per = SS_TILE_VALUES / state_p, tile = per < SS_TILE ? per : SS_TILE;
+  const int channels = SS_THREADS / m.lanes, es = f32 ? 4 : 2, unit = 16 / es;
+  auto whole = [&](const void* p, long long ld, int off) {       // rows of 16-byte units
+    return ((reinterpret_cast<uintptr_t>(p) + (uintptr_t)off * es) & 15) == 0 && ld % unit == 0;
+  };
+  const int row = (s.state + unit - 1) / unit * unit;
+  const bool tma = channels % unit == 0 && channels % 4 == 0 && row <= 256 && whole(in.x, in.ld_x, 0) && whole(in.proj, in.ld, in.z_off) &&
+                   whole(in.low, in.ld_low, in.b_off) && whole(in.low, in.ld_low, in.c_off) && whole(out, ldo, 0) &&
+                   ld_dt % 4 == 0 && (reinterpret_cast<uintptr_t>(dt) & 15) == 0;
+  TileMaps maps{};
+  if (tma) {
+    auto map = [&](const void* p, long long ld, int off, int cols, int box_cols, int size) {
+      uint64_t dims[2] = {(uint64_t)cols, (uint64_t)rb.rows}, strides[1] = {(uint64_t)ld * size};
+      uint32_t box[2] = {(uint32_t)box_cols, (uint32_t)tile};
+      return make_tensor_map((const char*)p + (long long)off * size, size == 4 ? TmaDType::F32 : TmaDType::BF16, 2, dims, strides, box,
+                             false);
+    };
+    maps.x = map(in.x, in.ld_x, 0, s.inner, channels, es);
+    maps.z = map(in.proj, in.ld, in.z_off, s.inner, channels, es);
+    maps.dt = map(dt, ld_dt, 0, s.inner, channels, 4);
+    maps.b = map(in.low, in.ld_low, in.b_off, s.state, row, es);
+    maps.c = map(in.low, in.ld_low, in.c_off, s.state, row, es);
+    maps.out = map(out, ldo, 0, s.inner, channels, es);
+  }
+  auto go = [&](auto kernel, auto layout, auto* o) {
+    layout.tokens = tile;
+    layout.channels = channels;
+    layout.row = row;
+    const int smem = (tma ? SS_STAGES : 1) * layout.bytes() + 2 * tile * state_p * 4 + 128;
+    MB_CUDA_CHECK(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    kernel<<<grid, SS_THREADS, smem, stream>>>(s, in, rb, m.lanes, p.chunk, p.chunks, dt, ld_dt, sc, o, ldo, layout, tma, maps, status);
+  };
+#define MB_SS_L(T, NR, L)                                                                         \
+  do {                                                                                            \
+    if (p.chunks > 1) go(selective_scan_kernel<T, NR, false, L>, TileLayout<T>{}, (T*)out);       \
+    go(selective_scan_kernel<T, NR, true, L>, TileLayout<T>{}, (T*)out);                          \
+  } while (0)
+#define MB_SS(T, NR) do { if (m.lanes == 1) MB_SS_L(T, NR, 1); else MB_SS_L(T, NR, 0); } while (0)
+#define MB_SS_BF(NR) MB_SS(__nv_bfloat16, NR)
+#define MB_SS_F(NR) MB_SS(float, NR)
   if (f32) { MB_SS_NR(MB_SS_F); } else { MB_SS_NR(MB_SS_BF); }
 #undef MB_SS_F
 #undef MB_SS_BF
 #undef MB_SS
+#undef MB_SS_L
   count_launch(p.chunks > 1 ? 2 : 1);
   check_launch();
 }

@@ -104,6 +104,7 @@ EXPAND_TOKENS = 16         # portions of at least this many tokens expand the la
 EXPAND_BYTES = 4 << 30     # unless the expanded keys and values would need more than this
 SEGMENT_GEMM_ROWS = 48     # mean rows per expert from which the prompt-sized grouped GEMM runs
 LOW_RANK_FUSE_ROWS = 16    # decode batches up to this size evaluate the low-rank maps inside the recurrence kernel
+STEP_FUSE_ROWS = 4         # the same for the step sizes of a selective scan, whose map every token reads again
 
 
 class HybridEngine(InferenceEngine):
@@ -499,15 +500,15 @@ class HybridEngine(InferenceEngine):
         sel.conv(proj, ctx.batch, one, x)
         low = self._gemm(x, L.x_maps.weight)
         dt = None
-        if not (one and ctx.rows <= LOW_RANK_FUSE_ROWS):
+        if not (one and ctx.rows <= STEP_FUSE_ROWS):
             dt = self._gemm(low[:, : L.w_dt.shape[1]], L.w_dt, dtype=torch.float32)
         if out.shape[1] != m.inner:
             out[:, m.inner:].zero_()
         if one:
             sel.step(proj, x, low, dt, ctx.batch, out)
         else:
-            scratch = torch.empty(sel.scratch_floats(ctx.n_seq, ctx.max_q), device=self.device, dtype=torch.float32)
-            sel.scan(proj, x, low, dt, ctx.batch, ctx.max_q, scratch, out)
+            scratch = torch.empty(sel.scratch_floats(ctx.n_seq, ctx.rows, ctx.max_q), device=self.device, dtype=torch.float32)
+            sel.scan(proj, x, low, dt, ctx.batch, ctx.max_q, scratch, out, self._status)
 
     def _parallel_selective(self, L, h, ctx):
         proj = self._gemm(h, L.proj.weight)

@@ -228,7 +228,7 @@ def _expert_rows(K, H, C, rnd, eng, L, T):
 
 def run_dogozen_kernels(peaks: dict, width: int = 2048) -> list[dict]:
     """Tempered and window attention (heads of 128), selective scan, routed and shared experts, soft-capped output."""
-    from ..infer.hybrid import LOW_RANK_FUSE_ROWS, HybridEngine
+    from ..infer.hybrid import STEP_FUSE_ROWS, HybridEngine
     from ..models.hybrid_config import dogozen_config
     from ..ops import functional as F, native
 
@@ -282,16 +282,16 @@ def run_dogozen_kernels(peaks: dict, width: int = 2048) -> list[dict]:
         n, b = B * S, _batch([S] * B, [0] * B)
         proj, x, low, out = rnd(n, N), rnd(n, c), rnd(n, par.x_maps.N), torch.empty(n, c, device="cuda", dtype=bf)
         dt, sizes = torch.randn(n, c, device="cuda") - 3.0, f"{B} x {S}, {c} channels, {ns} state values"
-        scratch = torch.empty(sel.scratch_floats(B, S), device="cuda")
+        scratch = torch.empty(sel.scratch_floats(B, n, S), device="cuda")
         K.add("selective_conv", sizes, lambda: sel.conv(proj, b, False, x), nbytes=4.0 * n * c, like="rope (dense)")
-        K.add("selective_scan", sizes, lambda: sel.scan(proj, x, low, dt, b, S, scratch, out),
+        K.add("selective_scan", sizes, lambda: sel.scan(proj, x, low, dt, b, S, scratch, out, st),
               nbytes=n * (c * 10.0 + 4 * ns) + 8.0 * B * c * ns, like="chunked recurrence + norm + gate")
         _recurrent_rows(K, H, st, "delta", h, 128, 128, [S] * B, False)
         _recurrent_rows(K, H, st, "gla", h, 64, 128, [S] * B, False)
     for T in (1, 16, 64):
         b = _batch([1] * T, [99] * T)
         proj, x, low, out = rnd(T, N), rnd(T, c), rnd(T, par.x_maps.N), torch.empty(T, c, device="cuda", dtype=bf)
-        dt = torch.randn(T, c, device="cuda") if T > LOW_RANK_FUSE_ROWS else None
+        dt = torch.randn(T, c, device="cuda") if T > STEP_FUSE_ROWS else None
         sizes = f"{T} tokens, {c} channels, {ns} state values"
         K.add("selective_conv, one token", sizes, lambda: sel.conv(proj, b, True, x), nbytes=T * c * (4.0 + 24), like="recurrent_decode")
         K.add("selective_step", sizes, lambda: sel.step(proj, x, low, dt, b, out),
