@@ -47,6 +47,41 @@ def lebedra(width, vocab, layers, side, mult=0.5, eps=1e-5):
             "layers": [{"type": "latent_attention", "mixer": m, "mlp": f} for m, f in layers]}
 
 
+def window_left(heads, kv, dim, vdim, rot, window, base=500.0, scaling=None, scale=None):
+    r = {"base": base, "dims": rot}
+    if scaling:
+        r["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    return {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5 if scale is None else scale, "rot": r,
+            "mask": {"size": window}}
+
+
+def selective(inner, state, rank, conv):
+    return {"inner": inner, "state": state, "dt_rank": rank, "conv": conv}
+
+
+def tempered_layer(heads, kv, dim, vdim, coef, every, scale=None, mlp=None, kv_from=None):
+    m = dict(attention(heads, kv, dim, vdim, scale), q_temp={"coef": coef, "every": every})
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def scan_layer(left, right, scales, mlp=None):
+    return {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": scales[0], "right_scale": scales[1]}, "mlp": mlp}
+
+
+def sigmoid_moe(experts, top, ff, groups, keep, scale=1.0, shared=0):
+    d = {"kind": "moe", "expert": {"ff": ff},
+         "router": {"experts": experts, "top": top, "scale": scale, "groups": {"count": groups, "keep": keep}}}
+    if shared:
+        d["shared"] = {"ff": shared}
+    return d
+
+
+def dogozen(width, vocab, layers, cap=20.0, eps=1e-5):
+    return {"architecture": "Dogozen", "vocab": vocab, "width": width, "norm": {"eps": eps}, "logit_softcap": cap, "layers": layers}
+
+
 CONFIGS = {
     # unaligned widths everywhere, grouped heads, three taps
     "ragged": config(100, 211, [gla_layer(3, 24, 40, 8.0, ff=52),
@@ -73,9 +108,49 @@ CONFIGS = {
                              8, 1.0, 1e-3),
     # widths beyond the prompt attention's, a token side wider than a tile
     "latent_plain": lebedra(136, 130, [(latent(2, 160, 72, 136, 40), moe(9, 5, 24, 3.0, 3, 3)), (latent(17, 16, 4, 24, 520), dense(40))], 136, 0.6),
+    # Dogozen: unaligned widths, shared keys and values with another temperature and scale, partial rotation of an odd
+    # number of pairs, three taps, fewer channels than a block
+    "scan_ragged": dogozen(100, 211, [
+        tempered_layer(6, 2, 20, 36, 0.4, 16, mlp=dense(52)),
+        scan_layer(window_left(4, 2, 20, 12, 10, 19), selective(52, 5, 3, 3), (0.7, 1.2), sigmoid_moe(6, 3, 20, 3, 2, 1.7, 28)),
+        tempered_layer(4, 2, 20, 36, 0.9, 7, 0.4, kv_from=0)]),
+    # widths of the tensor-core paths, more than eight query heads on one key head, stretched rotation, two lanes per
+    # channel, a layer that shares with the one before a parallel layer
+    "scan_wide": dogozen(256, 384, [
+        scan_layer(window_left(6, 2, 72, 104, 48, 70, 1e4, (4.0, 1.0, 3.0, 64)), selective(512, 16, 16, 4), (1.0, 0.6), dense(256)),
+        tempered_layer(12, 1, 128, 64, 0.2, 100, 0.11, sigmoid_moe(8, 2, 64, 2, 1, 2.0, 64)),
+        scan_layer(window_left(4, 4, 128, 128, 128, 33, 1e5, (8.0, 1.0, 4.0, 512)), selective(200, 24, 40, 4), (0.5, 0.9),
+                   sigmoid_moe(12, 4, 72, 1, 1)),
+        tempered_layer(9, 1, 128, 64, 0.3, 1, 0.09, dense(96), kv_from=1)], 18.0),
+    # one of everything: head, tap, state value, rank, window, expert, experts per group
+    "scan_single": dogozen(64, 96, [
+        scan_layer(window_left(1, 1, 16, 16, 2, 1), selective(8, 1, 1, 1), (1.0, 1.0), sigmoid_moe(4, 1, 24, 4, 2, 0.5, 8)),
+        tempered_layer(1, 1, 64, 64, 1.5, 3, mlp=sigmoid_moe(1, 1, 32, 1, 1)),
+        scan_layer(window_left(2, 1, 64, 64, 64, 16), selective(72, 4, 9, 2), (2.0, -0.5))], 50.0, 1e-3),
+    # widths beyond the prompt attention's, a window longer than the sequences, many state values, many taps
+    "scan_plain": dogozen(136, 130, [
+        tempered_layer(2, 2, 160, 136, 0.5, 32, mlp=dense(40)),
+        scan_layer(window_left(3, 1, 136, 24, 40, 2000), selective(40, 130, 24, 6), (0.9, 1.1), dense(56))], 10.0),
 }
-TEGANEX = [n for n in CONFIGS if not n.startswith("latent")]
+TEGANEX = [n for n in CONFIGS if not n.startswith(("latent", "scan"))]
 LEBEDRA = [n for n in CONFIGS if n.startswith("latent")]
+DOGOZEN = [n for n in CONFIGS if n.startswith("scan")]
+
+
+def _dogozen_weight(name: str, r: torch.Tensor) -> torch.Tensor:
+    """Norms around zero, decays from nearly one to nearly zero, biases and step sizes that show."""
+    leaf = name.rsplit(".", 1)[-1]
+    if leaf == "A_log":
+        return r * 1.2 - 0.5
+    if len(r.shape) == 1:
+        if name.endswith(".dt.b"):
+            return r * 1.5 - 2.0
+        return 1.0 + 0.3 * r if leaf == "D" else r * {"sink": 1.5, "b": 0.5}.get(leaf, 0.3)
+    if leaf == "conv":
+        return r * 0.5
+    if leaf == "embed":
+        return r
+    return r * ({"router": 2.0, "dt": 1.0}.get(leaf, 1.5) / r.shape[1] ** 0.5)
 
 
 def weights(cfg: dict, seed: int = 0, low_rank: int = 12, sure_routes: bool = False) -> dict:
@@ -91,7 +166,9 @@ def weights(cfg: dict, seed: int = 0, low_rank: int = 12, sure_routes: bool = Fa
         shape = tuple(low_rank if n is None else n for n in shape)
         leaf = name.rsplit(".", 1)[-1]
         r = torch.randn(shape, generator=g)
-        if len(shape) == 1:
+        if cfg["architecture"] == "Dogozen":
+            t = _dogozen_weight(name, r)
+        elif len(shape) == 1:
             if leaf == "A_log":
                 t = torch.linspace(-3.0, 2.7, shape[0]) if shape[0] > 1 else torch.zeros(1)
             elif leaf == "dt_bias":
@@ -112,7 +189,7 @@ def weights(cfg: dict, seed: int = 0, low_rank: int = 12, sure_routes: bool = Fa
             t = r * (1.0 if leaf == "embed" else 0.4)
         else:
             t = r * (1.5 / shape[1] ** 0.5)
-        if sure_routes and cfg["architecture"] == "Lebedra":
+        if sure_routes and cfg["architecture"] != "Teganex":
             n = max([x["mlp"]["router"]["experts"] for x in cfg["layers"] if (x["mlp"] or {}).get("kind") == "moe"] or [0])
             if leaf == "router":
                 t = torch.cat([r[:, :n] * 2.0 / n ** 0.5, torch.zeros(shape[0], shape[1] - n)], 1)

@@ -10,8 +10,8 @@ import hybrid_oracle as oracle
 import hybrid_util as hu
 from mythos_b200.infer.kv_paged import PagedKVCache, RecurrentStatePool
 from mythos_b200.models import registry
-from mythos_b200.models.hybrid import HybridModel
-from mythos_b200.models.hybrid_config import HybridConfig, lebedra_config, teganex_config
+from mythos_b200.models.hybrid import HybridModel, expected_shapes
+from mythos_b200.models.hybrid_config import FrequencyScaling, HybridConfig, Rotation, dogozen_config, lebedra_config, teganex_config
 from mythos_b200.oil.importers import read_safetensors_torch, write_safetensors
 from mythos_b200.oil.model_io import load_model
 
@@ -55,6 +55,47 @@ def test_bad_latent_configurations_are_refused(change):
         HybridConfig.from_dict(raw)
 
 
+@pytest.mark.parametrize("change", [
+    lambda c: c["layers"][2]["mixer"].update(kv_from=1),            # other widths
+    lambda c: c["layers"][2]["mixer"].update(kv_from=2),
+    lambda c: c["layers"][0]["mixer"].update(kv_from=2),            # a later layer
+    lambda c: c["layers"][0]["mixer"]["q_temp"].update(every=0),
+    lambda c: c["layers"][1]["mixer"]["left"]["rot"].update(dims=9),
+    lambda c: c["layers"][1]["mixer"]["left"]["rot"].update(dims=22),
+    lambda c: c["layers"][1]["mixer"]["left"]["mask"].update(size=-1),
+    lambda c: c["layers"][1]["mixer"]["right"].update(state=0),
+    lambda c: c["layers"][1]["mlp"]["router"]["groups"].update(keep=4),
+    lambda c: c["layers"][1]["mlp"].update(kind="other"),
+    lambda c: c["layers"][1].update(type="gla"),
+])
+def test_bad_scan_configurations_are_refused(change):
+    raw = json.loads(json.dumps(hu.CONFIGS["scan_ragged"]))
+    change(raw)
+    with pytest.raises((ValueError, KeyError)):
+        HybridConfig.from_dict(raw)
+
+
+def test_optional_parts_of_a_configuration():
+    raw = json.loads(json.dumps(hu.CONFIGS["scan_ragged"]))
+    del raw["layers"][0]["mixer"]["q_temp"], raw["layers"][1]["mixer"]["left"]["mask"], raw["layers"][1]["mlp"]["router"]["groups"]
+    raw["layers"][1]["mlp"]["shared"], raw["logit_softcap"], raw["layers"][0]["mlp"] = None, None, None
+    c = HybridConfig.from_dict(raw)
+    left, moe = c.layers[1].mixer.left, c.layers[1].mlp
+    assert c.layers[0].mixer.q_temp is None and left.window == 0 and (moe.groups, moe.keep, moe.shared) == (1, 1, 0)
+    assert c.logit_softcap == 0.0 and c.layers[0].mlp is None
+    shapes = expected_shapes(c)
+    assert "l1.mlp.shared.gate" not in shapes and "l2.mix.k" not in shapes and "l2.mix.v.b" not in shapes and "l0.mix.k.b" in shapes
+
+
+@pytest.mark.parametrize("rot", [{"base": 1e4, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 256}},
+                                 {"base": 500.0, "dims": 10}, {"base": 1e5, "dims": 48, "scaling": {"factor": 2.0, "low": 2.0, "high": 2.0, "original": 64}}])
+def test_rotation_frequencies(rot):
+    sc = rot.get("scaling")
+    r = Rotation(rot["base"], rot["dims"], FrequencyScaling(**sc) if sc else None)
+    want = torch.tensor(oracle.frequencies(rot), dtype=torch.float64) / (2 * torch.pi)
+    assert torch.allclose(torch.tensor(r.turns(), dtype=torch.float64), want, rtol=1e-12, atol=0)
+
+
 def _write(folder, cfg, w):
     os.makedirs(folder, exist_ok=True)
     with open(os.path.join(folder, "config.json"), "w") as f:
@@ -95,6 +136,21 @@ def test_lebedra_folder_loads_through_the_registry(tmp_path):
         HybridModel(HybridConfig.from_dict(cfg), w)
 
 
+def test_dogozen_folder_loads_through_the_registry(tmp_path):
+    cfg = hu.CONFIGS["scan_ragged"]
+    w = hu.weights(cfg, 3)
+    _write(str(tmp_path), cfg, w)
+    m, _ = load_model(str(tmp_path))
+    assert isinstance(m, HybridModel) and m.cfg.architecture == "Dogozen" and m.cfg.tied_head and m.cfg.norm_offset == 1.0
+    assert torch.equal(m.tensor("l1.mix.right.A_log"), w["l1.mix.right.A_log"]) and "head" not in dict(m.named_tensors())
+    from mythos_b200.tools.info import main as info_main
+
+    assert info_main([str(tmp_path)]) == 0
+    del w["l1.mix.left.sink"]
+    with pytest.raises(KeyError):
+        HybridModel(HybridConfig.from_dict(cfg), w)
+
+
 def test_missing_and_misshapen_tensors_are_refused():
     cfg = hu.CONFIGS["single"]
     hc = HybridConfig.from_dict(cfg)
@@ -112,6 +168,8 @@ def test_named_configuration_has_consistent_shapes():
     m = HybridModel.random(cfg, low_rank=8)
     assert m.param_count() == sum(t.numel() for _, t in m.named_tensors())
     assert [s.type for s in cfg.layers] == ["gla", "gla", "gla", "parallel"]
+    m = HybridModel.random(dogozen_config(width=256, layers=6, vocab=64, experts=16, top=2))
+    assert m.param_count() == sum(t.numel() for _, t in m.named_tensors()) and m.cfg.layers[4].mixer.kv_from == 2
     m = HybridModel.random(lebedra_config(width=256, layers=2, vocab=64, experts=8, top=2))
     assert m.param_count() == sum(t.numel() for _, t in m.named_tensors()) and m.tensor("l1.mlp.e7.gate").shape[1] == 256
 
@@ -334,3 +392,71 @@ def test_a_mistake_in_a_latent_or_expert_mechanism_shows(slip, monkeypatch):
     monkeypatch.setattr(oracle, fn, wrong)
     e = hu.row_errors(oracle.forward(cfg, w, toks), right)
     assert float(e.max()) > 0.06 and float((e > 1e-3).double().mean()) > 0.3, (float(e.max()), float(e.median()))
+
+
+def _scan_slips():
+    """Mistakes in Dogozen's mechanisms: name -> (function of the oracle, wrong version)."""
+    att, rot, freq, temp, scan, choose, cap, conv, norm, soft, shared = (
+        oracle.window_sink_attention, oracle.rotate_halves, oracle.frequencies, oracle.query_temperature, oracle.selective_scan,
+        oracle.choose_by_sigmoid, oracle.soft_cap, oracle.short_conv, oracle.rms_norm_around_zero, oracle.softplus, oracle.tempered_attention)
+
+    def interleaved(x, pos, r):
+        n = r["dims"]
+        order = torch.tensor([2 * i for i in range(n // 2)] + [2 * i + 1 for i in range(n // 2)] + list(range(n, x.shape[-1])))
+        out = torch.empty_like(x)
+        out[..., order] = rot(x[..., order], pos, r)
+        return out
+
+    def late_read(x, dt, A, B, C, D):                      # read-out before the current token's write
+        S, out = torch.zeros_like(A), torch.zeros_like(x)
+        for t in range(x.shape[0]):
+            S = torch.exp(dt[t][:, None] * A) * S
+            out[t] = S @ C[t] + D * x[t]
+            S = S + (dt[t] * x[t])[:, None] * B[t][None, :]
+        return out
+
+    def one_best(z, r):                                    # groups by their best expert alone
+        s, g = torch.sigmoid(z), r["groups"]
+        size = r["experts"] // g["count"]
+        best = torch.topk(s.view(g["count"], size).amax(1), g["keep"]).indices.tolist()
+        picked = sorted((e for e in range(r["experts"]) if e // size in best), key=lambda e: -float(s[e]))[: r["top"]]
+        total = sum(s[e] for e in picked)
+        return [(e, s[e] / total * r["scale"]) for e in picked]
+
+    def own_keys(h, W, p, c, eps, kv):                     # a sharing layer whose queries meet the previous layer's stream
+        return shared(h, W, p, {k: v for k, v in c.items() if k != "q_temp"}, eps, kv)
+
+    return {"window_longer": ("window_sink_attention", lambda q, k, v, sc, w=None, s=None: att(q, k, v, sc, w and w + 1, s)),
+            "window_shorter": ("window_sink_attention", lambda q, k, v, sc, w=None, s=None: att(q, k, v, sc, w and w - 1, s)),
+            "no_sink": ("window_sink_attention", lambda q, k, v, sc, w=None, s=None: att(q, k, v, sc, w)),
+            "scaled_sink": ("window_sink_attention", lambda q, k, v, sc, w=None, s=None: att(q, k, v, sc, w, None if s is None else s * sc)),
+            "no_rotation": ("rotate_halves", lambda x, pos, r: x), "interleaved": ("rotate_halves", interleaved),
+            "late_positions": ("rotate_halves", lambda x, pos, r: rot(x, pos if x.shape[1] == 2 else pos + 1, r)),
+            "no_temperature": ("query_temperature", lambda pos, c: torch.ones(pos.shape, dtype=torch.float64)),
+            "late_temperature": ("query_temperature", lambda pos, c: temp(pos - 1, c)),
+            "unused_temperature": ("tempered_attention", own_keys),
+            "late_read": ("selective_scan", late_read),
+            "no_skip": ("selective_scan", lambda x, dt, A, B, C, D: scan(x, dt, A, B, C, D * 0)),
+            "swapped_maps": ("selective_scan", lambda x, dt, A, B, C, D: scan(x, dt, A, C, B, D)),
+            "no_step_in_input": ("selective_scan", lambda x, dt, A, B, C, D: scan(x / dt, dt, A, B, C, D * dt.mean())),
+            "shifted_conv": ("short_conv", lambda x, w: conv(torch.cat([torch.zeros_like(x[:1]), x[:-1]]), w)),
+            "linear_steps": ("softplus", lambda z: torch.clamp(z, min=0)),
+            "one_best": ("choose_by_sigmoid", one_best),
+            "no_groups": ("choose_by_sigmoid", lambda z, r: choose(z, {**r, "groups": None})),
+            "no_router_scale": ("choose_by_sigmoid", lambda z, r: choose(z, {**r, "scale": 1.0})),
+            "plain_weights": ("choose_by_sigmoid", lambda z, r: [(e, torch.sigmoid(z[e]) * r["scale"]) for e, _ in choose(z, r)]),
+            "norm_without_one": ("rms_norm_around_zero", lambda x, w, e: norm(x, w - 1, e)),
+            "no_cap": ("soft_cap", lambda x, c: x)}
+
+
+@pytest.mark.parametrize("slip", sorted(_scan_slips()))
+def test_a_mistake_in_a_scan_or_window_mechanism_shows(slip, monkeypatch):
+    """Far above what 32-bit comparisons allow (5e-5) on many rows, and on some above the bf16 tolerance as well."""
+    cfg = json.loads(json.dumps(hu.CONFIGS["scan_ragged"]))
+    cfg["layers"][1]["mlp"] = hu.sigmoid_moe(12, 2, 20, 3, 1, 1.7, 28)
+    w, toks = hu.weights(cfg, 5), hu.tokens(cfg, 48)
+    right = oracle.forward(cfg, w, toks)
+    fn, wrong = _scan_slips()[slip]
+    monkeypatch.setattr(oracle, fn, wrong)
+    e = hu.row_errors(oracle.forward(cfg, w, toks), right)
+    assert float(e.max()) > 0.06 and float((e > 1e-3).double().mean()) > 0.25, (float(e.max()), float(e.median()))
