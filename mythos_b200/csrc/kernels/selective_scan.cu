@@ -61,6 +61,27 @@ __device__ __forceinline__ float log1p_unit(float e) {
   return 2.f * t * p;
 }
 __device__ __forceinline__ float softplus_fast(float z) { return fmaxf(z, 0.f) + log1p_unit(fast_exp2(-1.4426950408889634f * fabsf(z))); }
+// 2^x for x <= 0 by its Taylor series about the nearest integer, the last step one rounding: a decay just below one is
+// off by half a unit in the last place either way, so thousands of them in a row do not drift.
+__device__ __forceinline__ float exp2_series(float x) {
+  x = fmaxf(x, -126.f);
+  const float i = rintf(x), f = x - i;
+  float p = fmaf(f, 1.5252734e-5f, 1.5403530e-4f);       // ln(2)^k / k!, k = 7 .. 1
+  p = fmaf(p, f, 1.3333558e-3f);
+  p = fmaf(p, f, 9.6181291e-3f);
+  p = fmaf(p, f, 5.5504109e-2f);
+  p = fmaf(p, f, 2.4022651e-1f);
+  p = fmaf(p, f, 6.9314718e-1f);
+  p = fmaf(p, f, 1.f);
+  return x <= -126.f ? 0.f : p * __int_as_float(((int)i + 127) << 23);
+}
+// Decays, step sizes and gates: with 32-bit activations as exactly as 32-bit arithmetic goes, with 16-bit ones by the
+// special-function unit (relative error about 2^-22).
+template <typename T>
+__device__ __forceinline__ float decay_t(float x) {
+  if constexpr (sizeof(T) == 2) return fast_exp2(x);
+  else return exp2_series(x);
+}
 // z / (1 + e^-z)
 __device__ __forceinline__ float silu_fast(float z) { return z * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * z)); }
 
@@ -119,6 +140,11 @@ template <typename T>
 __device__ __forceinline__ float silu_t(float z) {
   if constexpr (sizeof(T) == 2) return silu_fast(z);
   else return silu_f(z);
+}
+template <typename T>
+__device__ __forceinline__ float softplus_t(float z) {
+  if constexpr (sizeof(T) == 2) return softplus_fast(z);
+  else return softplus_f(z);
 }
 template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(256)
@@ -283,7 +309,7 @@ struct ChunkScratch {
 };
 
 // State update of one token on packed pairs of state values; the read-out is formed when Y.
-template <int NR, bool Y>
+template <typename T, int NR, bool Y>
 __device__ __forceinline__ float advance(uint64_t (&S)[NR / 2], const uint64_t (&a)[NR / 2], float dt, float x, const float* sB,
                                          const float* sC) {
   const uint64_t dt2 = f32x2(dt, dt), dx2 = f32x2(dt * x, dt * x);
@@ -298,7 +324,7 @@ __device__ __forceinline__ float advance(uint64_t (&S)[NR / 2], const uint64_t (
       const int n = 2 * i + j;
       float e0, e1;
       f32x2_unpack(mul_f32x2(dt2, a[n]), e0, e1);
-      S[n] = fma_f32x2(f32x2(fast_exp2(e0), fast_exp2(e1)), S[n], mul_f32x2(dx2, j ? B.y : B.x));
+      S[n] = fma_f32x2(f32x2(decay_t<T>(e0), decay_t<T>(e1)), S[n], mul_f32x2(dx2, j ? B.y : B.x));
       if constexpr (Y) y[j] = fma_f32x2(S[n], j ? C.y : C.x, y[j]);
     }
   }
@@ -418,7 +444,7 @@ selective_scan_kernel(const __grid_constant__ SelectiveSpec s, const __grid_cons
       for (int n = 0; n < NR / 2; ++n) {
         float d0, d1;
         f32x2_unpack(mul_f32x2(f32x2(sum, sum), a[n]), d0, d1);
-        S[n] = fma_f32x2(f32x2(fast_exp2(d0), fast_exp2(d1)), S[n], e[n]);
+        S[n] = fma_f32x2(f32x2(decay_t<T>(d0), decay_t<T>(d1)), S[n], e[n]);
       }
     }
   } else {
@@ -472,17 +498,17 @@ selective_scan_kernel(const __grid_constant__ SelectiveSpec s, const __grid_cons
 #pragma unroll
       for (int g = 0; g < G; ++g) {
         x[g] = ldf(sx + (u0 + g) * channels);
-        d[g] = softplus_fast(sd[(u0 + g) * channels] + bias);
+        d[g] = softplus_t<T>(sd[(u0 + g) * channels] + bias);
         if constexpr (!OUT) total += d[g];
       }
 #pragma unroll
-      for (int g = 0; g < G; ++g) y[g] = advance<NR, OUT>(S, a, d[g], x[g], pB + (u0 + g) * state_p, pC + (u0 + g) * state_p);
+      for (int g = 0; g < G; ++g) y[g] = advance<T, NR, OUT>(S, a, d[g], x[g], pB + (u0 + g) * state_p, pC + (u0 + g) * state_p);
       if constexpr (OUT) {
         for (int o = 1; o < lanes; o <<= 1)
 #pragma unroll
           for (int g = 0; g < G; ++g) y[g] += __shfl_xor_sync(0xffffffffu, y[g], o);
 #pragma unroll
-        for (int g = 0; g < G; ++g) y[g] = fmaf(D, x[g], y[g]) * scale * silu_fast(ldf(sz + (u0 + g) * channels));
+        for (int g = 0; g < G; ++g) y[g] = fmaf(D, x[g], y[g]) * scale * silu_t<T>(ldf(sz + (u0 + g) * channels));
         if (sub == 0) {                            // the output takes x's place
 #pragma unroll
           for (int g = 0; g < G; ++g) stf(sx + (u0 + g) * channels, y[g]);
@@ -563,12 +589,12 @@ selective_step_kernel(SelectiveSpec s, SelectiveInputs in, RaggedBatch rb, int l
     }
     for (int o = 1; o < lanes; o <<= 1) pre += __shfl_xor_sync(0xffffffffu, pre, o);
   }
-  const float d = softplus_fast(pre + in.dt_bias[ch]);
-  float y = advance<NR, true>(S, a, d, x, sB + sub * NR, sC + sub * NR);
+  const float d = softplus_t<T>(pre + in.dt_bias[ch]);
+  float y = advance<T, NR, true>(S, a, d, x, sB + sub * NR, sC + sub * NR);
   for (int o = 1; o < lanes; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
   if (!live) return;
   store_pairs<NR>(slot, S);
-  if (sub == 0) stf(out + b * ldo + ch, fmaf(in.d[ch], x, y) * silu_fast(z) * s.out_scale);
+  if (sub == 0) stf(out + b * ldo + ch, fmaf(in.d[ch], x, y) * silu_t<T>(z) * s.out_scale);
 }
 
 void check_spec(const SelectiveSpec& s) {

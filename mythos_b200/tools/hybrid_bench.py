@@ -167,7 +167,7 @@ def _dense_attention_rows(K, H, C, st, rnd, h, kv):
           lambda: C.flash_attn_paged_prefill(q, kc, vc, table, b[0], b[1], o, S, 128 ** -0.5, st),
           flops=2.0 * B * h * (S * (S + 1) / 2) * 256)
     sms = torch.cuda.get_device_properties(0).multi_processor_count
-    for NB, ctx in ((16, 4096), (64, 1024)):
+    for NB, ctx in ((16, 4096), (64, 1024), (16, 1024)):
         pages = NB * ctx // PAGE
         table = torch.randperm(pages, device="cuda").to(torch.int32).view(NB, -1)
         kc, vc, q, o = rnd(pages, PAGE, kv, 128), rnd(pages, PAGE, kv, 128), rnd(NB, h, 128), rnd(NB, h, 128)
