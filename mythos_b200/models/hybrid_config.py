@@ -477,7 +477,7 @@ def dogozen_config(width: int = 2048, layers: int = 8, vocab: int = 32000, max_p
                                rotation=Rotation(500000.0, 128, FrequencyScaling(8.0, 1.0, 4.0, 8192))),
                 SelectiveMixer(2 * width, 16, max(8, width // 16), 4), (1.0, 1.0)), moe))
     return HybridConfig(vocab, width, out, 1e-6, max_seq_len=max_positions, architecture="Dogozen", position_table=False,
-                        norm_offset=1.0, tied_head=True, logit_softcap=30.0)
+                        norm_offset=1.0, tied_head=True, logit_softcap=50.0)
 
 
 register("Dogozen", HybridConfig.from_dict, "mythos_b200.models.hybrid:HybridModel")
