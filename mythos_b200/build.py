@@ -27,7 +27,7 @@ CSRC = PKG / "csrc"
 OBJ = PKG / "csrc" / "build"
 
 # Sources of the layer-list model module: those it has to itself, and those it shares with ``_C``.
-HYBRID_ONLY = ["hybrid_ops", "recurrent", "chunk_scan", "selective_scan", "gemm_decode", "expert_route", "latent"]
+HYBRID_ONLY = ["hybrid_ops", "recurrent", "chunk_scan", "selective_scan", "short_conv", "gemm_decode", "expert_route", "latent"]
 HYBRID_SOURCES = HYBRID_ONLY + ["host_util", "gemm", "gemm_2cta", "sampler", "attention_fwd", "attention_fwd2", "paged_attn"]
 
 NVCC_FLAGS = [

@@ -36,8 +36,53 @@ mb::RaggedBatch ragged(const std::vector<Tensor>& batch) {
                          batch[3].data_ptr<int>(), batch[4].data_ptr<int>(), (int)n, (int)rows};
 }
 
+// Short causal convolution of one layer's channels, built once per layer: w [taps, channels] (last row: the current
+// token's), state [slots, taps - 1, channels].
+struct Conv {
+  int channels = 0, taps = 0;
+  bool residual = false;
+  Tensor w;
+  OptTensor bias, state;
+
+  void validate() const {
+    TORCH_CHECK(channels > 0 && taps > 0 && taps <= 64, "convolution: sizes");
+    fptr(w, (int64_t)taps * channels, "convolution: w");
+    fptr(bias, channels, "convolution: bias");
+    TORCH_CHECK(taps == 1 || state.has_value(), "convolution: more than one tap needs a state");
+    if (taps > 1) fptr(state, state->size(0) * (taps - 1) * channels, "convolution: state");
+  }
+  mb::ShortConv raw() const {
+    return mb::ShortConv{channels, taps, residual, w.data_ptr<float>(), fptr(bias, channels, "bias"),
+                         taps > 1 ? const_cast<float*>(fptr(state, 0, "state")) : nullptr};
+  }
+  // x: [rows, >= off + channels], columns from off on
+  void run(const Tensor& x, int64_t off, const std::vector<Tensor>& batch, bool one_token, Tensor& y) const {
+    const auto rb = ragged(batch);
+    const bool f32 = is_f32(y, "y");
+    chk_rows(x, f32, rb.rows, off + channels, "x");
+    chk_rows(y, f32, rb.rows, channels, "y");
+    TORCH_CHECK(y.stride(0) == y.size(1), "convolution: y must be contiguous");
+    c10::cuda::CUDAGuard guard(y.device());
+    mb::short_conv(f32, raw(), static_cast<const char*>(x.data_ptr()) + off * (f32 ? 4 : 2), x.stride(0), rb, one_token, y.data_ptr(),
+                   y.stride(0), cur_stream());
+  }
+  // The same inside a kernel that writes the convolution's input, one token per sequence.
+  mb::ConvTail tail(const std::vector<Tensor>& batch, Tensor& out, bool f32, int64_t rows) const {
+    const auto rb = ragged(batch);
+    chk_rows(out, f32, rows, channels, "convolution output");
+    TORCH_CHECK(rb.rows == rows && rb.n_seq == rows && residual && !bias.has_value(), "convolution tail: one token per sequence");
+    return mb::ConvTail{raw(), rb.slots, rb.kv_lens, out.data_ptr(), out.stride(0)};
+  }
+};
+using ConvArg = std::optional<std::tuple<Conv, std::vector<Tensor>, Tensor>>;     // convolution, batch, output
+mb::ConvTail conv_tail(const ConvArg& a, bool f32, int64_t rows) {
+  if (!a.has_value()) return mb::ConvTail{};
+  Tensor out = std::get<2>(*a);
+  return std::get<0>(*a).tail(std::get<1>(*a), out, f32, rows);
+}
+
 void embed_pos_norm(const Tensor& ids, const Tensor& pos, const Tensor& embed, const OptTensor& pos_table, double scale,
-                    const OptTensor& gamma, Tensor& x, Tensor& h, double eps) {
+                    const OptTensor& gamma, Tensor& x, Tensor& h, double eps, const OptTensor& gamma0, const ConvArg& conv) {
   const bool f32 = is_f32(h, "h");
   const int64_t rows = ids.numel(), dim = embed.size(1);
   chk_c(ids, I32, "ids");
@@ -53,8 +98,33 @@ void embed_pos_norm(const Tensor& ids, const Tensor& pos, const Tensor& embed, c
   c10::cuda::CUDAGuard guard(h.device());
   mb::embed_pos_norm(f32, ids.data_ptr<int>(), pos.data_ptr<int>(), embed.data_ptr(), cptr(pos_table),
                      (int)embed.size(0), pos_table.has_value() ? (int)pos_table->size(0) : 1, (float)scale,
-                     fptr(gamma, dim, "gamma"), x.data_ptr<float>(), h.data_ptr(), h.stride(0), (int)rows, (int)dim,
-                     (float)eps, cur_stream());
+                     fptr(gamma0, dim, "gamma0"), fptr(gamma, dim, "gamma"), x.data_ptr<float>(), h.data_ptr(), h.stride(0),
+                     (int)rows, (int)dim, (float)eps, conv_tail(conv, f32, rows), cur_stream());
+}
+
+// x += mult * (y + bias); h = rms(x) * w_next, with conv also h + conv(h).
+void residual_norm(const Tensor& y, const OptTensor& bias, double mult, Tensor& x, const Tensor& w_next, Tensor& h, double eps,
+                   const ConvArg& conv) {
+  const bool f32 = is_f32(h, "h");
+  chk_c(x, F32, "x");
+  const int64_t rows = x.size(0), dim = x.size(1);
+  chk_rows(y, f32, rows, dim, "y");
+  chk_rows(h, f32, rows, dim, "h");
+  c10::cuda::CUDAGuard guard(h.device());
+  mb::residual_norm(f32, y.data_ptr(), y.stride(0), fptr(bias, dim, "bias"), (float)mult, x.data_ptr<float>(),
+                    fptr(w_next, dim, "w_next"), h.data_ptr(), h.stride(0), (int)rows, (int)dim, (float)eps,
+                    conv_tail(conv, f32, rows), cur_stream());
+}
+
+// out[:, :width] from y + bias; the rest of out's columns are zeroed.
+void poly_norm(const Tensor& y, const OptTensor& bias, const Tensor& abce, int64_t width, Tensor& out, double eps) {
+  const bool f32 = is_f32(out, "out");
+  const int64_t rows = out.size(0);
+  chk_rows(y, f32, rows, width, "y");
+  chk_rows(out, f32, rows, width, "out");
+  c10::cuda::CUDAGuard guard(out.device());
+  mb::poly_norm(f32, y.data_ptr(), y.stride(0), fptr(bias, width, "bias"), fptr(abce, 4, "abce"), out.data_ptr(), out.stride(0),
+                (int)rows, (int)width, (int)out.size(1), (float)eps, cur_stream());
 }
 
 void sandwich_norm(const Tensor& y1, const OptTensor& y2, const OptTensor& w1, const OptTensor& w2, const Tensor& w_post,
@@ -218,7 +288,7 @@ void gemm_decode(const Tensor& x, const Tensor& w, Tensor& out, int64_t f, int64
                   x.size(1) == w.size(1), "gemm_decode: operands");
   const int64_t n = f > 0 ? f : w.size(0);
   TORCH_CHECK(out.size(0) == x.size(0) && out.size(1) >= n && (f == 0 || f_off + f <= w.size(0)), "gemm_decode: shapes");
-  mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0, (float)cap};
+  mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0, (float)cap, nullptr, 0, 0};
   if (mul.has_value()) {
     TORCH_CHECK(ids.has_value() && mul->dim() == 2 && mul->stride(1) == 1 && mul->size(1) >= n, "gemm_decode: mul");
     chk(*mul, BF16, "mul");
@@ -234,8 +304,9 @@ void gemm_decode(const Tensor& x, const Tensor& w, Tensor& out, int64_t f, int64
                   (int)x.size(0), (int)n, (int)x.size(1), (float)alpha, tail, mb::GemmGroup{}, status_ptr(status), cur_stream());
 }
 
-// out[:, b] = x[:, b] w[b]^T for every b: x [rows, b, K], w [b, N, K], out [rows, b, N], inner strides 1.
-void gemm_heads(const Tensor& x, const Tensor& w, Tensor& out, const OptTensor& status) {
+// out[:, b] = x[:, b] w[b]^T for every b: x [rows, b, K], w [b, N, K], out [rows, b, N], inner strides 1. With gate
+// [rows, b * N] times its sigmoid.
+void gemm_heads(const Tensor& x, const Tensor& w, Tensor& out, const OptTensor& status, const OptTensor& gate) {
   const bool f32 = is_f32(x, "x");
   for (const Tensor* t : {&x, &w, (const Tensor*)&out}) {
     chk(*t, f32 ? F32 : BF16, "gemm_heads operand");
@@ -244,14 +315,25 @@ void gemm_heads(const Tensor& x, const Tensor& w, Tensor& out, const OptTensor& 
   const int64_t rows = x.size(0), b = x.size(1), K = x.size(2), N = w.size(1);
   TORCH_CHECK(w.size(0) == b && w.size(2) == K && out.size(0) == rows && out.size(1) == b && out.size(2) == N, "gemm_heads: shapes");
   if (rows == 0) return;
+  mb::GemmTail tail{};
+  if (gate.has_value()) {
+    chk_rows(*gate, f32, rows, b * N, "gate");
+    TORCH_CHECK(out.stride(1) == N, "gemm_heads: a gated output has its products side by side");
+    tail.gate = gate->data_ptr();
+    tail.ld_gate = gate->stride(0);
+    tail.gate_batch = N;
+  }
   c10::cuda::CUDAGuard guard(x.device());
-  if (f32)
+  if (f32) {
     mb::gemm_f32(x.data_ptr<float>(), x.stride(0), w.data_ptr<float>(), w.stride(1), out.data_ptr<float>(), out.stride(0), (int)rows,
                  (int)N, (int)K, 1.f, cur_stream(), (int)b, x.stride(1), w.stride(0), out.stride(1));
-  else
+    if (gate.has_value())
+      mb::sigmoid_mul(true, out.data_ptr(), out.stride(0), gate->data_ptr(), gate->stride(0), (int)rows, (int)(b * N), cur_stream());
+  } else {
     mb::gemm_decode(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(1), out.data_ptr(), false, out.stride(0), (int)rows, (int)N,
-                    (int)K, 1.f, mb::GemmTail{}, mb::GemmGroup{(int)b, x.stride(1), w.stride(0), out.stride(1), nullptr, 0},
+                    (int)K, 1.f, tail, mb::GemmGroup{(int)b, x.stride(1), w.stride(0), out.stride(1), nullptr, 0},
                     status_ptr(status), cur_stream());
+  }
 }
 
 mb::TileList tile_list(const Tensor& tiles, const Tensor& count) {
@@ -274,7 +356,7 @@ void gemm_tiles(const Tensor& x, const Tensor& w, Tensor& out, const Tensor& til
   const int64_t n = f > 0 ? f : w.size(1);
   TORCH_CHECK(out.size(1) >= n && (f == 0 || f_off + f <= w.size(1)), "gemm_tiles: shapes");
   const mb::TileList list = tile_list(tiles, count);
-  const mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0, 0.f};
+  const mb::GemmTail tail{f > 0 ? (int)f_off : 0, gate(act), nullptr, nullptr, 0, 0, 0.f, nullptr, 0, 0};
   c10::cuda::CUDAGuard guard(x.device());
   if (f32) {
     TORCH_CHECK(f == 0 && tile_rows == 64, "gemm_tiles: fp32 takes 64-row tiles and no tail");
@@ -355,9 +437,10 @@ void gelu_mul(Tensor& y, const Tensor& table, const Tensor& ids) {
 // ---- latent attention of one layer: sizes, offsets in the projection and parameters, built once per layer
 struct Latent {
   mb::LatentSpec s{};
-  int qr_off = 0, c_off = 0, kr_off = 0;
+  int qr_off = 0, c_off = 0, kr_off = 0, low_off = -1, low_rank = 0;   // c_off < 0: another layer's latents
   float scale = 1.f, eps = 1e-6f;
-  Tensor gamma, turns, sink;
+  OptTensor gamma, sink, low_gamma;
+  Tensor turns;
 
   mb::LatentPages pages(const Tensor& table, const Tensor& cache, bool f32, int64_t n_seq) const {
     chk_c(table, I32, "block_table");
@@ -366,21 +449,31 @@ struct Latent {
     TORCH_CHECK(cache.dim() == 4 && cache.size(2) == 1 && cache.size(3) == s.row(), "cache: [pages, page_size, 1, latent row]");
     return mb::LatentPages{cache.data_ptr(), table.data_ptr<int>(), (int)table.size(1), (int)cache.size(1), (int)cache.size(0)};
   }
-  void prep(Tensor& proj, const std::vector<Tensor>& batch, const Tensor& table, const Tensor& cache) const {
+  // What of a projection is prepared: latents (and what queries are a map of), rotated query columns, or both.
+  void prep(Tensor& proj, const std::vector<Tensor>& batch, const Tensor& table, const Tensor& cache, bool latents, bool queries) const {
     const auto rb = ragged(batch);
-    const bool f32 = is_f32(proj, "proj");
-    chk_rows(proj, f32, rb.rows, std::max({qr_off + s.heads * s.rot_p, c_off + s.rank_p, kr_off + s.rot_p}), "proj");
+    const bool f32 = is_f32(proj, "proj"), own = latents && c_off >= 0, low = latents && low_off >= 0;
+    int cols = 0;
+    if (queries) cols = qr_off + s.heads * s.rot_p;
+    if (own) cols = std::max({cols, c_off + s.rank_p, kr_off + s.rot_p});
+    if (low) cols = std::max(cols, low_off + (low_rank + 7) / 8 * 8);
+    if (cols == 0) return;
+    chk_rows(proj, f32, rb.rows, cols, "proj");
+    const mb::LatentPrep p{low ? low_off : -1, low_rank, queries ? qr_off : -1, own ? c_off : -1, own ? kr_off : -1,
+                           fptr(low_gamma, low_rank, "low_gamma"), fptr(gamma, s.rank, "gamma"), turns.data_ptr<double>()};
     c10::cuda::CUDAGuard guard(proj.device());
-    mb::latent_prep(f32, proj.data_ptr(), proj.stride(0), qr_off, c_off, kr_off, gamma.data_ptr<float>(),
-                    turns.data_ptr<double>(), s, rb, pages(table, cache, f32, rb.n_seq), eps, cur_stream());
+    mb::latent_prep(f32, proj.data_ptr(), proj.stride(0), p, s, rb, pages(table, cache, f32, rb.n_seq), eps, cur_stream());
   }
-  void gather(const Tensor& table, const Tensor& cache, const Tensor& cu_k, int64_t max_kv, Tensor& out) const {
+  void gather(const Tensor& table, const Tensor& cache, const Tensor& cu_k, const Tensor& first, int64_t max_kv, Tensor& out) const {
     chk_c(out, BF16, "out");
     chk_c(cu_k, I32, "cu_k");
     TORCH_CHECK(out.dim() == 2 && out.size(1) == s.row(), "gather: out");
     const int n_seq = (int)cu_k.numel() - 1;
+    chk_c(first, I32, "first");
+    TORCH_CHECK(first.numel() == n_seq, "gather: first");
     c10::cuda::CUDAGuard guard(out.device());
-    mb::latent_gather(s, pages(table, cache, false, n_seq), cu_k.data_ptr<int>(), n_seq, (int)max_kv, out.data_ptr(), cur_stream());
+    mb::latent_gather(s, pages(table, cache, false, n_seq), cu_k.data_ptr<int>(), first.data_ptr<int>(), n_seq, (int)max_kv,
+                      out.data_ptr(), cur_stream());
   }
   mb::LatentQuery query(const Tensor& q_lat, const Tensor& proj, const Tensor& row_seq, const Tensor& pos, const Tensor& o,
                         bool f32) const {
@@ -401,7 +494,7 @@ struct Latent {
     const bool f32 = is_f32(q_lat, "q_lat");
     const auto q = query(q_lat, proj, row_seq, pos, o, f32);
     c10::cuda::CUDAGuard guard(o.device());
-    mb::latent_attn_any(f32, q, s, pages(table, cache, f32, 0), sink.data_ptr<float>(), o.data_ptr(), scale, cur_stream());
+    mb::latent_attn_any(f32, q, s, pages(table, cache, f32, 0), fptr(sink, s.heads, "sink"), o.data_ptr(), scale, cur_stream());
   }
   bool decode_ok(int64_t page_size) const { return mb::latent_decode_ok(s, (int)page_size); }
   void attn_decode(const Tensor& q_lat, const Tensor& proj, const Tensor& row_seq, const Tensor& pos, const Tensor& table,
@@ -410,14 +503,15 @@ struct Latent {
     chk_c(scratch, F32, "scratch");
     TORCH_CHECK(splits == 1 || scratch.numel() >= (int64_t)q.rows * s.heads * splits * (s.rank_p + 4), "attn_decode: scratch");
     c10::cuda::CUDAGuard guard(o.device());
-    mb::latent_attn_decode(q, s, pages(table, cache, false, 0), sink.data_ptr<float>(), o.data_ptr(), scratch.data_ptr<float>(),
+    mb::latent_attn_decode(q, s, pages(table, cache, false, 0), fptr(sink, s.heads, "sink"), o.data_ptr(), scratch.data_ptr<float>(),
                            (int)splits, scale, status_ptr(status), cur_stream());
   }
   bool prefill_ok(int64_t dim_p, int64_t vdim_p) const { return mb::flash_attn_ragged_ok((int)dim_p, s.rot_p, (int)vdim_p); }
-  // q, kv: [rows, heads, width] views (unrotated queries; expanded keys and values), latents [keys, row], o [rows, heads, vdim]
+  // q, kv: [rows, heads, width] views (unrotated queries; expanded keys and values), latents [keys, row], key_lens keys of every
+  // sequence, o [rows, heads, vdim], gate [rows, heads * vdim] or null
   void attn_prefill(const Tensor& q, const Tensor& proj, const Tensor& k, const Tensor& v, const Tensor& latents,
-                    const std::vector<Tensor>& batch, const Tensor& cu_k, int64_t max_q, int64_t min_q, Tensor& o,
-                    const OptTensor& status) const {
+                    const std::vector<Tensor>& batch, const Tensor& cu_k, const Tensor& key_lens, int64_t max_q, int64_t min_q,
+                    const OptTensor& gate, Tensor& o, const OptTensor& status) const {
     const auto rb = ragged(batch);
     for (const Tensor* t : {&q, &k, &v, (const Tensor*)&o}) {
       chk(*t, BF16, "attn_prefill operand");
@@ -426,6 +520,8 @@ struct Latent {
     chk_rows(proj, false, rb.rows, qr_off + s.heads * s.rot_p, "proj");
     chk_c(latents, BF16, "latents");
     chk_c(cu_k, I32, "cu_k");
+    chk_c(key_lens, I32, "key_lens");
+    TORCH_CHECK(key_lens.numel() == rb.n_seq, "attn_prefill: key_lens");
     TORCH_CHECK(q.size(0) == rb.rows && o.size(0) == rb.rows && k.size(0) == v.size(0) && k.stride(0) == v.stride(0) &&
                     q.size(2) == k.size(2) && v.size(2) == o.size(2) && proj.stride(0) == q.stride(0) && latents.size(0) == k.size(0) &&
                     latents.size(1) == s.row() && cu_k.numel() == rb.n_seq + 1, "attn_prefill: shapes");
@@ -442,8 +538,14 @@ struct Latent {
     a.ldo = o.stride(0);
     a.cu_q = rb.cu_q;
     a.cu_k = cu_k.data_ptr<int>();
-    a.kv_lens = rb.kv_lens;
-    a.sink = sink.data_ptr<float>();
+    a.key_lens = key_lens.data_ptr<int>();
+    a.sink = fptr(sink, s.heads, "sink");
+    if (gate.has_value()) {
+      chk_rows(*gate, false, rb.rows, s.heads * o.size(2), "gate");
+      a.gate = gate->data_ptr();
+      a.ld_gate = gate->stride(0);
+    }
+    a.window = s.window;
     a.batch = rb.n_seq;
     a.total_q = rb.rows;
     a.total_k = (int)k.size(0);
@@ -624,36 +726,28 @@ struct Recurrent {
 // The selective scan of one layer with its parameters and state, built once per layer.
 struct Selective {
   mb::SelectiveSpec s{};
-  int x_off = 0, z_off = 0, b_off = 0, c_off = 0;
-  Tensor conv_w, conv_b, a, d, dt_b, state, w_dt;
-  OptTensor conv_state;
+  int z_off = 0, b_off = 0, c_off = 0;
+  Tensor a, d, dt_b, state, w_dt;
 
   void validate() const {
     const int64_t sp = mb::selective_padded_state(s.state);
-    TORCH_CHECK(s.inner > 0 && s.state > 0 && s.rank > 0 && s.taps > 0, "selective: sizes");
+    TORCH_CHECK(s.inner > 0 && s.state > 0 && s.rank > 0, "selective: sizes");
     chk_c(state, F32, "state");
     TORCH_CHECK(state.dim() == 3 && state.size(1) == s.inner && state.size(2) == sp, "state: [slots, inner, padded state]");
-    fptr(conv_w, (int64_t)s.taps * s.inner, "conv_w");
-    for (const Tensor* t : {&conv_b, &d, &dt_b}) fptr(*t, s.inner, "selective: channel parameters");
+    for (const Tensor* t : {&d, &dt_b}) fptr(*t, s.inner, "selective: channel parameters");
     fptr(a, s.inner * sp, "a");
-    TORCH_CHECK(s.taps == 1 || conv_state.has_value(), "selective: conv_state");
-    fptr(conv_state, state.size(0) * (s.taps - 1) * s.inner, "conv_state");
     is_f32(w_dt, "w_dt");
     TORCH_CHECK(w_dt.dim() == 2 && w_dt.size(0) == s.inner && w_dt.stride(1) == 1 && w_dt.size(1) >= (s.rank + 7) / 8 * 8, "w_dt");
   }
   mb::SelectiveInputs inputs(const Tensor& proj, bool f32, int64_t rows) const {
-    chk_rows(proj, f32, rows, std::max(x_off, z_off) + s.inner, "proj");
+    chk_rows(proj, f32, rows, z_off + s.inner, "proj");
     mb::SelectiveInputs in{};
     in.proj = proj.data_ptr();
     in.ld = proj.stride(0);
-    in.x_off = x_off;
     in.z_off = z_off;
-    in.conv_w = conv_w.data_ptr<float>();
-    in.conv_b = conv_b.data_ptr<float>();
     in.a = a.data_ptr<float>();
     in.d = d.data_ptr<float>();
     in.dt_bias = dt_b.data_ptr<float>();
-    in.conv_state = const_cast<float*>(fptr(conv_state, 0, "conv_state"));
     in.state = state.data_ptr<float>();
     in.b_off = b_off;
     in.c_off = c_off;
@@ -668,14 +762,6 @@ struct Selective {
     in.low = low.data_ptr();
     in.ld_low = low.stride(0);
     return in;
-  }
-  void conv(const Tensor& proj, const std::vector<Tensor>& batch, bool one_token, Tensor& x) const {
-    const auto rb = ragged(batch);
-    const bool f32 = is_f32(x, "x");
-    chk_rows(x, f32, rb.rows, s.inner, "x");
-    TORCH_CHECK(x.stride(0) == x.size(1), "conv: x must be contiguous");
-    c10::cuda::CUDAGuard guard(x.device());
-    mb::selective_conv(f32, s, inputs(proj, f32, rb.rows), rb, one_token, x.data_ptr(), x.stride(0), cur_stream());
   }
   int64_t scratch_floats(int64_t n_seq, int64_t rows, int64_t max_q) const {
     return mb::selective_scratch(s, (int)n_seq, (int)rows, (int)max_q);
@@ -716,8 +802,27 @@ void soft_cap(Tensor& y, double cap) {
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.doc() = "sm_100a kernels of layer-list models";
-  m.def("embed_pos_norm", &embed_pos_norm);
   namespace py = pybind11;
+  py::class_<Conv>(m, "Conv")
+      .def(py::init([](int64_t channels, bool residual, const Tensor& w, const OptTensor& bias, const OptTensor& state) {
+             Conv c;
+             TORCH_CHECK(w.dim() == 2 && w.size(1) == channels, "convolution: w [taps, channels]");
+             c.channels = (int)channels;
+             c.taps = (int)w.size(0);
+             c.residual = residual;
+             c.w = w;
+             c.bias = bias;
+             c.state = state;
+             c.validate();
+             return c;
+           }),
+           py::arg("channels"), py::arg("residual"), py::arg("w"), py::arg("bias") = OptTensor(), py::arg("state") = OptTensor())
+      .def("run", &Conv::run);
+  m.def("embed_pos_norm", &embed_pos_norm, py::arg("ids"), py::arg("pos"), py::arg("embed"), py::arg("pos_table"), py::arg("scale"),
+        py::arg("gamma"), py::arg("x"), py::arg("h"), py::arg("eps"), py::arg("gamma0") = OptTensor(), py::arg("conv") = ConvArg());
+  m.def("residual_norm", &residual_norm, py::arg("y"), py::arg("bias"), py::arg("mult"), py::arg("x"), py::arg("w_next"), py::arg("h"),
+        py::arg("eps"), py::arg("conv") = ConvArg());
+  m.def("poly_norm", &poly_norm);
   m.def("sandwich_norm", &sandwich_norm, py::arg("y1"), py::arg("y2"), py::arg("w1"), py::arg("w2"), py::arg("w_post"), py::arg("x"),
         py::arg("w_next"), py::arg("h"), py::arg("eps"), py::arg("mult") = 1.0);
   m.def("expert_norm", &expert_norm, py::arg("y"), py::arg("shared"), py::arg("row"), py::arg("weight"), py::arg("w_post"), py::arg("x"),
@@ -725,7 +830,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_decode", &gemm_decode, py::arg("x"), py::arg("w"), py::arg("out"), py::arg("f"), py::arg("f_off"), py::arg("alpha"),
         py::arg("status"), py::arg("act") = Act(0, 0.0, 0.0), py::arg("mul") = OptTensor(), py::arg("ids") = OptTensor(),
         py::arg("cap") = 0.0);
-  m.def("gemm_heads", &gemm_heads);
+  m.def("gemm_heads", &gemm_heads, py::arg("x"), py::arg("w"), py::arg("out"), py::arg("status"), py::arg("gate") = OptTensor());
   m.def("gemm_tiles", &gemm_tiles);
   m.def("expert_select", &expert_select, py::arg("logits"), py::arg("correction"), py::arg("spec"), py::arg("tile_rows"), py::arg("idx"),
         py::arg("weight"), py::arg("slot"), py::arg("counts"), py::arg("offset"), py::arg("tiles"), py::arg("count"),
@@ -781,28 +886,41 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
       .def("decode", &Recurrent::decode)
       .def("norm_gate", &Recurrent::norm_gate);
   py::class_<Latent>(m, "Latent")
-      .def(py::init([](py::dict d, const Tensor& gamma, const Tensor& turns, const Tensor& sink) {
+      .def(py::init([](py::dict d, const OptTensor& gamma, const Tensor& turns, const OptTensor& sink, const OptTensor& low_gamma) {
         Latent l;
         auto geti = [&](const char* k) { return d[k].cast<int>(); };
-        l.s = mb::LatentSpec{geti("heads"), geti("rank"), geti("rot"), geti("rank_p"), geti("rot_p")};
+        l.s = mb::LatentSpec{geti("heads"), geti("rank"), geti("rot"), geti("rank_p"), geti("rot_p"),
+                             d.contains("window") ? geti("window") : 0, d.contains("rot_amp") ? d["rot_amp"].cast<float>() : 1.f};
+        TORCH_CHECK(l.s.window >= 0, "latent: window");
+        if (d.contains("low_off")) {
+          l.low_off = geti("low_off");
+          l.low_rank = geti("low_rank");
+          TORCH_CHECK(l.low_off >= 0 && l.low_off % 8 == 0 && l.low_rank > 0 && low_gamma.has_value(), "latent: low-rank queries");
+        }
         TORCH_CHECK(l.s.heads > 0 && l.s.rank > 0 && l.s.rot > 0 && l.s.rank_p >= l.s.rank && l.s.rot_p >= l.s.rot &&
                         l.s.rank_p % 8 == 0 && l.s.rot_p % 8 == 0, "latent: sizes");
         l.qr_off = geti("qr_off");
-        l.c_off = geti("c_off");
-        l.kr_off = geti("kr_off");
-        TORCH_CHECK((l.qr_off | l.c_off | l.kr_off) % 8 == 0, "latent: offsets");
+        l.c_off = d.contains("c_off") ? geti("c_off") : -1;
+        if (l.c_off >= 0) {
+          l.kr_off = geti("kr_off");
+          TORCH_CHECK(l.kr_off >= 0 && (l.c_off | l.kr_off) % 8 == 0 && gamma.has_value(), "latent: offsets");
+        }
+        TORCH_CHECK(l.qr_off >= 0 && l.qr_off % 8 == 0, "latent: offsets");
         l.scale = d["scale"].cast<float>();
         l.eps = d["eps"].cast<float>();
         fptr(gamma, l.s.rank, "gamma");
         fptr(sink, l.s.heads, "sink");
         chk_c(turns, torch::kFloat64, "turns");
         TORCH_CHECK(turns.numel() >= l.s.rot / 2, "latent: turns");
+        fptr(low_gamma, l.low_rank, "low_gamma");
         l.gamma = gamma;
         l.turns = turns;
         l.sink = sink;
+        l.low_gamma = low_gamma;
         return l;
-      }))
-      .def("prep", &Latent::prep)
+      }), py::arg("spec"), py::arg("gamma"), py::arg("turns"), py::arg("sink"), py::arg("low_gamma") = OptTensor())
+      .def("prep", &Latent::prep, py::arg("proj"), py::arg("batch"), py::arg("table"), py::arg("cache"), py::arg("latents") = true,
+           py::arg("queries") = true)
       .def("gather", &Latent::gather)
       .def("attn_any", &Latent::attn_any)
       .def("decode_ok", &Latent::decode_ok)
@@ -828,6 +946,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         t.p.v_off = geti("v_off", 0);
         t.p.norm_dim = geti("norm_dim", 0);
         t.p.rot = geti("rot", 0);
+        t.p.pairs = geti("pairs", 0) != 0;
+        t.p.rot_amp = getf("rot_amp", 1.f);
         t.p.temp_coef = getf("temp_coef", 0.f);
         t.p.temp_every = getf("temp_every", 1.f);
         t.p.eps = getf("eps", 1e-6f);
@@ -869,23 +989,18 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         Selective t;
         auto geti = [&](const char* k) { return spec[k].cast<int>(); };
         auto gett = [&](const char* k) { return tensors[k].cast<Tensor>(); };
-        t.s = mb::SelectiveSpec{geti("inner"), geti("state"), geti("rank"), geti("taps"), spec["out_scale"].cast<float>()};
-        t.x_off = geti("x_off");
+        t.s = mb::SelectiveSpec{geti("inner"), geti("state"), geti("rank"), spec["out_scale"].cast<float>()};
         t.z_off = geti("z_off");
         t.b_off = geti("b_off");
         t.c_off = geti("c_off");
-        t.conv_w = gett("conv_w");
-        t.conv_b = gett("conv_b");
         t.a = gett("a");
         t.d = gett("d");
         t.dt_b = gett("dt_b");
         t.state = gett("state");
         t.w_dt = gett("w_dt");
-        if (tensors.contains("conv_state")) t.conv_state = gett("conv_state");
         t.validate();
         return t;
       }))
-      .def("conv", &Selective::conv)
       .def("scratch_floats", &Selective::scratch_floats)
       .def("scan", &Selective::scan)
       .def("step", &Selective::step);

@@ -191,18 +191,22 @@ void flash_attn_paged_prefill(const void* q, long long q_tok_stride, const void*
 // whose key is shared by all heads and one more denominator logit per head (attention_fwd.cu, FA_RAGGED). Queries
 // [total_q, heads, dim] and [total_q, heads, rot] with row stride ldq, keys / values [total_k, heads, dim / vdim] with
 // row stride ldkv, shared key part [total_k, rot] with row stride ldk_rot, output [total_q, heads, vdim]. Sequence b:
-// query rows cu_q[b] .., key rows cu_k[b] .., kv_lens[b] keys; those with fewer than min_q new tokens are left out.
+// query rows cu_q[b] .., key rows cu_k[b] .., key_lens[b] keys, the last of which is its last query's (a window may have
+// left out earlier ones); sequences with fewer than min_q new tokens are left out. sink and gate (logits per output value,
+// [total_q, heads * vdim]) may be null; window 0: none.
 struct RaggedAttn {
   const void *q, *q_rot, *k, *k_rot, *v;
   void* o;
   long long ldq, ldkv, ldk_rot, ldo;
-  const int *cu_q, *cu_k, *kv_lens;
+  const int *cu_q, *cu_k, *key_lens;
   const float* sink;
-  int batch, total_q, total_k, max_q, min_q, heads, dim, rot, vdim;
+  const void* gate;
+  long long ld_gate;
+  int batch, total_q, total_k, max_q, min_q, heads, dim, rot, vdim, window;
   float scale;
 };
 bool flash_attn_ragged_ok(int dim, int rot, int vdim);
-void flash_attn_ragged(const RaggedAttn& a, int* status, cudaStream_t stream);   // gate: optional per-head output gate logits [total_q, heads]
+void flash_attn_ragged(const RaggedAttn& a, int* status, cudaStream_t stream);
 void flash_attn_bwd(const void* q, const void* k, const void* v, const void* o, const void* dout, const float* lse,
                     void* dq, void* dk, void* dv, float* dq_accum, float* delta, int batch, int seq, int heads,
                     int kv_heads, int head_dim, bool causal, float scale, int* status, cudaStream_t stream);

@@ -61,9 +61,10 @@ enum { FA_DENSE = 0, FA_PAGED = 1, FA_RAGGED = 2 };
 struct PagedPrefillArgs {
   const int* block_table;   // [batch, table_stride] page ids
   const int* cu_q;          // [batch + 1] first query row of every sequence
-  const int* kv_lens;       // [batch] keys visible to the LAST query of the sequence (prefix + new tokens)
+  const int* kv_lens;       // [batch] keys visible to the LAST query of the sequence (prefix + new tokens; FA_RAGGED: those
+                            // among its packed rows)
   int table_stride;
-  const __nv_bfloat16* gate;   // logits of an output gate (sigmoid), or null: [total_q, >= heads], or
+  const __nv_bfloat16* gate;   // logits of an output gate (sigmoid), or null: [total_q, >= heads] (FA_PAGED), or
   long long ld_gate;           // [total_q, heads * o_cols] with gate_channels
   bool gate_channels;
   const float* sink;           // [heads]
@@ -378,7 +379,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
               if (PAGED && c * 32 + i * 8 >= pa.o_cols) break;
-              if constexpr (MODE == FA_PAGED) {
+              if constexpr (PAGED) {
                 if (grow) {
                   float g[8];
                   unpack8(ldg8(grow, c * 32 + i * 8), g);
@@ -516,6 +517,8 @@ void flash_attn_ragged(const RaggedAttn& a, int* status, cudaStream_t stream) {
   MB_REQUIRE(flash_attn_ragged_ok(a.dim, a.rot, a.vdim), "flash_attn_ragged: head widths up to 128 + 64 and 128");
   MB_REQUIRE((a.dim | a.rot | a.vdim) % 8 == 0 && a.dim > 0 && a.rot > 0 && a.vdim > 0, "flash_attn_ragged: widths in units of 8");
   MB_REQUIRE((reinterpret_cast<uintptr_t>(a.o) & 15) == 0 && a.ldo % 8 == 0, "flash_attn_ragged: output alignment");
+  MB_REQUIRE(a.window >= 0 && (a.gate == nullptr || (a.ld_gate % 8 == 0 && (reinterpret_cast<uintptr_t>(a.gate) & 15) == 0)),
+             "flash_attn_ragged: window / gate alignment");
   if (a.batch == 0 || a.total_q == 0 || a.total_k == 0 || a.max_q == 0) return;
   // token-major [rows, heads, width] views: one box = 64 columns of one head
   auto map = [](const void* base, int rows, int heads, int width, long long ld, int box_rows) {
@@ -528,7 +531,8 @@ void flash_attn_ragged(const RaggedAttn& a, int* status, cudaStream_t stream) {
   const CUtensorMap tk = map(a.k, a.total_k, a.heads, a.dim, a.ldkv, FA_BN), tv = map(a.v, a.total_k, a.heads, a.vdim, a.ldkv, FA_BN);
   const CUtensorMap tk2 = map(a.k_rot, a.total_k, 1, a.rot, a.ldk_rot, FA_BN);
   const dim3 grid((a.max_q + 2 * FA_BM - 1) / (2 * FA_BM), a.heads, a.batch);
-  PagedPrefillArgs pa{nullptr, a.cu_q, a.kv_lens, 0, nullptr, 0, false, a.sink, 0, 1.f, a.cu_k, a.min_q, a.vdim};
+  PagedPrefillArgs pa{nullptr, a.cu_q, a.key_lens, 0, (const __nv_bfloat16*)a.gate, a.ld_gate, true, a.sink, a.window, 1.f, a.cu_k,
+                      a.min_q, a.vdim};
   auto go = [&](auto kern, int smem) {
     MB_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     kern<<<grid, FA_THREADS, smem, stream>>>(tq, tk, tv, (__nv_bfloat16*)a.o, nullptr, a.total_q, a.heads, a.heads, a.ldo, 1,

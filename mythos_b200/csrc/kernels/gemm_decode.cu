@@ -46,7 +46,9 @@ __device__ __forceinline__ float gd_ld_cluster(uint32_t addr) {
 }
 
 // Value of one output element before it is stored.
-__device__ __forceinline__ float gd_tail(const GemmTail& tail, float y, int token, int n) {
+__device__ __forceinline__ float gd_tail(const GemmTail& tail, float y, int token, int n, int batch) {
+  if (tail.gate != nullptr)
+    return y * sigmoid_f(__bfloat162float(static_cast<const __nv_bfloat16*>(tail.gate)[token * tail.ld_gate + batch * tail.gate_batch + n]));
   if (tail.cap > 0.f) return soft_cap_f(y, tail.cap);
   if (tail.mul == nullptr) return y;
   const int id = min(max(tail.mul_ids[token], 0), tail.vocab - 1);
@@ -179,7 +181,7 @@ gemm_decode_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
 #pragma unroll
       for (int p = 0; p < 8; ++p)
         if (p < splits) y += gd_ld_cluster(peer[p] + (t * GD_BM + threadIdx.x) * 4);
-      if (n < N) stf(out + (long long)(m0 + t) * ldo + n, gd_tail(tail, y * alpha, m0 + t, n));
+      if (n < N) stf(out + (long long)(m0 + t) * ldo + n, gd_tail(tail, y * alpha, m0 + t, n, x_batch));
     }
   } else {
     const int i = threadIdx.x & 63, n = n0 + i;
@@ -392,7 +394,7 @@ void gemm_decode(const void* x, long long ldx, const void* W, long long ldw, voi
   MB_REQUIRE(ldx % 8 == 0 && ldw % 8 == 0 && (!many || (group.x_batch % 8 == 0 && group.w_batch % 8 == 0)),
              "gemm_decode: strides must be multiples of 8 elements");
   MB_REQUIRE(f_off == 0 || f_off >= N, "gemm_decode: the up half starts after the gate half");
-  MB_REQUIRE((tail.mul != nullptr) + (f_off > 0) + (tail.cap > 0.f) <= 1, "gemm_decode: one tail at a time");
+  MB_REQUIRE((tail.mul != nullptr) + (f_off > 0) + (tail.cap > 0.f) + (tail.gate != nullptr) <= 1, "gemm_decode: one tail at a time");
   int mt = (M + 15) / 16 * 16;
   if (mt > 128) mt = 128;
   if (group.list) mt = group.mt;
@@ -432,7 +434,7 @@ void gemm_segments(const void* x, long long ldx, const void* W, long long ldw, l
   MB_REQUIRE(ldx % 8 == 0 && ldw % 8 == 0 && w_batch % 8 == 0 && ldo % 8 == 0 && N % 8 == 0 &&
                  (reinterpret_cast<uintptr_t>(out) & 15) == 0, "gemm_segments: alignment");
   MB_REQUIRE(tail.f_off == 0 || tail.f_off >= N, "gemm_segments: the up half starts after the gate half");
-  MB_REQUIRE(tail.mul == nullptr && tail.cap <= 0.f, "gemm_segments: gated tail only");
+  MB_REQUIRE(tail.mul == nullptr && tail.gate == nullptr && tail.cap <= 0.f, "gemm_segments: gated tail only");
   static bool configured = false;
   if (!configured) {
     MB_CUDA_CHECK(cudaFuncSetAttribute(gemm_segments_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, GS_SMEM));

@@ -20,11 +20,42 @@ struct RaggedBatch {
   int n_seq, rows;
 };
 
-// x[t] = embed[id] * scale + pos_table[pos] (fp32 stream; the table may be null),
+// ---- short causal convolution per channel (short_conv.cu): y = silu(conv(x) + bias), or residual: x + conv(x) + bias
+struct ShortConv {
+  int channels, taps;
+  bool residual;
+  const float *w, *bias;            // [taps, channels] (last row: the current token's), [channels] or null
+  float* state;                     // [slots][taps - 1][channels] last inputs of every sequence
+};
+// A ragged batch; columns [channels, ldy) are zeroed and the state advances. one_token: row b belongs to sequence b.
+void short_conv(bool f32, const ShortConv& s, const void* x, long long ldx, const RaggedBatch& rb, bool one_token, void* y,
+                long long ldy, cudaStream_t stream);
+
+// Where a kernel that writes a normalised row h of one token per sequence also writes h + conv(h): c.taps 0: nowhere.
+struct ConvTail {
+  ShortConv c;
+  const int *slots, *kv_lens;
+  void* out;
+  long long ld;
+};
+
+// x[t] = embed[id] * scale + pos_table[pos] (fp32 stream; the table may be null), with gamma0 normalised,
 // h[t] = rmsnorm(x[t]) * gamma, or x[t] with gamma null.
 void embed_pos_norm(bool f32, const int* ids, const int* pos, const void* embed, const void* pos_table, int vocab,
-                    int max_pos, float scale, const float* gamma, float* x, void* h, long long ldh, int rows, int dim,
-                    float eps, cudaStream_t stream);
+                    int max_pos, float scale, const float* gamma0, const float* gamma, float* x, void* h, long long ldh,
+                    int rows, int dim, float eps, const ConvTail& conv, cudaStream_t stream);
+
+// x += mult * (y + bias) (bias may be null);  h = rms(x) * w_next.
+void residual_norm(bool f32, const void* y, long long ldy, const float* bias, float mult, float* x, const float* w_next, void* h,
+                   long long ldh, int rows, int dim, float eps, const ConvTail& conv, cudaStream_t stream);
+
+// out = a N(z) + b N(z^2) + c N(z^3) + e with z = y + bias and abce = {a, b, c, e}, N dividing a row by its root mean
+// square over the `width` columns; columns [width, ldo) of out are zeroed.
+void poly_norm(bool f32, const void* y, long long ldy, const float* bias, const float* abce, void* out, long long ldo, int rows,
+               int width, int padded, float eps, cudaStream_t stream);
+
+// y[t, n] *= sigmoid(gate[t, n])
+void sigmoid_mul(bool f32, void* y, long long ldy, const void* gate, long long ld_gate, int rows, int width, cudaStream_t stream);
 
 // Output of a sublayer: y1 alone; (rms(y1) * w1 + rms(y2) * w2) / 2; or the sum over j < top of
 // weight[t, j] * y1[row[t, j]] (routed experts), plus y2[t] if there is one (their shared expert).
@@ -41,7 +72,8 @@ void sandwich_norm(bool f32, const SublayerOut& y, const float* w_post, float mu
                    long long ldh, int rows, int dim, float eps, cudaStream_t stream);
 
 // How projected heads become queries, keys and values: bias, RMS norm of every q and k head, rotation, query
-// temperature. q [rows, heads, dk] is written out, k and v go to their pages. dk and dv are the stored widths;
+// temperature. q [rows, heads, dk] is written out, k and v go to their pages; v may be the same columns as k (it is neither
+// normalised nor rotated). dk and dv are the stored widths;
 // columns past a head's true width are zero in the projection and stay zero.
 struct HeadPrep {
   int heads, kv_heads, dk, dv;
@@ -49,8 +81,10 @@ struct HeadPrep {
   const float *q_bias, *k_bias, *v_bias;      // [heads * dk], [kv_heads * dk], [kv_heads * dv], or null
   int norm_dim;                     // columns the norm averages over; 0: no norm
   const float *q_gamma, *k_gamma;   // [dk] norm weights, or null
-  const double* turns;              // revolutions per position of the pair (i, i + rot / 2)
+  const double* turns;              // revolutions per position of the pair (i, i + rot / 2), or (2i, 2i + 1) with pairs
   int rot;                          // rotated columns (0: none)
+  bool pairs;
+  float rot_amp;                    // factor of cosines and sines
   float temp_coef, temp_every;      // queries times 1 + coef ln(floor((pos + 1) / every) + 1); coef 0: none
   float eps;
 };
@@ -81,7 +115,8 @@ struct GateAct {
   float limit, alpha;       //    u' = u clamped to [-limit, limit]
 };
 // What a few-token GEMM does with the products of a row: nothing; a gated activation of two halves of W;
-// gelu_tanh(y) * mul[mul_ids[t] * ld_mul + n]; or a soft cap.
+// gelu_tanh(y) * mul[mul_ids[t] * ld_mul + n]; a soft cap; or y * sigmoid(gate[t * ld_gate + n]), in product b of a batch
+// + b * gate_batch.
 struct GemmTail {
   int f_off;                // > 0: W holds a gate matrix in rows [0, N) and an up matrix from row f_off
   GateAct act;
@@ -90,6 +125,8 @@ struct GemmTail {
   long long ld_mul;
   int vocab;                // rows of mul
   float cap;                // > 0: y <- cap tanh(y / cap)
+  const void* gate;
+  long long ld_gate, gate_batch;
 };
 // Several products in one launch: `batch` of them side by side (x, W and out advance by *_batch elements), or with
 // `list` (tile rows = mt: 16, 32, 64 or 128) rows grouped by matrix, W advancing by w_batch elements.
@@ -147,6 +184,8 @@ void expert_gather(const void* h, long long ldh_bytes, const RouterSpec& s, cons
 // multiple of 8 values with zeros; all heads read the same rows.
 struct LatentSpec {
   int heads, rank, rot, rank_p, rot_p;   // widths and their padded forms
+  int window;                            // keys a query sees, its own included (0: all earlier ones)
+  float rot_amp;                         // factor of cosines and sines
   __host__ __device__ int row() const { return rank_p + rot_p; }
 };
 struct LatentPages {
@@ -154,16 +193,22 @@ struct LatentPages {
   const int* table;
   int stride, page_size, pages;
 };
-// Latent norm, rotation of the key part and of the queries' rotated columns (in place), append to the pages.
-// turns[i]: revolutions per position of pair i.
-void latent_prep(bool f32, void* proj, long long ld, int qr_off, int c_off, int kr_off, const float* gamma,
-                 const double* turns, const LatentSpec& s, const RaggedBatch& rb, const LatentPages& pg, float eps,
-                 cudaStream_t stream);
-// Latent rows of the sequences' pages, packed: sequence b at rows cu_k[b] .. cu_k[b + 1] of out.
-void latent_gather(const LatentSpec& s, const LatentPages& pg, const int* cu_k, int n_seq, int max_kv, void* out,
+// Columns of a projection, each part left out with a negative offset: vectors that queries are a map of (low_off: RMS
+// norm over low_rank columns in place), the queries' rotated columns (qr_off: rotated in place), latent (c_off: RMS norm) and
+// rotated key part (kr_off: rotation), which go to the pages. Columns 2i and 2i + 1 are a pair, turns[i] its revolutions
+// per position.
+struct LatentPrep {
+  int low_off, low_rank, qr_off, c_off, kr_off;
+  const float *low_gamma, *gamma;
+  const double* turns;
+};
+void latent_prep(bool f32, void* proj, long long ld, const LatentPrep& p, const LatentSpec& s, const RaggedBatch& rb,
+                 const LatentPages& pg, float eps, cudaStream_t stream);
+// Latent rows of the sequences' pages, packed: sequence b, from its token first[b] on, at rows cu_k[b] .. cu_k[b + 1] of out.
+void latent_gather(const LatentSpec& s, const LatentPages& pg, const int* cu_k, const int* first, int n_seq, int max_kv, void* out,
                    cudaStream_t stream);
 // Queries of single tokens: q_lat [rows, heads, rank_p] (unrotated part taken into the latent's space) and the rotated
-// part at qr + t * ld_qr + h * rot_p; token t sees positions 0 .. pos[t] of sequence row_seq[t].
+// part at qr + t * ld_qr + h * rot_p; token t sees positions up to pos[t] of sequence row_seq[t].
 struct LatentQuery {
   const void* q_lat;
   const void* qr;
@@ -171,7 +216,7 @@ struct LatentQuery {
   const int *row_seq, *pos;
   int rows;
 };
-// out [rows, heads, rank_p]: softmax-weighted latents, with exp(sink[h]) in the denominator.
+// out [rows, heads, rank_p]: softmax-weighted latents, with exp(sink[h]) in the denominator (sink may be null).
 void latent_attn_any(bool f32, const LatentQuery& q, const LatentSpec& s, const LatentPages& pg, const float* sink, void* out,
                      float scale, cudaStream_t stream);
 bool latent_decode_ok(const LatentSpec& s, int page_size);
@@ -230,18 +275,16 @@ void conv_state_update(bool f32, const RecurrentSpec& s, const RecurrentInputs& 
 // S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n;  out_c = (sum_n S[c, n] C_n + D_c x_c) silu(z_c) out_scale
 // with x = silu(short convolution of the projection's x columns + bias) and dt = softplus(pre-activation + bias).
 struct SelectiveSpec {
-  int inner, state, rank, taps;     // channels, state values per channel, width of the map to dt, convolution taps
+  int inner, state, rank;           // channels, state values per channel, width of the map to dt
   float out_scale;
 };
 int selective_padded_state(int state);   // state values per channel as stored
 struct SelectiveInputs {
-  const void* proj;                 // [rows, ld]: x | z columns at the offsets below
+  const void* proj;                 // [rows, ld]: z columns at the offset below
   long long ld;
-  int x_off, z_off;
-  const float *conv_w, *conv_b;     // [taps, inner] (last row: the current token's), [inner]
+  int z_off;
   const float* a;                   // [inner, padded state]: A log2(e), zero in the padding
   const float *d, *dt_bias;         // [inner]
-  float* conv_state;                // [slots][taps - 1][inner]
   float* state;                     // [slots][inner][padded state]
   const void* low;                  // [rows, ld_low]: x's maps, dt columns from 0, B and C columns at the offsets below
   long long ld_low;
@@ -249,9 +292,6 @@ struct SelectiveInputs {
   const void* x;                    // [rows, ld_x] the convolved channels
   long long ld_x;
 };
-// x = silu(conv) of a ragged batch, columns [inner, ldx) zeroed; the convolution state advances.
-void selective_conv(bool f32, const SelectiveSpec& s, const SelectiveInputs& in, const RaggedBatch& rb, bool one_token,
-                    void* x, long long ldx, cudaStream_t stream);
 // Prompts and portions; dt [rows, ld_dt]: pre-activations without bias. Long portions are cut into chunks that run side
 // by side: a first kernel forms every chunk's own state and summed step sizes, the second starts each chunk from
 // the states before it. Scratch: selective_scratch floats.

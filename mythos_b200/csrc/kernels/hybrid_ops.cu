@@ -68,9 +68,10 @@ __device__ __forceinline__ void stv(__nv_bfloat16* p, const float (&f)[V]) {
 }
 
 // h = rms(row) * gamma (or the row itself) for a row held in shared memory; columns [dim, ldh) are zeroed (GEMM padding).
+// With a convolution tail, row t being the new token of sequence t, also h + conv(h).
 template <typename T, int V>
 __device__ __forceinline__ void write_normed(const float* row, float ss, const float* gamma, T* h, long long ldh,
-                                             int dim, float eps) {
+                                             int dim, float eps, const ConvTail& cv, long long t) {
   const float r = 1.f / sqrtf(ss / (float)dim + eps);
   for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
     float x[V], g[V];
@@ -83,14 +84,25 @@ __device__ __forceinline__ void write_normed(const float* row, float ss, const f
     stv<V>(h + i, x);
   }
   for (int i = dim + threadIdx.x; i < ldh; i += SN_THREADS) stf(h + i, 0.f);
+  if (cv.c.taps > 0) {
+    __syncthreads();                                   // h is complete; the convolution reads what the activation type keeps of it
+    T* out = static_cast<T*>(cv.out) + t * cv.ld;
+    float* state = cv.c.state ? cv.c.state + (long long)cv.slots[t] * (cv.c.taps - 1) * dim : nullptr;
+    const bool fresh = cv.kv_lens[t] <= 1;
+    for (int i = threadIdx.x; i < dim; i += SN_THREADS) {
+      const float cur = ldf(h + i);
+      stf(out + i, cur + conv_step(cv.c, state, fresh, i, cur));
+    }
+    for (int i = dim + threadIdx.x; i < cv.ld; i += SN_THREADS) stf(out + i, 0.f);
+  }
 }
 
 template <typename T, int V>
 __global__ void __launch_bounds__(SN_THREADS)
 embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ pos, const T* __restrict__ embed,
                       const T* __restrict__ pos_table, int vocab, int max_pos, float scale,
-                      const float* __restrict__ gamma, float* __restrict__ x, T* __restrict__ h, long long ldh, int dim,
-                      float eps) {
+                      const float* __restrict__ gamma0, const float* __restrict__ gamma, float* __restrict__ x,
+                      T* __restrict__ h, long long ldh, int dim, float eps, const __grid_constant__ ConvTail cv) {
   extern __shared__ __align__(16) float row[];
   __shared__ float scratch[32];
   const long long t = blockIdx.x;
@@ -111,10 +123,136 @@ embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ pos, 
       ss += y[j] * y[j];
     }
     stv<V>(row + i, y);
-    stv<V>(x + t * dim + i, y);
+    if (!gamma0) stv<V>(x + t * dim + i, y);
   }
   ss = block_sum(ss, scratch);
-  write_normed<T, V>(row, ss, gamma, h + t * ldh, ldh, dim, eps);
+  if (gamma0) {                                        // the stream starts from the normalised row
+    const float r = 1.f / sqrtf(ss / (float)dim + eps);
+    ss = 0.f;
+    for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
+      float y[V], g[V];
+      ldv<V>(row + i, y);
+      ldv<V>(gamma0 + i, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        y[j] *= r * g[j];
+        ss += y[j] * y[j];
+      }
+      stv<V>(row + i, y);
+      stv<V>(x + t * dim + i, y);
+    }
+    ss = block_sum(ss, scratch);
+  }
+  write_normed<T, V>(row, ss, gamma, h + t * ldh, ldh, dim, eps, cv, t);
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(SN_THREADS)
+residual_norm_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ bias, float mult, float* __restrict__ x,
+                     const float* __restrict__ w_next, T* __restrict__ h, long long ldh, int dim, float eps,
+                     const __grid_constant__ ConvTail cv) {
+  extern __shared__ __align__(16) float row[];
+  __shared__ float scratch[32];
+  const long long t = blockIdx.x;
+  float sx = 0.f;
+  for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
+    float a[V], b[V], xv[V];
+    ldv<V>(y + t * ldy + i, a);
+    ldv<V>(x + t * dim + i, xv);
+    if (bias) {
+      ldv<V>(bias + i, b);
+#pragma unroll
+      for (int j = 0; j < V; ++j) a[j] += b[j];
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      xv[j] = fmaf(mult, a[j], xv[j]);
+      sx += xv[j] * xv[j];
+    }
+    stv<V>(x + t * dim + i, xv);
+    stv<V>(row + i, xv);
+  }
+  sx = block_sum(sx, scratch);
+  write_normed<T, V>(row, sx, w_next, h + t * ldh, ldh, dim, eps, cv, t);
+}
+
+// One block per row. NV > 0: vectors of V values a thread keeps in registers; 0: any width, the row is read twice.
+template <typename T, int V, int NV>
+__global__ void __launch_bounds__(512)
+poly_norm_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ bias, const float* __restrict__ abce,
+                 T* __restrict__ out, long long ldo, int width, int padded, float eps) {
+  __shared__ float part[3][16];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, step = blockDim.x * V;
+  y += blockIdx.x * ldy;
+  out += blockIdx.x * ldo;
+  float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+  auto load = [&](int i, float (&z)[V]) {
+    load_v<V>(y + i, z);
+    if (bias) {
+      float b[V];
+      if constexpr (V == 8) {
+        float lo[4], hi[4];
+        load_v<4>(bias + i, lo);
+        load_v<4>(bias + i + 4, hi);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { b[j] = lo[j]; b[4 + j] = hi[j]; }
+      } else {
+        load_v<V>(bias + i, b);
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) z[j] += b[j];
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float q = z[j] * z[j], q2 = q * q;
+      s1 += q;
+      s2 += q2;
+      s3 = fmaf(q2, q, s3);
+    }
+  };
+  float keep[NV > 0 ? NV : 1][V];
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = threadIdx.x * V + k * step;
+      if (i < width) load(i, keep[k]);
+    }
+  } else {
+    for (int i = threadIdx.x * V; i < width; i += step) load(i, keep[0]);
+  }
+  s1 = warp_sum(s1);
+  s2 = warp_sum(s2);
+  s3 = warp_sum(s3);
+  if (lane == 0) {
+    part[0][warp] = s1;
+    part[1][warp] = s2;
+    part[2][warp] = s3;
+  }
+  __syncthreads();
+  s1 = warp_sum(lane < nw ? part[0][lane] : 0.f);
+  s2 = warp_sum(lane < nw ? part[1][lane] : 0.f);
+  s3 = warp_sum(lane < nw ? part[2][lane] : 0.f);
+  const float n = (float)width, e = abce[3];
+  const float a = abce[0] / sqrtf(s1 / n + eps), b = abce[1] / sqrtf(s2 / n + eps), c = abce[2] / sqrtf(s3 / n + eps);
+  auto store = [&](int i, float (&z)[V]) {
+#pragma unroll
+    for (int j = 0; j < V; ++j) z[j] = fmaf(fmaf(fmaf(c, z[j], b), z[j], a), z[j], e);
+    if constexpr (V == 8) *reinterpret_cast<bf16x8*>(out + i) = pack8(z);
+    else stv<V>(out + i, z);
+  };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = threadIdx.x * V + k * step;
+      if (i < width) store(i, keep[k]);
+    }
+  } else {
+    for (int i = threadIdx.x * V; i < width; i += step) {
+      load(i, keep[0]);
+      store(i, keep[0]);
+    }
+  }
+  for (int i = width + threadIdx.x; i < padded; i += blockDim.x) stf(out + i, 0.f);
 }
 
 enum { SUB_ONE, SUB_TWO, SUB_EXPERTS };
@@ -210,15 +348,15 @@ sandwich_norm_kernel(SublayerOut src, const float* __restrict__ w_post, float mu
     stv<V>(row + i, xv);
   }
   if (w_next) sx = block_sum(sx, scratch);
-  write_normed<T, V>(row, sx, w_next, h + t * ldh, ldh, dim, eps);
+  write_normed<T, V>(row, sx, w_next, h + t * ldh, ldh, dim, eps, ConvTail{}, t);
 }
 
 // Cosine and sine of a position's turn: position x revolutions, reduced to a fraction of a turn in double precision.
-__device__ __forceinline__ float2 turn(int pos, double revolutions) {
+__device__ __forceinline__ float2 turn(int pos, double revolutions, float amp) {
   const double a = pos * revolutions;
   float sn, co;
   sincospif(2.f * (float)(a - rint(a)), &sn, &co);
-  return make_float2(co, sn);
+  return make_float2(amp * co, amp * sn);
 }
 __device__ __forceinline__ float query_factor(const HeadPrep& p, int pos) {
   return p.temp_coef == 0.f ? 1.f : 1.f + p.temp_coef * logf(floorf((float)(pos + 1) / p.temp_every) + 1.f);
@@ -268,8 +406,10 @@ __global__ void attn_prep_kernel(const T* __restrict__ proj, long long ld, HeadP
   for (int i = lane; i < width; i += 32) {
     float x = normed(i);
     if (i < p.rot) {
-      const float2 cs = turn(pos, p.turns[i < half ? i : i - half]);
-      x = i < half ? x * cs.x - normed(i + half) * cs.y : x * cs.x + normed(i - half) * cs.y;
+      const float2 cs = turn(pos, p.turns[p.pairs ? i >> 1 : (i < half ? i : i - half)], p.rot_amp);
+      const bool first = p.pairs ? (i & 1) == 0 : i < half;
+      const int by = p.pairs ? 1 : half;
+      x = first ? x * cs.x - normed(i + by) * cs.y : x * cs.x + normed(i - by) * cs.y;
     }
     stf(dst + i, x * f);
   }
@@ -325,10 +465,10 @@ attn_prep8_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, const __
     s_page_row[i] = page < 0 ? -1 : page * page_size + pos % page_size;
     s_factor[i] = query_factor(p, pos);
   }
-  const bool spread = half % 8 == 0;                       // neighbouring lanes then read neighbouring entries
+  const bool spread = !p.pairs && half % 8 == 0;           // neighbouring lanes then read neighbouring entries
   for (int i = threadIdx.x; i < nt * half; i += AP_THREADS) {
     const int tl = i / half, k = i - tl * half;
-    cs_all[tl * half + (spread ? (k & 7) * (half >> 3) + (k >> 3) : k)] = turn(rb.pos[t0 + tl], p.turns[k]);
+    cs_all[tl * half + (spread ? (k & 7) * (half >> 3) + (k >> 3) : k)] = turn(rb.pos[t0 + tl], p.turns[k], p.rot_amp);
   }
   __syncthreads();
   for (int w0 = first; w0 < total; w0 += AP_THREADS >> 4) {
@@ -369,7 +509,18 @@ attn_prep8_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, const __
 #pragma unroll
         for (int i = 0; i < 8; ++i) f[i] *= q;
       }
-      if (c < p.rot) {
+      if (p.pairs) {
+        const float2* cs = cs_all + it.tl * half + c / 2;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          if (c + 2 * i < p.rot) {
+            const float2 t = cs[i];
+            const float u = f[2 * i], v = f[2 * i + 1];
+            f[2 * i] = u * t.x - v * t.y;
+            f[2 * i + 1] = v * t.x + u * t.y;
+          }
+        }
+      } else if (c < p.rot) {
         // column i < half turns with i + half; the partner's value is read again
         const float2* cs = cs_all + it.tl * half;
         if (spread) {
@@ -544,6 +695,16 @@ __global__ void gelu_mul_kernel(T* __restrict__ y, long long ldy, const T* __res
   }
 }
 
+template <typename T>
+__global__ void sigmoid_mul_kernel(T* __restrict__ y, long long ldy, const T* __restrict__ gate, long long ld_gate, long long rows,
+                                   int width) {
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < rows * width;
+       i += (long long)gridDim.x * blockDim.x) {
+    T* p = y + i / width * ldy + i % width;
+    stf(p, ldf(p) * sigmoid_f(ldf(gate + i / width * ld_gate + i % width)));
+  }
+}
+
 __global__ void soft_cap_kernel(float* __restrict__ y, long long ldy, long long rows, int width, float cap) {
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < rows * width;
        i += (long long)gridDim.x * blockDim.x) {
@@ -560,11 +721,16 @@ inline int grid_for(long long n, int threads, int per_sm) {
 
 template <typename T, int V>
 void embed_launch(const int* ids, const int* pos, const void* embed, const void* pos_table, int vocab, int max_pos,
-                  float scale, const float* gamma, float* x, void* h, long long ldh, int rows, int dim, float eps,
-                  cudaStream_t stream) {
-  embed_pos_norm_kernel<T, V><<<rows, SN_THREADS, dim * 4, stream>>>(ids, pos, (const T*)embed, (const T*)pos_table,
-                                                                     vocab, max_pos, scale, gamma, x, (T*)h, ldh, dim,
-                                                                     eps);
+                  float scale, const float* gamma0, const float* gamma, float* x, void* h, long long ldh, int rows, int dim,
+                  float eps, const ConvTail& conv, cudaStream_t stream) {
+  embed_pos_norm_kernel<T, V><<<rows, SN_THREADS, dim * 4, stream>>>(ids, pos, (const T*)embed, (const T*)pos_table, vocab, max_pos,
+                                                                     scale, gamma0, gamma, x, (T*)h, ldh, dim, eps, conv);
+}
+void check_tail(const ConvTail& conv, int dim) {
+  MB_REQUIRE(conv.c.taps >= 0 && conv.c.taps <= 64, "convolution tail: taps");
+  if (conv.c.taps == 0) return;
+  MB_REQUIRE(conv.c.channels == dim && conv.ld >= dim && conv.out && conv.c.w && conv.slots && conv.kv_lens &&
+                 (conv.c.taps == 1 || conv.c.state) && !conv.c.bias, "convolution tail: arguments");
 }
 template <typename T, int V>
 void sandwich_launch(const SublayerOut& y, const float* w_post, float mult, float* x, const float* w_next, void* h,
@@ -580,13 +746,14 @@ void sandwich_launch(const SublayerOut& y, const float* w_post, float mult, floa
 }  // namespace
 
 void embed_pos_norm(bool f32, const int* ids, const int* pos, const void* embed, const void* pos_table, int vocab,
-                    int max_pos, float scale, const float* gamma, float* x, void* h, long long ldh, int rows, int dim,
-                    float eps, cudaStream_t stream) {
+                    int max_pos, float scale, const float* gamma0, const float* gamma, float* x, void* h, long long ldh,
+                    int rows, int dim, float eps, const ConvTail& conv, cudaStream_t stream) {
+  check_tail(conv, dim);
   MB_REQUIRE(dim > 0 && dim <= 12000 && ldh >= dim, "embed_pos_norm: row width out of range");
   if (rows == 0) return;
   const bool v4 = dim % 4 == 0 && ldh % 4 == 0;
   auto go = [&](auto fn) {
-    fn(ids, pos, embed, pos_table, vocab, max_pos, scale, gamma, x, h, ldh, rows, dim, eps, stream);
+    fn(ids, pos, embed, pos_table, vocab, max_pos, scale, gamma0, gamma, x, h, ldh, rows, dim, eps, conv, stream);
   };
   if (f32) { if (v4) go(embed_launch<float, 4>); else go(embed_launch<float, 1>); }
   else     { if (v4) go(embed_launch<__nv_bfloat16, 4>); else go(embed_launch<__nv_bfloat16, 1>); }
@@ -604,6 +771,53 @@ void sandwich_norm(bool f32, const SublayerOut& y, const float* w_post, float mu
   auto go = [&](auto fn) { fn(y, w_post, mult, x, w_next, h, ldh, rows, dim, eps, stream); };
   if (f32) { if (v4) go(sandwich_launch<float, 4>); else go(sandwich_launch<float, 1>); }
   else     { if (v4) go(sandwich_launch<__nv_bfloat16, 4>); else go(sandwich_launch<__nv_bfloat16, 1>); }
+  count_launch();
+  check_launch();
+}
+
+void residual_norm(bool f32, const void* y, long long ldy, const float* bias, float mult, float* x, const float* w_next, void* h,
+                   long long ldh, int rows, int dim, float eps, const ConvTail& conv, cudaStream_t stream) {
+  MB_REQUIRE(dim > 0 && dim <= 12000 && ldh >= dim && ldy >= dim && w_next, "residual_norm: arguments");
+  check_tail(conv, dim);
+  if (rows == 0) return;
+  const bool v4 = dim % 4 == 0 && ldh % 4 == 0 && ldy % 4 == 0;
+#define MB_RN(T, V) \
+  residual_norm_kernel<T, V><<<rows, SN_THREADS, dim * 4, stream>>>((const T*)y, ldy, bias, mult, x, w_next, (T*)h, ldh, dim, eps, conv)
+  if (f32) { if (v4) MB_RN(float, 4); else MB_RN(float, 1); }
+  else     { if (v4) MB_RN(__nv_bfloat16, 4); else MB_RN(__nv_bfloat16, 1); }
+#undef MB_RN
+  count_launch();
+  check_launch();
+}
+
+void poly_norm(bool f32, const void* y, long long ldy, const float* bias, const float* abce, void* out, long long ldo, int rows,
+               int width, int padded, float eps, cudaStream_t stream) {
+  MB_REQUIRE(width > 0 && ldy >= width && padded >= width && ldo >= padded && abce, "poly_norm: arguments");
+  if (rows == 0) return;
+  const int V = f32 ? 4 : 8;
+  const bool vec = width % V == 0 && ldy % V == 0 && ldo % V == 0 &&
+                   ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(bias)) & 15) == 0;
+  const int units = vec ? width / V : width, threads = units <= 64 ? 64 : (units <= 1024 ? 256 : 512);
+  const int nv = (units + threads - 1) / threads;
+#define MB_PN(T, V, NV) poly_norm_kernel<T, V, NV><<<rows, threads, 0, stream>>>((const T*)y, ldy, bias, abce, (T*)out, ldo, width, padded, eps)
+#define MB_PNV(T, V) \
+  do { if (nv <= 1) MB_PN(T, V, 1); else if (nv <= 2) MB_PN(T, V, 2); else if (nv <= 4) MB_PN(T, V, 4); else MB_PN(T, V, 0); } while (0)
+  if (f32) { if (vec) MB_PNV(float, 4); else MB_PN(float, 1, 0); }
+  else     { if (vec) MB_PNV(__nv_bfloat16, 8); else MB_PN(__nv_bfloat16, 1, 0); }
+#undef MB_PNV
+#undef MB_PN
+  count_launch();
+  check_launch();
+}
+
+void sigmoid_mul(bool f32, void* y, long long ldy, const void* gate, long long ld_gate, int rows, int width, cudaStream_t stream) {
+  MB_REQUIRE(ldy >= width && ld_gate >= width, "sigmoid_mul: strides");
+  if (rows == 0 || width == 0) return;
+  const int grid = grid_for((long long)rows * width, 256, 16);
+  if (f32)
+    sigmoid_mul_kernel<float><<<grid, 256, 0, stream>>>((float*)y, ldy, (const float*)gate, ld_gate, rows, width);
+  else
+    sigmoid_mul_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((__nv_bfloat16*)y, ldy, (const __nv_bfloat16*)gate, ld_gate, rows, width);
   count_launch();
   check_launch();
 }

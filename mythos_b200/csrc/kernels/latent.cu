@@ -1,7 +1,7 @@
 // Attention over a cached latent (hybrid_api.h): every token stores one normalised latent row and one
 // rotated key part, shared by all heads.
 //
-//   latent_prep         latent norm, interleaved rotation, append to the pages
+//   latent_prep         norms of latents and of what queries are a map of, rotation of neighbouring columns, append to the pages
 //   latent_gather       latent rows of whole sequences, packed (keys and values of prompts are expanded from
 //                       them by one GEMM, and the attention kernel of attention_fwd.cu takes over)
 //   latent_attn_any     any widths, fp32 arithmetic, one warp per (token, head)
@@ -49,13 +49,33 @@ struct Vec16 {
   }
 };
 
+// Normalises `width` columns of a row by a warp (zeros up to padded): out = x / rms * gamma.
+template <typename T>
+__device__ __forceinline__ void lp_norm(const T* src, T* dst, int width, int padded, const float* gamma, float eps, int lane) {
+  constexpr int N = Vec16<T>::N;
+  float ss = 0.f;
+  for (int i = lane * N; i < padded; i += 32 * N) {
+    Vec16<T> x;
+    x.load(src + i);
+#pragma unroll
+    for (int j = 0; j < N; ++j) ss = fmaf(x.v[j], x.v[j], ss);
+  }
+  const float r = 1.f / sqrtf(warp_sum(ss) / (float)width + eps);
+  for (int i = lane * N; i < padded; i += 32 * N) {
+    Vec16<T> x;
+    x.load(src + i);
+#pragma unroll
+    for (int j = 0; j < N; ++j) x.v[j] *= i + j < width ? r * gamma[i + j] : 0.f;
+    x.store(dst + i);
+  }
+}
+
 // One warp per token. Angles: position x revolutions, reduced to a fraction of a turn in double precision. Padded
 // columns of the projection are zero, and so are those of a page row.
 constexpr int LP_WARPS = 4;
 template <typename T>
 __global__ void __launch_bounds__(LP_WARPS * 32)
-latent_prep_kernel(T* __restrict__ proj, long long ld, int qr_off, int c_off, int kr_off, const float* __restrict__ gamma,
-                   const double* __restrict__ turns, LatentSpec s, RaggedBatch rb, LatentPages pg, float eps) {
+latent_prep_kernel(T* __restrict__ proj, long long ld, LatentPrep p, LatentSpec s, RaggedBatch rb, LatentPages pg, float eps) {
   constexpr int N = Vec16<T>::N;
   extern __shared__ float2 cs_all[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -63,46 +83,36 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, int qr_off, int c_off, in
   if (t >= rb.rows) return;
   float2* cs = cs_all + warp * (s.rot_p / 2);
   const int pos = rb.pos[t];
-  const int page = pg.table[(long long)rb.row_seq[t] * pg.stride + pos / pg.page_size];
+  T* row = proj + (long long)t * ld;
+  if (p.low_off >= 0) lp_norm(row + p.low_off, row + p.low_off, p.low_rank, (p.low_rank + 7) / 8 * 8, p.low_gamma, eps, lane);
+  if (p.qr_off < 0 && p.c_off < 0) return;
   for (int i = lane; i < s.rot_p / 2; i += 32) {
     float sn = 0.f, co = 1.f;
     if (i < s.rot / 2) {
-      const double a = pos * turns[i];
+      const double a = pos * p.turns[i];
       sincospif(2.f * (float)(a - rint(a)), &sn, &co);
     }
-    cs[i] = make_float2(co, sn);
+    cs[i] = make_float2(s.rot_amp * co, s.rot_amp * sn);
   }
-  T* row = proj + (long long)t * ld;
-  float ss = 0.f;
-  for (int i = lane * N; i < s.rank_p; i += 32 * N) {
-    Vec16<T> x;
-    x.load(row + c_off + i);
-#pragma unroll
-    for (int j = 0; j < N; ++j) ss = fmaf(x.v[j], x.v[j], ss);
-  }
-  ss = warp_sum(ss);
   __syncwarp();                              // cs is complete
-  if (page >= 0) {
-    T* dst = static_cast<T*>(pg.cache) + ((long long)page * pg.page_size + pos % pg.page_size) * s.row();
-    const float r = 1.f / sqrtf(ss / (float)s.rank + eps);
-    for (int i = lane * N; i < s.rank_p; i += 32 * N) {
-      Vec16<T> x;
-      x.load(row + c_off + i);
-#pragma unroll
-      for (int j = 0; j < N; ++j) x.v[j] *= i + j < s.rank ? r * gamma[i + j] : 0.f;
-      x.store(dst + i);
-    }
-    for (int i = lane * N; i < s.rot_p; i += 32 * N) {
-      Vec16<T> x;
-      x.load(row + kr_off + i);
-      x.rotate(cs + i / 2);
-      x.store(dst + s.rank_p + i);
+  if (p.c_off >= 0) {
+    const int page = pg.table[(long long)rb.row_seq[t] * pg.stride + pos / pg.page_size];
+    if (page >= 0) {
+      T* dst = static_cast<T*>(pg.cache) + ((long long)page * pg.page_size + pos % pg.page_size) * s.row();
+      lp_norm(row + p.c_off, dst, s.rank, s.rank_p, p.gamma, eps, lane);
+      for (int i = lane * N; i < s.rot_p; i += 32 * N) {
+        Vec16<T> x;
+        x.load(row + p.kr_off + i);
+        x.rotate(cs + i / 2);
+        x.store(dst + s.rank_p + i);
+      }
     }
   }
+  if (p.qr_off < 0) return;
   const int per = s.rot_p / N;               // vectors per head
   for (int j = lane; j < s.heads * per; j += 32) {
     Vec16<T> x;
-    T* q = row + qr_off + j * N;
+    T* q = row + p.qr_off + j * N;
     x.load(q);
     x.rotate(cs + (j % per) * (N / 2));
     x.store(q);
@@ -111,15 +121,15 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, int qr_off, int c_off, in
 
 // grid (token blocks, sequences); 16-byte units.
 __global__ void __launch_bounds__(256)
-latent_gather_kernel(LatentPages pg, const int* __restrict__ cu_k, uint4* __restrict__ out, int units) {
-  const int b = blockIdx.y, lo = cu_k[b], n = cu_k[b + 1] - lo;
+latent_gather_kernel(LatentPages pg, const int* __restrict__ cu_k, const int* __restrict__ first, uint4* __restrict__ out, int units) {
+  const int b = blockIdx.y, lo = cu_k[b], n = cu_k[b + 1] - lo, skip = first[b];
   const int* table = pg.table + (long long)b * pg.stride;
   const uint4* cache = static_cast<const uint4*>(pg.cache);
   const long long total = (long long)n * units;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
-    const int t = (int)(i / units), c = (int)(i % units);
+    const int r = (int)(i / units), t = skip + r, c = (int)(i % units);
     const int page = max(table[t / pg.page_size], 0);
-    out[((long long)lo + t) * units + c] = cache[((long long)page * pg.page_size + t % pg.page_size) * units + c];
+    out[((long long)lo + r) * units + c] = cache[((long long)page * pg.page_size + t % pg.page_size) * units + c];
   }
 }
 
@@ -141,11 +151,11 @@ latent_attn_any_kernel(LatentQuery q, LatentSpec s, LatentPages pg, const float*
   __syncwarp();
   const int* bt = pg.table + (long long)q.row_seq[t] * pg.stride;
   const T* cache = static_cast<const T*>(pg.cache);
-  const int n = q.pos[t] + 1;
-  float m = sink[h], l = 1.f, acc[ND];         // the sink is a key without value
+  const int n = q.pos[t] + 1, first = s.window > 0 ? max(0, n - s.window) : 0;
+  float m = sink ? sink[h] : -INFINITY, l = sink ? 1.f : 0.f, acc[ND];         // the sink is a key without value
 #pragma unroll
   for (int j = 0; j < ND; ++j) acc[j] = 0.f;
-  for (int j0 = 0; j0 < n; j0 += 32) {
+  for (int j0 = first; j0 < n; j0 += 32) {
     const int key = j0 + lane;
     float sc = -INFINITY;
     long long tok = 0;
@@ -246,8 +256,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_c, LatentQuery q, La
   }
   __syncthreads();
   const int ctx = q.pos[b] + 1;
-  const int n_tiles = (ctx + LD_TOK - 1) / LD_TOK, per = (n_tiles + splits - 1) / splits;
-  const int j0 = split * per, j1 = min(n_tiles, j0 + per);
+  const int lo = s.window > 0 ? max(0, ctx - s.window) : 0;         // first visible token
+  const int first = lo / LD_TOK, n_tiles = (ctx + LD_TOK - 1) / LD_TOK, per = (n_tiles - first + splits - 1) / splits;
+  const int j0 = first + split * per, j1 = min(n_tiles, j0 + per);
   const int* bt = pg.table + (long long)q.row_seq[b] * pg.stride;
   auto issue = [&](int j) {                                         // warp 0: tile j0 + j
     const int st = j % L.stages;
@@ -328,7 +339,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_c, LatentQuery q, La
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        v[i] = tok + i < ctx ? v[i] * scale_log2 : -INFINITY;
+        v[i] = tok + i < ctx && tok + i >= lo ? v[i] * scale_log2 : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
 #pragma unroll
@@ -386,7 +397,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_c, LatentQuery q, La
   const int r0 = lane >> 2;
   if (splits == 1) {                            // nothing to merge: the sink, then the quotient
     if (slane == 0) {
-      const float sk = srow < G ? sink[h0 + srow] * 1.4426950408889634f : -INFINITY, M = fmaxf(m_run, sk);
+      const float sk = sink && srow < G ? sink[h0 + srow] * 1.4426950408889634f : -INFINITY, M = fmaxf(m_run, sk);
       const float w = exp2f(m_run - M);
       s_alpha[srow] = w / (w * l_run + exp2f(sk - M));
     }
@@ -429,7 +440,7 @@ latent_merge_kernel(const float* __restrict__ scratch, const float* __restrict__
   if (threadIdx.x < 32) {
     const int lane = threadIdx.x;
     float2 ml[2];
-    const float sk = sink[blockIdx.x % heads] * 1.4426950408889634f;
+    const float sk = sink ? sink[blockIdx.x % heads] * 1.4426950408889634f : -INFINITY;
     float M = sk;
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
@@ -470,30 +481,29 @@ latent_merge_kernel(const float* __restrict__ scratch, const float* __restrict__
 
 }  // namespace
 
-void latent_prep(bool f32, void* proj, long long ld, int qr_off, int c_off, int kr_off, const float* gamma,
-                 const double* turns, const LatentSpec& s, const RaggedBatch& rb, const LatentPages& pg, float eps,
-                 cudaStream_t stream) {
+void latent_prep(bool f32, void* proj, long long ld, const LatentPrep& p, const LatentSpec& s, const RaggedBatch& rb,
+                 const LatentPages& pg, float eps, cudaStream_t stream) {
   MB_REQUIRE(s.rot > 0 && s.rot % 2 == 0 && s.rot <= 2048, "latent_prep: rotated width");
-  MB_REQUIRE(ld % 8 == 0 && ((qr_off | c_off | kr_off) & 7) == 0, "latent_prep: columns in units of 8");
+  for (int off : {p.low_off, p.qr_off, p.c_off, p.kr_off}) MB_REQUIRE(off < 0 || off % 8 == 0, "latent_prep: columns in units of 8");
+  MB_REQUIRE(ld % 8 == 0 && (p.c_off < 0 || (p.kr_off >= 0 && p.gamma)) && (p.low_off < 0 || (p.low_gamma && p.low_rank > 0)) &&
+                 (reinterpret_cast<uintptr_t>(proj) & 15) == 0, "latent_prep: arguments");
   if (rb.rows == 0) return;
   const int smem = LP_WARPS * (s.rot_p / 2) * (int)sizeof(float2), grid = (rb.rows + LP_WARPS - 1) / LP_WARPS;
   if (f32)
-    latent_prep_kernel<float><<<grid, LP_WARPS * 32, smem, stream>>>((float*)proj, ld, qr_off, c_off, kr_off, gamma, turns, s, rb,
-                                                                     pg, eps);
+    latent_prep_kernel<float><<<grid, LP_WARPS * 32, smem, stream>>>((float*)proj, ld, p, s, rb, pg, eps);
   else
-    latent_prep_kernel<__nv_bfloat16><<<grid, LP_WARPS * 32, smem, stream>>>((__nv_bfloat16*)proj, ld, qr_off, c_off, kr_off, gamma,
-                                                                             turns, s, rb, pg, eps);
+    latent_prep_kernel<__nv_bfloat16><<<grid, LP_WARPS * 32, smem, stream>>>((__nv_bfloat16*)proj, ld, p, s, rb, pg, eps);
   count_launch();
   check_launch();
 }
 
-void latent_gather(const LatentSpec& s, const LatentPages& pg, const int* cu_k, int n_seq, int max_kv, void* out,
+void latent_gather(const LatentSpec& s, const LatentPages& pg, const int* cu_k, const int* first, int n_seq, int max_kv, void* out,
                    cudaStream_t stream) {
   if (n_seq == 0 || max_kv == 0) return;
   const int units = s.row() / 8;
   const long long want = ((long long)max_kv * units + 1023) / 1024;
   const dim3 grid((unsigned)(want < 2048 ? want : 2048), n_seq);
-  latent_gather_kernel<<<grid, 256, 0, stream>>>(pg, cu_k, (uint4*)out, units);
+  latent_gather_kernel<<<grid, 256, 0, stream>>>(pg, cu_k, first, (uint4*)out, units);
   count_launch();
   check_launch();
 }

@@ -1,7 +1,6 @@
 // Selective scan (hybrid_api.h): a diagonal recurrence per channel whose step size, input map and read-out map
 // depend on the token.
 //
-//   selective_conv  short causal convolution + silu of the channels, and its state
 //   selective_scan  prompts and portions: a thread owns NR state values of a channel in registers and walks the
 //                   tokens of a chunk; tiles of inputs pass through shared memory by TMA, B and C of a token are read
 //                   by all channels.
@@ -10,6 +9,8 @@
 //                   a chunk, walks it again and reads out.
 //   selective_step  one token per sequence: the same update on the stored state, for few sequences with the map to
 //                   the step sizes inside.
+//
+// The short convolution in front of it is short_conv.cu.
 //
 // Step sizes, decays, states and the read-out are fp32 in both activation types. A is stored times log2(e), so a
 // decay is one exp2.
@@ -44,11 +45,6 @@ StateMap state_map(int state) {
 }
 
 // ln(1 + e) for 0 <= e <= 1 as 2 artanh(e / (2 + e)), series in t^2 <= 1/9.
-__device__ __forceinline__ float fast_rcp(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 __device__ __forceinline__ float log1p_unit(float e) {
   const float t = e * fast_rcp(2.f + e), t2 = t * t;
   float p = fmaf(t2, 1.f / 15.f, 1.f / 13.f);
@@ -82,225 +78,11 @@ __device__ __forceinline__ float decay_t(float x) {
   if constexpr (sizeof(T) == 2) return fast_exp2(x);
   else return exp2_series(x);
 }
-// z / (1 + e^-z)
-__device__ __forceinline__ float silu_fast(float z) { return z * fast_rcp(1.f + fast_exp2(-1.4426950408889634f * z)); }
-
-template <int V>
-__device__ __forceinline__ void load_v(const float* p, float (&f)[V]) {
-  if constexpr (V % 4 == 0) {
-#pragma unroll
-    for (int i = 0; i < V / 4; ++i) {
-      const float4 t = reinterpret_cast<const float4*>(p)[i];
-      f[4 * i] = t.x; f[4 * i + 1] = t.y; f[4 * i + 2] = t.z; f[4 * i + 3] = t.w;
-    }
-  } else {
-#pragma unroll
-    for (int i = 0; i < V; ++i) f[i] = p[i];
-  }
-}
-template <int V>
-__device__ __forceinline__ void load_v(const __nv_bfloat16* p, float (&f)[V]) {
-  if constexpr (V == 8) {
-    unpack8(*reinterpret_cast<const bf16x8*>(p), f);
-  } else if constexpr (V == 4) {
-    const uint2 t = *reinterpret_cast<const uint2*>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.y));
-    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
-  } else {
-#pragma unroll
-    for (int i = 0; i < V; ++i) f[i] = __bfloat162float(p[i]);
-  }
-}
-template <int V>
-__device__ __forceinline__ void store_v(float* p, const float (&f)[V]) {
-  if constexpr (V % 4 == 0) {
-#pragma unroll
-    for (int i = 0; i < V / 4; ++i) reinterpret_cast<float4*>(p)[i] = make_float4(f[4 * i], f[4 * i + 1], f[4 * i + 2], f[4 * i + 3]);
-  } else {
-#pragma unroll
-    for (int i = 0; i < V; ++i) p[i] = f[i];
-  }
-}
-template <int V>
-__device__ __forceinline__ void store_v(__nv_bfloat16* p, const float (&f)[V]) {
-  if constexpr (V == 4) {
-    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
-  } else {
-#pragma unroll
-    for (int i = 0; i < V; ++i) p[i] = __float2bfloat16(f[i]);
-  }
-}
-
-// ---------------------------------------------------------------------------------------------
-// V channels of SC_ROWS neighbouring rows per thread; the rows' inputs pass through registers (TAPS > 0), so each is read
-// once. TAPS: number of taps, 0: any number, read from the cache.
-constexpr int SC_ROWS = 16, SC_STEP = 4;
-template <typename T>
-__device__ __forceinline__ float silu_t(float z) {
-  if constexpr (sizeof(T) == 2) return silu_fast(z);
-  else return silu_f(z);
-}
 template <typename T>
 __device__ __forceinline__ float softplus_t(float z) {
   if constexpr (sizeof(T) == 2) return softplus_fast(z);
   else return softplus_f(z);
 }
-template <typename T, int V, int TAPS>
-__global__ void __launch_bounds__(256)
-selective_conv_kernel(SelectiveSpec s, SelectiveInputs in, RaggedBatch rb, T* __restrict__ x, long long ldx) {
-  __shared__ int s_index[SC_ROWS];                 // row within its sequence's portion
-  __shared__ long long s_state[SC_ROWS];           // its sequence's convolution state, -1: it has no earlier tokens
-  const long long c = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
-  const int r0 = blockIdx.y * SC_ROWS, n = min(SC_ROWS, rb.rows - r0), taps = TAPS > 0 ? TAPS : s.taps;
-  if (threadIdx.x < n) {
-    const int b = rb.row_seq[r0 + threadIdx.x], lo = rb.cu_q[b];
-    s_index[threadIdx.x] = r0 + threadIdx.x - lo;
-    s_state[threadIdx.x] = rb.kv_lens[b] > rb.cu_q[b + 1] - lo ? (long long)rb.slots[b] * (taps - 1) * s.inner : -1;
-  }
-  __syncthreads();
-  if (c >= ldx) return;
-  if (c >= s.inner) {                              // padding (V = 1)
-    for (int r = 0; r < n; ++r) stf(x + (r0 + r) * ldx + c, 0.f);
-    return;
-  }
-  const T* col = static_cast<const T*>(in.proj) + (long long)r0 * in.ld + in.x_off + c;
-  T* dst = x + (long long)r0 * ldx + c;
-  const float* w = in.conv_w + c;
-  float bias[V];
-  load_v<V>(in.conv_b + c, bias);
-  // inputs j tokens before row r that lie before its portion: from the state, zeros before the start
-  auto early = [&](int r, int j, float (&v)[V]) {
-    const long long st = s_state[r];
-    if (st >= 0) {
-      load_v<V>(in.conv_state + st + (long long)(taps - 1 + s_index[r] - j) * s.inner + c, v);
-    } else {
-#pragma unroll
-      for (int i = 0; i < V; ++i) v[i] = 0.f;
-    }
-  };
-  if constexpr (TAPS > 0) {
-    float wr[TAPS][V], h[TAPS - 1 + SC_STEP][V];   // h: inputs from row r - (TAPS - 1) on
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) load_v<V>(w + (long long)j * s.inner, wr[j]);
-#pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) {
-      if (r0 - (TAPS - 1) + j >= 0) {
-        load_v<V>(col + (long long)(j - (TAPS - 1)) * in.ld, h[j]);
-      } else {
-#pragma unroll
-        for (int i = 0; i < V; ++i) h[j][i] = 0.f;
-      }
-    }
-#pragma unroll 1
-    for (int r = 0; r < n; r += SC_STEP) {
-#pragma unroll
-      for (int u = 0; u < SC_STEP; ++u)
-        if (r + u < n) load_v<V>(col + (long long)(r + u) * in.ld, h[TAPS - 1 + u]);
-#pragma unroll
-      for (int u = 0; u < SC_STEP; ++u) {
-        if (r + u >= n) break;
-        const int i0 = s_index[r + u];
-        float acc[V];
-#pragma unroll
-        for (int i = 0; i < V; ++i) acc[i] = fmaf(wr[TAPS - 1][i], h[TAPS - 1 + u][i], bias[i]);
-#pragma unroll
-        for (int j = 1; j < TAPS; ++j) {
-          if (j <= i0) {                           // the same for the whole block
-#pragma unroll
-            for (int i = 0; i < V; ++i) acc[i] = fmaf(wr[TAPS - 1 - j][i], h[TAPS - 1 + u - j][i], acc[i]);
-          } else {
-            float v[V];
-            early(r + u, j, v);
-#pragma unroll
-            for (int i = 0; i < V; ++i) acc[i] = fmaf(wr[TAPS - 1 - j][i], v[i], acc[i]);
-          }
-        }
-#pragma unroll
-        for (int i = 0; i < V; ++i) acc[i] = silu_t<T>(acc[i]);
-        store_v<V>(dst + (long long)(r + u) * ldx, acc);
-      }
-#pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j)
-#pragma unroll
-        for (int i = 0; i < V; ++i) h[j][i] = h[j + SC_STEP][i];
-    }
-  } else {
-    for (int r = 0; r < n; ++r) {
-      float acc[V];
-#pragma unroll
-      for (int i = 0; i < V; ++i) acc[i] = bias[i];
-      for (int j = 0; j < taps; ++j) {
-        float v[V], wj[V];
-        if (j <= s_index[r]) load_v<V>(col + (long long)(r - j) * in.ld, v);
-        else early(r, j, v);
-        load_v<V>(w + (long long)(taps - 1 - j) * s.inner, wj);
-#pragma unroll
-        for (int i = 0; i < V; ++i) acc[i] = fmaf(wj[i], v[i], acc[i]);
-      }
-#pragma unroll
-      for (int i = 0; i < V; ++i) acc[i] = silu_t<T>(acc[i]);
-      store_v<V>(dst + (long long)r * ldx, acc);
-    }
-  }
-}
-
-// One thread per (sequence, channel): the last taps - 1 inputs of the sequence become the state.
-template <typename T>
-__global__ void selective_conv_state_kernel(SelectiveSpec s, SelectiveInputs in, RaggedBatch rb) {
-  const int c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y;
-  if (c >= s.inner) return;
-  const int r0 = rb.cu_q[b], len = rb.cu_q[b + 1] - r0, n = s.taps - 1;
-  if (len <= 0) return;
-  const bool fresh = rb.kv_lens[b] == len;
-  float* st = in.conv_state + (long long)rb.slots[b] * n * s.inner + c;
-  const T* col = static_cast<const T*>(in.proj) + in.x_off + c;
-  // entry j holds the input of token len - n + j; an entry moves down, never up, so in-place order is safe
-  for (int j = 0; j < n; ++j) {
-    const int i = len - n + j;
-    float v;
-    if (i >= 0) v = ldf(col + (long long)(r0 + i) * in.ld);
-    else v = fresh ? 0.f : st[(long long)(n + i) * s.inner];
-    st[(long long)j * s.inner] = v;
-  }
-}
-
-// One token per sequence: convolution and its state in one pass, one channel per thread.
-template <typename T>
-__global__ void __launch_bounds__(256)
-selective_conv_step_kernel(SelectiveSpec s, SelectiveInputs in, RaggedBatch rb, T* __restrict__ x, long long ldx) {
-  const int c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y;
-  if (c >= ldx) return;
-  if (c >= s.inner) {
-    stf(x + b * ldx + c, 0.f);
-    return;
-  }
-  const bool fresh = rb.kv_lens[b] <= 1;
-  const float cur = ldf(static_cast<const T*>(in.proj) + b * in.ld + in.x_off + c);
-  float acc = fmaf(in.conv_w[(long long)(s.taps - 1) * s.inner + c], cur, in.conv_b[c]);
-  float* st = in.conv_state + (long long)rb.slots[b] * (s.taps - 1) * s.inner + c;
-  const float* w = in.conv_w + c;
-  if (s.taps == 4) {                               // all loads before the stores
-    float old[3];
-#pragma unroll
-    for (int j = 0; j < 3; ++j) old[j] = fresh ? 0.f : st[(long long)j * s.inner];
-#pragma unroll
-    for (int j = 0; j < 3; ++j) acc = fmaf(w[(long long)j * s.inner], old[j], acc);
-    st[0] = old[1];
-    st[s.inner] = old[2];
-    st[2ll * s.inner] = cur;
-  } else {
-    float nxt = cur;                               // newest first: entry j moves to j - 1
-    for (int j = s.taps - 2; j >= 0; --j) {
-      const float old = fresh ? 0.f : st[(long long)j * s.inner];
-      acc = fmaf(w[(long long)j * s.inner], old, acc);
-      st[(long long)j * s.inner] = nxt;
-      nxt = old;
-    }
-  }
-  stf(x + b * ldx + c, silu_f(acc));
-}
-
 // ---------------------------------------------------------------------------------------------
 // Scratch of a chunked scan: the state every sequence starts from, and per chunk its own state (from zero) and the sum
 // of its step sizes.
@@ -598,7 +380,7 @@ selective_step_kernel(SelectiveSpec s, SelectiveInputs in, RaggedBatch rb, int l
 }
 
 void check_spec(const SelectiveSpec& s) {
-  MB_REQUIRE(s.inner > 0 && s.rank > 0 && s.taps > 0 && s.taps <= 64, "selective scan: sizes");
+  MB_REQUIRE(s.inner > 0 && s.rank > 0, "selective scan: sizes");
   MB_REQUIRE(s.state > 0 && s.state <= 512, "selective scan: at most 512 state values per channel");
 }
 
@@ -625,44 +407,6 @@ ChunkPlan plan_chunks(const SelectiveSpec& s, int rows, int max_q) {
 int selective_padded_state(int state) {
   const StateMap m = state_map(state);
   return m.nr * m.lanes;
-}
-
-void selective_conv(bool f32, const SelectiveSpec& s, const SelectiveInputs& in, const RaggedBatch& rb, bool one_token,
-                    void* x, long long ldx, cudaStream_t stream) {
-  check_spec(s);
-  MB_REQUIRE(ldx >= s.inner, "selective_conv: output width");
-  if (rb.rows == 0) return;
-  if (one_token) {
-    MB_REQUIRE(rb.rows == rb.n_seq, "selective_conv: one token per sequence");
-    const dim3 grid((int)((ldx + 255) / 256), rb.n_seq);
-    if (f32) selective_conv_step_kernel<float><<<grid, 256, 0, stream>>>(s, in, rb, (float*)x, ldx);
-    else selective_conv_step_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(s, in, rb, (__nv_bfloat16*)x, ldx);
-    count_launch();
-    check_launch();
-    return;
-  }
-  const int V = 4;
-  const bool vec = s.inner % V == 0 && ldx == s.inner && in.ld % V == 0 && in.x_off % V == 0 &&
-                   ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(in.proj)) & 15) == 0;
-  const int units = (int)(vec ? ldx / V : ldx), threads = units >= 128 ? 128 : (units + 31) / 32 * 32;
-  const dim3 grid((units + threads - 1) / threads, (rb.rows + SC_ROWS - 1) / SC_ROWS);
-  MB_REQUIRE(grid.y <= 65535, "selective_conv: too many rows in one batch");
-#define MB_SC(T, V, TAPS) selective_conv_kernel<T, V, TAPS><<<grid, threads, 0, stream>>>(s, in, rb, (T*)x, ldx)
-  if (f32) {
-    if (vec && s.taps == 4) MB_SC(float, 4, 4); else if (vec) MB_SC(float, 4, 0); else MB_SC(float, 1, 0);
-  } else {
-    if (vec && s.taps == 4) MB_SC(__nv_bfloat16, 4, 4); else if (vec) MB_SC(__nv_bfloat16, 4, 0); else MB_SC(__nv_bfloat16, 1, 0);
-  }
-#undef MB_SC
-  count_launch();
-  check_launch();
-  if (s.taps > 1) {
-    const dim3 sgrid((s.inner + 255) / 256, rb.n_seq);
-    if (f32) selective_conv_state_kernel<float><<<sgrid, 256, 0, stream>>>(s, in, rb);
-    else selective_conv_state_kernel<__nv_bfloat16><<<sgrid, 256, 0, stream>>>(s, in, rb);
-    count_launch();
-    check_launch();
-  }
 }
 
 long long selective_scratch(const SelectiveSpec& s, int n_seq, int rows, int max_q) {

@@ -20,9 +20,14 @@ and input / read-out maps -> GEMM to the channels' step sizes -> scan with its o
 Latent attention caches one row per token (latent | rotated key part) that all heads share. Tokens of
 sequences that bring few of them at once (decoding, short portions) attend in the latent's space: queries go
 through W_uk, the result through W_uv. Longer portions expand the latents of their sequence to keys and
-values once per pass and run the tensor-core prompt attention. A batch with both runs both. Routed experts:
+values once per pass (with a window those of its reach) and run the tensor-core prompt attention. A batch with both
+runs both. The order of rotated columns is free, so halves are stored as neighbouring pairs. Routed experts:
 router GEMM -> selection and row segments -> row gather -> two grouped GEMMs -> (weighted sum + shared expert +
 norm + residual).
+
+Parallel designs: mixer and feed-forward write side by side into one row and share one output GEMM; one kernel adds it
+to the stream and normalises, and for single tokens also runs the convolution in front of the next mixer (its last
+inputs are a state of every layer). Longer portions run that convolution as a kernel of its own.
 
 ``dtype``: "bfloat16" (matrix products and activations in bf16 with 32-bit accumulation; residual,
 norms, decays, states and scores in 32-bit) or "float32" (everything in 32-bit).
@@ -81,20 +86,23 @@ class _Sublayer:
 class _Ctx:
     """One pass: token ids, the ragged batch (cu_q, kv_lens, slots, row_seq, pos), its block-table rows and sizes.
     ``decode``: one token of every sequence. ``split`` (passes with a long portion and latent layers):
-    ``_LatentSplit``, else every token attends in the latent's space."""
+    ``_LatentSplit``, else every token attends in the latent's space. ``conv``: what mixers read behind an input
+    convolution."""
 
     def __init__(self, ids, batch, table, rows, n_seq, max_q, max_kv, split=None):
         self.ids, self.batch, self.table, self.rows, self.n_seq = ids, batch, table, rows, n_seq
         self.max_q, self.max_kv, self.split = max_q, max_kv, split
         self.decode = max_q == 1
+        self.conv = None
 
 
 class _LatentSplit:
     """Which tokens attend how: ``cu_k`` first expanded row of every sequence with a long portion (``keys`` in all,
-    at most ``max_k`` of one), ``short`` the rows of the other sequences (None: there are none)."""
+    ``key_lens`` of each, at most ``max_k``), which holds its token ``first``; ``short`` the rows of the other sequences
+    (None: there are none)."""
 
-    def __init__(self, cu_k, keys, max_k, short, short_seq, short_pos):
-        self.cu_k, self.keys, self.max_k = cu_k, keys, max_k
+    def __init__(self, cu_k, first, key_lens, keys, max_k, short, short_seq, short_pos):
+        self.cu_k, self.first, self.key_lens, self.keys, self.max_k = cu_k, first, key_lens, keys, max_k
         self.short, self.short_seq, self.short_pos = short, short_seq, short_pos
 
 
@@ -132,13 +140,13 @@ class HybridEngine(InferenceEngine):
         pages_per_seq = (self.max_seq_len + page_size - 1) // page_size
         att = [s.attention for s in cfg.layers if s.attention is not None]
         recurrent = any(s.recurrent is not None for s in cfg.layers)
-        self.states = RecurrentStatePool(max_batch, self.device) if recurrent else None
+        self.states = RecurrentStatePool(max_batch, self.device) if recurrent or cfg.input_conv > 1 else None
         shapes = []                # per caching layer; a latent layer's rows are keys and values at once
         for s in cfg.layers:
             if s.attention is not None:
                 if s.attention.kv_from is None:
                     shapes.append((s.attention.kv_heads, _pad8(s.attention.dim), _pad8(s.attention.vdim)))
-            elif s.latent is not None:
+            elif s.latent is not None and s.latent.kv_from is None:
                 shapes.append((1, _pad8(s.latent.kv_rank) + _pad8(s.latent.rot_dim), 0))
         self.cache = PagedKVCache(len(shapes), 0, 0, kv_pages or max_batch * pages_per_seq, page_size, max_batch,
                                   pages_per_seq, self.device, dtype=self.dtype, layer_shapes=shapes, states=self.states)
@@ -180,7 +188,7 @@ class HybridEngine(InferenceEngine):
         return w.to(device=self.device, dtype=torch.float32).contiguous()
 
     def _norm(self, w: torch.Tensor) -> torch.Tensor:
-        return self._vector(w) + self.cfg.norm_offset
+        return self._vector(w.expand(self.cfg.hidden_size) if w.dim() == 0 else w) + self.cfg.norm_offset
 
     def _pack(self, model) -> None:
         t = model.tensor
@@ -189,21 +197,23 @@ class HybridEngine(InferenceEngine):
         self.pos_table = t("pos").to(self.device, self.dtype).contiguous() if cfg.position_table else None
         self.side_table = t("side.embed").to(self.device, self.dtype).contiguous() if cfg.token_side else None
         self.final_norm = self._norm(t("final.norm"))
+        self.embed_norm = self._norm(t("embed.norm")) if cfg.embed_norm else None
         if not cfg.tied_head:
             self.head = self._matrix(t("head"))
         else:
             self.head = self.embed_table if cfg.hidden_size % 8 == 0 else self._matrix(self.embed_table)
         pages_of = {}                                 # layer -> its entry of the cache
         for i, spec in enumerate(cfg.layers):
-            share = spec.attention.kv_from if spec.attention is not None else None
+            keeps = spec.attention or spec.latent
+            share = keeps.kv_from if keeps is not None else None
             if share is not None:
                 pages_of[i] = pages_of[share]
-            elif spec.attention is not None or spec.latent is not None:
+            elif keeps is not None:
                 pages_of[i] = len(set(pages_of.values()))
 
         def norms(p: str, n: int) -> _Sublayer:
             if cfg.pre_norm:
-                return _Sublayer(self._norm(t(p + f"norm{n}")), self._norm(t(p + f"norm{n}b")))
+                return _Sublayer(self._norm(t(p + f"norm{n}")), self._norm(t(p + f"norm{n}b")) if cfg.post_norm else None)
             return _Sublayer(None, self._norm(t(p + f"norm{n}")))
 
         for i, spec in enumerate(cfg.layers):
@@ -227,7 +237,11 @@ class HybridEngine(InferenceEngine):
             else:
                 L.run = self._gla
                 self._pack_gla(L, t, p + "mix.")
-            if spec.mlp is not None:
+            if cfg.input_conv:
+                L.conv = self._input_conv(t(p + "canon1"))
+            if cfg.parallel:
+                self._pack_side_by_side(L, t, p + "mlp.")
+            elif spec.mlp is not None:
                 L.ff_norms = norms(p, 2)
                 if isinstance(spec.mlp, MoeFF):
                     self._pack_experts(L, t, p + "mlp.")
@@ -263,9 +277,33 @@ class HybridEngine(InferenceEngine):
                                 {"z_bias": self._vector(t(p + "a2.b")), "gamma": self._vector(t(p + "norm")), "a2": L.a2})
         L.out = self._matrix(t(p + "o"))
 
+    def _input_conv(self, w: torch.Tensor):
+        channels, taps = w.shape
+        return self.H.Conv(channels, True, self._vector(w.t()), state=self.states.add(taps - 1, channels) if taps > 1 else None)
+
+    def _pack_side_by_side(self, L, t, p: str) -> None:
+        """Feed-forward beside a mixer: its down matrix continues the rows of the mixer's output matrix."""
+        mixer = L.run
+        L.run, L.heads_of = self._side_by_side, {self._attention_layer: self._attention_heads, self._latent: self._latent_heads}[mixer]
+        L.mixer_cols = L.out.shape[1]
+        f = L.spec.mlp
+        if f is None:
+            return
+        down = self._matrix(t(p + "down"))
+        L.out = torch.cat([L.out, down], 1)
+        L.down_bias = None
+        if f.gated:
+            L.gate_up = FusedProjection([("gate", t(p + "gate")), ("up", t(p + "up"))], self.dtype, self.device)
+            L.act = (ACT_KINDS[f.act], 0.0, 0.0)
+        else:
+            L.up, L.up_bias = self._matrix(t(p + "up")), self._vector(t(p + "up.b"))
+            L.poly, L.down_bias = self._vector(t(p + "act")), self._vector(t(p + "down.b"))
+
     # ---- attention: projection parts under a prefix, then the kernel-side object over their offsets
     def _attention_parts(self, m: AttentionMixer, t, p: str, prefix: str = "") -> list:
-        parts = [("q", m.heads)] + ([("k", m.kv_heads), ("v", m.kv_heads)] if m.kv_from is None else [])
+        parts = [("q", m.heads)]
+        if m.kv_from is None:
+            parts += [("k", m.kv_heads)] + ([("v", m.kv_heads)] if m.values == "own" else [])
         parts = [(prefix + n, _pad_heads(t(p + n), heads)) for n, heads in parts]
         if m.gate is not None:
             parts.append((prefix + "g", _pad_heads(t(p + "g"), m.heads) if m.gate == "channel" else t(p + "g")))
@@ -277,22 +315,27 @@ class HybridEngine(InferenceEngine):
                 "scale": m.scale, "out_scale": out_scale, "window": m.window, "gate_channels": int(m.gate == "channel"),
                 "norm_dim": m.dim if m.qk_norm else 0, "eps": self.cfg.norm_eps}
         if own:
-            spec.update(k_off=off[prefix + "k"], v_off=off[prefix + "v"])
+            spec.update(k_off=off[prefix + "k"], v_off=off[prefix + ("v" if m.values == "own" else "k")])
         tensors = {}
         if m.bias:
             for n, heads in [("q", m.heads)] + ([("k", m.kv_heads), ("v", m.kv_heads)] if own else []):
-                tensors[n + "_bias"] = self._vector(_pad_heads(t(p + n + ".b"), heads))
+                source = "k" if n == "v" and m.values == "keys" else n
+                tensors[n + "_bias"] = self._vector(_pad_heads(t(p + source + ".b"), heads))
         if m.qk_norm == "weighted":
             for n in ("q", "k") if own else ("q",):
                 tensors[n + "_gamma"] = self._vector(_pad_heads(t(p + n + ".norm"), 1))
-        if m.sink:
-            tensors["sink"] = self._vector(t(p + "sink"))
+        tensors.update(self._sink(m, t, p))
         if m.rotation is not None:
-            spec["rot"] = m.rotation.dims
+            spec.update(rot=m.rotation.dims, pairs=int(m.rotation.layout == "pairs"), rot_amp=m.rotation.amplitude)
             tensors["turns"] = torch.tensor(m.rotation.turns(), dtype=torch.float64, device=self.device)
         if m.q_temp is not None:
             spec.update(temp_coef=m.q_temp.coef, temp_every=m.q_temp.every)
         return self.H.Attention(spec, tensors)
+
+    def _sink(self, m, t, p: str) -> dict:
+        if m.sink is None:
+            return {}
+        return {"sink": self._vector(t(p + "sink")) if m.sink == "learned" else torch.zeros(m.heads, device=self.device)}
 
     @staticmethod
     def _attention_out(m: AttentionMixer, w: torch.Tensor) -> torch.Tensor:
@@ -320,13 +363,11 @@ class HybridEngine(InferenceEngine):
         padded = self.H.selective_padded_state(n)
         decay = torch.zeros(r.inner, padded, dtype=torch.float64)
         decay[:, :n] = -torch.exp(t(right + "A_log").double().cpu()) / math.log(2.0)
-        tensors = {"conv_w": self._vector(t(right + "conv").t()), "conv_b": self._vector(t(right + "conv.b")),
-                   "a": self._vector(decay), "d": self._vector(t(right + "D")), "dt_b": self._vector(t(right + "dt.b")),
+        tensors = {"a": self._vector(decay), "d": self._vector(t(right + "D")), "dt_b": self._vector(t(right + "dt.b")),
                    "w_dt": L.w_dt, "state": self.states.add(r.inner, padded)}
-        if r.conv > 1:
-            tensors["conv_state"] = self.states.add(r.conv - 1, r.inner)
-        L.sel = self.H.Selective({"inner": r.inner, "state": n, "rank": k, "taps": r.conv, "out_scale": scale_r,
-                                  "x_off": L.proj.off["rx"], "z_off": L.proj.off["rz"], "b_off": L.x_maps.off["B"],
+        L.conv = self.H.Conv(r.inner, False, self._vector(t(right + "conv").t()), self._vector(t(right + "conv.b")),
+                             self.states.add(r.conv - 1, r.inner) if r.conv > 1 else None)
+        L.sel = self.H.Selective({"inner": r.inner, "state": n, "rank": k, "out_scale": scale_r, "z_off": L.proj.off["rz"], "b_off": L.x_maps.off["B"],
                                   "c_off": L.x_maps.off["C"]}, tensors)
         L.out = self._matrix(torch.cat([self._attention_out(a, t(left + "o")), t(right + "o")], 1))
 
@@ -348,8 +389,8 @@ class HybridEngine(InferenceEngine):
         L.rec = self._recurrent(r, {"q": off["rq"], "k": off["rk"], "v": off["rv"], "b": off["rb"]}, tensors)
 
     def _pack_latent(self, L, t, p: str) -> None:
-        """Projection columns: unrotated queries per head | rotated queries per head | latent | rotated key part, each
-        part of a head padded to a multiple of 8."""
+        """Projection columns: unrotated queries per head | rotated queries per head (or, of low-rank queries, what a
+        second matrix makes both from) | latent | rotated key part | gate, each part of a head padded to a multiple of 8."""
         m = L.spec.mixer
         H, dn, dr, dv, r = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank
         dn_p, dr_p, dv_p, r_p = _pad8(dn), _pad8(dr), _pad8(dv), _pad8(r)
@@ -359,21 +400,35 @@ class HybridEngine(InferenceEngine):
             out[:, :width] = w.view(H, width, -1)
             return out.view(H * padded, -1)
 
-        q = t(p + "q").view(H, dn + dr, -1)
-        dkv = t(p + "dkv")
-        L.proj = FusedProjection([("q", heads(q[:, :dn].reshape(H * dn, -1), dn, dn_p)),
-                                  ("qr", heads(q[:, dn:].reshape(H * dr, -1), dr, dr_p)),
-                                  ("c", dkv[:r]), ("kr", dkv[r:])], self.dtype, self.device)
+        order = torch.arange(dr)                       # rotated columns as neighbouring pairs
+        if m.rotation.layout == "halves":
+            order = torch.stack([order[: dr // 2], order[dr // 2:]], 1).flatten()
+        q = t(p + ("uq" if m.q_rank else "q")).view(H, dn + dr, -1)
+        queries = [("q", heads(q[:, :dn].reshape(H * dn, -1), dn, dn_p)),
+                   ("qr", heads(q[:, dn:][:, order.to(q.device)].reshape(H * dr, -1), dr, dr_p))]
+        parts = [("low", t(p + "dq"))] if m.q_rank else queries
+        if m.kv_from is None:
+            dkv = t(p + "dkv")
+            parts = parts + [("c", dkv[:r]), ("kr", dkv[r:][order.to(dkv.device)])]
+        if m.gate:
+            parts = parts + [("g", heads(t(p + "g"), dv, dv_p))]
+        L.proj = FusedProjection(parts, self.dtype, self.device)
+        L.low = FusedProjection(queries, self.dtype, self.device) if m.q_rank else None
         uk, uv = t(p + "uk").view(H, dn, r), t(p + "uv").view(H, dv, r)
         L.uk_t = torch.zeros(H, r_p, dn_p, dtype=self.dtype, device=self.device)       # queries into the latent's space
         L.uk_t[:, :r, :dn] = uk.transpose(1, 2).to(self.device, self.dtype)
         L.uv = torch.zeros(H, dv_p, r_p, dtype=self.dtype, device=self.device)         # latents to a head's values
         L.uv[:, :dv, :r] = uv.to(self.device, self.dtype)
-        off = L.proj.off
-        turns = torch.tensor([m.rot_base ** (-2.0 * i / dr) / (2.0 * math.pi) for i in range(dr // 2)], dtype=torch.float64)
-        L.lat = self.H.Latent({"heads": H, "rank": r, "rot": dr, "rank_p": r_p, "rot_p": dr_p, "qr_off": off["qr"],
-                               "c_off": off["c"], "kr_off": off["kr"], "scale": m.scale, "eps": self.cfg.norm_eps},
-                              self._vector(t(p + "dkv.norm")), turns.to(self.device), self._vector(t(p + "sink")))
+        off, own = L.proj.off, m.kv_from is None
+        spec = {"heads": H, "rank": r, "rot": dr, "rank_p": r_p, "rot_p": dr_p, "qr_off": (L.low or L.proj).off["qr"],
+                "scale": m.scale, "eps": self.cfg.norm_eps, "window": m.window, "rot_amp": m.rotation.amplitude}
+        if own:
+            spec.update(c_off=off["c"], kr_off=off["kr"])
+        if m.q_rank:
+            spec.update(low_off=off["low"], low_rank=m.q_rank)
+        turns = torch.tensor(m.rotation.turns(), dtype=torch.float64, device=self.device)
+        L.lat = self.H.Latent(spec, self._vector(t(p + "dkv.norm")) if own else None, turns, self._sink(m, t, p).get("sink"),
+                              self._vector(t(p + "dq.norm")) if m.q_rank else None)
         L.expand = None
         if self.tensor_kernels and not self.f32 and L.lat.prefill_ok(dn_p, dv_p):      # keys and values of all heads
             L.expand = torch.zeros(H * (dn_p + dv_p), r_p, dtype=self.dtype, device=self.device)
@@ -409,7 +464,7 @@ class HybridEngine(InferenceEngine):
         n = sum(x.numel() * x.element_size() for x in tables if x is not None)
         for L in self.layers:
             mats = [L.proj.weight, L.a2, L.g2, L.out, L.left_out, L.right_out, L.down, L.uk_t, L.uv, L.router, L.w_in, L.w_out,
-                    L.side_gate, L.side_proj, L.w_dt] + [f.weight for f in (L.gate_up, L.x_maps) if f is not None]
+                    L.side_gate, L.side_proj, L.w_dt, L.up] + [f.weight for f in (L.gate_up, L.x_maps, L.low) if f is not None]
             n += sum(x.numel() * x.element_size() for x in mats if x is not None)
         return n
 
@@ -489,15 +544,18 @@ class HybridEngine(InferenceEngine):
             att.prefill(q, kc, vc, ctx.batch, ctx.table, gate, o, ctx.max_q, self._status)
         return o
 
+    def _attention_heads(self, L, h, ctx, out=None):
+        return self._attention(L, self._gemm(h, L.proj.weight), ctx, out=out)
+
     def _attention_layer(self, L, h, ctx):
-        return self._gemm(self._attention(L, self._gemm(h, L.proj.weight), ctx), L.out), None
+        return self._gemm(self._attention_heads(L, h, ctx), L.out), None
 
     def _selective(self, L, proj, ctx, out):
         """Selective scan of a layer over the batch with its output gate -> out [rows, padded channels]."""
         m, sel = L.spec.recurrent, L.sel
         one = ctx.decode and self.tensor_kernels
         x = self._new(ctx.rows, _pad8(m.inner))
-        sel.conv(proj, ctx.batch, one, x)
+        L.conv.run(proj, L.proj.off["rx"], ctx.batch, one, x)
         low = self._gemm(x, L.x_maps.weight)
         dt = None
         if not (one and ctx.rows <= STEP_FUSE_ROWS):
@@ -526,23 +584,24 @@ class HybridEngine(InferenceEngine):
         return y_left, y_right
 
     # ---- latent attention
-    def _latent_tokens(self, L, proj, row_seq, pos, ctx):
+    def _latent_tokens(self, L, queries, gate, row_seq, pos, ctx, out=None):
         """Tokens that attend in the latent's space -> [rows, heads, padded value width]."""
         m, H = L.spec.mixer, L.spec.mixer.heads
-        n, cache = proj.shape[0], self.cache.k[L.att_index]
+        n, cache = queries.shape[0], self.cache.k[L.att_index]
         r_p, dn_p = L.uk_t.shape[1:]
-        q = proj[:, : H * dn_p].unflatten(1, (H, dn_p))
+        q = queries[:, : H * dn_p].unflatten(1, (H, dn_p))
         q_lat = torch.empty(n, H, r_p, device=self.device, dtype=self.dtype)
         o_lat = torch.empty_like(q_lat)
         self.H.gemm_heads(q, L.uk_t, q_lat, self._status)
         if self._fast and L.lat.decode_ok(self.page_size):
-            splits = self._latent_splits(n, H, ctx.max_kv)
+            splits = self._latent_splits(n, H, min(ctx.max_kv, m.window + 64) if m.window else ctx.max_kv)
             scratch = torch.empty(n * H * splits * (r_p + 4) if splits > 1 else 0, device=self.device, dtype=torch.float32)
-            L.lat.attn_decode(q_lat, proj, row_seq, pos, ctx.table, cache, o_lat, scratch, splits, self._status)
+            L.lat.attn_decode(q_lat, queries, row_seq, pos, ctx.table, cache, o_lat, scratch, splits, self._status)
         else:
-            L.lat.attn_any(q_lat, proj, row_seq, pos, ctx.table, cache, o_lat)
-        out = torch.empty(n, H, L.uv.shape[1], device=self.device, dtype=self.dtype)
-        self.H.gemm_heads(o_lat, L.uv, out, self._status)
+            L.lat.attn_any(q_lat, queries, row_seq, pos, ctx.table, cache, o_lat)
+        if out is None:
+            out = torch.empty(n, H, L.uv.shape[1], device=self.device, dtype=self.dtype)
+        self.H.gemm_heads(o_lat, L.uv, out, self._status, gate)
         return out
 
     def _latent_splits(self, rows: int, heads: int, max_kv: int) -> int:
@@ -550,26 +609,39 @@ class HybridEngine(InferenceEngine):
         pairs = rows * ((heads + 15) // 16)
         return max(1, min(64, self._sms // pairs, (max_kv + 127) // 128))
 
-    def _latent(self, L, h, ctx):
+    def _latent_heads(self, L, h, ctx, out=None):
+        """Latent attention up to its output projection -> [rows, heads * padded value width]."""
         m, H = L.spec.mixer, L.spec.mixer.heads
         proj = self._gemm(h, L.proj.weight)
         cache = self.cache.k[L.att_index]
-        L.lat.prep(proj, ctx.batch, ctx.table, cache)
+        queries = proj
+        if L.low is not None:                          # the vector that both query parts are a map of comes first
+            L.lat.prep(proj, ctx.batch, ctx.table, cache, queries=False)
+            queries = self._gemm(proj[:, : L.low.K], L.low.weight)
+        L.lat.prep(queries, ctx.batch, ctx.table, cache, latents=L.low is None)
+        dn_p, dv_p = L.uk_t.shape[2], L.uv.shape[1]
+        gate = proj[:, L.proj.off["g"]:][:, : H * dv_p] if m.gate else None
+        if out is None:
+            out = self._new(ctx.rows, H * dv_p)
+        o = out.unflatten(1, (H, dv_p))
         sp = ctx.split
         if sp is None or L.expand is None or not self._fast or sp.keys * L.expand.shape[0] * 2 > EXPAND_BYTES:
-            o = self._latent_tokens(L, proj, ctx.batch[3], ctx.batch[4], ctx)
-            return self._gemm(o.flatten(1), L.out), None
-        dn_p, dv_p = L.uk_t.shape[2], L.uv.shape[1]
+            self._latent_tokens(L, queries, gate, ctx.batch[3], ctx.batch[4], ctx, o)
+            return out
         latents = self._new(sp.keys, cache.shape[3])
-        L.lat.gather(ctx.table, cache, sp.cu_k, sp.max_k, latents)
+        L.lat.gather(ctx.table, cache, sp.cu_k, sp.first, sp.max_k, latents)
         kv = self._gemm(latents[:, : L.expand.shape[1]], L.expand)
-        o = torch.empty(ctx.rows, H, dv_p, device=self.device, dtype=self.dtype)
-        L.lat.attn_prefill(proj[:, : H * dn_p].unflatten(1, (H, dn_p)), proj, kv[:, : H * dn_p].unflatten(1, (H, dn_p)),
-                           kv[:, H * dn_p:].unflatten(1, (H, dv_p)), latents, ctx.batch, sp.cu_k, ctx.max_q, EXPAND_TOKENS, o,
-                           self._status)
+        L.lat.attn_prefill(queries[:, : H * dn_p].unflatten(1, (H, dn_p)), queries, kv[:, : H * dn_p].unflatten(1, (H, dn_p)),
+                           kv[:, H * dn_p:].unflatten(1, (H, dv_p)), latents, ctx.batch, sp.cu_k, sp.key_lens, ctx.max_q,
+                           EXPAND_TOKENS, gate, o, self._status)
         if sp.short is not None:
-            o.index_copy_(0, sp.short, self._latent_tokens(L, proj.index_select(0, sp.short), sp.short_seq, sp.short_pos, ctx))
-        return self._gemm(o.flatten(1), L.out), None
+            o.index_copy_(0, sp.short, self._latent_tokens(L, queries.index_select(0, sp.short),
+                                                           gate.index_select(0, sp.short) if gate is not None else None,
+                                                           sp.short_seq, sp.short_pos, ctx))
+        return out
+
+    def _latent(self, L, h, ctx):
+        return self._gemm(self._latent_heads(L, h, ctx), L.out), None
 
     # ---- feed-forwards
     def _expert_tile(self, rows: int, m) -> int:
@@ -622,6 +694,24 @@ class HybridEngine(InferenceEngine):
             self.H.gate_pair(gu, f, L.gate_up.off["up"], L.act, a)
         return self._gemm(a, L.down, out)
 
+    def _poly(self, L, h, out):
+        """Ungated feed-forward up to its down matrix."""
+        self.H.poly_norm(self._gemm(h, L.up), L.up_bias, L.poly, L.spec.mlp.ff, out, self.cfg.norm_eps)
+
+    def _side_by_side(self, L, h, ctx):
+        """Mixer and feed-forward of a parallel design -> their sum."""
+        y = self._new(ctx.rows, L.out.shape[1])
+        n = L.mixer_cols
+        L.heads_of(L, ctx.conv if L.conv is not None else h, ctx, y[:, :n])
+        if L.up is not None:
+            self._poly(L, h, y[:, n:])
+        elif L.gate_up is not None:
+            gu = self._gemm(h, L.gate_up.weight)
+            a = self._new(ctx.rows, L.out.shape[1] - n)
+            self.H.gate_pair(gu, L.spec.mlp.ff, L.gate_up.off["up"], L.act, a)
+            y[:, n:].copy_(a)
+        return self._gemm(y, L.out)
+
     def _feed_forward(self, L, h, ctx):
         return self._gated(L, L.spec.mlp.ff, h, ctx)
 
@@ -659,13 +749,16 @@ class HybridEngine(InferenceEngine):
         return self._run_layers(ids, pos, ctx)
 
     def _batch_plan(self, lens, bases):
-        if not any(s.latent is not None for s in self.cfg.layers) or max(lens) < EXPAND_TOKENS:
+        windows = [s.latent.window for s in self.cfg.layers if s.latent is not None]
+        if not windows or max(lens) < EXPAND_TOKENS:
             return [], None
-        cu_k, short, short_seq, short_pos, at, max_k = [0], [], [], [], 0, 0
+        reach = max(windows) if min(windows) > 0 else 0        # keys in front of a query that some layer sees, 0: all
+        cu_k, first, key_lens, short, short_seq, short_pos, at = [0], [], [], [], [], [], 0
         for i, (n, base) in enumerate(zip(lens, bases)):
+            first.append(max(0, base - reach + 1) if reach and n >= EXPAND_TOKENS else 0)
+            key_lens.append(base + n - first[-1])
             if n >= EXPAND_TOKENS:
-                cu_k.append(cu_k[-1] + base + n)
-                max_k = max(max_k, base + n)
+                cu_k.append(cu_k[-1] + key_lens[-1])
             else:
                 cu_k.append(cu_k[-1])
                 short += range(at, at + n)
@@ -673,29 +766,41 @@ class HybridEngine(InferenceEngine):
                 short_pos += range(base, base + n)
             at += n
 
-        def build(cu, rows, seq, pos):
-            return _LatentSplit(cu, cu_k[-1], max_k, rows.long() if short else None, seq, pos)
+        max_k = max(b - a for a, b in zip(cu_k, cu_k[1:]))
 
-        return [cu_k, short, short_seq, short_pos], build
+        def build(cu, skipped, keys, rows, seq, pos):
+            return _LatentSplit(cu, skipped, keys, cu_k[-1], max_k, rows.long() if short else None, seq, pos)
+
+        return [cu_k, first, key_lens, short, short_seq, short_pos], build
 
     def _run_layers(self, ids, pos, ctx, trace=None):
         cfg, H = self.cfg, self.H
         d, eps = cfg.hidden_size, cfg.norm_eps
         x = self._new(ctx.rows, d, torch.float32)
         h = self._new(ctx.rows, _pad8(d))
+        if cfg.input_conv:
+            ctx.conv = self._new(ctx.rows, _pad8(d))
         subs = []                                    # (layer, sublayer function, its norms)
         for L in self.layers:
             subs.append((L, L.run, L.norms))
-            if L.spec.mlp is not None:
+            if L.spec.mlp is not None and not cfg.parallel:
                 subs.append((L, self._experts if L.router is not None else self._feed_forward, L.ff_norms))
             if L.side_gate is not None:
                 subs.append((L, self._token_side, L.side_norms))
+
+        def conv_tail(j):                            # single tokens: the kernel that writes h runs sublayer j's convolution
+            return (subs[j][0].conv, ctx.batch, ctx.conv) if cfg.input_conv and ctx.decode and j < len(subs) else None
+
         H.embed_pos_norm(ids, pos, self.embed_table, self.pos_table, cfg.embed_scale,
-                         subs[0][2].pre if subs else self.final_norm, x, h, eps)
+                         subs[0][2].pre if subs else self.final_norm, x, h, eps, self.embed_norm, conv_tail(0))
         for j, (L, fn, norms) in enumerate(subs):
             nxt = subs[j + 1][2].pre if j + 1 < len(subs) else self.final_norm
+            if cfg.input_conv and not ctx.decode:
+                L.conv.run(h, 0, ctx.batch, False, ctx.conv)
             y = fn(L, h, ctx)
-            if fn == self._experts:
+            if cfg.parallel:
+                H.residual_norm(y, L.down_bias, cfg.residual_mult, x, nxt, h, eps, conv_tail(j + 1))
+            elif fn == self._experts:
                 H.expert_norm(*y, norms.post, x, nxt, h, eps, cfg.residual_mult)
             else:
                 y1, y2 = y if isinstance(y, tuple) else (y, None)
@@ -718,6 +823,8 @@ class HybridEngine(InferenceEngine):
 class _HybridLayer:
     spec = norms = ff_norms = proj = a2 = g2 = out = left_out = right_out = left_norm = right_norm = rec = None
     att = sel = x_maps = w_dt = None
+    conv = low = up = up_bias = poly = down_bias = heads_of = None
+    mixer_cols = 0
     gate_up = down = act = router = correction = rule = w_in = w_out = None
     lat = uk_t = uv = expand = run = None
     side_gate = side_proj = side_embed = side_norms = None

@@ -17,7 +17,9 @@ from .hybrid_config import (AttentionMixer, HybridConfig, LatentAttentionMixer, 
 def _attention_shapes(p: str, m: AttentionMixer, d: int) -> dict:
     out = {p + "q": (m.heads * m.dim, d)}
     if m.kv_from is None:
-        out.update({p + "k": (m.kv_heads * m.dim, d), p + "v": (m.kv_heads * m.vdim, d)})
+        out[p + "k"] = (m.kv_heads * m.dim, d)
+        if m.values == "own":
+            out[p + "v"] = (m.kv_heads * m.vdim, d)
     if m.bias:
         out.update({name + ".b": shape[:1] for name, shape in out.items()})
     if m.qk_norm == "weighted":
@@ -26,7 +28,7 @@ def _attention_shapes(p: str, m: AttentionMixer, d: int) -> dict:
             out[p + "k.norm"] = (m.dim,)
     if m.gate is not None:
         out[p + "g"] = (m.heads * (m.vdim if m.gate == "channel" else 1), d)
-    if m.sink:
+    if m.sink == "learned":
         out[p + "sink"] = (m.heads,)
     out[p + "o"] = (d, m.heads * m.vdim)
     return out
@@ -54,9 +56,17 @@ def _delta_shapes(p: str, m: RecurrentMixer, d: int) -> dict:
 
 
 def _latent_shapes(p: str, m: LatentAttentionMixer, d: int) -> dict:
-    return {p + "q": (m.heads * (m.dim + m.rot_dim), d), p + "dkv": (m.kv_rank + m.rot_dim, d), p + "dkv.norm": (m.kv_rank,),
-            p + "uk": (m.heads * m.dim, m.kv_rank), p + "uv": (m.heads * m.vdim, m.kv_rank), p + "sink": (m.heads,),
-            p + "o": (d, m.heads * m.vdim)}
+    q = m.heads * (m.dim + m.rot_dim)
+    out = {p + "dq": (m.q_rank, d), p + "dq.norm": (m.q_rank,), p + "uq": (q, m.q_rank)} if m.q_rank else {p + "q": (q, d)}
+    if m.kv_from is None:
+        out.update({p + "dkv": (m.kv_rank + m.rot_dim, d), p + "dkv.norm": (m.kv_rank,)})
+    out.update({p + "uk": (m.heads * m.dim, m.kv_rank), p + "uv": (m.heads * m.vdim, m.kv_rank)})
+    if m.sink == "learned":
+        out[p + "sink"] = (m.heads,)
+    if m.gate:
+        out[p + "g"] = (m.heads * m.vdim, d)
+    out[p + "o"] = (d, m.heads * m.vdim)
+    return out
 
 
 def _gated_shapes(p: str, ff: int, d: int) -> dict:
@@ -65,7 +75,9 @@ def _gated_shapes(p: str, ff: int, d: int) -> dict:
 
 def _mlp_shapes(p: str, f, d: int) -> dict:
     if not isinstance(f, MoeFF):
-        return _gated_shapes(p, f.ff, d)
+        if f.gated:
+            return _gated_shapes(p, f.ff, d)
+        return {p + "up": (f.ff, d), p + "up.b": (f.ff,), p + "down": (d, f.ff), p + "down.b": (d,), p + "act": (4,)}
     out = {p + "router": (f.experts, d)}
     if f.correction:
         out[p + "correction"] = (f.experts,)
@@ -82,20 +94,25 @@ def expected_shapes(cfg: HybridConfig) -> dict:
     out = {"embed": (cfg.vocab_size, d)}
     if cfg.position_table:
         out["pos"] = (cfg.max_seq_len, d)
-    out["final.norm"] = (d,)
+    norm = () if cfg.scalar_norms else (d,)
+    out["final.norm"] = norm
+    if cfg.embed_norm:
+        out["embed.norm"] = norm
     if not cfg.tied_head:
         out["head"] = (cfg.vocab_size, d)
     if cfg.token_side:
         out["side.embed"] = (cfg.vocab_size, cfg.num_layers * cfg.token_side)
 
     def norms(p: str, n: int) -> None:                 # a sublayer's norms: before (if the design has one), after
-        out[p + f"norm{n}"] = (d,)
-        if cfg.pre_norm:
-            out[p + f"norm{n}b"] = (d,)
+        out[p + f"norm{n}"] = norm
+        if cfg.pre_norm and cfg.post_norm:
+            out[p + f"norm{n}b"] = norm
 
     for i, spec in enumerate(cfg.layers):
         p = f"l{i}."
         norms(p, 1)
+        if cfg.input_conv:
+            out[p + "canon1"] = (d, cfg.input_conv)
         m = spec.mixer
         if isinstance(m, ParallelMixer):
             right = _selective_shapes if isinstance(m.right, SelectiveMixer) else _delta_shapes
@@ -110,7 +127,8 @@ def expected_shapes(cfg: HybridConfig) -> dict:
         else:
             out.update(_gla_shapes(p + "mix.", m, d))
         if spec.mlp is not None:
-            norms(p, 2)
+            if not cfg.parallel:
+                norms(p, 2)
             out.update(_mlp_shapes(p + "mlp.", spec.mlp, d))
         if cfg.token_side:
             out.update({p + "side.gate": (cfg.token_side, d), p + "side.proj": (d, cfg.token_side), p + "side.norm": (d,)})
@@ -153,11 +171,13 @@ class HybridModel(nn.Module):
                 t = torch.full(shape, 1.0 - cfg.norm_offset, device=device)
             elif leaf == "A_log" and len(shape) == 2:
                 t = torch.log(torch.arange(1, shape[1] + 1, device=device, dtype=torch.float32)).expand(shape)
+            elif leaf == "act":
+                t = torch.tensor([0.6, 0.3, 0.2, 0.0], device=device)
             elif leaf == "D":
                 t = torch.ones(shape, device=device)
             elif name.endswith(".dt.b"):
                 t = -5.0 + 3.0 * torch.rand(shape, device=device, generator=g)
-            elif name.endswith((".q.b", ".k.b", ".v.b", ".conv.b")):
+            elif name.endswith((".q.b", ".k.b", ".v.b", ".conv.b", ".up.b", ".down.b")):
                 t = torch.randn(shape, device=device, generator=g) * std
             elif leaf == "A_log":
                 t = torch.log(1.0 + 3.0 * torch.rand(shape, device=device, generator=g))
@@ -169,7 +189,7 @@ class HybridModel(nn.Module):
                 t = (torch.rand(shape, device=device, generator=g) * 4 + 1 if len(shape) == 1
                      else torch.randn(shape, device=device, generator=g) * std)
             else:
-                t = torch.randn(shape, device=device, generator=g) * (0.5 if leaf == "conv" else std)
+                t = torch.randn(shape, device=device, generator=g) * ({"conv": 0.5, "canon1": 0.25}.get(leaf, std))
             out[name] = t.to(dtype)
         return cls(cfg, out)
 

@@ -12,16 +12,19 @@ Mixers (``LayerSpec.mixer``):
 * ``ParallelMixer``: an attention and a recurrent mixer on the same input, averaged after their own norms or
   added with constant scales;
 * ``LatentAttentionMixer``: attention whose keys and values are linear maps of one normalised latent per
-  token, plus a rotated key part that all heads share; only the latent and that part are cached. A
-  learned sink per head enters the softmax denominator.
+  token, plus a rotated key part that all heads share; only the latent and that part are cached. Low-rank queries,
+  sliding window, sink and output gate as its fields say; a layer may use an earlier one's latents (``kv_from``).
 
-Feed-forwards (``LayerSpec.mlp``): ``DenseFF`` (gated, with its activation) and ``MoeFF`` (a router that
-scores by softmax or sigmoid, with expert groups, over gated experts, and optionally a shared expert).
+Feed-forwards (``LayerSpec.mlp``): ``DenseFF`` (gated, or one projection and a polynomial of normalised powers) and
+``MoeFF`` (a router that scores by softmax or sigmoid, with expert groups, over gated experts, and optionally a shared
+expert).
 
 The designs served under this configuration are Teganex (norms before and after every sublayer, learned
-positions), Lebedra (norms on the sublayer outputs only, latent attention, experts, per-layer token input) and
+positions), Lebedra (norms on the sublayer outputs only, latent attention, experts, per-layer token input),
 Dogozen (norms around sublayers with weights stored around zero, tempered full attention with shared caches,
-window attention beside a selective scan, sigmoid-routed experts, tied and soft-capped output).
+window attention beside a selective scan, sigmoid-routed experts, tied and soft-capped output) and Zigivik (mixer and
+feed-forward side by side behind one norm with a single weight, a short convolution in front of every mixer, window
+latent attention with shared latents, attention whose values are its keys).
 """
 from __future__ import annotations
 
@@ -51,16 +54,49 @@ class FrequencyScaling:
 
 
 @dataclass
+class RampScaling:
+    """YaRN: slows pairs by ``factor`` along a ramp over their number, from the pair that turns ``fast`` times within
+    ``original`` positions (not slowed) to the one that turns ``slow`` times; what is rotated grows by ``amplitude``."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    @property
+    def amplitude(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0
+
+    def ramp(self, base: float, dims: int) -> list:
+        """Share of the slowed frequency in every pair's."""
+        def pair(turns: float) -> float:
+            return dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+        lo, hi = max(math.floor(pair(self.fast)), 0), min(math.ceil(pair(self.slow)), dims - 1)
+        return [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(dims // 2)]
+
+
+@dataclass
 class Rotation:
-    """Rotary positions on the first ``dims`` columns of a head, column i paired with i + dims / 2."""
+    """Rotary positions on the first ``dims`` columns of a head: column i paired with i + dims / 2 (``halves``) or
+    column 2i with 2i + 1 (``pairs``)."""
     base: float
     dims: int
-    scaling: FrequencyScaling | None = None
+    scaling: FrequencyScaling | RampScaling | None = None
+    layout: str = "halves"
 
     def turns(self) -> list:
         """Revolutions per position of every pair."""
         f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
-        return [(self.scaling.apply(x) if self.scaling else x) / (2.0 * math.pi) for x in f]
+        if isinstance(self.scaling, RampScaling):
+            f = [x / self.scaling.factor * r + x * (1.0 - r) for x, r in zip(f, self.scaling.ramp(self.base, self.dims))]
+        elif self.scaling:
+            f = [self.scaling.apply(x) for x in f]
+        return [x / (2.0 * math.pi) for x in f]
+
+    @property
+    def amplitude(self) -> float:
+        """Factor of cosines and sines."""
+        return self.scaling.amplitude if isinstance(self.scaling, RampScaling) else 1.0
 
 
 @dataclass
@@ -68,6 +104,9 @@ class QueryTemperature:
     """Queries at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
     coef: float
     every: float
+
+
+SINKS = ("learned", "zero", None)
 
 
 @dataclass
@@ -80,9 +119,10 @@ class AttentionMixer:
     qk_norm: str | None = "weighted"   # RMS norm of every q / k head: "weighted", "plain" (no weight) or None
     gate: str | None = "head"          # sigmoid output gate: one value per head, per "channel", or None
     bias: bool = False                 # on q, k and v
+    values: str = "own"                # "own", or "keys": the projected keys, before norm and rotation
     rotation: Rotation | None = None
     window: int = 0                    # keys a query sees, itself included; 0: all earlier ones
-    sink: bool = False                 # one more logit per head in the softmax denominator
+    sink: str | None = None            # one more logit per head in the softmax denominator: "learned", or "zero"
     q_temp: QueryTemperature | None = None
     kv_from: int | None = None         # layer whose cached keys and values are used
 
@@ -94,6 +134,10 @@ class AttentionMixer:
             raise ValueError(f"attention: unknown norm {self.qk_norm!r} or gate {self.gate!r}")
         if self.window < 0:
             raise ValueError(f"attention: negative window {self.window}")
+        if self.sink not in SINKS or self.values not in ("own", "keys"):
+            raise ValueError(f"attention: unknown sink {self.sink!r} or values {self.values!r}")
+        if self.values == "keys" and self.dim != self.vdim:
+            raise ValueError(f"attention: keys of width {self.dim} cannot be values of width {self.vdim}")
         r = self.rotation
         if r is not None and (r.dims <= 0 or r.dims % 2 or r.dims > self.dim):
             raise ValueError(f"attention: {r.dims} rotated columns of {self.dim}")
@@ -150,24 +194,38 @@ class LatentAttentionMixer:
     vdim: int
     kv_rank: int               # width of the latent
     scale: float
-    rot_base: float
+    rotation: Rotation         # of all rot_dim columns
+    q_rank: int = 0            # queries are a map of a normalised vector of this width, 0: of the input itself
+    window: int = 0            # keys a query sees, itself included; 0: all earlier ones
+    sink: str | None = "learned"
+    gate: bool = False         # sigmoid output gate per channel
+    kv_from: int | None = None # layer whose cached latents and rotated key parts are used
 
     def __post_init__(self):
         _positive(self, "heads", "dim", "rot_dim", "vdim", "kv_rank")
         if self.rot_dim % 2:
             raise ValueError(f"latent attention: the rotated width must be even, got {self.rot_dim}")
+        if self.rotation.dims != self.rot_dim:
+            raise ValueError(f"latent attention: rotated dimensions {self.rotation.dims} and rotated width {self.rot_dim} differ")
+        if self.sink not in SINKS or self.window < 0 or self.q_rank < 0:
+            raise ValueError(f"latent attention: sink {self.sink!r}, window {self.window} or query rank {self.q_rank}")
 
 
 @dataclass
 class DenseFF:
-    """``down(act(gate h) * (up h))``"""
+    """``down(act(gate h) * (up h))``; with ``act`` "poly_norm" ``down(act(up h + b)) + b``, where act(z) is
+    a N(z) + b N(z^2) + c N(z^3) + e of four weights, N dividing a token's vector by its root mean square."""
     ff: int
-    act: str = "silu"          # "silu" | "relu"
+    act: str = "silu"          # "silu" | "relu" | "poly_norm"
 
     def __post_init__(self):
         _positive(self, "ff")
-        if self.act not in ("silu", "relu"):
+        if self.act not in ("silu", "relu", "poly_norm"):
             raise ValueError(f"feed-forward: unknown activation {self.act!r}")
+
+    @property
+    def gated(self) -> bool:
+        return self.act != "poly_norm"
 
 
 @dataclass
@@ -242,7 +300,12 @@ class HybridConfig:
     architecture: str = "Teganex"
     position_table: bool = True    # learned positions, ``max_seq_len`` rows
     pre_norm: bool = True          # sublayers read a normalised copy of the stream (else the stream itself)
-    residual_mult: float = 1.0     # x <- x + residual_mult * norm(sublayer)
+    post_norm: bool = True         # sublayer outputs are normalised before they are added
+    parallel: bool = False         # mixer and feed-forward read the same norm and are added together
+    scalar_norms: bool = False     # the model's norms have one weight for all coordinates
+    embed_norm: bool = False       # the stream starts from a normalised embedding
+    input_conv: int = 0            # mixers read h + a causal convolution of h over this many tokens, 0: h
+    residual_mult: float = 1.0     # x <- x + residual_mult * sublayer
     token_side: int = 0            # width of the per-layer token input, 0: none
     norm_offset: float = 0.0       # added to every stored norm weight
     tied_head: bool = False        # the embedding table is the output matrix
@@ -251,7 +314,19 @@ class HybridConfig:
 
     def __post_init__(self):
         _positive(self, "vocab_size", "hidden_size", "max_seq_len")
+        if self.input_conv < 0:
+            raise ValueError(f"input convolution over {self.input_conv} tokens")
+        if self.parallel and (self.post_norm or not self.pre_norm or self.token_side or self.position_table):
+            raise ValueError("sublayers side by side come with a norm in front only, no token input and no position table")
         for i, x in enumerate(self.layers):
+            if self.parallel and (x.attention is None and x.latent is None or isinstance(x.mixer, ParallelMixer)
+                                  or isinstance(x.mlp, MoeFF)):
+                raise ValueError(f"layer {i}: only attention and dense feed-forwards run side by side")
+            a = x.latent
+            if a is not None and a.kv_from is not None:
+                b = self.layers[a.kv_from].latent if 0 <= a.kv_from < i else None
+                if b is None or b.kv_from is not None or (b.kv_rank, b.rot_dim, b.rotation) != (a.kv_rank, a.rot_dim, a.rotation):
+                    raise ValueError(f"layer {i}: layer {a.kv_from} has no latents of its shape and rotation to share")
             a = x.attention
             if a is None or a.kv_from is None:
                 continue
@@ -281,12 +356,16 @@ class HybridConfig:
             return cls(layers=[_dogozen_layer(i, x) for i, x in enumerate(d["layers"])],
                        position_table=False, norm_offset=1.0, tied_head=True, logit_softcap=float(d.get("logit_softcap") or 0.0),
                        **common)
+        if arch == "Zigivik":
+            return cls(layers=[_zigivik_layer(i, x) for i, x in enumerate(d["layers"])], position_table=False, post_norm=False,
+                       parallel=True, scalar_norms=True, embed_norm=True, input_conv=int(d["canon"]["taps"]),
+                       residual_mult=float(d["residual_mult"]), **common)
         return cls(layers=[_layer_from_dict(i, x, ("gla", "parallel"), "silu") for i, x in enumerate(d["layers"])],
                    embed_scale=float(d["embedding"]["scale"]), logit_scale=float(d["logit_scale"]),
                    max_seq_len=int(d["max_positions"]), **common)
 
     def to_dict(self) -> dict:
-        layer = _dogozen_layer_to_dict if self.architecture == "Dogozen" else _layer_to_dict
+        layer = {"Dogozen": _dogozen_layer_to_dict, "Zigivik": _zigivik_layer_to_dict}.get(self.architecture, _layer_to_dict)
         d = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
              "norm": {"eps": self.norm_eps}, "layers": [layer(x) for x in self.layers]}
         if self.architecture == "Lebedra":
@@ -296,6 +375,8 @@ class HybridConfig:
         elif self.architecture == "Dogozen":
             if self.logit_softcap:
                 d["logit_softcap"] = self.logit_softcap
+        elif self.architecture == "Zigivik":
+            d.update(residual_mult=self.residual_mult, canon={"taps": self.input_conv})
         else:
             d.update(max_positions=self.max_seq_len, embedding={"scale": self.embed_scale}, logit_scale=self.logit_scale)
         return d
@@ -320,10 +401,8 @@ def _layer_from_dict(index: int, d: dict, kinds: tuple, act: str) -> LayerSpec:
             RecurrentMixer("delta", int(r["heads"]), int(r["kv_heads"]), int(r["dim"]), int(r["vdim"]), conv=int(r["conv"])))
     else:
         rot = m["rot"]
-        if int(rot.get("dims", m["rot_dim"])) != int(m["rot_dim"]):
-            raise ValueError(f"layer {index}: rotated dimensions {rot['dims']} and rotated width {m['rot_dim']} differ")
         mixer = LatentAttentionMixer(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]),
-                                     float(m["scale"]), float(rot["base"]))
+                                     float(m["scale"]), Rotation(float(rot["base"]), int(rot.get("dims", m["rot_dim"])), layout="pairs"))
     return LayerSpec(kind, mixer, _mlp_from_dict(index, d.get("mlp"), act))
 
 
@@ -348,7 +427,7 @@ def _layer_to_dict(x: LayerSpec) -> dict:
                            "conv": m.right.conv}}
     elif isinstance(m, LatentAttentionMixer):
         mixer = {"heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank, "scale": m.scale,
-                 "rot": {"base": m.rot_base, "dims": m.rot_dim}}
+                 "rot": {"base": m.rotation.base, "dims": m.rot_dim}}
     else:
         mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "tau": m.tau}
     f = x.mlp
@@ -380,7 +459,7 @@ def _dogozen_layer(index: int, d: dict) -> LayerSpec:
         mixer = _dogozen_attention(m, qk_norm="plain", gate="channel", bias=True)
     elif kind == "parallel":
         r = m["right"]
-        mixer = ParallelMixer(_dogozen_attention(m["left"], qk_norm=None, gate=None, sink=True),
+        mixer = ParallelMixer(_dogozen_attention(m["left"], qk_norm=None, gate=None, sink="learned"),
                               SelectiveMixer(int(r["inner"]), int(r["state"]), int(r["dt_rank"]), int(r["conv"])),
                               (float(m["left_scale"]), float(m["right_scale"])))
     else:
@@ -424,6 +503,46 @@ def _dogozen_layer_to_dict(x: LayerSpec) -> dict:
     return {"type": x.type, "mixer": mixer, "mlp": mlp}
 
 
+# ---- Zigivik
+def _zigivik_layer(index: int, d: dict) -> LayerSpec:
+    kind, m, mlp = d["type"], d["mixer"], d.get("mlp")
+    if kind not in ("attention", "latent_attention"):
+        raise ValueError(f"layer {index}: unknown mixer type {kind!r}")
+    rot = m["rot"]
+    scaling = rot.get("scaling")
+    if scaling:
+        scaling = RampScaling(*(float(scaling[n]) for n in ("factor", "original", "fast", "slow")))
+    rotation = Rotation(float(rot["base"]), int(rot["dims"]), scaling or None, "pairs" if kind == "attention" else "halves")
+    window = int((m.get("mask") or {}).get("size", 0))
+    if kind == "attention":
+        mixer = AttentionMixer(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), qk_norm=None,
+                               gate=None, bias=True, values="keys", rotation=rotation, window=window, sink="zero")
+    else:
+        mixer = LatentAttentionMixer(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]),
+                                     float(m["scale"]), rotation, q_rank=int(m["q_rank"]), window=window, sink=None, gate=True,
+                                     kv_from=int(m["kv_from"]) if m.get("kv_from") is not None else None)
+        _positive(mixer, "q_rank")
+    return LayerSpec(kind, mixer, _mlp_from_dict(index, mlp, "poly_norm"))
+
+
+def _zigivik_layer_to_dict(x: LayerSpec) -> dict:
+    m = x.mixer
+    r = m.rotation
+    rot = {"base": r.base, "dims": r.dims}
+    if r.scaling:
+        rot["scaling"] = dict(vars(r.scaling))
+    mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale, "rot": rot}
+    if isinstance(m, AttentionMixer):
+        mixer["kv_heads"] = m.kv_heads
+    else:
+        mixer.update(rot_dim=m.rot_dim, kv_rank=m.kv_rank, q_rank=m.q_rank)
+        if m.kv_from is not None:
+            mixer["kv_from"] = m.kv_from
+    if m.window:
+        mixer["mask"] = {"size": m.window}
+    return {"type": x.type, "mixer": mixer, "mlp": {"kind": "dense", "ff": x.mlp.ff} if x.mlp is not None else None}
+
+
 # ------------------------------------------------------------------ named configurations
 def teganex_config(width: int = 2048, layers: int = 8, vocab: int = 32000, max_positions: int = 8192,
                    parallel_every: int = 4) -> HybridConfig:
@@ -445,7 +564,8 @@ def lebedra_config(width: int = 2048, layers: int = 8, vocab: int = 32000, max_p
                    top: int = 6) -> HybridConfig:
     """Lebedra at the layer sizes of a real model: latents of 512 with heads of 128 + 64 rotated, a dense first
     layer, then experts whose ``top`` together are about as wide as the dense feed-forward."""
-    mixer = LatentAttentionMixer(width // 128, 128, 64, 128, 512, 192 ** -0.5, 10000.0)
+    mixer = LatentAttentionMixer(width // 128, 128, 64, 128, 512, 192 ** -0.5,
+                                 Rotation(10000.0, 64, layout="pairs"))
     dense = width * 11 // 4 // 128 * 128
     moe = MoeFF(experts, top, max(128, dense // top // 128 * 128), 7.0, 8, 3)
     out = [LayerSpec("latent_attention", mixer, DenseFF(dense, "relu") if i == 0 else moe) for i in range(layers)]
@@ -473,13 +593,36 @@ def dogozen_config(width: int = 2048, layers: int = 8, vocab: int = 32000, max_p
                 q_temp=QueryTemperature(0.1, 8192), kv_from=share), DenseFF(dense)))
         else:
             out.append(LayerSpec("parallel", ParallelMixer(
-                AttentionMixer(h, max(1, h // 8), 128, 128, 128 ** -0.5, qk_norm=None, gate=None, sink=True, window=window,
+                AttentionMixer(h, max(1, h // 8), 128, 128, 128 ** -0.5, qk_norm=None, gate=None, sink="learned", window=window,
                                rotation=Rotation(500000.0, 128, FrequencyScaling(8.0, 1.0, 4.0, 8192))),
                 SelectiveMixer(2 * width, 16, max(8, width // 16), 4), (1.0, 1.0)), moe))
     return HybridConfig(vocab, width, out, 1e-6, max_seq_len=max_positions, architecture="Dogozen", position_table=False,
                         norm_offset=1.0, tied_head=True, logit_softcap=50.0)
 
 
+def zigivik_config(width: int = 2048, layers: int = 8, vocab: int = 32000, max_positions: int = 8192,
+                   window: int = 1024) -> HybridConfig:
+    """Zigivik at the layer sizes of a real model: every fourth layer full attention (one key head for eight query
+    heads, 128 wide), the others window attention over latents of 512 with heads of 128 + 64 rotated; the second of
+    three neighbours uses the first one's latents. The ungated feed-forward is as wide as a gated one is in all."""
+    h = width // 128
+    ff = DenseFF(width * 11 // 4 // 128 * 128 * 3 // 2 // 128 * 128, "poly_norm")
+    rot = Rotation(500000.0, 64, RampScaling(8.0, 8192, 32.0, 1.0), "halves")
+    out = []
+    for i in range(layers):
+        if i % 4 == 3:
+            out.append(LayerSpec("attention", AttentionMixer(
+                h, max(1, h // 8), 128, 128, 128 ** -0.5, qk_norm=None, gate=None, bias=True, values="keys",
+                rotation=Rotation(500000.0, 128, layout="pairs"), sink="zero"), ff))
+        else:
+            out.append(LayerSpec("latent_attention", LatentAttentionMixer(
+                h, 128, 64, 128, 512, 192 ** -0.5, rot, q_rank=width * 3 // 8 // 128 * 128, window=window, sink=None, gate=True,
+                kv_from=i - 1 if i % 4 == 1 else None), ff))
+    return HybridConfig(vocab, width, out, 1e-6, max_seq_len=max_positions, architecture="Zigivik", position_table=False,
+                        post_norm=False, parallel=True, scalar_norms=True, embed_norm=True, input_conv=4, residual_mult=0.7)
+
+
 register("Dogozen", HybridConfig.from_dict, "mythos_b200.models.hybrid:HybridModel")
 register("Lebedra", HybridConfig.from_dict, "mythos_b200.models.hybrid:HybridModel")
 register("Teganex", HybridConfig.from_dict, "mythos_b200.models.hybrid:HybridModel")
+register("Zigivik", HybridConfig.from_dict, "mythos_b200.models.hybrid:HybridModel")

@@ -283,7 +283,7 @@ def run_dogozen_kernels(peaks: dict, width: int = 2048) -> list[dict]:
         proj, x, low, out = rnd(n, N), rnd(n, c), rnd(n, par.x_maps.N), torch.empty(n, c, device="cuda", dtype=bf)
         dt, sizes = torch.randn(n, c, device="cuda") - 3.0, f"{B} x {S}, {c} channels, {ns} state values"
         scratch = torch.empty(sel.scratch_floats(B, n, S), device="cuda")
-        K.add("selective_conv", sizes, lambda: sel.conv(proj, b, False, x), nbytes=4.0 * n * c, like="rope (dense)")
+        K.add("selective_conv", sizes, lambda: par.conv.run(proj, par.proj.off["rx"], b, False, x), nbytes=4.0 * n * c, like="rope (dense)")
         K.add("selective_scan", sizes, lambda: sel.scan(proj, x, low, dt, b, S, scratch, out, st),
               nbytes=n * (c * 10.0 + 4 * ns) + 8.0 * B * c * ns, like="chunked recurrence + norm + gate")
         _recurrent_rows(K, H, st, "delta", h, 128, 128, [S] * B, False)
@@ -293,7 +293,7 @@ def run_dogozen_kernels(peaks: dict, width: int = 2048) -> list[dict]:
         proj, x, low, out = rnd(T, N), rnd(T, c), rnd(T, par.x_maps.N), torch.empty(T, c, device="cuda", dtype=bf)
         dt = torch.randn(T, c, device="cuda") if T > STEP_FUSE_ROWS else None
         sizes = f"{T} tokens, {c} channels, {ns} state values"
-        K.add("selective_conv, one token", sizes, lambda: sel.conv(proj, b, True, x), nbytes=T * c * (4.0 + 24), like="recurrent_decode")
+        K.add("selective_conv, one token", sizes, lambda: par.conv.run(proj, par.proj.off["rx"], b, True, x), nbytes=T * c * (4.0 + 24), like="recurrent_decode")
         K.add("selective_step", sizes, lambda: sel.step(proj, x, low, dt, b, out),
               nbytes=T * c * (8.0 * ns + 6 + 4 * (dt is not None)) + 2.0 * c * r.dt_rank * (dt is None), like="recurrent_decode")
         _recurrent_rows(K, H, st, "delta", h, 128, 128, [1] * T, True)
@@ -346,17 +346,17 @@ def run_lebedra_kernels(peaks: dict, width: int = 2048) -> list[dict]:
 
     for B, S in ((4, 2048), (1, 8192)):
         table, cache = pages(B, S)
-        b, n = _batch([S] * B, [0] * B), B * S
+        b, n, zero = _batch([S] * B, [0] * B), B * S, torch.zeros(B, device="cuda", dtype=torch.int32)
         proj, o = rnd(n, L.proj.N), torch.empty(n, h, m.vdim, device="cuda", dtype=bf)
         lat, kv = torch.empty(n, W, device="cuda", dtype=bf), rnd(n, h * (m.dim + m.vdim))
         q, k, v = (t.unflatten(1, (h, 128)) for t in (proj[:, : h * m.dim], kv[:, : h * m.dim], kv[:, h * m.dim:]))
         K.add("latent_prep", f"{n} tokens, {h} heads", lambda: L.lat.prep(proj, b, table, cache),
               nbytes=2.0 * n * (2 * h * m.rot_dim + 2 * W), like="rope (dense)")
-        K.add("latent_gather", f"{n} tokens", lambda: L.lat.gather(table, cache, b[0], S, lat), nbytes=4.0 * n * W, like="rope (dense)")
+        K.add("latent_gather", f"{n} tokens", lambda: L.lat.gather(table, cache, b[0], zero, S, lat), nbytes=4.0 * n * W, like="rope (dense)")
         K.add("expand latents (GEMM)", f"{n} x {L.expand.shape[0]} x {r}", lambda: H.gemm_nt(lat[:, :r], L.expand, kv, 1.0, st),
               flops=2.0 * n * L.expand.shape[0] * r, like="gemm (dense bf16)")
         K.add("latent prefill attention", f"{B} x {S}, {h} heads, 128 + 64 / 128",
-              lambda: L.lat.attn_prefill(q, proj, k, v, lat, b, b[0], S, 16, o, st),
+              lambda: L.lat.attn_prefill(q, proj, k, v, lat, b, b[0], b[1], S, 16, None, o, st),
               flops=2.0 * B * h * (S * (S + 1) / 2) * (m.dim + m.rot_dim + m.vdim), like="paged prefill attention (dense)")
     qkv, pos = rnd(8192, h + 2, 128), torch.arange(2048, device="cuda", dtype=torch.int32).repeat(4)
     K.add("rope (dense)", f"8192 tokens, {h} heads, 128", lambda: C.rope(qkv[:, :h], pos, 10000.0, False), nbytes=4.0 * 8192 * h * 128)

@@ -1,5 +1,7 @@
 """Plain, slow PyTorch statement of the hybrid designs (one function per mechanism, token by token where
 there is a recurrence). It is the yardstick of the hybrid tests and shares no code with the package."""
+import math
+
 import torch
 
 
@@ -386,12 +388,143 @@ def forward_dogozen(cfg, W, tokens, dtype=torch.float64, trace=None):
     return soft_cap(rms_norm_around_zero(x, W["final.norm"], eps) @ W["embed"].T, cfg["logit_softcap"])
 
 
+# ------------------------------------------------------------------ Zigivik
+def one_number_norm(x, g, eps):
+    return rms(x, eps) * g
+
+
+def input_conv(h, w):
+    """What a mixer reads: h plus a causal convolution of it per channel."""
+    return h + short_conv(h, w)
+
+
+def yarn_frequencies(r):
+    """(angle per position of every rotated pair, factor of cosines and sines). Pairs up to the one that turns ``fast``
+    times within ``original`` positions keep their frequency, those from the one that turns ``slow`` times on are
+    slowed by ``factor``, with a linear ramp over the pair's number between."""
+    n, base, sc = r["dims"], float(r["base"]), r.get("scaling")
+    f = [base ** (-2.0 * i / n) for i in range(n // 2)]
+    if not sc:
+        return f, 1.0
+    pair = lambda turns: n * math.log(sc["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
+    lo, hi = max(math.floor(pair(sc["fast"])), 0), min(math.ceil(pair(sc["slow"])), n - 1)
+    out = []
+    for i, x in enumerate(f):
+        ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        out.append(x / sc["factor"] * ramp + x * (1 - ramp))
+    return out, 0.1 * math.log(sc["factor"]) + 1
+
+
+def turn_halves(x, pos, r):
+    """Components i and i + dims / 2 of x [T, heads, n] turn together, with yarn_frequencies; the rest stays."""
+    out, half = x.clone(), r["dims"] // 2
+    freq, amp = yarn_frequencies(r)
+    for i, f in enumerate(freq):
+        a = pos.to(torch.float64) * f
+        c, s = (amp * torch.cos(a)).to(x.dtype)[:, None], (amp * torch.sin(a)).to(x.dtype)[:, None]
+        u, v = x[..., i], x[..., i + half]
+        out[..., i], out[..., i + half] = u * c - v * s, v * c + u * s
+    return out
+
+
+def turn_pairs(x, pos, r):
+    """Components 2i and 2i + 1 of the first ``dims`` of x [T, heads, n] turn together; the rest stays."""
+    out = x.clone()
+    out[..., : r["dims"]] = rotate_pairs(x[..., : r["dims"]], pos, r["base"])
+    return out
+
+
+def banded_attention(q, k, v, scale, window=None, plus_one=False):
+    """Query i sees keys j <= i, with ``window`` only those with i - j < window; ``plus_one``: one is added to the
+    denominator. q [T, H, dk]; k [T, G, dk]; v [T, G, dv]."""
+    T, H, _ = q.shape
+    G = k.shape[1]
+    i = torch.arange(T)
+    hidden = i[None, :] > i[:, None]
+    if window is not None:
+        hidden = hidden | (i[:, None] - i[None, :] >= window)
+    out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    for h in range(H):
+        g = h // (H // G)
+        s = ((q[:, h] @ k[:, g].T) * scale).masked_fill(hidden, float("-inf"))
+        m = s.max(-1, keepdim=True).values
+        if plus_one:
+            m = torch.clamp(m, min=0.0)
+        e = torch.exp(s - m)
+        out[:, h] = (e @ v[:, g]) / (e.sum(-1, keepdim=True) + (torch.exp(-m) if plus_one else 0.0))
+    return out
+
+
+def low_rank_queries(h, W, p, eps):
+    return rms_norm(h @ W[p + "dq"].T, W[p + "dq.norm"], eps) @ W[p + "uq"].T
+
+
+def window_latent_attention(h, W, p, c, eps, kept):
+    """``kept`` (layer -> latent and rotated key part) receives the layer's own and gives those of a layer that shares
+    them."""
+    T, H, dn, dr, dv = h.shape[0], c["heads"], c["dim"], c["rot_dim"], c["vdim"]
+    pos = torch.arange(T)
+    q = low_rank_queries(h, W, p, eps).view(T, H, dn + dr)
+    q = torch.cat([q[..., :dn], turn_halves(q[..., dn:], pos, c["rot"])], -1)
+    if c.get("kv_from") is None:
+        kv = h @ W[p + "dkv"].T
+        lat = rms_norm(kv[:, : c["kv_rank"]], W[p + "dkv.norm"], eps)
+        kr = turn_halves(kv[:, None, c["kv_rank"]:], pos, c["rot"])[:, 0]
+        kept[p] = (lat, kr)
+    else:
+        lat, kr = kept[f"l{c['kv_from']}.mix."]
+    k = torch.cat([(lat @ W[p + "uk"].T).view(T, H, dn), kr[:, None].expand(T, H, dr)], -1)
+    v = (lat @ W[p + "uv"].T).view(T, H, dv)
+    o = banded_attention(q, k, v, c["scale"], (c.get("mask") or {}).get("size")).reshape(T, H * dv)
+    return (o * torch.sigmoid(h @ W[p + "g"].T)) @ W[p + "o"].T
+
+
+def key_value_attention(h, W, p, c):
+    """The values are the keys before their rotation."""
+    T, H, G = h.shape[0], c["heads"], c["kv_heads"]
+    pos = torch.arange(T)
+    q = (h @ W[p + "q"].T + W[p + "q.b"]).view(T, H, c["dim"])
+    k = (h @ W[p + "k"].T + W[p + "k.b"]).view(T, G, c["dim"])
+    o = banded_attention(turn_pairs(q, pos, c["rot"]), turn_pairs(k, pos, c["rot"]), k, c["scale"], plus_one=True)
+    return o.reshape(T, H * c["vdim"]) @ W[p + "o"].T
+
+
+def poly_norm(z, act, eps):
+    a, b, c, e = act
+    return a * rms(z, eps) + b * rms(z ** 2, eps) + c * rms(z ** 3, eps) + e
+
+
+def poly_ff(h, W, p, eps):
+    return poly_norm(h @ W[p + "up"].T + W[p + "up.b"], W[p + "act"], eps) @ W[p + "down"].T + W[p + "down.b"]
+
+
+def forward_zigivik(cfg, W, tokens, dtype=torch.float64, trace=None):
+    W = {k: v.to(dtype) for k, v in W.items()}
+    eps, m = cfg["norm"]["eps"], cfg["residual_mult"]
+    x = one_number_norm(W["embed"][torch.as_tensor(tokens, dtype=torch.long)], W["embed.norm"], eps)
+    kept = {}
+    for i, L in enumerate(cfg["layers"]):
+        p = f"l{i}."
+        h = one_number_norm(x, W[p + "norm1"], eps)
+        g = input_conv(h, W[p + "canon1"])
+        y = (key_value_attention(g, W, p + "mix.", L["mixer"]) if L["type"] == "attention"
+             else window_latent_attention(g, W, p + "mix.", L["mixer"], eps, kept))
+        if L["mlp"] is not None:
+            y = y + poly_ff(h, W, p + "mlp.", eps)
+        x = x + m * y
+        if trace is not None:
+            trace.append(x)
+    return one_number_norm(x, W["final.norm"], eps) @ W["head"].T
+
+
 def forward(cfg, W, tokens, dtype=torch.float64, trace=None):
     """Logits [T, vocab] of one sequence; ``trace`` (a list) receives the stream after every layer."""
     if cfg["architecture"] == "Lebedra":
         return forward_lebedra(cfg, W, tokens, dtype, trace)
     if cfg["architecture"] == "Dogozen":
         return forward_dogozen(cfg, W, tokens, dtype, trace)
+    if cfg["architecture"] == "Zigivik":
+        return forward_zigivik(cfg, W, tokens, dtype, trace)
     W = {k: v.to(dtype) for k, v in W.items()}
     eps = cfg["norm"]["eps"]
     tok = torch.as_tensor(tokens, dtype=torch.long)

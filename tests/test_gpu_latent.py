@@ -85,13 +85,13 @@ class Case:
             keys = sum(self.total)
             cu = torch.tensor([sum(self.total[:i]) for i in range(len(self.total) + 1)], dtype=torch.int32, device="cuda")
             lat = torch.full((keys, self.W), float("nan"), device="cuda", dtype=self.dtype)
-            self.lat.gather(self.table, self.cache, cu, max(self.total), lat)
+            self.lat.gather(self.table, self.cache, cu, torch.zeros_like(cu[1:]), max(self.total), lat)
             kv = torch.zeros(keys, Hn * (self.dim_p + self.vdim_p), device="cuda", dtype=self.dtype)
             k, v = kv[:, : Hn * self.dim_p].unflatten(1, (Hn, self.dim_p)), kv[:, Hn * self.dim_p:].unflatten(1, (Hn, self.vdim_p))
             c = lat[:, : self.rank].float()
             k[..., : self.dim] = torch.einsum("tr,hdr->thd", c, self.uk.float()).to(self.dtype)
             v[..., : self.vdim] = torch.einsum("tr,hdr->thd", c, self.uv.float()).to(self.dtype)
-            self.lat.attn_prefill(q, self.proj, k, v, lat, self.batch, cu, max(self.lens), 1, out, status())
+            self.lat.attn_prefill(q, self.proj, k, v, lat, self.batch, cu, self.batch[1], max(self.lens), 1, None, out, status())
             return out[..., : self.vdim]
         uk = torch.zeros(Hn, self.rank_p, self.dim_p, device="cuda", dtype=self.dtype)
         uk[:, : self.rank, : self.dim] = self.uk.transpose(1, 2)
@@ -207,13 +207,13 @@ def test_short_and_long_portions_in_one_batch_stay_apart():
     want = c.want()
     cu = torch.tensor([0, 0, 45, 45], dtype=torch.int32, device="cuda")
     lat = torch.empty(45, c.W, device="cuda", dtype=BF16)
-    c.lat.gather(c.table, c.cache, cu, 45, lat)
+    c.lat.gather(c.table, c.cache, cu, torch.zeros_like(cu[1:]), 45, lat)
     kv = torch.zeros(45, 4 * 128, device="cuda", dtype=BF16)
     k, v = kv[:, :256].unflatten(1, (4, 64)), kv[:, 256:].unflatten(1, (4, 64))
     k.copy_(torch.einsum("tr,hdr->thd", lat[:, :96].float(), c.uk.float()))
     v.copy_(torch.einsum("tr,hdr->thd", lat[:, :96].float(), c.uv.float()))
     out = torch.full((44, 4, 64), 7.0, device="cuda", dtype=BF16)
-    c.lat.attn_prefill(c.queries()[0], c.proj, k, v, lat, c.batch, cu, 40, 16, out, status())
+    c.lat.attn_prefill(c.queries()[0], c.proj, k, v, lat, c.batch, cu, c.batch[1], 40, 16, None, out, status())
     close(out[3:43], want[3:43], 2.5e-2)
     assert float((out[:3] - 7.0).abs().max()) == 0.0 and float((out[43:] - 7.0).abs().max()) == 0.0
 

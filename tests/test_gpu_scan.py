@@ -258,12 +258,14 @@ class Scan:
         a = torch.zeros(inner, sp)
         a[:, :state] = self.A.double() / math.log(2.0)
         self.conv_w, self.conv_b, self.D, self.dt_b = rnd(inner, taps) * 0.5, rnd(inner) * 0.3, 1 + 0.3 * rnd(inner), rnd(inner) * 1.5 - 2.0
-        self.t = {"conv_w": self.conv_w.t(), "conv_b": self.conv_b, "a": a, "d": self.D, "dt_b": self.dt_b,
-                  "state": torch.full((slots, inner, sp), 7.0), "conv_state": torch.full((slots, max(1, taps - 1), inner), 7.0)}
+        self.t = {"a": a, "d": self.D, "dt_b": self.dt_b,
+                  "state": torch.full((slots, inner, sp), 7.0)}
         self.t = {k: v.contiguous().cuda() for k, v in self.t.items()}
         self.t["w_dt"] = self.w_dt
-        self.sel = H().Selective({"inner": inner, "state": state, "rank": rank, "taps": taps, "out_scale": out_scale, "x_off": 0,
-                                  "z_off": self.z_off, "b_off": self.b_off, "c_off": self.c_off}, self.t)
+        self.conv = H().Conv(inner, False, self.conv_w.t().contiguous().cuda(), self.conv_b.cuda(),
+                             torch.full((slots, taps - 1, inner), 7.0, device="cuda") if taps > 1 else None)
+        self.sel = H().Selective({"inner": inner, "state": state, "rank": rank, "out_scale": out_scale, "z_off": self.z_off,
+                                  "b_off": self.b_off, "c_off": self.c_off}, self.t)
 
     def want(self, lo, hi):
         """Rows [lo, hi) as one sequence from the start; the convolved channels and the maps are rounded as the kernels
@@ -282,7 +284,7 @@ class Scan:
         proj, batch, n = self.proj[idx].contiguous(), ragged(lens, bases, slots), sum(lens)
         full = lambda *s, t=self.dtype: torch.full(s, float("nan"), device="cuda", dtype=t)
         x = full(n, pad8(self.inner))
-        self.sel.conv(proj, batch, one, x)
+        self.conv.run(proj, 0, batch, one, x)
         assert float(x[:, self.inner:].float().abs().sum()) == 0.0
         low = (d(x)[:, : self.inner] @ d(self.w_low)[:, : self.inner].t()).to("cuda", self.dtype)
         dt = (d(low)[:, : self.rank] @ d(self.w_dt)[:, : self.rank].t()).float().cuda()

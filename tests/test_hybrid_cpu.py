@@ -224,11 +224,11 @@ def test_batch_plan_separates_long_and_short_portions():
     n = EXPAND_TOKENS
     assert HybridEngine._batch_plan(Cfg, [1, n - 1], [5, 0]) == ([], None)
     lists, build = HybridEngine._batch_plan(Cfg, [2, n, 1, n + 3], [7, 0, 0, 100])
-    assert lists == [[0, 0, n, n, 2 * n + 103], [0, 1, n + 2], [0, 0, 2], [7, 8, 0]]
+    assert lists == [[0, 0, n, n, 2 * n + 103], [0] * 4, [9, n, 1, n + 103], [0, 1, n + 2], [0, 0, 2], [7, 8, 0]]
     sp = build(*[torch.tensor(x, dtype=torch.int32) for x in lists])
     assert sp.keys == 2 * n + 103 and sp.max_k == n + 103 and sp.short.dtype == torch.int64
     lists, build = HybridEngine._batch_plan(Cfg, [n], [3])
-    assert lists == [[0, n + 3], [], [], []] and build(*[torch.tensor(x) for x in lists]).short is None
+    assert lists == [[0, n + 3], [0], [n + 3], [], [], []] and build(*[torch.tensor(x) for x in lists]).short is None
 
 
 class _FakeEngine:
