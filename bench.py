@@ -194,7 +194,7 @@ def main() -> int:
                     help="data-parallel gradient path: fused peer-memory kernels or plain NCCL collectives")
     ap.add_argument("--activation-checkpointing", action="store_true",
                     help="recompute block activations in the backward pass (memory for one extra forward)")
-    ap.add_argument("--hybrid", nargs="?", const="teganex", default=None, choices=["teganex", "lebedra", "dogozen"],
+    ap.add_argument("--hybrid", nargs="?", const="teganex", default=None, choices=["teganex", "lebedra", "dogozen", "zigivik"],
                     help="instead of the headline workload: prefill / decode throughput and kernel times of layer-list layers "
                          "of this design (default: teganex) beside the dense engine of equal size, one JSON line (1 GPU)")
     ap.add_argument("--no-decode", action="store_true", help="skip the tensor-parallel decode measurement")

@@ -49,6 +49,12 @@ __device__ __forceinline__ void ldv(const __nv_bfloat16* p, float (&f)[V]) {
     f[0] = __bfloat162float(*p);
   }
 }
+// What type T keeps of a value.
+template <typename T>
+__device__ __forceinline__ float kept(float v) {
+  if constexpr (sizeof(T) == 2) return __bfloat162float(__float2bfloat16(v));
+  else return v;
+}
 template <int V>
 __device__ __forceinline__ void stv(float* p, const float (&f)[V]) {
   if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
@@ -67,14 +73,54 @@ __device__ __forceinline__ void stv(__nv_bfloat16* p, const float (&f)[V]) {
   }
 }
 
+// The state and weights that row t's convolution will want, on their way to L2 while the row is reduced.
+__device__ __forceinline__ void prefetch_tail(const ConvTail& cv, int dim, long long t) {
+  if (cv.c.taps <= 1) return;
+  const float* state = cv.c.state + (long long)cv.slots[t] * (cv.c.taps - 1) * dim;
+  const int n = (cv.c.taps - 1) * dim;
+  for (int i = threadIdx.x * 32; i < n; i += SN_THREADS * 32) {
+    asm volatile("prefetch.global.L2 [%0];" ::"l"(state + i));
+    asm volatile("prefetch.global.L2 [%0];" ::"l"(cv.c.w + i));
+  }
+}
+
 // h = rms(row) * gamma (or the row itself) for a row held in shared memory; columns [dim, ldh) are zeroed (GEMM padding).
-// With a convolution tail, row t being the new token of sequence t, also h + conv(h).
+// With a convolution tail, row t being the new token of sequence t, also h + conv(h) of what the activation type keeps of h.
 template <typename T, int V>
 __device__ __forceinline__ void write_normed(const float* row, float ss, const float* gamma, T* h, long long ldh,
                                              int dim, float eps, const ConvTail& cv, long long t) {
   const float r = 1.f / sqrtf(ss / (float)dim + eps);
+  const int taps = cv.c.taps;
+  T* out = taps > 0 ? static_cast<T*>(cv.out) + t * cv.ld : nullptr;
+  float* state = taps > 1 ? cv.c.state + (long long)cv.slots[t] * (taps - 1) * dim : nullptr;
+  const bool fresh = taps > 0 && cv.kv_lens[t] <= 1;
   for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
     float x[V], g[V];
+    if (V == 4 && taps == 4) {                         // all loads first
+      float w[4][V], old[3][V];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ldv<V>(cv.c.w + (long long)j * dim + i, w[j]);
+#pragma unroll
+      for (int j = 0; j < 3; ++j) ldv<V>(state + (long long)j * dim + i, old[j]);
+      ldv<V>(row + i, x);
+      ldv<V>(gamma + i, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        x[j] = kept<T>(x[j] * r * g[j]);
+#pragma unroll
+        for (int k = 0; k < 3; ++k) old[k][j] = fresh ? 0.f : old[k][j];
+        float y = fmaf(w[3][j], x[j], x[j]);
+#pragma unroll
+        for (int k = 0; k < 3; ++k) y = fmaf(w[k][j], old[k][j], y);
+        g[j] = y;
+      }
+      stv<V>(h + i, x);
+      stv<V>(out + i, g);
+      stv<V>(state + i, old[1]);
+      stv<V>(state + dim + i, old[2]);
+      stv<V>(state + 2ll * dim + i, x);
+      continue;
+    }
     ldv<V>(row + i, x);
     if (gamma) {
       ldv<V>(gamma + i, g);
@@ -82,19 +128,17 @@ __device__ __forceinline__ void write_normed(const float* row, float ss, const f
       for (int j = 0; j < V; ++j) x[j] *= r * g[j];
     }
     stv<V>(h + i, x);
+    if (taps > 0) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        const float cur = kept<T>(x[j]);
+        stf(out + i + j, cur + conv_step(cv.c, state, fresh, i + j, cur));
+      }
+    }
   }
   for (int i = dim + threadIdx.x; i < ldh; i += SN_THREADS) stf(h + i, 0.f);
-  if (cv.c.taps > 0) {
-    __syncthreads();                                   // h is complete; the convolution reads what the activation type keeps of it
-    T* out = static_cast<T*>(cv.out) + t * cv.ld;
-    float* state = cv.c.state ? cv.c.state + (long long)cv.slots[t] * (cv.c.taps - 1) * dim : nullptr;
-    const bool fresh = cv.kv_lens[t] <= 1;
-    for (int i = threadIdx.x; i < dim; i += SN_THREADS) {
-      const float cur = ldf(h + i);
-      stf(out + i, cur + conv_step(cv.c, state, fresh, i, cur));
-    }
+  if (taps > 0)
     for (int i = dim + threadIdx.x; i < cv.ld; i += SN_THREADS) stf(out + i, 0.f);
-  }
 }
 
 template <typename T, int V>
@@ -106,6 +150,7 @@ embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ pos, 
   extern __shared__ __align__(16) float row[];
   __shared__ float scratch[32];
   const long long t = blockIdx.x;
+  prefetch_tail(cv, dim, t);
   int id = ids[t];
   id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
   int p = pos[t];
@@ -154,6 +199,7 @@ residual_norm_kernel(const T* __restrict__ y, long long ldy, const float* __rest
   extern __shared__ __align__(16) float row[];
   __shared__ float scratch[32];
   const long long t = blockIdx.x;
+  prefetch_tail(cv, dim, t);
   float sx = 0.f;
   for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
     float a[V], b[V], xv[V];
@@ -176,83 +222,113 @@ residual_norm_kernel(const T* __restrict__ y, long long ldy, const float* __rest
   write_normed<T, V>(row, sx, w_next, h + t * ldh, ldh, dim, eps, cv, t);
 }
 
-// One block per row. NV > 0: vectors of V values a thread keeps in registers; 0: any width, the row is read twice.
-template <typename T, int V, int NV>
-__global__ void __launch_bounds__(512)
-poly_norm_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ bias, const float* __restrict__ abce,
-                 T* __restrict__ out, long long ldo, int width, int padded, float eps) {
-  __shared__ float part[3][16];
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, step = blockDim.x * V;
-  y += blockIdx.x * ldy;
-  out += blockIdx.x * ldo;
-  float s1 = 0.f, s2 = 0.f, s3 = 0.f;
-  auto load = [&](int i, float (&z)[V]) {
-    load_v<V>(y + i, z);
-    if (bias) {
-      float b[V];
-      if constexpr (V == 8) {
-        float lo[4], hi[4];
-        load_v<4>(bias + i, lo);
-        load_v<4>(bias + i + 4, hi);
+template <int V>
+__device__ __forceinline__ void load_bias(const float* bias, int i, float (&b)[V]) {
+  if constexpr (V == 8) {
+    float lo[4], hi[4];
+    load_v<4>(bias + i, lo);
+    load_v<4>(bias + i + 4, hi);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) { b[j] = lo[j]; b[4 + j] = hi[j]; }
-      } else {
-        load_v<V>(bias + i, b);
-      }
-#pragma unroll
-      for (int j = 0; j < V; ++j) z[j] += b[j];
-    }
-#pragma unroll
-    for (int j = 0; j < V; ++j) {
-      const float q = z[j] * z[j], q2 = q * q;
-      s1 += q;
-      s2 += q2;
-      s3 = fmaf(q2, q, s3);
-    }
-  };
-  float keep[NV > 0 ? NV : 1][V];
-  if constexpr (NV > 0) {
-#pragma unroll
-    for (int k = 0; k < NV; ++k) {
-      const int i = threadIdx.x * V + k * step;
-      if (i < width) load(i, keep[k]);
-    }
+    for (int j = 0; j < 4; ++j) { b[j] = lo[j]; b[4 + j] = hi[j]; }
   } else {
-    for (int i = threadIdx.x * V; i < width; i += step) load(i, keep[0]);
+    load_v<V>(bias + i, b);
   }
-  s1 = warp_sum(s1);
-  s2 = warp_sum(s2);
-  s3 = warp_sum(s3);
+}
+template <int V>
+__device__ __forceinline__ void add_powers(const float (&z)[V], float3& s) {
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    const float q = z[j] * z[j], q2 = q * q;
+    s.x += q;
+    s.y += q2;
+    s.z = fmaf(q2, q, s.z);
+  }
+}
+// Factors of z, z^2 and z^3 from a block's sums of squares.
+__device__ __forceinline__ float3 power_factors(float3 s, float (*part)[16], const float4& abce, float width, float eps) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  s = make_float3(warp_sum(s.x), warp_sum(s.y), warp_sum(s.z));
   if (lane == 0) {
-    part[0][warp] = s1;
-    part[1][warp] = s2;
-    part[2][warp] = s3;
+    part[0][warp] = s.x;
+    part[1][warp] = s.y;
+    part[2][warp] = s.z;
   }
   __syncthreads();
-  s1 = warp_sum(lane < nw ? part[0][lane] : 0.f);
-  s2 = warp_sum(lane < nw ? part[1][lane] : 0.f);
-  s3 = warp_sum(lane < nw ? part[2][lane] : 0.f);
-  const float n = (float)width, e = abce[3];
-  const float a = abce[0] / sqrtf(s1 / n + eps), b = abce[1] / sqrtf(s2 / n + eps), c = abce[2] / sqrtf(s3 / n + eps);
-  auto store = [&](int i, float (&z)[V]) {
+  s.x = warp_sum(lane < nw ? part[0][lane] : 0.f);
+  s.y = warp_sum(lane < nw ? part[1][lane] : 0.f);
+  s.z = warp_sum(lane < nw ? part[2][lane] : 0.f);
+  return make_float3(abce.x / sqrtf(s.x / width + eps), abce.y / sqrtf(s.y / width + eps), abce.z / sqrtf(s.z / width + eps));
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_poly(T* out, float (&z)[V], const float3& f, float e) {
 #pragma unroll
-    for (int j = 0; j < V; ++j) z[j] = fmaf(fmaf(fmaf(c, z[j], b), z[j], a), z[j], e);
-    if constexpr (V == 8) *reinterpret_cast<bf16x8*>(out + i) = pack8(z);
-    else stv<V>(out + i, z);
-  };
-  if constexpr (NV > 0) {
+  for (int j = 0; j < V; ++j) z[j] = fmaf(fmaf(fmaf(f.z, z[j], f.y), z[j], f.x), z[j], e);
+  if constexpr (V == 8) *reinterpret_cast<bf16x8*>(out) = pack8(z);
+  else stv<V>(out, z);
+}
+
+// One block per row; a thread holds NV vectors of V values (16 bytes).
+template <typename T, int V, int NV>
+__global__ void __launch_bounds__(512)
+poly_norm_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ bias, const float* __restrict__ abce_p,
+                 T* __restrict__ out, long long ldo, int width, int padded, float eps) {
+  __shared__ float part[3][16];
+  const int step = blockDim.x * V, c = threadIdx.x * V;
+  y += blockIdx.x * ldy;
+  out += blockIdx.x * ldo;
+  uint4 raw[NV];
 #pragma unroll
-    for (int k = 0; k < NV; ++k) {
-      const int i = threadIdx.x * V + k * step;
-      if (i < width) store(i, keep[k]);
+  for (int k = 0; k < NV; ++k)
+    if (c + k * step < width) raw[k] = *reinterpret_cast<const uint4*>(y + c + k * step);
+  const float4 abce = make_float4(abce_p[0], abce_p[1], abce_p[2], abce_p[3]);
+  float z[NV][V];
+  float3 s = make_float3(0.f, 0.f, 0.f);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = c + k * step;
+    if (i >= width) continue;
+    load_v<V>(reinterpret_cast<const T*>(&raw[k]), z[k]);
+    if (bias) {
+      float b[V];
+      load_bias<V>(bias, i, b);
+#pragma unroll
+      for (int j = 0; j < V; ++j) z[k][j] += b[j];
     }
-  } else {
-    for (int i = threadIdx.x * V; i < width; i += step) {
-      load(i, keep[0]);
-      store(i, keep[0]);
-    }
+    add_powers<V>(z[k], s);
+  }
+  const float3 f = power_factors(s, part, abce, (float)width, eps);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = c + k * step;
+    if (i < width) store_poly<T, V>(out + i, z[k], f, abce.w);
   }
   for (int i = width + threadIdx.x; i < padded; i += blockDim.x) stf(out + i, 0.f);
+}
+
+// Any width and alignment, one block per row, the row is read twice.
+template <typename T>
+__global__ void __launch_bounds__(256)
+poly_norm_any_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ bias, const float* __restrict__ abce_p,
+                     T* __restrict__ out, long long ldo, int width, int padded, float eps) {
+  __shared__ float part[3][16];
+  const float4 abce = make_float4(abce_p[0], abce_p[1], abce_p[2], abce_p[3]);
+  y += blockIdx.x * ldy;
+  out += blockIdx.x * ldo;
+  float3 s = make_float3(0.f, 0.f, 0.f);
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float z[1] = {ldf(y + i) + (bias ? bias[i] : 0.f)};
+    add_powers<1>(z, s);
+  }
+  const float3 f = power_factors(s, part, abce, (float)width, eps);
+  for (int i = threadIdx.x; i < padded; i += blockDim.x) {
+    float z[1] = {0.f};
+    if (i < width) {
+      z[0] = ldf(y + i) + (bias ? bias[i] : 0.f);
+      store_poly<T, 1>(out + i, z, f, abce.w);
+    } else {
+      stf(out + i, 0.f);
+    }
+  }
 }
 
 enum { SUB_ONE, SUB_TWO, SUB_EXPERTS };
@@ -731,6 +807,8 @@ void check_tail(const ConvTail& conv, int dim) {
   if (conv.c.taps == 0) return;
   MB_REQUIRE(conv.c.channels == dim && conv.ld >= dim && conv.out && conv.c.w && conv.slots && conv.kv_lens &&
                  (conv.c.taps == 1 || conv.c.state) && !conv.c.bias, "convolution tail: arguments");
+  MB_REQUIRE(((reinterpret_cast<uintptr_t>(conv.c.w) | reinterpret_cast<uintptr_t>(conv.c.state) | reinterpret_cast<uintptr_t>(conv.out)) & 15) == 0 &&
+                 (dim % 4 != 0 || conv.ld % 4 == 0), "convolution tail: alignment");
 }
 template <typename T, int V>
 void sandwich_launch(const SublayerOut& y, const float* w_post, float mult, float* x, const float* w_next, void* h,
@@ -797,15 +875,26 @@ void poly_norm(bool f32, const void* y, long long ldy, const float* bias, const 
   const int V = f32 ? 4 : 8;
   const bool vec = width % V == 0 && ldy % V == 0 && ldo % V == 0 &&
                    ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(bias)) & 15) == 0;
-  const int units = vec ? width / V : width, threads = units <= 64 ? 64 : (units <= 1024 ? 256 : 512);
-  const int nv = (units + threads - 1) / threads;
-#define MB_PN(T, V, NV) poly_norm_kernel<T, V, NV><<<rows, threads, 0, stream>>>((const T*)y, ldy, bias, abce, (T*)out, ldo, width, padded, eps)
-#define MB_PNV(T, V) \
-  do { if (nv <= 1) MB_PN(T, V, 1); else if (nv <= 2) MB_PN(T, V, 2); else if (nv <= 4) MB_PN(T, V, 4); else MB_PN(T, V, 0); } while (0)
-  if (f32) { if (vec) MB_PNV(float, 4); else MB_PN(float, 1, 0); }
-  else     { if (vec) MB_PNV(__nv_bfloat16, 8); else MB_PN(__nv_bfloat16, 1, 0); }
+  const int units = width / V;
+  if (!vec || units > 4096) {
+    if (f32) poly_norm_any_kernel<float><<<rows, 256, 0, stream>>>((const float*)y, ldy, bias, abce, (float*)out, ldo, width, padded, eps);
+    else
+      poly_norm_any_kernel<__nv_bfloat16><<<rows, 256, 0, stream>>>((const __nv_bfloat16*)y, ldy, bias, abce, (__nv_bfloat16*)out, ldo,
+                                                                    width, padded, eps);
+  } else {
+    const int nv = units <= 384 ? 1 : (units <= 768 ? 2 : (units <= 1152 ? 3 : (units <= 1536 ? 4 : (units <= 2304 ? 6 : 8))));
+    const int threads = ((units + nv - 1) / nv + 31) / 32 * 32;
+#define MB_PN(T, V, NV) \
+  poly_norm_kernel<T, V, NV><<<rows, threads, 0, stream>>>((const T*)y, ldy, bias, abce, (T*)out, ldo, width, padded, eps)
+#define MB_PNV(T, V)                                                                                               \
+  do {                                                                                                             \
+    if (nv == 1) MB_PN(T, V, 1); else if (nv == 2) MB_PN(T, V, 2); else if (nv == 3) MB_PN(T, V, 3);               \
+    else if (nv == 4) MB_PN(T, V, 4); else if (nv == 6) MB_PN(T, V, 6); else MB_PN(T, V, 8);                       \
+  } while (0)
+    if (f32) MB_PNV(float, 4); else MB_PNV(__nv_bfloat16, 8);
 #undef MB_PNV
 #undef MB_PN
+  }
   count_launch();
   check_launch();
 }

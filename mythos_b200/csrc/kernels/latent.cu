@@ -52,28 +52,67 @@ struct Vec16 {
 // Normalises `width` columns of a row by a warp (zeros up to padded): out = x / rms * gamma.
 template <typename T>
 __device__ __forceinline__ void lp_norm(const T* src, T* dst, int width, int padded, const float* gamma, float eps, int lane) {
-  constexpr int N = Vec16<T>::N;
+  constexpr int N = Vec16<T>::N, KEEP = 4;       // vectors that stay in registers
+  uint4 raw[KEEP];
   float ss = 0.f;
-  for (int i = lane * N; i < padded; i += 32 * N) {
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = (lane + 32 * k) * N;
+    if (i < padded) raw[k] = *reinterpret_cast<const uint4*>(src + i);
+  }
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = (lane + 32 * k) * N;
+    if (i < padded) {
+      Vec16<T> x;
+      x.load(reinterpret_cast<const T*>(&raw[k]));
+#pragma unroll
+      for (int j = 0; j < N; ++j) ss = fmaf(x.v[j], x.v[j], ss);
+    }
+  }
+  for (int i = (lane + 32 * KEEP) * N; i < padded; i += 32 * N) {
     Vec16<T> x;
     x.load(src + i);
 #pragma unroll
     for (int j = 0; j < N; ++j) ss = fmaf(x.v[j], x.v[j], ss);
   }
   const float r = 1.f / sqrtf(warp_sum(ss) / (float)width + eps);
-  for (int i = lane * N; i < padded; i += 32 * N) {
+  auto put = [&](Vec16<T>& x, int i) {
+    if (i + N <= width) {
+#pragma unroll
+      for (int j = 0; j < N; j += 4) {
+        const float4 g = *reinterpret_cast<const float4*>(gamma + i + j);
+        x.v[j] *= r * g.x;
+        x.v[j + 1] *= r * g.y;
+        x.v[j + 2] *= r * g.z;
+        x.v[j + 3] *= r * g.w;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < N; ++j) x.v[j] *= i + j < width ? r * gamma[i + j] : 0.f;
+    }
+    x.store(dst + i);
+  };
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = (lane + 32 * k) * N;
+    if (i < padded) {
+      Vec16<T> x;
+      x.load(reinterpret_cast<const T*>(&raw[k]));
+      put(x, i);
+    }
+  }
+  for (int i = (lane + 32 * KEEP) * N; i < padded; i += 32 * N) {
     Vec16<T> x;
     x.load(src + i);
-#pragma unroll
-    for (int j = 0; j < N; ++j) x.v[j] *= i + j < width ? r * gamma[i + j] : 0.f;
-    x.store(dst + i);
+    put(x, i);
   }
 }
 
 // One warp per token. Angles: position x revolutions, reduced to a fraction of a turn in double precision. Padded
-// columns of the projection are zero, and so are those of a page row.
+// columns of the projection are zero, and so are those of a page row. ROWS: norms and page rows (else queries only).
 constexpr int LP_WARPS = 4;
-template <typename T>
+template <typename T, bool ROWS>
 __global__ void __launch_bounds__(LP_WARPS * 32)
 latent_prep_kernel(T* __restrict__ proj, long long ld, LatentPrep p, LatentSpec s, RaggedBatch rb, LatentPages pg, float eps) {
   constexpr int N = Vec16<T>::N;
@@ -84,8 +123,10 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, LatentPrep p, LatentSpec 
   float2* cs = cs_all + warp * (s.rot_p / 2);
   const int pos = rb.pos[t];
   T* row = proj + (long long)t * ld;
-  if (p.low_off >= 0) lp_norm(row + p.low_off, row + p.low_off, p.low_rank, (p.low_rank + 7) / 8 * 8, p.low_gamma, eps, lane);
-  if (p.qr_off < 0 && p.c_off < 0) return;
+  if constexpr (ROWS) {
+    if (p.low_off >= 0) lp_norm(row + p.low_off, row + p.low_off, p.low_rank, (p.low_rank + 7) / 8 * 8, p.low_gamma, eps, lane);
+    if (p.qr_off < 0 && p.c_off < 0) return;
+  }
   for (int i = lane; i < s.rot_p / 2; i += 32) {
     float sn = 0.f, co = 1.f;
     if (i < s.rot / 2) {
@@ -95,7 +136,7 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, LatentPrep p, LatentSpec 
     cs[i] = make_float2(s.rot_amp * co, s.rot_amp * sn);
   }
   __syncwarp();                              // cs is complete
-  if (p.c_off >= 0) {
+  if (ROWS && p.c_off >= 0) {
     const int page = pg.table[(long long)rb.row_seq[t] * pg.stride + pos / pg.page_size];
     if (page >= 0) {
       T* dst = static_cast<T*>(pg.cache) + ((long long)page * pg.page_size + pos % pg.page_size) * s.row();
@@ -110,6 +151,7 @@ latent_prep_kernel(T* __restrict__ proj, long long ld, LatentPrep p, LatentSpec 
   }
   if (p.qr_off < 0) return;
   const int per = s.rot_p / N;               // vectors per head
+#pragma unroll 4
   for (int j = lane; j < s.heads * per; j += 32) {
     Vec16<T> x;
     T* q = row + p.qr_off + j * N;
@@ -486,13 +528,15 @@ void latent_prep(bool f32, void* proj, long long ld, const LatentPrep& p, const 
   MB_REQUIRE(s.rot > 0 && s.rot % 2 == 0 && s.rot <= 2048, "latent_prep: rotated width");
   for (int off : {p.low_off, p.qr_off, p.c_off, p.kr_off}) MB_REQUIRE(off < 0 || off % 8 == 0, "latent_prep: columns in units of 8");
   MB_REQUIRE(ld % 8 == 0 && (p.c_off < 0 || (p.kr_off >= 0 && p.gamma)) && (p.low_off < 0 || (p.low_gamma && p.low_rank > 0)) &&
-                 (reinterpret_cast<uintptr_t>(proj) & 15) == 0, "latent_prep: arguments");
+                 ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(p.gamma) | reinterpret_cast<uintptr_t>(p.low_gamma)) & 15) == 0,
+             "latent_prep: arguments");
   if (rb.rows == 0) return;
   const int smem = LP_WARPS * (s.rot_p / 2) * (int)sizeof(float2), grid = (rb.rows + LP_WARPS - 1) / LP_WARPS;
-  if (f32)
-    latent_prep_kernel<float><<<grid, LP_WARPS * 32, smem, stream>>>((float*)proj, ld, p, s, rb, pg, eps);
-  else
-    latent_prep_kernel<__nv_bfloat16><<<grid, LP_WARPS * 32, smem, stream>>>((__nv_bfloat16*)proj, ld, p, s, rb, pg, eps);
+  const bool rows = p.low_off >= 0 || p.c_off >= 0;
+#define MB_LP(T, ROWS) latent_prep_kernel<T, ROWS><<<grid, LP_WARPS * 32, smem, stream>>>((T*)proj, ld, p, s, rb, pg, eps)
+  if (f32) { if (rows) MB_LP(float, true); else MB_LP(float, false); }
+  else     { if (rows) MB_LP(__nv_bfloat16, true); else MB_LP(__nv_bfloat16, false); }
+#undef MB_LP
   count_launch();
   check_launch();
 }

@@ -111,6 +111,7 @@ DECODE_GEMM_ROWS = 128     # up to this many tokens a product goes through the f
 EXPAND_TOKENS = 16         # portions of at least this many tokens expand the latents of their sequence
 EXPAND_BYTES = 4 << 30     # unless the expanded keys and values would need more than this
 SEGMENT_GEMM_ROWS = 48     # mean rows per expert from which the prompt-sized grouped GEMM runs
+SIDE_STREAM_ROWS = 128     # up to this many tokens a parallel design's mixer and feed-forward run on two streams
 LOW_RANK_FUSE_ROWS = 16    # decode batches up to this size evaluate the low-rank maps inside the recurrence kernel
 STEP_FUSE_ROWS = 4         # the same for the step sizes of a selective scan, whose map every token reads again
 
@@ -157,6 +158,7 @@ class HybridEngine(InferenceEngine):
         self._sms = torch.cuda.get_device_properties(self.device).multi_processor_count if self.device.type == "cuda" else 1
         self.H = native.require_hybrid() if self.device.type == "cuda" else None
         self._status = native.status_word(self.device)
+        self._side = torch.cuda.Stream(self.device) if cfg.parallel and self.device.type == "cuda" else None
         groups = max([m.kv_heads * ((m.heads // m.kv_heads + 7) // 8) for m in att] or [1])
         self._counters = torch.zeros(max_batch * groups, device=self.device, dtype=torch.int32)
         experts = max([s.mlp.experts for s in cfg.layers if isinstance(s.mlp, MoeFF)] or [0])
@@ -694,22 +696,31 @@ class HybridEngine(InferenceEngine):
             self.H.gate_pair(gu, f, L.gate_up.off["up"], L.act, a)
         return self._gemm(a, L.down, out)
 
-    def _poly(self, L, h, out):
-        """Ungated feed-forward up to its down matrix."""
-        self.H.poly_norm(self._gemm(h, L.up), L.up_bias, L.poly, L.spec.mlp.ff, out, self.cfg.norm_eps)
+    def _ff_columns(self, L, h, out):
+        """Feed-forward up to its down matrix."""
+        if L.up is not None:
+            self.H.poly_norm(self._gemm(h, L.up), L.up_bias, L.poly, L.spec.mlp.ff, out, self.cfg.norm_eps)
+        elif L.gate_up is not None:
+            gu, a = self._gemm(h, L.gate_up.weight), self._new(*out.shape)
+            self.H.gate_pair(gu, L.spec.mlp.ff, L.gate_up.off["up"], L.act, a)
+            out.copy_(a)
 
     def _side_by_side(self, L, h, ctx):
-        """Mixer and feed-forward of a parallel design -> their sum."""
+        """Mixer and feed-forward of a parallel design -> their sum. Few tokens leave most of the GPU idle: the two run
+        on streams of their own."""
         y = self._new(ctx.rows, L.out.shape[1])
         n = L.mixer_cols
-        L.heads_of(L, ctx.conv if L.conv is not None else h, ctx, y[:, :n])
-        if L.up is not None:
-            self._poly(L, h, y[:, n:])
-        elif L.gate_up is not None:
-            gu = self._gemm(h, L.gate_up.weight)
-            a = self._new(ctx.rows, L.out.shape[1] - n)
-            self.H.gate_pair(gu, L.spec.mlp.ff, L.gate_up.off["up"], L.act, a)
-            y[:, n:].copy_(a)
+        mixer_in = ctx.conv if L.conv is not None else h
+        if ctx.rows <= SIDE_STREAM_ROWS and L.spec.mlp is not None:
+            main = torch.cuda.current_stream(self.device)
+            self._side.wait_stream(main)
+            with torch.cuda.stream(self._side):
+                self._ff_columns(L, h, y[:, n:])
+            L.heads_of(L, mixer_in, ctx, y[:, :n])
+            main.wait_stream(self._side)
+        else:
+            L.heads_of(L, mixer_in, ctx, y[:, :n])
+            self._ff_columns(L, h, y[:, n:])
         return self._gemm(y, L.out)
 
     def _feed_forward(self, L, h, ctx):

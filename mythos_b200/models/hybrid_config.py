@@ -616,7 +616,7 @@ def zigivik_config(width: int = 2048, layers: int = 8, vocab: int = 32000, max_p
                 rotation=Rotation(500000.0, 128, layout="pairs"), sink="zero"), ff))
         else:
             out.append(LayerSpec("latent_attention", LatentAttentionMixer(
-                h, 128, 64, 128, 512, 192 ** -0.5, rot, q_rank=width * 3 // 8 // 128 * 128, window=window, sink=None, gate=True,
+                h, 128, 64, 128, 512, 192 ** -0.5, rot, q_rank=max(128, width * 3 // 8 // 128 * 128), window=window, sink=None, gate=True,
                 kv_from=i - 1 if i % 4 == 1 else None), ff))
     return HybridConfig(vocab, width, out, 1e-6, max_seq_len=max_positions, architecture="Zigivik", position_table=False,
                         post_norm=False, parallel=True, scalar_norms=True, embed_norm=True, input_conv=4, residual_mult=0.7)

@@ -1,4 +1,4 @@
-"""Speed of layer-list models (Teganex, Lebedra or Dogozen layers at the sizes of a real model, random weights) beside
+"""Speed of layer-list models (Teganex, Lebedra, Dogozen or Zigivik layers at the sizes of a real model, random weights) beside
 the dense transformer engine of equal width, depth and feed-forward (Lebedra, Dogozen: the dense layers', and the
 experts of a token together about as wide), both with bf16 weights.
 
@@ -31,7 +31,7 @@ def _engines(design, width, layers, vocab, batch, max_len):
     from ..models import hybrid_config as hc
 
     kw = dict(seed=1, device="cuda", max_batch=batch, max_seq_len=max_len)
-    make = {"teganex": hc.teganex_config, "lebedra": hc.lebedra_config, "dogozen": hc.dogozen_config}[design]
+    make = {"teganex": hc.teganex_config, "lebedra": hc.lebedra_config, "dogozen": hc.dogozen_config, "zigivik": hc.zigivik_config}[design]
     yield design, HybridEngine.random(make(width, layers, vocab, max_len), **kw)
     yield "dense", InferenceEngine.random(_dense_config(width, layers, vocab, max_len), **kw)
 
@@ -167,7 +167,7 @@ def _dense_attention_rows(K, H, C, st, rnd, h, kv):
           lambda: C.flash_attn_paged_prefill(q, kc, vc, table, b[0], b[1], o, S, 128 ** -0.5, st),
           flops=2.0 * B * h * (S * (S + 1) / 2) * 256)
     sms = torch.cuda.get_device_properties(0).multi_processor_count
-    for NB, ctx in ((16, 4096), (64, 1024), (16, 1024)):
+    for NB, ctx in ((16, 4096), (64, 1024), (16, 1024), (1, 1024)):
         pages = NB * ctx // PAGE
         table = torch.randperm(pages, device="cuda").to(torch.int32).view(NB, -1)
         kc, vc, q, o = rnd(pages, PAGE, kv, 128), rnd(pages, PAGE, kv, 128), rnd(NB, h, 128), rnd(NB, h, 128)
@@ -226,6 +226,122 @@ def _expert_rows(K, H, C, rnd, eng, L, T):
     return hid, hh
 
 
+def _visible(S, w):
+    """Query-key pairs of a sequence of S tokens."""
+    return S * (S + 1) / 2 if not w or w >= S else w * (w + 1) / 2 + (S - w) * w
+
+
+def run_zigivik_kernels(peaks: dict, width: int = 2048) -> list[dict]:
+    """Window attention over latents, attention whose values are its keys, input convolution, PolyNorm and the stream."""
+    from ..infer.hybrid import HybridEngine
+    from ..models.hybrid_config import zigivik_config
+    from ..ops import functional as F, native
+
+    H, C, st = native.require_hybrid(), native.require(), native.status_word("cuda")
+    K, bf, d = _Kernels(peaks), torch.bfloat16, width
+    rnd = lambda *s: torch.randn(*s, device="cuda").to(bf)
+    cfg = zigivik_config(width, 4, 32000)
+    eng = HybridEngine.random(cfg, device="cuda", max_batch=64, max_seq_len=4096, kv_pages=64)
+    L, full = eng.layers[0], eng.layers[3]
+    m, a, ff, eps = L.spec.mixer, full.spec.mixer, L.spec.mlp.ff, cfg.norm_eps
+    h, kv, r, W, win = m.heads, a.kv_heads, m.kv_rank, m.kv_rank + m.rot_dim, m.window
+    dn, dv = m.dim, m.vdim
+    _dense_attention_rows(K, H, C, st, rnd, h, kv)
+    # ---- stream, convolution, PolyNorm
+    for T in (1, 16, 64, 8192):
+        b = _batch([1] * T, [99] * T) if T <= 64 else _batch([2048] * 4, [0] * 4)
+        y, g, x = rnd(T, d), rnd(T, d), torch.randn(T, d, device="cuda")
+        hid, bias, one = rnd(T, d), torch.zeros(d, device="cuda"), torch.ones(d, device="cuda")
+        tail = (L.conv, b, g) if T <= 64 else None
+        K.add("residual_norm" + (" + convolution" if tail else ""), f"{T} x {d}",
+              lambda: H.residual_norm(y, bias, 0.7, x, one, hid, eps, tail), nbytes=T * d * (12.0 + (26 if tail else 0)),
+              like="rmsnorm + residual (dense)")
+        w16, res = torch.ones(d, device="cuda", dtype=bf), rnd(T, d)
+        K.add("rmsnorm + residual (dense)", f"{T} x {d}", lambda: F.rmsnorm(hid, w16, 1e-6, res), nbytes=T * d * 8.0)
+        if T > 64:
+            K.add("input convolution", f"{T} x {d}", lambda: L.conv.run(hid, 0, b, False, g), nbytes=T * d * 4.0, like="rope (dense)")
+        z, out = rnd(T, ff), rnd(T, L.out.shape[1])[:, L.mixer_cols:]
+        K.add("poly_norm", f"{T} x {ff}", lambda: H.poly_norm(z, L.up_bias, L.poly, ff, out, eps), nbytes=T * ff * 4.0,
+              like="rmsnorm + residual (dense)")
+    # ---- attention whose values are its keys
+    def pages(B, S):
+        n = B * S // PAGE
+        return torch.randperm(n, device="cuda").to(torch.int32).view(B, -1), rnd(n, PAGE, kv, 128), rnd(n, PAGE, kv, 128)
+
+    for B, S in ((4, 2048), (1, 8192)):
+        (table, kc, vc), b, n = pages(B, S), _batch([S] * B, [0] * B), B * S
+        q, o, proj = rnd(n, h, 128), torch.empty(n, h * 128, device="cuda", dtype=bf), rnd(n, full.proj.N)
+        K.add("attn_prep, pairs, keys as values", f"{n} tokens, {h}/{kv} heads, 128", lambda: full.att.prep(proj, b, table, q, kc, vc),
+              nbytes=n * 128 * (4.0 * h + 6 * kv), like="rope (dense)")
+        K.add("paged prefill attention, one in the denominator", f"{B} x {S}, {h}/{kv} heads, 128",
+              lambda: full.att.prefill(q, kc, vc, b, table, None, o, S, st), flops=2.0 * B * h * _visible(S, 0) * 256,
+              like="paged prefill attention (dense)")
+    qkv, pos = rnd(8192, h + 2 * kv, 128), torch.arange(2048, device="cuda", dtype=torch.int32).repeat(4)
+    K.add("rope (dense)", f"8192 tokens, {h}/{kv} heads, 128", lambda: C.rope(qkv[:, : h + kv], pos, 10000.0, False),
+          nbytes=4.0 * 8192 * (h + kv) * 128)
+    sms = torch.cuda.get_device_properties(0).multi_processor_count
+    for NB, ctx in ((16, 4096), (64, 1024)):
+        (table, kc, vc), b = pages(NB, ctx), _batch([1] * NB, [ctx - 1] * NB)
+        q, o = rnd(NB, h, 128), torch.empty(NB, h * 128, device="cuda", dtype=bf)
+        splits = max(1, min(32, (6 * sms + NB * kv - 1) // (NB * kv), (ctx + 255) // 256))
+        scratch = torch.empty(full.att.decode_scratch(NB, splits), device="cuda")
+        K.add("paged decode attention, one in the denominator", f"{NB} x {ctx}, {h}/{kv} heads, 128",
+              lambda: full.att.decode(q, kc, vc, b, table, None, o, scratch, eng._counters, splits, st), nbytes=4.0 * NB * ctx * kv * 128,
+              like="paged decode attention (dense)")
+    # ---- window attention over latents
+    def latents(B, S):
+        return torch.randperm(B * S // PAGE, device="cuda").to(torch.int32).view(B, -1), rnd(B * S // PAGE, PAGE, 1, W)
+
+    for B, S, past in ((4, 2048, 0), (1, 8192, 0), (4, 2048, 2048)):
+        table, cache = latents(B, S + past)
+        b, n, held = _batch([S] * B, [past] * B), B * S, S + min(past, win - 1)
+        i32 = dict(device="cuda", dtype=torch.int32)
+        cu = torch.arange(B + 1, **i32) * held
+        first, keys = torch.full((B,), S + past - held, **i32), torch.full((B,), held, **i32)
+        proj, qs, o = rnd(n, L.proj.N), rnd(n, L.low.N), torch.empty(n, h, dv, device="cuda", dtype=bf)
+        lat, ex = torch.empty(B * held, W, device="cuda", dtype=bf), rnd(B * held, h * (dn + dv))
+        q, k, v = qs[:, : h * dn].unflatten(1, (h, dn)), ex[:, : h * dn].unflatten(1, (h, dn)), ex[:, h * dn:].unflatten(1, (h, dv))
+        gate, sizes = proj[:, L.proj.off["g"]:][:, : h * dv], f"{B} x {S}" + (f" behind {past}" if past else "")
+        K.add("latent_prep, latents", sizes, lambda: L.lat.prep(proj, b, table, cache, queries=False),
+              nbytes=4.0 * n * (W + m.q_rank), like="rope (dense)")
+        K.add("latent_prep, queries", sizes, lambda: L.lat.prep(qs, b, table, cache, latents=False), nbytes=4.0 * n * h * m.rot_dim,
+              like="rope (dense)")
+        K.add("latent_gather", sizes, lambda: L.lat.gather(table, cache, cu, first, held, lat), nbytes=4.0 * B * held * W, like="rope (dense)")
+        K.add(f"latent prefill attention, window {win}, gated", f"{sizes}, {h} heads, {dn} + {m.rot_dim} / {dv}",
+              lambda: L.lat.attn_prefill(q, qs, k, v, lat, b, cu, keys, S, 16, gate, o, st),
+              flops=2.0 * B * h * (_visible(S + past, win) - _visible(past, win)) * (dn + m.rot_dim + dv),
+              nbytes=2.0 * n * h * (dn + m.rot_dim + 2 * dv), like="paged prefill attention (dense)")
+    for NB, ctx in ((1, 4096), (16, 4096), (64, 4096)):
+        table, cache = latents(NB, ctx)
+        b, proj, qs = _batch([1] * NB, [ctx - 1] * NB), rnd(NB, L.proj.N), rnd(NB, L.low.N)
+        ql, ol, out = rnd(NB, h, r), rnd(NB, h, r), rnd(NB, h, dv)
+        q, gate = qs[:, : h * dn].unflatten(1, (h, dn)), proj[:, L.proj.off["g"]:][:, : h * dv]
+        K.add("W_uk per head", f"{NB} tokens, {h} heads", lambda: H.gemm_heads(q, L.uk_t, ql, st),
+              nbytes=2.0 * (L.uk_t.numel() + NB * h * (dn + r)), like="gemm_decode")
+        splits = eng._latent_splits(NB, h, min(ctx, win + 64))
+        sc = torch.empty(NB * h * splits * (r + 4), device="cuda")
+        K.add(f"latent decode attention, window {win}", f"{NB} x {ctx}, {h} heads", lambda: L.lat.attn_decode(
+            ql, qs, b[3], b[4], table, cache, ol, sc, splits, st),
+            nbytes=2.0 * NB * (min(ctx, win) * W + h * (W + r)), flops=2.0 * NB * h * min(ctx, win) * (W + r),
+            like=f"paged decode attention (dense), {NB} x {win}")
+        K.add("W_uv per head, gated", f"{NB} tokens, {h} heads", lambda: H.gemm_heads(ol, L.uv, out, st, gate),
+              nbytes=2.0 * (L.uv.numel() + NB * h * (2 * dv + r)), like="gemm_decode")
+        x, w, y = rnd(NB, dn * 4), rnd(h * r // 4, dn * 4), rnd(NB, h * r // 4)
+        K.add("gemm_decode", f"{NB} x {h * r // 4} x {dn * 4}", lambda: H.gemm_decode(x, w, y, 0, 0, 1.0, st),
+              nbytes=2.0 * (w.numel() + x.numel() + y.numel()))
+    # ---- products
+    for T in (1, 16, 64, 8192):
+        for name, ww in (("latent layer in", L.proj.weight), ("low-rank queries", L.low.weight), ("attention in", full.proj.weight),
+                         ("feed-forward up", L.up), ("mixer and feed-forward out", L.out)):
+            n_out, k_in = ww.shape
+            xx, oo, sizes = rnd(T, k_in), torch.empty(T, n_out, device="cuda", dtype=bf), f"{T} x {n_out} x {k_in}"
+            work = dict(nbytes=2.0 * (n_out * k_in + T * (k_in + n_out)), flops=2.0 * T * n_out * k_in)
+            K.add(f"{name} (GEMM)", sizes, lambda: eng._gemm(xx, ww, out=oo), like="gemm (dense bf16)", **work)
+            K.add("gemm (dense bf16)", sizes, lambda: F.gemm(xx, ww, out=oo), **work)
+    native.check_status("cuda")
+    return K.rows
+
+
 def run_dogozen_kernels(peaks: dict, width: int = 2048) -> list[dict]:
     """Tempered and window attention (heads of 128), selective scan, routed and shared experts, soft-capped output."""
     from ..infer.hybrid import STEP_FUSE_ROWS, HybridEngine
@@ -242,9 +358,6 @@ def run_dogozen_kernels(peaks: dict, width: int = 2048) -> list[dict]:
     win, sms = par.spec.mixer.left.window, torch.cuda.get_device_properties(0).multi_processor_count
     _dense_attention_rows(K, H, C, st, rnd, h, kv)
 
-    def visible(S, w):                                 # query-key pairs of a sequence
-        return S * (S + 1) / 2 if not w or w >= S else w * (w + 1) / 2 + (S - w) * w
-
     def pages(B, S):
         n = B * S // PAGE
         return torch.randperm(n, device="cuda").to(torch.int32).view(B, -1), rnd(n, PAGE, kv, 128), rnd(n, PAGE, kv, 128)
@@ -260,7 +373,7 @@ def run_dogozen_kernels(peaks: dict, width: int = 2048) -> list[dict]:
             K.add(f"attn_prep, {name}", f"{n} tokens, {h}/{kv} heads, 128", lambda: L.att.prep(proj, b, table, q, kc, vc),
                   nbytes=4.0 * n * (h + 2 * kv) * 128, like="rope (dense)")
             K.add(f"paged prefill attention, {name}", f"{B} x {S}, {h}/{kv} heads, 128",
-                  lambda: L.att.prefill(q, kc, vc, b, table, gate, o, S, st), flops=2.0 * B * h * visible(S, w) * 256,
+                  lambda: L.att.prefill(q, kc, vc, b, table, gate, o, S, st), flops=2.0 * B * h * _visible(S, w) * 256,
                   nbytes=n * (h * 128 * (4.0 + 2 * (gate is not None)) + 512 * kv), like="paged prefill attention (dense)")
     qkv, pos = rnd(8192, h + 2 * kv, 128), torch.arange(2048, device="cuda", dtype=torch.int32).repeat(4)
     K.add("rope (dense)", f"8192 tokens, {h}/{kv} heads, 128", lambda: C.rope(qkv[:, : h + kv], pos, 10000.0, False),
@@ -402,6 +515,8 @@ def run_kernels(peaks: dict, width: int = 2048, design: str = "teganex") -> list
         return run_lebedra_kernels(peaks, width)
     if design == "dogozen":
         return run_dogozen_kernels(peaks, width)
+    if design == "zigivik":
+        return run_zigivik_kernels(peaks, width)
     from ..ops import functional as F, native
 
     H, C, st = native.require_hybrid(), native.require(), native.status_word("cuda")
@@ -490,7 +605,7 @@ def main(argv=None) -> int:
     ap.add_argument("--kernels", action="store_true")
     ap.add_argument("--models", action="store_true")
     ap.add_argument("--width", type=int, default=2048)
-    ap.add_argument("--design", default="teganex", choices=["teganex", "lebedra", "dogozen"])
+    ap.add_argument("--design", default="teganex", choices=["teganex", "lebedra", "dogozen", "zigivik"])
     a = ap.parse_args(argv)
     peaks = {}
     path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")

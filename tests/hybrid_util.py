@@ -82,6 +82,32 @@ def dogozen(width, vocab, layers, cap=20.0, eps=1e-5):
     return {"architecture": "Dogozen", "vocab": vocab, "width": width, "norm": {"eps": eps}, "logit_softcap": cap, "layers": layers}
 
 
+def ramp(base, dims, factor=None, original=64, fast=8.0, slow=1.0):
+    """Rotation with slowed long wavelengths (without, where ``factor`` is None)."""
+    r = {"base": base, "dims": dims}
+    if factor is not None:
+        r["scaling"] = {"factor": factor, "original": float(original), "fast": fast, "slow": slow}
+    return r
+
+
+def window_latent(heads, dim, rot, vdim, rank, q_rank, window, turn=None, scale=None, kv_from=None, ff=0):
+    m = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "q_rank": q_rank, "mask": {"size": window},
+         "rot": turn or ramp(300.0, rot), "scale": (dim + rot) ** -0.5 if scale is None else scale}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": m, "mlp": dense(ff) if ff else None}
+
+
+def key_value(heads, kv, dim, rot, base=400.0, scale=None, ff=0):
+    m = dict(attention(heads, kv, dim, dim, scale), rot={"base": base, "dims": rot})
+    return {"type": "attention", "mixer": m, "mlp": dense(ff) if ff else None}
+
+
+def zigivik(width, vocab, layers, taps, mult, eps=1e-5):
+    return {"architecture": "Zigivik", "vocab": vocab, "width": width, "norm": {"eps": eps}, "residual_mult": mult, "canon": {"taps": taps},
+            "layers": layers}
+
+
 CONFIGS = {
     # unaligned widths everywhere, grouped heads, three taps
     "ragged": config(100, 211, [gla_layer(3, 24, 40, 8.0, ff=52),
@@ -131,10 +157,50 @@ CONFIGS = {
     "scan_plain": dogozen(136, 130, [
         tempered_layer(2, 2, 160, 136, 0.5, 32, mlp=dense(40)),
         scan_layer(window_left(3, 1, 136, 24, 40, 2000), selective(40, 130, 24, 6), (0.9, 1.1), dense(56))], 10.0),
+    # Zigivik: unaligned widths, grouped heads, partial rotation of an odd number of pairs, three taps, a layer without
+    # feed-forward, latents shared with other heads, another window and scale
+    "side_ragged": zigivik(100, 211, [
+        window_latent(3, 20, 6, 36, 44, 28, 19, ramp(300.0, 6, 4.0), ff=52),
+        key_value(6, 2, 20, 10, ff=44),
+        window_latent(5, 12, 6, 20, 44, 21, 33, ramp(300.0, 6, 4.0), 0.35, kv_from=0),
+        key_value(3, 3, 28, 28, scale=0.3)], 3, 0.55),
+    # widths of the tensor-core paths, more than 16 latent heads, more than eight query heads on one key head, a window
+    # longer than a key tile, the sharing layer behind another that has latents of its own
+    "side_wide": zigivik(256, 384, [
+        key_value(12, 1, 128, 128, 1e4, 0.11, ff=512),
+        window_latent(20, 128, 64, 128, 256, 136, 70, ramp(1e4, 64, 8.0, 128, 32.0), ff=256),
+        window_latent(2, 64, 32, 64, 512, 64, 100, ramp(500.0, 32), ff=264),
+        window_latent(4, 72, 64, 104, 256, 80, 64, ramp(1e4, 64, 8.0, 128, 32.0), kv_from=1, ff=328),
+        key_value(4, 4, 64, 48, 1e5, ff=128)], 4, 0.4),
+    # one head, pair, tap, key and rank; whole residuals; every layer narrow
+    "side_single": zigivik(64, 96, [
+        window_latent(1, 16, 2, 16, 8, 1, 1, ramp(100.0, 2, 2.0, 16, 2.0, 1.0), ff=1),
+        key_value(1, 1, 64, 2, 10.0, ff=64),
+        window_latent(1, 8, 8, 8, 16, 64, 16, ff=8)], 1, 1.0, 1e-3),
+    # widths beyond the prompt attention's, latents beyond the decode kernel's, a window longer than the sequences, many taps
+    "side_plain": zigivik(136, 130, [
+        window_latent(2, 160, 72, 136, 40, 136, 2000, ramp(1e4, 72, 16.0, 32, 4.0, 0.5), ff=40),
+        key_value(2, 1, 136, 72, ff=2100),
+        window_latent(3, 16, 4, 24, 520, 30, 40, ff=24)], 6, 0.6),
 }
-TEGANEX = [n for n in CONFIGS if not n.startswith(("latent", "scan"))]
+TEGANEX = [n for n in CONFIGS if not n.startswith(("latent", "scan", "side"))]
 LEBEDRA = [n for n in CONFIGS if n.startswith("latent")]
 DOGOZEN = [n for n in CONFIGS if n.startswith("scan")]
+ZIGIVIK = [n for n in CONFIGS if n.startswith("side")]
+
+
+def _zigivik_weight(name: str, r: torch.Tensor) -> torch.Tensor:
+    """Norm weights away from one, every power of the activation and every bias and tap visible."""
+    leaf = name.rsplit(".", 1)[-1]
+    if leaf == "act":
+        return torch.tensor([0.7, -0.5, 0.4, 0.3]) + 0.1 * r
+    if len(r.shape) == 0 or leaf == "norm":
+        return 1.0 + 0.3 * r
+    if len(r.shape) == 1:
+        return 0.5 * r
+    if leaf == "canon1":
+        return 0.4 * r
+    return r if leaf == "embed" else r * (1.5 / r.shape[1] ** 0.5)
 
 
 def _dogozen_weight(name: str, r: torch.Tensor) -> torch.Tensor:
@@ -166,8 +232,8 @@ def weights(cfg: dict, seed: int = 0, low_rank: int = 12, sure_routes: bool = Fa
         shape = tuple(low_rank if n is None else n for n in shape)
         leaf = name.rsplit(".", 1)[-1]
         r = torch.randn(shape, generator=g)
-        if cfg["architecture"] == "Dogozen":
-            t = _dogozen_weight(name, r)
+        if cfg["architecture"] in ("Dogozen", "Zigivik"):
+            t = {"Dogozen": _dogozen_weight, "Zigivik": _zigivik_weight}[cfg["architecture"]](name, r)
         elif len(shape) == 1:
             if leaf == "A_log":
                 t = torch.linspace(-3.0, 2.7, shape[0]) if shape[0] > 1 else torch.zeros(1)

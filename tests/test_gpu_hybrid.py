@@ -62,7 +62,7 @@ class Truth:
     """The oracle's logits and streams for one sequence."""
 
     def __init__(self, cfg, w, toks):
-        self.layers, self.routed = [], cfg["architecture"] != "Teganex"
+        self.layers, self.routed = [], cfg["architecture"] in ("Lebedra", "Dogozen")
         self.logits = oracle.forward(cfg, w, toks, trace=self.layers)
 
     def agrees(self, got, dtype, rows=slice(None), layer=None):
@@ -426,7 +426,8 @@ def test_portions_and_single_tokens_give_the_whole_prompt(name, tensor_kernels):
 def test_mixed_batches_reuse_pages_and_slots(dtype):
     """Requests of unequal length come and go in a pool that holds two or three of them at a time; portions
     run beside decoded tokens and a request is left out of some steps."""
-    for name in ("deep", "ragged", "latent_ragged", "latent_wide", "latent_plain", "scan_ragged", "scan_wide", "scan_plain"):
+    for name in ("deep", "ragged", "latent_ragged", "latent_wide", "latent_plain", "scan_ragged", "scan_wide", "scan_plain", "side_ragged",
+                 "side_wide", "side_plain"):
         cfg = hu.CONFIGS[name]
         w = model_weights(cfg, 9, dtype)
         eng = engine(cfg, dtype, w=w, kv_pages=22)
@@ -465,7 +466,7 @@ def test_mixed_batches_reuse_pages_and_slots(dtype):
             assert Truth(cfg, w, t).agrees(torch.cat(o), dtype), (name, len(t))
 
 
-@pytest.mark.parametrize("name", ["wide", "latent_wide", "scan_wide"])
+@pytest.mark.parametrize("name", ["wide", "latent_wide", "scan_wide", "side_wide"])
 def test_long_decoding_does_not_drift(name):
     cfg = hu.CONFIGS[name]
     toks = hu.tokens(cfg, 420, 5)
@@ -482,7 +483,7 @@ def test_long_decoding_does_not_drift(name):
         assert truth.agrees(lg, dtype, slice(-1, None))
 
 
-@pytest.mark.parametrize("name", ["deep", "latent_ragged", "scan_ragged"])
+@pytest.mark.parametrize("name", ["deep", "latent_ragged", "scan_ragged", "side_ragged"])
 def test_offloaded_sequence_continues_in_another_slot(name):
     cfg = hu.CONFIGS[name]
     w, toks = hu.weights(cfg, 8), hu.tokens(cfg, 60)
@@ -507,7 +508,7 @@ def _greedy(cfg, w, prompt, n):
     return seq[len(prompt):], gaps
 
 
-@pytest.mark.parametrize("name,wide", [("ragged", "wide"), ("latent_ragged", "latent_wide"), ("scan_ragged", "scan_wide")])
+@pytest.mark.parametrize("name,wide", [("ragged", "wide"), ("latent_ragged", "latent_wide"), ("scan_ragged", "scan_wide"), ("side_ragged", "side_wide")])
 def test_greedy_generation_and_scheduler(name, wide):
     from mythos_b200.infer.sampler import SamplerConfig
     from mythos_b200.infer.serving import ContinuousBatcher
@@ -538,7 +539,7 @@ def test_greedy_generation_and_scheduler(name, wide):
     assert e16.generate(ps, max_new_tokens=20).tokens == e16.generate(ps, max_new_tokens=20, use_graph=False).tokens
 
 
-@pytest.mark.parametrize("name", ["ragged", "latent_ragged", "scan_ragged"])
+@pytest.mark.parametrize("name", ["ragged", "latent_ragged", "scan_ragged", "side_ragged"])
 def test_model_helpers_and_command_line(tmp_path, name):
     from mythos_b200.infer.engine import InferenceEngine
     from mythos_b200.infer.serving import compute_logprobs

@@ -25,12 +25,14 @@ def d(t):
 # ------------------------------------------------------------------------------- latent attention
 class Case:
     """New tokens of several sequences whose earlier tokens already lie in shuffled pages. ``proj`` holds unrotated
-    queries | rotated queries | latent | key part as the layer's projection leaves them."""
+    queries | rotated queries | latent | key part as the layer's projection leaves them. ``sink``: a number for every head,
+    "none", or None for random ones."""
 
-    def __init__(self, dtype, heads, dim, rot, vdim, rank, lens, bases, seed=0, base=10000.0, scale=None, sink=None):
+    def __init__(self, dtype, heads, dim, rot, vdim, rank, lens, bases, seed=0, base=10000.0, scale=None, sink=None, window=0,
+                 gate=False, amp=1.0):
         g = torch.Generator().manual_seed(seed)
         self.dtype, self.heads, self.dim, self.rot, self.vdim, self.rank = dtype, heads, dim, rot, vdim, rank
-        self.lens, self.bases, self.base = lens, bases, base
+        self.lens, self.bases, self.base, self.window, self.amp = lens, bases, base, window, amp
         self.scale = (dim + rot) ** -0.5 if scale is None else scale
         self.rank_p, self.rot_p, self.dim_p, self.vdim_p = pad8(rank), pad8(rot), pad8(dim), pad8(vdim)
         self.total = [b + n for b, n in zip(bases, lens)]
@@ -55,15 +57,22 @@ class Case:
         c = lambda t: t.to("cuda", dtype)
         self.table, self.cache, self.proj = table.cuda(), c(cache), c(proj)
         self.gamma = (1 + 0.3 * torch.randn(rank, generator=g)).cuda()
-        self.sink = (torch.randn(heads, generator=g) * 1.5 if sink is None else torch.full((heads,), float(sink))).cuda()
+        self.sink = None
+        if sink != "none":
+            self.sink = (torch.randn(heads, generator=g) * 1.5 if sink is None else torch.full((heads,), float(sink))).cuda()
         self.uk = c(torch.randn(heads, dim, rank, generator=g) * rank ** -0.5)
         self.uv = c(torch.randn(heads, vdim, rank, generator=g) * rank ** -0.5)
         turns = torch.tensor([base ** (-2.0 * i / rot) / (2 * math.pi) for i in range(rot // 2)], dtype=torch.float64)
         self.lat = H().Latent({"heads": heads, "rank": rank, "rot": rot, "rank_p": self.rank_p, "rot_p": self.rot_p,
                                "qr_off": self.off["qr"], "c_off": self.off["c"], "kr_off": self.off["kr"], "scale": self.scale,
-                               "eps": 1e-5}, self.gamma, turns.cuda(), self.sink)
+                               "eps": 1e-5, "window": window, "rot_amp": amp}, self.gamma, turns.cuda(), self.sink)
         self.batch = ragged(lens, bases)
         self.raw = self.proj.clone()
+        self.gate = None
+        if gate:
+            self.gate = torch.zeros(T, 8 + heads * self.vdim_p)
+            self.gate[:, 8:].view(T, heads, self.vdim_p)[..., :vdim] = torch.randn(T, heads, vdim, generator=g)
+            self.gate = c(self.gate)[:, 8:]
 
     def prep(self):
         self.lat.prep(self.proj, self.batch, self.table, self.cache)
@@ -82,16 +91,19 @@ class Case:
         out = torch.full((T, Hn, self.vdim_p), float("nan"), device="cuda", dtype=self.dtype)
         q, _ = self.queries()
         if how == "prefill":
-            keys = sum(self.total)
-            cu = torch.tensor([sum(self.total[:i]) for i in range(len(self.total) + 1)], dtype=torch.int32, device="cuda")
+            first = [max(0, b - self.window + 1) if self.window else 0 for b in self.bases]
+            held = [t - f for t, f in zip(self.total, first)]
+            keys, i32 = sum(held), dict(dtype=torch.int32, device="cuda")
+            cu = torch.tensor([sum(held[:i]) for i in range(len(held) + 1)], **i32)
             lat = torch.full((keys, self.W), float("nan"), device="cuda", dtype=self.dtype)
-            self.lat.gather(self.table, self.cache, cu, torch.zeros_like(cu[1:]), max(self.total), lat)
+            self.lat.gather(self.table, self.cache, cu, torch.tensor(first, **i32), max(held), lat)
             kv = torch.zeros(keys, Hn * (self.dim_p + self.vdim_p), device="cuda", dtype=self.dtype)
             k, v = kv[:, : Hn * self.dim_p].unflatten(1, (Hn, self.dim_p)), kv[:, Hn * self.dim_p:].unflatten(1, (Hn, self.vdim_p))
             c = lat[:, : self.rank].float()
             k[..., : self.dim] = torch.einsum("tr,hdr->thd", c, self.uk.float()).to(self.dtype)
             v[..., : self.vdim] = torch.einsum("tr,hdr->thd", c, self.uv.float()).to(self.dtype)
-            self.lat.attn_prefill(q, self.proj, k, v, lat, self.batch, cu, self.batch[1], max(self.lens), 1, None, out, status())
+            self.lat.attn_prefill(q, self.proj, k, v, lat, self.batch, cu, torch.tensor(held, **i32), max(self.lens), 1, self.gate,
+                                  out, status())
             return out[..., : self.vdim]
         uk = torch.zeros(Hn, self.rank_p, self.dim_p, device="cuda", dtype=self.dtype)
         uk[:, : self.rank, : self.dim] = self.uk.transpose(1, 2)
@@ -106,7 +118,7 @@ class Case:
             assert self.lat.decode_ok(PAGE)
             scratch = torch.full((T * Hn * splits * (self.rank_p + 4),), float("nan"), device="cuda")
             self.lat.attn_decode(ql, self.proj, self.batch[3], self.batch[4], self.table, self.cache, ol, scratch, splits, status())
-        H().gemm_heads(ol, uv, out, status())
+        H().gemm_heads(ol, uv, out, status(), self.gate)
         return out[..., : self.vdim]
 
     def want(self):
@@ -122,9 +134,14 @@ class Case:
             v = torch.einsum("tr,hdr->thd", c, uv)
             full = torch.zeros(self.total[s], self.heads, q.shape[-1], dtype=torch.float64)
             full[self.bases[s]:] = q[at:at + n]
-            out.append(oracle.sink_attention(full, k, v, self.scale, d(self.sink))[self.bases[s]:])
+            o = (oracle.sink_attention(full, k, v, self.scale, d(self.sink)) if self.sink is not None
+                 else oracle.banded_attention(full, k, v, self.scale, self.window or None))
+            out.append(o[self.bases[s]:])
             at += n
-        return torch.cat(out)
+        o = torch.cat(out)
+        if self.gate is not None:
+            o = o * torch.sigmoid(d(self.gate).view(-1, self.heads, self.vdim_p)[..., : self.vdim])
+        return o
 
 
 SHAPES = [(3, 20, 6, 36, 44), (1, 64, 64, 64, 64), (20, 128, 64, 128, 512), (17, 72, 2, 40, 256), (2, 8, 8, 8, 8), (16, 128, 32, 96, 200)]

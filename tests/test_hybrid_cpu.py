@@ -11,7 +11,8 @@ import hybrid_util as hu
 from mythos_b200.infer.kv_paged import PagedKVCache, RecurrentStatePool
 from mythos_b200.models import registry
 from mythos_b200.models.hybrid import HybridModel, expected_shapes
-from mythos_b200.models.hybrid_config import FrequencyScaling, HybridConfig, Rotation, dogozen_config, lebedra_config, teganex_config
+from mythos_b200.models.hybrid_config import (FrequencyScaling, HybridConfig, RampScaling, Rotation, dogozen_config, lebedra_config,
+                                               teganex_config, zigivik_config)
 from mythos_b200.oil.importers import read_safetensors_torch, write_safetensors
 from mythos_b200.oil.model_io import load_model
 
@@ -75,6 +76,38 @@ def test_bad_scan_configurations_are_refused(change):
         HybridConfig.from_dict(raw)
 
 
+@pytest.mark.parametrize("change", [
+    lambda c: c["layers"][2]["mixer"].update(kv_from=1),            # not latents
+    lambda c: c["layers"][2]["mixer"].update(kv_from=2),
+    lambda c: c["layers"][2]["mixer"].update(kv_rank=40),
+    lambda c: c["layers"][2]["mixer"]["rot"].update(base=301.0),    # rotated otherwise than the latents it uses
+    lambda c: c["layers"][0]["mixer"]["rot"].update(dims=4),
+    lambda c: c["layers"][0]["mixer"].update(q_rank=0),
+    lambda c: c["layers"][1]["mixer"].update(vdim=24),              # the keys are the values
+    lambda c: c["layers"][1]["mixer"].update(kv_heads=4),
+    lambda c: c["layers"][1]["mlp"].update(kind="moe"),
+    lambda c: c["layers"][3].update(type="parallel"),
+    lambda c: c["canon"].update(taps=-1),
+])
+def test_bad_parallel_configurations_are_refused(change):
+    raw = json.loads(json.dumps(hu.CONFIGS["side_ragged"]))
+    change(raw)
+    with pytest.raises((ValueError, KeyError)):
+        HybridConfig.from_dict(raw)
+
+
+def test_shapes_of_parallel_sublayers():
+    raw = json.loads(json.dumps(hu.CONFIGS["side_ragged"]))
+    del raw["layers"][2]["mixer"]["mask"]
+    c = HybridConfig.from_dict(raw)
+    shapes = expected_shapes(c)
+    assert c.layers[2].mixer.window == 0 and c.layers[2].mixer.rotation == c.layers[0].mixer.rotation
+    assert shapes["embed.norm"] == shapes["l2.norm1"] == shapes["final.norm"] == () and shapes["l3.canon1"] == (100, 3)
+    for absent in ("l0.norm2", "l0.norm1b", "l1.mix.v", "l1.mix.sink", "l2.mix.dkv", "l2.mix.dkv.norm", "l2.mlp.up", "l0.mix.q", "l1.mlp.gate"):
+        assert absent not in shapes
+    assert shapes["l2.mix.uq"] == (5 * 18, 21) and shapes["l1.mlp.act"] == (4,) and shapes["l1.mix.k.b"] == (40,)
+
+
 def test_optional_parts_of_a_configuration():
     raw = json.loads(json.dumps(hu.CONFIGS["scan_ragged"]))
     del raw["layers"][0]["mixer"]["q_temp"], raw["layers"][1]["mixer"]["left"]["mask"], raw["layers"][1]["mlp"]["router"]["groups"]
@@ -94,6 +127,16 @@ def test_rotation_frequencies(rot):
     r = Rotation(rot["base"], rot["dims"], FrequencyScaling(**sc) if sc else None)
     want = torch.tensor(oracle.frequencies(rot), dtype=torch.float64) / (2 * torch.pi)
     assert torch.allclose(torch.tensor(r.turns(), dtype=torch.float64), want, rtol=1e-12, atol=0)
+
+
+@pytest.mark.parametrize("rot", [hu.ramp(1e4, 64, 8.0, 256, 32.0), hu.ramp(500.0, 10, 2.5, 4096, 32.0), hu.ramp(300.0, 6, 4.0, 64, 3.0, 3.0),
+                                 hu.ramp(100.0, 2, 16.0, 16, 4.0, 0.5), hu.ramp(1e5, 48), hu.ramp(10.0, 16, 1.0, 32, 4.0)])
+def test_ramped_rotation_frequencies(rot):
+    sc = rot.get("scaling")
+    r = Rotation(rot["base"], rot["dims"], RampScaling(**sc) if sc else None)
+    freq, amp = oracle.yarn_frequencies(rot)
+    want = torch.tensor(freq, dtype=torch.float64) / (2 * torch.pi)
+    assert torch.allclose(torch.tensor(r.turns(), dtype=torch.float64), want, rtol=1e-12, atol=0) and r.amplitude == pytest.approx(amp, rel=1e-12)
 
 
 def _write(folder, cfg, w):
@@ -151,6 +194,21 @@ def test_dogozen_folder_loads_through_the_registry(tmp_path):
         HybridModel(HybridConfig.from_dict(cfg), w)
 
 
+def test_zigivik_folder_loads_through_the_registry(tmp_path):
+    cfg = hu.CONFIGS["side_ragged"]
+    w = hu.weights(cfg, 3)
+    _write(str(tmp_path), cfg, w)
+    m, _ = load_model(str(tmp_path))
+    assert isinstance(m, HybridModel) and m.cfg.architecture == "Zigivik" and m.cfg.parallel and m.cfg.input_conv == 3
+    assert m.tensor("embed.norm").shape == () and torch.equal(m.tensor("l2.mix.uk"), w["l2.mix.uk"])
+    from mythos_b200.tools.info import main as info_main
+
+    assert info_main([str(tmp_path)]) == 0
+    del w["l1.mlp.act"]
+    with pytest.raises(KeyError):
+        HybridModel(HybridConfig.from_dict(cfg), w)
+
+
 def test_missing_and_misshapen_tensors_are_refused():
     cfg = hu.CONFIGS["single"]
     hc = HybridConfig.from_dict(cfg)
@@ -170,6 +228,8 @@ def test_named_configuration_has_consistent_shapes():
     assert [s.type for s in cfg.layers] == ["gla", "gla", "gla", "parallel"]
     m = HybridModel.random(dogozen_config(width=256, layers=6, vocab=64, experts=16, top=2))
     assert m.param_count() == sum(t.numel() for _, t in m.named_tensors()) and m.cfg.layers[4].mixer.kv_from == 2
+    m = HybridModel.random(zigivik_config(width=512, layers=5, vocab=64))
+    assert m.param_count() == sum(t.numel() for _, t in m.named_tensors()) and m.cfg.layers[1].mixer.kv_from == 0
     m = HybridModel.random(lebedra_config(width=256, layers=2, vocab=64, experts=8, top=2))
     assert m.param_count() == sum(t.numel() for _, t in m.named_tensors()) and m.tensor("l1.mlp.e7.gate").shape[1] == 256
 
@@ -229,6 +289,20 @@ def test_batch_plan_separates_long_and_short_portions():
     assert sp.keys == 2 * n + 103 and sp.max_k == n + 103 and sp.short.dtype == torch.int64
     lists, build = HybridEngine._batch_plan(Cfg, [n], [3])
     assert lists == [[0, n + 3], [0], [n + 3], [], [], []] and build(*[torch.tensor(x) for x in lists]).short is None
+
+
+def test_batch_plan_leaves_out_what_no_window_reaches():
+    from mythos_b200.infer.hybrid import EXPAND_TOKENS, HybridEngine
+
+    class Cfg:
+        cfg = HybridConfig.from_dict(hu.CONFIGS["side_ragged"])          # windows of 19 and 33
+
+    n = EXPAND_TOKENS
+    lists, build = HybridEngine._batch_plan(Cfg, [n, 2, n + 5], [100, 90, 32])
+    assert lists == [[0, n + 32, n + 32, 2 * n + 69], [68, 0, 0], [n + 32, 92, n + 37], [n, n + 1], [1, 1], [90, 91]]
+    assert build(*[torch.tensor(x, dtype=torch.int32) for x in lists]).max_k == n + 37
+    Cfg.cfg.layers[0].mixer.window = 0                                   # a layer that sees everything
+    assert HybridEngine._batch_plan(Cfg, [n], [100])[0][:3] == [[0, n + 100], [0], [n + 100]]
 
 
 class _FakeEngine:
@@ -457,6 +531,73 @@ def test_a_mistake_in_a_scan_or_window_mechanism_shows(slip, monkeypatch):
     w, toks = hu.weights(cfg, 5), hu.tokens(cfg, 48)
     right = oracle.forward(cfg, w, toks)
     fn, wrong = _scan_slips()[slip]
+    monkeypatch.setattr(oracle, fn, wrong)
+    e = hu.row_errors(oracle.forward(cfg, w, toks), right)
+    assert float(e.max()) > 0.06 and float((e > 1e-3).double().mean()) > 0.25, (float(e.max()), float(e.median()))
+
+
+def _side_slips():
+    """Mistakes in Zigivik's mechanisms: name -> (function of the oracle, wrong version)."""
+    att, halves, pairs, freq, conv, poly, low, norm, lat, kv, ff = (
+        oracle.banded_attention, oracle.turn_halves, oracle.turn_pairs, oracle.yarn_frequencies, oracle.input_conv, oracle.poly_norm,
+        oracle.low_rank_queries, oracle.one_number_norm, oracle.window_latent_attention, oracle.key_value_attention, oracle.poly_ff)
+
+    def as_pairs(x, pos, r):
+        n = r["dims"]
+        order = torch.tensor([i // 2 + (i % 2) * (n // 2) for i in range(n)])
+        out = x.clone()
+        out[..., order] = halves(x[..., order], pos, r)
+        return halves(x[..., torch.tensor([2 * i for i in range(n // 2)] + [2 * i + 1 for i in range(n // 2)])], pos, r)
+
+    def as_halves(x, pos, r):
+        n = r["dims"]
+        order = torch.tensor([i // 2 + (i % 2) * (n // 2) for i in range(n)])
+        out = x.clone()
+        out[..., order] = pairs(x[..., order], pos, r)
+        return out
+
+    def own_values(h, W, p, c):                            # values behind the rotation
+        T, G = h.shape[0], c["kv_heads"]
+        pos = torch.arange(T)
+        q = pairs((h @ W[p + "q"].T + W[p + "q.b"]).view(T, c["heads"], c["dim"]), pos, c["rot"])
+        k = pairs((h @ W[p + "k"].T + W[p + "k.b"]).view(T, G, c["dim"]), pos, c["rot"])
+        return att(q, k, k, c["scale"], plus_one=True).reshape(T, -1) @ W[p + "o"].T
+
+    def one_rms(z, act, eps):                              # every power divided by the rms of z itself
+        n = oracle.rms(z, eps)
+        return act[0] * n + act[1] * n ** 2 + act[2] * n ** 3 + act[3]
+
+    def shifted(h, w):
+        return h + conv(torch.cat([torch.zeros_like(h[:1]), h[:-1]]), w) - torch.cat([torch.zeros_like(h[:1]), h[:-1]])
+
+    return {"window_longer": ("banded_attention", lambda q, k, v, s, w=None, plus_one=False: att(q, k, v, s, w and w + 1, plus_one)),
+            "window_shorter": ("banded_attention", lambda q, k, v, s, w=None, plus_one=False: att(q, k, v, s, w and w - 1, plus_one)),
+            "no_one": ("banded_attention", lambda q, k, v, s, w=None, plus_one=False: att(q, k, v, s, w)),
+            "one_everywhere": ("banded_attention", lambda q, k, v, s, w=None, plus_one=False: att(q, k, v, s, w, True)),
+            "as_pairs": ("turn_halves", as_pairs), "as_halves": ("turn_pairs", as_halves),
+            "no_ramp": ("yarn_frequencies", lambda r: ([float(r["base"]) ** (-2.0 * i / r["dims"]) for i in range(r["dims"] // 2)], freq(r)[1])),
+            "no_amplitude": ("yarn_frequencies", lambda r: (freq(r)[0], 1.0)),
+            "amplitude_in_scale": ("yarn_frequencies", lambda r: (freq(r)[0], freq(r)[1] ** 2)),
+            "late_positions": ("turn_pairs", lambda x, pos, r: pairs(x, pos if x.shape[1] == 2 else pos + 1, r)),
+            "values_behind_rotation": ("key_value_attention", own_values),
+            "no_conv": ("input_conv", lambda h, w: h), "conv_alone": ("input_conv", lambda h, w: conv(h, w) - h),
+            "reversed_taps": ("input_conv", lambda h, w: conv(h, w.flip(1))), "shifted_conv": ("input_conv", shifted),
+            "one_rms": ("poly_norm", one_rms), "no_constant": ("poly_norm", lambda z, a, e: poly(z, a, e) - a[3]),
+            "swapped_powers": ("poly_norm", lambda z, a, e: poly(z, a[torch.tensor([2, 1, 0, 3])], e)),
+            "no_query_norm": ("low_rank_queries", lambda h, W, p, e: (h @ W[p + "dq"].T) @ W[p + "uq"].T),
+            "no_down_bias": ("poly_ff", lambda h, W, p, e: ff(h, W, p, e) - W[p + "down.b"]),
+            "norm_around_zero": ("one_number_norm", lambda x, g, e: norm(x, 1 + g, e)),
+            "own_latents": ("window_latent_attention", lambda h, W, p, c, e, kept: lat(h, W, p, c, e, {k: (a.flip(0), b) for k, (a, b) in kept.items()}
+                                                                                       if c.get("kv_from") is not None else kept))}
+
+
+@pytest.mark.parametrize("slip", sorted(_side_slips()))
+def test_a_mistake_in_a_parallel_layer_shows(slip, monkeypatch):
+    """Far above what 32-bit comparisons allow (5e-5) on many rows, and on some above the bf16 tolerance as well."""
+    cfg = hu.CONFIGS["side_ragged"]
+    w, toks = hu.weights(cfg, 5), hu.tokens(cfg, 60)
+    right = oracle.forward(cfg, w, toks)
+    fn, wrong = _side_slips()[slip]
     monkeypatch.setattr(oracle, fn, wrong)
     e = hu.row_errors(oracle.forward(cfg, w, toks), right)
     assert float(e.max()) > 0.06 and float((e > 1e-3).double().mean()) > 0.25, (float(e.max()), float(e.median()))
