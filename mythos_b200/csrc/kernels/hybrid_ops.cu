@@ -86,17 +86,17 @@ __device__ __forceinline__ void prefetch_tail(const ConvTail& cv, int dim, long 
 
 // h = rms(row) * gamma (or the row itself) for a row held in shared memory; columns [dim, ldh) are zeroed (GEMM padding).
 // With a convolution tail, row t being the new token of sequence t, also h + conv(h) of what the activation type keeps of h.
-template <typename T, int V>
+template <typename T, int V, bool CONV>
 __device__ __forceinline__ void write_normed(const float* row, float ss, const float* gamma, T* h, long long ldh,
                                              int dim, float eps, const ConvTail& cv, long long t) {
   const float r = 1.f / sqrtf(ss / (float)dim + eps);
-  const int taps = cv.c.taps;
+  const int taps = CONV ? cv.c.taps : 0;
   T* out = taps > 0 ? static_cast<T*>(cv.out) + t * cv.ld : nullptr;
   float* state = taps > 1 ? cv.c.state + (long long)cv.slots[t] * (taps - 1) * dim : nullptr;
   const bool fresh = taps > 0 && cv.kv_lens[t] <= 1;
   for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
     float x[V], g[V];
-    if (V == 4 && taps == 4) {                         // all loads first
+    if (CONV && V == 4 && taps == 4) {                 // all loads first
       float w[4][V], old[3][V];
 #pragma unroll
       for (int j = 0; j < 4; ++j) ldv<V>(cv.c.w + (long long)j * dim + i, w[j]);
@@ -128,7 +128,7 @@ __device__ __forceinline__ void write_normed(const float* row, float ss, const f
       for (int j = 0; j < V; ++j) x[j] *= r * g[j];
     }
     stv<V>(h + i, x);
-    if (taps > 0) {
+    if (CONV) {
 #pragma unroll
       for (int j = 0; j < V; ++j) {
         const float cur = kept<T>(x[j]);
@@ -141,7 +141,7 @@ __device__ __forceinline__ void write_normed(const float* row, float ss, const f
     for (int i = dim + threadIdx.x; i < cv.ld; i += SN_THREADS) stf(out + i, 0.f);
 }
 
-template <typename T, int V>
+template <typename T, int V, bool CONV>
 __global__ void __launch_bounds__(SN_THREADS)
 embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ pos, const T* __restrict__ embed,
                       const T* __restrict__ pos_table, int vocab, int max_pos, float scale,
@@ -150,7 +150,7 @@ embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ pos, 
   extern __shared__ __align__(16) float row[];
   __shared__ float scratch[32];
   const long long t = blockIdx.x;
-  prefetch_tail(cv, dim, t);
+  if constexpr (CONV) prefetch_tail(cv, dim, t);
   int id = ids[t];
   id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
   int p = pos[t];
@@ -188,10 +188,10 @@ embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ pos, 
     }
     ss = block_sum(ss, scratch);
   }
-  write_normed<T, V>(row, ss, gamma, h + t * ldh, ldh, dim, eps, cv, t);
+  write_normed<T, V, CONV>(row, ss, gamma, h + t * ldh, ldh, dim, eps, cv, t);
 }
 
-template <typename T, int V>
+template <typename T, int V, bool CONV>
 __global__ void __launch_bounds__(SN_THREADS)
 residual_norm_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ bias, float mult, float* __restrict__ x,
                      const float* __restrict__ w_next, T* __restrict__ h, long long ldh, int dim, float eps,
@@ -199,7 +199,7 @@ residual_norm_kernel(const T* __restrict__ y, long long ldy, const float* __rest
   extern __shared__ __align__(16) float row[];
   __shared__ float scratch[32];
   const long long t = blockIdx.x;
-  prefetch_tail(cv, dim, t);
+  if constexpr (CONV) prefetch_tail(cv, dim, t);
   float sx = 0.f;
   for (int i = threadIdx.x * V; i < dim; i += SN_THREADS * V) {
     float a[V], b[V], xv[V];
@@ -219,7 +219,7 @@ residual_norm_kernel(const T* __restrict__ y, long long ldy, const float* __rest
     stv<V>(row + i, xv);
   }
   sx = block_sum(sx, scratch);
-  write_normed<T, V>(row, sx, w_next, h + t * ldh, ldh, dim, eps, cv, t);
+  write_normed<T, V, CONV>(row, sx, w_next, h + t * ldh, ldh, dim, eps, cv, t);
 }
 
 template <int V>
@@ -424,7 +424,7 @@ sandwich_norm_kernel(SublayerOut src, const float* __restrict__ w_post, float mu
     stv<V>(row + i, xv);
   }
   if (w_next) sx = block_sum(sx, scratch);
-  write_normed<T, V>(row, sx, w_next, h + t * ldh, ldh, dim, eps, ConvTail{}, t);
+  write_normed<T, V, false>(row, sx, w_next, h + t * ldh, ldh, dim, eps, ConvTail{}, t);
 }
 
 // Cosine and sine of a position's turn: position x revolutions, reduced to a fraction of a turn in double precision.
@@ -799,8 +799,12 @@ template <typename T, int V>
 void embed_launch(const int* ids, const int* pos, const void* embed, const void* pos_table, int vocab, int max_pos,
                   float scale, const float* gamma0, const float* gamma, float* x, void* h, long long ldh, int rows, int dim,
                   float eps, const ConvTail& conv, cudaStream_t stream) {
-  embed_pos_norm_kernel<T, V><<<rows, SN_THREADS, dim * 4, stream>>>(ids, pos, (const T*)embed, (const T*)pos_table, vocab, max_pos,
-                                                                     scale, gamma0, gamma, x, (T*)h, ldh, dim, eps, conv);
+  auto go = [&](auto kern) {
+    kern<<<rows, SN_THREADS, dim * 4, stream>>>(ids, pos, (const T*)embed, (const T*)pos_table, vocab, max_pos, scale, gamma0, gamma, x,
+                                                (T*)h, ldh, dim, eps, conv);
+  };
+  if (conv.c.taps > 0) go(embed_pos_norm_kernel<T, V, true>);
+  else go(embed_pos_norm_kernel<T, V, false>);
 }
 void check_tail(const ConvTail& conv, int dim) {
   MB_REQUIRE(conv.c.taps >= 0 && conv.c.taps <= 64, "convolution tail: taps");
@@ -859,11 +863,14 @@ void residual_norm(bool f32, const void* y, long long ldy, const float* bias, fl
   check_tail(conv, dim);
   if (rows == 0) return;
   const bool v4 = dim % 4 == 0 && ldh % 4 == 0 && ldy % 4 == 0;
-#define MB_RN(T, V) \
-  residual_norm_kernel<T, V><<<rows, SN_THREADS, dim * 4, stream>>>((const T*)y, ldy, bias, mult, x, w_next, (T*)h, ldh, dim, eps, conv)
+#define MB_RNC(T, V, CONV)                                                                                                  \
+  residual_norm_kernel<T, V, CONV><<<rows, SN_THREADS, dim * 4, stream>>>((const T*)y, ldy, bias, mult, x, w_next, (T*)h, ldh, \
+                                                                          dim, eps, conv)
+#define MB_RN(T, V) do { if (conv.c.taps > 0) MB_RNC(T, V, true); else MB_RNC(T, V, false); } while (0)
   if (f32) { if (v4) MB_RN(float, 4); else MB_RN(float, 1); }
   else     { if (v4) MB_RN(__nv_bfloat16, 4); else MB_RN(__nv_bfloat16, 1); }
 #undef MB_RN
+#undef MB_RNC
   count_launch();
   check_launch();
 }
